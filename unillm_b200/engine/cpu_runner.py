@@ -6,14 +6,12 @@ Works on any torch device; every op is a plain torch op.
 """
 from __future__ import annotations
 
-import math
 from typing import List, Optional
 
 import torch
-import torch.nn.functional as F
 
 from ..models.decoder import DecoderModel
-from ..precompute import RoPECache, alibi_slopes, apply_rope
+from ..precompute import alibi_slopes, apply_rope
 from ..sampling import Sampler, SamplingParams
 from ..tensor_core import ops_fn
 from .runner import StepBatch
@@ -25,70 +23,57 @@ class CpuModelRunner:
         s = self.spec
         self.block_size, self.num_blocks, self.max_model_len = block_size, num_blocks, max_model_len
         dev, dt = model.device, model.dtype
-        self.k_cache = [torch.zeros(num_blocks, s.num_kv_heads, block_size, s.head_dim, dtype=dt, device=dev)
-                        for _ in range(s.num_layers)]
-        self.v_cache = [torch.zeros_like(k) for k in self.k_cache]
-        self._rope: Optional[RoPECache] = None
+        self.k_cache, self.v_cache = [], []
+        for i in range(s.num_layers):
+            ls = s.layer(i)
+            if ls.kv_from is not None:                  # reads that layer's pages
+                self.k_cache.append(self.k_cache[ls.kv_from])
+                self.v_cache.append(self.v_cache[ls.kv_from])
+                continue
+            for cache, d in ((self.k_cache, ls.head_dim), (self.v_cache, ls.v_head_dim)):
+                cache.append(torch.zeros(num_blocks, ls.num_kv_heads, block_size, d, dtype=dt, device=dev))
         self._alibi = alibi_slopes(s.num_heads).to(dev) if s.pos == "alibi" else None
         self.launches = 0
         self.h2d_bytes = self.d2h_bytes = 0
         self._sampler = Sampler()
 
-    def _rope_at(self, positions: torch.Tensor):
-        s = self.spec
-        need = int(positions.max()) + 1
-        if self._rope is None or self._rope.max_seq_len < need:
-            self._rope = RoPECache(s.head_dim, max(need, 4096), s.rope_theta, rotary_dim=s.rd,
-                                   position_scale=s.rope_pos_scale, llama3=s.rope_llama3, device=self.model.device)
-        return self._rope.at(positions)
-
     def _attention(self, i: int, h: torch.Tensor, b: StepBatch, pos: torch.Tensor, slots: torch.Tensor) -> torch.Tensor:
-        s, m = self.spec, self.model
+        s, m, ls = self.spec, self.model, self.spec.layer(i)
         L = f"layers.{i}."
         T = h.shape[0]
-        qkv = ops_fn.linear(h, m.p[L + "wqkv"], m.p.get(L + "bqkv"))
-        q, k, v = qkv.split([s.q_size, s.kv_size, s.kv_size], dim=-1)
-        q = q.reshape(T, s.num_heads, s.head_dim)
-        k = k.reshape(T, s.num_kv_heads, s.head_dim)
-        v = v.reshape(T, s.num_kv_heads, s.head_dim)
-        if s.qk_norm:
-            q = ops_fn.rms_norm(q, m.p[L + "q_norm"], s.norm_eps)
-            k = ops_fn.rms_norm(k, m.p[L + "k_norm"], s.norm_eps)
-        if s.pos == "rope" and s.rd > 0:
-            cos, sin = self._rope_at(pos)
-            q = apply_rope(q, cos, sin, s.rd, s.rope_interleaved)
-            k = apply_rope(k, cos, sin, s.rd, s.rope_interleaved)
-        ok = slots >= 0
-        blk, off = slots[ok] // self.block_size, slots[ok] % self.block_size
-        self.k_cache[i][blk, :, off] = k[ok]
-        self.v_cache[i][blk, :, off] = v[ok]
-        out = torch.empty(T, s.num_heads, s.head_dim, dtype=h.dtype, device=h.device)
-        scale = s.attn_scale if s.attn_scale is not None else 1.0 / math.sqrt(s.head_dim)
-        g = s.num_heads // s.num_kv_heads
+        q, k, v = m._project_qkv(i, h)
+        if ls.rotary_dim > 0:
+            cos, sin = m._rope_cache(int(pos.max()) + 1, ls).at(pos)
+            q = apply_rope(q, cos, sin, ls.rotary_dim, s.rope_interleaved)
+            if k is not None:
+                k = apply_rope(k, cos, sin, ls.rotary_dim, s.rope_interleaved)
+        if k is not None:
+            ok = slots >= 0
+            blk, off = slots[ok] // self.block_size, slots[ok] % self.block_size
+            self.k_cache[i][blk, :, off] = k[ok]
+            self.v_cache[i][blk, :, off] = v[ok]
+        out = torch.empty(T, ls.num_heads, ls.v_head_dim, dtype=h.dtype, device=h.device)
         row = 0
         q_lens = [1] * b.num_decode + list(b.prefill_q_lens)
         for si, ql in enumerate(q_lens):
             kv_len = b.seq_lens[si]
             bt = torch.as_tensor(b.block_tables[si][: (kv_len + self.block_size - 1) // self.block_size],
                                  device=h.device, dtype=torch.long)
-            kk = self.k_cache[i][bt].permute(1, 0, 2, 3).reshape(s.num_kv_heads, -1, s.head_dim)[:, :kv_len]
-            vv = self.v_cache[i][bt].permute(1, 0, 2, 3).reshape(s.num_kv_heads, -1, s.head_dim)[:, :kv_len]
-            if g > 1:
-                kk, vv = kk.repeat_interleave(g, 0), vv.repeat_interleave(g, 0)
+            kk = self.k_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.head_dim)[:, :kv_len]
+            vv = self.v_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.v_head_dim)[:, :kv_len]
             qq = q[row:row + ql].transpose(0, 1).float()              # [H, ql, D]
             qpos = torch.arange(kv_len - ql, kv_len, device=h.device)[:, None]
             kpos = torch.arange(kv_len, device=h.device)[None, :]
             vis = kpos <= qpos
-            if s.window > 0:
-                vis = vis & (kpos > qpos - s.window)
+            if ls.window > 0:
+                vis = vis & (kpos > qpos - ls.window)
             bias = torch.zeros(ql, kv_len, device=h.device).masked_fill(~vis, float("-inf"))
             if self._alibi is not None:
                 bias = bias[None] + self._alibi[:, None, None] * (kpos - qpos)[None].float()
-            y = F.scaled_dot_product_attention(qq[None], kk.float()[None], vv.float()[None],
-                                               attn_mask=bias if bias.dim() == 2 else bias[None], scale=scale)[0]
+            y = m._attend(i, qq[None], kk.float()[None], vv.float()[None], bias if bias.dim() == 2 else bias[None])[0]
             out[row:row + ql] = y.transpose(0, 1).to(h.dtype)
             row += ql
-        return ops_fn.linear(out.reshape(T, s.q_size), m.p[L + "wo"], m.p.get(L + "bo"))
+        return ops_fn.linear(out.reshape(T, ls.o_size), m.p[L + "wo"], m.p.get(L + "bo"))
 
     @torch.no_grad()
     def forward_logits(self, b: StepBatch) -> torch.Tensor:
@@ -106,21 +91,8 @@ class CpuModelRunner:
             x = x + m.p["pos_embed"][pos + s.learned_pos_offset]
         if s.embed_norm:
             x = ops_fn.layer_norm(x, m.p["embed_norm.w"], m.p["embed_norm.b"], s.norm_eps)
-        rs = s.residual_scale
         for i in range(s.num_layers):
-            L = f"layers.{i}."
-            if s.post_ln:
-                x = m._norm(x + self._attention(i, x, b, pos, slots) * rs, L + "ln1")
-                x = m._norm(x + m._mlp(i, x[None])[0] * rs, L + "ln2")
-                continue
-            h = m._norm(x, L + "ln1")
-            a = self._attention(i, h, b, pos, slots)
-            if s.parallel_residual:
-                m_in = h if s.parallel_shared_norm else m._norm(x, L + "ln2")
-                x = x + (a + m._mlp(i, m_in[None])[0]) * rs
-            else:
-                x = x + a * rs
-                x = x + m._mlp(i, m._norm(x, L + "ln2")[None])[0] * rs
+            x = m.block(i, x[None], lambda h, i=i: self._attention(i, h[0], b, pos, slots)[None])[0]
         rows = torch.as_tensor(b.sample_rows, dtype=torch.long, device=dev)
         xs = x[rows]
         if s.final_norm:

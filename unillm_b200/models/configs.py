@@ -314,6 +314,29 @@ class FlorenceConfig:
 
 
 @model_config
+class GekapelConfig:
+    """Gekapel: every layer is described on its own.  ``layers[i]`` holds ``mixer`` (heads, kv_heads, dim, vdim, scale,
+    mask.size, rot.{base, dims, scaling}, optionally kv_from) and ``mlp`` (router.{experts, top}, expert.ff, shared.ff;
+    null for a layer without a feed-forward)."""
+
+    vocab_size: int = 32000
+    hidden_size: int = 2048
+    num_hidden_layers: int = 0
+    norm_eps: float = 1e-6
+    layers: List[Any] = []
+    max_position_embeddings: int = 131072
+    initializer_range: float = 0.02
+
+    @classmethod
+    def from_hf_config(cls, d):
+        if "layers" not in d or "width" not in d:
+            return super(GekapelConfig, cls).from_hf_config(d)
+        kw = {k: d[k] for k in ("max_position_embeddings", "initializer_range") if k in d}
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], num_hidden_layers=len(d["layers"]),
+                   norm_eps=d["norm"]["eps"], layers=list(d["layers"]), **kw)
+
+
+@model_config
 class GemmaConfig:
     vocab_size: int = 256000
     hidden_size: int = 3072

@@ -27,7 +27,7 @@ from ..model_core import Model, ModelInputs, ModelOutputs, ModelWeights, WeightM
 from ..precompute import RoPECache, alibi_slopes, apply_rope
 from ..tensor_core import ops_fn
 from ..types import InvalidInput, LoadingError
-from .spec import DecoderSpec, KeyScheme, MoESpec
+from .spec import DecoderSpec, KeyScheme, LayerSpec, MoESpec
 
 
 def _f(x):
@@ -44,7 +44,7 @@ class DecoderModel(Model):
         self.spec: DecoderSpec = self.spec_from_config(config)
         self.reference_quirks = reference_quirks
         self.p: Dict[str, torch.Tensor] = {}
-        self._rope: Optional[RoPECache] = None
+        self._rope: Optional[Dict[tuple, RoPECache]] = None
         self._alibi: Optional[torch.Tensor] = None
 
     @classmethod
@@ -56,7 +56,7 @@ class DecoderModel(Model):
     # ------------------------------------------------------------------------------------------
     def param_shapes(self) -> Dict[str, tuple]:
         s = self.spec
-        H, D = s.hidden_size, s.head_dim
+        H = s.hidden_size
         E = s.embed_proj_dim or H
         shp: Dict[str, tuple] = {"embed": (s.vocab_size, E)}
         if s.embed_proj_dim:
@@ -69,24 +69,28 @@ class DecoderModel(Model):
             shp["embed_norm.b"] = (H,)
         for i in range(s.num_layers):
             L = f"layers.{i}."
+            ls = s.layer(i)
             shp[L + "ln1.w"] = (H,)
             if s.norm_bias:
                 shp[L + "ln1.b"] = (H,)
-            if not (s.parallel_residual and s.parallel_shared_norm):
+            if not (s.parallel_residual and s.parallel_shared_norm) and ls.mlp is not None:
                 shp[L + "ln2.w"] = (H,)
                 if s.norm_bias:
                     shp[L + "ln2.b"] = (H,)
-            shp[L + "wqkv"] = (s.q_size + 2 * s.kv_size, H)
+            shp[L + "wqkv"] = (ls.qkv_size, H)
             if s.qkv_bias:
-                shp[L + "bqkv"] = (s.q_size + 2 * s.kv_size,)
+                shp[L + "bqkv"] = (ls.qkv_size,)
             if s.qk_norm:
-                shp[L + "q_norm"] = (D,)
-                shp[L + "k_norm"] = (D,)
-            shp[L + "wo"] = (H, s.q_size)
+                shp[L + "q_norm"] = (ls.head_dim,)
+                if ls.kv_from is None:
+                    shp[L + "k_norm"] = (ls.head_dim,)
+            if ls.sink:
+                shp[L + "sink"] = (ls.num_heads,)
+            shp[L + "wo"] = (H, ls.o_size)
             if s.o_bias:
                 shp[L + "bo"] = (H,)
-            moe = s.layer_is_moe(i)
-            if (not moe) or s.moe.dense_parallel:
+            moe = ls.mlp == "moe"
+            if ls.mlp == "dense" or (moe and ls.moe.dense_parallel):
                 I = s.intermediate_size
                 if s.mlp == "gated":
                     shp[L + "w_gate_up"] = (2 * I, H)
@@ -98,13 +102,15 @@ class DecoderModel(Model):
                 if s.mlp_bias:
                     shp[L + "b_down"] = (H,)
             if moe:
-                m = s.moe
+                m = ls.moe
                 shp[L + "router"] = (m.num_experts, H)
+                if m.router_bias:
+                    shp[L + "router_b"] = (m.num_experts,)
                 shp[L + "experts_gate_up"] = (m.num_experts, (2 if m.gated else 1) * m.intermediate_size, H)
                 shp[L + "experts_down"] = (m.num_experts, H, m.intermediate_size)
                 if m.num_shared_experts:
-                    Is = m.num_shared_experts * m.intermediate_size
-                    shp[L + "shared_gate_up"] = (2 * Is, H)
+                    Is = m.shared_width
+                    shp[L + "shared_gate_up"] = ((2 if m.gated else 1) * Is, H)
                     shp[L + "shared_down"] = (H, Is)
         if s.final_norm:
             shp["final_norm.w"] = (H,)
@@ -126,7 +132,7 @@ class DecoderModel(Model):
                 t = torch.zeros(shape, dtype=dtype)
             elif is_norm_w:
                 t = torch.zeros(shape, dtype=dtype) if self.spec.norm_weight_offset_one else torch.ones(shape, dtype=dtype)
-            elif name.endswith((".b", "bqkv", "bo", "b_up", "b_down", "lm_head_bias")):
+            elif name.endswith((".b", "bqkv", "bo", "b_up", "b_down", "lm_head_bias", "router_b", "sink")):
                 t = torch.zeros(shape, dtype=dtype)
             else:
                 t = (torch.randn(shape, generator=g, dtype=torch.float32) * std).to(dtype)
@@ -137,9 +143,9 @@ class DecoderModel(Model):
     # ------------------------------------------------------------------------------------------
     # loading from / exporting to the family's on-disk names
     # ------------------------------------------------------------------------------------------
-    @staticmethod
-    def _find(w: ModelWeights, prefixes, names, suffix=".weight"):
+    def _find(self, w: ModelWeights, prefixes, names, suffix=".weight"):
         """First present alias; block-quantised (GGUF) tensors are dequantised on the way in."""
+        suffix = {".weight": self.scheme.weight_suffix, ".bias": self.scheme.bias_suffix}.get(suffix, suffix)
         for pre in prefixes:
             for n in names:
                 t = w.get(pre + n + suffix)
@@ -186,6 +192,7 @@ class DecoderModel(Model):
             out["embed_norm.b"] = b if b is not None else torch.zeros(s.hidden_size)
         for i in range(s.num_layers):
             L = f"layers.{i}."
+            ls = s.layer(i)
             pre = tuple(p.format(i=i) for p in k.layer)
             out[L + "ln1.w"] = need(self._find(weights, pre, k.ln1), f"layer {i} ln1")
             if s.norm_bias:
@@ -210,8 +217,12 @@ class DecoderModel(Model):
                     names = [p + n + ".weight" for p in pre for n in k.q]
                     q, kk, v = deq(names), deq([n.replace(k.q[0], k.k[0]) for n in names]), \
                         deq([n.replace(k.q[0], k.v[0]) for n in names])
-                need(q, f"layer {i} q_proj"), need(kk, f"layer {i} k_proj"), need(v, f"layer {i} v_proj")
-                out[L + "wqkv"] = torch.cat([q, kk, v], dim=0)
+                need(q, f"layer {i} q_proj")
+                if ls.kv_from is None:
+                    need(kk, f"layer {i} k_proj"), need(v, f"layer {i} v_proj")
+                    out[L + "wqkv"] = torch.cat([q, kk, v], dim=0)
+                else:
+                    out[L + "wqkv"] = q
                 bq = None
                 qb = self._find(weights, pre, k.q, ".bias")
                 if qb is not None:
@@ -223,7 +234,10 @@ class DecoderModel(Model):
                 out[L + "bqkv"] = bq if bq is not None else torch.zeros(s.q_size + 2 * s.kv_size)
             if s.qk_norm:
                 out[L + "q_norm"] = need(self._find(weights, pre, k.q_norm), "q_norm")
-                out[L + "k_norm"] = need(self._find(weights, pre, k.k_norm), "k_norm")
+                if ls.kv_from is None:
+                    out[L + "k_norm"] = need(self._find(weights, pre, k.k_norm), "k_norm")
+            if ls.sink:
+                out[L + "sink"] = need(self._find(weights, pre, k.sink, ""), f"layer {i} sinks")
             wo = T(self._find(weights, pre, k.o))
             if wo is None:
                 wo = deq([p + n + ".weight" for p in pre for n in k.o])
@@ -232,8 +246,8 @@ class DecoderModel(Model):
                 b = self._find(weights, pre, k.o, ".bias")
                 out[L + "bo"] = b if b is not None else torch.zeros(s.hidden_size)
             # ---- MLP ----
-            moe = s.layer_is_moe(i)
-            if (not moe) or s.moe.dense_parallel:
+            moe = ls.mlp == "moe"
+            if ls.mlp == "dense" or (moe and ls.moe.dense_parallel):
                 if s.mlp == "gated":
                     gu = T(self._find(weights, pre, k.gate_up)) if k.gate_up else None
                     if gu is None:
@@ -257,8 +271,10 @@ class DecoderModel(Model):
                     b = self._find(weights, pre, k.down, ".bias")
                     out[L + "b_down"] = b if b is not None else torch.zeros(s.hidden_size)
             if moe:
-                m = s.moe
+                m = ls.moe
                 out[L + "router"] = need(self._find(weights, pre, k.router), f"layer {i} router")
+                if m.router_bias:
+                    out[L + "router_b"] = need(self._find(weights, pre, k.router, ".bias"), f"layer {i} router bias")
                 gus, dns = [], []
                 for e in range(m.num_experts):
                     epre = tuple(p + x.format(e=e) for p in pre for x in k.expert)
@@ -272,8 +288,9 @@ class DecoderModel(Model):
                 out[L + "experts_down"] = torch.stack(dns)
                 if m.num_shared_experts:
                     g = need(self._find(weights, pre, k.shared_gate), "shared gate")
-                    u = need(self._find(weights, pre, k.shared_up), "shared up")
-                    out[L + "shared_gate_up"] = torch.cat([g, u], 0)
+                    if m.gated:
+                        g = torch.cat([g, need(self._find(weights, pre, k.shared_up), "shared up")], 0)
+                    out[L + "shared_gate_up"] = g
                     out[L + "shared_down"] = need(self._find(weights, pre, k.shared_down), "shared down")
         if s.final_norm:
             out["final_norm.w"] = need(self._find(weights, root, k.final_norm), "final norm")
@@ -338,83 +355,95 @@ class DecoderModel(Model):
         """Parameters under the family's on-disk names (first alias of each scheme entry)."""
         s, k = self.spec, self.scheme
         out: Dict[str, torch.Tensor] = {}
+        WS, BS = k.weight_suffix, k.bias_suffix
 
         def T(t):
             return t.t().contiguous() if k.transposed and t.dim() == 2 else t
 
-        out[k.embed[0] + ".weight"] = self.p["embed"]
+        out[k.embed[0] + WS] = self.p["embed"]
         if s.embed_proj_dim:
-            out[k.project_in[0] + ".weight"] = self.p["project_in"]
-            out[k.project_out[0] + ".weight"] = self.p["project_out"]
+            out[k.project_in[0] + WS] = self.p["project_in"]
+            out[k.project_out[0] + WS] = self.p["project_out"]
         if s.pos == "learned":
-            out[k.pos_embed[0] + ".weight"] = self.p["pos_embed"]
+            out[k.pos_embed[0] + WS] = self.p["pos_embed"]
         if s.embed_norm:
-            out[k.embed_norm[0] + ".weight"] = self.p["embed_norm.w"]
-            out[k.embed_norm[0] + ".bias"] = self.p["embed_norm.b"]
+            out[k.embed_norm[0] + WS] = self.p["embed_norm.w"]
+            out[k.embed_norm[0] + BS] = self.p["embed_norm.b"]
         for i in range(s.num_layers):
             L, pre = f"layers.{i}.", k.layer[0].format(i=i)
-            out[pre + k.ln1[0] + ".weight"] = self.p[L + "ln1.w"]
+            ls = s.layer(i)
+            out[pre + k.ln1[0] + WS] = self.p[L + "ln1.w"]
             if s.norm_bias:
-                out[pre + k.ln1[0] + ".bias"] = self.p[L + "ln1.b"]
+                out[pre + k.ln1[0] + BS] = self.p[L + "ln1.b"]
             if L + "ln2.w" in self.p:
-                out[pre + k.ln2[0] + ".weight"] = self.p[L + "ln2.w"]
+                out[pre + k.ln2[0] + WS] = self.p[L + "ln2.w"]
                 if s.norm_bias:
-                    out[pre + k.ln2[0] + ".bias"] = self.p[L + "ln2.b"]
+                    out[pre + k.ln2[0] + BS] = self.p[L + "ln2.b"]
             wqkv = self.p[L + "wqkv"]
             if k.qkv:
-                out[pre + k.qkv[0] + ".weight"] = T(self._pack_qkv(wqkv))
+                out[pre + k.qkv[0] + WS] = T(self._pack_qkv(wqkv))
                 if s.qkv_bias:
-                    out[pre + k.qkv[0] + ".bias"] = self._pack_qkv(self.p[L + "bqkv"][:, None])[:, 0]
+                    out[pre + k.qkv[0] + BS] = self._pack_qkv(self.p[L + "bqkv"][:, None])[:, 0]
+            elif ls.kv_from is not None:
+                out[pre + k.q[0] + WS] = T(wqkv)
             else:
-                q, kk, v = wqkv.split([s.q_size, s.kv_size, s.kv_size])
-                out[pre + k.q[0] + ".weight"], out[pre + k.k[0] + ".weight"], out[pre + k.v[0] + ".weight"] = T(q), T(kk), T(v)
+                q, kk, v = wqkv.split([ls.q_size, ls.k_size, ls.v_size])
+                out[pre + k.q[0] + WS], out[pre + k.k[0] + WS], out[pre + k.v[0] + WS] = T(q), T(kk), T(v)
                 if s.qkv_bias:
                     qb, kb, vb = self.p[L + "bqkv"].split([s.q_size, s.kv_size, s.kv_size])
-                    out[pre + k.q[0] + ".bias"], out[pre + k.k[0] + ".bias"], out[pre + k.v[0] + ".bias"] = qb, kb, vb
+                    out[pre + k.q[0] + BS], out[pre + k.k[0] + BS], out[pre + k.v[0] + BS] = qb, kb, vb
             if s.qk_norm:
-                out[pre + k.q_norm[0] + ".weight"] = self.p[L + "q_norm"]
-                out[pre + k.k_norm[0] + ".weight"] = self.p[L + "k_norm"]
-            out[pre + k.o[0] + ".weight"] = T(self.p[L + "wo"])
+                out[pre + k.q_norm[0] + WS] = self.p[L + "q_norm"]
+                if ls.kv_from is None:
+                    out[pre + k.k_norm[0] + WS] = self.p[L + "k_norm"]
+            if ls.sink:
+                out[pre + k.sink[0]] = self.p[L + "sink"]
+            out[pre + k.o[0] + WS] = T(self.p[L + "wo"])
             if s.o_bias:
-                out[pre + k.o[0] + ".bias"] = self.p[L + "bo"]
+                out[pre + k.o[0] + BS] = self.p[L + "bo"]
             if L + "w_gate_up" in self.p:
                 if k.gate_up:
-                    out[pre + k.gate_up[0] + ".weight"] = T(self.p[L + "w_gate_up"])
+                    out[pre + k.gate_up[0] + WS] = T(self.p[L + "w_gate_up"])
                 else:
                     g, u = self.p[L + "w_gate_up"].chunk(2, 0)
-                    out[pre + k.gate[0] + ".weight"], out[pre + k.up[0] + ".weight"] = T(g), T(u)
+                    out[pre + k.gate[0] + WS], out[pre + k.up[0] + WS] = T(g), T(u)
             if L + "w_up" in self.p:
-                out[pre + k.up[0] + ".weight"] = T(self.p[L + "w_up"])
+                out[pre + k.up[0] + WS] = T(self.p[L + "w_up"])
                 if s.mlp_bias:
-                    out[pre + k.up[0] + ".bias"] = self.p[L + "b_up"]
+                    out[pre + k.up[0] + BS] = self.p[L + "b_up"]
             if L + "w_down" in self.p:
-                out[pre + k.down[0] + ".weight"] = T(self.p[L + "w_down"])
+                out[pre + k.down[0] + WS] = T(self.p[L + "w_down"])
                 if s.mlp_bias:
-                    out[pre + k.down[0] + ".bias"] = self.p[L + "b_down"]
+                    out[pre + k.down[0] + BS] = self.p[L + "b_down"]
             if L + "router" in self.p:
-                m = s.moe
-                out[pre + k.router[0] + ".weight"] = self.p[L + "router"]
+                m = ls.moe
+                out[pre + k.router[0] + WS] = self.p[L + "router"]
+                if m.router_bias:
+                    out[pre + k.router[0] + BS] = self.p[L + "router_b"]
                 for e in range(m.num_experts):
                     ep = pre + k.expert[0].format(e=e)
                     gu = self.p[L + "experts_gate_up"][e]
                     if m.gated:
                         g, u = gu.chunk(2, 0)
-                        out[ep + k.e_gate[0] + ".weight"], out[ep + k.e_up[0] + ".weight"] = g, u
+                        out[ep + k.e_gate[0] + WS], out[ep + k.e_up[0] + WS] = g, u
                     else:
-                        out[ep + k.e_gate[0] + ".weight"] = gu
-                    out[ep + k.e_down[0] + ".weight"] = self.p[L + "experts_down"][e]
+                        out[ep + k.e_gate[0] + WS] = gu
+                    out[ep + k.e_down[0] + WS] = self.p[L + "experts_down"][e]
                 if m.num_shared_experts:
-                    g, u = self.p[L + "shared_gate_up"].chunk(2, 0)
-                    out[pre + k.shared_gate[0] + ".weight"], out[pre + k.shared_up[0] + ".weight"] = g, u
-                    out[pre + k.shared_down[0] + ".weight"] = self.p[L + "shared_down"]
+                    if m.gated:
+                        g, u = self.p[L + "shared_gate_up"].chunk(2, 0)
+                        out[pre + k.shared_gate[0] + WS], out[pre + k.shared_up[0] + WS] = g, u
+                    else:
+                        out[pre + k.shared_gate[0] + WS] = self.p[L + "shared_gate_up"]
+                    out[pre + k.shared_down[0] + WS] = self.p[L + "shared_down"]
         if s.final_norm:
-            out[k.final_norm[0] + ".weight"] = self.p["final_norm.w"]
+            out[k.final_norm[0] + WS] = self.p["final_norm.w"]
             if s.norm_bias:
-                out[k.final_norm[0] + ".bias"] = self.p["final_norm.b"]
+                out[k.final_norm[0] + BS] = self.p["final_norm.b"]
         if not s.tie_embeddings:
-            out[k.lm_head[0] + ".weight"] = self.p["lm_head"]
+            out[k.lm_head[0] + WS] = self.p["lm_head"]
         if s.lm_head_bias:
-            out[k.lm_head[0] + ".bias"] = self.p["lm_head_bias"]
+            out[k.lm_head[0] + BS] = self.p["lm_head_bias"]
         md = WeightMetadata(architecture=type(self._config).__name__, total_params=sum(t.numel() for t in out.values()),
                             format="memory", dtype=str(self.dtype))
         return ModelWeights({n: t.contiguous() for n, t in out.items()}, md)
@@ -444,54 +473,89 @@ class DecoderModel(Model):
             return ops_fn.rms_norm(x, (w.float() + 1.0).to(w.dtype), eps)
         return ops_fn.rms_norm(x, w, eps)
 
-    def _rope_cache(self, need_len: int) -> RoPECache:
+    def _rope_cache(self, need_len: int, ls: Optional[LayerSpec] = None) -> RoPECache:
+        """Tables of one rotation; layers with the same rotation share them."""
         s = self.spec
-        if self._rope is None or self._rope.max_seq_len < need_len or self._rope.cos.device != self.device:
+        ls = ls or s.layer(0)
+        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3)
+        if self._rope is None:
+            self._rope = {}
+        c = self._rope.get(key)
+        if c is None or c.max_seq_len < need_len or c.cos.device != self.device:
             n = max(need_len, min(s.max_position_embeddings, 8192))
-            self._rope = RoPECache(s.head_dim, n, s.rope_theta, rotary_dim=s.rd, position_scale=s.rope_pos_scale,
-                                   llama3=s.rope_llama3, device=self.device)
-        return self._rope
+            c = self._rope[key] = RoPECache(ls.head_dim, n, ls.rope_theta, rotary_dim=ls.rotary_dim,
+                                            position_scale=s.rope_pos_scale, llama3=ls.rope_llama3, device=self.device)
+        return c
 
-    def _attention(self, i: int, h: torch.Tensor, past: int, cache: Optional[KVCache]) -> torch.Tensor:
-        s = self.spec
+    def _project_qkv(self, i: int, h: torch.Tensor):
+        """(q, k, v) of layer ``i`` as [..., heads, size] before rotation, normalised where the design has it; k and v
+        are None when the layer reads another layer's."""
+        s, ls = self.spec, self.spec.layer(i)
         L = f"layers.{i}."
-        B, T, _ = h.shape
         qkv = ops_fn.linear(h, self.p[L + "wqkv"], self.p.get(L + "bqkv"))
-        q, k, v = qkv.split([s.q_size, s.kv_size, s.kv_size], dim=-1)
-        q = q.reshape(B, T, s.num_heads, s.head_dim)
-        k = k.reshape(B, T, s.num_kv_heads, s.head_dim)
-        v = v.reshape(B, T, s.num_kv_heads, s.head_dim)
+        lead = h.shape[:-1]
+        k = v = None
+        if ls.kv_from is None:
+            q, k, v = qkv.split([ls.q_size, ls.k_size, ls.v_size], dim=-1)
+            k = k.reshape(*lead, ls.num_kv_heads, ls.head_dim)
+            v = v.reshape(*lead, ls.num_kv_heads, ls.v_head_dim)
+        else:
+            q = qkv
+        q = q.reshape(*lead, ls.num_heads, ls.head_dim)
         if s.qk_norm:
             q = ops_fn.rms_norm(q, self.p[L + "q_norm"], s.norm_eps)
-            k = ops_fn.rms_norm(k, self.p[L + "k_norm"], s.norm_eps)
-        if s.pos == "rope" and s.rd > 0:
-            cos, sin = self._rope_cache(past + T).get_range(past, past + T)
-            q = apply_rope(q, cos, sin, s.rd, s.rope_interleaved)
-            k = apply_rope(k, cos, sin, s.rd, s.rope_interleaved)
-        k, v = k.transpose(1, 2), v.transpose(1, 2)      # [B, Hkv, T, D]
-        if cache is not None:
-            lc = cache.layer(i)
-            lc.append(k, v)
-            k, v = lc.get_kv()
+            if k is not None:
+                k = ops_fn.rms_norm(k, self.p[L + "k_norm"], s.norm_eps)
+        return q, k, v
+
+    def _attend(self, i: int, q, k, v, bias):
+        """q [B, Hq, T, Dk], k / v [B, Hkv, S, ...] in fp32, additive ``bias`` [T, S] or [Hq, T, S] -> [B, Hq, T, Dv]."""
+        ls = self.spec.layer(i)
+        g = ls.num_heads // ls.num_kv_heads
+        if g > 1:
+            k, v = k.repeat_interleave(g, dim=1), v.repeat_interleave(g, dim=1)
+        scale = ls.scale if ls.scale is not None else 1.0 / math.sqrt(ls.head_dim)
+        if not ls.sink:
+            return F.scaled_dot_product_attention(q, k, v, attn_mask=bias, scale=scale)
+        sc = torch.matmul(q, k.transpose(-1, -2)) * scale + bias
+        sink = self.p[f"layers.{i}.sink"].to(sc).reshape(-1, 1, 1).expand(*sc.shape[:-1], 1)
+        # the sink is one more column of the softmax that has no value
+        p = torch.softmax(torch.cat([sc, sink], dim=-1), dim=-1)[..., :-1]
+        return torch.matmul(p, v)
+
+    def _attention(self, i: int, h: torch.Tensor, past: int, cache: Optional[KVCache], shared: dict) -> torch.Tensor:
+        s, ls = self.spec, self.spec.layer(i)
+        L = f"layers.{i}."
+        B, T, _ = h.shape
+        q, k, v = self._project_qkv(i, h)
+        if ls.rotary_dim > 0:
+            cos, sin = self._rope_cache(past + T, ls).get_range(past, past + T)
+            q = apply_rope(q, cos, sin, ls.rotary_dim, s.rope_interleaved)
+            if k is not None:
+                k = apply_rope(k, cos, sin, ls.rotary_dim, s.rope_interleaved)
+        if ls.kv_from is not None:
+            k, v = shared[ls.kv_from]
+        else:
+            k, v = k.transpose(1, 2), v.transpose(1, 2)      # [B, Hkv, T, D]
+            if cache is not None:
+                lc = cache.layer(i)
+                lc.append(k, v)
+                k, v = lc.get_kv()
+            shared[i] = (k, v)
         q = q.transpose(1, 2)                             # [B, Hq, T, D]
         S = k.shape[2]
-        g = s.num_heads // s.num_kv_heads
-        kf, vf = _f(k), _f(v)
-        if g > 1:
-            kf, vf = kf.repeat_interleave(g, dim=1), vf.repeat_interleave(g, dim=1)
-        scale = s.attn_scale if s.attn_scale is not None else 1.0 / math.sqrt(s.head_dim)
         qpos = torch.arange(past, past + T, device=h.device)[:, None]
         kpos = torch.arange(S, device=h.device)[None, :]
         vis = kpos <= qpos
-        if s.window > 0:
-            vis = vis & (kpos > qpos - s.window)
+        if ls.window > 0:
+            vis = vis & (kpos > qpos - ls.window)
         bias = torch.zeros(T, S, device=h.device, dtype=torch.float32).masked_fill(~vis, float("-inf"))
         if s.pos == "alibi":
             if self._alibi is None or self._alibi.device != h.device:
                 self._alibi = alibi_slopes(s.num_heads).to(h.device)
             bias = bias[None] + self._alibi[:, None, None] * (kpos - qpos)[None].float()
-        y = F.scaled_dot_product_attention(_f(q), kf, vf, attn_mask=bias, scale=scale)
-        y = y.transpose(1, 2).reshape(B, T, s.q_size).to(h.dtype)
+        y = self._attend(i, _f(q), _f(k), _f(v), bias)
+        y = y.transpose(1, 2).reshape(B, T, ls.o_size).to(h.dtype)
         return ops_fn.linear(y, self.p[L + "wo"], self.p.get(L + "bo"))
 
     def _dense_mlp(self, x, w_gate_up=None, w_up=None, b_up=None, w_down=None, b_down=None, act="silu"):
@@ -504,11 +568,12 @@ class DecoderModel(Model):
         return ops_fn.linear(hdn, w_down, b_down)
 
     def _moe(self, i: int, x: torch.Tensor) -> torch.Tensor:
-        s, m = self.spec, self.spec.moe
+        m = self.spec.layer(i).moe
         L = f"layers.{i}."
         shape = x.shape
         x2 = x.reshape(-1, shape[-1])
-        logits = F.linear(_f(x2), _f(self.p[L + "router"]))
+        rb = self.p.get(L + "router_b")
+        logits = F.linear(_f(x2), _f(self.p[L + "router"]), None if rb is None else _f(rb))
         if m.normalize_topk:
             v, idx = torch.topk(logits, m.top_k, dim=-1)
             w = torch.softmax(v, dim=-1)
@@ -526,8 +591,9 @@ class DecoderModel(Model):
                 y = self._dense_mlp(x2[tok], w_up=gu[e], w_down=dn[e], act=m.act)
             out.index_add_(0, tok, _f(y) * w[tok, slot].unsqueeze(-1))
         if m.num_shared_experts:
-            out = out + _f(self._dense_mlp(x2, w_gate_up=self.p[L + "shared_gate_up"], w_down=self.p[L + "shared_down"],
-                                           act=m.act))
+            w = self.p[L + "shared_gate_up"]
+            out = out + _f(self._dense_mlp(x2, w_gate_up=w if m.gated else None, w_up=None if m.gated else w,
+                                           w_down=self.p[L + "shared_down"], act=m.act))
         return out.to(x.dtype).reshape(shape)
 
     def _mlp(self, i: int, x: torch.Tensor) -> torch.Tensor:
@@ -542,20 +608,24 @@ class DecoderModel(Model):
             y = mo if y is None else y + mo
         return y
 
-    def _layer(self, i: int, x: torch.Tensor, past: int, cache: Optional[KVCache]) -> torch.Tensor:
+    def block(self, i: int, x: torch.Tensor, attention) -> torch.Tensor:
+        """One layer around ``attention(h)``: where the norms sit and how the sublayers join the residual stream."""
         s = self.spec
         L = f"layers.{i}."
         rs = s.residual_scale
         if s.post_ln:
-            x = self._norm(x + self._attention(i, x, past, cache) * rs, L + "ln1")
+            x = self._norm(x + attention(x) * rs, L + "ln1")
             return self._norm(x + self._mlp(i, x) * rs, L + "ln2")
+        if s.norm_placement == "output":
+            x = x + self._norm(attention(x), L + "ln1") * rs
+            return x if s.layer(i).mlp is None else x + self._norm(self._mlp(i, x), L + "ln2") * rs
         h = self._norm(x, L + "ln1")
-        a = self._attention(i, h, past, cache)
+        a = attention(h)
         if s.parallel_residual:
             m_in = h if s.parallel_shared_norm else self._norm(x, L + "ln2")
             return x + (a + self._mlp(i, m_in)) * rs
         x = x + a * rs
-        return x + self._mlp(i, self._norm(x, L + "ln2")) * rs
+        return x if s.layer(i).mlp is None else x + self._mlp(i, self._norm(x, L + "ln2")) * rs
 
     def hidden_states(self, input_ids: torch.Tensor, cache: Optional[KVCache] = None,
                       inputs_embeds: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -579,8 +649,9 @@ class DecoderModel(Model):
             x = x + self.p["pos_embed"][pos][None]
         if s.embed_norm:
             x = ops_fn.layer_norm(x, self.p["embed_norm.w"], self.p["embed_norm.b"], s.norm_eps)
+        shared: dict = {}                     # keys and values of this call's layers, for those that read an earlier one's
         for i in range(s.num_layers):
-            x = self._layer(i, x, past, cache)
+            x = self.block(i, x, lambda h, i=i: self._attention(i, h, past, cache, shared))
         if cache is not None:
             cache.set_seq_len(past + T)
         if s.final_norm:

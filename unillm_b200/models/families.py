@@ -11,7 +11,8 @@ import math
 
 from . import configs as C
 from .decoder import DecoderModel
-from .spec import DecoderSpec, KeyScheme, MoESpec
+from ..types import ConfigurationError
+from .spec import DecoderSpec, KeyScheme, LayerSpec, MoESpec
 
 
 def _base(c, **kw) -> DecoderSpec:
@@ -448,11 +449,65 @@ class ArcticModel(DecoderModel):
                                     intermediate_size=c.moe_intermediate_size, dense_parallel=True, act=c.hidden_act))
 
 
+class GekapelModel(DecoderModel):
+    """Gekapel: norms on the sublayers' outputs only (the sublayers read the 32-bit residual stream itself), windowed
+    attention with per-head query / key norms, partial interleaved rotation and softmax sinks, layers that reuse an
+    earlier layer's keys and values, and mixture-of-experts feed-forwards (squared-relu experts without gates, a biased
+    router, an always-on shared expert).  Not one of the reference's families."""
+
+    config_class = C.GekapelConfig
+    scheme = KeyScheme(embed=("embed",), layer=("l{i}.",), ln1=("norm1",), ln2=("norm2",), q=("mix.q",), k=("mix.k",),
+                       v=("mix.v",), q_norm=("mix.q.norm",), k_norm=("mix.k.norm",), sink=("mix.sink",), o=("mix.o",),
+                       router=("mlp.router",), expert=("mlp.e{e}.",), e_gate=("up",), e_down=("down",),
+                       shared_gate=("mlp.shared.up",), shared_down=("mlp.shared.down",), final_norm=("final.norm",),
+                       lm_head=("head",), weight_suffix="", bias_suffix=".b")
+
+    @staticmethod
+    def _layer_spec(i: int, d: dict, layers) -> LayerSpec:
+        if d.get("type", "attention") != "attention":
+            raise ConfigurationError(f"layer {i}: unknown mixer {d.get('type')!r}")
+        mx, mlp, rot = d["mixer"], d.get("mlp"), d["mixer"].get("rot")
+        sc = rot.get("scaling") if rot else None
+        src = mx.get("kv_from")
+        if src is not None:
+            if not 0 <= src < i or layers[src]["mixer"].get("kv_from") is not None:
+                raise ConfigurationError(f"layer {i}: kv_from {src} is not an earlier layer with keys of its own")
+            if any(layers[src]["mixer"][n] != mx[n] for n in ("kv_heads", "dim", "vdim")):
+                raise ConfigurationError(f"layer {i}: keys of layer {src} have other sizes")
+        if mx["heads"] % mx["kv_heads"]:
+            raise ConfigurationError(f"layer {i}: {mx['heads']} heads over {mx['kv_heads']} key/value heads")
+        moe = None
+        if mlp is not None:
+            if mlp.get("kind", "moe") != "moe":
+                raise ConfigurationError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
+            sh = mlp.get("shared")
+            moe = MoESpec(num_experts=mlp["router"]["experts"], top_k=mlp["router"]["top"],
+                          intermediate_size=mlp["expert"]["ff"], normalize_topk=True, act="relu2", gated=False,
+                          router_bias=True, num_shared_experts=0 if sh is None else 1,
+                          shared_intermediate_size=None if sh is None else sh["ff"])
+        return LayerSpec(num_heads=mx["heads"], num_kv_heads=mx["kv_heads"], head_dim=mx["dim"], v_head_dim=mx["vdim"],
+                         window=mx["mask"]["size"] if mx.get("mask") else 0, scale=float(mx["scale"]),
+                         rotary_dim=rot["dims"] if rot else 0, rope_theta=float(rot["base"]) if rot else 10000.0,
+                         rope_llama3=None if sc is None else tuple(float(sc[n]) for n in ("factor", "low", "high", "original")),
+                         kv_from=src, sink=True, mlp=None if moe is None else "moe", moe=moe)
+
+    @classmethod
+    def spec_from_config(cls, c):
+        layers = tuple(cls._layer_spec(i, d, c.layers) for i, d in enumerate(c.layers))
+        first = layers[0] if layers else None
+        return DecoderSpec(vocab_size=c.vocab_size, hidden_size=c.hidden_size, num_layers=len(layers), layers=layers,
+                           num_heads=first.num_heads if first else 0, num_kv_heads=first.num_kv_heads if first else 0,
+                           head_dim=first.head_dim if first else 0, intermediate_size=0,
+                           max_position_embeddings=c.max_position_embeddings, norm="layer", norm_eps=c.norm_eps,
+                           norm_bias=True, norm_placement="output", residual_fp32=True, qk_norm=True,
+                           rope_interleaved=True, initializer_range=c.initializer_range)
+
+
 DECODER_FAMILIES = {
     "llama": LlamaModel, "qwen": QwenModel, "gemma": GemmaModel, "phi": PhiModel, "deepseek": DeepSeekModel,
     "mistral": MistralModel, "mixtral": MixtralModel, "gpt2": GPT2Model, "gptj": GPTJModel, "gptneox": GPTNeoXModel,
     "opt": OPTModel, "bloom": BLOOMModel, "mpt": MPTModel, "starcoder": StarCoderModel, "codellama": CodeLlamaModel,
     "olmo": OlmoModel, "granite": GraniteModel, "yi": YiModel, "falcon": FalconModel, "baichuan": BaichuanModel,
     "internlm": InternLMModel, "chatglm": ChatGLMModel, "minicpm": MiniCPMModel, "deepseek_moe": DeepSeekMoEModel,
-    "dbrx": DbrxModel, "grok": GrokModel, "arctic": ArcticModel,
+    "dbrx": DbrxModel, "grok": GrokModel, "arctic": ArcticModel, "gekapel": GekapelModel,
 }

@@ -9,6 +9,10 @@ linear or Llama-3 scaling / interleaved), ALiBi, learned positions, sliding wind
 residual topology (sequential / parallel, shared or separate norms, post-LN), MLP kind (gated /
 plain, activation), biases, embedding / logit / residual / attention scalings, tied embeddings, and
 mixture-of-experts (experts, top-k, shared experts, dense-parallel MLP, leading dense layers).
+
+Designs whose layers differ from one another (head counts, head sizes, windows, rotations, feed-forward sizes, layers
+without a feed-forward, layers that read another layer's keys and values) list a ``LayerSpec`` per layer;
+``DecoderSpec.layer(i)`` answers for every spec, so the loaders and runners ask it instead of the uniform fields.
 """
 from __future__ import annotations
 
@@ -26,7 +30,57 @@ class MoESpec:
     dense_parallel: bool = False         # Arctic: dense MLP output + MoE output
     first_k_dense: int = 0               # leading layers that use the dense MLP instead of MoE
     act: str = "silu"
-    gated: bool = True
+    gated: bool = True                   # False: down(act(up x)) experts (and shared experts)
+    router_bias: bool = False            # logits = W x + b
+    shared_intermediate_size: Optional[int] = None   # width of the always-on expert; None: num_shared * intermediate_size
+
+    @property
+    def shared_width(self) -> int:
+        if self.shared_intermediate_size is not None:
+            return self.shared_intermediate_size
+        return self.num_shared_experts * self.intermediate_size
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """What one layer's sublayers look like.  ``kv_from``: the layer has no key / value projections and attends to the
+    cached keys and values of that earlier layer (its own queries, window, scale and sinks).  ``mlp``: "dense", "moe" or
+    None (no feed-forward)."""
+
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int                        # query / key size
+    v_head_dim: int
+    window: int = 0                      # keys p - window + 1 .. p; 0 = all
+    scale: Optional[float] = None        # None = 1/sqrt(head_dim)
+    rotary_dim: int = 0
+    rope_theta: float = 10000.0
+    rope_llama3: Optional[Tuple[float, float, float, float]] = None
+    kv_from: Optional[int] = None
+    sink: bool = False                   # one learned logit per head in the softmax denominator
+    mlp: Optional[str] = "dense"
+    moe: Optional[MoESpec] = None
+
+    @property
+    def q_size(self) -> int:
+        return self.num_heads * self.head_dim
+
+    @property
+    def k_size(self) -> int:
+        return self.num_kv_heads * self.head_dim
+
+    @property
+    def v_size(self) -> int:
+        return self.num_kv_heads * self.v_head_dim
+
+    @property
+    def o_size(self) -> int:
+        return self.num_heads * self.v_head_dim
+
+    @property
+    def qkv_size(self) -> int:
+        """Rows of the fused projection: [Q; K; V], or Q alone for a layer that reads another layer's keys."""
+        return self.q_size if self.kv_from is not None else self.q_size + self.k_size + self.v_size
 
 
 @dataclass
@@ -67,6 +121,9 @@ class DecoderSpec:
     parallel_residual: bool = False      # x + attn(n1(x)) + mlp(n2(x))
     parallel_shared_norm: bool = False   # ... with mlp reading n1(x) (GPT-J, Phi, Falcon-7B)
     post_ln: bool = False                # OPT-350m style: norm after the residual add
+    norm_placement: str = "input"        # "input": x + f(norm(x)) | "output": x + norm(f(x)), sublayers read x itself
+    residual_fp32: bool = False          # the residual stream is kept in 32 bits between the layers
+    layers: Optional[Tuple[LayerSpec, ...]] = None   # per-layer description; None: all layers as the fields above say
     # scalings
     embed_scale: float = 1.0
     logit_scale: float = 1.0
@@ -93,14 +150,30 @@ class DecoderSpec:
     def rd(self) -> int:
         return self.head_dim if self.rotary_dim is None else self.rotary_dim
 
+    def layer(self, i: int) -> LayerSpec:
+        if self.layers is not None:
+            return self.layers[i]
+        return LayerSpec(num_heads=self.num_heads, num_kv_heads=self.num_kv_heads, head_dim=self.head_dim,
+                         v_head_dim=self.head_dim, window=self.window, scale=self.attn_scale,
+                         rotary_dim=self.rd if self.pos == "rope" else 0, rope_theta=self.rope_theta,
+                         rope_llama3=self.rope_llama3, mlp="moe" if self.layer_is_moe(i) else "dense",
+                         moe=self.moe if self.layer_is_moe(i) else None)
+
     def layer_is_moe(self, i: int) -> bool:
+        if self.layers is not None:
+            return self.layers[i].mlp == "moe"
         return self.moe is not None and i >= self.moe.first_k_dense
+
+    @property
+    def kv_layers(self) -> Tuple[int, ...]:
+        """Layers that own keys and values (the others read one of these)."""
+        return tuple(i for i in range(self.num_layers) if self.layer(i).kv_from is None)
 
 
 @dataclass
 class KeyScheme:
     """Tensor names of one family.  Every entry is a tuple of aliases, tried in order; layer-level
-    names are relative to ``layer.format(i=...)``.  ``.weight`` / ``.bias`` are appended."""
+    names are relative to ``layer.format(i=...)``.  ``weight_suffix`` / ``bias_suffix`` are appended (sinks have none)."""
 
     embed: Tuple[str, ...] = ("model.embed_tokens",)
     pos_embed: Tuple[str, ...] = ()
@@ -124,6 +197,9 @@ class KeyScheme:
     gate_up: Tuple[str, ...] = ()        # packed [gate; up]
     final_norm: Tuple[str, ...] = ("model.norm",)
     lm_head: Tuple[str, ...] = ("lm_head",)
+    sink: Tuple[str, ...] = ()           # per-head softmax sinks
+    weight_suffix: str = ".weight"
+    bias_suffix: str = ".bias"
     transposed: bool = False             # GPT-2 Conv1D stores [in, out]
     router: Tuple[str, ...] = ("block_sparse_moe.gate",)
     expert: Tuple[str, ...] = ("block_sparse_moe.experts.{e}.",)
