@@ -269,28 +269,29 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const UbAttnArgs a, co
 }
 
 // Merge the split partials: out = sum_i O_i * exp(lse_i - lse_max) / sum_i exp(lse_i - lse_max).
+// A softmax sink (one logit per head without a value) joins the denominator here, once.
 __global__ void attn_split_merge_kernel(const float* scratch, __nv_bfloat16* out, float* lse_out, int Hq, int D,
-                                        int splits, long long o_stride) {
+                                        int splits, long long o_stride, const float* sinks) {
   const int seq = blockIdx.x, h = blockIdx.y;
   const float* sp = scratch + ((long long)seq * Hq + h) * splits * (D + 2);
-  float mx = -CUDART_INF_F;
+  float mx = sinks != nullptr ? sinks[h] : -CUDART_INF_F;
   for (int i = 0; i < splits; ++i) mx = fmaxf(mx, sp[i * (D + 2) + D]);
-  float den = 0.f;
+  float den = sinks != nullptr ? expf(sinks[h] - mx) : 0.f;
   for (int i = 0; i < splits; ++i) {
     const float ls = sp[i * (D + 2) + D];
-    den += (ls == -CUDART_INF_F) ? 0.f : __expf(ls - mx);
+    den += (ls == -CUDART_INF_F) ? 0.f : expf(ls - mx);
   }
   for (int d = threadIdx.x; d < D; d += blockDim.x) {
     float o = 0.f;
     for (int i = 0; i < splits; ++i) {
       const float ls = sp[i * (D + 2) + D];
-      const float w = (ls == -CUDART_INF_F) ? 0.f : __expf(ls - mx);
+      const float w = (ls == -CUDART_INF_F) ? 0.f : expf(ls - mx);
       o += sp[i * (D + 2) + d] * w;
     }
     out[(long long)seq * o_stride + (long long)h * D + d] = __float2bfloat16(den > 0.f ? o / den : 0.f);
   }
   if (threadIdx.x == 0 && lse_out != nullptr)
-    lse_out[(long long)seq * Hq + h] = den > 0.f ? mx + __logf(den) : -CUDART_INF_F;
+    lse_out[(long long)seq * Hq + h] = den > 0.f ? mx + logf(den) : -CUDART_INF_F;
 }
 
 // Merge two independently computed attention partials over disjoint key sets.
@@ -355,28 +356,30 @@ static bool decode_warp_enabled() {
   return v == 1;
 }
 
+// The warp-MMA kernel and, for split ranges, the merge of the partials.
+static int launch_mma(const UbAttnArgs& a, cudaStream_t st) {
+  const int rc = ub_attn_decode_mma_main(&a, st);
+  if (rc != 0 || a.splits == 1) return rc;
+  const int dv = a.Dv > 0 ? a.Dv : a.D;
+  attn_split_merge_kernel<<<dim3(a.num_seqs, a.Hq), dv <= 128 ? dv : 128, 0, st>>>(
+      a.scratch, reinterpret_cast<__nv_bfloat16*>(a.out), a.lse, a.Hq, dv, a.splits, a.o_stride, a.sinks);
+  const cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -(int)e;
+}
+
 template <int D>
 static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
-  const bool mma_ok = D <= 128 && decode_mma_enabled() && ub_attn_decode_mma_supported(&a);
+  const bool plain = a.sinks == nullptr && (a.Dv == 0 || a.Dv == D);     // what the older kernels take
+  const bool mma_ok = (D <= 128 || !plain) && (decode_mma_enabled() || !plain) && ub_attn_decode_mma_supported(&a);
   if (a.merge_o != nullptr && (!mma_ok || a.splits != 1)) return -7;   // fused merge lives in the warp-MMA kernels only
   // one warp per item needs enough items to keep every SM's copy engines busy; with fewer, an item is better served by
   // the four warps of a CTA
-  if (mma_ok && a.splits == 1 && a.num_seqs * a.Hkv >= 256 && decode_warp_enabled() && ub_attn_decode_warp_supported(&a))
+  if (!plain && !mma_ok) return -4;
+  if (plain && mma_ok && a.splits == 1 && a.num_seqs * a.Hkv >= 256 && decode_warp_enabled() && ub_attn_decode_warp_supported(&a))
     return ub_attn_decode_warp(&a, st);
-  if (mma_ok && a.kv_start > 0 && decode_persist_enabled() && ub_attn_decode_persist_supported(&a))
+  if (plain && mma_ok && a.kv_start > 0 && decode_persist_enabled() && ub_attn_decode_persist_supported(&a))
     return ub_attn_decode_persist(&a, st);
-  if (mma_ok) {
-    int rc = ub_attn_decode_mma_main(&a, st);
-    if (rc != 0) return rc;
-    if (a.splits > 1) {
-      dim3 g2(a.num_seqs, a.Hq);
-      attn_split_merge_kernel<<<g2, D <= 128 ? D : 128, 0, st>>>(a.scratch, reinterpret_cast<__nv_bfloat16*>(a.out),
-                                                                 a.lse, a.Hq, D, a.splits, a.o_stride);
-      cudaError_t e = cudaGetLastError();
-      if (e != cudaSuccess) return -(int)e;
-    }
-    return 0;
-  }
+  if (mma_ok) return launch_mma(a, st);
   const int Gtot = a.Hq / a.Hkv;
   int G = 1;
   while (G < Gtot && G < 8) G <<= 1;
@@ -396,7 +399,7 @@ static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
   if (a.splits > 1) {
     dim3 g2(a.num_seqs, a.Hq);
     attn_split_merge_kernel<<<g2, D <= 128 ? D : 128, 0, st>>>(a.scratch, reinterpret_cast<__nv_bfloat16*>(a.out),
-                                                               a.lse, a.Hq, D, a.splits, a.o_stride);
+                                                               a.lse, a.Hq, D, a.splits, a.o_stride, nullptr);
     e = cudaGetLastError();
     if (e != cudaSuccess) return -(int)e;
   }
@@ -415,7 +418,7 @@ extern "C" int ub_attn_decode(const UbAttnArgs* a, void* stream_v) {
     case 64: return launch_decode<64>(*a, st);
     case 128: return launch_decode<128>(*a, st);
     case 256: return launch_decode<256>(*a, st);
-    default: return -4;
+    default: return a->merge_o == nullptr && ub_attn_decode_mma_supported(a) ? launch_mma(*a, st) : -4;
   }
 }
 

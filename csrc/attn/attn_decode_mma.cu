@@ -1,4 +1,5 @@
-// K4 on warp-level tensor-core MMA: paged decode attention (one query token per sequence) for head sizes 64 / 128.
+// K4 on warp-level tensor-core MMA: paged decode attention (one query token per sequence) for head sizes 64 / 128, and
+// for any others up to 256 (multiples of 8, value size apart from the query / key size) and softmax sinks.
 //
 // One CTA handles (sequence, kv head, split).  The up-to-16 query heads that share the kv head form the 16 rows of
 // an m16n8k16 A operand, so the score and P*V products for all heads of the group cost one MMA stream instead of
@@ -50,27 +51,30 @@ __device__ __forceinline__ uint32_t tile_off(int row, int chunk) {
 // STAGES = 3 for long key ranges (two tiles in flight behind the one being used, two CTAs per SM); STAGES = 2 for
 // the short suffix ranges of the cascade, where a CTA has only two to four tiles and what hides the latency of its
 // dependent loads is a third resident CTA.
-template <int D, int STAGES>
+// DK / DV: query-key and value head sizes rounded up to a compiled size; the runtime sizes may be any multiple of 8 up to
+// them (the missing chunks are zero-filled in shared memory).
+template <int DK, int DV, int STAGES>
 struct Smem {
-  static constexpr int STAGE_BYTES = 2 * KT * D * 2;                 // K tile then V tile
-  static constexpr int RED_BYTES = 4 * ROWS * D * 4;                 // per-warp partial outputs (fp32)
+  static constexpr int STAGE_BYTES = KT * (DK + DV) * 2;             // K tile then V tile
+  static constexpr int RED_BYTES = 4 * ROWS * DV * 4;                // per-warp partial outputs (fp32)
   static constexpr int PIPE_BYTES = STAGES * STAGE_BYTES > RED_BYTES ? STAGES * STAGE_BYTES : RED_BYTES;
   static constexpr int Q_OFF = PIPE_BYTES;                           // [16][D] bf16, swizzled
-  static constexpr int ML_OFF = Q_OFF + ROWS * D * 2;                // [4][16][2] floats
+  static constexpr int ML_OFF = Q_OFF + ROWS * DK * 2;               // [4][16][2] floats
   static constexpr int BT_OFF = ML_OFF + 4 * ROWS * 2 * 4;           // block-table entries of this CTA's key range
   static constexpr int BT_MAX = 256;
   static constexpr int TOTAL = BT_OFF + BT_MAX * 4;
 };
 
-template <int D, int STAGES>
+template <int DK, int DV, int STAGES>
 __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a, const int gchunks) {
   pdl_launch_dependents();
   pdl_wait();          // no global access before the previous kernel has completed
-  constexpr int CPR = D / 8;
-  using S = Smem<D, STAGES>;
+  constexpr int CPK = DK / 8, CPV = DV / 8;
+  using S = Smem<DK, DV, STAGES>;
+  const int dk = a.D, dv = a.Dv;                       // real sizes
   extern __shared__ __align__(128) uint8_t dsm[];
   uint8_t* q_sm = dsm + S::Q_OFF;
-  float (*red_o)[ROWS][D] = reinterpret_cast<float (*)[ROWS][D]>(dsm);
+  float (*red_o)[ROWS][DV] = reinterpret_cast<float (*)[ROWS][DV]>(dsm);
   float (*red_ml)[ROWS][2] = reinterpret_cast<float (*)[ROWS][2]>(dsm + S::ML_OFF);
 
   const int seq = blockIdx.x;
@@ -105,11 +109,11 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
   const __nv_bfloat16* qp = reinterpret_cast<const __nv_bfloat16*>(a.q) + (long long)seq * a.q_stride;
 
   // Q rows (heads of the group; rows past gn are zero)
-  for (int i = threadIdx.x; i < ROWS * CPR; i += 128) {
-    const int r = i / CPR, c = i % CPR;
+  for (int i = threadIdx.x; i < ROWS * CPK; i += 128) {
+    const int r = i / CPK, c = i % CPK;
     uint4 v = make_uint4(0, 0, 0, 0);
-    if (r < gn) v = *reinterpret_cast<const uint4*>(qp + (long long)(h0 + r) * D + c * 8);
-    *reinterpret_cast<uint4*>(q_sm + tile_off<D>(r, c)) = v;
+    if (r < gn && c * 8 < dk) v = *reinterpret_cast<const uint4*>(qp + (long long)(h0 + r) * dk + c * 8);
+    *reinterpret_cast<uint4*>(q_sm + tile_off<DK>(r, c)) = v;
   }
 
   // Tiles start on a page boundary, so a tile is KT / block_size whole pages: one block-table lookup and one
@@ -125,7 +129,6 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
       bt_sm[i] = (page0 + i) < a.max_blocks_per_seq ? bt[page0 + i] : -1;
   __syncthreads();                                       // q_sm and bt_sm complete
   const int pages_per_tile = KT >> bs_shift;
-  const int chunks_per_page = CPR << bs_shift;
   auto issue_tile = [&](int t) {
     if (t < n_tiles) {
       uint8_t* st = dsm + (t % STAGES) * S::STAGE_BYTES;
@@ -138,15 +141,29 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
           const int bi = pos0 >> bs_shift;
           const int blk = bi >= a.max_blocks_per_seq ? -1 : ((bi - page0) < S::BT_MAX ? bt_sm[bi - page0] : bt[bi]);
           if (blk < 0 || blk >= a.num_blocks) set_err(a.err, ERR_BOUNDS, seq);
-          else base = (((long long)blk * a.Hkv + kvh) << bs_shift) * D;
+          else base = ((long long)blk * a.Hkv + kvh) << bs_shift;         // first cache row of the page
         }
-        for (int c = threadIdx.x; c < chunks_per_page; c += 128) {
-          const int tr = c / CPR;                                        // token inside the page (CPR is a power of two)
-          const int r = (pg << bs_shift) + tr;
-          const bool ok = tr < nvalid;
-          const uint32_t dst = tile_off<D>(r, c % CPR);
-          cp_async16(st + dst, kc + base + c * 8, ok);
-          cp_async16(st + KT * D * 2 + dst, vc + base + c * 8, ok);
+        if (DK == DV && dk == DK && dv == DV) {
+          const long long off = base * DK;
+          for (int c = threadIdx.x; c < (CPK << bs_shift); c += 128) {
+            const int tr = c / CPK;                                      // token inside the page (CPK is a power of two)
+            const int r = (pg << bs_shift) + tr;
+            const bool ok = tr < nvalid;
+            const uint32_t dst = tile_off<DK>(r, c % CPK);
+            cp_async16(st + dst, kc + off + c * 8, ok);
+            cp_async16(st + KT * DK * 2 + dst, vc + off + c * 8, ok);
+          }
+        } else {
+          for (int c = threadIdx.x; c < (CPK << bs_shift); c += 128) {
+            const int tr = c / CPK, ch = c % CPK, r = (pg << bs_shift) + tr;
+            const bool ok = tr < nvalid && ch * 8 < dk;
+            cp_async16(st + tile_off<DK>(r, ch), kc + (ok ? (base + tr) * dk + ch * 8 : 0), ok);
+          }
+          for (int c = threadIdx.x; c < (CPV << bs_shift); c += 128) {
+            const int tr = c / CPV, ch = c % CPV, r = (pg << bs_shift) + tr;
+            const bool ok = tr < nvalid && ch * 8 < dv;
+            cp_async16(st + KT * DK * 2 + tile_off<DV>(r, ch), vc + (ok ? (base + tr) * dv + ch * 8 : 0), ok);
+          }
         }
       }
     }
@@ -154,12 +171,12 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
   };
   for (int t = 0; t < STAGES - 1; ++t) issue_tile(t);
 
-  uint32_t qf[D / 16][4];
+  uint32_t qf[DK / 16][4];
 #pragma unroll
-  for (int ks = 0; ks < D / 16; ++ks) {
+  for (int ks = 0; ks < DK / 16; ++ks) {
     const int r = (lane & 7) + ((lane >> 3) & 1) * 8;
     const int c = ks * 2 + (lane >> 4);
-    ldsm_x4(smem_u32(q_sm + tile_off<D>(r, c)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+    ldsm_x4(smem_u32(q_sm + tile_off<DK>(r, c)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
   }
 
   // this thread's rows: r_a = lane / 4 and r_b = r_a + 8 (rows are query heads)
@@ -170,9 +187,9 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
     if (rb < gn) slope_b = a.alibi_slopes[h0 + rb] * LOG2E;
   }
   const float sc = a.scale * LOG2E;
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+  for (int i = 0; i < DV / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_a = -CUDART_INF_F, m_b = -CUDART_INF_F, l_a = 0.f, l_b = 0.f;
 
   // The partial over the shared prefix that the epilogue folds in: fetched now, so that its latency runs under the
@@ -184,10 +201,10 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
     const int i = threadIdx.x + k * 128;
     pre_la[k] = 0.f;
     pre_oa[k] = 0.f;
-    if (a.merge_o != nullptr && a.splits == 1 && i < gn * D) {
-      const int h = h0 + i / D;
+    if (a.merge_o != nullptr && a.splits == 1 && i < gn * DV) {
+      const int h = h0 + i / DV;                     // the merge form has dv == DV
       pre_la[k] = a.merge_lse[(long long)seq * a.Hq + h];
-      pre_oa[k] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.merge_o)[((long long)seq * a.Hq + h) * D + i % D]);
+      pre_oa[k] = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.merge_o)[((long long)seq * a.Hq + h) * DV + i % DV]);
     }
   }
 
@@ -196,21 +213,21 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
     __syncthreads();                       // tile t visible to all; all are done with tile t-1
     issue_tile(t + STAGES - 1);
     const uint8_t* kb = dsm + (t % STAGES) * S::STAGE_BYTES;
-    const uint8_t* vb = kb + KT * D * 2;
+    const uint8_t* vb = kb + KT * DK * 2;
     const int tw0 = warp * 16;             // this warp's 16 tokens inside the tile
     const int t0 = tile_origin + t * KT + tw0;
-    if (t0 >= kv_hi || t0 + 16 <= kv_lo) continue;   // warp-uniform: nothing visible in this warp's slice             // warp-uniform: nothing visible in this warp's slice
+    if (t0 >= kv_hi || t0 + 16 <= kv_lo) continue;   // warp-uniform: nothing visible in this warp's slice
 
     float s[2][4];
 #pragma unroll
     for (int j = 0; j < 2; ++j) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks) {
+    for (int ks = 0; ks < DK / 16; ++ks) {
       const int mi = lane >> 3;
       const int r = tw0 + (mi >> 1) * 8 + (lane & 7);
       const int c = ks * 2 + (mi & 1);
       uint32_t b0, b1, b2, b3;
-      ldsm_x4(smem_u32(kb + tile_off<D>(r, c)), b0, b1, b2, b3);
+      ldsm_x4(smem_u32(kb + tile_off<DK>(r, c)), b0, b1, b2, b3);
       mma_bf16(s[0], qf[ks], b0, b1);
       mma_bf16(s[1], qf[ks], b2, b3);
     }
@@ -249,14 +266,14 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
     l_a = l_a * al_a + ps_a;
     l_b = l_b * al_b + ps_b;
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) { o[i][0] *= al_a; o[i][1] *= al_a; o[i][2] *= al_b; o[i][3] *= al_b; }
+    for (int i = 0; i < DV / 8; ++i) { o[i][0] *= al_a; o[i][1] *= al_a; o[i][2] *= al_b; o[i][3] *= al_b; }
 #pragma unroll
-    for (int dp = 0; dp < D / 16; ++dp) {
+    for (int dp = 0; dp < DV / 16; ++dp) {
       const int mi = lane >> 3;
       const int r = tw0 + (mi & 1) * 8 + (lane & 7);
       const int c = dp * 2 + (mi >> 1);
       uint32_t b0, b1, b2, b3;
-      ldsm_x4_t(smem_u32(vb + tile_off<D>(r, c)), b0, b1, b2, b3);
+      ldsm_x4_t(smem_u32(vb + tile_off<DV>(r, c)), b0, b1, b2, b3);
       mma_bf16(o[dp * 2], pf, b0, b1);
       mma_bf16(o[dp * 2 + 1], pf, b2, b3);
     }
@@ -269,7 +286,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) {
+  for (int i = 0; i < DV / 8; ++i) {
     const int d = i * 8 + (lane & 3) * 2;
     if (ra < gn) { red_o[warp][ra][d] = o[i][0]; red_o[warp][ra][d + 1] = o[i][1]; }
     if (rb < gn) { red_o[warp][rb][d] = o[i][2]; red_o[warp][rb][d + 1] = o[i][3]; }
@@ -279,8 +296,9 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
     if (rb < gn) { red_ml[warp][rb][0] = m_b; red_ml[warp][rb][1] = l_b; }
   }
   __syncthreads();
-  for (int i = threadIdx.x, it = 0; i < gn * D; i += 128, ++it) {
-    const int g = i / D, d = i % D;
+  for (int i = threadIdx.x, it = 0; i < gn * DV; i += 128, ++it) {
+    const int g = i / DV, d = i % DV;
+    if (d >= dv) continue;
     float mx = -CUDART_INF_F;
 #pragma unroll
     for (int w = 0; w < 4; ++w) mx = fmaxf(mx, red_ml[w][g][0]);
@@ -291,9 +309,17 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
       lt += red_ml[w][g][1] * scw;
       ov += red_o[w][g][d] * scw;
     }
+    const int h = h0 + g;
+    if (a.sinks != nullptr && a.splits == 1) {
+      // the sink joins the denominator (of split ranges: in the merge, once)
+      const float sk = a.sinks[h] * LOG2E;
+      const float m2 = fmaxf(mx, sk), al = mx == -CUDART_INF_F ? 0.f : exp2f(mx - m2);
+      lt = lt * al + exp2f(sk - m2);
+      ov *= al;
+      mx = m2;
+    }
     const float inv = lt > 0.f ? 1.f / lt : 0.f;
     float lse = lt > 0.f ? (mx + log2f(lt)) * LN2 : -CUDART_INF_F;
-    const int h = h0 + g;
     if (a.splits == 1) {
       float val = ov * inv;
       if (a.merge_o != nullptr) {
@@ -305,7 +331,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
           oa = it == 0 ? pre_oa[0] : it == 1 ? pre_oa[1] : it == 2 ? pre_oa[2] : pre_oa[3];
         } else {
           la = a.merge_lse[(long long)seq * a.Hq + h];
-          oa = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.merge_o)[((long long)seq * a.Hq + h) * D + d]);
+          oa = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.merge_o)[((long long)seq * a.Hq + h) * dv + d]);
         }
         const float mm = fmaxf(la, lse);
         const float wa = (la == -CUDART_INF_F) ? 0.f : __expf(la - mm);
@@ -314,33 +340,42 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
         val = den > 0.f ? (wa * oa + wb * val) / den : 0.f;
         lse = den > 0.f ? mm + __logf(den) : -CUDART_INF_F;
       }
-      reinterpret_cast<__nv_bfloat16*>(a.out)[(long long)seq * a.o_stride + (long long)h * D + d] = __float2bfloat16(val);
+      reinterpret_cast<__nv_bfloat16*>(a.out)[(long long)seq * a.o_stride + (long long)h * dv + d] = __float2bfloat16(val);
       if (d == 0 && a.lse != nullptr) a.lse[(long long)seq * a.Hq + h] = lse;
     } else {
-      float* sp = a.scratch + (((long long)seq * a.Hq + h) * a.splits + split) * (D + 2);
+      float* sp = a.scratch + (((long long)seq * a.Hq + h) * a.splits + split) * (dv + 2);
       sp[d] = ov * inv;
-      if (d == 0) sp[D] = lse;
+      if (d == 0) sp[dv] = lse;
     }
   }
 }
 
-template <int D, int STAGES>
+template <int DK, int DV, int STAGES>
 static int launch(const UbAttnArgs& a, cudaStream_t st) {
-  constexpr int SMEM = Smem<D, STAGES>::TOTAL;
+  constexpr int SMEM = Smem<DK, DV, STAGES>::TOTAL;
   static bool attr_set[UB_MAX_DEVICES] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < UB_MAX_DEVICES && !attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<D, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<DK, DV, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return -(int)e;
     attr_set[dev] = true;
   }
   const int Gtot = a.Hq / a.Hkv;
   const int gchunks = (Gtot + ROWS - 1) / ROWS;
   dim3 grid(a.num_seqs, a.Hkv * gchunks, a.splits);
-  ub::launch_pdl(attn_decode_mma_kernel<D, STAGES>, grid, dim3(128), (size_t)SMEM, st, a, gchunks);
+  ub::launch_pdl(attn_decode_mma_kernel<DK, DV, STAGES>, grid, dim3(128), (size_t)SMEM, st, a, gchunks);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
+}
+
+// Sizes of other designs: each head size rounded up to a compiled one (64, 128 or 256).
+template <int DK>
+static int launch_sized(const UbAttnArgs& a, cudaStream_t st) {
+  constexpr int S = DK > 128 ? 2 : 3;
+  if (a.Dv <= 64) return launch<DK, 64, S>(a, st);
+  if (a.Dv <= 128) return launch<DK, 128, S>(a, st);
+  return launch<DK, 256, 2>(a, st);
 }
 
 }  // namespace dmma
@@ -348,7 +383,9 @@ static int launch(const UbAttnArgs& a, cudaStream_t st) {
 
 // The main kernel of the decode step for head sizes 64 / 128 (the split merge, if any, is launched by the caller).
 extern "C" int ub_attn_decode_mma_supported(const UbAttnArgs* a) {
-  if (a->D != 64 && a->D != 128) return 0;
+  const int dv = a->Dv > 0 ? a->Dv : a->D;
+  if (a->D > 256 || dv > 256 || a->D % 8 != 0 || dv % 8 != 0) return 0;
+  if (a->merge_o != nullptr && (a->D != dv || (dv != 64 && dv != 128) || a->sinks != nullptr)) return 0;
   if (a->block_size < 8 || a->block_size > 64 || (a->block_size & (a->block_size - 1))) return 0;   // whole pages per 64-token tile
   if (a->Hkv <= 0 || a->Hq % a->Hkv != 0 || a->q_stride % 8 != 0) return 0;
   if ((reinterpret_cast<uintptr_t>(a->q) & 15) || (reinterpret_cast<uintptr_t>(a->k_cache) & 15) ||
@@ -357,8 +394,16 @@ extern "C" int ub_attn_decode_mma_supported(const UbAttnArgs* a) {
   return 1;
 }
 
-extern "C" int ub_attn_decode_mma_main(const UbAttnArgs* a, void* stream) {
+extern "C" int ub_attn_decode_mma_main(const UbAttnArgs* args, void* stream) {
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  UbAttnArgs sized = *args;
+  if (sized.Dv <= 0) sized.Dv = sized.D;
+  const UbAttnArgs* a = &sized;
+  if (a->D != a->Dv || (a->D != 64 && a->D != 128)) {
+    if (a->D <= 64) return ub::dmma::launch_sized<64>(*a, st);
+    if (a->D <= 128) return ub::dmma::launch_sized<128>(*a, st);
+    return ub::dmma::launch_sized<256>(*a, st);
+  }
   // suffix ranges after a shared prefix are short (two to four tiles): a third resident CTA per SM hides more of the
   // chain of dependent latencies than a deeper ring does (68.8 us vs 83.3 us per layer on the serving step);
   // UB_DECODE_STAGES=3 keeps the deep ring there
@@ -366,6 +411,6 @@ extern "C" int ub_attn_decode_mma_main(const UbAttnArgs* a, void* stream) {
     const char* e = getenv("UB_DECODE_STAGES");
     return (e != nullptr && atoi(e) == 3) ? 3 : 2;
   }();
-  if (a->kv_start > 0 && suffix_stages == 2) return a->D == 64 ? ub::dmma::launch<64, 2>(*a, st) : ub::dmma::launch<128, 2>(*a, st);
-  return a->D == 64 ? ub::dmma::launch<64, 3>(*a, st) : ub::dmma::launch<128, 3>(*a, st);
+  if (a->kv_start > 0 && suffix_stages == 2) return a->D == 64 ? ub::dmma::launch<64, 64, 2>(*a, st) : ub::dmma::launch<128, 128, 2>(*a, st);
+  return a->D == 64 ? ub::dmma::launch<64, 64, 3>(*a, st) : ub::dmma::launch<128, 128, 3>(*a, st);
 }

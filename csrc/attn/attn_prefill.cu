@@ -10,7 +10,8 @@
 // attention over a shared radix prefix; split-KV).
 //
 // This kernel uses warp-level mma (m16n8k16) with fp32 accumulation; the GEMM-shaped bulk of the
-// model runs on tcgen05 (csrc/gemm).  Head dims 64 and 128.
+// model runs on tcgen05 (csrc/gemm).  Head sizes up to 256 (multiples of 8; the value size may differ from the
+// query / key size), windows and softmax sinks.
 //
 // Replaces in the reference: ops_fn::flash_attention (crates/runtime/src/tensor_core.rs:1318-1383,
 // which materialises the full score matrix and a host-built mask) and the prefill case of
@@ -57,13 +58,17 @@ __device__ __forceinline__ uint32_t tile_off(int row, int chunk) {
   return (uint32_t)(row * D * 2 + ((chunk ^ (row & 7)) << 4));
 }
 
-template <int D>
+// DK / DV: query-key and value head sizes rounded up to a compiled size; the runtime sizes may be any multiple of 8 up to
+// them (the missing 16-byte chunks are zero-filled in shared memory).
+template <int DK, int DV>
 __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
-  constexpr int CPR = D / 8;  // 16-byte chunks per row
+  constexpr int CPK = DK / 8, CPV = DV / 8;  // 16-byte chunks per row
+  constexpr bool Q_REGS = DK <= 128;         // query fragments held in registers, else read per use
+  const int dk = a.D, dv = a.Dv;             // real sizes
   extern __shared__ __align__(128) uint8_t smem_p[];
-  uint8_t* q_sm = smem_p;                    // [QT][D]
-  uint8_t* k_sm = q_sm + QT * D * 2;         // [2][KT][D]
-  uint8_t* v_sm = k_sm + 2 * KT * D * 2;     // [2][KT][D]
+  uint8_t* q_sm = smem_p;                    // [QT][DK]
+  uint8_t* k_sm = q_sm + QT * DK * 2;        // [2][KT][DK]
+  uint8_t* v_sm = k_sm + 2 * KT * DK * 2;    // [2][KT][DV]
 
   const int seq = blockIdx.z, kvh = blockIdx.y;
   const int G = a.Hq / a.Hkv;
@@ -80,13 +85,13 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
   const __nv_bfloat16* qg = reinterpret_cast<const __nv_bfloat16*>(a.q);
 
   // ---- load the Q tile (packed rows) ----
-  for (int i = threadIdx.x; i < QT * CPR; i += 128) {
-    const int r = i / CPR, c = i % CPR;
+  for (int i = threadIdx.x; i < QT * CPK; i += 128) {
+    const int r = i / CPK, c = i % CPK;
     const int row = row0 + r;
-    const bool ok = row < rows_total;
+    const bool ok = row < rows_total && c * 8 < dk;
     const int tok = ok ? row / G : 0, hg = ok ? row % G : 0;
-    const __nv_bfloat16* src = qg + (long long)(qs + tok) * a.q_stride + (long long)(kvh * G + hg) * D + c * 8;
-    cp_async16(q_sm + tile_off<D>(r, c), src, ok);
+    const __nv_bfloat16* src = qg + (ok ? (long long)(qs + tok) * a.q_stride + (long long)(kvh * G + hg) * dk + c * 8 : 0);
+    cp_async16(q_sm + tile_off<DK>(r, c), src, ok);
   }
   cp_async_commit();
 
@@ -102,23 +107,35 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
 
   auto load_kv = [&](int tile, int buf) {
     const int t0 = kv_begin + tile * KT;
-    for (int i = threadIdx.x; i < KT * CPR; i += 128) {
-      const int r = i / CPR, c = i % CPR;
-      const int pos = t0 + r;
-      bool ok = pos < kv_end;
-      long long off = 0;
-      if (ok) {
-        const int bi = pos / a.block_size;
-        const int blk = bi < a.max_blocks_per_seq ? bt[bi] : -1;
-        if (blk < 0 || blk >= a.num_blocks) {
-          set_err(a.err, ERR_BOUNDS, seq);
-          ok = false;
-        } else {
-          off = (((long long)blk * a.Hkv + kvh) * a.block_size + (pos % a.block_size)) * D + c * 8;
-        }
+    auto cache_row = [&](int pos) -> long long {      // row of the caches that holds this position, -1 = outside
+      if (pos >= kv_end) return -1;
+      const int bi = pos / a.block_size;
+      const int blk = bi < a.max_blocks_per_seq ? bt[bi] : -1;
+      if (blk < 0 || blk >= a.num_blocks) {
+        set_err(a.err, ERR_BOUNDS, seq);
+        return -1;
       }
-      cp_async16(k_sm + buf * KT * D * 2 + tile_off<D>(r, c), kc + off, ok);
-      cp_async16(v_sm + buf * KT * D * 2 + tile_off<D>(r, c), vc + off, ok);
+      return ((long long)blk * a.Hkv + kvh) * a.block_size + (pos % a.block_size);
+    };
+    if (DK == DV && dk == DK && dv == DV) {
+      for (int i = threadIdx.x; i < KT * CPK; i += 128) {
+        const int r = i / CPK, c = i % CPK;
+        const long long row = cache_row(t0 + r);
+        const long long off = row >= 0 ? row * DK + c * 8 : 0;
+        cp_async16(k_sm + buf * KT * DK * 2 + tile_off<DK>(r, c), kc + off, row >= 0);
+        cp_async16(v_sm + buf * KT * DV * 2 + tile_off<DV>(r, c), vc + off, row >= 0);
+      }
+    } else {
+      for (int i = threadIdx.x; i < KT * CPK; i += 128) {
+        const int r = i / CPK, c = i % CPK;
+        const long long row = c * 8 < dk ? cache_row(t0 + r) : -1;
+        cp_async16(k_sm + buf * KT * DK * 2 + tile_off<DK>(r, c), kc + (row >= 0 ? row * dk + c * 8 : 0), row >= 0);
+      }
+      for (int i = threadIdx.x; i < KT * CPV; i += 128) {
+        const int r = i / CPV, c = i % CPV;
+        const long long row = c * 8 < dv ? cache_row(t0 + r) : -1;
+        cp_async16(v_sm + buf * KT * DV * 2 + tile_off<DV>(r, c), vc + (row >= 0 ? row * dv + c * 8 : 0), row >= 0);
+      }
     }
   };
 
@@ -137,19 +154,22 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
   }
   const float sc = a.scale * P_LOG2E;
 
-  float o[D / 8][4];
+  float o[DV / 8][4];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
+  for (int i = 0; i < DV / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
   float m_a = -CUDART_INF_F, m_b = -CUDART_INF_F, l_a = 0.f, l_b = 0.f;
 
   cp_async_wait<1>();  // Q has landed (first kv tile may still be in flight)
   __syncthreads();
-  uint32_t qf[D / 16][4];
-#pragma unroll
-  for (int ks = 0; ks < D / 16; ++ks) {
+  uint32_t qf[Q_REGS ? DK / 16 : 1][4];
+  auto load_q = [&](int ks, uint32_t (&f)[4]) {
     const int r = warp * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
     const int c = ks * 2 + (lane >> 4);
-    ldsm_x4(smem_u32(q_sm + tile_off<D>(r, c)), qf[ks][0], qf[ks][1], qf[ks][2], qf[ks][3]);
+    ldsm_x4(smem_u32(q_sm + tile_off<DK>(r, c)), f[0], f[1], f[2], f[3]);
+  };
+  if constexpr (Q_REGS) {
+#pragma unroll
+    for (int ks = 0; ks < DK / 16; ++ks) load_q(ks, qf[ks]);
   }
 
   for (int tile = 0; tile < ntiles; ++tile) {
@@ -158,8 +178,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
     cp_async_commit();
     cp_async_wait<1>();
     __syncthreads();
-    const uint8_t* kb = k_sm + buf * KT * D * 2;
-    const uint8_t* vb = v_sm + buf * KT * D * 2;
+    const uint8_t* kb = k_sm + buf * KT * DK * 2;
+    const uint8_t* vb = v_sm + buf * KT * DV * 2;
     const int t0 = kv_begin + tile * KT;
 
     // S = Q K^T  (16 x 64 per warp)
@@ -167,16 +187,18 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
 #pragma unroll
     for (int j = 0; j < KT / 8; ++j) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
 #pragma unroll
-    for (int ks = 0; ks < D / 16; ++ks) {
+    for (int ks = 0; ks < DK / 16; ++ks) {
+      if constexpr (!Q_REGS) load_q(ks, qf[0]);
+      const uint32_t (&qk)[4] = qf[Q_REGS ? ks : 0];
 #pragma unroll
       for (int jp = 0; jp < KT / 16; ++jp) {
         const int mi = lane >> 3;
         const int r = jp * 16 + (mi >> 1) * 8 + (lane & 7);
         const int c = ks * 2 + (mi & 1);
         uint32_t b0, b1, b2, b3;
-        ldsm_x4(smem_u32(kb + tile_off<D>(r, c)), b0, b1, b2, b3);
-        mma_bf16(s[jp * 2], qf[ks], b0, b1);
-        mma_bf16(s[jp * 2 + 1], qf[ks], b2, b3);
+        ldsm_x4(smem_u32(kb + tile_off<DK>(r, c)), b0, b1, b2, b3);
+        mma_bf16(s[jp * 2], qk, b0, b1);
+        mma_bf16(s[jp * 2 + 1], qk, b2, b3);
       }
     }
     // scale, mask, online softmax
@@ -220,17 +242,17 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
     l_a = l_a * al_a + ps_a;
     l_b = l_b * al_b + ps_b;
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) { o[i][0] *= al_a; o[i][1] *= al_a; o[i][2] *= al_b; o[i][3] *= al_b; }
+    for (int i = 0; i < DV / 8; ++i) { o[i][0] *= al_a; o[i][1] *= al_a; o[i][2] *= al_b; o[i][3] *= al_b; }
     // O += P V
 #pragma unroll
     for (int kk = 0; kk < KT / 16; ++kk) {
 #pragma unroll
-      for (int dp = 0; dp < D / 16; ++dp) {
+      for (int dp = 0; dp < DV / 16; ++dp) {
         const int mi = lane >> 3;
         const int r = kk * 16 + (mi & 1) * 8 + (lane & 7);
         const int c = dp * 2 + (mi >> 1);
         uint32_t b0, b1, b2, b3;
-        ldsm_x4_t(smem_u32(vb + tile_off<D>(r, c)), b0, b1, b2, b3);
+        ldsm_x4_t(smem_u32(vb + tile_off<DV>(r, c)), b0, b1, b2, b3);
         mma_bf16(o[dp * 2], pf[kk], b0, b1);
         mma_bf16(o[dp * 2 + 1], pf[kk], b2, b3);
       }
@@ -243,7 +265,19 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
-  const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
+  float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
+  if (a.sinks != nullptr) {
+    // the sink joins the denominator: o / (l + exp(sink - m)), taken relative to the larger of the two exponents
+    auto with_sink = [&](float& m, float& l, int row) {
+      const float sk = a.sinks[kvh * G + min(row, rows_total - 1) % G] * P_LOG2E;
+      const float mx = fmaxf(m, sk), al = m == -CUDART_INF_F ? 0.f : exp2f(m - mx);
+      l = l * al + exp2f(sk - mx);
+      m = mx;
+      return al / l;
+    };
+    inv_a = with_sink(m_a, l_a, rowa);
+    inv_b = with_sink(m_b, l_b, rowb);
+  }
   __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(a.out);
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
@@ -251,11 +285,11 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
     if (row >= rows_total) continue;
     const int tok = row / G, hg = row % G;
     const float inv = half ? inv_b : inv_a;
-    __nv_bfloat16* dst = og + (long long)(qs + tok) * a.o_stride + (long long)(kvh * G + hg) * D;
+    __nv_bfloat16* dst = og + (long long)(qs + tok) * a.o_stride + (long long)(kvh * G + hg) * dv;
 #pragma unroll
-    for (int i = 0; i < D / 8; ++i) {
+    for (int i = 0; i < DV / 8; ++i) {
       const int d = i * 8 + (lane & 3) * 2;
-      *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(o[i][half * 2] * inv, o[i][half * 2 + 1] * inv);
+      if (d < dv) *reinterpret_cast<uint32_t*>(dst + d) = pack_bf16x2(o[i][half * 2] * inv, o[i][half * 2 + 1] * inv);
     }
     if ((lane & 3) == 0 && a.lse != nullptr) {
       const float l = half ? l_b : l_a, m = half ? m_b : m_a;
@@ -264,21 +298,29 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
   }
 }
 
-template <int D>
+template <int DK, int DV>
 static int launch_prefill(const UbAttnArgs& a, cudaStream_t st) {
   const int G = a.Hq / a.Hkv;
-  const size_t smem = (size_t)(QT + 4 * KT) * D * 2;
+  const size_t smem = (size_t)QT * DK * 2 + (size_t)2 * KT * (DK + DV) * 2;
   static bool attr_set[UB_MAX_DEVICES] = {};
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < UB_MAX_DEVICES && !attr_set[dev]) {
-    cudaFuncSetAttribute(attn_prefill_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaFuncSetAttribute(attn_prefill_kernel<DK, DV>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     attr_set[dev] = true;
   }
   dim3 grid(((long long)a.max_q_len * G + QT - 1) / QT, a.Hkv, a.num_seqs);
-  attn_prefill_kernel<D><<<grid, 128, smem, st>>>(a);
+  attn_prefill_kernel<DK, DV><<<grid, 128, smem, st>>>(a);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
+}
+
+// Each head size rounded up to a compiled one (64, 128 or 256).
+template <int DK>
+static int launch_sized(const UbAttnArgs& a, cudaStream_t st) {
+  if (a.Dv <= 64) return launch_prefill<DK, 64>(a, st);
+  if (a.Dv <= 128) return launch_prefill<DK, 128>(a, st);
+  return launch_prefill<DK, 256>(a, st);
 }
 
 }  // namespace ub
@@ -302,7 +344,8 @@ extern "C" int ub_attn_prefill_last_path() { return g_last_path; }
 extern "C" int ub_attn_prefill(const UbAttnArgs* a, void* stream_v) {
   using namespace ub;
   if (a->num_seqs <= 0 || a->max_q_len <= 0) return 0;
-  if (tc_enabled() && ub_attn_prefill_tc_supported(a)) {
+  const bool plain = a->sinks == nullptr && (a->Dv == 0 || a->Dv == a->D);   // what the tensor-core kernel takes
+  if (plain && tc_enabled() && ub_attn_prefill_tc_supported(a)) {
     g_last_path = 1;
     return ub_attn_prefill_tc(a, stream_v);
   }
@@ -311,9 +354,10 @@ extern "C" int ub_attn_prefill(const UbAttnArgs* a, void* stream_v) {
   if (a->Hq % a->Hkv != 0) return -2;
   if (a->q_stride % 8 != 0) return -3;
   cudaStream_t st = (cudaStream_t)stream_v;
-  switch (a->D) {
-    case 64: return launch_prefill<64>(*a, st);
-    case 128: return launch_prefill<128>(*a, st);
-    default: return -4;
-  }
+  UbAttnArgs b = *a;
+  if (b.Dv <= 0) b.Dv = b.D;
+  if (b.D > 256 || b.Dv > 256 || b.D % 8 != 0 || b.Dv % 8 != 0) return -4;
+  if (b.D <= 64) return launch_sized<64>(b, st);
+  if (b.D <= 128) return launch_sized<128>(b, st);
+  return launch_sized<256>(b, st);
 }

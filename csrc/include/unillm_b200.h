@@ -118,6 +118,32 @@ typedef struct UbNormArgs {
 } UbNormArgs;
 int ub_norm(const UbNormArgs* args, void* stream);
 
+/* ---------------- K1f : GEMM with fp32 operands and 32-bit arithmetic (x, w, bias, residual, out all fp32; grouped and
+   gated forms as ub_gemm_tn, no fused collectives) ---------------- */
+int ub_gemm_f32(const UbGemmArgs* args, void* stream);
+
+/* ---------------- K5r : norms around a 32-bit residual stream (csrc/norm/residual_norm.cu) ----------------
+   Rows of x, y, yx and out are Hp elements apart (Hp = H rounded up to 8); y, yx, weight, bias and out have the element type
+   of the matrix products: bf16, or fp32 with f32 = 1. */
+typedef struct UbResidualNormArgs {
+  const void* y;            /* [T, Hp] sublayer rows, or NULL when yx alone gives them */
+  const void* yx;           /* [slots, Hp] expert rows to be combined onto y, or NULL */
+  const int* row_slot;      /* [T, K] row of yx per choice, negative = none */
+  const float* topk_w;      /* [T, K] */
+  float* x;                 /* residual stream */
+  const int* rows;          /* ub_row_norm: row of x per output row, or NULL */
+  void* out;                /* [T, Hp] */
+  const void* weight;       /* [Hp], zero in the pad columns */
+  const void* bias;         /* [Hp] or NULL */
+  int* err;
+  int T, H, Hp, K, slots, x_rows, kind /* 0 RMS, 1 LayerNorm */, f32;
+  float eps;
+} UbResidualNormArgs;
+int ub_residual_norm(const UbResidualNormArgs* args, void* stream);   /* x += norm(y + sum_k w yx); out = x */
+int ub_row_norm(const UbResidualNormArgs* args, void* stream);        /* out[t] = norm(x[rows[t]]) */
+int ub_embed_residual(const int* ids, const void* table, float* x, void* out, int rows, int Hp, int V, float scale, int f32,
+                      int* err, void* stream);
+
 /* ---------------- K6 : (q/k head RMSNorm) + RoPE + paged KV append ---------------- */
 typedef struct UbRopeArgs {
   void* qkv;                 /* bf16 [T, (Hq + 2 Hkv) * D]; q and k are rotated in place */
@@ -138,6 +164,10 @@ typedef struct UbRopeArgs {
   int interleaved;           /* 0 = half-split pairs (i, i + rd/2); 1 = adjacent pairs (2i, 2i+1) */
   /* Llama-3 style frequency scaling; factor <= 0 disables */
   float l3_factor, l3_low_freq_factor, l3_high_freq_factor, l3_orig_ctx;
+  const float* inv_freq;     /* [rotary_dim / 2] frequencies, or NULL: computed from theta and the scaling above */
+  int Dv;                    /* value head size (0 = D); rows are [Hq * D | Hkv * D | Hkv * Dv] */
+  int norm_dim;              /* elements of a head that the RMS norm averages over (0 = D; less when heads are padded) */
+  int f32;                   /* qkv, caches and norm weights are fp32 */
 } UbRopeArgs;
 int ub_rope_kv_append(const UbRopeArgs* args, void* stream);
 
@@ -169,7 +199,14 @@ typedef struct UbAttnArgs {
      and the warp-MMA decode kernel with splits == 1; other paths answer -7. */
   const void* merge_o;
   const float* merge_lse;
+  /* One learned logit per query head, fp32 [Hq], or NULL: exp(sink) joins the softmax denominator once and has no value.
+     The tensor-core prefill kernel and the warp / persistent decode kernels do not take sinks; the dispatchers choose a
+     kernel that does. */
+  const float* sinks;
+  int Dv;                    /* value head size (0 = D): v_cache [.., Dv], out [T, Hq, Dv], scratch [.., Dv + 2] */
 } UbAttnArgs;
+/* fp32 q, caches and output, 32-bit arithmetic; q_start = NULL: one query per sequence */
+int ub_attn_f32(const UbAttnArgs* args, void* stream);
 int ub_attn_decode(const UbAttnArgs* args, void* stream);
 int ub_attn_prefill(const UbAttnArgs* args, void* stream);
 /* merge two partial attention results (o_a, lse_a) and (o_b, lse_b) -> out; rows = T*Hq, D columns */
@@ -269,9 +306,13 @@ typedef struct UbMoeRouteArgs {
      get row_slot = -1 and no tile; expert_counts/offsets/tiles use local expert indices.  0 = all experts local. */
   int expert_lo;
   int num_local_experts;
+  const void* router_b;     /* [E] added to the logits (router_w mode), or NULL */
+  int x_f32;                /* x is fp32 (the residual stream itself) */
+  int router_f32;           /* router_w and router_b are fp32 */
 } UbMoeRouteArgs;
 int ub_moe_route(const UbMoeRouteArgs* args, void* stream);
 int ub_moe_gather(const void* x, const int* sorted_rows, void* out, int rows, int K, int H, void* stream);
+int ub_moe_gather_f32(const float* x, const int* sorted_rows, float* out, int rows, int K, int H, void* stream);
 int ub_moe_combine(const void* y, const int* row_slot, const float* topk_w, const void* residual, void* out, int T,
                    int K, int H, void* stream);
 /* F6: combine fused with the reduce-scatter: token t's partial row is stored into the receive slot

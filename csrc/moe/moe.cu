@@ -9,7 +9,7 @@
 #include <cuda_runtime.h>
 #include <stdint.h>
 
-#include "../common/ptx.cuh"
+#include "../common/elem.cuh"
 #include "../include/unillm_b200.h"
 
 namespace ub {
@@ -18,26 +18,28 @@ constexpr int MOE_MAX_E = 256;
 constexpr int MOE_MAX_K = 16;
 
 // One CTA of 128 threads per token: logits (from x and the router matrix, or given), top-k, weights.
+// XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.
+template <typename XT, typename WT>
 __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) {
   __shared__ float logit[MOE_MAX_E];
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int E = a.E, K = a.K;
   if (a.router_w != nullptr) {
-    const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x) + (long long)t * a.H;
-    const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.router_w);
+    const XT* x = reinterpret_cast<const XT*>(a.x) + (long long)t * a.H;
+    const WT* w = reinterpret_cast<const WT*>(a.router_w);
     for (int e = warp; e < E; e += 4) {
-      const __nv_bfloat16* we = w + (long long)e * a.H;
+      const WT* we = w + (long long)e * a.H;
       float acc = 0.f;
       for (int h = lane * 8; h < a.H; h += 256) {
-        const uint4 xv = *reinterpret_cast<const uint4*>(x + h);
-        const uint4 wv = __ldg(reinterpret_cast<const uint4*>(we + h));
-        const uint32_t* xs = reinterpret_cast<const uint32_t*>(&xv);
-        const uint32_t* ws = reinterpret_cast<const uint32_t*>(&wv);
+        float xs[8], ws[8];
+        load8(x + h, xs);
+        load8(we + h, ws);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) acc += bf16_lo(xs[j]) * bf16_lo(ws[j]) + bf16_hi(xs[j]) * bf16_hi(ws[j]);
+        for (int j = 0; j < 8; ++j) acc = fmaf(xs[j], ws[j], acc);
       }
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
+      if (a.router_b != nullptr) acc += (float)reinterpret_cast<const WT*>(a.router_b)[e];
       // the reference model keeps router logits in the activation dtype: round like a bf16 linear layer would
       if (lane == 0) logit[e] = a.round_logits_bf16 ? __bfloat162float(__float2bfloat16(acc)) : acc;
     }
@@ -54,7 +56,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
   float den = 0.f;
-  for (int e = lane; e < E; e += 32) den += __expf(logit[e] - mx);
+  for (int e = lane; e < E; e += 32) den += expf(logit[e] - mx);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
   uint32_t taken = 0;  // bit j: expert lane + 32*j already selected
@@ -80,7 +82,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
   }
   if (lane == 0) {
     float s = 0.f;
-    for (int k = 0; k < K; ++k) { sel_l[k] = __expf(sel_l[k] - mx); s += sel_l[k]; }
+    for (int k = 0; k < K; ++k) { sel_l[k] = expf(sel_l[k] - mx); s += sel_l[k]; }
     const float inv = a.norm_topk ? 1.f / s : 1.f / den;
     for (int k = 0; k < K; ++k) {
       a.topk_ids[(long long)t * K + k] = sel_e[k];
@@ -132,10 +134,11 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const UbMoeRouteArgs a) 
   for (int i = off[E] + threadIdx.x; i < n; i += blockDim.x) a.sorted_rows[i] = -1;   // unused tail
 }
 
-// out[slot, :] = x[sorted_rows[slot] / K, :]
-__global__ void __launch_bounds__(256) moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ sorted_rows,
-                                                         __nv_bfloat16* __restrict__ out, int rows, int K, int H) {
-  const int vec = H / 8;
+// out[slot, :] = x[sorted_rows[slot] / K, :]; V 16-byte vectors per 8 bf16 / 4 fp32 elements
+template <typename T>
+__global__ void __launch_bounds__(256) moe_gather_kernel(const T* __restrict__ x, const int* __restrict__ sorted_rows,
+                                                         T* __restrict__ out, int rows, int K, int H) {
+  const int vec = H / (16 / (int)sizeof(T));
   for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < (long long)rows * vec;
        i += (long long)gridDim.x * blockDim.x) {
     const int slot = int(i / vec), c = int(i % vec);
@@ -380,8 +383,21 @@ extern "C" int ub_moe_route(const UbMoeRouteArgs* a, void* stream_v) {
   if (a->tiles != nullptr && (a->tile_tokens <= 0 || a->max_tiles <= 0)) return -4;
   UbMoeRouteArgs b = *a;
   if (b.weight_scale == 0.f) b.weight_scale = 1.f;
-  ub::moe_route_kernel<<<a->T, 128, 0, st>>>(b);
+  if (b.router_w != nullptr && b.x_f32 && b.router_f32) ub::moe_route_kernel<float, float><<<a->T, 128, 0, st>>>(b);
+  else if (b.router_w != nullptr && b.x_f32) ub::moe_route_kernel<float, __nv_bfloat16><<<a->T, 128, 0, st>>>(b);
+  else if (b.router_w != nullptr && b.router_f32) ub::moe_route_kernel<__nv_bfloat16, float><<<a->T, 128, 0, st>>>(b);
+  else ub::moe_route_kernel<__nv_bfloat16, __nv_bfloat16><<<a->T, 128, 0, st>>>(b);
   ub::moe_sort_kernel<<<1, 1024, 0, st>>>(b);
+  cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -(int)e;
+}
+
+extern "C" int ub_moe_gather_f32(const float* x, const int* sorted_rows, float* out, int rows, int K, int H, void* stream_v) {
+  if (rows <= 0) return 0;
+  if (H % 4 != 0) return -2;
+  const long long work = (long long)rows * (H / 4);
+  int blocks = int((work + 255) / 256 < 148 * 8 ? (work + 255) / 256 : 148 * 8);
+  ub::moe_gather_kernel<float><<<blocks, 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(x, sorted_rows, out, rows, K, H);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }
@@ -392,7 +408,7 @@ extern "C" int ub_moe_gather(const void* x, const int* sorted_rows, void* out, i
   const long long work = (long long)rows * (H / 8);
   int blocks = int((work + 255) / 256);
   if (blocks > 148 * 8) blocks = 148 * 8;
-  ub::moe_gather_kernel<<<blocks, 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(
+  ub::moe_gather_kernel<__nv_bfloat16><<<blocks, 256, 0, reinterpret_cast<cudaStream_t>(stream_v)>>>(
       reinterpret_cast<const __nv_bfloat16*>(x), sorted_rows, reinterpret_cast<__nv_bfloat16*>(out), rows, K, H);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;

@@ -4,12 +4,14 @@
 // is a contiguous block_size x D tile that attention kernels can fetch with bulk copies.
 // One CTA per token, one warp per head (round-robin).  cos/sin are computed on the fly from the
 // position (no table in HBM); partial rotary, linear position scaling and Llama-3 frequency
-// scaling are parameters.  Slots are bounds-checked: a bad slot sets the error word and is skipped.
+// scaling are parameters (or a table of frequencies).  Heads with a norm, interleaved pairs or a value size of its own go
+// through a second kernel in which a few lanes own a head, eight elements each; it also has a 32-bit form.
+// Slots are bounds-checked: a bad slot sets the error word and is skipped.
 //
 // Replaces in the reference: apply_rope / apply_rope_with_offset (crates/runtime/src/models_v2/
 // llama.rs:761-883), LayerKVCache::append (crates/runtime/src/kv_cache.rs:91-134) and the scalar /
 // NEON apply_rope (crates/runtime/src/simd/arch/scalar.rs:112-153).
-#include "../common/ptx.cuh"
+#include "../common/elem.cuh"
 #include "../include/unillm_b200.h"
 
 namespace ub {
@@ -182,11 +184,121 @@ __global__ void __launch_bounds__(128) rope_kv_append_kernel(const UbRopeArgs a)
   }
 }
 
+// LPH lanes per head (a power of two, LPH * 8 >= D), eight consecutive elements of the head per lane: the norm is a shuffle
+// reduction among the lanes of the head, interleaved pairs are lane-local, half-split pairs come from the lane that holds
+// the other half.  K goes to the cache (and back into the row only when there is no cache), V is copied to the cache.
+template <typename T, int LPH>
+__global__ void __launch_bounds__(128) head_norm_rope_kernel(const UbRopeArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ float cs[];                   // cos [half] then sin [half]
+  const int t = blockIdx.x, D = a.D, Dv = a.Dv, half = a.rotary_dim / 2;
+  const float pos = (float)a.positions[t] * a.pos_scale;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * (a.inv_freq != nullptr ? a.inv_freq[i] : rope_inv_freq(i, a)), &s, &c);
+    cs[i] = c;
+    cs[half + i] = s;
+  }
+  __syncthreads();
+  const long long slot = a.slot_mapping != nullptr ? (long long)a.slot_mapping[t] : -1;
+  bool slot_ok = slot >= 0;
+  if (slot >= a.num_slots) {
+    slot_ok = false;
+    if (threadIdx.x == 0) set_err(a.err, ERR_BOUNDS, t);
+  }
+  const long long blk = slot_ok ? slot / a.block_size : 0, off = slot_ok ? slot % a.block_size : 0;
+  T* row = reinterpret_cast<T*>(a.qkv) + (long long)t * ((long long)(a.Hq + a.Hkv) * D + (long long)a.Hkv * Dv);
+  const int grp = threadIdx.x / LPH, c = threadIdx.x % LPH, ngrp = 128 / LPH;
+  const int nrot = a.Hq + a.Hkv;
+  const bool have = c * 8 < D;                    // the last lanes of a group may own nothing
+  const float inv_n = 1.f / (float)(a.norm_dim > 0 ? a.norm_dim : D);
+  const int hc = half / 8;                        // half-split form: chunks per half
+  for (int h0 = 0; h0 < nrot; h0 += ngrp) {
+    const int h = h0 + grp;
+    const bool ok = h < nrot && have;
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = 0.f;
+    if (ok) load8(row + (long long)h * D + c * 8, v);
+    const T* nw = reinterpret_cast<const T*>(h < a.Hq ? a.q_norm_w : a.k_norm_w);
+    if (a.q_norm_w != nullptr || a.k_norm_w != nullptr) {
+      float ss = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
+#pragma unroll
+      for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+      if (ok && nw != nullptr) {
+        const float r = 1.f / sqrtf(ss * inv_n + a.norm_eps);
+        float w[8];
+        load8(nw + c * 8, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * r * w[e];
+      }
+    }
+    if (a.interleaved) {
+#pragma unroll
+      for (int e = 0; e < 8; e += 2) {
+        const int i = c * 4 + e / 2;
+        if (i < half) {
+          const float co = cs[i], si = cs[half + i], x0 = v[e], x1 = v[e + 1];
+          v[e] = x0 * co - x1 * si;
+          v[e + 1] = x1 * co + x0 * si;
+        }
+      }
+    } else if (half > 0) {                        // half % 8 == 0 (host check)
+      const int partner = c < hc ? c + hc : (c < 2 * hc ? c - hc : c);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float other = __shfl_sync(0xffffffffu, v[e], partner, LPH);
+        if (c < hc) v[e] = v[e] * cs[c * 8 + e] - other * cs[half + c * 8 + e];
+        else if (c < 2 * hc) v[e] = v[e] * cs[(c - hc) * 8 + e] + other * cs[half + (c - hc) * 8 + e];
+      }
+    }
+    if (!ok) continue;
+    if (h < a.Hq || a.k_cache == nullptr) store8(row + (long long)h * D + c * 8, v);
+    if (h >= a.Hq && slot_ok && a.k_cache != nullptr)
+      store8(reinterpret_cast<T*>(a.k_cache) + ((blk * a.Hkv + (h - a.Hq)) * a.block_size + off) * D + c * 8, v);
+  }
+  if (slot_ok && a.v_cache != nullptr) {
+    const int cpr = Dv / 8;
+    const T* vr = row + (long long)nrot * D;
+    for (int it = threadIdx.x; it < a.Hkv * cpr; it += 128) {
+      const int hk = it / cpr, ch = it - hk * cpr;
+      float v[8];
+      load8(vr + (long long)hk * Dv + ch * 8, v);
+      store8(reinterpret_cast<T*>(a.v_cache) + ((blk * a.Hkv + hk) * a.block_size + off) * Dv + ch * 8, v);
+    }
+  }
+}
+
+template <typename T>
+static cudaError_t launch_head_norm_rope(const UbRopeArgs& a, cudaStream_t st) {
+  const size_t smem = (size_t)(a.rotary_dim > 0 ? a.rotary_dim : 1) * sizeof(float);
+  const dim3 grid(a.T), block(128);
+  if (a.D <= 32) return launch_pdl(head_norm_rope_kernel<T, 4>, grid, block, smem, st, a);
+  if (a.D <= 64) return launch_pdl(head_norm_rope_kernel<T, 8>, grid, block, smem, st, a);
+  if (a.D <= 128) return launch_pdl(head_norm_rope_kernel<T, 16>, grid, block, smem, st, a);
+  return launch_pdl(head_norm_rope_kernel<T, 32>, grid, block, smem, st, a);
+}
+
 }  // namespace ub
 
 extern "C" int ub_rope_kv_append(const UbRopeArgs* a, void* stream_v) {
   if (a->T <= 0) return 0;
   if (a->D > 512 || (a->rotary_dim & 1) || a->rotary_dim > a->D) return -2;
+  const int Dv = a->Dv > 0 ? a->Dv : a->D;
+  const bool general = a->f32 || Dv != a->D || a->inv_freq != nullptr || (a->norm_dim > 0 && a->norm_dim != a->D);
+  const bool wide_ok = a->D % 8 == 0 && Dv % 8 == 0 && a->D <= 256 && (a->interleaved || a->rotary_dim % 16 == 0);
+  if (general && !wide_ok) return -4;
+  if (wide_ok && (general || a->interleaved || a->q_norm_w != nullptr || a->k_norm_w != nullptr)) {
+    UbRopeArgs b = *a;
+    b.Dv = Dv;
+    cudaError_t e = b.f32 ? ub::launch_head_norm_rope<float>(b, (cudaStream_t)stream_v)
+                          : ub::launch_head_norm_rope<__nv_bfloat16>(b, (cudaStream_t)stream_v);
+    if (e == cudaSuccess) e = cudaGetLastError();
+    return e == cudaSuccess ? 0 : -(int)e;
+  }
   ub::launch_pdl(ub::rope_kv_append_kernel, dim3(a->T), dim3(128), (4 * a->D + a->rotary_dim) * sizeof(float), (cudaStream_t)stream_v, *a);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;

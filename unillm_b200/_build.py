@@ -1,10 +1,14 @@
 """In-tree build of the native libraries.
 
-Two shared objects are produced next to this file's package, so that they travel with the source
+The shared objects are produced next to this file's package, so that they travel with the source
 tree and are visible to whatever inspects the process's loaded libraries:
 
-* ``unillm_b200/_native/libunillm_b200_cuda.so``  -- every CUDA kernel (``csrc/**/*.cu``), compiled
-  with ``nvcc -gencode arch=compute_100a,code=sm_100a`` (Blackwell only; no other arch is built).
+* ``unillm_b200/_native/libunillm_b200_cuda.so``  -- the CUDA kernels that serving a decoder on one GPU
+  launches (``csrc/{gemm,attn,norm,norm_rope,moe,eltwise,sample,kv}``), compiled with
+  ``nvcc -gencode arch=compute_100a,code=sm_100a`` (Blackwell only; no other arch is built).
+* ``unillm_b200/_native/libunillm_b200_cuda_more.so``  -- the rest of ``csrc/**/*.cu``: peer-memory
+  collectives, recurrences, block-quantised matrices, probes.  A process that needs none of them neither
+  builds nor loads it.
 * ``unillm_b200/_native/libunillm_b200_host.so``  -- host-side C++ runtime (``csrc/**/*.cpp``): KV block
   pool, radix tree, GGUF block (de)quantisation oracle, scheduler core.
 
@@ -62,12 +66,20 @@ def nvcc_path() -> str:
     return p
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> Path:
+SERVING_DIRS = ("attn", "eltwise", "gemm", "kv", "moe", "norm", "norm_rope", "sample")
+CUDA_LIBS = {"serving": "libunillm_b200_cuda.so", "more": "libunillm_b200_cuda_more.so"}
+
+
+def cuda_sources(part: str) -> list:
+    return [s for s in sorted(CSRC.rglob("*.cu")) if (s.relative_to(CSRC).parts[0] in SERVING_DIRS) == (part == "serving")]
+
+
+def build_cuda(force: bool = False, verbose: bool = False, part: str = "serving") -> Path:
     OBJ.mkdir(parents=True, exist_ok=True)
     nvcc = nvcc_path()
-    srcs = sorted(CSRC.rglob("*.cu"))
+    srcs = cuda_sources(part)
     hdr_m = _newest_header_mtime()
-    lib = OUT / "libunillm_b200_cuda.so"
+    lib = OUT / CUDA_LIBS[part]
     jobs = []
     objs = []
     for s in srcs:
@@ -123,7 +135,8 @@ def build_host(force: bool = False, verbose: bool = False) -> Path:
 
 
 def build_all(force: bool = False, verbose: bool = False) -> None:
-    build_cuda(force, verbose)
+    for part in CUDA_LIBS:
+        build_cuda(force, verbose, part)
     build_host(force, verbose)
 
 

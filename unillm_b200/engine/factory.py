@@ -32,18 +32,24 @@ def why_not_gpu(model) -> Optional[str]:
         return "post-LN / projected-embedding topologies run on the whole-model path"
     if getattr(model, "reference_quirks", False):
         return "reference_quirks changes the normalisation; the kernels implement the published architecture"
-    if s.hidden_size % 8 or s.head_dim % 8:
+    if s.layers is None and (s.hidden_size % 8 or s.head_dim % 8):
         return "hidden size and head size must be multiples of 8 (16-byte rows for the TMA copies)"
+    for i in range(s.num_layers):
+        ls = s.layer(i)
+        if s.layers is not None and (max(ls.head_dim, ls.v_head_dim) > 256 or s.hidden_size > 16384):
+            return f"layer {i}: head sizes above 256 or a width above 16384"
+        if ls.moe is not None and (ls.moe.num_experts > 256 or ls.moe.top_k > 16):
+            return f"layer {i}: more than 256 experts or more than 16 per token"
     return None
 
 
-def _auto_num_blocks(spec, weights, block_size: int, device, gpu_memory_fraction: float, max_model_len: int,
+def _auto_num_blocks(weights, block_size: int, device, gpu_memory_fraction: float, max_model_len: int,
                      max_num_seqs: int) -> int:
     """KV blocks that fit in ``gpu_memory_fraction`` of the device after the weights, capped by what the sequence
     limits can ever use."""
     free, total = torch.cuda.mem_get_info(device)
     budget = int(total * gpu_memory_fraction) - (total - free)
-    per_block = 2 * spec.num_layers * weights.hkv * block_size * spec.head_dim * 2
+    per_block = weights.kv_bytes_per_token() * block_size
     fit = max(budget // max(per_block, 1), 0)
     useful = max_num_seqs * (-(-max_model_len // block_size) + 1) + 64
     n = int(min(fit, useful))
@@ -57,11 +63,13 @@ def build_engine(model, *, device="cuda", max_num_seqs: int = 64, max_num_batche
                  max_model_len: Optional[int] = None, block_size: int = 16, num_blocks: Optional[int] = None,
                  gpu_memory_fraction: float = 0.9, enable_prefix_caching: bool = True, async_scheduling: bool = False,
                  use_cuda_graphs: bool = True, eos_token_id: Optional[int] = None, rank: int = 0, world: int = 1,
-                 tp=None, quantize: Optional[str] = None):
+                 tp=None, quantize: Optional[str] = None, dtype: torch.dtype = torch.bfloat16):
     """An ``LLMEngine`` that runs ``model`` on the hand-written kernels of ``device``.
 
     ``quantize`` ("q4_k", "q8_0", "q4_0"): keep the projection matrices block-quantised on the device (4.5 - 8.5 bits
     per weight, see ``RunnerWeights.quantize``) instead of bf16.
+
+    ``dtype=torch.float32``: weights, caches and all arithmetic in 32 bits (models with a 32-bit residual stream).
 
     Raises ``UnsupportedOperation`` (with the reason) when the model cannot take that path; see ``why_not_gpu``."""
     from .llm_engine import LLMEngine
@@ -76,11 +84,11 @@ def build_engine(model, *, device="cuda", max_num_seqs: int = 64, max_num_batche
     spec = model.spec
     if max_model_len is None:
         max_model_len = min(spec.max_position_embeddings, 8192)
-    weights = RunnerWeights(spec, model.p, dev, rank, world)
+    weights = RunnerWeights(spec, model.p, dev, rank, world, dtype=dtype)
     if quantize:
         weights.quantize(quantize)
     if num_blocks is None:
-        num_blocks = _auto_num_blocks(spec, weights, block_size, dev, gpu_memory_fraction, max_model_len, max_num_seqs)
+        num_blocks = _auto_num_blocks(weights, block_size, dev, gpu_memory_fraction, max_model_len, max_num_seqs)
     runner = GpuModelRunner(spec, weights, num_blocks=num_blocks, block_size=block_size, max_num_seqs=max_num_seqs,
                             max_num_batched_tokens=max_num_batched_tokens, max_model_len=max_model_len, tp=tp, device=dev,
                             use_cuda_graphs=use_cuda_graphs)

@@ -125,6 +125,7 @@ class LLMEngine:
         self.waiting: Deque[Sequence] = deque()
         self.running: List[Sequence] = []
         self.seqs: Dict[int, Sequence] = {}
+        self.scored: Dict[object, Sequence] = {}    # sequences of ``score_step``, by the caller's key
         self._next_id = 0
         self.stats = EngineStats()
         self.async_scheduling = async_scheduling
@@ -307,26 +308,52 @@ class LLMEngine:
             self._publish(s, s.num_computed + n)
         if not decode and not chunks:
             return None, []
+        batch = self._build_batch(decode, chunks)
+        plan: List[Tuple[Sequence, int, bool]] = [(s, 1, True) for s in decode]
+        batch.sample_rows = list(range(len(decode)))
+        row = len(decode)
+        for s, n in chunks:
+            row += n
+            done = s.num_computed + n >= s.total_len
+            if done:
+                batch.sample_rows.append(row - 1)
+            plan.append((s, n, done))
+        shared = self._shared_prefix(decode) if len(decode) >= 8 else 0
+        # prefill chunks can join the shared-prefix pass when they start at or after the prefix and reuse its blocks
+        nshared = shared // bs
+        pfx_ok = bool(chunks) and shared > 0 and all(
+            s.num_computed >= shared and s.blocks[:nshared] == decode[0].blocks[:nshared] for s, _ in chunks)
+        sampled = [s for s, _, smp in plan if smp]
+        greedy = all(s.params.greedy for s in sampled)
+        batch.shared_prefix_len, batch.prefill_shares_prefix = shared, pfx_ok
+        batch.seed, batch.step = self.seed, self.stats.steps
+        if not greedy:
+            batch.temperature = [s.params.temperature for s in sampled]
+            batch.top_p = [s.params.top_p for s in sampled]
+            batch.top_k = [s.params.top_k or 0 for s in sampled]
+        return batch, plan
+
+    def _build_batch(self, decode: List[Sequence], chunks: List[Tuple[Sequence, int]]) -> StepBatch:
+        """Packs one decode token per sequence of ``decode`` and the next ``n`` tokens of every (sequence, n) of ``chunks``;
+        the blocks for them are already held."""
+        bs = self.block_size
         token_ids: List[int] = []
         positions: List[int] = []
         slots: List[int] = []
         seq_lens: List[int] = []
         tables: List[List[int]] = []
-        sample_rows: List[int] = []
-        plan: List[Tuple[Sequence, int, bool]] = []
         token_src: Optional[List[int]] = None
         if decode:
-            positions = [len(s.prompt_ids) + len(s.output_ids) - 1 for s in decode]
+            positions = [s.total_len - 1 for s in decode]
+            last = [s.output_ids[-1] if s.output_ids else s.prompt_ids[-1] for s in decode]
             if self._inflight is not None:
                 token_src = [s.pending_src for s in decode]
-                token_ids = [0 if s.pending_src >= 0 else s.output_ids[-1] for s in decode]
+                token_ids = [0 if s.pending_src >= 0 else t for s, t in zip(decode, last)]
             else:
-                token_ids = [s.output_ids[-1] for s in decode]
+                token_ids = last
             slots = [s.blocks[p // bs] * bs + p % bs for s, p in zip(decode, positions)]
             seq_lens = [p + 1 for p in positions]
             tables = [s.blocks_array() for s in decode]
-            sample_rows = list(range(len(decode)))
-            plan = [(s, 1, True) for s in decode]
         q_lens: List[int] = []
         for s, n in chunks:
             a, b = s.num_computed, s.num_computed + n
@@ -338,27 +365,10 @@ class LLMEngine:
             positions.extend(range(a, b))
             blk = s.blocks
             slots.extend([blk[p // bs] * bs + p % bs for p in range(a, b)])
-            seq_lens.append(s.num_computed + n)
+            seq_lens.append(b)
             tables.append(s.blocks_array())
             q_lens.append(n)
-            done = s.num_computed + n >= s.total_len
-            if done:
-                sample_rows.append(len(token_ids) - 1)
-            plan.append((s, n, done))
-        shared = self._shared_prefix(decode) if len(decode) >= 8 else 0
-        # prefill chunks can join the shared-prefix pass when they start at or after the prefix and reuse its blocks
-        nshared = shared // bs
-        pfx_ok = bool(chunks) and shared > 0 and all(
-            s.num_computed >= shared and s.blocks[:nshared] == decode[0].blocks[:nshared] for s, _ in chunks)
-        sampled = [s for s, _, smp in plan if smp]
-        greedy = all(s.params.greedy for s in sampled)
-        batch = StepBatch(token_ids, positions, slots, len(decode), seq_lens, tables, q_lens, sample_rows, shared,
-                          prefill_shares_prefix=pfx_ok, seed=self.seed, step=self.stats.steps, token_src=token_src)
-        if not greedy:
-            batch.temperature = [s.params.temperature for s in sampled]
-            batch.top_p = [s.params.top_p for s in sampled]
-            batch.top_k = [s.params.top_k or 0 for s in sampled]
-        return batch, plan
+        return StepBatch(token_ids, positions, slots, len(decode), seq_lens, tables, q_lens, token_src=token_src)
 
     def _ensure_blocks_no_preempt(self, s: Sequence, upto_tokens: int) -> bool:
         need = (upto_tokens + self.block_size - 1) // self.block_size - len(s.blocks)
@@ -558,6 +568,67 @@ class LLMEngine:
                 self.stats.finished += 1
             outs.append(StepOutput(s.seq_id, tok, reason is not None, reason))
         return outs
+
+    # ------------------------------------------------------------------------------------------
+    # scoring: the caller brings every token
+    # ------------------------------------------------------------------------------------------
+    def score_step(self, entries: Sequence[Tuple[object, Sequence[int], Sequence[int]]], end: Sequence[object] = ()):
+        """One engine step over token ids that the caller gives: ``entries`` is a list of ``(key, next tokens, wanted
+        places among them)``.  A key seen for the first time opens a sequence; later entries of the key continue it from
+        the cache.  All entries run as one batch through the runner's step function -- entries with a single token beside
+        the decode rows, longer ones as prompt portions.  Returns the fp32 logits [wanted, vocab] in the order of the
+        entries and of their wanted places (on the runner's device).  Sequences named in ``end`` give their blocks back
+        after the step.  Scored sequences are outside the request queue and the prefix cache; nothing is sampled."""
+        n_tokens = sum(len(t) for _, t, _ in entries)
+        if n_tokens > self.max_tokens:
+            raise InvalidInput(f"step of {n_tokens} tokens exceeds max_num_batched_tokens {self.max_tokens}")
+        if len({k for k, _, _ in entries}) != len(entries):
+            raise InvalidInput("a sequence appears twice in a step")
+        for key, toks, want in entries:
+            s = self.scored.get(key)
+            if len(toks) == 0 or any(not 0 <= w < len(toks) for w in want):
+                raise InvalidInput(f"sequence {key!r}: no tokens, or a wanted place outside them")
+            if (s.total_len if s is not None else 0) + len(toks) > self.max_model_len:
+                raise InvalidInput(f"sequence {key!r} exceeds max_model_len {self.max_model_len}")
+        if len(self.running) + len(set(self.scored) | {k for k, _, _ in entries}) > self.max_num_seqs:
+            raise InvalidInput(f"more than {self.max_num_seqs} live sequences")
+        self._late.extend(self._drain())
+        decode: List[Sequence] = []
+        chunks: List[Tuple[Sequence, int]] = []
+        for key, toks, _ in entries:
+            s = self.scored.get(key)
+            if s is None:
+                s = self.scored[key] = Sequence(-1, [], SamplingParams(), status=RUNNING)
+            s.prompt_ids.extend(int(t) for t in toks)
+            if not self._ensure_blocks_no_preempt(s, s.total_len):
+                raise MemoryError_(f"no KV blocks left for sequence {key!r}")
+            if len(toks) == 1:
+                decode.append(s)
+            else:
+                chunks.append((s, len(toks)))
+        if not entries:
+            logits = None
+        else:
+            batch = self._build_batch(decode, chunks)
+            first = {id(s): i for i, s in enumerate(decode)}        # first row of each sequence in the batch
+            row = len(decode)
+            for s, n in chunks:
+                first[id(s)] = row
+                row += n
+            batch.sample_rows = [first[id(self.scored[k])] + w for k, _, want in entries for w in want]
+            logits = self.runner.forward_logits(batch)
+            for s in decode + [s for s, _ in chunks]:
+                s.num_computed = s.total_len
+            self.stats.steps += 1
+            self.stats.decode_tokens += len(decode)
+            self.stats.prefill_tokens += n_tokens - len(decode)
+        for key in end:
+            s = self.scored.pop(key, None)
+            if s is None:
+                raise InvalidInput(f"unknown sequence {key!r}")
+            self._release(s, publish=False)
+            s.status = FINISHED
+        return logits
 
     def run_to_completion(self, max_steps: int = 1 << 30) -> Dict[int, List[int]]:
         n = 0

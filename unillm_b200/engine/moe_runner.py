@@ -24,18 +24,16 @@ import torch
 from ..ops import cuda_ops as K
 
 
-def moe_partial(runner, i: int, h: torch.Tensor, residual=None, combine_rs=None) -> torch.Tensor:
-    """MoE output for hidden rows ``h`` ([T, H]).  With ``residual`` (single rank only) it is added in the combine.
-    ``combine_rs`` (peer pointers as for ``gemm_tn(rs=...)``) makes the combine kernel push its partial rows to the
-    ranks that own them instead of returning them."""
-    s, t = runner.spec, runner.w.t
-    m = s.moe
+def _experts(runner, i: int, h: torch.Tensor, router_x: torch.Tensor):
+    """Routing of ``router_x`` and the experts' outputs for ``h``: (rows in expert order, routing)."""
+    t = runner.w.t
+    m = runner.layers[i].moe
     L = f"layers.{i}."
     T = h.shape[0]
     with runner._prof("moe_route"):
-        r = K.moe_route(h, t[L + "router"], m.top_k, norm_topk=m.normalize_topk, round_logits_bf16=False,
+        r = K.moe_route(router_x, t[L + "router"], m.top_k, norm_topk=m.normalize_topk, round_logits_bf16=False,
                         expert_lo=runner.w.expert_lo if runner.w.ep else 0,
-                        num_local_experts=runner.w.experts_local if runner.w.ep else 0)
+                        num_local_experts=runner.w.experts_local if runner.w.ep else 0, router_b=t.get(L + "router_b"))
         xs = K.moe_gather(h, r)
     runner.launches += 3
     gu, dn = t[L + "experts_gate_up"], t[L + "experts_down"]
@@ -46,11 +44,44 @@ def moe_partial(runner, i: int, h: torch.Tensor, residual=None, combine_rs=None)
             a = K.grouped_gemm(xs, gu, r, act=m.act)
     with runner._prof(f"moe_down[{T * m.top_k}x{dn.shape[1]}x{dn.shape[2]}]"):
         y = K.grouped_gemm(a, dn, r)
+    runner.launches += 2
+    return y, r
+
+
+def _shared_expert(runner, i: int, h: torch.Tensor, residual=None) -> torch.Tensor:
+    """The always-on expert's rows (+ residual)."""
+    t = runner.w.t
+    m = runner.layers[i].moe
+    w = t[f"layers.{i}.shared_gate_up"]
+    sh = runner._gemm(h, w, dual_rows=w.shape[0] // 2 if m.gated else 0, act=m.act)
+    return runner._gemm(sh, t[f"layers.{i}.shared_down"], residual=residual)
+
+
+def moe_branch(runner, i: int, h: torch.Tensor, router_x: torch.Tensor):
+    """The mixture's output for a layer that normalises it before the residual add: ``(base rows or None, expert rows or
+    None, routing)``, to be summed by the norm kernel.  ``router_x``: what the router reads (the 32-bit stream)."""
+    m = runner.layers[i].moe
+    y, r = _experts(runner, i, h, router_x)
+    base = _shared_expert(runner, i, h) if m.num_shared_experts else None
+    if runner.tp.world == 1:
+        return base, y, r
+    out = K.moe_combine(y, r, residual=base)          # partial rows of this rank's share of every expert
+    runner.tp.all_reduce(out)
+    runner.launches += 2
+    return out, None, None
+
+
+def moe_partial(runner, i: int, h: torch.Tensor, residual=None, combine_rs=None) -> torch.Tensor:
+    """MoE output for hidden rows ``h`` ([T, H]).  With ``residual`` (single rank only) it is added in the combine.
+    ``combine_rs`` (peer pointers as for ``gemm_tn(rs=...)``) makes the combine kernel push its partial rows to the
+    ranks that own them instead of returning them."""
+    t = runner.w.t
+    m = runner.layers[i].moe
+    L = f"layers.{i}."
+    y, r = _experts(runner, i, h, h)
     base = residual
     if m.num_shared_experts:
-        Is = t[L + "shared_gate_up"].shape[0] // 2
-        sh = runner._gemm(h, t[L + "shared_gate_up"], dual_rows=Is, act=m.act)
-        base = runner._gemm(sh, t[L + "shared_down"], residual=residual)
+        base = _shared_expert(runner, i, h, residual)
     if m.dense_parallel and (L + "w_down") in t:
         d = runner._mlp_noresid(i, h, dense_only=True)
         base = d if base is None else K.add(base, d)
@@ -63,7 +94,7 @@ def moe_partial(runner, i: int, h: torch.Tensor, residual=None, combine_rs=None)
             out = None
         else:
             out = K.moe_combine(y, r, residual=base)
-    runner.launches += 3
+    runner.launches += 1
     return out
 
 

@@ -34,7 +34,7 @@ import torch
 
 from ..models.spec import DecoderSpec
 from ..ops import cuda_ops as K
-from ..precompute import alibi_slopes
+from ..precompute import alibi_slopes, rope_inv_freq
 from ..types import InvalidInput, UnsupportedOperation
 
 
@@ -106,52 +106,95 @@ class QWeight:
 QUANT_NAMES = {"q4_0": 2, "q8_0": 8, "q4_k": 12}
 
 
+def _round8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def _pad(t: torch.Tensor, dim: int, size: int) -> torch.Tensor:
+    """``t`` with zeros appended along ``dim`` up to ``size`` entries."""
+    n = size - t.shape[dim]
+    if n == 0:
+        return t
+    shape = list(t.shape)
+    shape[dim] = n
+    return torch.cat([t, t.new_zeros(shape)], dim)
+
+
+@dataclass(frozen=True)
+class KernelHeads:
+    """One layer's attention heads as this rank's kernels see them: head sizes are rounded up to multiples of 8 (16-byte
+    rows); the pad entries of the projections are zero, so they add nothing to scores or outputs."""
+
+    hq: int
+    hkv: int
+    kv_lo: int
+    dk: int
+    dv: int
+    own_kv: bool
+
+    @property
+    def qkv_rows(self) -> int:
+        return self.hq * self.dk + (self.hkv * (self.dk + self.dv) if self.own_kv else 0)
+
+
 class RunnerWeights:
-    """Device weights of one rank in kernel layout (bf16, fused QKV / gate-up, TP-sharded)."""
+    """Device weights of one rank in kernel layout (fused QKV / gate-up, TP-sharded), bf16 or fp32.  For per-layer specs, row
+    sizes that are not multiples of 8 (model width, head sizes, feed-forward widths) are zero-padded to the next one."""
 
     def __init__(self, spec: DecoderSpec, params: Dict[str, torch.Tensor], device, rank: int = 0, world: int = 1,
-                 expert_parallel: bool = False):
-        self.spec, self.rank, self.world = spec, rank, world
+                 expert_parallel: bool = False, dtype: torch.dtype = torch.bfloat16):
+        self._init_layout(spec, rank, world, expert_parallel, dtype)
         s = spec
-        self._set_ep(expert_parallel)
-        if s.num_heads % world != 0:
-            raise InvalidInput(f"{s.num_heads} heads not divisible by tensor parallel size {world}")
-        self.hq = s.num_heads // world
-        self.hkv, self.kv_lo = self.kv_layout(s.num_kv_heads, rank, world)
-        D = s.head_dim
-
-        def kv_rows(t):
-            """Rows (or elements) of this rank's KV heads inside a [num_kv_heads * D, ...] tensor."""
-            return t[self.kv_lo * D:(self.kv_lo + self.hkv) * D]
+        H = self.width
 
         def dev(t):
-            return t.to(device=device, dtype=torch.bfloat16).contiguous()
+            return t.to(device=device, dtype=dtype).contiguous()
+
+        def heads(t, n, d, dp, lo, cnt):
+            """Rows (or elements) of heads [lo, lo + cnt) of a [n * d, ...] tensor, every head padded to dp rows."""
+            t = t.reshape(n, d, *t.shape[1:])[lo:lo + cnt]
+            t = _pad(t, 1, dp)
+            return t.reshape(cnt * dp, *t.shape[2:])
 
         self.t: Dict[str, torch.Tensor] = {}
         p = params
-        self.t["embed"] = dev(p["embed"])
-        for n in ("pos_embed", "embed_norm.w", "embed_norm.b", "final_norm.w", "final_norm.b", "project_in", "project_out"):
+        self.t["embed"] = dev(_pad(p["embed"], 1, H))
+        for n in ("embed_norm.w", "embed_norm.b", "final_norm.w", "final_norm.b"):
+            if n in p:
+                self.t[n] = dev(_pad(p[n], 0, H))
+        for n in ("pos_embed", "project_in", "project_out"):
             if n in p:
                 self.t[n] = dev(p[n])
         lm = p["embed"] if s.tie_embeddings else p["lm_head"]
-        if s.vocab_size % world != 0:
-            raise InvalidInput(f"vocab {s.vocab_size} not divisible by tensor parallel size {world}")
-        self.vocab_shard = s.vocab_size // world
-        self.t["lm_head"] = dev(shard_rows(lm, rank, world)) if (world > 1 or not s.tie_embeddings) else self.t["embed"]
+        self.t["lm_head"] = dev(_pad(shard_rows(lm, rank, world), 1, H)) if (world > 1 or not s.tie_embeddings) \
+            else self.t["embed"]
         if "lm_head_bias" in p:
             self.t["lm_head_bias"] = dev(shard_rows(p["lm_head_bias"], rank, world))
         for i in range(s.num_layers):
             L = f"layers.{i}."
-            for n in ("ln1.w", "ln1.b", "ln2.w", "ln2.b", "q_norm", "k_norm"):
+            ls, kh = s.layer(i), self.heads[i]
+            for n in ("ln1.w", "ln1.b", "ln2.w", "ln2.b"):
                 if L + n in p:
-                    self.t[L + n] = dev(p[L + n])
-            wqkv = p[L + "wqkv"]
-            q, k, v = wqkv.split([s.q_size, s.kv_size, s.kv_size], dim=0)
-            self.t[L + "wqkv"] = dev(torch.cat([shard_rows(q, rank, world), kv_rows(k), kv_rows(v)], 0))
+                    self.t[L + n] = dev(_pad(p[L + n], 0, H))
+            for n in ("q_norm", "k_norm"):
+                if L + n in p:
+                    self.t[L + n] = dev(_pad(p[L + n], 0, kh.dk))
+            if L + "sink" in p:
+                self.t[L + "sink"] = p[L + "sink"][rank * kh.hq:(rank + 1) * kh.hq].to(device=device, dtype=torch.float32).contiguous()
+
+            def fused_rows(t):
+                parts = t.split([ls.q_size, ls.k_size, ls.v_size]) if kh.own_kv else (t,)
+                out = [heads(parts[0], ls.num_heads, ls.head_dim, kh.dk, rank * kh.hq, kh.hq)]
+                if kh.own_kv:
+                    out.append(heads(parts[1], ls.num_kv_heads, ls.head_dim, kh.dk, kh.kv_lo, kh.hkv))
+                    out.append(heads(parts[2], ls.num_kv_heads, ls.v_head_dim, kh.dv, kh.kv_lo, kh.hkv))
+                return torch.cat(out, 0)
+
+            self.t[L + "wqkv"] = dev(_pad(fused_rows(p[L + "wqkv"]), 1, H))
             if L + "bqkv" in p:
-                qb, kb, vb = p[L + "bqkv"].split([s.q_size, s.kv_size, s.kv_size])
-                self.t[L + "bqkv"] = dev(torch.cat([shard_rows(qb, rank, world), kv_rows(kb), kv_rows(vb)]))
-            self.t[L + "wo"] = dev(shard_cols(p[L + "wo"], rank, world))
+                self.t[L + "bqkv"] = dev(fused_rows(p[L + "bqkv"]))
+            wo = p[L + "wo"].t()                              # [heads * v size, H]: sharded and padded like the head rows
+            self.t[L + "wo"] = dev(_pad(heads(wo, ls.num_heads, ls.v_head_dim, kh.dv, rank * kh.hq, kh.hq).t(), 0, H))
             if L + "bo" in p:
                 self.t[L + "bo"] = dev(p[L + "bo"] if rank == 0 else torch.zeros_like(p[L + "bo"]))
             if L + "w_gate_up" in p:
@@ -167,30 +210,63 @@ class RunnerWeights:
                     self.t[L + "b_down"] = dev(p[L + "b_down"] if rank == 0 else torch.zeros_like(p[L + "b_down"]))
             if L + "router" in p:
                 # experts: tensor-parallel inside each expert here; expert-parallel layouts are built by MoeRunner
-                self.t[L + "router"] = dev(p[L + "router"])
-                gu = p[L + "experts_gate_up"]
-                E = gu.shape[0]
+                m = ls.moe
+                self.t[L + "router"] = dev(_pad(p[L + "router"], 1, H))
+                if m.router_bias:
+                    self.t[L + "router_b"] = dev(p[L + "router_b"])
+
+                def up_rows(t, r, w):
+                    """This rank's rows of an up (or [gate; up]) matrix [.., rows, H], each half padded to 8."""
+                    halves = t.chunk(2, -2) if m.gated else (t,)
+                    n = halves[0].shape[-2] // w
+                    cut = [_pad(h[..., r * n:(r + 1) * n, :], h.dim() - 2, self._round(n)) for h in halves]
+                    return _pad(torch.cat(cut, -2), t.dim() - 1, H)
+
+                def down_cols(t, r, w):
+                    n = t.shape[-1] // w
+                    return _pad(_pad(t[..., r * n:(r + 1) * n], t.dim() - 1, self._round(n)), t.dim() - 2, H)
+
+                gu, dn = p[L + "experts_gate_up"], p[L + "experts_down"]
                 if self.ep:
                     # expert parallel: whole experts [expert_lo, expert_lo + experts_local) live here
                     lo, hi = self.expert_lo, self.expert_lo + self.experts_local
-                    self.t[L + "experts_gate_up"] = dev(gu[lo:hi])
-                    self.t[L + "experts_down"] = dev(p[L + "experts_down"][lo:hi])
-                elif s.moe.gated:
-                    g, u = gu.chunk(2, 1)
-                    n = g.shape[1] // world
-                    gu = torch.cat([g[:, rank * n:(rank + 1) * n], u[:, rank * n:(rank + 1) * n]], 1)
+                    self.t[L + "experts_gate_up"] = dev(up_rows(gu[lo:hi], 0, 1))
+                    self.t[L + "experts_down"] = dev(down_cols(dn[lo:hi], 0, 1))
                 else:
-                    n = gu.shape[1] // world
-                    gu = gu[:, rank * n:(rank + 1) * n]
-                if not self.ep:
-                    self.t[L + "experts_gate_up"] = dev(gu)
-                    dn = p[L + "experts_down"]
-                    n = dn.shape[2] // world
-                    self.t[L + "experts_down"] = dev(dn[:, :, rank * n:(rank + 1) * n])
+                    self.t[L + "experts_gate_up"] = dev(up_rows(gu, rank, world))
+                    self.t[L + "experts_down"] = dev(down_cols(dn, rank, world))
                 if L + "shared_gate_up" in p:
-                    g, u = p[L + "shared_gate_up"].chunk(2, 0)
-                    self.t[L + "shared_gate_up"] = dev(torch.cat([shard_rows(g, rank, world), shard_rows(u, rank, world)], 0))
-                    self.t[L + "shared_down"] = dev(shard_cols(p[L + "shared_down"], rank, world))
+                    self.t[L + "shared_gate_up"] = dev(up_rows(p[L + "shared_gate_up"], rank, world))
+                    self.t[L + "shared_down"] = dev(down_cols(p[L + "shared_down"], rank, world))
+
+    def _init_layout(self, spec: DecoderSpec, rank: int, world: int, expert_parallel: bool, dtype=torch.bfloat16) -> None:
+        """Everything that follows from the spec and the rank alone: head layout per layer, padded width, shard sizes."""
+        self.spec, self.rank, self.world, self.dtype = spec, rank, world, dtype
+        self._round = _round8 if spec.layers is not None else (lambda n: n)
+        self._set_ep(expert_parallel)
+        if spec.vocab_size % world != 0:
+            raise InvalidInput(f"vocab {spec.vocab_size} not divisible by tensor parallel size {world}")
+        self.vocab_shard = spec.vocab_size // world
+        self.width = self._round(spec.hidden_size)
+        self.heads: List[KernelHeads] = []
+        for i in range(spec.num_layers):
+            ls = spec.layer(i)
+            if ls.num_heads % world != 0:
+                raise InvalidInput(f"{ls.num_heads} heads not divisible by tensor parallel size {world}")
+            if ls.moe is not None and not self.ep and (ls.moe.intermediate_size % world or ls.moe.shared_width % world):
+                raise InvalidInput(f"layer {i}: expert widths not divisible by tensor parallel size {world}")
+            hkv, kv_lo = self.kv_layout(ls.num_kv_heads, rank, world)
+            self.heads.append(KernelHeads(ls.num_heads // world, hkv, kv_lo, self._round(ls.head_dim), self._round(ls.v_head_dim),
+                                          ls.kv_from is None))
+        # uniform specs: one layout for all layers
+        self.hq = self.heads[0].hq if self.heads else spec.num_heads // world
+        self.hkv, self.kv_lo = (self.heads[0].hkv, self.heads[0].kv_lo) if self.heads else \
+            self.kv_layout(spec.num_kv_heads, rank, world)
+
+    def kv_bytes_per_token(self) -> int:
+        """Cache bytes that one token takes on this rank over all layers that own keys and values."""
+        e = torch.empty(0, dtype=self.dtype).element_size()
+        return e * sum(k.hkv * (k.dk + k.dv) for k in self.heads if k.own_kv)
 
     @staticmethod
     def kv_layout(num_kv_heads: int, rank: int, world: int) -> Tuple[int, int]:
@@ -219,12 +295,8 @@ class RunnerWeights:
         benchmark path for 8B-70B architectures.  Every rank draws the same full-size tensor for a given
         name from a per-tensor seed and keeps its shard, so TP=1 and TP=N hold the same model."""
         self = RunnerWeights.__new__(RunnerWeights)
-        self.spec, self.rank, self.world = spec, rank, world
         s = spec
-        self._set_ep(expert_parallel)
-        self.hq = s.num_heads // world
-        self.hkv, self.kv_lo = self.kv_layout(s.num_kv_heads, rank, world)
-        self.vocab_shard = s.vocab_size // world
+        self._init_layout(spec, rank, world, expert_parallel)
         self.t = {}
         H, I = s.hidden_size, s.intermediate_size
         std = s.initializer_range
@@ -257,6 +329,9 @@ class RunnerWeights:
             self.t["lm_head"] = self.t["embed"][rank * vs:(rank + 1) * vs] if world > 1 else self.t["embed"]
         else:
             self.t["lm_head"] = rnd(s.vocab_size, H, rank * vs, vs)
+        if s.layers is not None:
+            self._random_layers(rnd, ones)
+            return self
         qs, ks = s.q_size // world, self.hkv * s.head_dim
         k0 = self.kv_lo * s.head_dim
         for i in range(s.num_layers):
@@ -292,6 +367,41 @@ class RunnerWeights:
                 self.t[L + "w_gate_up"] = torch.cat([g, u], 0)
                 self.t[L + "w_down"] = rnd(H, I, 0, H, rank * Is, Is)
         return self
+
+    def _random_layers(self, rnd, ones) -> None:
+        """Random weights of a per-layer spec on one rank, in kernel layout."""
+        s, H = self.spec, self.width
+        if self.world != 1 or H != s.hidden_size:
+            raise UnsupportedOperation("random per-layer weights: one rank, width a multiple of 8")
+        zeros = lambda n: torch.zeros_like(ones(n))
+        if s.norm_bias:
+            self.t["final_norm.b"] = zeros(H)
+        for i, (kh, ls) in enumerate(zip(self.heads, s.layers)):
+            L = f"layers.{i}."
+            for n in ("ln1", "ln2"):
+                self.t[L + n + ".w"] = ones(H)
+                if s.norm_bias:
+                    self.t[L + n + ".b"] = zeros(H)
+            self.t[L + "wqkv"] = rnd(kh.qkv_rows, H)
+            self.t[L + "wo"] = rnd(H, kh.hq * kh.dv)
+            if s.qk_norm:
+                self.t[L + "q_norm"] = ones(kh.dk)
+                if kh.own_kv:
+                    self.t[L + "k_norm"] = ones(kh.dk)
+            if ls.sink:
+                self.t[L + "sink"] = zeros(kh.hq).float()
+            m = ls.moe
+            if m is None:
+                continue
+            up = (2 if m.gated else 1) * self._round(m.intermediate_size)
+            self.t[L + "router"] = rnd(m.num_experts, H)
+            if m.router_bias:
+                self.t[L + "router_b"] = zeros(m.num_experts)
+            self.t[L + "experts_gate_up"] = torch.stack([rnd(up, H) for _ in range(m.num_experts)])
+            self.t[L + "experts_down"] = torch.stack([rnd(H, self._round(m.intermediate_size)) for _ in range(m.num_experts)])
+            if m.num_shared_experts:
+                self.t[L + "shared_gate_up"] = rnd((2 if m.gated else 1) * self._round(m.shared_width), H)
+                self.t[L + "shared_down"] = rnd(H, self._round(m.shared_width))
 
     def quantize(self, qtype="q4_k") -> "RunnerWeights":
         """Re-encodes every projection matrix (QKV, attention output, MLP, ``lm_head``; not embeddings, norms, routers
@@ -501,6 +611,11 @@ class GpuModelRunner:
                  tp: Optional[TpContext] = None, device=None, use_cuda_graphs: bool = True):
         if spec.norm not in ("rms", "layer") or spec.post_ln or spec.embed_proj_dim:
             raise UnsupportedOperation("this spec is served by the generic model path, not the fused runner")
+        if spec.norm_placement == "output" and (not spec.residual_fp32 or spec.pos == "learned" or spec.embed_norm
+                                                or spec.residual_scale != 1.0 or spec.parallel_residual):
+            raise UnsupportedOperation("norms on sublayer outputs: 32-bit residual stream, no learned positions")
+        if spec.norm_placement == "input" and (spec.residual_fp32 or weights.dtype != torch.bfloat16):
+            raise UnsupportedOperation("a 32-bit residual stream or 32-bit weights: only with norms on sublayer outputs")
         self.spec, self.w = spec, weights
         self.tp = tp or TpContext()
         self.device = torch.device(device if device is not None else f"cuda:{torch.cuda.current_device()}")
@@ -510,11 +625,19 @@ class GpuModelRunner:
         # NCCL collectives inside a captured graph stalled on this stack; the baseline path launches eagerly
         self.use_cuda_graphs = use_cuda_graphs and (self.tp.world == 1 or self.tp.fused)
         s, dev = spec, self.device
-        hkv, D = weights.hkv, s.head_dim
-        self.k_cache = [torch.zeros(num_blocks, hkv, block_size, D, dtype=torch.bfloat16, device=dev)
-                        for _ in range(s.num_layers)]
-        self.v_cache = [torch.zeros(num_blocks, hkv, block_size, D, dtype=torch.bfloat16, device=dev)
-                        for _ in range(s.num_layers)]
+        self.layers = [s.layer(i) for i in range(s.num_layers)]
+        # a window that no sequence can outgrow is full attention (and keeps the kernels for that)
+        self.windows = [ls.window if 0 < ls.window < max_model_len else 0 for ls in self.layers]
+        self.k_cache: List[torch.Tensor] = []
+        self.v_cache: List[torch.Tensor] = []
+        for ls, kh in zip(self.layers, weights.heads):
+            if ls.kv_from is not None:                   # attends to that layer's pages
+                self.k_cache.append(self.k_cache[ls.kv_from])
+                self.v_cache.append(self.v_cache[ls.kv_from])
+                continue
+            for cache, d in ((self.k_cache, kh.dk), (self.v_cache, kh.dv)):
+                cache.append(torch.zeros(num_blocks, kh.hkv, block_size, d, dtype=weights.dtype, device=dev))
+        self._inv_freq: Dict[tuple, torch.Tensor] = {}   # rotation tables of per-layer specs
         self.alibi = None
         if s.pos == "alibi":
             sl = alibi_slopes(s.num_heads)
@@ -534,7 +657,8 @@ class GpuModelRunner:
         self._out_events = [torch.cuda.Event(), torch.cuda.Event()]
         self._sel: List[int] = []
         self._handle = None
-        self.attn_scratch = torch.empty(max_num_seqs * weights.hq * 16 * (D + 2), dtype=torch.float32, device=dev)
+        self.attn_scratch = torch.empty(max_num_seqs * 16 * max((k.hq * (k.dv + 2) for k in weights.heads), default=0),
+                                        dtype=torch.float32, device=dev)
         self.prefix_scratch = None     # workspace of the key-split shared-prefix pass, allocated on first use
         self._deq_scratch = None       # bf16 expansion of one quantised matrix at a time (quantised weights, > 8 rows)
         if getattr(weights, "quantized", None):
@@ -666,29 +790,52 @@ class GpuModelRunner:
         self.launches += 1
         return K.gemm_tn(x, dense, **kw)
 
+    def _rope_append(self, i, qkv, pos, slots):
+        """Head norms and rotation of q and k in place, keys and values into the cache (of a layer that owns some)."""
+        s, t, ls, kh = self.spec, self.w.t, self.layers[i], self.w.heads[i]
+        L = f"layers.{i}."
+        kw = dict(theta=ls.rope_theta, llama3_scaling=ls.rope_llama3)
+        if s.layers is not None:
+            # frequencies from the host in 64 bits, and only for the layers' own rotation
+            key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3)
+            if key not in self._inv_freq:
+                self._inv_freq[key] = rope_inv_freq(*key).to(self.device)
+            kw = dict(inv_freq=self._inv_freq[key] if ls.rotary_dim > 0 else None, v_head_dim=kh.dv, norm_dim=ls.head_dim)
+        own = kh.own_kv
+        with self._prof("rope_kv_append"):
+            K.rope_kv_append(qkv, pos, slots if own else None, self.k_cache[i] if own else None,
+                             self.v_cache[i] if own else None, num_q_heads=kh.hq, num_kv_heads=kh.hkv if own else 0,
+                             head_dim=kh.dk, rotary_dim=ls.rotary_dim, pos_scale=s.rope_pos_scale,
+                             interleaved=s.rope_interleaved, q_norm_w=t.get(L + "q_norm"), k_norm_w=t.get(L + "k_norm"),
+                             norm_eps=s.norm_eps, **kw)
+        self.launches += 1
+
     def _attention(self, i, qkv, lay, shared_prefix_len):
-        """qkv [T, (hq + 2 hkv) * D] already rotated and appended -> attention output [T, hq * D]."""
-        s, w = self.spec, self.w
-        D, hq, hkv = s.head_dim, w.hq, w.hkv
+        """qkv [T, q | k | v] already rotated and appended -> attention output [T, hq * Dv]."""
+        kh, ls = self.w.heads[i], self.layers[i]
+        D, hq, hkv, window = kh.dk, kh.hq, kh.hkv, self.windows[i]
+        sinks = self.w.t.get(f"layers.{i}.sink")
         T, Dp, P = lay["_T"], lay["_Dp"], lay["_P"]
-        q = qkv.view(T, hq + 2 * hkv, D)[:, :hq]           # strided view: row stride (hq + 2 hkv) * D
-        out = torch.empty(T, hq, D, dtype=torch.bfloat16, device=qkv.device)
+        q = qkv[:, :hq * D].unflatten(1, (hq, D))          # strided view: row stride of the fused projection
+        out = torch.empty(T, hq, kh.dv, dtype=qkv.dtype, device=qkv.device)
         kc, vc = self.k_cache[i], self.v_cache[i]
         bt = self._view(lay, "block_tables").view(Dp + P, self.max_blocks_per_seq)
-        scale = s.attn_scale
-        cascade = shared_prefix_len >= 4 * self.block_size and Dp >= 8
+        scale = ls.scale if ls.scale is not None else 1.0 / math.sqrt(ls.head_dim)
+        # the shared-prefix pass has no window, position bias or sink
+        plain = window == 0 and self.alibi is None and sinks is None and kh.dk == kh.dv and qkv.dtype == torch.bfloat16
+        cascade = plain and shared_prefix_len >= 4 * self.block_size and Dp >= 8
         # prefill rows join the cascade when their chunks start after the shared prefix and share its blocks
-        pp = cascade and P > 0 and lay.get("_pp", False) and s.window == 0 and self.alibi is None
+        pp = cascade and P > 0 and lay.get("_pp", False)
         if cascade:
             # one GEMM-shaped pass of all queries over the shared prefix blocks, one pass per sequence over the
             # unique suffixes, then a merge of the two partials
             R = T if pp else Dp
-            # the suffix kernels fold the prefix partial into their output themselves (head dim 128, page 16, no
-            # window / ALiBi); otherwise a separate merge kernel combines the two partials
-            fused = D == 128 and self.block_size == 16 and s.window == 0 and self.alibi is None
+            # the suffix kernels fold the prefix partial into their output themselves (head dim 128, page 16);
+            # otherwise a separate merge kernel combines the two partials
+            fused = D == 128 and self.block_size == 16
             lse_a = torch.empty(R, hq, dtype=torch.float32, device=qkv.device)
             oa = torch.empty(R, hq, D, dtype=torch.bfloat16, device=qkv.device)
-            kvs = self._prefix_splits(R, shared_prefix_len)
+            kvs = self._prefix_splits(i, R, shared_prefix_len)
             with self._prof("attn_shared_prefix"):
                 K.attn_prefill(q[:R], kc, vc, bt[:1], self._prefix_len_dev(shared_prefix_len), self._q_start_all(R),
                                R, scale=scale, causal=False, window=0, alibi_slopes=None, out=oa, lse=lse_a,
@@ -724,9 +871,8 @@ class GpuModelRunner:
                 lse_b = torch.empty(R, hq, dtype=torch.float32, device=qkv.device)
                 ob = torch.empty(R, hq, D, dtype=torch.bfloat16, device=qkv.device)
                 with self._prof("attn_decode_suffix"):
-                    K.attn_decode(q[:Dp], kc, vc, bt[:Dp], self._view(lay, "seq_lens_d"), scale=scale, window=s.window,
-                                  kv_start=shared_prefix_len, alibi_slopes=self.alibi, out=ob[:Dp], lse=lse_b[:Dp],
-                                  return_lse=True, splits=1)
+                    K.attn_decode(q[:Dp], kc, vc, bt[:Dp], self._view(lay, "seq_lens_d"), scale=scale,
+                                  kv_start=shared_prefix_len, out=ob[:Dp], lse=lse_b[:Dp], return_lse=True, splits=1)
                 if pp:
                     with self._prof("attn_prefill_suffix"):
                         K.attn_prefill(q[Dp:], kc, vc, bt[Dp:], self._view(lay, "seq_lens_p"), self._view(lay, "q_start"),
@@ -738,17 +884,17 @@ class GpuModelRunner:
                 self.launches += 3
         elif Dp > 0:
             with self._prof("attn_decode"):
-                K.attn_decode(q[:Dp], kc, vc, bt[:Dp], self._view(lay, "seq_lens_d"), scale=scale, window=s.window,
-                              alibi_slopes=self.alibi, out=out[:Dp], scratch=self.attn_scratch,
+                K.attn_decode(q[:Dp], kc, vc, bt[:Dp], self._view(lay, "seq_lens_d"), scale=scale, window=window,
+                              alibi_slopes=self.alibi, sinks=sinks, out=out[:Dp], scratch=self.attn_scratch,
                               max_seq_len=self.max_model_len if self._graph_mode else int(self._max_len_d))
             self.launches += 1
         if P > 0 and not pp:
             with self._prof("attn_prefill"):
                 K.attn_prefill(q[Dp:], kc, vc, bt[Dp:], self._view(lay, "seq_lens_p"), self._view(lay, "q_start"),
-                               lay["_max_q"], scale=scale, causal=True, window=s.window, alibi_slopes=self.alibi,
-                               out=out[Dp:])
+                               lay["_max_q"], scale=scale, causal=True, window=window, alibi_slopes=self.alibi,
+                               sinks=sinks, out=out[Dp:])
             self.launches += 1
-        return out.view(T, hq * D)
+        return out.view(T, hq * kh.dv)
 
     def _side_stream(self):
         if self._side is None:
@@ -757,12 +903,12 @@ class GpuModelRunner:
 
     PREFIX_SPLIT_ROWS = 160 * 128     # (query row, head) pairs x splits the key-split workspace can hold
 
-    def _prefix_splits(self, R: int, prefix_len: int) -> int:
+    def _prefix_splits(self, i: int, R: int, prefix_len: int) -> int:
         """Key splits of the shared-prefix pass.  The pass has one CTA per 128 packed (token, head-of-group) rows and KV
         head; a tensor-parallel rank with one KV head and a few hundred rows would keep a fraction of the SMs busy while
         every CTA walks the whole prefix, so the key tiles are divided until about one wave of CTAs exists."""
-        s, w = self.spec, self.w
-        if s.head_dim != 128 or self.block_size != 16 or s.window or self.alibi is not None:
+        w = self.w.heads[i]
+        if w.dk != 128 or self.block_size != 16:
             return 1
         G = w.hq // w.hkv
         if 128 % G:
@@ -821,6 +967,8 @@ class GpuModelRunner:
             self._last_fused = True
             return self._forward_tokens_fused(lay, shared_prefix_len)
         self._last_fused = False
+        if s.norm_placement == "output":
+            return self._forward_tokens_output_norm(lay, shared_prefix_len)
         ids = self._view(lay, "token_ids")
         pos = self._view(lay, "positions")
         slots = self._view(lay, "slot_mapping")
@@ -835,14 +983,7 @@ class GpuModelRunner:
             L = f"layers.{i}."
             h = self._norm(x, L + "ln1")
             qkv = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
-            with self._prof("rope_kv_append"):
-                K.rope_kv_append(qkv, pos, slots, self.k_cache[i], self.v_cache[i], num_q_heads=self.w.hq,
-                                 num_kv_heads=self.w.hkv, head_dim=s.head_dim,
-                                 rotary_dim=s.rd if s.pos == "rope" else 0, theta=s.rope_theta,
-                                 pos_scale=s.rope_pos_scale, interleaved=s.rope_interleaved,
-                                 q_norm_w=t.get(L + "q_norm"), k_norm_w=t.get(L + "k_norm"), norm_eps=s.norm_eps,
-                                 llama3_scaling=s.rope_llama3)
-            self.launches += 1
+            self._rope_append(i, qkv, pos, slots)
             a = self._attention(i, qkv, lay, shared_prefix_len)
             if s.parallel_residual:
                 m_in = h if s.parallel_shared_norm else self._norm(x, L + "ln2")
@@ -872,12 +1013,47 @@ class GpuModelRunner:
                 self.launches += 1
         return x
 
+    def _forward_tokens_output_norm(self, lay, shared_prefix_len: int) -> torch.Tensor:
+        """Layers of the form ``x += norm(f(x))`` around a 32-bit residual stream.  ``h`` is the stream in the element type
+        of the matrix products; the norm of a sublayer's output, the residual add and the next ``h`` are one kernel, which
+        for a mixture-of-experts also sums the chosen experts' rows and the shared expert's."""
+        s, t, tp = self.spec, self.w.t, self.tp
+        pos, slots = self._view(lay, "positions"), self._view(lay, "slot_mapping")
+        x, h = K.embed_residual(self._view(lay, "token_ids"), t["embed"], scale=s.embed_scale)
+        self.launches += 1
+        for i, ls in enumerate(self.layers):
+            L = f"layers.{i}."
+            qkv = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
+            self._rope_append(i, qkv, pos, slots)
+            a = self._attention(i, qkv, lay, shared_prefix_len)
+            y = self._gemm(a, t[L + "wo"], bias=t.get(L + "bo"))
+            tp.all_reduce(y)
+            h = self._residual_norm(x, y, L + "ln1")
+            if ls.mlp == "moe":
+                from .moe_runner import moe_branch
+
+                y, experts, routing = moe_branch(self, i, h, router_x=x)
+                h = self._residual_norm(x, y, L + "ln2", experts=experts, routing=routing)
+            elif ls.mlp == "dense":
+                y = self._mlp_noresid(i, h)
+                tp.all_reduce(y)
+                h = self._residual_norm(x, y, L + "ln2")
+        return x
+
+    def _residual_norm(self, x, y, name, **kw):
+        s, t = self.spec, self.w.t
+        self.launches += 1
+        with self._prof("residual_norm"):
+            return K.residual_norm(x, y, t[name + ".w"], t.get(name + ".b"), eps=s.norm_eps,
+                                   kind="rms" if s.norm == "rms" else "layer", width=s.hidden_size,
+                                   out=x if self.w.dtype == torch.float32 else None, **kw)
+
     # ------------------------------------------------------------------------------------------
     # fused tensor-parallel path (F1 / F3)
     # ------------------------------------------------------------------------------------------
     def _fused_ok(self, T: int) -> bool:
         s, tp = self.spec, self.tp
-        return (tp.fused and tp.comm is not None and T % tp.world == 0 and T // tp.world <= tp.comm.max_rows
+        return (tp.fused and tp.comm is not None and s.layers is None and s.norm_placement == "input" and T % tp.world == 0 and T // tp.world <= tp.comm.max_rows
                 and not s.parallel_residual and s.residual_scale == 1.0 and s.pos != "learned"
                 and not s.embed_norm and s.final_norm
                 and (s.moe is None or (s.moe.num_shared_experts == 0 and not s.moe.dense_parallel)))
@@ -914,14 +1090,7 @@ class GpuModelRunner:
         for i in range(s.num_layers):
             L = f"layers.{i}."
             qkv = self._gemm(h_full, t[L + "wqkv"], bias=t.get(L + "bqkv"), ag=ag_args, tag="gemm_ag" if ag_args else "gemm")
-            with self._prof("rope_kv_append"):
-                K.rope_kv_append(qkv, pos, slots, self.k_cache[i], self.v_cache[i], num_q_heads=self.w.hq,
-                                 num_kv_heads=self.w.hkv, head_dim=s.head_dim,
-                                 rotary_dim=s.rd if s.pos == "rope" else 0, theta=s.rope_theta,
-                                 pos_scale=s.rope_pos_scale, interleaved=s.rope_interleaved,
-                                 q_norm_w=t.get(L + "q_norm"), k_norm_w=t.get(L + "k_norm"), norm_eps=s.norm_eps,
-                                 llama3_scaling=s.rope_llama3)
-            self.launches += 1
+            self._rope_append(i, qkv, pos, slots)
             a = self._attention(i, qkv, lay, shared_prefix_len)
             # o_proj: partial rows go straight to their owner's receive slot
             self._gemm(a, t[L + "wo"], bias=t.get(L + "bo"), out=rs0_out.view(W * R, H)[:T], rs=c.gemm_rs(0, R),
@@ -1003,13 +1172,24 @@ class GpuModelRunner:
             a = self._gemm(h, t[L + "w_up"], bias=t.get(L + "b_up"), act=s.act)
         return self._gemm(a, t[L + "w_down"], bias=t.get(L + "b_down"))
 
+    def _final_rows(self, x, lay) -> torch.Tensor:
+        """Final-normed rows of the step whose logits are asked for."""
+        s, t = self.spec, self.w.t
+        rows = self._view(lay, "sample_rows")
+        if s.residual_fp32:
+            self.launches += 1
+            with self._prof("norm"):
+                return K.row_norm(x, t["final_norm.w"], t.get("final_norm.b"), eps=s.norm_eps, rows=rows,
+                                  kind="rms" if s.norm == "rms" else "layer", width=s.hidden_size)
+        xs = x.index_select(0, rows.long()) if lay["_S"] != x.shape[0] else x
+        if s.final_norm and not self._final_norm_done:
+            xs = self._norm(xs, "final_norm")
+        return xs
+
     def _logits_and_sample(self, x, lay, b: Optional[StepBatch], fl) -> torch.Tensor:
         s, t, tp = self.spec, self.w.t, self.tp
         S = lay["_S"]
-        rows = self._view(lay, "sample_rows")
-        xs = x.index_select(0, rows.long()) if S != x.shape[0] else x
-        if s.final_norm and not self._final_norm_done:
-            xs = self._norm(xs, "final_norm")
+        xs = self._final_rows(x, lay)
         logits = self._gemm(xs, t["lm_head"], bias=t.get("lm_head_bias"), out_scale=s.logit_scale)
         out = self.out_ids_dev[:S]
         greedy = fl is None
@@ -1224,19 +1404,27 @@ class GpuModelRunner:
         torch.cuda.synchronize(self.device)
 
     def kv_cache_bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.k_cache) * 2
+        own = [i for i, ls in enumerate(self.layers) if ls.kv_from is None]
+        return sum(c[i].numel() * c[i].element_size() for c in (self.k_cache, self.v_cache) for i in own)
 
-    def logits_for(self, b: StepBatch) -> torch.Tensor:
-        """Test hook: full logits [S, vocab_shard] of a step (eager, no sampling)."""
+    def forward_logits(self, b: StepBatch) -> torch.Tensor:
+        """Runs a step as plain launches without sampling: fp32 logits [len(b.sample_rows), vocab shard] of any of its
+        rows (an empty list just appends to the cache)."""
         self._graph_mode = False
         self._max_len_d = max(b.seq_lens[:b.num_decode]) if b.num_decode else 0
         lay = self._pack(b, bucketed=False)
         lay["_pp"] = b.prefill_shares_prefix
         self._upload(lay)
         x = self._forward_tokens(lay, b.shared_prefix_len)
-        rows = self._view(lay, "sample_rows")
-        xs = x.index_select(0, rows.long())
-        if self.spec.final_norm and not self._final_norm_done:
-            xs = self._norm(xs, "final_norm")
-        return self._gemm(xs, self.w.t["lm_head"], bias=self.w.t.get("lm_head_bias"), out_scale=self.spec.logit_scale,
-                          out_dtype=torch.float32)
+        if lay["_S"] == 0:
+            return torch.empty(0, self.w.vocab_shard, dtype=torch.float32, device=self.device)
+        return self._gemm(self._final_rows(x, lay), self.w.t["lm_head"], bias=self.w.t.get("lm_head_bias"),
+                          out_scale=self.spec.logit_scale, out_dtype=torch.float32)
+
+    logits_for = forward_logits
+
+    def raise_on_device_error(self) -> None:
+        """Waits for the work launched so far and raises if a kernel recorded an error."""
+        code, detail = K.err_word(self.device).tolist()
+        if code != 0:
+            raise DeviceStepError(code, detail)

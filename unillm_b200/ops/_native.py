@@ -1,9 +1,11 @@
 """ctypes bindings of the in-tree native libraries.
 
-``cuda_lib()`` loads ``_native/libunillm_b200_cuda.so`` (all sm_100a kernels, C ABI declared in
-``csrc/include/unillm_b200.h``) and ``host_lib()`` loads ``_native/libunillm_b200_host.so`` (C++ host
-runtime).  Both are built on demand by ``unillm_b200._build``.  On a machine with a GPU a missing or
-unloadable CUDA library is an error, never a silent fallback.
+``cuda_lib()`` answers for all sm_100a kernels (C ABI declared in ``csrc/include/unillm_b200.h``): it loads
+``_native/libunillm_b200_cuda.so`` (the kernels that serve a decoder on one GPU) and, when a symbol of it is first
+asked for, ``_native/libunillm_b200_cuda_more.so`` (collectives, recurrences, block-quantised matrices).
+``host_lib()`` loads ``_native/libunillm_b200_host.so`` (C++ host runtime).  Each is built on demand by
+``unillm_b200._build``.  On a machine with a GPU a missing or unloadable CUDA library is an error, never a silent
+fallback.
 """
 from __future__ import annotations
 
@@ -66,6 +68,15 @@ class UbRopeArgs(C.Structure):
         ("T", i32), ("Hq", i32), ("Hkv", i32), ("D", i32), ("rotary_dim", i32), ("block_size", i32),
         ("num_slots", i64), ("theta", f32), ("pos_scale", f32), ("norm_eps", f32), ("interleaved", i32),
         ("l3_factor", f32), ("l3_low_freq_factor", f32), ("l3_high_freq_factor", f32), ("l3_orig_ctx", f32),
+        ("inv_freq", vp), ("Dv", i32), ("norm_dim", i32), ("f32", i32),
+    ]
+
+
+class UbResidualNormArgs(C.Structure):
+    _fields_ = [
+        ("y", vp), ("yx", vp), ("row_slot", vp), ("topk_w", vp), ("x", vp), ("rows", vp), ("out", vp), ("weight", vp),
+        ("bias", vp), ("err", vp), ("T", i32), ("H", i32), ("Hp", i32), ("K", i32), ("slots", i32), ("x_rows", i32),
+        ("kind", i32), ("f32", i32), ("eps", f32),
     ]
 
 
@@ -77,7 +88,7 @@ class UbAttnArgs(C.Structure):
         ("block_size", i32), ("max_blocks_per_seq", i32), ("num_blocks", i32),
         ("q_stride", i64), ("o_stride", i64), ("scale", f32),
         ("causal", i32), ("window", i32), ("splits", i32), ("kv_start", i32), ("total_q", i32), ("max_q_len", i32),
-        ("merge_o", vp), ("merge_lse", vp),
+        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32),
     ]
 
 
@@ -105,7 +116,7 @@ class UbMoeRouteArgs(C.Structure):
         ("expert_offsets", vp), ("sorted_rows", vp), ("row_slot", vp), ("tiles", vp), ("err", vp),
         ("logits_f32", i32), ("T", i32), ("E", i32), ("K", i32), ("H", i32), ("norm_topk", i32),
         ("round_logits_bf16", i32), ("weight_scale", f32), ("tile_tokens", i32), ("max_tiles", i32),
-        ("expert_lo", i32), ("num_local_experts", i32),
+        ("expert_lo", i32), ("num_local_experts", i32), ("router_b", vp), ("x_f32", i32), ("router_f32", i32),
     ]
 
 
@@ -158,12 +169,6 @@ class UbDeviceProps(C.Structure):
     ]
 
 
-def _ensure_built() -> None:
-    from .. import _build
-
-    _build.build_all()
-
-
 def cuda_lib_path() -> Path:
     return _NATIVE_DIR / "libunillm_b200_cuda.so"
 
@@ -172,31 +177,58 @@ def host_lib_path() -> Path:
     return _NATIVE_DIR / "libunillm_b200_host.so"
 
 
-def cuda_lib() -> C.CDLL:
-    """The CUDA kernel library.  Raises if it cannot be built or loaded."""
-    global _cuda
-    if _cuda is not None:
-        return _cuda
-    with _lock:
-        if _cuda is not None:
-            return _cuda
-        if not cuda_lib_path().exists() or os.environ.get("UNILLM_REBUILD"):
-            _ensure_built()
-        lib = C.CDLL(str(cuda_lib_path()))
-        for name in (
-            "ub_gemm_tn", "ub_norm", "ub_rope_kv_append", "ub_attn_decode", "ub_attn_prefill", "ub_sample",
-            "ub_moe_route", "ub_allreduce_oneshot", "ub_tp_argmax_merge",
-        ):
-            if hasattr(lib, name):
-                getattr(lib, name).restype = i32
-                getattr(lib, name).argtypes = [vp, vp]
+class _CudaLibs:
+    """The CUDA libraries behind one namespace; the second is opened when a symbol is not in the first."""
+
+    ARGS_AND_STREAM = {
+        "serving": ("ub_gemm_tn", "ub_norm", "ub_rope_kv_append", "ub_attn_decode", "ub_attn_prefill", "ub_sample",
+                    "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm"),
+        "more": ("ub_allreduce_oneshot", "ub_tp_argmax_merge"),
+    }
+
+    def __init__(self):
+        self._parts = {}
+        lib = self.part("serving")
         lib.ub_gemm_num_ctas.restype = i32
         lib.ub_gemm_num_ctas.argtypes = [vp]
         lib.ub_gemm_streamk_reset.restype = i32
         lib.ub_gemm_streamk_reset.argtypes = [vp]
         lib.ub_cuda_error_string.restype = C.c_char_p
-        _cuda = lib
-        return lib
+
+    def part(self, name: str) -> C.CDLL:
+        if name not in self._parts:
+            from .. import _build
+
+            path = _NATIVE_DIR / _build.CUDA_LIBS[name]
+            if not path.exists() or os.environ.get("UNILLM_REBUILD"):
+                _build.build_cuda(part=name)
+            lib = C.CDLL(str(path))
+            for fn in self.ARGS_AND_STREAM[name]:
+                getattr(lib, fn).restype = i32
+                getattr(lib, fn).argtypes = [vp, vp]
+            self._parts[name] = lib
+        return self._parts[name]
+
+    def __getattr__(self, symbol: str):
+        if not symbol.startswith("ub_"):
+            raise AttributeError(symbol)
+        try:
+            fn = getattr(self.part("serving"), symbol)
+        except AttributeError:
+            with _lock:
+                fn = getattr(self.part("more"), symbol)
+        setattr(self, symbol, fn)
+        return fn
+
+
+def cuda_lib() -> _CudaLibs:
+    """The CUDA kernel libraries.  Raises if they cannot be built or loaded."""
+    global _cuda
+    if _cuda is None:
+        with _lock:
+            if _cuda is None:
+                _cuda = _CudaLibs()
+    return _cuda
 
 
 def host_lib() -> C.CDLL:
@@ -208,7 +240,9 @@ def host_lib() -> C.CDLL:
         if _host is not None:
             return _host
         if not host_lib_path().exists() or os.environ.get("UNILLM_REBUILD"):
-            _ensure_built()
+            from .. import _build
+
+            _build.build_host()
         _host = C.CDLL(str(host_lib_path()))
         return _host
 

@@ -66,6 +66,20 @@ def _bf16c(t: torch.Tensor, name: str) -> None:
         raise ValueError(f"{name} must be a CUDA tensor")
 
 
+def _elem(name: str, t: torch.Tensor, *others: Optional[torch.Tensor]) -> bool:
+    """Checks that ``t`` and the given others are CUDA tensors of one element type, bf16 or fp32; True for fp32."""
+    if t.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"{name} must be bfloat16 or float32, got {t.dtype}")
+    for o in (t, *others):
+        if o is None:
+            continue
+        if o.dtype != t.dtype:
+            raise TypeError(f"{name}: operands of different types ({t.dtype}, {o.dtype})")
+        if not o.is_cuda:
+            raise ValueError(f"{name}: operands must be CUDA tensors")
+    return t.dtype == torch.float32
+
+
 # ---------------------------------------------------------------------------------------------
 # GEMM
 # ---------------------------------------------------------------------------------------------
@@ -78,12 +92,17 @@ def gemm_tn(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = 
 
     ``dual_rows = I`` switches to the gated form: ``w`` is ``[2*I, K]`` with gate rows first and the
     result is ``act(x @ w[:I]^T) * (x @ w[I:]^T)`` of shape ``[M, I]``.
+    With fp32 operands everything runs in 32-bit arithmetic and the result is fp32.
     ``rs`` / ``ag`` carry the peer pointers for the fused reduce-scatter / all-gather variants (see
     :mod:`unillm_b200.dist.fused`).
     """
-    _bf16c(x, "x"), _bf16c(w, "w")
+    f32 = _elem("gemm_tn", x, w, bias, residual)      # fp32 operands: 32-bit arithmetic (ub_gemm_f32)
     if x.dim() != 2 or w.dim() != 2:
         raise ValueError("gemm_tn takes 2-D operands")
+    if f32:
+        if rs is not None or ag is not None or (out is not None and out.dtype != torch.float32):
+            raise ValueError("gemm_tn in fp32: no fused collectives, fp32 output")
+        out_dtype = torch.float32
     if x.stride(1) != 1 or w.stride(1) != 1:
         raise ValueError("operands must be K-contiguous")
     M, K = x.shape
@@ -115,10 +134,6 @@ def gemm_tn(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = 
     a.splits = splits
     a.cta_pair = cta_pair
     a.pair_splits = pair_splits
-    if bias is not None:
-        _bf16c(bias, "bias")
-    if residual is not None:
-        _bf16c(residual, "residual")
     if rs is not None:
         a.rs_world, a.rs_rank, a.rs_rows_per_rank = rs["world"], rs["rank"], rs["rows_per_rank"]
         for i in range(rs["world"]):
@@ -131,7 +146,10 @@ def gemm_tn(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = 
     if grouped is not None:
         a.grp_tiles, a.grp_max_tiles, a.grp_w_rows = grouped["tiles"], grouped["max_tiles"], grouped["w_rows"]
         a.tile_tokens = grouped["tile_tokens"]
-    N.check(N.cuda_lib().ub_gemm_tn(C.byref(a), _stream(x)), "ub_gemm_tn")
+    if f32:
+        N.check(N.cuda_lib().ub_gemm_f32(C.byref(a), _stream(x)), "ub_gemm_f32")
+    else:
+        N.check(N.cuda_lib().ub_gemm_tn(C.byref(a), _stream(x)), "ub_gemm_tn")
     return out
 
 
@@ -208,6 +226,77 @@ def norm(x: torch.Tensor, weight: Optional[torch.Tensor], *, bias: Optional[torc
 
 
 # ---------------------------------------------------------------------------------------------
+# Norms around a 32-bit residual stream
+# ---------------------------------------------------------------------------------------------
+def _resid_args(what: str, x: torch.Tensor, weight, bias, out, H: int, eps: float, kind: str):
+    f32 = _elem(what, weight, bias, out)
+    if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous() or out.shape[1:] != x.shape[1:]:
+        raise ValueError(f"{what}: the residual stream is a contiguous fp32 [T, width] tensor, out has its rows' size")
+    if not out.is_contiguous() or weight.numel() != x.shape[1] or (bias is not None and bias.numel() != x.shape[1]):
+        raise ValueError(f"{what}: weights must cover the (padded) row")
+    a = N.UbResidualNormArgs()
+    a.x, a.out, a.weight, a.bias = x.data_ptr(), out.data_ptr(), weight.data_ptr(), _p(bias)
+    a.err = err_word(x.device).data_ptr()
+    a.T, a.H, a.Hp, a.x_rows = out.shape[0], H, x.shape[1], x.shape[0]
+    a.kind, a.f32, a.eps = (0 if kind == "rms" else 1), int(f32), eps
+    return a
+
+
+def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, bias: Optional[torch.Tensor] = None, *,
+                  eps: float, kind: str = "rms", width: Optional[int] = None, out: Optional[torch.Tensor] = None,
+                  experts: Optional[torch.Tensor] = None, routing: Optional["MoeRouting"] = None) -> torch.Tensor:
+    """``x += norm(y)`` on the fp32 residual stream ``x`` (in place); returns the new rows in the type of ``weight``.
+
+    ``experts`` / ``routing``: the rows to be normalised are ``y + sum_k w[t, k] * experts[row_slot[t, k]]`` (``y`` may then
+    be None).  ``width``: real row size when rows are zero-padded to a multiple of 8."""
+    if out is None:
+        out = torch.empty(x.shape, dtype=weight.dtype, device=x.device)
+    a = _resid_args("residual_norm", x, weight, bias, out, width or x.shape[1], eps, kind)
+    for t in (y, experts):
+        if t is not None and (t.dtype != weight.dtype or t.shape[1] != x.shape[1] or not t.is_contiguous()):
+            raise ValueError("residual_norm: sublayer rows must be contiguous, of the weights' type and the stream's width")
+    if y is not None and y.shape[0] != x.shape[0]:
+        raise ValueError("residual_norm: one sublayer row per token")
+    a.y = _p(y)
+    if experts is not None:
+        if routing.T != x.shape[0]:
+            raise ValueError("residual_norm: the routing is of another step")
+        a.yx, a.row_slot, a.topk_w = experts.data_ptr(), routing.row_slot.data_ptr(), routing.topk_w.data_ptr()
+        a.K, a.slots = routing.K, experts.shape[0]
+    N.check(N.cuda_lib().ub_residual_norm(C.byref(a), _stream(x)), "ub_residual_norm")
+    return out
+
+
+def row_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None, *, eps: float, kind: str = "rms",
+             rows: Optional[torch.Tensor] = None, width: Optional[int] = None) -> torch.Tensor:
+    """``norm(x[rows])`` of an fp32 residual stream (all rows when ``rows`` is None) in the type of ``weight``."""
+    if rows is not None and rows.dtype != torch.int32:
+        raise TypeError("rows must be int32")
+    n = x.shape[0] if rows is None else rows.numel()
+    out = torch.empty(n, x.shape[1], dtype=weight.dtype, device=x.device)
+    a = _resid_args("row_norm", x, weight, bias, out, width or x.shape[1], eps, kind)
+    a.rows = _p(rows)
+    N.check(N.cuda_lib().ub_row_norm(C.byref(a), _stream(x)), "ub_row_norm")
+    return out
+
+
+def embed_residual(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0):
+    """First value of an fp32 residual stream: ``(x fp32, the same rows in the table's type)``."""
+    f32 = _elem("embed_residual", table)
+    if ids.dtype != torch.int32 or not table.is_contiguous():
+        raise ValueError("embed_residual: int32 ids, contiguous table")
+    T, (V, Hp) = ids.numel(), table.shape
+    x = torch.empty(T, Hp, dtype=torch.float32, device=table.device)
+    out = x if f32 else torch.empty(T, Hp, dtype=table.dtype, device=table.device)
+    lib = N.cuda_lib()
+    lib.ub_embed_residual.restype = C.c_int
+    lib.ub_embed_residual.argtypes = [N.vp, N.vp, N.vp, N.vp, N.i32, N.i32, N.i32, N.f32, N.i32, N.vp, N.vp]
+    N.check(lib.ub_embed_residual(ids.data_ptr(), table.data_ptr(), x.data_ptr(), out.data_ptr(), T, Hp, V, scale, int(f32),
+                                  err_word(table.device).data_ptr(), _stream(table)), "ub_embed_residual")
+    return x, out
+
+
+# ---------------------------------------------------------------------------------------------
 # RoPE + KV append
 # ---------------------------------------------------------------------------------------------
 def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Optional[torch.Tensor],
@@ -215,9 +304,14 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
                    num_kv_heads: int, head_dim: int, rotary_dim: Optional[int] = None, theta: float = 10000.0,
                    pos_scale: float = 1.0, interleaved: bool = False, q_norm_w: Optional[torch.Tensor] = None,
                    k_norm_w: Optional[torch.Tensor] = None, norm_eps: float = 1e-6,
-                   llama3_scaling: Optional[Sequence[float]] = None) -> torch.Tensor:
-    """Rotates q and k inside ``qkv`` [T, (Hq+2Hkv)*D] in place and appends k, v to the paged cache."""
-    _bf16c(qkv, "qkv")
+                   llama3_scaling: Optional[Sequence[float]] = None, v_head_dim: Optional[int] = None,
+                   norm_dim: int = 0, inv_freq: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Rotates q and k inside ``qkv`` [T, (Hq+Hkv)*D + Hkv*Dv] in place and appends k, v to the paged cache.
+
+    ``num_kv_heads = 0``: rows hold queries only (a layer that reads another layer's keys).  ``inv_freq`` (fp32
+    [rotary_dim / 2]) replaces the frequencies that ``theta`` and the scaling give; ``norm_dim`` is the number of elements
+    the head norm averages over when heads are zero-padded."""
+    f32 = _elem("rope_kv_append", qkv, k_cache, v_cache, q_norm_w, k_norm_w)
     if not qkv.is_contiguous():
         raise ValueError("qkv must be contiguous")
     T = qkv.shape[0]
@@ -238,6 +332,15 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
         a.slot_mapping = None
     a.theta, a.pos_scale, a.norm_eps = theta, pos_scale, norm_eps
     a.interleaved = 1 if interleaved else 0
+    a.Dv, a.norm_dim, a.f32 = v_head_dim or head_dim, norm_dim, int(f32)
+    if qkv.shape[1] != (num_q_heads + num_kv_heads) * head_dim + num_kv_heads * a.Dv:
+        raise ValueError(f"rope_kv_append: rows of {qkv.shape[1]} elements do not hold these heads")
+    if k_cache is not None and (k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]) != (num_kv_heads, head_dim, a.Dv):
+        raise ValueError("rope_kv_append: cache shapes do not match the heads")
+    if inv_freq is not None:
+        if inv_freq.dtype != torch.float32 or inv_freq.numel() != a.rotary_dim // 2:
+            raise ValueError("inv_freq: fp32, one entry per rotated pair")
+        a.inv_freq = inv_freq.data_ptr()
     if llama3_scaling is not None:
         a.l3_factor, a.l3_low_freq_factor, a.l3_high_freq_factor, a.l3_orig_ctx = llama3_scaling
     N.check(N.cuda_lib().ub_rope_kv_append(C.byref(a), _stream(qkv)), "ub_rope_kv_append")
@@ -247,7 +350,7 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
 # ---------------------------------------------------------------------------------------------
 # Attention
 # ---------------------------------------------------------------------------------------------
-def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale):
+def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks=None):
     a = N.UbAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out, a.lse = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(lse)
     a.block_tables, a.seq_lens = block_tables.data_ptr(), seq_lens.data_ptr()
@@ -256,6 +359,13 @@ def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D
     a.block_size, a.max_blocks_per_seq, a.num_blocks = k_cache.shape[2], block_tables.shape[1], k_cache.shape[0]
     a.q_stride, a.o_stride = q.stride(0), out.stride(0)
     a.scale = scale if scale is not None else 1.0 / math.sqrt(D)
+    a.Dv = v_cache.shape[3]
+    if k_cache.shape[3] != D or out.shape[-1] != a.Dv:
+        raise ValueError("attention: head sizes of q, caches and out do not match")
+    if sinks is not None:
+        if sinks.dtype != torch.float32 or sinks.numel() != Hq:
+            raise ValueError("sinks: fp32, one per query head")
+        a.sinks = sinks.data_ptr()
     return a
 
 
@@ -263,27 +373,34 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, b
                 seq_lens: torch.Tensor, *, scale: Optional[float] = None, window: int = 0, kv_start: int = 0,
                 alibi_slopes: Optional[torch.Tensor] = None, splits: int = 0, scratch: Optional[torch.Tensor] = None,
                 out: Optional[torch.Tensor] = None, return_lse: bool = False, lse: Optional[torch.Tensor] = None,
-                max_seq_len: Optional[int] = None, merge: Optional[tuple] = None, kernel: Optional[str] = None):
-    """One query token per sequence.  q: [B, Hq, D] (last two dims contiguous); caches [nb, Hkv, bs, D].
+                max_seq_len: Optional[int] = None, merge: Optional[tuple] = None, kernel: Optional[str] = None,
+                sinks: Optional[torch.Tensor] = None):
+    """One query token per sequence.  q: [B, Hq, D] (last two dims contiguous); caches [nb, Hkv, bs, D] (the value cache may
+    have a head size of its own).  ``sinks``: fp32 [Hq], one logit per head that joins the softmax denominator.  fp32
+    operands run in 32-bit arithmetic.
 
     ``kernel="warp"`` calls the warp-per-item kernel directly (page size 16, head size 64 / 128, ``splits == 1``, no
     window, no ALiBi) instead of going through the dispatcher's choice."""
-    _bf16c(q, "q")
+    f32 = _elem("attn_decode", q, k_cache, v_cache, out)
     B, Hq, D = q.shape
-    Hkv = k_cache.shape[1]
+    Hkv, Dv = k_cache.shape[1], v_cache.shape[3]
     if out is None:
-        out = torch.empty((B, Hq, D), dtype=torch.bfloat16, device=q.device)
+        out = torch.empty((B, Hq, Dv), dtype=q.dtype, device=q.device)
     if return_lse and lse is None:
         lse = torch.empty((B, Hq), dtype=torch.float32, device=q.device)
+    if f32:
+        splits = 1
     if splits <= 0:
         ctx = max_seq_len if max_seq_len is not None else block_tables.shape[1] * k_cache.shape[2]
+        if window > 0:
+            ctx = min(ctx, window)
         ctas = B * Hkv
         splits = 1
         while ctas * splits < 2 * 148 and ctx // (splits * 2) >= 256 and splits < 16:
             splits *= 2
-    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale)
+    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks)
     if splits > 1:
-        need = B * Hq * splits * (D + 2)
+        need = B * Hq * splits * (Dv + 2)
         if scratch is None or scratch.numel() < need:
             scratch = torch.empty(need, dtype=torch.float32, device=q.device)
         a.scratch = scratch.data_ptr()
@@ -291,7 +408,9 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, b
     a.alibi_slopes = _p(alibi_slopes)
     if merge is not None:        # (o [B, Hq, D] bf16 contiguous, lse [B, Hq] fp32): partial over a disjoint key set
         a.merge_o, a.merge_lse = merge[0].data_ptr(), merge[1].data_ptr()
-    if kernel == "warp":
+    if f32:
+        N.check(N.cuda_lib().ub_attn_f32(C.byref(a), _stream(q)), "ub_attn_f32")
+    elif kernel == "warp":
         lib = N.cuda_lib()
         if not lib.ub_attn_decode_warp_supported(C.byref(a)):
             raise ValueError("attn_decode(kernel='warp'): page size 16, head size 64 / 128, one split, no window / ALiBi")
@@ -306,7 +425,7 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
                  causal: bool = True, window: int = 0, kv_start: int = 0,
                  alibi_slopes: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
                  return_lse: bool = False, lse: Optional[torch.Tensor] = None, merge: Optional[tuple] = None,
-                 kv_splits: int = 1, scratch: Optional[torch.Tensor] = None):
+                 kv_splits: int = 1, scratch: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
     """Ragged prefill: q [T, Hq, D]; sequence i owns query rows q_start[i]:q_start[i+1] and sees
     seq_lens[i] keys, its last query at kv position seq_lens[i]-1.
 
@@ -314,14 +433,14 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
     folds the partial results with a second small kernel: for launches with few query tiles and many keys, such as
     the shared-prefix pass of a tensor-parallel rank that holds one KV head.  ``scratch`` (fp32, at least
     :func:`attn_prefill_split_scratch_floats` elements) holds the partials."""
-    _bf16c(q, "q")
+    f32 = _elem("attn_prefill", q, k_cache, v_cache, out)
     T, Hq, D = q.shape
     Hkv = k_cache.shape[1]
     if out is None:
-        out = torch.empty((T, Hq, D), dtype=torch.bfloat16, device=q.device)
+        out = torch.empty((T, Hq, v_cache.shape[3]), dtype=q.dtype, device=q.device)
     if return_lse and lse is None:
         lse = torch.empty((T, Hq), dtype=torch.float32, device=q.device)
-    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale)
+    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks)
     a.q_start = q_start.data_ptr()
     a.causal, a.window, a.kv_start = (1 if causal else 0), window, kv_start
     a.total_q, a.max_q_len = T, max_q_len
@@ -335,7 +454,10 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
         if scratch.dtype != torch.float32:
             raise TypeError("scratch must be float32")
         a.splits, a.scratch = kv_splits, scratch.data_ptr()
-    N.check(N.cuda_lib().ub_attn_prefill(C.byref(a), _stream(q)), "ub_attn_prefill")
+    if f32:
+        N.check(N.cuda_lib().ub_attn_f32(C.byref(a), _stream(q)), "ub_attn_f32")
+    else:
+        N.check(N.cuda_lib().ub_attn_prefill(C.byref(a), _stream(q)), "ub_attn_prefill")
     return (out, lse) if return_lse else out
 
 
@@ -606,14 +728,17 @@ def moe_tile_tokens(T: int, K: int, E: int) -> int:
 def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k: int, *, norm_topk: bool = True,
               logits: Optional[torch.Tensor] = None, weight_scale: float = 1.0, tile_tokens: int = 0,
               round_logits_bf16: bool = True, routing: Optional[MoeRouting] = None, expert_lo: int = 0,
-              num_local_experts: int = 0) -> MoeRouting:
-    """Router GEMV + top-k + softmax weights + expert sort + grouped-GEMM tile table, two launches.
+              num_local_experts: int = 0, router_b: Optional[torch.Tensor] = None) -> MoeRouting:
+    """Router GEMV (+ bias) + top-k + softmax weights + expert sort + grouped-GEMM tile table, two launches.  ``x`` may be
+    bf16 or an fp32 residual stream, whatever the type of the router.
 
     ``expert_lo`` / ``num_local_experts`` restrict the sort to the experts of this rank (expert parallelism): pairs
     routed to other ranks get ``row_slot = -1`` and take no part in the grouped GEMMs."""
     if router_w is not None:
-        _bf16c(x, "x"), _bf16c(router_w, "router_w")
+        _elem("moe_route x", x), _elem("moe_route router", router_w, router_b)
         T, H = x.shape
+        if router_w.shape[1] != H or not x.is_contiguous() or not router_w.is_contiguous():
+            raise ValueError("moe_route: x [T, H] and router [E, H] must be contiguous")
         E = router_w.shape[0]
         dev = x.device
     else:
@@ -635,6 +760,8 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
     a.norm_topk = 1 if norm_topk else 0
     a.round_logits_bf16 = 1 if round_logits_bf16 else 0
     a.weight_scale = weight_scale
+    if router_w is not None:
+        a.router_b, a.x_f32, a.router_f32 = _p(router_b), int(x.dtype == torch.float32), int(router_w.dtype == torch.float32)
     a.tile_tokens, a.max_tiles = r.tile_tokens, r.max_tiles
     a.expert_lo, a.num_local_experts = expert_lo, num_local_experts
     N.check(N.cuda_lib().ub_moe_route(C.byref(a), torch.cuda.current_stream(dev).cuda_stream), "ub_moe_route")
@@ -643,14 +770,15 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
 
 def moe_gather(x: torch.Tensor, r: MoeRouting, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``out[slot] = x[sorted_rows[slot] // K]``: activations in expert order."""
-    _bf16c(x, "x")
+    f32 = _elem("moe_gather", x, out)
     T, H = x.shape
     if out is None:
-        out = torch.empty(T * r.K, H, dtype=torch.bfloat16, device=x.device)
+        out = torch.empty(T * r.K, H, dtype=x.dtype, device=x.device)
     lib = N.cuda_lib()
-    lib.ub_moe_gather.restype = C.c_int
-    lib.ub_moe_gather.argtypes = [N.vp, N.vp, N.vp, N.i32, N.i32, N.i32, N.vp]
-    N.check(lib.ub_moe_gather(x.data_ptr(), r.sorted_rows.data_ptr(), out.data_ptr(), T * r.K, r.K, H, _stream(x)),
+    gather = lib.ub_moe_gather_f32 if f32 else lib.ub_moe_gather
+    gather.restype = C.c_int
+    gather.argtypes = [N.vp, N.vp, N.vp, N.i32, N.i32, N.i32, N.vp]
+    N.check(gather(x.data_ptr(), r.sorted_rows.data_ptr(), out.data_ptr(), T * r.K, r.K, H, _stream(x)),
             "ub_moe_gather")
     return out
 
@@ -792,16 +920,17 @@ def grouped_gemm(x_sorted: torch.Tensor, w: torch.Tensor, r: MoeRouting, *, dual
     E, rows, Kd = w.shape
     g = {"tiles": r.tiles.data_ptr(), "max_tiles": r.max_tiles, "w_rows": rows, "tile_tokens": r.tile_tokens}
     n_out = dual_rows if dual_rows else rows
+    f32 = _elem("grouped_gemm", x_sorted, w, out)
     if out is None:
-        out = torch.empty(x_sorted.shape[0], n_out, dtype=torch.bfloat16, device=x_sorted.device)
+        out = torch.empty(x_sorted.shape[0], n_out, dtype=x_sorted.dtype, device=x_sorted.device)
     w2 = w.view(E * rows, Kd)
     if dual_rows:
         return gemm_tn(x_sorted, w2, dual_rows=dual_rows, act=act, out=out, grouped=g)
     # non-dual: N is the per-expert row count while w2 has E*rows rows
-    return _gemm_grouped_plain(x_sorted, w2, rows, act, out, g)
+    return _gemm_grouped_plain(x_sorted, w2, rows, act, out, g, f32)
 
 
-def _gemm_grouped_plain(x, w2, rows, act, out, g):
+def _gemm_grouped_plain(x, w2, rows, act, out, g, f32=False):
     a = N.UbGemmArgs()
     a.x, a.w, a.out = x.data_ptr(), w2.data_ptr(), out.data_ptr()
     a.err = err_word(x.device).data_ptr()
@@ -811,5 +940,6 @@ def _gemm_grouped_plain(x, w2, rows, act, out, g):
     a.w_rows_total = w2.shape[0]
     a.out_scale = 1.0
     a.grp_tiles, a.grp_max_tiles, a.grp_w_rows, a.tile_tokens = g["tiles"], g["max_tiles"], g["w_rows"], g["tile_tokens"]
-    N.check(N.cuda_lib().ub_gemm_tn(C.byref(a), _stream(x)), "ub_gemm_tn(grouped)")
+    lib = N.cuda_lib()
+    N.check((lib.ub_gemm_f32 if f32 else lib.ub_gemm_tn)(C.byref(a), _stream(x)), "ub_gemm_tn(grouped)")
     return out
