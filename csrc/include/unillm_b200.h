@@ -168,6 +168,7 @@ typedef struct UbRopeArgs {
   int Dv;                    /* value head size (0 = D); rows are [Hq * D | Hkv * D | Hkv * Dv] */
   int norm_dim;              /* elements of a head that the RMS norm averages over (0 = D; less when heads are padded) */
   int f32;                   /* qkv, caches and norm weights are fp32 */
+  int k_cache_only;          /* 1: the rotated k need not be written back into qkv (it is in the cache) */
 } UbRopeArgs;
 int ub_rope_kv_append(const UbRopeArgs* args, void* stream);
 

@@ -186,7 +186,7 @@ __global__ void __launch_bounds__(128) rope_kv_append_kernel(const UbRopeArgs a)
 
 // LPH lanes per head (a power of two, LPH * 8 >= D), eight consecutive elements of the head per lane: the norm is a shuffle
 // reduction among the lanes of the head, interleaved pairs are lane-local, half-split pairs come from the lane that holds
-// the other half.  K goes to the cache (and back into the row only when there is no cache), V is copied to the cache.
+// the other half.  K goes to the cache and, unless k_cache_only, back into the row; V is copied to the cache.
 template <typename T, int LPH>
 __global__ void __launch_bounds__(128) head_norm_rope_kernel(const UbRopeArgs a) {
   pdl_launch_dependents();
@@ -256,7 +256,7 @@ __global__ void __launch_bounds__(128) head_norm_rope_kernel(const UbRopeArgs a)
       }
     }
     if (!ok) continue;
-    if (h < a.Hq || a.k_cache == nullptr) store8(row + (long long)h * D + c * 8, v);
+    if (h < a.Hq || !a.k_cache_only || !slot_ok) store8(row + (long long)h * D + c * 8, v);
     if (h >= a.Hq && slot_ok && a.k_cache != nullptr)
       store8(reinterpret_cast<T*>(a.k_cache) + ((blk * a.Hkv + (h - a.Hq)) * a.block_size + off) * D + c * 8, v);
   }

@@ -78,6 +78,11 @@ def build_cuda(force: bool = False, verbose: bool = False, part: str = "serving"
     OBJ.mkdir(parents=True, exist_ok=True)
     nvcc = nvcc_path()
     srcs = cuda_sources(part)
+    deps = []
+    if part != "serving":
+        # the second library may use host functions of the first; they lie side by side
+        first = build_cuda(force=False, verbose=verbose)
+        deps = ["-L", str(OUT), f"-l:{first.name}", "-Xlinker", "-rpath=$ORIGIN"]
     hdr_m = _newest_header_mtime()
     lib = OUT / CUDA_LIBS[part]
     jobs = []
@@ -100,7 +105,7 @@ def build_cuda(force: bool = False, verbose: bool = False, part: str = "serving"
     if jobs or not lib.exists():
         # link beside the target and rename: a reader (another process, a snapshot) never sees a half-written library
         tmp = lib.with_suffix(".so.tmp")
-        _run([nvcc, "-shared", "-o", str(tmp), *map(str, objs), "-cudart", "static"])
+        _run([nvcc, "-shared", "-o", str(tmp), *map(str, objs), *deps, "-cudart", "static"])
         os.replace(tmp, lib)
     return lib
 

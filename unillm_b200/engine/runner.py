@@ -807,7 +807,7 @@ class GpuModelRunner:
                              self.v_cache[i] if own else None, num_q_heads=kh.hq, num_kv_heads=kh.hkv if own else 0,
                              head_dim=kh.dk, rotary_dim=ls.rotary_dim, pos_scale=s.rope_pos_scale,
                              interleaved=s.rope_interleaved, q_norm_w=t.get(L + "q_norm"), k_norm_w=t.get(L + "k_norm"),
-                             norm_eps=s.norm_eps, **kw)
+                             norm_eps=s.norm_eps, k_cache_only=own, **kw)
         self.launches += 1
 
     def _attention(self, i, qkv, lay, shared_prefix_len):

@@ -68,7 +68,7 @@ class UbRopeArgs(C.Structure):
         ("T", i32), ("Hq", i32), ("Hkv", i32), ("D", i32), ("rotary_dim", i32), ("block_size", i32),
         ("num_slots", i64), ("theta", f32), ("pos_scale", f32), ("norm_eps", f32), ("interleaved", i32),
         ("l3_factor", f32), ("l3_low_freq_factor", f32), ("l3_high_freq_factor", f32), ("l3_orig_ctx", f32),
-        ("inv_freq", vp), ("Dv", i32), ("norm_dim", i32), ("f32", i32),
+        ("inv_freq", vp), ("Dv", i32), ("norm_dim", i32), ("f32", i32), ("k_cache_only", i32),
     ]
 
 

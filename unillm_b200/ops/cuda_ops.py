@@ -305,12 +305,12 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
                    pos_scale: float = 1.0, interleaved: bool = False, q_norm_w: Optional[torch.Tensor] = None,
                    k_norm_w: Optional[torch.Tensor] = None, norm_eps: float = 1e-6,
                    llama3_scaling: Optional[Sequence[float]] = None, v_head_dim: Optional[int] = None,
-                   norm_dim: int = 0, inv_freq: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   norm_dim: int = 0, inv_freq: Optional[torch.Tensor] = None, k_cache_only: bool = False) -> torch.Tensor:
     """Rotates q and k inside ``qkv`` [T, (Hq+Hkv)*D + Hkv*Dv] in place and appends k, v to the paged cache.
 
     ``num_kv_heads = 0``: rows hold queries only (a layer that reads another layer's keys).  ``inv_freq`` (fp32
     [rotary_dim / 2]) replaces the frequencies that ``theta`` and the scaling give; ``norm_dim`` is the number of elements
-    the head norm averages over when heads are zero-padded."""
+    the head norm averages over when heads are zero-padded.  ``k_cache_only``: the rotated k is needed in the cache only."""
     f32 = _elem("rope_kv_append", qkv, k_cache, v_cache, q_norm_w, k_norm_w)
     if not qkv.is_contiguous():
         raise ValueError("qkv must be contiguous")
@@ -333,6 +333,7 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
     a.theta, a.pos_scale, a.norm_eps = theta, pos_scale, norm_eps
     a.interleaved = 1 if interleaved else 0
     a.Dv, a.norm_dim, a.f32 = v_head_dim or head_dim, norm_dim, int(f32)
+    a.k_cache_only = int(k_cache_only)
     if qkv.shape[1] != (num_q_heads + num_kv_heads) * head_dim + num_kv_heads * a.Dv:
         raise ValueError(f"rope_kv_append: rows of {qkv.shape[1]} elements do not hold these heads")
     if k_cache is not None and (k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]) != (num_kv_heads, head_dim, a.Dv):
