@@ -182,6 +182,20 @@ def reference_arm(args):
     return 0
 
 
+def design_bench(args) -> int:
+    import torch
+
+    torch.cuda.set_device(0)
+    from unillm_b200.benchmark import designs
+
+    sampler = ClockSampler(0)
+    sampler.prepare()
+    sampler.start()
+    rows = designs.main(args.design_sizes.split(",") if args.design_sizes else None, args.design_kernels)
+    print(json.dumps({"design": args.design, "dtype": "bf16", "data": "synthetic", "rows": rows, "clocks": sampler.stop()}))
+    return 0
+
+
 def _median(xs):
     xs = sorted(xs)
     n = len(xs)
@@ -214,9 +228,16 @@ def main(argv=None) -> int:
                     help="1 GPU: run the per-rank shapes of W-way tensor parallelism (heads, KV heads, MLP width and "
                          "vocabulary divided by W) without any communication -- the compute floor of one rank; "
                          "the token counts it prints are not a throughput of the full model")
+    ap.add_argument("--design", default=None, choices=["gekapel"],
+                    help="1 GPU: instead of the serving workload, prefill and decode steps of this design beside the closest "
+                         "existing family at equal size (random weights, a few layers)")
+    ap.add_argument("--design-sizes", default=None, help="--design: comma-separated subset of the sizes (1k,2k,4k)")
+    ap.add_argument("--design-kernels", action="store_true", help="--design: also every kernel of the steps against its roofline")
     args = ap.parse_args(argv)
     if args.impl == "reference":
         return reference_arm(args)
+    if args.design:
+        return design_bench(args)
     args.warmup = max(args.warmup, 3)
 
     import torch

@@ -1,0 +1,232 @@
+"""Prefill and decode throughput of one design beside the closest existing family at equal size, and the same
+comparison kernel by kernel (``python bench.py --design gekapel [--design-kernels]``).
+
+Both models are random-weight stacks of a few layers with a real model's layer sizes, run by the same
+``GpuModelRunner`` steps that serve requests: a prefill step is one batch of whole prompts, a decode step one token of
+every sequence at a given context through the captured CUDA graph.  Device time of a step is the CUDA-event interval
+around its launch (metadata upload, kernels, read-back of the samples); the layers' weights are larger than L2.
+
+The kernel table replays every call of one step alone (CUDA graph, L2 flushed between calls, ``microbench.time_ms``) and
+sets its time against the roofline of the call: the larger of its bytes over the copy bandwidth and its multiply-adds
+over the bf16 matrix throughput (MEASURED_PEAKS.json).
+
+The closest family to Gekapel is DeepSeek-MoE (routed experts plus always-on ones), here with Mistral's sliding window.
+Its experts have a gate, so at equal size they are two thirds as wide.
+"""
+from __future__ import annotations
+
+import contextlib
+import statistics
+from typing import Dict, List, Optional
+
+import torch
+
+from ..engine.runner import GpuModelRunner, RunnerWeights, StepBatch
+from ..models import configs as C
+from ..models.families import GekapelModel
+from ..models.spec import DecoderSpec, MoESpec
+from ..ops import cuda_ops as K
+from .microbench import _peaks, time_ms
+
+# per size: width, heads, kv heads, head dim, window, experts, top, expert width, shared width, vocabulary, layers
+SIZES = {
+    "1k": dict(width=1024, heads=16, kv=4, dim=64, window=256, experts=64, top=8, ff=384, shared=768, vocab=32000, layers=4),
+    "2k": dict(width=2048, heads=16, kv=4, dim=128, window=512, experts=32, top=4, ff=1536, shared=3072, vocab=32000, layers=4),
+    "4k": dict(width=4096, heads=32, kv=8, dim=128, window=1024, experts=16, top=2, ff=6144, shared=6144, vocab=32000, layers=4),
+}
+PREFILL = [(4, 2048), (1, 512)]            # (prompts, tokens each)
+DECODE = [(1, 2048), (32, 2048), (256, 2048)]   # (sequences, context)
+
+
+def gekapel_spec(z: dict) -> DecoderSpec:
+    layers = []
+    for i in range(z["layers"]):
+        mx = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "mask": {"size": z["window"]},
+              "rot": {"base": 10000.0, "dims": z["dim"] // 2,
+                      "scaling": {"factor": 4.0, "low": 1.0, "high": 4.0, "original": 4096}}, "scale": z["dim"] ** -0.5}
+        if i >= z["layers"] // 2:                       # the upper half reads the keys of the last layer that has some
+            mx["kv_from"] = z["layers"] // 2 - 1
+        layers.append({"type": "attention", "mixer": mx,
+                       "mlp": {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"]}, "expert": {"ff": z["ff"]},
+                               "shared": {"ff": z["shared"]}}})
+    return GekapelModel.spec_from_config(C.GekapelConfig(vocab_size=z["vocab"], hidden_size=z["width"],
+                                                         num_hidden_layers=z["layers"], layers=layers))
+
+
+def closest_spec(z: dict) -> DecoderSpec:
+    ff = z["ff"] * 2 // 3
+    return DecoderSpec(vocab_size=z["vocab"], hidden_size=z["width"], num_layers=z["layers"], num_heads=z["heads"],
+                       num_kv_heads=z["kv"], head_dim=z["dim"], intermediate_size=ff, max_position_embeddings=8192,
+                       window=z["window"],
+                       moe=MoESpec(num_experts=z["experts"], top_k=z["top"], intermediate_size=ff, num_shared_experts=1,
+                                   shared_intermediate_size=z["shared"] * 2 // 3))
+
+
+ARMS = {"gekapel": gekapel_spec, "deepseek_moe + window": closest_spec}
+
+
+def _runner(spec: DecoderSpec, tokens: int, max_len: int, seqs: int) -> GpuModelRunner:
+    w = RunnerWeights.random(spec, f"cuda:{torch.cuda.current_device()}", seed=7)
+    return GpuModelRunner(spec, w, num_blocks=tokens // 16 + 8, max_num_seqs=max(seqs, 8), max_num_batched_tokens=8192,
+                          max_model_len=max_len)
+
+
+def _batch(vocab: int, seqs: int, context: int, decode: bool, seed: int = 0) -> StepBatch:
+    """Whole prompts of ``context`` tokens, or one token of every sequence at position ``context - 1``."""
+    g = torch.Generator().manual_seed(seed)
+    nb = -(-context // 16)
+    tables = [list(range(s * nb, (s + 1) * nb)) for s in range(seqs)]
+    ids = torch.randint(0, vocab, (seqs * (1 if decode else context),), generator=g).tolist()
+    if decode:
+        pos = [context - 1] * seqs
+        slots = [t[-1] * 16 + (context - 1) % 16 for t in tables]
+        return StepBatch(ids, pos, slots, seqs, [context] * seqs, tables, [], list(range(seqs)))
+    pos = list(range(context)) * seqs
+    slots = [t[p // 16] * 16 + p % 16 for t in tables for p in range(context)]
+    return StepBatch(ids, pos, slots, 0, [context] * seqs, tables, [context] * seqs, [(s + 1) * context - 1 for s in range(seqs)])
+
+
+def step_ms(runner: GpuModelRunner, b: StepBatch, iters: int = 20, warmup: int = 4) -> Dict[str, float]:
+    for _ in range(warmup):
+        runner.execute(b)
+    times = []
+    for _ in range(iters):
+        torch.cuda.synchronize()
+        a, z = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        runner.launch(b)
+        z.record()
+        runner.fetch()
+        torch.cuda.synchronize()
+        times.append(a.elapsed_time(z))
+    return {"ms": round(statistics.median(times), 4), "ms_min": round(min(times), 4)}
+
+
+# ------------------------------------------------------------------------------------------------
+# kernel by kernel
+# ------------------------------------------------------------------------------------------------
+RECORDED = ("gemm_tn", "grouped_gemm", "norm", "residual_norm", "row_norm", "embed_residual", "embed_gather", "rope_kv_append",
+            "attn_decode", "attn_prefill", "moe_route", "moe_gather", "moe_combine", "sample")
+
+
+@contextlib.contextmanager
+def _record(calls: list):
+    """Collects the calls of the kernel front end made inside the block (outermost calls only)."""
+    saved = {n: getattr(K, n) for n in RECORDED}
+    depth = [0]
+
+    def wrap(name, fn):
+        def f(*a, **kw):
+            depth[0] += 1
+            try:
+                r = fn(*a, **kw)
+            finally:
+                depth[0] -= 1
+            if depth[0] == 0:
+                calls.append((name, fn, a, kw, r))
+            return r
+        return f
+
+    for n, fn in saved.items():
+        setattr(K, n, wrap(n, fn))
+    try:
+        yield
+    finally:
+        for n, fn in saved.items():
+            setattr(K, n, fn)
+
+
+def _nbytes(*ts) -> int:
+    return sum(t.numel() * t.element_size() for t in ts if isinstance(t, torch.Tensor))
+
+
+def _cost(name: str, a, kw, r, b: StepBatch, windows) -> tuple:
+    """(label, bytes moved, multiply-add flops) of one call, counting every operand once."""
+    if name == "gemm_tn":
+        x, w = a[0], a[1]
+        return (f"gemm {x.shape[0]}x{w.shape[0]}x{w.shape[1]}", _nbytes(x, w, r, kw.get("residual")),
+                2.0 * x.shape[0] * w.shape[0] * w.shape[1])
+    if name == "grouped_gemm":
+        x, w, rt = a[0], a[1], a[2]
+        used = min(w.shape[0], int((rt.counts > 0).sum()))
+        return (f"expert gemm {x.shape[0]}x{w.shape[1]}x{w.shape[2]} ({'up' if kw.get('act') else 'down'})",
+                _nbytes(x, r) + used * _nbytes(w[0]), 2.0 * x.shape[0] * w.shape[1] * w.shape[2])
+    if name in ("attn_decode", "attn_prefill"):
+        q, kc, vc = a[0], a[1], a[2]
+        win = kw.get("window") or 10 ** 9
+        lens = b.seq_lens
+        q_lens = [1] * b.num_decode + list(b.prefill_q_lens)
+        row = (kc.shape[3] + vc.shape[3]) * kc.shape[1] * kc.element_size()
+        keys = sum(min(n, win + ql - 1) for n, ql in zip(lens, q_lens))
+        pairs = 0
+        for n, ql in zip(lens, q_lens):
+            first = n - ql + 1
+            full = max(0, min(n, win) - first + 1) if first <= win else 0       # queries that see fewer keys than the window
+            pairs += full * (first + first + full - 1) // 2 + (ql - full) * min(n, win)
+        return name, _nbytes(q, r) + keys * row, 2.0 * pairs * q.shape[1] * (kc.shape[3] + vc.shape[3])
+    if name == "residual_norm":
+        x, y, ex = a[0], a[1], kw.get("experts")
+        return ("norm + residual" + (" + expert sum" if ex is not None else "")), _nbytes(x, x, y, ex, r), 0.0
+    if name == "moe_combine":
+        return "expert sum + residual", _nbytes(a[0], kw.get("residual"), r), 0.0
+    if name == "norm":
+        return "norm", _nbytes(a[0], r), 0.0
+    if name == "rope_kv_append":
+        q = kw["num_q_heads"] * kw["head_dim"] / a[0].shape[1]
+        kv = 1.0 - q
+        return "rope + append", int(_nbytes(a[0]) * (2 * q + 2 * kv)), 0.0
+    if name == "moe_route":
+        return "route + sort", _nbytes(a[0], a[1]), 2.0 * a[0].shape[0] * a[1].numel()
+    if name == "moe_gather":
+        return "gather", _nbytes(a[0], r), 0.0
+    ts = [t for t in (*a, *(r if isinstance(r, tuple) else (r,))) if isinstance(t, torch.Tensor)]
+    if name in ("embed_gather", "embed_residual"):
+        return "embedding", 2 * _nbytes(*(r if isinstance(r, tuple) else (r,))), 0.0
+    return name, _nbytes(*ts), 0.0
+
+
+def kernel_rows(runner: GpuModelRunner, b: StepBatch) -> List[dict]:
+    """One row per distinct kernel call of a step: calls, microseconds each, fraction of its roofline."""
+    hbm, tf, _ = _peaks()
+    calls: list = []
+    with _record(calls):
+        runner.forward_logits(b)
+    torch.cuda.synchronize()
+    rows: Dict[str, dict] = {}
+    for name, fn, a, kw, r in calls:
+        label, nbytes, flops = _cost(name, a, kw, r, b, None)
+        if label in rows:
+            rows[label]["calls"] += 1
+            continue
+        ms, _ = time_ms(lambda: fn(*a, **kw))
+        floor = max(nbytes / (hbm * 1e9), flops / (tf * 1e12)) * 1e6
+        rows[label] = {"kernel": label, "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2),
+                       "fraction": round(floor / (ms * 1e3), 3)}
+    return list(rows.values())
+
+
+def main(sizes: Optional[List[str]] = None, kernels: bool = False) -> List[dict]:
+    out = []
+    for size in sizes or list(SIZES):
+        z = SIZES[size]
+        for arm, make in ARMS.items():
+            spec = make(z)
+            tokens = max([n * c for n, c in PREFILL] + [n * c for n, c in DECODE])
+            runner = _runner(spec, tokens, max(c for _, c in PREFILL + DECODE) + 16, max(n for n, _ in DECODE))
+            for kind, cases in (("prefill", PREFILL), ("decode", DECODE)):
+                for n, c in cases:
+                    b = _batch(spec.vocab_size, n, c, kind == "decode")
+                    t = step_ms(runner, b)
+                    row = {"size": size, "model": arm, "layers": spec.num_layers, "params_m": round(runner.w.nbytes() / 2e6),
+                           "step": kind, "sequences": n, "context": c, **t,
+                           "tokens_per_s": round(len(b.token_ids) / t["ms"] * 1e3)}
+                    out.append(row)
+                    print(row, flush=True)
+                    if kernels:
+                        for k in kernel_rows(runner, b):
+                            out.append({"size": size, "model": arm, "step": kind, "sequences": n, "context": c, **k})
+                            print("   ", k, flush=True)
+            K.check_device_errors()
+            del runner
+            torch.cuda.empty_cache()
+    return out

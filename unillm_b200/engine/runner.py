@@ -360,6 +360,11 @@ class RunnerWeights:
                     gu[j, Ie:] = rnd(m.intermediate_size, H, c0, Ie)
                     dn[j] = rnd(H, m.intermediate_size, 0, H, c0, Ie)
                 self.t[L + "experts_gate_up"], self.t[L + "experts_down"] = gu, dn
+                if m.num_shared_experts:
+                    Is = m.shared_width // world
+                    r0 = rank * Is
+                    self.t[L + "shared_gate_up"] = torch.cat([rnd(m.shared_width, H, r0, Is) for _ in range(2 if m.gated else 1)], 0)
+                    self.t[L + "shared_down"] = rnd(H, m.shared_width, 0, H, r0, Is)
             else:
                 Is = I // world
                 g = rnd(I, H, rank * Is, Is)
