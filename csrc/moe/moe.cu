@@ -17,121 +17,188 @@ namespace ub {
 constexpr int MOE_MAX_E = 256;
 constexpr int MOE_MAX_K = 16;
 
-// One CTA of 128 threads per token: logits (from x and the router matrix, or given), top-k, weights.
-// XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.
-template <typename XT, typename WT>
+// Logits of TB tokens per CTA of 128 threads (from x and the router matrix, or given), then top-k and weights, one warp
+// per token.  XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.  A warp
+// takes four experts at a time for all TB tokens, so a router row is read once per TB tokens and an activation once per
+// four experts.  A logit's sum runs over h in the same order whatever TB is.
+template <typename XT, typename WT, int TB>
 __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) {
-  __shared__ float logit[MOE_MAX_E];
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int EB = 4;
+  __shared__ float logits_s[TB][MOE_MAX_E];
+  const int t0 = blockIdx.x * TB, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int E = a.E, K = a.K;
   if (a.router_w != nullptr) {
-    const XT* x = reinterpret_cast<const XT*>(a.x) + (long long)t * a.H;
+    const XT* x = reinterpret_cast<const XT*>(a.x);
     const WT* w = reinterpret_cast<const WT*>(a.router_w);
-    for (int e = warp; e < E; e += 4) {
-      const WT* we = w + (long long)e * a.H;
-      float acc = 0.f;
-      for (int h = lane * 8; h < a.H; h += 256) {
-        float xs[8], ws[8];
-        load8(x + h, xs);
-        load8(we + h, ws);
+    for (int e0 = warp * EB; e0 < E; e0 += 4 * EB) {
+      float acc[TB][EB];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) acc = fmaf(xs[j], ws[j], acc);
+      for (int i = 0; i < TB; ++i)
+#pragma unroll
+        for (int j = 0; j < EB; ++j) acc[i][j] = 0.f;
+      for (int h = lane * 8; h < a.H; h += 256) {
+        float ws[EB][8];
+#pragma unroll
+        for (int j = 0; j < EB; ++j) load8(w + (long long)min(e0 + j, E - 1) * a.H + h, ws[j]);
+#pragma unroll
+        for (int i = 0; i < TB; ++i) {
+          float xs[8];
+          load8(x + (long long)min(t0 + i, a.T - 1) * a.H + h, xs);
+#pragma unroll
+          for (int j = 0; j < EB; ++j)
+#pragma unroll
+            for (int c = 0; c < 8; ++c) acc[i][j] = fmaf(xs[c], ws[j][c], acc[i][j]);
+        }
       }
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-      if (a.router_b != nullptr) acc += (float)reinterpret_cast<const WT*>(a.router_b)[e];
-      // the reference model keeps router logits in the activation dtype: round like a bf16 linear layer would
-      if (lane == 0) logit[e] = a.round_logits_bf16 ? __bfloat162float(__float2bfloat16(acc)) : acc;
+      for (int i = 0; i < TB; ++i)
+#pragma unroll
+        for (int j = 0; j < EB; ++j) {
+          float v = warp_sum(acc[i][j]);
+          const int e = e0 + j;
+          if (e >= E) continue;
+          if (a.router_b != nullptr) v += (float)reinterpret_cast<const WT*>(a.router_b)[e];
+          // the reference model keeps router logits in the activation dtype: round like a bf16 linear layer would
+          if (lane == 0) logits_s[i][e] = a.round_logits_bf16 ? __bfloat162float(__float2bfloat16(v)) : v;
+        }
     }
   } else {
-    for (int e = threadIdx.x; e < E; e += 128)
-      logit[e] = a.logits_f32 ? reinterpret_cast<const float*>(a.logits)[(long long)t * E + e]
-                              : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.logits)[(long long)t * E + e]);
+    for (int i = threadIdx.x; i < TB * E; i += 128) {
+      const int t = t0 + i / E, e = i % E;
+      if (t >= a.T) continue;
+      logits_s[i / E][e] = a.logits_f32 ? reinterpret_cast<const float*>(a.logits)[(long long)t * E + e]
+                                        : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.logits)[(long long)t * E + e]);
+    }
   }
   __syncthreads();
-  if (warp != 0) return;
-  // Softmax statistics over all experts (used when the weights are not renormalised over the selection).
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, logit[e]);
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-  float den = 0.f;
-  for (int e = lane; e < E; e += 32) den += expf(logit[e] - mx);
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
-  uint32_t taken = 0;  // bit j: expert lane + 32*j already selected
-  float sel_l[MOE_MAX_K];
-  int sel_e[MOE_MAX_K];
-  for (int k = 0; k < K; ++k) {
-    float best = -INFINITY;
-    int bi = 0x7fffffff;
-    for (int e = lane, j = 0; e < E; e += 32, ++j) {
-      if (taken >> j & 1u) continue;
-      const float v = logit[e];
-      if (v > best || (v == best && e < bi)) { best = v; bi = e; }
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
-    }
-    if (bi < E && (bi & 31) == lane) taken |= 1u << (bi >> 5);
-    sel_l[k] = best;
-    sel_e[k] = bi < E ? bi : 0;
-  }
-  if (lane == 0) {
-    float s = 0.f;
-    for (int k = 0; k < K; ++k) { sel_l[k] = expf(sel_l[k] - mx); s += sel_l[k]; }
-    const float inv = a.norm_topk ? 1.f / s : 1.f / den;
+  for (int i = warp; i < TB; i += 4) {
+    const int t = t0 + i;
+    if (t >= a.T) continue;                       // warp-uniform
+    const float* logit = logits_s[i];
+    // Softmax statistics over all experts (used when the weights are not renormalised over the selection).
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, logit[e]);
+    mx = warp_max(mx);
+    float den = 0.f;
+    for (int e = lane; e < E; e += 32) den += expf(logit[e] - mx);
+    den = warp_sum(den);
+    uint32_t taken = 0;  // bit j: expert lane + 32*j already selected
+    float mine = 0.f;    // lane k keeps the k-th choice
+    int mine_e = 0;
     for (int k = 0; k < K; ++k) {
-      a.topk_ids[(long long)t * K + k] = sel_e[k];
-      a.topk_w[(long long)t * K + k] = sel_l[k] * inv * a.weight_scale;
+      float best = -INFINITY;
+      int bi = 0x7fffffff;
+      for (int e = lane, j = 0; e < E; e += 32, ++j) {
+        if (taken >> j & 1u) continue;
+        const float v = logit[e];
+        if (v > best || (v == best && e < bi)) { best = v; bi = e; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+      }
+      if (bi < E && (bi & 31) == lane) taken |= 1u << (bi >> 5);
+      if (lane == k) { mine = expf(best - mx); mine_e = bi < E ? bi : 0; }
+    }
+    const float s = warp_sum(lane < K ? mine : 0.f);
+    const float inv = a.norm_topk ? 1.f / s : 1.f / den;
+    if (lane < K) {
+      a.topk_ids[(long long)t * K + lane] = mine_e;
+      a.topk_w[(long long)t * K + lane] = mine * inv * a.weight_scale;
     }
   }
 }
 
 // One CTA: counts, exclusive offsets, slot assignment and the token-tile table of the grouped GEMM.
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const UbMoeRouteArgs a) {
-  __shared__ int cnt[MOE_MAX_E], off[MOE_MAX_E + 1], cur[MOE_MAX_E];
+  __shared__ int cnt[MOE_MAX_E], off[MOE_MAX_E + 1], first_tile[MOE_MAX_E + 1];
   const int E = a.num_local_experts > 0 ? a.num_local_experts : a.E, n = a.T * a.K;
-  for (int e = threadIdx.x; e < E; e += blockDim.x) { cnt[e] = 0; cur[e] = 0; }
+  for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
   // Expert parallelism: only experts [expert_lo, expert_lo + E) live on this rank; the rest get no slot.
   const int lo = a.expert_lo;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const int e = a.topk_ids[i] - lo;
-    if (e >= 0 && e < E) atomicAdd(&cnt[e], 1);
-  }
-  __syncthreads();
-  if (threadIdx.x == 0) {
-    int acc = 0, tile = 0;
-    int4* tiles = reinterpret_cast<int4*>(a.tiles);
-    for (int e = 0; e < E; ++e) {
-      off[e] = acc;
-      if (tiles != nullptr) {
-        for (int r = 0; r < cnt[e] && tile < a.max_tiles; r += a.tile_tokens, ++tile)
-          tiles[tile] = make_int4(e, acc + r, acc + cnt[e], 0);
-      }
-      acc += cnt[e];
+  constexpr int U = 4;                            // ids in flight per thread
+  for (int i0 = threadIdx.x; i0 < n; i0 += U * blockDim.x) {
+    int id[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * blockDim.x;
+      id[u] = i < n ? a.topk_ids[i] - lo : -1;
     }
-    off[E] = acc;
-    if (tiles != nullptr)
-      for (; tile < a.max_tiles; ++tile) tiles[tile] = make_int4(-1, 0, 0, 0);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * blockDim.x;
+      if (i >= n) continue;
+      // the place among the expert's rows, kept in row_slot until the offsets are known
+      a.row_slot[i] = id[u] >= 0 && id[u] < E ? atomicAdd(&cnt[id[u]], 1) : -1;
+    }
   }
   __syncthreads();
+  const int tile = a.tiles != nullptr ? a.tile_tokens : 1;
+  if (threadIdx.x < 32) {
+    // exclusive sums of the rows and of the tiles, a warp of experts at a time
+    int acc = 0, tacc = 0;
+    for (int e0 = 0; e0 < E; e0 += 32) {
+      const int e = e0 + threadIdx.x, c = e < E ? cnt[e] : 0, tc = (c + tile - 1) / tile;
+      int s = c, ts = tc;
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const int v = __shfl_up_sync(0xffffffffu, s, o), tv = __shfl_up_sync(0xffffffffu, ts, o);
+        if ((int)threadIdx.x >= o) { s += v; ts += tv; }
+      }
+      if (e < E) { off[e] = acc + s - c; first_tile[e] = tacc + ts - tc; }
+      acc += __shfl_sync(0xffffffffu, s, 31);
+      tacc += __shfl_sync(0xffffffffu, ts, 31);
+    }
+    if (threadIdx.x == 0) { off[E] = acc; first_tile[E] = tacc; }
+  }
+  __syncthreads();
+  if (a.tiles != nullptr) {
+    int4* tiles = reinterpret_cast<int4*>(a.tiles);
+    const int used = min(first_tile[E], a.max_tiles);
+    for (int i = threadIdx.x; i < a.max_tiles; i += blockDim.x) {
+      int4 t = make_int4(-1, 0, 0, 0);
+      if (i < used) {
+        int l = 0, r = E - 1;                     // the last expert whose first tile is <= i and that has tiles
+        while (l < r) {
+          const int m = (l + r + 1) >> 1;
+          if (first_tile[m] <= i) l = m; else r = m - 1;
+        }
+        t = make_int4(l, off[l] + (i - first_tile[l]) * tile, off[l] + cnt[l], 0);
+      }
+      tiles[i] = t;
+    }
+  }
   for (int e = threadIdx.x; e <= E; e += blockDim.x) {
     a.expert_offsets[e] = off[e];
     if (e < E) a.expert_counts[e] = cnt[e];
   }
-  for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    const int e = a.topk_ids[i] - lo;
-    if (e < 0 || e >= E) { a.row_slot[i] = -1; continue; }
-    const int slot = off[e] + atomicAdd(&cur[e], 1);
-    a.sorted_rows[slot] = i;
-    a.row_slot[i] = slot;
+  for (int i0 = threadIdx.x; i0 < n; i0 += U * blockDim.x) {
+    int id[U], place[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * blockDim.x;
+      place[u] = -1;
+      if (i < n) { id[u] = a.topk_ids[i] - lo; place[u] = a.row_slot[i]; }
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * blockDim.x;
+      if (place[u] < 0) continue;
+      const int slot = off[id[u]] + place[u];
+      a.sorted_rows[slot] = i;
+      a.row_slot[i] = slot;
+    }
   }
   for (int i = off[E] + threadIdx.x; i < n; i += blockDim.x) a.sorted_rows[i] = -1;   // unused tail
+}
+
+template <typename XT, typename WT>
+static void launch_route(const UbMoeRouteArgs& a, cudaStream_t st) {
+  if (a.T >= 148 * 8) moe_route_kernel<XT, WT, 4><<<(a.T + 3) / 4, 128, 0, st>>>(a);
+  else moe_route_kernel<XT, WT, 1><<<a.T, 128, 0, st>>>(a);
 }
 
 // out[slot, :] = x[sorted_rows[slot] / K, :]; V 16-byte vectors per 8 bf16 / 4 fp32 elements
@@ -383,10 +450,10 @@ extern "C" int ub_moe_route(const UbMoeRouteArgs* a, void* stream_v) {
   if (a->tiles != nullptr && (a->tile_tokens <= 0 || a->max_tiles <= 0)) return -4;
   UbMoeRouteArgs b = *a;
   if (b.weight_scale == 0.f) b.weight_scale = 1.f;
-  if (b.router_w != nullptr && b.x_f32 && b.router_f32) ub::moe_route_kernel<float, float><<<a->T, 128, 0, st>>>(b);
-  else if (b.router_w != nullptr && b.x_f32) ub::moe_route_kernel<float, __nv_bfloat16><<<a->T, 128, 0, st>>>(b);
-  else if (b.router_w != nullptr && b.router_f32) ub::moe_route_kernel<__nv_bfloat16, float><<<a->T, 128, 0, st>>>(b);
-  else ub::moe_route_kernel<__nv_bfloat16, __nv_bfloat16><<<a->T, 128, 0, st>>>(b);
+  if (b.router_w != nullptr && b.x_f32 && b.router_f32) ub::launch_route<float, float>(b, st);
+  else if (b.router_w != nullptr && b.x_f32) ub::launch_route<float, __nv_bfloat16>(b, st);
+  else if (b.router_w != nullptr && b.router_f32) ub::launch_route<__nv_bfloat16, float>(b, st);
+  else ub::launch_route<__nv_bfloat16, __nv_bfloat16>(b, st);
   ub::moe_sort_kernel<<<1, 1024, 0, st>>>(b);
   cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;

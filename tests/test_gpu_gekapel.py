@@ -126,10 +126,10 @@ def test_head_norm_rotation_and_append(dtype, Hq, Hkv, dim, vdim, dims, scaled):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("E,top,H,bias", [(5, 2, 96, True), (7, 7, 56, True), (1, 1, 8, True), (64, 8, 1024, True), (256, 16, 64, False)])
-def test_router(dtype, E, top, H, bias):
+@pytest.mark.parametrize("T", [1, 21, 1501])
+def test_router(dtype, E, top, H, bias, T):
     from unillm_b200.ops import cuda_ops as K
 
-    T = 21
     x, w = _rand(T, H, seed=1, dtype=torch.float32, scale=2.0), _rand(E, H, seed=2, scale=H ** -0.5)
     b = _rand(E, seed=3) if bias else torch.zeros(E)
     idx, wt = P.route(x.double(), w.double(), b.double(), top)
@@ -137,6 +137,14 @@ def test_router(dtype, E, top, H, bias):
     got = torch.zeros(T, E, dtype=torch.float64).scatter_(1, r.topk_ids.cpu().long(), r.topk_w.cpu().double())
     want = torch.zeros(T, E, dtype=torch.float64).scatter_(1, idx, wt)
     assert (got - want).abs().max() < 1e-5
+    # expert order: every (token, choice) pair has a slot of its own inside its expert's rows, covered by the tile table
+    ids, slot, off = r.topk_ids.cpu().flatten().long(), r.row_slot.cpu().long(), r.offsets.cpu().long()
+    assert torch.equal(slot.sort().values, torch.arange(T * top)) and torch.equal(r.sorted_rows.cpu().long()[slot], torch.arange(T * top))
+    assert ((slot >= off[ids]) & (slot < off[ids + 1])).all()
+    assert torch.equal(r.counts.cpu().long(), torch.bincount(ids, minlength=E))
+    tiles = [t for t in r.tiles.cpu().tolist() if t[0] >= 0]
+    covered = [(e, x) for e, a, z, _ in tiles for x in range(a, min(z, a + r.tile_tokens))]
+    assert len(covered) == T * top and all(off[e] <= x < off[e + 1] for e, x in covered)
     K.check_device_errors()
 
 
