@@ -44,6 +44,16 @@ def test_model_directory_loads_and_exports(tmp_path, case):
     assert all(torch.equal(out[n].float(), t.float()) for n, t in w.items())
 
 
+def test_cache_cost_counts_only_layers_with_keys(case):
+    from unillm_b200.scheduler.policies import KvShape
+
+    cfg, _, m, _, _ = case
+    per_token = sum(x["mixer"]["kv_heads"] * (x["mixer"]["dim"] + x["mixer"]["vdim"]) for x in cfg["layers"]
+                    if x["mixer"].get("kv_from") is None)
+    assert KvShape.from_spec(m.spec).bytes_per_token() == 2 * per_token
+    assert m.memory_requirements().kv_cache_memory == 2 * per_token * m.spec.max_position_embeddings
+
+
 def test_bad_configurations_are_refused():
     from unillm_b200.types import ConfigurationError
 

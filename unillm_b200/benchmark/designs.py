@@ -140,7 +140,7 @@ def _nbytes(*ts) -> int:
     return sum(t.numel() * t.element_size() for t in ts if isinstance(t, torch.Tensor))
 
 
-def _cost(name: str, a, kw, r, b: StepBatch, windows) -> tuple:
+def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
     """(label, bytes moved, multiply-add flops) of one call, counting every operand once."""
     if name == "gemm_tn":
         x, w = a[0], a[1]
@@ -181,7 +181,10 @@ def _cost(name: str, a, kw, r, b: StepBatch, windows) -> tuple:
         return "gather", _nbytes(a[0], r), 0.0
     ts = [t for t in (*a, *(r if isinstance(r, tuple) else (r,))) if isinstance(t, torch.Tensor)]
     if name in ("embed_gather", "embed_residual"):
-        return "embedding", 2 * _nbytes(*(r if isinstance(r, tuple) else (r,))), 0.0
+        rs = r if isinstance(r, tuple) else (r,)
+        return "embedding", _nbytes(*rs) + _nbytes(rs[-1]), 0.0
+    if name == "row_norm":
+        return "row norm", _nbytes(r) + 4 * r.numel(), 0.0
     return name, _nbytes(*ts), 0.0
 
 
@@ -194,7 +197,7 @@ def kernel_rows(runner: GpuModelRunner, b: StepBatch) -> List[dict]:
     torch.cuda.synchronize()
     rows: Dict[str, dict] = {}
     for name, fn, a, kw, r in calls:
-        label, nbytes, flops = _cost(name, a, kw, r, b, None)
+        label, nbytes, flops = _cost(name, a, kw, r, b)
         if label in rows:
             rows[label]["calls"] += 1
             continue

@@ -49,13 +49,16 @@ def cmd_generate(a) -> int:
     from .config import GenerationConfig
     from .pipeline import InferencePipelineBuilder
 
+    import torch
+
     cuda = a.device.startswith("cuda")
     # for a GPU run the weights are loaded on the host and handed to the kernel runner, which keeps its own bf16
     # copy in kernel layout on the device; a model the runner does not cover is moved to the device as a whole
     model = _load(a.model, "cpu" if cuda else a.device)
     b = InferencePipelineBuilder().model(model).use_engine(a.engine)
     if cuda:
-        b = b.device(a.device).engine_options(max_num_seqs=8, max_num_batched_tokens=2048, quantize=a.quantize)
+        b = b.device(a.device).engine_options(max_num_seqs=8, max_num_batched_tokens=2048, quantize=a.quantize,
+                                             dtype=getattr(torch, a.dtype))
     pipe = b.build()
     if cuda:
         if pipe.engine_note is None:
@@ -143,6 +146,8 @@ def build_parser() -> argparse.ArgumentParser:
     g.add_argument("--engine", action="store_true", help="run on the paged continuous-batching engine")
     g.add_argument("--quantize", default=None, choices=["q4_k", "q8_0", "q4_0"],
                    help="--device cuda: keep the projection weights block-quantised on the device")
+    g.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"],
+                   help="--device cuda: float32 runs weights, cache and arithmetic in 32 bits (models with a 32-bit residual stream)")
     g.add_argument("--stream", action="store_true")
     g.set_defaults(fn=cmd_generate)
     m = sub.add_parser("models", help="list architectures and cached models")

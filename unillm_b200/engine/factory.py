@@ -84,6 +84,8 @@ def build_engine(model, *, device="cuda", max_num_seqs: int = 64, max_num_batche
     spec = model.spec
     if max_model_len is None:
         max_model_len = min(spec.max_position_embeddings, 8192)
+    if quantize and dtype != torch.bfloat16:
+        raise UnsupportedOperation("block-quantised weights go with bf16 arithmetic")
     weights = RunnerWeights(spec, model.p, dev, rank, world, dtype=dtype)
     if quantize:
         weights.quantize(quantize)

@@ -1,4 +1,4 @@
-"""Configuration classes of all 47 architectures.
+"""Configuration classes of all architectures: the reference's 47, and Gekapel.
 
 Field names and defaults follow the reference's ``model_config!`` blocks one for one
 (``crates/runtime/src/models_v2/<family>.rs``, e.g. ``llama.rs:20-38``, ``mixtral.rs:16-38``), so a

@@ -165,6 +165,11 @@ class DecoderSpec:
         return self.moe is not None and i >= self.moe.first_k_dense
 
     @property
+    def kv_elements_per_token(self) -> int:
+        """Cache elements that one token takes over all layers that own keys and values."""
+        return sum(self.layer(i).k_size + self.layer(i).v_size for i in self.kv_layers)
+
+    @property
     def kv_layers(self) -> Tuple[int, ...]:
         """Layers that own keys and values (the others read one of these)."""
         return tuple(i for i in range(self.num_layers) if self.layer(i).kv_from is None)

@@ -39,15 +39,24 @@ class SchedulingPolicy(enum.Enum):
 
 @dataclass
 class KvShape:
-    """What one cached token costs: 2 (K,V) * layers * kv_heads * head_dim * bytes."""
+    """What one cached token costs: 2 (K,V) * layers * kv_heads * head_dim * bytes, or ``elements`` * bytes where the layers
+    differ (``from_spec``)."""
 
     num_layers: int = 32
     num_kv_heads: int = 32
     head_dim: int = 128
     dtype_bytes: int = 2
     tp: int = 1
+    elements: Optional[int] = None
+
+    @classmethod
+    def from_spec(cls, spec, dtype_bytes: int = 2, tp: int = 1) -> "KvShape":
+        return cls(spec.num_layers, spec.num_kv_heads, spec.head_dim, dtype_bytes, tp,
+                   spec.kv_elements_per_token if spec.layers is not None else None)
 
     def bytes_per_token(self) -> int:
+        if self.elements is not None:
+            return -(-self.elements // self.tp) * self.dtype_bytes
         return 2 * self.num_layers * max(1, self.num_kv_heads // self.tp) * self.head_dim * self.dtype_bytes
 
 
