@@ -81,7 +81,7 @@ def test_embed_residual_and_bad_ids(dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("Hq,Hkv,dim,vdim,dims", [(4, 2, 64, 64, 16), (6, 2, 32, 48, 8), (5, 5, 20, 12, 6), (3, 1, 40, 24, 40),
+@pytest.mark.parametrize("Hq,Hkv,dim,vdim,dims", [(6, 3, 64, 64, 24), (6, 2, 32, 48, 8), (5, 5, 20, 12, 6), (3, 1, 40, 24, 40),
                                                   (2, 1, 128, 96, 64), (2, 1, 192, 256, 2), (1, 1, 16, 8, 0), (18, 1, 72, 136, 72)])
 @pytest.mark.parametrize("scaled", [True, False])
 def test_head_norm_rotation_and_append(dtype, Hq, Hkv, dim, vdim, dims, scaled):
@@ -208,7 +208,7 @@ def _paged(lens, Hkv, dim, vdim, dtype, bs=16, seed=0):
     return kc, vc, bt, ks, vs, dev
 
 
-SIZES = [(4, 2, 64, 64), (4, 1, 128, 128), (6, 2, 32, 48), (5, 5, 24, 16), (18, 1, 72, 136), (2, 1, 192, 256), (4, 2, 256, 64), (3, 3, 8, 200)]
+SIZES = [(6, 2, 64, 64), (4, 1, 128, 128), (6, 2, 32, 48), (5, 5, 24, 16), (18, 1, 72, 136), (2, 1, 192, 256), (4, 2, 256, 64), (3, 3, 8, 200)]
 
 
 def _plant(k, q, pos, h, g, scale):
