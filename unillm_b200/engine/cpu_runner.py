@@ -6,10 +6,12 @@ Works on any torch device; every op is a plain torch op.
 """
 from __future__ import annotations
 
-from typing import List, Optional
+import copy
+from typing import Dict, List, Optional
 
 import torch
 
+from ..models import mixers as MX
 from ..models.decoder import DecoderModel
 from ..precompute import alibi_slopes, apply_rope
 from ..sampling import Sampler, SamplingParams
@@ -30,8 +32,10 @@ class CpuModelRunner:
                 self.k_cache.append(self.k_cache[ls.kv_from])
                 self.v_cache.append(self.v_cache[ls.kv_from])
                 continue
-            for cache, d in ((self.k_cache, ls.head_dim), (self.v_cache, ls.v_head_dim)):
-                cache.append(torch.zeros(num_blocks, ls.num_kv_heads, block_size, d, dtype=dt, device=dev))
+            heads, dk, dv = (1, ls.cache_row, 0) if ls.mixer == "latent" else (ls.num_kv_heads, ls.head_dim, ls.v_head_dim)
+            for cache, d in ((self.k_cache, dk), (self.v_cache, dv)):
+                cache.append(torch.zeros(num_blocks, heads, block_size, d, dtype=dt, device=dev) if ls.has_kv else None)
+        self.states: Dict[int, List[dict]] = {}         # state row -> what each layer carries on
         self._alibi = alibi_slopes(s.num_heads).to(dev) if s.pos == "alibi" else None
         self.launches = 0
         self.h2d_bytes = self.d2h_bytes = 0
@@ -41,12 +45,17 @@ class CpuModelRunner:
         s, m, ls = self.spec, self.model, self.spec.layer(i)
         L = f"layers.{i}."
         T = h.shape[0]
-        q, k, v = m._project_qkv(i, h)
-        if ls.rotary_dim > 0:
-            cos, sin = m._rope_cache(int(pos.max()) + 1, ls).at(pos)
-            q = apply_rope(q, cos, sin, ls.rotary_dim, s.rope_interleaved)
-            if k is not None:
-                k = apply_rope(k, cos, sin, ls.rotary_dim, s.rope_interleaved)
+        rope = m._rope_cache(int(pos.max()) + 1, ls).at(pos) if ls.rotary_dim > 0 else None
+        latent = ls.mixer == "latent"
+        if latent:
+            q, rows = m._latent_rows(i, h, rope)
+            k, v = rows[:, None], rows[:, None, :0]
+        else:
+            q, k, v = m._project_qkv(i, h)
+            if rope is not None:
+                q = apply_rope(q, *rope, ls.rotary_dim, s.rope_interleaved)
+                if k is not None:
+                    k = apply_rope(k, *rope, ls.rotary_dim, s.rope_interleaved)
         if k is not None:
             ok = slots >= 0
             blk, off = slots[ok] // self.block_size, slots[ok] % self.block_size
@@ -59,8 +68,11 @@ class CpuModelRunner:
             kv_len = b.seq_lens[si]
             bt = torch.as_tensor(b.block_tables[si][: (kv_len + self.block_size - 1) // self.block_size],
                                  device=h.device, dtype=torch.long)
-            kk = self.k_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.head_dim)[:, :kv_len]
-            vv = self.v_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.v_head_dim)[:, :kv_len]
+            if latent:
+                kk, vv = MX.latent_expand(m.p, L, ls, self.k_cache[i][bt][:, 0].flatten(0, 1)[:kv_len])
+            else:
+                kk = self.k_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.head_dim)[:, :kv_len]
+                vv = self.v_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.v_head_dim)[:, :kv_len]
             qq = q[row:row + ql].transpose(0, 1).float()              # [H, ql, D]
             qpos = torch.arange(kv_len - ql, kv_len, device=h.device)[:, None]
             kpos = torch.arange(kv_len, device=h.device)[None, :]
@@ -74,6 +86,18 @@ class CpuModelRunner:
             out[row:row + ql] = y.transpose(0, 1).to(h.dtype)
             row += ql
         return ops_fn.linear(out.reshape(T, ls.o_size), m.p[L + "wo"], m.p.get(L + "bo"))
+
+    def _per_sequence(self, h: torch.Tensor, b: StepBatch, st: List[dict], fn) -> torch.Tensor:
+        """``fn(rows [1, n, H], state)`` on the rows of each sequence of the step."""
+        out = [fn(x[None], st[si])[0] for si, x in enumerate(h.split([1] * b.num_decode + list(b.prefill_q_lens)))]
+        return torch.cat(out)
+
+    def _mixer(self, i: int, h: torch.Tensor, b: StepBatch, pos, slots, st: List[dict]) -> torch.Tensor:
+        ls, m, L = self.spec.layer(i), self.model, f"layers.{i}."
+        if ls.mixer == "wkv":
+            y = self._per_sequence(h, b, st, lambda x, d: MX.wkv(m.p, L, ls, x, d, self.spec.norm_eps))
+            return ops_fn.linear(y, m.p[L + "wo"])
+        return self._attention(i, h, b, pos, slots)
 
     @torch.no_grad()
     def forward_logits(self, b: StepBatch) -> torch.Tensor:
@@ -91,8 +115,17 @@ class CpuModelRunner:
             x = x + m.p["pos_embed"][pos + s.learned_pos_offset]
         if s.embed_norm:
             x = ops_fn.layer_norm(x, m.p["embed_norm.w"], m.p["embed_norm.b"], s.norm_eps)
+        nseq = len(b.seq_lens)
+        read = b.state_in if b.state_in is not None else [-1] * nseq
+        states = [copy.deepcopy(self.states[r]) if r >= 0 else [{} for _ in range(s.num_layers)] for r in read]
         for i in range(s.num_layers):
-            x = m.block(i, x[None], lambda h, i=i: self._attention(i, h[0], b, pos, slots)[None])[0]
+            st = [d[i] for d in states]
+            conv = lambda h, n, i=i, st=st: self._per_sequence(
+                h[0], b, st, lambda y, d: MX.input_conv(y, m.p[f"layers.{i}.{n}"], d, n))[None]
+            x = m.block(i, x[None], lambda h, i=i, st=st: self._mixer(i, h[0], b, pos, slots, st)[None], conv)[0]
+        for w, d in zip(b.state_out or (), states):
+            if w >= 0:
+                self.states[w] = d
         rows = torch.as_tensor(b.sample_rows, dtype=torch.long, device=dev)
         xs = x[rows]
         if s.final_norm:
@@ -156,7 +189,6 @@ class TpCpuModelRunner(CpuModelRunner):
 
     def __init__(self, model: DecoderModel, rank: int, world: int, group=None, *, num_blocks: int, block_size: int = 16,
                  max_model_len: int = 8192):
-        import copy
         import dataclasses
 
         from .runner import RunnerWeights

@@ -35,6 +35,7 @@ from dataclasses import dataclass, field
 from typing import Callable, Deque, Dict, List, Optional, Sequence, Tuple
 
 from ..kv.block_pool import BlockPool, RadixTree
+from ..kv.state_slots import StateSlots
 from ..sampling import SamplingParams
 from ..types import InvalidInput, MemoryError_
 from .runner import DeviceStepError, StepBatch
@@ -63,6 +64,7 @@ class Sequence:
     preemptions: int = 0
     pending_src: int = -1            # sample index, in the step in flight, of the token that output_ids[pending_at] awaits
     pending_at: int = -1
+    state_slot: int = -1             # recurrent models: the slot of its carried state, -1 = none yet
     _blocks_np: Optional[object] = field(default=None, repr=False)
 
     def blocks_array(self):
@@ -116,7 +118,10 @@ class LLMEngine:
         self.runner = runner
         self.block_size = block_size
         self.pool = BlockPool(num_blocks, block_size)
-        self.radix = RadixTree(self.pool) if enable_prefix_caching else None
+        # a model with carried state cannot start behind a cached prefix: the blocks hold keys, not the state at their end
+        stateful = bool(getattr(getattr(runner, "spec", None), "has_state", False))
+        self.slots = StateSlots(max_num_seqs) if stateful else None
+        self.radix = RadixTree(self.pool) if enable_prefix_caching and not stateful else None
         self.max_num_seqs, self.max_tokens, self.max_model_len = max_num_seqs, max_num_batched_tokens, max_model_len
         self.chunked = enable_chunked_prefill
         self.eos_token_id = eos_token_id
@@ -193,6 +198,9 @@ class LLMEngine:
             self.radix.unlock(s.radix_node)
         s.radix_node = 0
         s.published_blocks = 0
+        if s.state_slot >= 0:
+            self.slots.free(s.state_slot)
+            s.state_slot = -1
 
     def _publish(self, s: Sequence, upto_tokens: int) -> None:
         """Offer the blocks that are completely filled by the first ``upto_tokens`` tokens to the radix tree."""
@@ -290,7 +298,7 @@ class LLMEngine:
         if self.policy is not None:
             order = self.policy(order)
         for s in order:
-            if budget <= 0 or len(self.running) >= self.max_num_seqs:
+            if budget <= 0 or len(self.running) + len(self.scored) >= self.max_num_seqs:
                 break
             self._admit(s)
             remaining = s.total_len - s.num_computed
@@ -368,7 +376,15 @@ class LLMEngine:
             seq_lens.append(b)
             tables.append(s.blocks_array())
             q_lens.append(n)
-        return StepBatch(token_ids, positions, slots, len(decode), seq_lens, tables, q_lens, token_src=token_src)
+        batch = StepBatch(token_ids, positions, slots, len(decode), seq_lens, tables, q_lens, token_src=token_src)
+        if self.slots is not None:
+            batch.state_in, batch.state_out = [], []
+            for s in decode + [s for s, _ in chunks]:
+                if s.state_slot < 0:
+                    s.state_slot = self.slots.allocate()
+                a, b = self.slots.advance(s.state_slot, fresh=s.num_computed == 0)
+                batch.state_in.append(a), batch.state_out.append(b)
+        return batch
 
     def _ensure_blocks_no_preempt(self, s: Sequence, upto_tokens: int) -> bool:
         need = (upto_tokens + self.block_size - 1) // self.block_size - len(s.blocks)

@@ -77,6 +77,10 @@ class StepBatch:
     # when ``token_ids`` already holds it.  Lets a step be launched before the host has read the previous
     # step's samples.
     token_src: Optional[List[int]] = None
+    # recurrent models, per sequence (decode rows, then prefill chunks): rows of the state tensors to read (-1: the
+    # sequence starts, zero state) and to write (-1: none)
+    state_in: Optional[List[int]] = None
+    state_out: Optional[List[int]] = None
 
 
 def shard_rows(w: torch.Tensor, rank: int, world: int) -> torch.Tensor:
@@ -566,6 +570,9 @@ class StepPacker:
         for ql in q_lens:
             qs.append(qs[-1] + ql)
         put("q_start", qs)
+        if b.state_in is not None:
+            for name, v in (("state_in", b.state_in), ("state_out", b.state_out)):
+                put(name, list(v[:D]) + [-1] * pad + list(v[D:]) + [-1] * (Pp - P))
         if bucketed:
             rows = list(range(Dp)) + [Dp + max(qs[j + 1] - 1, 0) for j in range(Pp)]
             sel = []

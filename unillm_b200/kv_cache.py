@@ -10,7 +10,7 @@ The serving engine uses the paged cache in ``unillm_b200.kv`` instead.
 """
 from __future__ import annotations
 
-from typing import List, Optional, Tuple
+from typing import Dict, List, Optional, Tuple
 
 import torch
 
@@ -24,6 +24,7 @@ class LayerKVCache:
         self.max_seq_len = max_seq_len
         self.k: Optional[torch.Tensor] = None
         self.v: Optional[torch.Tensor] = None
+        self.state: Dict[str, torch.Tensor] = {}     # what a recurrent layer or an input convolution carries on
         self.len = 0
 
     def is_allocated(self) -> bool:
@@ -50,16 +51,19 @@ class LayerKVCache:
         return self.len
 
     def clear(self) -> None:
+        self.state = {}
         self.len = 0
 
     def deallocate(self) -> None:
         self.k = self.v = None
+        self.state = {}
         self.len = 0
 
     def memory_bytes(self) -> int:
+        state = sum(t.numel() * t.element_size() for t in self.state.values())
         if self.k is None:
-            return 0
-        return self.k.numel() * self.k.element_size() + self.v.numel() * self.v.element_size()
+            return state
+        return state + self.k.numel() * self.k.element_size() + self.v.numel() * self.v.element_size()
 
 
 class KVCache:

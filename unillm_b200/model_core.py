@@ -295,7 +295,7 @@ class Model:
             kv = 2 * c.num_hidden_layers * nkv * hd * ctx * 2
         spec = getattr(self, "spec", None)
         if getattr(spec, "layers", None) is not None:      # layers differ: the spec knows what a token takes
-            kv = 2 * spec.kv_elements_per_token * spec.max_position_embeddings
+            kv = 2 * spec.kv_elements_per_token * spec.max_position_embeddings + 4 * spec.state_elements
         on_gpu = self.device.type == "cuda"
         return MemoryRequirements(gpu_memory=nbytes if on_gpu else 0, cpu_memory=0 if on_gpu else nbytes,
                                   kv_cache_memory=kv, peak_memory=nbytes + kv + nbytes // 10)

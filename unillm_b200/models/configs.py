@@ -1,4 +1,4 @@
-"""Configuration classes of all architectures: the reference's 47, and Gekapel.
+"""Configuration classes of all architectures: the reference's 47, Gekapel and Nipulorn.
 
 Field names and defaults follow the reference's ``model_config!`` blocks one for one
 (``crates/runtime/src/models_v2/<family>.rs``, e.g. ``llama.rs:20-38``, ``mixtral.rs:16-38``), so a
@@ -334,6 +334,33 @@ class GekapelConfig:
         kw = {k: d[k] for k in ("max_position_embeddings", "initializer_range") if k in d}
         return cls(vocab_size=d["vocab"], hidden_size=d["width"], num_hidden_layers=len(d["layers"]),
                    norm_eps=d["norm"]["eps"], layers=list(d["layers"]), **kw)
+
+
+@model_config
+class NipulornConfig:
+    """Nipulorn: every layer is described on its own.  ``layers[i]`` holds ``type`` ("wkv" or "latent_attention"), ``mixer``
+    (heads and dim; latent attention also vdim, q_rank, kv_rank, rot_dim, scale and rot.{base, dims, scaling}) and ``mlp``
+    (ff, or null for a layer without a feed-forward)."""
+
+    vocab_size: int = 32000
+    hidden_size: int = 2048
+    num_hidden_layers: int = 0
+    norm_eps: float = 1e-5
+    embedding_scale: float = 1.0
+    logit_scale: float = 1.0
+    canon_taps: int = 4
+    layers: List[Any] = []
+    max_position_embeddings: int = 131072
+    initializer_range: float = 0.02
+
+    @classmethod
+    def from_hf_config(cls, d):
+        if "layers" not in d or "width" not in d:
+            return super(NipulornConfig, cls).from_hf_config(d)
+        kw = {k: d[k] for k in ("max_position_embeddings", "initializer_range") if k in d}
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], num_hidden_layers=len(d["layers"]), norm_eps=d["norm"]["eps"],
+                   embedding_scale=d["embedding"]["scale"], logit_scale=d["logit_scale"], canon_taps=d["canon"]["taps"],
+                   layers=list(d["layers"]), **kw)
 
 
 @model_config

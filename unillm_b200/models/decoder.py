@@ -16,6 +16,7 @@ Reference: ``crates/runtime/src/models_v2/llama.rs`` -- ``forward`` ``:203-236``
 """
 from __future__ import annotations
 
+import dataclasses
 import math
 from typing import Dict, List, Optional
 
@@ -27,6 +28,7 @@ from ..model_core import Model, ModelInputs, ModelOutputs, ModelWeights, WeightM
 from ..precompute import RoPECache, alibi_slopes, apply_rope
 from ..tensor_core import ops_fn
 from ..types import InvalidInput, LoadingError
+from . import mixers as MX
 from .spec import DecoderSpec, KeyScheme, LayerSpec, MoESpec
 
 
@@ -77,21 +79,34 @@ class DecoderModel(Model):
                 shp[L + "ln2.w"] = (H,)
                 if s.norm_bias:
                     shp[L + "ln2.b"] = (H,)
-            shp[L + "wqkv"] = (ls.qkv_size, H)
-            if s.qkv_bias:
-                shp[L + "bqkv"] = (ls.qkv_size,)
-            if s.qk_norm:
-                shp[L + "q_norm"] = (ls.head_dim,)
-                if ls.kv_from is None:
-                    shp[L + "k_norm"] = (ls.head_dim,)
-            if ls.sink:
-                shp[L + "sink"] = (ls.num_heads,)
-            shp[L + "wo"] = (H, ls.o_size)
-            if s.o_bias:
-                shp[L + "bo"] = (H,)
+            if s.norm_placement == "both":
+                shp[L + "ln1b.w"] = (H,)
+                if ls.mlp is not None:
+                    shp[L + "ln2b.w"] = (H,)
+            if s.input_conv:
+                shp[L + "conv1"] = (H, s.input_conv)
+                if ls.mlp is not None:
+                    shp[L + "conv2"] = (H, s.input_conv)
+            if ls.mixer != "attention":
+                shp.update({L + n: t for n, t in MX.mixer_shapes(ls, H).items()})
+            else:
+                shp[L + "wqkv"] = (ls.qkv_size, H)
+                if s.qkv_bias:
+                    shp[L + "bqkv"] = (ls.qkv_size,)
+                if s.qk_norm:
+                    shp[L + "q_norm"] = (ls.head_dim,)
+                    if ls.kv_from is None:
+                        shp[L + "k_norm"] = (ls.head_dim,)
+                if ls.sink:
+                    shp[L + "sink"] = (ls.num_heads,)
+                shp[L + "wo"] = (H, ls.o_size)
+                if s.o_bias:
+                    shp[L + "bo"] = (H,)
             moe = ls.mlp == "moe"
             if ls.mlp == "dense" or (moe and ls.moe.dense_parallel):
-                I = s.intermediate_size
+                I = s.layer_intermediate(i)
+                if s.act == "xielu":
+                    shp[L + "act"] = (2,)
                 if s.mlp == "gated":
                     shp[L + "w_gate_up"] = (2 * I, H)
                 else:
@@ -132,6 +147,8 @@ class DecoderModel(Model):
                 t = torch.zeros(shape, dtype=dtype)
             elif is_norm_w:
                 t = torch.zeros(shape, dtype=dtype) if self.spec.norm_weight_offset_one else torch.ones(shape, dtype=dtype)
+            elif name.endswith(("q_a_norm", "kv_a_norm", "o_norm")):         # weights that are not stored around zero
+                t = torch.ones(shape, dtype=dtype)
             elif name.endswith((".b", "bqkv", "bo", "b_up", "b_down", "lm_head_bias", "router_b", "sink")):
                 t = torch.zeros(shape, dtype=dtype)
             else:
@@ -156,7 +173,31 @@ class DecoderModel(Model):
                     return q.dequantize()
         return None
 
+    def _complete_spec(self, weights: ModelWeights) -> DecoderSpec:
+        """The spec with the sizes that only the tensors' shapes give (the rank of a wkv layer's decay)."""
+        s = self.spec
+        if s.layers is None or all(ls.mixer != "wkv" or ls.decay_rank for ls in s.layers):
+            return s
+        layers = list(s.layers)
+        for i, ls in enumerate(layers):
+            if ls.mixer == "wkv" and not ls.decay_rank:
+                t = self._find(weights, tuple(p.format(i=i) for p in self.scheme.layer), self.scheme.mixers["wkv"]["w_d1"])
+                if t is None:
+                    raise LoadingError(f"{type(self).__name__}: missing weight layer {i} decay")
+                layers[i] = dataclasses.replace(ls, decay_rank=t.shape[0])
+        return dataclasses.replace(s, layers=tuple(layers))
+
+    def _load_mixer(self, weights: ModelWeights, i: int, pre, out: Dict[str, torch.Tensor]) -> None:
+        """Parameters of a layer's latent or wkv mixer, each put together from the tensors the scheme names."""
+        ls = self.spec.layer(i)
+        for name, shape in MX.mixer_shapes(ls, self.spec.hidden_size).items():
+            parts = [self._find(weights, pre, (n,)) for n in self.scheme.mixers[ls.mixer][name]]
+            if any(t is None for t in parts):
+                raise LoadingError(f"{type(self).__name__}: missing weight layer {i} {name} {self.scheme.mixers[ls.mixer][name]}")
+            out[f"layers.{i}.{name}"] = MX.join_parts(parts, shape)
+
     def _load(self, weights: ModelWeights, dtype=None, device=None):
+        self.spec = self._complete_spec(weights)
         s, k = self.spec, self.scheme
         dtype = dtype or torch.float32
         dev = torch.device(device) if device is not None else torch.device("cpu")
@@ -204,47 +245,14 @@ class DecoderModel(Model):
                 if s.norm_bias:
                     b = self._find(weights, pre, k.ln2, ".bias")
                     out[L + "ln2.b"] = b if b is not None else torch.zeros(s.hidden_size)
-            # ---- attention projections ----
-            packed = T(self._find(weights, pre, k.qkv)) if k.qkv else None
-            pb = self._find(weights, pre, k.qkv, ".bias") if k.qkv else None
-            if packed is not None:
-                out[L + "wqkv"], bq = self._unpack_qkv(packed, pb)
+            for n, names in (("ln1b.w", k.ln1b), ("ln2b.w", k.ln2b), ("conv1", k.conv1), ("conv2", k.conv2), ("act", k.act)):
+                if L + n in shapes:
+                    out[L + n] = need(self._find(weights, pre, names), f"layer {i} {n}")
+            # ---- mixer ----
+            if ls.mixer != "attention":
+                self._load_mixer(weights, i, pre, out)
             else:
-                q = T(self._find(weights, pre, k.q))
-                kk = T(self._find(weights, pre, k.k))
-                v = T(self._find(weights, pre, k.v))
-                if q is None:
-                    names = [p + n + ".weight" for p in pre for n in k.q]
-                    q, kk, v = deq(names), deq([n.replace(k.q[0], k.k[0]) for n in names]), \
-                        deq([n.replace(k.q[0], k.v[0]) for n in names])
-                need(q, f"layer {i} q_proj")
-                if ls.kv_from is None:
-                    need(kk, f"layer {i} k_proj"), need(v, f"layer {i} v_proj")
-                    out[L + "wqkv"] = torch.cat([q, kk, v], dim=0)
-                else:
-                    out[L + "wqkv"] = q
-                bq = None
-                qb = self._find(weights, pre, k.q, ".bias")
-                if qb is not None:
-                    kb = self._find(weights, pre, k.k, ".bias")
-                    vb = self._find(weights, pre, k.v, ".bias")
-                    bq = torch.cat([qb, kb if kb is not None else torch.zeros(s.kv_size),
-                                    vb if vb is not None else torch.zeros(s.kv_size)])
-            if s.qkv_bias:
-                out[L + "bqkv"] = bq if bq is not None else torch.zeros(s.q_size + 2 * s.kv_size)
-            if s.qk_norm:
-                out[L + "q_norm"] = need(self._find(weights, pre, k.q_norm), "q_norm")
-                if ls.kv_from is None:
-                    out[L + "k_norm"] = need(self._find(weights, pre, k.k_norm), "k_norm")
-            if ls.sink:
-                out[L + "sink"] = need(self._find(weights, pre, k.sink, ""), f"layer {i} sinks")
-            wo = T(self._find(weights, pre, k.o))
-            if wo is None:
-                wo = deq([p + n + ".weight" for p in pre for n in k.o])
-            out[L + "wo"] = need(wo, f"layer {i} o_proj")
-            if s.o_bias:
-                b = self._find(weights, pre, k.o, ".bias")
-                out[L + "bo"] = b if b is not None else torch.zeros(s.hidden_size)
+                self._load_attention(weights, i, pre, out, T, need, deq)
             # ---- MLP ----
             moe = ls.mlp == "moe"
             if ls.mlp == "dense" or (moe and ls.moe.dense_parallel):
@@ -314,6 +322,51 @@ class DecoderModel(Model):
         self.device, self.dtype = dev, dtype
         self._rope = self._alibi = None
 
+    def _load_attention(self, weights: ModelWeights, i: int, pre, out: Dict[str, torch.Tensor], T, need, deq) -> None:
+        """Projections, head norms and sinks of one layer's attention."""
+        s, k, ls = self.spec, self.scheme, self.spec.layer(i)
+        L = f"layers.{i}."
+        packed = T(self._find(weights, pre, k.qkv)) if k.qkv else None
+        pb = self._find(weights, pre, k.qkv, ".bias") if k.qkv else None
+        if packed is not None:
+            out[L + "wqkv"], bq = self._unpack_qkv(packed, pb)
+        else:
+            q = T(self._find(weights, pre, k.q))
+            kk = T(self._find(weights, pre, k.k))
+            v = T(self._find(weights, pre, k.v))
+            if q is None:
+                names = [p + n + ".weight" for p in pre for n in k.q]
+                q, kk, v = deq(names), deq([n.replace(k.q[0], k.k[0]) for n in names]), \
+                    deq([n.replace(k.q[0], k.v[0]) for n in names])
+            need(q, f"layer {i} q_proj")
+            if ls.kv_from is None:
+                need(kk, f"layer {i} k_proj"), need(v, f"layer {i} v_proj")
+                out[L + "wqkv"] = torch.cat([q, kk, v], dim=0)
+            else:
+                out[L + "wqkv"] = q
+            bq = None
+            qb = self._find(weights, pre, k.q, ".bias")
+            if qb is not None:
+                kb = self._find(weights, pre, k.k, ".bias")
+                vb = self._find(weights, pre, k.v, ".bias")
+                bq = torch.cat([qb, kb if kb is not None else torch.zeros(s.kv_size),
+                                vb if vb is not None else torch.zeros(s.kv_size)])
+        if s.qkv_bias:
+            out[L + "bqkv"] = bq if bq is not None else torch.zeros(s.q_size + 2 * s.kv_size)
+        if s.qk_norm:
+            out[L + "q_norm"] = need(self._find(weights, pre, k.q_norm), "q_norm")
+            if ls.kv_from is None:
+                out[L + "k_norm"] = need(self._find(weights, pre, k.k_norm), "k_norm")
+        if ls.sink:
+            out[L + "sink"] = need(self._find(weights, pre, k.sink, ""), f"layer {i} sinks")
+        wo = T(self._find(weights, pre, k.o))
+        if wo is None:
+            wo = deq([p + n + ".weight" for p in pre for n in k.o])
+        out[L + "wo"] = need(wo, f"layer {i} o_proj")
+        if s.o_bias:
+            b = self._find(weights, pre, k.o, ".bias")
+            out[L + "bo"] = b if b is not None else torch.zeros(s.hidden_size)
+
     def _unpack_qkv(self, w: torch.Tensor, b: Optional[torch.Tensor]):
         """On-disk packed QKV -> canonical [Q; K; V] row order."""
         s, lay = self.spec, self.scheme.qkv_layout
@@ -379,28 +432,38 @@ class DecoderModel(Model):
                 out[pre + k.ln2[0] + WS] = self.p[L + "ln2.w"]
                 if s.norm_bias:
                     out[pre + k.ln2[0] + BS] = self.p[L + "ln2.b"]
-            wqkv = self.p[L + "wqkv"]
-            if k.qkv:
-                out[pre + k.qkv[0] + WS] = T(self._pack_qkv(wqkv))
-                if s.qkv_bias:
-                    out[pre + k.qkv[0] + BS] = self._pack_qkv(self.p[L + "bqkv"][:, None])[:, 0]
-            elif ls.kv_from is not None:
-                out[pre + k.q[0] + WS] = T(wqkv)
+            for n, names, suffix in (("ln1b.w", k.ln1b, WS), ("ln2b.w", k.ln2b, WS), ("conv1", k.conv1, WS), ("conv2", k.conv2, WS),
+                                     ("act", k.act, WS)):
+                if L + n in self.p:
+                    out[pre + names[0] + suffix] = self.p[L + n]
+            if ls.mixer != "attention":
+                for n in MX.mixer_shapes(ls, s.hidden_size):
+                    names = k.mixers[ls.mixer][n]
+                    for name, t in zip(names, MX.split_parts(self.p[L + n], ls, n, len(names))):
+                        out[pre + name + WS] = t
             else:
-                q, kk, v = wqkv.split([ls.q_size, ls.k_size, ls.v_size])
-                out[pre + k.q[0] + WS], out[pre + k.k[0] + WS], out[pre + k.v[0] + WS] = T(q), T(kk), T(v)
-                if s.qkv_bias:
-                    qb, kb, vb = self.p[L + "bqkv"].split([s.q_size, s.kv_size, s.kv_size])
-                    out[pre + k.q[0] + BS], out[pre + k.k[0] + BS], out[pre + k.v[0] + BS] = qb, kb, vb
-            if s.qk_norm:
-                out[pre + k.q_norm[0] + WS] = self.p[L + "q_norm"]
-                if ls.kv_from is None:
-                    out[pre + k.k_norm[0] + WS] = self.p[L + "k_norm"]
-            if ls.sink:
-                out[pre + k.sink[0]] = self.p[L + "sink"]
-            out[pre + k.o[0] + WS] = T(self.p[L + "wo"])
-            if s.o_bias:
-                out[pre + k.o[0] + BS] = self.p[L + "bo"]
+                wqkv = self.p[L + "wqkv"]
+                if k.qkv:
+                    out[pre + k.qkv[0] + WS] = T(self._pack_qkv(wqkv))
+                    if s.qkv_bias:
+                        out[pre + k.qkv[0] + BS] = self._pack_qkv(self.p[L + "bqkv"][:, None])[:, 0]
+                elif ls.kv_from is not None:
+                    out[pre + k.q[0] + WS] = T(wqkv)
+                else:
+                    q, kk, v = wqkv.split([ls.q_size, ls.k_size, ls.v_size])
+                    out[pre + k.q[0] + WS], out[pre + k.k[0] + WS], out[pre + k.v[0] + WS] = T(q), T(kk), T(v)
+                    if s.qkv_bias:
+                        qb, kb, vb = self.p[L + "bqkv"].split([s.q_size, s.kv_size, s.kv_size])
+                        out[pre + k.q[0] + BS], out[pre + k.k[0] + BS], out[pre + k.v[0] + BS] = qb, kb, vb
+                if s.qk_norm:
+                    out[pre + k.q_norm[0] + WS] = self.p[L + "q_norm"]
+                    if ls.kv_from is None:
+                        out[pre + k.k_norm[0] + WS] = self.p[L + "k_norm"]
+                if ls.sink:
+                    out[pre + k.sink[0]] = self.p[L + "sink"]
+                out[pre + k.o[0] + WS] = T(self.p[L + "wo"])
+                if s.o_bias:
+                    out[pre + k.o[0] + BS] = self.p[L + "bo"]
             if L + "w_gate_up" in self.p:
                 if k.gate_up:
                     out[pre + k.gate_up[0] + WS] = T(self.p[L + "w_gate_up"])
@@ -477,14 +540,15 @@ class DecoderModel(Model):
         """Tables of one rotation; layers with the same rotation share them."""
         s = self.spec
         ls = ls or s.layer(0)
-        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3)
+        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3, ls.rope_yarn)
         if self._rope is None:
             self._rope = {}
         c = self._rope.get(key)
         if c is None or c.max_seq_len < need_len or c.cos.device != self.device:
             n = max(need_len, min(s.max_position_embeddings, 8192))
             c = self._rope[key] = RoPECache(ls.head_dim, n, ls.rope_theta, rotary_dim=ls.rotary_dim,
-                                            position_scale=s.rope_pos_scale, llama3=ls.rope_llama3, device=self.device)
+                                            position_scale=s.rope_pos_scale, llama3=ls.rope_llama3, yarn=ls.rope_yarn,
+                                            device=self.device)
         return c
 
     def _project_qkv(self, i: int, h: torch.Tensor):
@@ -508,6 +572,23 @@ class DecoderModel(Model):
                 k = ops_fn.rms_norm(k, self.p[L + "k_norm"], s.norm_eps)
         return q, k, v
 
+    def _latent_rows(self, i: int, h: torch.Tensor, rope):
+        """Rotated queries [.., heads, head_dim + rot_dim] and the rows to be cached [.., kv_rank + rot_dim] of a latent layer."""
+        s, ls = self.spec, self.spec.layer(i)
+        q, c, kr = MX.latent_project(self.p, f"layers.{i}.", ls, h, s.norm_eps)
+        if rope is not None:
+            qn, qr = q.split([ls.head_dim, ls.rot_dim], dim=-1)
+            q = torch.cat([qn, apply_rope(qr, *rope, ls.rotary_dim, s.rope_interleaved)], -1)
+            kr = apply_rope(kr, *rope, ls.rotary_dim, s.rope_interleaved)
+        return q, torch.cat([c, kr.squeeze(-2)], -1)
+
+    def mixer(self, i: int, h: torch.Tensor, past: int, cache: Optional[KVCache], shared: dict, st: dict) -> torch.Tensor:
+        """The first sublayer of layer ``i`` on whole sequences; ``st`` is the layer's carried state."""
+        ls, L = self.spec.layer(i), f"layers.{i}."
+        if ls.mixer == "wkv":
+            return ops_fn.linear(MX.wkv(self.p, L, ls, h, st, self.spec.norm_eps), self.p[L + "wo"])
+        return self._attention(i, h, past, cache, shared)
+
     def _attend(self, i: int, q, k, v, bias):
         """q [B, Hq, T, Dk], k / v [B, Hkv, S, ...] in fp32, additive ``bias`` [T, S] or [Hq, T, S] -> [B, Hq, T, Dv]."""
         ls = self.spec.layer(i)
@@ -527,13 +608,23 @@ class DecoderModel(Model):
         s, ls = self.spec, self.spec.layer(i)
         L = f"layers.{i}."
         B, T, _ = h.shape
-        q, k, v = self._project_qkv(i, h)
-        if ls.rotary_dim > 0:
-            cos, sin = self._rope_cache(past + T, ls).get_range(past, past + T)
-            q = apply_rope(q, cos, sin, ls.rotary_dim, s.rope_interleaved)
-            if k is not None:
-                k = apply_rope(k, cos, sin, ls.rotary_dim, s.rope_interleaved)
-        if ls.kv_from is not None:
+        rope = self._rope_cache(past + T, ls).get_range(past, past + T) if ls.rotary_dim > 0 else None
+        if ls.mixer == "latent":
+            q, rows = self._latent_rows(i, h, rope)
+            rows = rows[:, None]                              # one row of width kv_rank + rot_dim for all heads
+            if cache is not None:
+                cache.layer(i).append(rows, rows[..., :0])
+                rows, _ = cache.layer(i).get_kv()
+            k, v = MX.latent_expand(self.p, L, ls, rows[:, 0])
+        else:
+            q, k, v = self._project_qkv(i, h)
+            if rope is not None:
+                q = apply_rope(q, *rope, ls.rotary_dim, s.rope_interleaved)
+                if k is not None:
+                    k = apply_rope(k, *rope, ls.rotary_dim, s.rope_interleaved)
+        if ls.mixer == "latent":
+            pass
+        elif ls.kv_from is not None:
             k, v = shared[ls.kv_from]
         else:
             k, v = k.transpose(1, 2), v.transpose(1, 2)      # [B, Hkv, T, D]
@@ -558,13 +649,14 @@ class DecoderModel(Model):
         y = y.transpose(1, 2).reshape(B, T, ls.o_size).to(h.dtype)
         return ops_fn.linear(y, self.p[L + "wo"], self.p.get(L + "bo"))
 
-    def _dense_mlp(self, x, w_gate_up=None, w_up=None, b_up=None, w_down=None, b_down=None, act="silu"):
+    def _dense_mlp(self, x, w_gate_up=None, w_up=None, b_up=None, w_down=None, b_down=None, act="silu", act_p=None):
         if w_gate_up is not None:
             gu = ops_fn.linear(x, w_gate_up)
             g, u = gu.chunk(2, dim=-1)
             hdn = (ops_fn.activation(act)(_f(g)) * _f(u)).to(x.dtype)
         else:
-            hdn = ops_fn.activation(act)(_f(ops_fn.linear(x, w_up, b_up))).to(x.dtype)
+            z = _f(ops_fn.linear(x, w_up, b_up))
+            hdn = (MX.xielu(z, act_p) if act == "xielu" else ops_fn.activation(act)(z)).to(x.dtype)
         return ops_fn.linear(hdn, w_down, b_down)
 
     def _moe(self, i: int, x: torch.Tensor) -> torch.Tensor:
@@ -602,14 +694,15 @@ class DecoderModel(Model):
         y = None
         if L + "w_down" in self.p:
             y = self._dense_mlp(x, self.p.get(L + "w_gate_up"), self.p.get(L + "w_up"), self.p.get(L + "b_up"),
-                                self.p[L + "w_down"], self.p.get(L + "b_down"), s.act)
+                                self.p[L + "w_down"], self.p.get(L + "b_down"), s.act, self.p.get(L + "act"))
         if s.layer_is_moe(i):
             mo = self._moe(i, x)
             y = mo if y is None else y + mo
         return y
 
-    def block(self, i: int, x: torch.Tensor, attention) -> torch.Tensor:
-        """One layer around ``attention(h)``: where the norms sit and how the sublayers join the residual stream."""
+    def block(self, i: int, x: torch.Tensor, attention, conv=None) -> torch.Tensor:
+        """One layer around ``attention(h)``: where the norms sit and how the sublayers join the residual stream.
+        ``conv(h, name)`` puts the input convolution of that name in front of a sublayer."""
         s = self.spec
         L = f"layers.{i}."
         rs = s.residual_scale
@@ -619,6 +712,13 @@ class DecoderModel(Model):
         if s.norm_placement == "output":
             x = x + self._norm(attention(x), L + "ln1") * rs
             return x if s.layer(i).mlp is None else x + self._norm(self._mlp(i, x), L + "ln2") * rs
+        if s.norm_placement == "both":
+            h = self._norm(x, L + "ln1")
+            x = x + self._norm(attention(conv(h, "conv1") if s.input_conv else h), L + "ln1b") * rs
+            if s.layer(i).mlp is None:
+                return x
+            h = self._norm(x, L + "ln2")
+            return x + self._norm(self._mlp(i, conv(h, "conv2") if s.input_conv else h), L + "ln2b") * rs
         h = self._norm(x, L + "ln1")
         a = attention(h)
         if s.parallel_residual:
@@ -651,7 +751,9 @@ class DecoderModel(Model):
             x = ops_fn.layer_norm(x, self.p["embed_norm.w"], self.p["embed_norm.b"], s.norm_eps)
         shared: dict = {}                     # keys and values of this call's layers, for those that read an earlier one's
         for i in range(s.num_layers):
-            x = self.block(i, x, lambda h, i=i: self._attention(i, h, past, cache, shared))
+            st: dict = cache.layer(i).state if cache is not None else {}
+            x = self.block(i, x, lambda h, i=i, st=st: self.mixer(i, h, past, cache, shared, st),
+                           lambda h, n, i=i, st=st: MX.input_conv(h, self.p[f"layers.{i}.{n}"], st, n))
         if cache is not None:
             cache.set_seq_len(past + T)
         if s.final_norm:

@@ -503,6 +503,55 @@ class GekapelModel(DecoderModel):
                            rope_interleaved=True, initializer_range=c.initializer_range)
 
 
+class NipulornModel(DecoderModel):
+    """Nipulorn: norms before and after each sublayer around a 32-bit residual stream, a short causal convolution in front of
+    every sublayer, layers of RWKV-6 style recurrences and of multi-head latent attention (softmax sinks, YaRN rotation),
+    xIELU feed-forwards where a layer has one, tied and scaled embeddings.  Not one of the reference's families."""
+
+    config_class = C.NipulornConfig
+    scheme = KeyScheme(embed=("embed",), layer=("l{i}.",), ln1=("norm1",), ln2=("norm2",), ln1b=("norm1b",), ln2b=("norm2b",),
+                       conv1=("canon1",), conv2=("canon2",), up=("mlp.up",), down=("mlp.down",), act=("mlp.act",),
+                       final_norm=("final.norm",), weight_suffix="", bias_suffix=".b",
+                       mixers={"latent": {"w_dqkv": ("mix.dq", "mix.dkv"), "q_a_norm": ("mix.dq.norm",),
+                                          "kv_a_norm": ("mix.dkv.norm",), "w_uq": ("mix.uq",), "w_uk": ("mix.uk",),
+                                          "w_uv": ("mix.uv",), "sink": ("mix.sink",), "wo": ("mix.o",)},
+                               "wkv": {"mu": tuple("mix.mu." + n for n in "rkvgw"),
+                                       "w_rkvg": tuple("mix." + n for n in "rkvg"), "w_d1": ("mix.w1",), "w_d2": ("mix.w2",),
+                                       "d0": ("mix.w0",), "u": ("mix.u",), "o_norm": ("mix.norm",), "wo": ("mix.o",)}})
+
+    @staticmethod
+    def _layer_spec(i: int, d: dict) -> LayerSpec:
+        mx, mlp = d["mixer"], d.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ConfigurationError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
+        ff = dict(mlp=None if mlp is None else "dense", intermediate_size=None if mlp is None else mlp["ff"])
+        if d["type"] == "wkv":
+            return LayerSpec(num_heads=mx["heads"], num_kv_heads=mx["heads"], head_dim=mx["dim"], v_head_dim=mx["dim"],
+                             mixer="wkv", **ff)
+        if d["type"] != "latent_attention":
+            raise ConfigurationError(f"layer {i}: unknown mixer {d['type']!r}")
+        rot = mx["rot"]
+        sc = rot.get("scaling")
+        if rot["dims"] > mx["rot_dim"] or rot["dims"] % 2:
+            raise ConfigurationError(f"layer {i}: {rot['dims']} rotated dimensions of {mx['rot_dim']}")
+        return LayerSpec(num_heads=mx["heads"], num_kv_heads=mx["heads"], head_dim=mx["dim"], v_head_dim=mx["vdim"],
+                         scale=float(mx["scale"]), rotary_dim=rot["dims"], rope_theta=float(rot["base"]),
+                         rope_yarn=None if sc is None else tuple(float(sc[n]) for n in ("factor", "original", "fast", "slow")),
+                         sink=True, mixer="latent", q_rank=mx["q_rank"], kv_rank=mx["kv_rank"], rot_dim=mx["rot_dim"], **ff)
+
+    @classmethod
+    def spec_from_config(cls, c):
+        layers = tuple(cls._layer_spec(i, d) for i, d in enumerate(c.layers))
+        first = layers[0] if layers else None
+        return DecoderSpec(vocab_size=c.vocab_size, hidden_size=c.hidden_size, num_layers=len(layers), layers=layers,
+                           num_heads=first.num_heads if first else 0, num_kv_heads=first.num_kv_heads if first else 0,
+                           head_dim=first.head_dim if first else 0, intermediate_size=0,
+                           max_position_embeddings=c.max_position_embeddings, norm="rms", norm_eps=c.norm_eps,
+                           norm_weight_offset_one=True, norm_placement="both", residual_fp32=True, input_conv=c.canon_taps,
+                           rope_interleaved=True, mlp="plain", act="xielu", embed_scale=c.embedding_scale,
+                           logit_scale=c.logit_scale, tie_embeddings=True, initializer_range=c.initializer_range)
+
+
 DECODER_FAMILIES = {
     "llama": LlamaModel, "qwen": QwenModel, "gemma": GemmaModel, "phi": PhiModel, "deepseek": DeepSeekModel,
     "mistral": MistralModel, "mixtral": MixtralModel, "gpt2": GPT2Model, "gptj": GPTJModel, "gptneox": GPTNeoXModel,
@@ -510,4 +559,5 @@ DECODER_FAMILIES = {
     "olmo": OlmoModel, "granite": GraniteModel, "yi": YiModel, "falcon": FalconModel, "baichuan": BaichuanModel,
     "internlm": InternLMModel, "chatglm": ChatGLMModel, "minicpm": MiniCPMModel, "deepseek_moe": DeepSeekMoEModel,
     "dbrx": DbrxModel, "grok": GrokModel, "arctic": ArcticModel, "gekapel": GekapelModel,
+    "nipulorn": NipulornModel,
 }

@@ -1,0 +1,108 @@
+"""Sublayer parts of per-layer specs beyond plain attention: latent attention, the wkv recurrence, the input convolution and
+the xIELU activation, as PyTorch on any device -- the whole-model path and the CPU runner; the serving kernels are
+``csrc/attn/attn_latent.cu``, ``csrc/scan/wkv_mixer.cu`` and ``csrc/norm/sublayer_in.cu``.
+
+State that a sequence carries lives in a dictionary per layer (``st``); a missing entry stands for the start of a sequence.
+
+Latent attention follows DeepSeek-V2 ("DeepSeek-V2: A Strong, Economical, and Efficient Mixture-of-Experts Language
+Model"), the recurrence RWKV-6 (the reference's ``models_v2/rwkv6.rs:483-553`` in another parametrisation).
+"""
+from __future__ import annotations
+
+from typing import Dict, Tuple
+
+import torch
+import torch.nn.functional as F
+
+from ..ops import recurrent as R
+from ..tensor_core import ops_fn
+from .spec import LayerSpec
+
+MU = ("r", "k", "v", "g", "w")           # order of the token-shift mixes in the parameter ``mu``
+
+
+def mixer_shapes(ls: LayerSpec, H: int) -> Dict[str, Tuple[int, ...]]:
+    """Canonical parameters of a latent or wkv mixer."""
+    n, d = ls.num_heads, ls.head_dim
+    if ls.mixer == "latent":
+        return {"w_dqkv": (ls.q_rank + ls.kv_rank + ls.rot_dim, H), "q_a_norm": (ls.q_rank,), "kv_a_norm": (ls.kv_rank,),
+                "w_uq": (ls.q_size, ls.q_rank), "w_uk": (n * d, ls.kv_rank), "w_uv": (n * ls.v_head_dim, ls.kv_rank),
+                **({"sink": (n,)} if ls.sink else {}), "wo": (H, ls.o_size)}
+    if ls.mixer == "wkv":
+        C = n * d
+        return {"mu": (5, H), "w_rkvg": (4, C, H), "w_d1": (ls.decay_rank, H), "w_d2": (C, ls.decay_rank), "d0": (C,),
+                "u": (n, d), "o_norm": (C,), "wo": (H, C)}
+    raise ValueError(f"no such mixer: {ls.mixer!r}")
+
+
+def join_parts(parts, shape) -> torch.Tensor:
+    """The parameter that several tensors make up: stacked where it has one axis more than they have, else concatenated."""
+    if len(parts) == 1:
+        return parts[0]
+    return torch.stack(list(parts)) if len(shape) == parts[0].dim() + 1 else torch.cat(list(parts), 0)
+
+
+def split_parts(t: torch.Tensor, ls: LayerSpec, name: str, n: int):
+    """Inverse of ``join_parts`` for the parameters above."""
+    if n == 1:
+        return [t]
+    if name == "w_dqkv":
+        return list(t.split([ls.q_rank, ls.kv_rank + ls.rot_dim]))
+    return list(t.unbind(0))
+
+
+def input_conv(h: torch.Tensor, w: torch.Tensor, st: dict, key: str) -> torch.Tensor:
+    """h [B, T, H] plus its causal depthwise convolution with the taps w [H, n] (the last tap meets the token itself)."""
+    n = w.shape[1] - 1
+    if key not in st:
+        st[key] = torch.zeros(h.shape[0], n, h.shape[2], dtype=h.dtype, device=h.device)
+    return h + R.causal_dwconv1d(h, w, None, st[key])
+
+
+def wkv(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, st: dict, eps: float) -> torch.Tensor:
+    """h [B, T, H] -> [B, T, heads * dim], before the output projection."""
+    B, T, H = h.shape
+    n, d = ls.num_heads, ls.head_dim
+    first = st["shift"] if "shift" in st else torch.zeros(B, H, dtype=h.dtype, device=h.device)
+    dx = torch.cat([first[:, None], h[:, :-1]], 1) - h
+    st["shift"] = h[:, -1].clone()
+    mix = [h + dx * m.to(h.dtype) for m in p[L + "mu"]]
+    r, k, v, g = (ops_fn.linear(x, w) for x, w in zip(mix, p[L + "w_rkvg"]))
+    low = torch.tanh(F.linear(mix[4].float(), p[L + "w_d1"].float()))
+    ww = F.linear(low, p[L + "w_d2"].float()) + p[L + "d0"].float()          # decay = exp(-exp(ww))
+    if "wkv" not in st:
+        st["wkv"] = torch.zeros(B, n, d, d, dtype=torch.float32, device=h.device)
+    y = R.wkv6(r, k, v, ww.contiguous(), p[L + "u"].float(), n, st["wkv"]).float().reshape(B, T, n, d)
+    y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+    return (y.reshape(B, T, n * d) * p[L + "o_norm"].float() * F.silu(g.float())).to(h.dtype)
+
+
+def latent_project(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, eps: float):
+    """(queries [.., heads, dim + rot_dim], normalised latents [.., kv_rank], key part [.., 1, rot_dim]) before rotation."""
+    cq, c, kr = ops_fn.linear(h, p[L + "w_dqkv"]).split([ls.q_rank, ls.kv_rank, ls.rot_dim], dim=-1)
+    q = ops_fn.linear(ops_fn.rms_norm(cq.contiguous(), p[L + "q_a_norm"], eps), p[L + "w_uq"])
+    c = ops_fn.rms_norm(c.contiguous(), p[L + "kv_a_norm"], eps)
+    return q.reshape(*h.shape[:-1], ls.num_heads, ls.head_dim + ls.rot_dim), c, kr.unsqueeze(-2)
+
+
+def latent_expand(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, rows: torch.Tensor):
+    """Cached rows [.., S, kv_rank + rot_dim] -> keys [.., heads, S, dim + rot_dim] and values [.., heads, S, v size]."""
+    c, kr = rows.split([ls.kv_rank, ls.rot_dim], dim=-1)
+    lead = rows.shape[:-1]
+    k = ops_fn.linear(c.contiguous(), p[L + "w_uk"]).reshape(*lead, ls.num_heads, ls.head_dim).transpose(-2, -3)
+    v = ops_fn.linear(c.contiguous(), p[L + "w_uv"]).reshape(*lead, ls.num_heads, ls.v_head_dim).transpose(-2, -3)
+    kr = kr.unsqueeze(-3).expand(*k.shape[:-1], ls.rot_dim)
+    return torch.cat([k, kr], -1), v
+
+
+def xielu_coefficients(act: torch.Tensor) -> Tuple[float, float]:
+    """The two learned numbers as the activation uses them: softplus(p) in front of z^2, 1/2 + softplus(q) in front of the
+    exponential part."""
+    a = F.softplus(act.detach().double().cpu())
+    return float(a[0]), float(a[1]) + 0.5
+
+
+def xielu(z: torch.Tensor, act: torch.Tensor) -> torch.Tensor:
+    """z > 0: a z^2 + z / 2; z <= 0: b (e^z - 1 - z) + z / 2."""
+    a, b = xielu_coefficients(act)
+    return torch.where(z > 0, a * z * z, b * (torch.expm1(z) - z)) + 0.5 * z

@@ -11,8 +11,9 @@ plain, activation), biases, embedding / logit / residual / attention scalings, t
 mixture-of-experts (experts, top-k, shared experts, dense-parallel MLP, leading dense layers).
 
 Designs whose layers differ from one another (head counts, head sizes, windows, rotations, feed-forward sizes, layers
-without a feed-forward, layers that read another layer's keys and values) list a ``LayerSpec`` per layer;
-``DecoderSpec.layer(i)`` answers for every spec, so the loaders and runners ask it instead of the uniform fields.
+without a feed-forward, layers that read another layer's keys and values, layers with another mixer than attention) list
+a ``LayerSpec`` per layer; ``DecoderSpec.layer(i)`` answers for every spec, so the loaders and runners ask it instead of
+the uniform fields.
 """
 from __future__ import annotations
 
@@ -45,7 +46,12 @@ class MoESpec:
 class LayerSpec:
     """What one layer's sublayers look like.  ``kv_from``: the layer has no key / value projections and attends to the
     cached keys and values of that earlier layer (its own queries, window, scale and sinks).  ``mlp``: "dense", "moe" or
-    None (no feed-forward)."""
+    None (no feed-forward).
+
+    ``mixer``: "attention"; "latent" (multi-head latent attention: queries through a normalised latent of ``q_rank``, keys
+    and values of all heads from one cached, normalised latent of ``kv_rank`` and one cached rotated key part of
+    ``rot_dim`` shared by the heads; ``head_dim`` is the unrotated key size); or "wkv" (RWKV-6 style recurrence with a
+    ``head_dim`` x ``head_dim`` state per head, five token-shift mixes and a low-rank decay of ``decay_rank``)."""
 
     num_heads: int
     num_kv_heads: int
@@ -56,14 +62,31 @@ class LayerSpec:
     rotary_dim: int = 0
     rope_theta: float = 10000.0
     rope_llama3: Optional[Tuple[float, float, float, float]] = None
+    rope_yarn: Optional[Tuple[float, float, float, float]] = None   # (factor, original_ctx, fast turns, slow turns)
     kv_from: Optional[int] = None
     sink: bool = False                   # one learned logit per head in the softmax denominator
     mlp: Optional[str] = "dense"
     moe: Optional[MoESpec] = None
+    mixer: str = "attention"
+    q_rank: int = 0
+    kv_rank: int = 0
+    rot_dim: int = 0
+    decay_rank: int = 0
+    intermediate_size: Optional[int] = None   # dense feed-forward width (None: the model's)
+
+    @property
+    def has_kv(self) -> bool:
+        """The layer owns cache rows."""
+        return self.mixer != "wkv" and self.kv_from is None
+
+    @property
+    def cache_row(self) -> int:
+        """Cache elements per token of a layer that owns some: keys and values, or the latent and its rotated part."""
+        return self.kv_rank + self.rot_dim if self.mixer == "latent" else self.k_size + self.v_size
 
     @property
     def q_size(self) -> int:
-        return self.num_heads * self.head_dim
+        return self.num_heads * (self.head_dim + self.rot_dim)
 
     @property
     def k_size(self) -> int:
@@ -121,7 +144,9 @@ class DecoderSpec:
     parallel_residual: bool = False      # x + attn(n1(x)) + mlp(n2(x))
     parallel_shared_norm: bool = False   # ... with mlp reading n1(x) (GPT-J, Phi, Falcon-7B)
     post_ln: bool = False                # OPT-350m style: norm after the residual add
-    norm_placement: str = "input"        # "input": x + f(norm(x)) | "output": x + norm(f(x)), sublayers read x itself
+    norm_placement: str = "input"        # "input": x + f(norm(x)) | "output": x + norm(f(x)), sublayers read x itself |
+    #                                      "both": x + norm_b(f(norm(x)))
+    input_conv: int = 0                  # taps of the causal depthwise convolution added to what every sublayer reads (0: none)
     residual_fp32: bool = False          # the residual stream is kept in 32 bits between the layers
     layers: Optional[Tuple[LayerSpec, ...]] = None   # per-layer description; None: all layers as the fields above say
     # scalings
@@ -167,12 +192,34 @@ class DecoderSpec:
     @property
     def kv_elements_per_token(self) -> int:
         """Cache elements that one token takes over all layers that own keys and values."""
-        return sum(self.layer(i).k_size + self.layer(i).v_size for i in self.kv_layers)
+        return sum(self.layer(i).cache_row for i in self.kv_layers)
 
     @property
     def kv_layers(self) -> Tuple[int, ...]:
-        """Layers that own keys and values (the others read one of these)."""
-        return tuple(i for i in range(self.num_layers) if self.layer(i).kv_from is None)
+        """Layers that own cache rows (the others read one of these, or have no keys)."""
+        return tuple(i for i in range(self.num_layers) if self.layer(i).has_kv)
+
+    def layer_intermediate(self, i: int) -> int:
+        n = self.layer(i).intermediate_size
+        return self.intermediate_size if n is None else n
+
+    @property
+    def state_elements(self) -> int:
+        """fp32 elements of state that one sequence carries from token to token besides cache rows: the last inputs of the
+        convolutions, the previous token's input and the recurrent state of the wkv layers."""
+        n = 0
+        for i in range(self.num_layers):
+            ls = self.layer(i)
+            if self.input_conv:
+                n += (self.input_conv - 1) * self.hidden_size * (2 if ls.mlp is not None else 1)
+            if ls.mixer == "wkv":
+                n += self.hidden_size + ls.num_heads * ls.head_dim * ls.head_dim
+        return n
+
+    @property
+    def has_state(self) -> bool:
+        """Sequences carry state that cannot be rebuilt from cached blocks (so prompts cannot skip a cached prefix)."""
+        return self.state_elements > 0
 
 
 @dataclass
@@ -203,6 +250,12 @@ class KeyScheme:
     final_norm: Tuple[str, ...] = ("model.norm",)
     lm_head: Tuple[str, ...] = ("lm_head",)
     sink: Tuple[str, ...] = ()           # per-head softmax sinks
+    ln1b: Tuple[str, ...] = ()           # norms on the sublayers' outputs where the inputs are normed as well
+    ln2b: Tuple[str, ...] = ()
+    conv1: Tuple[str, ...] = ()          # input convolutions
+    conv2: Tuple[str, ...] = ()
+    act: Tuple[str, ...] = ()            # learned numbers of the activation
+    mixers: Optional[dict] = None        # {mixer: {parameter: names, several = stacked or concatenated}}, see decoder.MIXER_PARAMS
     weight_suffix: str = ".weight"
     bias_suffix: str = ".bias"
     transposed: bool = False             # GPT-2 Conv1D stores [in, out]

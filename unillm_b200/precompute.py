@@ -6,7 +6,7 @@ Parity with ``crates/runtime/src/precompute.rs``: ``RoPECache(head_dim, max_seq,
 (``:153-218``); ``SlidingWindowMaskCache(window)`` (``:224-289``).  The reference never uses these from
 its models; here the CPU oracle decoder does, and the device kernels compute the same quantities on
 the fly (``csrc/norm_rope/rope_kv_append.cu``), so the tables double as their test oracle.
-RoPE scaling variants: ``linear`` (positions divided by a factor, CodeLlama) and ``llama3``.
+RoPE scaling variants: ``linear`` (positions divided by a factor, CodeLlama), ``llama3`` and ``yarn``.
 """
 from __future__ import annotations
 
@@ -16,7 +16,11 @@ from typing import Optional, Tuple
 import torch
 
 
-def rope_inv_freq(rotary_dim: int, base: float, llama3: Optional[Tuple[float, float, float, float]] = None) -> torch.Tensor:
+def rope_inv_freq(rotary_dim: int, base: float, llama3: Optional[Tuple[float, float, float, float]] = None,
+                  yarn: Optional[Tuple[float, float, float, float]] = None) -> torch.Tensor:
+    """Frequencies of the rotated pairs.  ``yarn`` = (factor, original context, fast, slow): pairs that turn more than ``fast``
+    times within the original context keep their frequency, those that turn less than ``slow`` times are slowed down by
+    ``factor``, with a linear ramp over the pair index between the two (see ``rope_gain`` for the other half of it)."""
     inv = base ** (-torch.arange(0, rotary_dim // 2, dtype=torch.float64) * 2.0 / rotary_dim)
     if llama3 is not None:
         factor, low, high, orig = llama3
@@ -25,19 +29,31 @@ def rope_inv_freq(rotary_dim: int, base: float, llama3: Optional[Tuple[float, fl
         smooth = (orig / wavelen - low) / (high - low)
         mid = (1 - smooth) * inv / factor + smooth * inv
         inv = torch.where(wavelen > low_wl, inv / factor, torch.where(wavelen >= high_wl, mid, inv))
+    if yarn is not None:
+        factor, orig, fast, slow = yarn
+        pair = lambda turns: rotary_dim * math.log(orig / (turns * 2 * math.pi)) / (2 * math.log(base))
+        lo, hi = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), rotary_dim - 1)
+        ramp = ((torch.arange(rotary_dim // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+        inv = inv / factor * ramp + inv * (1 - ramp)
     return inv.float()
+
+
+def rope_gain(yarn: Optional[Tuple[float, float, float, float]]) -> float:
+    """Factor on cosine and sine that goes with ``yarn`` frequencies."""
+    return 1.0 if yarn is None else 0.1 * math.log(yarn[0]) + 1.0
 
 
 class RoPECache:
     def __init__(self, head_dim: int, max_seq_len: int = 2048, base: float = 10000.0, *, rotary_dim: Optional[int] = None,
                  position_scale: float = 1.0, llama3: Optional[Tuple[float, float, float, float]] = None,
-                 device="cpu"):
+                 yarn: Optional[Tuple[float, float, float, float]] = None, device="cpu"):
         self.head_dim, self.max_seq_len, self.base = head_dim, max_seq_len, base
         self.rotary_dim = rotary_dim if rotary_dim is not None else head_dim
-        inv = rope_inv_freq(self.rotary_dim, base, llama3).to(device)
+        inv = rope_inv_freq(self.rotary_dim, base, llama3, yarn).to(device)
         pos = torch.arange(max_seq_len, dtype=torch.float32, device=device) * position_scale
         ang = pos[:, None] * inv[None, :]
-        self.cos, self.sin = ang.cos(), ang.sin()
+        g = rope_gain(yarn)
+        self.cos, self.sin = ang.cos() * g, ang.sin() * g
 
     def get(self, seq_len: int):
         return self.cos[:seq_len], self.sin[:seq_len]
