@@ -25,6 +25,7 @@ extern "C" int ub_attn_decode_persist_supported(const UbAttnArgs* a);
 extern "C" int ub_attn_decode_persist(const UbAttnArgs* a, void* stream);
 extern "C" int ub_attn_decode_warp_supported(const UbAttnArgs* a);
 extern "C" int ub_attn_decode_warp(const UbAttnArgs* a, void* stream);
+extern "C" int ub_attn_split_merge(const UbAttnArgs* a, void* stream);
 
 namespace ub {
 
@@ -359,12 +360,7 @@ static bool decode_warp_enabled() {
 // The warp-MMA kernel and, for split ranges, the merge of the partials.
 static int launch_mma(const UbAttnArgs& a, cudaStream_t st) {
   const int rc = ub_attn_decode_mma_main(&a, st);
-  if (rc != 0 || a.splits == 1) return rc;
-  const int dv = a.Dv > 0 ? a.Dv : a.D;
-  attn_split_merge_kernel<<<dim3(a.num_seqs, a.Hq), dv <= 128 ? dv : 128, 0, st>>>(
-      a.scratch, reinterpret_cast<__nv_bfloat16*>(a.out), a.lse, a.Hq, dv, a.splits, a.o_stride, a.sinks);
-  const cudaError_t e = cudaGetLastError();
-  return e == cudaSuccess ? 0 : -(int)e;
+  return rc != 0 || a.splits == 1 ? rc : ub_attn_split_merge(&a, st);
 }
 
 template <int D>
@@ -407,6 +403,14 @@ static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
 }
 
 }  // namespace ub
+
+extern "C" int ub_attn_split_merge(const UbAttnArgs* a, void* stream) {
+  const int dv = a->Dv > 0 ? a->Dv : a->D;
+  ub::attn_split_merge_kernel<<<dim3(a->num_seqs, a->Hq), dv <= 128 ? dv : 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+      a->scratch, reinterpret_cast<__nv_bfloat16*>(a->out), a->lse, a->Hq, dv, a->splits, a->o_stride, a->sinks);
+  const cudaError_t e = cudaGetLastError();
+  return e == cudaSuccess ? 0 : -(int)e;
+}
 
 extern "C" int ub_attn_decode(const UbAttnArgs* a, void* stream_v) {
   using namespace ub;

@@ -13,8 +13,8 @@ namespace ub {
 namespace af32 {
 
 constexpr int WARPS = 4;
-constexpr int MAX_D = 256;
 
+template <int MAX_D>
 __global__ void __launch_bounds__(WARPS * 32) attn_f32_kernel(const UbAttnArgs a, const int Dv) {
   pdl_launch_dependents();
   pdl_wait();
@@ -33,7 +33,8 @@ __global__ void __launch_bounds__(WARPS * 32) attn_f32_kernel(const UbAttnArgs a
   for (int d = lane; d < D; d += 32) q_s[warp][d] = q[d];
   __syncwarp();
   const float* kc = reinterpret_cast<const float*>(a.k_cache);
-  const float* vc = reinterpret_cast<const float*>(a.v_cache);
+  const float* vc = reinterpret_cast<const float*>(a.kv_shared ? a.k_cache : a.v_cache);
+  const int v_ld = a.kv_shared ? D : Dv;         // shared rows: the value is the front of the key row
   const int* bt = a.block_tables + (long long)seq * a.max_blocks_per_seq;
   const int hi = a.causal || a.q_start == nullptr ? min(kv_len, qpos + 1) : kv_len;
   int lo = max(a.kv_start, 0);
@@ -77,7 +78,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_f32_kernel(const UbAttnArgs a
       const float pj = __shfl_sync(0xffffffffu, p, j);
       const long long rj = __shfl_sync(0xffffffffu, row, j);
       if (rj < 0) continue;
-      const float* vr = vc + rj * Dv;
+      const float* vr = vc + rj * v_ld;
 #pragma unroll
       for (int i = 0; i < MAX_D / 32; ++i)
         if (i * 32 + lane < Dv) acc[i] = fmaf(pj, vr[i * 32 + lane], acc[i]);
@@ -110,11 +111,14 @@ extern "C" int ub_attn_f32(const UbAttnArgs* a, void* stream) {
   if (a->num_seqs <= 0) return 0;
   if (a->q_start != nullptr && a->max_q_len <= 0) return 0;
   if (a->Hkv <= 0 || a->Hq % a->Hkv != 0) return -2;
-  if (a->D > MAX_D || Dv > MAX_D || a->D % 4 != 0 || (reinterpret_cast<uintptr_t>(a->k_cache) & 15)) return -4;
+  const int top = a->D > Dv ? a->D : Dv;
+  if (top > 640 || (a->kv_shared && Dv > a->D) || a->D % 4 != 0 || (reinterpret_cast<uintptr_t>(a->k_cache) & 15)) return -4;
   if (a->merge_o != nullptr || a->splits > 1) return -7;
   const int mq = a->q_start != nullptr ? a->max_q_len : 1;
-  cudaError_t e = ub::launch_pdl(attn_f32_kernel, dim3((mq + WARPS - 1) / WARPS, a->Hq, a->num_seqs), dim3(WARPS * 32), (size_t)0,
-                                 reinterpret_cast<cudaStream_t>(stream), *a, Dv);
+  const dim3 grid((mq + WARPS - 1) / WARPS, a->Hq, a->num_seqs), block(WARPS * 32);
+  cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
+  cudaError_t e = top <= 256 ? ub::launch_pdl(attn_f32_kernel<256>, grid, block, (size_t)0, st, *a, Dv)
+                             : ub::launch_pdl(attn_f32_kernel<640>, grid, block, (size_t)0, st, *a, Dv);
   if (e == cudaSuccess) e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }

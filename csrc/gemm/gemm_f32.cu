@@ -13,8 +13,8 @@ namespace gf32 {
 
 constexpr int BM = 64, BN = 64, BKF = 16;
 
-__device__ __forceinline__ float act_apply(float v, int act) {
-  switch (act) {
+__device__ __forceinline__ float act_apply(float v, const UbGemmArgs& a) {
+  switch (a.act) {
     case UB_ACT_SILU: return v / (1.f + expf(-v));
     case UB_ACT_GELU: return 0.5f * v * (1.f + erff(v * 0.70710678118654752f));
     case UB_ACT_GELU_TANH: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
@@ -24,6 +24,7 @@ __device__ __forceinline__ float act_apply(float v, int act) {
     case UB_ACT_SIGMOID: return 1.f / (1.f + expf(-v));
     case UB_ACT_TANH: return tanhf(v);
     case UB_ACT_SOFTPLUS: return v > 20.f ? v : log1pf(expf(v));
+    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? a.act_a * v * v : a.act_b * (expm1f(v) - v));
     default: return v;
   }
 }
@@ -105,10 +106,10 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const UbGemmArgs a) {
       if (n >= a.N) continue;
       float v = acc[0][i][j] * sc;
       if (DUAL) {
-        v = act_apply(v, a.act) * (acc[NT - 1][i][j] * sc);
+        v = act_apply(v, a) * (acc[NT - 1][i][j] * sc);
       } else {
         if (a.bias != nullptr) v += reinterpret_cast<const float*>(a.bias)[n];
-        v = act_apply(v, a.act);
+        v = act_apply(v, a);
       }
       if (a.residual != nullptr) v += reinterpret_cast<const float*>(a.residual)[(long long)m * a.ldr + n];
       out[(long long)m * a.ldo + n] = v;

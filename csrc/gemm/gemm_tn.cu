@@ -53,6 +53,7 @@ struct GemmParams {
   int up_row_off;   // DUAL: row offset of the "up" half inside w
   int out_f32;      // 1: out is float* (ldo in floats)
   float out_scale;  // multiplies the accumulator before bias / activation
+  float act_a, act_b;   // coefficients of UB_ACT_XIELU
   int* err;
   int splits;       // SPLIT-K: cluster size
   // F1: reduce-scatter push.  rs_world == 0 disables.
@@ -96,7 +97,7 @@ __device__ __forceinline__ TileCoord tile_coord(const GemmParams& p, int u, int 
   return c;
 }
 
-__device__ __forceinline__ float apply_act(float v, int act) {
+__device__ __forceinline__ float apply_act(float v, int act, float pa, float pb) {
   switch (act) {
     case UB_ACT_SILU: {
       // v * sigmoid(v) with sigmoid(v) = 0.5 * (1 + tanh(v / 2)): one MUFU instruction, no division
@@ -114,6 +115,7 @@ __device__ __forceinline__ float apply_act(float v, int act) {
     case UB_ACT_QUICK_GELU: return v / (1.f + __expf(-1.702f * v));
     case UB_ACT_SIGMOID: return 1.f / (1.f + __expf(-v));
     case UB_ACT_TANH: return tanhf(v);
+    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? pa * v * v : pb * (expm1f(v) - v));
     default: return v;
   }
 }
@@ -121,7 +123,7 @@ __device__ __forceinline__ float apply_act(float v, int act) {
 // The activation is chosen ONCE per chunk of accumulator values: a switch inside the per-value loop makes the
 // compiler evaluate every branch (erf, tanh, exp ...) for every value, which dominated the epilogue.
 template <int N, bool DUAL, int ACT>
-__device__ __forceinline__ void epi_values_t(uint32_t (&r)[N], const uint32_t (&r2)[N], float scale, float bias_v) {
+__device__ __forceinline__ void epi_values_t(uint32_t (&r)[N], const uint32_t (&r2)[N], float scale, float bias_v, float pa, float pb) {
   // The two hot forms run on packed fp32x2 instructions (the epilogue warps are bound by instruction issue):
   // silu(gate) * up with sigmoid(v) = 0.5 * (1 + tanh(v / 2)), four instructions per value instead of seven, and the
   // plain scale-and-bias as one multiply-add per two values.
@@ -156,24 +158,25 @@ __device__ __forceinline__ void epi_values_t(uint32_t (&r)[N], const uint32_t (&
 #pragma unroll
   for (int j = 0; j < N; ++j) {
     float v = __uint_as_float(r[j]) * scale;
-    if (DUAL) v = apply_act(v, ACT) * (__uint_as_float(r2[j]) * scale);
-    else v = apply_act(v + bias_v, ACT);
+    if (DUAL) v = apply_act(v, ACT, pa, pb) * (__uint_as_float(r2[j]) * scale);
+    else v = apply_act(v + bias_v, ACT, pa, pb);
     r[j] = __float_as_uint(v);
   }
 }
 template <int N, bool DUAL>
-__device__ __forceinline__ void epi_values(uint32_t (&r)[N], const uint32_t (&r2)[N], float scale, float bias_v, int act) {
+__device__ __forceinline__ void epi_values(uint32_t (&r)[N], const uint32_t (&r2)[N], float scale, float bias_v, int act, float pa, float pb) {
   switch (act) {
-    case UB_ACT_NONE: epi_values_t<N, DUAL, UB_ACT_NONE>(r, r2, scale, bias_v); break;
-    case UB_ACT_SILU: epi_values_t<N, DUAL, UB_ACT_SILU>(r, r2, scale, bias_v); break;
-    case UB_ACT_GELU: epi_values_t<N, DUAL, UB_ACT_GELU>(r, r2, scale, bias_v); break;
-    case UB_ACT_GELU_TANH: epi_values_t<N, DUAL, UB_ACT_GELU_TANH>(r, r2, scale, bias_v); break;
-    case UB_ACT_RELU: epi_values_t<N, DUAL, UB_ACT_RELU>(r, r2, scale, bias_v); break;
-    case UB_ACT_RELU2: epi_values_t<N, DUAL, UB_ACT_RELU2>(r, r2, scale, bias_v); break;
-    case UB_ACT_QUICK_GELU: epi_values_t<N, DUAL, UB_ACT_QUICK_GELU>(r, r2, scale, bias_v); break;
-    case UB_ACT_SIGMOID: epi_values_t<N, DUAL, UB_ACT_SIGMOID>(r, r2, scale, bias_v); break;
-    case UB_ACT_TANH: epi_values_t<N, DUAL, UB_ACT_TANH>(r, r2, scale, bias_v); break;
-    default: epi_values_t<N, DUAL, UB_ACT_NONE>(r, r2, scale, bias_v); break;
+    case UB_ACT_NONE: epi_values_t<N, DUAL, UB_ACT_NONE>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_SILU: epi_values_t<N, DUAL, UB_ACT_SILU>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_GELU: epi_values_t<N, DUAL, UB_ACT_GELU>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_GELU_TANH: epi_values_t<N, DUAL, UB_ACT_GELU_TANH>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_RELU: epi_values_t<N, DUAL, UB_ACT_RELU>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_RELU2: epi_values_t<N, DUAL, UB_ACT_RELU2>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_QUICK_GELU: epi_values_t<N, DUAL, UB_ACT_QUICK_GELU>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_SIGMOID: epi_values_t<N, DUAL, UB_ACT_SIGMOID>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_TANH: epi_values_t<N, DUAL, UB_ACT_TANH>(r, r2, scale, bias_v, pa, pb); break;
+    case UB_ACT_XIELU: if constexpr (!DUAL) epi_values_t<N, false, UB_ACT_XIELU>(r, r2, scale, bias_v, pa, pb); break;
+    default: epi_values_t<N, DUAL, UB_ACT_NONE>(r, r2, scale, bias_v, pa, pb); break;
   }
 }
 
@@ -347,7 +350,7 @@ __device__ __forceinline__ void splitk_finish_t(const GemmParams& p, const uint8
       gv[e] = __float_as_uint(x);
       uv[e] = __float_as_uint(up[e]);
     }
-    epi_values_t<8, DUAL, ACT>(gv, uv, p.out_scale, 0.f);
+    epi_values_t<8, DUAL, ACT>(gv, uv, p.out_scale, 0.f, p.act_a, p.act_b);
     float v[8];
 #pragma unroll
     for (int e = 0; e < 8; ++e) v[e] = __uint_as_float(gv[e]);
@@ -369,6 +372,7 @@ __device__ __forceinline__ void splitk_finish(const GemmParams& p, const uint8_t
     case UB_ACT_QUICK_GELU: splitk_finish_t<DUAL, UB_ACT_QUICK_GELU>(p, smem, tn, r0, r1, tid_e, m0, n0, vec_ok); break;
     case UB_ACT_SIGMOID: splitk_finish_t<DUAL, UB_ACT_SIGMOID>(p, smem, tn, r0, r1, tid_e, m0, n0, vec_ok); break;
     case UB_ACT_TANH: splitk_finish_t<DUAL, UB_ACT_TANH>(p, smem, tn, r0, r1, tid_e, m0, n0, vec_ok); break;
+    case UB_ACT_XIELU: if constexpr (!DUAL) splitk_finish_t<false, UB_ACT_XIELU>(p, smem, tn, r0, r1, tid_e, m0, n0, vec_ok); break;
     default: splitk_finish_t<DUAL, UB_ACT_NONE>(p, smem, tn, r0, r1, tid_e, m0, n0, vec_ok); break;
   }
 }
@@ -609,7 +613,7 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_constant
             tc_fence_before();
             mbar_arrive(&tmem_empty_bar[ab]);
           }
-          epi_values<CH, DUAL>(r, r2, p.out_scale, bias_v, p.act);
+          epi_values<CH, DUAL>(r, r2, p.out_scale, bias_v, p.act, p.act_a, p.act_b);
           if (p.out_f32) {
             // fp32 rows are twice as wide: the group's 8 KB buffer holds 16 tokens at a time
             float* stf = reinterpret_cast<float*>(staging);
@@ -1107,7 +1111,7 @@ gemm_tn_2cta_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_con
           }
           if (c + 2 < NCH) sk_prefetch(c + 2);       // in flight while this chunk is converted, staged and stored
         }
-        epi_values<CH, DUAL>(r, r2, p.out_scale, bias_v, p.act);
+        epi_values<CH, DUAL>(r, r2, p.out_scale, bias_v, p.act, p.act_a, p.act_b);
         if (p.out_f32) {
           float* stf = reinterpret_cast<float*>(staging);
 #pragma unroll
@@ -1699,6 +1703,9 @@ extern "C" int ub_gemm_tn(const UbGemmArgs* a, void* stream_v) {
   p.residual = reinterpret_cast<const __nv_bfloat16*>(a->residual);
   p.ldr = a->ldr;
   p.act = a->act;
+  p.act_a = a->act_a;
+  p.act_b = a->act_b;
+  if (a->batch > 1 || (a->act == UB_ACT_XIELU && dual)) return -6;   // batches: ub_gemv only
   p.up_row_off = a->up_row_off;
   p.out_f32 = a->out_f32;
   p.out_scale = a->out_scale == 0.f ? 1.f : a->out_scale;

@@ -21,8 +21,8 @@ namespace gemv {
 
 
 // same formulas as the tcgen05 GEMM's epilogue
-__device__ __forceinline__ float act_apply(float v, int act) {
-  switch (act) {
+__device__ __forceinline__ float act_apply(float v, const UbGemmArgs& a) {
+  switch (a.act) {
     case UB_ACT_SILU: {
       float t;
       asm("tanh.approx.f32 %0, %1;" : "=f"(t) : "f"(0.5f * v));
@@ -39,6 +39,7 @@ __device__ __forceinline__ float act_apply(float v, int act) {
     case UB_ACT_SIGMOID: return 1.f / (1.f + __expf(-v));
     case UB_ACT_TANH: return tanhf(v);
     case UB_ACT_SOFTPLUS: return v > 20.f ? v : log1pf(__expf(v));
+    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? a.act_a * v * v : a.act_b * (expm1f(v) - v));
     default: return v;
   }
 }
@@ -72,8 +73,8 @@ __global__ void __launch_bounds__(NW * 32) gemv_kernel(const UbGemmArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   const int col0 = blockIdx.x * 16;
-  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x);
-  const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.w);
+  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(a.x) + blockIdx.y * a.x_batch;
+  const __nv_bfloat16* w = reinterpret_cast<const __nv_bfloat16*>(a.w) + blockIdx.y * a.w_batch;
   const uint4* wlo[NT];
   const uint4* whi[NT];
 #pragma unroll
@@ -161,28 +162,29 @@ __global__ void __launch_bounds__(NW * 32) gemv_kernel(const UbGemmArgs a) {
     gsum *= sc;
     float v;
     if (DUAL) {
-      v = act_apply(gsum, a.act) * (usum * sc);
+      v = act_apply(gsum, a) * (usum * sc);
     } else {
       if (a.bias != nullptr) gsum += __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.bias)[col]);
-      v = act_apply(gsum, a.act);
+      v = act_apply(gsum, a);
     }
     if (a.residual != nullptr) v += __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.residual)[(long long)m * a.ldr + col]);
-    if (a.out_f32) reinterpret_cast<float*>(a.out)[(long long)m * a.ldo + col] = v;
-    else reinterpret_cast<__nv_bfloat16*>(a.out)[(long long)m * a.ldo + col] = __float2bfloat16(v);
+    const long long at = blockIdx.y * a.out_batch + (long long)m * a.ldo + col;
+    if (a.out_f32) reinterpret_cast<float*>(a.out)[at] = v;
+    else reinterpret_cast<__nv_bfloat16*>(a.out)[at] = __float2bfloat16(v);
   }
 }
 
 template <bool DUAL, bool TWO>
 static int launch(const UbGemmArgs& a, cudaStream_t st, int nw) {
-  const int grid = (a.N + 15) / 16;
+  const dim3 grid((a.N + 15) / 16, a.batch > 1 ? a.batch : 1);
   cudaError_t e;
   // The number of warps fixes the order in which a column's partial sums are added, so it depends on N and K only:
   // a row gives the same bits whatever the token count of the launch (CUDA-graph steps are padded, eager ones are not).
   if (DUAL && nw > 8) nw = 8;
   switch (nw) {
-    case 4: e = ub::launch_pdl(gemv_kernel<4, DUAL, TWO>, dim3(grid), dim3(128), (size_t)0, st, a); break;
-    case 8: e = ub::launch_pdl(gemv_kernel<8, DUAL, TWO>, dim3(grid), dim3(256), (size_t)0, st, a); break;
-    default: e = ub::launch_pdl(gemv_kernel<DUAL ? 8 : 16, DUAL, TWO>, dim3(grid), dim3(DUAL ? 256 : 512), (size_t)0, st, a); break;
+    case 4: e = ub::launch_pdl(gemv_kernel<4, DUAL, TWO>, grid, dim3(128), (size_t)0, st, a); break;
+    case 8: e = ub::launch_pdl(gemv_kernel<8, DUAL, TWO>, grid, dim3(256), (size_t)0, st, a); break;
+    default: e = ub::launch_pdl(gemv_kernel<DUAL ? 8 : 16, DUAL, TWO>, grid, dim3(DUAL ? 256 : 512), (size_t)0, st, a); break;
   }
   if (e == cudaSuccess) e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
@@ -195,6 +197,8 @@ static int launch(const UbGemmArgs& a, cudaStream_t st, int nw) {
 extern "C" int ub_gemv_supported(const UbGemmArgs* a) {
   if (a->M < 1 || a->M > 16 || a->N < 1 || a->K < 8 || a->K % 8 != 0) return 0;
   if (a->ldx % 8 != 0 || a->ldw % 8 != 0) return 0;
+  if (a->batch > 1 && (a->batch > 65535 || a->dual || a->bias != nullptr || a->residual != nullptr || a->x_batch % 8 != 0 || a->w_batch % 8 != 0))
+    return 0;
   if ((reinterpret_cast<uintptr_t>(a->x) & 15) || (reinterpret_cast<uintptr_t>(a->w) & 15)) return 0;
   if (a->rs_world > 0 || a->ag_world > 0 || a->grp_tiles != nullptr) return 0;
   return 1;
@@ -205,7 +209,7 @@ extern "C" int ub_gemv(const UbGemmArgs* a, void* stream) {
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   if (!ub_gemv_supported(a)) return -2;
   // warps per CTA: enough warps on the device to keep its copy engines busy (about 16 per SM), at least two k-steps each
-  const int tiles = (a->N + 15) / 16;
+  const int tiles = (a->N + 15) / 16 * (a->batch > 1 ? a->batch : 1);
   const int steps = (a->K / 8 + 3) / 4;
   int nw = 4;
   while (nw < 16 && tiles * nw < 148 * 16 && steps >= 4 * nw) nw <<= 1;

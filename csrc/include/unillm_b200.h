@@ -26,6 +26,7 @@ enum UbAct {
   UB_ACT_TANH = 8,
   UB_ACT_SOFTPLUS = 9,
   UB_ACT_EXP = 10,
+  UB_ACT_XIELU = 11, /* z > 0: act_a z^2 + z / 2; else act_b (e^z - 1 - z) + z / 2; epilogues of the GEMMs only */
 };
 
 /* ---------------- K1 / K2 / F1 / F3 : tcgen05 GEMM  out[M,N] = epi(x[M,K] @ w[N,K]^T) ---------------- */
@@ -67,6 +68,11 @@ typedef struct UbGemmArgs {
   /* F1: a zeroed u32 in LOCAL memory on which the CTAs of this GEMM arrive; the last one bumps every rs_peer_flag
      once (one arrival per source rank and use at the consumer).  Required when rs_world > 0. */
   uint32_t* rs_local_count;
+  float act_a, act_b;   /* coefficients of UB_ACT_XIELU */
+  /* up to 16 rows (ub_gemv) only: `batch` > 1 independent products of the same sizes, x, w and out these many elements
+     apart; no bias, residual or gated form */
+  int batch;
+  long long x_batch, w_batch, out_batch;
 } UbGemmArgs;
 int ub_gemm_tn(const UbGemmArgs* args, void* stream);
 /* Number of CTAs the launch for `args` will use; each CTA signals every peer once in F1 mode. */
@@ -138,11 +144,84 @@ typedef struct UbResidualNormArgs {
   int* err;
   int T, H, Hp, K, slots, x_rows, kind /* 0 RMS, 1 LayerNorm */, f32;
   float eps;
+  float w_off;              /* added to the weight (1: stored around zero) */
 } UbResidualNormArgs;
 int ub_residual_norm(const UbResidualNormArgs* args, void* stream);   /* x += norm(y + sum_k w yx); out = x */
 int ub_row_norm(const UbResidualNormArgs* args, void* stream);        /* out[t] = norm(x[rows[t]]) */
 int ub_embed_residual(const int* ids, const void* table, float* x, void* out, int rows, int Hp, int V, float scale, int f32,
                       int* err, void* stream);
+
+/* ---------------- K5s : input of a sublayer with norms on both sides (csrc/norm/sublayer_in.cu) ---------------- */
+typedef struct UbSublayerInArgs {
+  const float* x;           /* residual stream [rows, Hp] */
+  const void* y;            /* the previous sublayer's rows [rows, Hp], or NULL */
+  const void* wy;           /* weight of the norm on y */
+  float* x_out;             /* x + norm(y); another buffer than x; unused without y */
+  const void* wn;           /* weight of the norm on the result */
+  const float* conv;        /* [taps, Hp] or NULL */
+  float* conv_state;        /* [state_rows, taps - 1, Hp] last values of the norm */
+  const float* mu;          /* [n_mix, Hp] or NULL */
+  float* shift_state;       /* [state_rows, Hp] last value after the convolution */
+  void* out;                /* [rows, Hp], or n_mix of them out_mix_stride elements apart */
+  const int* state_in;      /* per sequence: state row to read, negative = start of the sequence */
+  const int* state_out;     /* ... and to write, negative = none; never a row that this launch reads */
+  const int* q_start;       /* [num_seqs + 1] rows of the sequences from row0 on; NULL: one row each */
+  int* err;
+  long long row0, out_mix_stride;
+  int H, Hp, taps, n_mix, num_seqs, max_q, state_rows, tile /* tokens per CTA */, f32;
+  float eps, w_off;
+} UbSublayerInArgs;
+int ub_sublayer_in(const UbSublayerInArgs* args, void* stream);
+
+/* ---------------- K16c : matrix-state recurrence with head norm and gate (csrc/wkv/wkv_mixer.cu) ---------------- */
+typedef struct UbWkvArgs {
+  const void *r, *k, *v, *g; /* [.., ld] rows of heads * D elements */
+  const float* ww;           /* decay = exp(-exp(ww)) */
+  const float* u;            /* [H, D] bonus of the current token */
+  const float* norm_w;       /* [H * D] */
+  float* state;              /* [state_rows, H, D, D], key channel first */
+  const int *state_in, *state_out, *q_start;   /* as in UbSublayerInArgs */
+  void* out;
+  float* ws;                 /* chunked form: ub_wkv_workspace_floats(rows of q_start, ..) floats */
+  int* err;
+  long long row0, ld;
+  int H, D /* padded to 8, <= 128 */, norm_dim /* real head size */, num_seqs, state_rows, f32;
+  int chunk;                 /* 0: one CTA walks a portion; else tokens per parallel chunk */
+  int rows, max_chunks;      /* chunked form: rows and an upper bound of the chunks of all sequences */
+  float eps;
+} UbWkvArgs;
+int ub_wkv_mixer(const UbWkvArgs* args, void* stream);
+long long ub_wkv_workspace_floats(int rows, int ld, int H, int D, int max_chunks);
+
+/* ---------------- K1h : one matrix per head, out[t, h] = x[t, h] @ w[h]^T (csrc/gemm/gemm_heads.cu) ---------------- */
+typedef struct UbHeadGemmArgs {
+  const void* x;
+  const void* w;            /* [H, N, K] */
+  void* out;
+  long long x_stride, x_head, out_stride, out_head;   /* elements between tokens / heads */
+  int M, N, K, H, f32;
+} UbHeadGemmArgs;
+int ub_gemm_heads(const UbHeadGemmArgs* args, void* stream);
+
+/* ---------------- K6m : norms, rotation and cache rows of latent attention (csrc/norm_rope/latent_rows.cu) ---------------- */
+typedef struct UbLatentArgs {
+  const void* down;         /* [T, q_rank + kv_rank + rot] */
+  void* q_latent;           /* [T, q_rank] */
+  void* cache;              /* [num_blocks, block_size, kv_rank + rot] */
+  const void *q_norm_w, *kv_norm_w;
+  const int* positions;
+  const int* slot_mapping;
+  const float* inv_freq;    /* [rot_dims / 2] */
+  const void* q;            /* ub_latent_rotate: rotated parts of the queries */
+  void* q_out;
+  int* err;
+  long long num_slots, q_stride, qo_stride;           /* elements between tokens */
+  int q_off, q_head, qo_off, qo_head;                 /* first rotated element of head 0, elements between heads */
+  int T, H, q_rank, kv_rank, rot, rot_dims, q_real, kv_real /* elements the norms average over */, f32;
+  float eps, gain;
+} UbLatentArgs;
+int ub_latent_rows(const UbLatentArgs* args, void* stream);
+int ub_latent_rotate(const UbLatentArgs* args, void* stream);
 
 /* ---------------- K6 : (q/k head RMSNorm) + RoPE + paged KV append ---------------- */
 typedef struct UbRopeArgs {
@@ -205,7 +284,12 @@ typedef struct UbAttnArgs {
      kernel that does. */
   const float* sinks;
   int Dv;                    /* value head size (0 = D): v_cache [.., Dv], out [T, Hq, Dv], scratch [.., Dv + 2] */
+  int kv_shared;             /* ub_attn_f32: values are the first Dv elements of the key rows (ub_attn_latent: always so) */
 } UbAttnArgs;
+/* one cache row per token for all heads: key = the row [D], value = its first Dv elements (csrc/attn/attn_latent.cu) */
+int ub_attn_latent(const UbAttnArgs* args, void* stream);
+/* merges the partials that a decode kernel left in args->scratch */
+int ub_attn_split_merge(const UbAttnArgs* args, void* stream);
 /* fp32 q, caches and output, 32-bit arithmetic; q_start = NULL: one query per sequence */
 int ub_attn_f32(const UbAttnArgs* args, void* stream);
 int ub_attn_decode(const UbAttnArgs* args, void* stream);

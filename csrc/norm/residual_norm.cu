@@ -106,7 +106,7 @@ __global__ void __launch_bounds__(256) residual_norm_kernel(const UbResidualNorm
     float* xr = a.x + (long long)t * a.Hp + ch * 8;
     load8(xr, x);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) x[e] += (f[c][e] - mean) * rstd * w[e] + b[e];
+    for (int e = 0; e < 8; ++e) x[e] += (f[c][e] - mean) * rstd * (a.w_off + w[e]) + b[e];
     store8(xr, x);
     store8(reinterpret_cast<T*>(a.out) + (long long)t * a.Hp + ch * 8, x);
   }
@@ -164,7 +164,7 @@ __global__ void __launch_bounds__(256) row_norm_kernel(const UbResidualNormArgs 
       for (int e = 0; e < 8; ++e) b[e] = 0.f;
     }
 #pragma unroll
-    for (int e = 0; e < 8; ++e) f[c][e] = (f[c][e] - mean) * rstd * w[e] + b[e];
+    for (int e = 0; e < 8; ++e) f[c][e] = (f[c][e] - mean) * rstd * (a.w_off + w[e]) + b[e];
     store8(reinterpret_cast<T*>(a.out) + (long long)t * a.Hp + ch * 8, f[c]);
   }
 }

@@ -25,11 +25,10 @@ def input_conv(h, taps):
     """h_t + sum_j taps[:, j] * h_(t - n + 1 + j), zeros in front of the sequence."""
     T, n = h.shape[0], taps.shape[1]
     y = h.clone()
-    for t in range(T):
-        for j in range(n):
-            s = t - n + 1 + j
-            if s >= 0:
-                y[t] += taps[:, j] * h[s]
+    for j in range(n):
+        back = n - 1 - j
+        if back < T:
+            y[back:] += taps[:, j] * h[:T - back]
     return y
 
 
@@ -53,12 +52,11 @@ def wkv_recurrence(r, k, v, d, u):
     """r, k, v, d [T, heads, dim], u [heads, dim] -> [T, heads, dim].  The state holds one row per key channel."""
     T, H, D = r.shape
     out = torch.zeros_like(v)
-    for h in range(H):
-        S = torch.zeros(D, D, dtype=r.dtype)
-        for t in range(T):
-            kv = torch.outer(k[t, h], v[t, h])
-            out[t, h] = (S + u[h][:, None] * kv).T @ r[t, h]
-            S = d[t, h][:, None] * S + kv
+    S = torch.zeros(H, D, D, dtype=r.dtype)
+    for t in range(T):
+        kv = k[t, :, :, None] * v[t, :, None, :]
+        out[t] = ((S + u[:, :, None] * kv) * r[t, :, :, None]).sum(1)
+        S = d[t, :, :, None] * S + kv
     return out
 
 
@@ -100,26 +98,22 @@ def rotate(v, positions, rot):
 
 def sink_softmax(scores, sink):
     """Softmax over the last axis with one more term exp(sink) in the denominator that has no value."""
-    m = torch.maximum(scores.max(), sink)
+    m = torch.maximum(scores.max(-1, keepdim=True).values, sink)
     e = torch.exp(scores - m)
-    return e / (e.sum() + torch.exp(sink - m))
-
-
-def latent_scores(qn, qr, c, kr, wuk, scale):
-    """Scores of one query (unrotated part qn [dim], rotated part qr) of one head with all latents c [n, rank]."""
-    return ((c @ wuk.T) @ qn + kr @ qr) * scale
+    return e / (e.sum(-1, keepdim=True) + torch.exp(sink - m))
 
 
 def latent_attention(qn, qr, c, kr, wuk, wuv, sink, scale):
     """qn [T, H, dim], qr [T, H, rot], latents c [S, rank], shared rotated keys kr [S, rot], wuk [H, dim, rank],
-    wuv [H, vdim, rank]; the queries are the last T of the S positions.  -> [T, H, vdim]."""
+    wuv [H, vdim, rank]; the queries are the last T of the S positions and see everything up to their own.
+    -> [T, H, vdim]."""
     T, H, S = qn.shape[0], qn.shape[1], c.shape[0]
     out = torch.zeros(T, H, wuv.shape[1], dtype=qn.dtype)
+    later = torch.arange(S)[None, :] > torch.arange(S - T, S)[:, None]
     for h in range(H):
-        v = c @ wuv[h].T
-        for i in range(T):
-            n = S - T + i + 1
-            out[i, h] = sink_softmax(latent_scores(qn[i, h], qr[i, h], c[:n], kr[:n], wuk[h], scale), sink[h]) @ v[:n]
+        k, v = c @ wuk[h].T, c @ wuv[h].T
+        scores = (qn[:, h] @ k.T + qr[:, h] @ kr.T) * scale
+        out[:, h] = sink_softmax(scores.masked_fill(later, -math.inf), sink[h]) @ v
     return out
 
 

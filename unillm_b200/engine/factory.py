@@ -36,10 +36,18 @@ def why_not_gpu(model) -> Optional[str]:
         return "hidden size and head size must be multiples of 8 (16-byte rows for the TMA copies)"
     for i in range(s.num_layers):
         ls = s.layer(i)
-        if s.layers is not None and (max(ls.head_dim, ls.v_head_dim) > 256 or s.hidden_size > 16384):
-            return f"layer {i}: head sizes above 256 or a width above 16384"
+        if s.layers is not None and s.hidden_size > 16384:
+            return "a width above 16384"
+        if ls.mixer == "wkv" and ls.head_dim > 128:
+            return f"layer {i}: wkv heads above 128"
+        if ls.mixer == "latent" and (ls.kv_rank > 512 or ls.kv_rank + ls.rot_dim > 624):
+            return f"layer {i}: a latent above 512, or above 624 with its rotated part"
+        if ls.mixer == "attention" and s.layers is not None and max(ls.head_dim, ls.v_head_dim) > 256:
+            return f"layer {i}: head sizes above 256"
         if ls.moe is not None and (ls.moe.num_experts > 256 or ls.moe.top_k > 16):
             return f"layer {i}: more than 256 experts or more than 16 per token"
+    if (s.input_conv - 1) * s.hidden_size * 4 > 220 * 1024:
+        return f"{s.input_conv} taps over {s.hidden_size} channels do not fit in shared memory"
     return None
 
 
@@ -48,7 +56,7 @@ def _auto_num_blocks(weights, block_size: int, device, gpu_memory_fraction: floa
     """KV blocks that fit in ``gpu_memory_fraction`` of the device after the weights, capped by what the sequence
     limits can ever use."""
     free, total = torch.cuda.mem_get_info(device)
-    budget = int(total * gpu_memory_fraction) - (total - free)
+    budget = int(total * gpu_memory_fraction) - (total - free) - max_num_seqs * weights.state_bytes_per_seq()
     per_block = weights.kv_bytes_per_token() * block_size
     fit = max(budget // max(per_block, 1), 0)
     useful = max_num_seqs * (-(-max_model_len // block_size) + 1) + 64

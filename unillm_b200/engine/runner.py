@@ -34,7 +34,7 @@ import torch
 
 from ..models.spec import DecoderSpec
 from ..ops import cuda_ops as K
-from ..precompute import alibi_slopes, rope_inv_freq
+from ..precompute import alibi_slopes, rope_gain, rope_inv_freq
 from ..types import InvalidInput, UnsupportedOperation
 
 
@@ -127,7 +127,10 @@ def _pad(t: torch.Tensor, dim: int, size: int) -> torch.Tensor:
 @dataclass(frozen=True)
 class KernelHeads:
     """One layer's attention heads as this rank's kernels see them: head sizes are rounded up to multiples of 8 (16-byte
-    rows); the pad entries of the projections are zero, so they add nothing to scores or outputs."""
+    rows); the pad entries of the projections are zero, so they add nothing to scores or outputs.
+
+    Latent attention: one cache row of ``dk`` = kv_rank + rot elements whose first ``dv`` = kv_rank are the value; ``dim``,
+    ``rot``, ``vdim`` and ``q_rank`` are the padded sizes around it.  wkv: ``dk`` x ``dv`` states, no cache row."""
 
     hq: int
     hkv: int
@@ -135,10 +138,20 @@ class KernelHeads:
     dk: int
     dv: int
     own_kv: bool
+    dim: int = 0
+    rot: int = 0
+    vdim: int = 0
+    q_rank: int = 0
 
     @property
     def qkv_rows(self) -> int:
         return self.hq * self.dk + (self.hkv * (self.dk + self.dv) if self.own_kv else 0)
+
+    @property
+    def cache_row(self) -> int:
+        if not self.own_kv:
+            return 0
+        return self.dk if self.q_rank else self.hkv * (self.dk + self.dv)
 
 
 class RunnerWeights:
@@ -177,9 +190,20 @@ class RunnerWeights:
         for i in range(s.num_layers):
             L = f"layers.{i}."
             ls, kh = s.layer(i), self.heads[i]
-            for n in ("ln1.w", "ln1.b", "ln2.w", "ln2.b"):
+            for n in ("ln1.w", "ln1.b", "ln2.w", "ln2.b", "ln1b.w", "ln2b.w"):
                 if L + n in p:
                     self.t[L + n] = dev(_pad(p[L + n], 0, H))
+            for n in ("conv1", "conv2"):
+                if L + n in p:                                # [taps, H] in fp32: the kernel walks the taps of a channel
+                    self.t[L + n] = _pad(p[L + n].t(), 1, H).to(device=device, dtype=torch.float32).contiguous()
+            if L + "act" in p:
+                from ..models.mixers import xielu_coefficients
+
+                self.act_params[i] = xielu_coefficients(p[L + "act"])
+            if ls.mixer != "attention":
+                self._mixer_weights(i, p, device, dev, heads)
+                self._dense_weights(i, p, dev)
+                continue
             for n in ("q_norm", "k_norm"):
                 if L + n in p:
                     self.t[L + n] = dev(_pad(p[L + n], 0, kh.dk))
@@ -201,17 +225,7 @@ class RunnerWeights:
             self.t[L + "wo"] = dev(_pad(heads(wo, ls.num_heads, ls.v_head_dim, kh.dv, rank * kh.hq, kh.hq).t(), 0, H))
             if L + "bo" in p:
                 self.t[L + "bo"] = dev(p[L + "bo"] if rank == 0 else torch.zeros_like(p[L + "bo"]))
-            if L + "w_gate_up" in p:
-                g, u = p[L + "w_gate_up"].chunk(2, 0)
-                self.t[L + "w_gate_up"] = dev(torch.cat([shard_rows(g, rank, world), shard_rows(u, rank, world)], 0))
-            if L + "w_up" in p:
-                self.t[L + "w_up"] = dev(shard_rows(p[L + "w_up"], rank, world))
-                if L + "b_up" in p:
-                    self.t[L + "b_up"] = dev(shard_rows(p[L + "b_up"], rank, world))
-            if L + "w_down" in p:
-                self.t[L + "w_down"] = dev(shard_cols(p[L + "w_down"], rank, world))
-                if L + "b_down" in p:
-                    self.t[L + "b_down"] = dev(p[L + "b_down"] if rank == 0 else torch.zeros_like(p[L + "b_down"]))
+            self._dense_weights(i, p, dev)
             if L + "router" in p:
                 # experts: tensor-parallel inside each expert here; expert-parallel layouts are built by MoeRunner
                 m = ls.moe
@@ -243,6 +257,59 @@ class RunnerWeights:
                     self.t[L + "shared_gate_up"] = dev(up_rows(p[L + "shared_gate_up"], rank, world))
                     self.t[L + "shared_down"] = dev(down_cols(p[L + "shared_down"], rank, world))
 
+    def _dense_weights(self, i: int, p, dev) -> None:
+        """Dense feed-forward of one layer."""
+        L, rank, world = f"layers.{i}.", self.rank, self.world
+        if L + "w_gate_up" in p:
+            g, u = p[L + "w_gate_up"].chunk(2, 0)
+            self.t[L + "w_gate_up"] = dev(torch.cat([shard_rows(g, rank, world), shard_rows(u, rank, world)], 0))
+        if L + "w_up" in p:
+            up = shard_rows(p[L + "w_up"], rank, world)
+            self.t[L + "w_up"] = dev(_pad(_pad(up, 0, self._round(up.shape[0])), 1, self.width))
+            if L + "b_up" in p:
+                self.t[L + "b_up"] = dev(shard_rows(p[L + "b_up"], rank, world))
+        if L + "w_down" in p:
+            dn = shard_cols(p[L + "w_down"], rank, world)
+            self.t[L + "w_down"] = dev(_pad(_pad(dn, 1, self._round(dn.shape[1])), 0, self.width))
+            if L + "b_down" in p:
+                self.t[L + "b_down"] = dev(p[L + "b_down"] if rank == 0 else torch.zeros_like(p[L + "b_down"]))
+
+    def _mixer_weights(self, i: int, p, device, dev, heads) -> None:
+        """Latent attention or wkv parameters of one layer in kernel layout."""
+        L, ls, kh, H = f"layers.{i}.", self.spec.layer(i), self.heads[i], self.width
+        n, t = ls.num_heads, self.t
+
+        def f32(x):
+            return x.to(device=device, dtype=torch.float32).contiguous()
+
+        def head_cols(w, d, dp):                              # [H, heads * d] -> [width, heads * dp]
+            return dev(_pad(heads(w.t(), n, d, dp, 0, n).t(), 0, H))
+
+        if ls.mixer == "wkv":
+            d, dp, rank = ls.head_dim, kh.dk, self._round(ls.decay_rank)
+            t[L + "mu"] = f32(_pad(p[L + "mu"], 1, H))
+            t[L + "w_rkvg"] = dev(torch.stack([_pad(heads(w, n, d, dp, 0, n), 1, H) for w in p[L + "w_rkvg"]]))
+            t[L + "w_d1"] = dev(_pad(_pad(p[L + "w_d1"], 0, rank), 1, H))
+            t[L + "w_d2"] = dev(_pad(heads(p[L + "w_d2"], n, d, dp, 0, n), 1, rank))
+            t[L + "d0"] = dev(heads(p[L + "d0"], n, d, dp, 0, n))
+            t[L + "u"] = f32(_pad(p[L + "u"], 1, dp))
+            t[L + "o_norm"] = f32(heads(p[L + "o_norm"], n, d, dp, 0, n))
+            t[L + "wo"] = head_cols(p[L + "wo"], d, dp)
+            return
+        dq, dc, dr = p[L + "w_dqkv"].split([ls.q_rank, ls.kv_rank, ls.rot_dim])
+        t[L + "w_dqkv"] = dev(_pad(torch.cat([_pad(dq, 0, kh.q_rank), _pad(dc, 0, kh.dv), _pad(dr, 0, kh.rot)]), 1, H))
+        t[L + "q_a_norm"], t[L + "kv_a_norm"] = dev(_pad(p[L + "q_a_norm"], 0, kh.q_rank)), dev(_pad(p[L + "kv_a_norm"], 0, kh.dv))
+        uq = p[L + "w_uq"].reshape(n, ls.head_dim + ls.rot_dim, ls.q_rank)
+        uq = torch.cat([_pad(uq[:, :ls.head_dim], 1, kh.dim), _pad(uq[:, ls.head_dim:], 1, kh.rot)], 1)
+        t[L + "w_uq"] = dev(_pad(uq.flatten(0, 1), 1, kh.q_rank))
+        uk = _pad(_pad(p[L + "w_uk"].reshape(n, ls.head_dim, ls.kv_rank), 1, kh.dim), 2, kh.dv)
+        uv = _pad(_pad(p[L + "w_uv"].reshape(n, ls.v_head_dim, ls.kv_rank), 1, kh.vdim), 2, kh.dv)
+        t[L + "w_uk_t"] = dev(uk.transpose(1, 2))             # [heads, kv_rank, dim]: taken to the query side
+        t[L + "w_uv"] = dev(uv)                               # [heads, vdim, kv_rank]
+        if ls.sink:
+            t[L + "sink"] = f32(p[L + "sink"])
+        t[L + "wo"] = head_cols(p[L + "wo"], ls.v_head_dim, kh.vdim)
+
     def _init_layout(self, spec: DecoderSpec, rank: int, world: int, expert_parallel: bool, dtype=torch.bfloat16) -> None:
         """Everything that follows from the spec and the rank alone: head layout per layer, padded width, shard sizes."""
         self.spec, self.rank, self.world, self.dtype = spec, rank, world, dtype
@@ -253,8 +320,22 @@ class RunnerWeights:
         self.vocab_shard = spec.vocab_size // world
         self.width = self._round(spec.hidden_size)
         self.heads: List[KernelHeads] = []
+        self.act_params: Dict[int, Tuple[float, float]] = {}   # coefficients of activations with learned numbers, per layer
+        r8 = self._round
         for i in range(spec.num_layers):
             ls = spec.layer(i)
+            if ls.mixer != "attention" or spec.norm_placement == "both":
+                if world > 1:
+                    raise UnsupportedOperation("latent attention, wkv layers and norms on both sides of a sublayer: one rank")
+            if ls.mixer == "wkv":
+                d = r8(ls.head_dim)
+                self.heads.append(KernelHeads(ls.num_heads, 0, 0, d, d, False))
+                continue
+            if ls.mixer == "latent":
+                rank_p, rot = r8(ls.kv_rank), r8(ls.rot_dim)
+                self.heads.append(KernelHeads(ls.num_heads, 1, 0, rank_p + rot, rank_p, True, r8(ls.head_dim), rot,
+                                              r8(ls.v_head_dim), r8(ls.q_rank)))
+                continue
             if ls.num_heads % world != 0:
                 raise InvalidInput(f"{ls.num_heads} heads not divisible by tensor parallel size {world}")
             if ls.moe is not None and not self.ep and (ls.moe.intermediate_size % world or ls.moe.shared_width % world):
@@ -270,7 +351,22 @@ class RunnerWeights:
     def kv_bytes_per_token(self) -> int:
         """Cache bytes that one token takes on this rank over all layers that own keys and values."""
         e = torch.empty(0, dtype=self.dtype).element_size()
-        return e * sum(k.hkv * (k.dk + k.dv) for k in self.heads if k.own_kv)
+        return e * sum(k.cache_row for k in self.heads)
+
+    def state_bytes_per_seq(self) -> int:
+        """Bytes of carried state of one live sequence (both halves of its slot)."""
+        return 8 * sum(math.prod(shape) for _, shape in self.state_shapes())
+
+    def state_shapes(self):
+        """((layer, name), shape per state row) of everything that sequences carry from step to step, all fp32."""
+        s, out = self.spec, []
+        for i in range(s.num_layers):
+            ls, kh = s.layer(i), self.heads[i]
+            if s.input_conv:
+                out += [((i, n), (s.input_conv - 1, self.width)) for n in (("conv1", "conv2") if ls.mlp is not None else ("conv1",))]
+            if ls.mixer == "wkv":
+                out += [((i, "shift"), (self.width,)), ((i, "wkv"), (kh.hq, kh.dk, kh.dv))]
+        return out
 
     @staticmethod
     def kv_layout(num_kv_heads: int, rank: int, world: int) -> Tuple[int, int]:
@@ -387,10 +483,37 @@ class RunnerWeights:
             self.t["final_norm.b"] = zeros(H)
         for i, (kh, ls) in enumerate(zip(self.heads, s.layers)):
             L = f"layers.{i}."
-            for n in ("ln1", "ln2"):
-                self.t[L + n + ".w"] = ones(H)
+            norm_w = zeros if s.norm_weight_offset_one else ones
+            for n in ("ln1", "ln2") if s.norm_placement != "both" else ("ln1", "ln2", "ln1b", "ln2b"):
+                self.t[L + n + ".w"] = norm_w(H)
                 if s.norm_bias:
                     self.t[L + n + ".b"] = zeros(H)
+            if s.input_conv:
+                for n in ("conv1", "conv2"):
+                    self.t[L + n] = rnd(s.input_conv, H).float()
+            if ls.mlp == "dense":
+                width = self._round(s.layer_intermediate(i))
+                self.t[L + "w_up"], self.t[L + "w_down"] = rnd(width, H), rnd(H, width)
+                if s.mlp == "gated":
+                    self.t[L + "w_gate_up"] = torch.cat([self.t.pop(L + "w_up"), rnd(width, H)])
+                if s.act == "xielu":
+                    self.act_params[i] = (0.8, 1.3)
+            if ls.mixer == "wkv":
+                rank, C = self._round(ls.decay_rank or 64), kh.hq * kh.dk
+                self.t[L + "mu"] = torch.full((5, H), 0.5, device=self.t["embed"].device)
+                self.t[L + "w_rkvg"] = torch.stack([rnd(C, H) for _ in range(4)])
+                self.t[L + "w_d1"], self.t[L + "w_d2"], self.t[L + "d0"] = rnd(rank, H), rnd(C, rank), zeros(C) - 2.0
+                self.t[L + "u"], self.t[L + "o_norm"] = rnd(kh.hq, kh.dk).float(), ones(C).float()
+                self.t[L + "wo"] = rnd(H, C)
+                continue
+            if ls.mixer == "latent":
+                self.t[L + "w_dqkv"] = rnd(kh.q_rank + kh.dk, H)
+                self.t[L + "q_a_norm"], self.t[L + "kv_a_norm"] = ones(kh.q_rank), ones(kh.dv)
+                self.t[L + "w_uq"] = rnd(kh.hq * (kh.dim + kh.rot), kh.q_rank)
+                self.t[L + "w_uk_t"] = rnd(kh.hq * kh.dv, kh.dim).view(kh.hq, kh.dv, kh.dim)
+                self.t[L + "w_uv"] = rnd(kh.hq * kh.vdim, kh.dv).view(kh.hq, kh.vdim, kh.dv)
+                self.t[L + "sink"], self.t[L + "wo"] = zeros(kh.hq).float(), rnd(H, kh.hq * kh.vdim)
+                continue
             self.t[L + "wqkv"] = rnd(kh.qkv_rows, H)
             self.t[L + "wo"] = rnd(H, kh.hq * kh.dv)
             if s.qk_norm:
@@ -626,6 +749,14 @@ class GpuModelRunner:
         if spec.norm_placement == "output" and (not spec.residual_fp32 or spec.pos == "learned" or spec.embed_norm
                                                 or spec.residual_scale != 1.0 or spec.parallel_residual):
             raise UnsupportedOperation("norms on sublayer outputs: 32-bit residual stream, no learned positions")
+        if spec.norm_placement == "both" and (not spec.residual_fp32 or spec.norm != "rms" or spec.norm_bias or spec.pos == "learned"
+                                              or spec.embed_norm or spec.residual_scale != 1.0 or spec.parallel_residual
+                                              or any(spec.layer_is_moe(i) for i in range(spec.num_layers))):
+            raise UnsupportedOperation("norms on both sides of a sublayer: RMS, 32-bit residual stream, dense feed-forwards")
+        if spec.norm_placement != "both" and (spec.input_conv or any(spec.layer(i).mixer != "attention" for i in range(spec.num_layers))):
+            raise UnsupportedOperation("input convolutions, latent attention and wkv layers: with norms on both sides of a sublayer")
+        if spec.norm_placement == "both" and any(spec.layer(i).mixer == "attention" for i in range(spec.num_layers)):
+            raise UnsupportedOperation("norms on both sides of a sublayer: latent attention and wkv layers")
         if spec.norm_placement == "input" and (spec.residual_fp32 or weights.dtype != torch.bfloat16):
             raise UnsupportedOperation("a 32-bit residual stream or 32-bit weights: only with norms on sublayer outputs")
         self.spec, self.w = spec, weights
@@ -647,8 +778,14 @@ class GpuModelRunner:
                 self.k_cache.append(self.k_cache[ls.kv_from])
                 self.v_cache.append(self.v_cache[ls.kv_from])
                 continue
-            for cache, d in ((self.k_cache, kh.dk), (self.v_cache, kh.dv)):
+            if not kh.own_kv:                            # no keys at all
+                self.k_cache.append(None), self.v_cache.append(None)
+                continue
+            for cache, d in ((self.k_cache, kh.dk), (self.v_cache, 0 if ls.mixer == "latent" else kh.dv)):
                 cache.append(torch.zeros(num_blocks, kh.hkv, block_size, d, dtype=weights.dtype, device=dev))
+        # carried state: two rows per live sequence (a step reads one and writes the other)
+        self.state: Dict[tuple, torch.Tensor] = {key: torch.zeros(2 * max_num_seqs, *shape, dtype=torch.float32, device=dev)
+                                                 for key, shape in weights.state_shapes()}
         self._inv_freq: Dict[tuple, torch.Tensor] = {}   # rotation tables of per-layer specs
         self.alibi = None
         if s.pos == "alibi":
@@ -809,10 +946,7 @@ class GpuModelRunner:
         kw = dict(theta=ls.rope_theta, llama3_scaling=ls.rope_llama3)
         if s.layers is not None:
             # frequencies from the host in 64 bits, and only for the layers' own rotation
-            key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3)
-            if key not in self._inv_freq:
-                self._inv_freq[key] = rope_inv_freq(*key).to(self.device)
-            kw = dict(inv_freq=self._inv_freq[key] if ls.rotary_dim > 0 else None, v_head_dim=kh.dv, norm_dim=ls.head_dim)
+            kw = dict(inv_freq=self._rotation(ls)[0] if ls.rotary_dim > 0 else None, v_head_dim=kh.dv, norm_dim=ls.head_dim)
         own = kh.own_kv
         with self._prof("rope_kv_append"):
             K.rope_kv_append(qkv, pos, slots if own else None, self.k_cache[i] if own else None,
@@ -981,6 +1115,8 @@ class GpuModelRunner:
         self._last_fused = False
         if s.norm_placement == "output":
             return self._forward_tokens_output_norm(lay, shared_prefix_len)
+        if s.norm_placement == "both":
+            return self._forward_tokens_both_norms(lay)
         ids = self._view(lay, "token_ids")
         pos = self._view(lay, "positions")
         slots = self._view(lay, "slot_mapping")
@@ -1052,13 +1188,115 @@ class GpuModelRunner:
                 h = self._residual_norm(x, y, L + "ln2")
         return x
 
+    def _forward_tokens_both_norms(self, lay) -> torch.Tensor:
+        """Layers of the form ``x += norm_b(f(conv(norm(x))))`` around a 32-bit residual stream.  Adding a sublayer's normed
+        output, the next norm, its convolution over time and (in front of a recurrent mixer) the token-shift mixes are one
+        kernel; what it needs from earlier steps is in the sequences' state rows."""
+        s, t = self.spec, self.w.t
+        pos, slots = self._view(lay, "positions"), self._view(lay, "slot_mapping")
+        parts = self._portions(lay)
+        x, _ = K.embed_residual(self._view(lay, "token_ids"), t["embed"], scale=s.embed_scale)
+        self.launches += 1
+        y = y_name = None
+        for i, ls in enumerate(self.layers):
+            L = f"layers.{i}."
+            x, h = self._sublayer_in(i, 1, x, parts, y, y_name)
+            if ls.mixer == "wkv":
+                a = self._wkv(i, h, parts)
+            else:
+                a = self._latent_attention(i, h, pos, slots, lay)
+            y, y_name = self._gemm(a, t[L + "wo"]), L + "ln1b"
+            if ls.mlp is not None:
+                x, h = self._sublayer_in(i, 2, x, parts, y, y_name)
+                up = self._gemm(h, t[L + "w_up"], act=s.act, act_params=self.w.act_params.get(i))
+                y, y_name = self._gemm(up, t[L + "w_down"]), L + "ln2b"
+        if y is not None:
+            self._residual_norm(x, y, y_name)
+        return x
+
+    def _portions(self, lay) -> List["K.Portions"]:
+        """The step's rows as portions of sequences: one-token rows of decoding sequences, then pieces of prompts."""
+        T, Dp, P = lay["_T"], lay["_Dp"], lay["_P"]
+        si = so = None
+        if "state_in" in lay:
+            si, so = self._view(lay, "state_in"), self._view(lay, "state_out")
+        cut = lambda t, a, b: None if t is None else t[a:b]
+        out = []
+        if Dp:
+            out.append(K.Portions(0, Dp, Dp, 1, None, cut(si, 0, Dp), cut(so, 0, Dp)))
+        if P:
+            out.append(K.Portions(Dp, T - Dp, P, lay["_max_q"], self._view(lay, "q_start"), cut(si, Dp, Dp + P), cut(so, Dp, Dp + P)))
+        return out
+
+    def _sublayer_in(self, i, which, x, parts, y, y_name):
+        s, t, L = self.spec, self.w.t, f"layers.{i}."
+        conv = f"conv{which}"
+        mix = which == 1 and self.layers[i].mixer == "wkv"
+        self.launches += len(parts)
+        with self._prof("sublayer_in"):
+            return K.sublayer_in(x, parts, t[f"{L}ln{which}.w"], eps=s.norm_eps, y=y, y_weight=None if y is None else t[y_name + ".w"],
+                                 conv=t.get(L + conv), conv_state=self.state.get((i, conv)), mu=t[L + "mu"] if mix else None,
+                                 shift_state=self.state[(i, "shift")] if mix else None, width=s.hidden_size,
+                                 offset_one=s.norm_weight_offset_one)
+
+    def _wkv(self, i, h, parts):
+        """``h`` [5, T, width]: the mixes for receptance, key, value, gate and decay."""
+        t, L, kh = self.w.t, f"layers.{i}.", self.w.heads[i]
+        with self._prof(f"gemm_rkvg[4x{h.shape[1]}x{kh.hq * kh.dk}x{h.shape[2]}]"):
+            rkvg = K.gemm_stacked(h[:4], t[L + "w_rkvg"])
+        low = self._gemm(h[4], t[L + "w_d1"], act="tanh")
+        ww = self._gemm(low, t[L + "w_d2"], bias=t[L + "d0"], out_dtype=torch.float32)
+        self.launches += 1 + len(parts)
+        with self._prof("wkv"):
+            return K.wkv_mixer(rkvg, ww, t[L + "u"], t[L + "o_norm"], self.state[(i, "wkv")], parts, eps=self.spec.norm_eps,
+                               norm_dim=self.layers[i].head_dim)
+
+    def _latent_attention(self, i, h, pos, slots, lay):
+        """Latent attention with the key matrices on the query side and the value matrices on the output side, over the
+        cached latents themselves."""
+        s, t, ls, kh, L = self.spec, self.w.t, self.layers[i], self.w.heads[i], f"layers.{i}."
+        T, Dp, P = lay["_T"], lay["_Dp"], lay["_P"]
+        freq, gain = self._rotation(ls)
+        down = self._gemm(h, t[L + "w_dqkv"])
+        with self._prof("latent_rows"):
+            cq = K.latent_rows(down, pos, slots, self.k_cache[i], t[L + "q_a_norm"], t[L + "kv_a_norm"], freq, eps=s.norm_eps,
+                               gain=gain, q_real=ls.q_rank, kv_real=ls.kv_rank)
+        q = self._gemm(cq, t[L + "w_uq"]).view(T, kh.hq, kh.dim + kh.rot)
+        bt = self._view(lay, "block_tables").view(Dp + P, self.max_blocks_per_seq)
+        qa = torch.empty(T, kh.hq, kh.dk, dtype=q.dtype, device=q.device)
+        lat = torch.empty(T, kh.hq, kh.dv, dtype=q.dtype, device=q.device)
+        out = torch.empty(T, kh.hq, kh.vdim, dtype=q.dtype, device=q.device)
+        with self._prof("latent_query"):
+            K.gemm_heads(q[..., :kh.dim], t[L + "w_uk_t"], qa[..., :kh.dv])
+            K.latent_rotate(q, pos, freq, kh.rot, out=qa, gain=gain)
+        kw = dict(scale=ls.scale, sinks=t.get(L + "sink"))
+        if Dp:
+            with self._prof("attn_latent_decode"):
+                K.attn_latent(qa[:Dp], self.k_cache[i], kh.dv, bt[:Dp], self._view(lay, "seq_lens_d"), out=lat[:Dp],
+                              scratch=self.attn_scratch, max_seq_len=self.max_model_len if self._graph_mode else int(self._max_len_d), **kw)
+        if P:
+            with self._prof("attn_latent_prefill"):
+                K.attn_latent(qa[Dp:], self.k_cache[i], kh.dv, bt[Dp:], self._view(lay, "seq_lens_p"), out=lat[Dp:],
+                              q_start=self._view(lay, "q_start"), max_q_len=lay["_max_q"], **kw)
+        with self._prof("latent_value"):
+            K.gemm_heads(lat, t[L + "w_uv"], out)
+        self.launches += 4 + (Dp > 0) + (P > 0)
+        return out.view(T, kh.hq * kh.vdim)
+
+    def _rotation(self, ls):
+        """(device table of a layer's rotation frequencies, gain on cosine and sine)."""
+        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3, ls.rope_yarn)
+        if key not in self._inv_freq:
+            self._inv_freq[key] = rope_inv_freq(*key).to(self.device)
+        return self._inv_freq[key], rope_gain(ls.rope_yarn)
+
     def _residual_norm(self, x, y, name, **kw):
         s, t = self.spec, self.w.t
         self.launches += 1
         with self._prof("residual_norm"):
             return K.residual_norm(x, y, t[name + ".w"], t.get(name + ".b"), eps=s.norm_eps,
                                    kind="rms" if s.norm == "rms" else "layer", width=s.hidden_size,
-                                   out=x if self.w.dtype == torch.float32 else None, **kw)
+                                   offset_one=s.norm_weight_offset_one, out=x if self.w.dtype == torch.float32 else None, **kw)
 
     # ------------------------------------------------------------------------------------------
     # fused tensor-parallel path (F1 / F3)
@@ -1192,7 +1430,8 @@ class GpuModelRunner:
             self.launches += 1
             with self._prof("norm"):
                 return K.row_norm(x, t["final_norm.w"], t.get("final_norm.b"), eps=s.norm_eps, rows=rows,
-                                  kind="rms" if s.norm == "rms" else "layer", width=s.hidden_size)
+                                  kind="rms" if s.norm == "rms" else "layer", width=s.hidden_size,
+                                  offset_one=s.norm_weight_offset_one)
         xs = x.index_select(0, rows.long()) if lay["_S"] != x.shape[0] else x
         if s.final_norm and not self._final_norm_done:
             xs = self._norm(xs, "final_norm")
@@ -1416,7 +1655,7 @@ class GpuModelRunner:
         torch.cuda.synchronize(self.device)
 
     def kv_cache_bytes(self) -> int:
-        own = [i for i, ls in enumerate(self.layers) if ls.kv_from is None]
+        own = [i for i, ls in enumerate(self.layers) if ls.has_kv]
         return sum(c[i].numel() * c[i].element_size() for c in (self.k_cache, self.v_cache) for i in own)
 
     def forward_logits(self, b: StepBatch) -> torch.Tensor:

@@ -24,6 +24,7 @@ UB_MAX_RANKS = 8
 ACT = {
     None: 0, "none": 0, "silu": 1, "swish": 1, "gelu": 2, "gelu_tanh": 3, "gelu_new": 3, "gelu_pytorch_tanh": 3,
     "relu": 4, "relu2": 5, "quick_gelu": 6, "sigmoid": 7, "tanh": 8, "softplus": 9, "exp": 10,
+    "xielu": 11,
 }
 
 vp = C.c_void_p
@@ -46,7 +47,8 @@ class UbGemmArgs(C.Structure):
         ("ag_world", i32), ("ag_rows_per_rank", i32),
         ("ag_flags", vp), ("ag_epoch", vp), ("ag_signals_per_use", u32),
         ("grp_tiles", vp), ("grp_max_tiles", i32), ("grp_w_rows", i32), ("tail_split", i32), ("cta_pair", i32), ("pair_splits", i32),
-        ("rs_local_count", vp),
+        ("rs_local_count", vp), ("act_a", f32), ("act_b", f32),
+        ("batch", i32), ("x_batch", i64), ("w_batch", i64), ("out_batch", i64),
     ]
 
 
@@ -76,7 +78,45 @@ class UbResidualNormArgs(C.Structure):
     _fields_ = [
         ("y", vp), ("yx", vp), ("row_slot", vp), ("topk_w", vp), ("x", vp), ("rows", vp), ("out", vp), ("weight", vp),
         ("bias", vp), ("err", vp), ("T", i32), ("H", i32), ("Hp", i32), ("K", i32), ("slots", i32), ("x_rows", i32),
-        ("kind", i32), ("f32", i32), ("eps", f32),
+        ("kind", i32), ("f32", i32), ("eps", f32), ("w_off", f32),
+    ]
+
+
+class UbSublayerInArgs(C.Structure):
+    _fields_ = [
+        ("x", vp), ("y", vp), ("wy", vp), ("x_out", vp), ("wn", vp), ("conv", vp), ("conv_state", vp), ("mu", vp),
+        ("shift_state", vp), ("out", vp), ("state_in", vp), ("state_out", vp), ("q_start", vp), ("err", vp),
+        ("row0", i64), ("out_mix_stride", i64),
+        ("H", i32), ("Hp", i32), ("taps", i32), ("n_mix", i32), ("num_seqs", i32), ("max_q", i32), ("state_rows", i32),
+        ("tile", i32), ("f32", i32), ("eps", f32), ("w_off", f32),
+    ]
+
+
+class UbWkvArgs(C.Structure):
+    _fields_ = [
+        ("r", vp), ("k", vp), ("v", vp), ("g", vp), ("ww", vp), ("u", vp), ("norm_w", vp), ("state", vp),
+        ("state_in", vp), ("state_out", vp), ("q_start", vp), ("out", vp), ("ws", vp), ("err", vp),
+        ("row0", i64), ("ld", i64),
+        ("H", i32), ("D", i32), ("norm_dim", i32), ("num_seqs", i32), ("state_rows", i32), ("f32", i32),
+        ("chunk", i32), ("rows", i32), ("max_chunks", i32), ("eps", f32),
+    ]
+
+
+class UbHeadGemmArgs(C.Structure):
+    _fields_ = [
+        ("x", vp), ("w", vp), ("out", vp), ("x_stride", i64), ("x_head", i64), ("out_stride", i64), ("out_head", i64),
+        ("M", i32), ("N", i32), ("K", i32), ("H", i32), ("f32", i32),
+    ]
+
+
+class UbLatentArgs(C.Structure):
+    _fields_ = [
+        ("down", vp), ("q_latent", vp), ("cache", vp), ("q_norm_w", vp), ("kv_norm_w", vp), ("positions", vp),
+        ("slot_mapping", vp), ("inv_freq", vp), ("q", vp), ("q_out", vp), ("err", vp),
+        ("num_slots", i64), ("q_stride", i64), ("qo_stride", i64),
+        ("q_off", i32), ("q_head", i32), ("qo_off", i32), ("qo_head", i32),
+        ("T", i32), ("H", i32), ("q_rank", i32), ("kv_rank", i32), ("rot", i32), ("rot_dims", i32), ("q_real", i32),
+        ("kv_real", i32), ("f32", i32), ("eps", f32), ("gain", f32),
     ]
 
 
@@ -88,7 +128,7 @@ class UbAttnArgs(C.Structure):
         ("block_size", i32), ("max_blocks_per_seq", i32), ("num_blocks", i32),
         ("q_stride", i64), ("o_stride", i64), ("scale", f32),
         ("causal", i32), ("window", i32), ("splits", i32), ("kv_start", i32), ("total_q", i32), ("max_q_len", i32),
-        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32),
+        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32), ("kv_shared", i32),
     ]
 
 
@@ -182,7 +222,8 @@ class _CudaLibs:
 
     ARGS_AND_STREAM = {
         "serving": ("ub_gemm_tn", "ub_norm", "ub_rope_kv_append", "ub_attn_decode", "ub_attn_prefill", "ub_sample",
-                    "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm"),
+                    "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm", "ub_sublayer_in", "ub_wkv_mixer",
+                    "ub_gemm_heads", "ub_latent_rows", "ub_latent_rotate", "ub_attn_latent"),
         "more": ("ub_allreduce_oneshot", "ub_tp_argmax_merge"),
     }
 
@@ -193,6 +234,7 @@ class _CudaLibs:
         lib.ub_gemm_num_ctas.argtypes = [vp]
         lib.ub_gemm_streamk_reset.restype = i32
         lib.ub_gemm_streamk_reset.argtypes = [vp]
+        lib.ub_wkv_workspace_floats.restype = i64
         lib.ub_cuda_error_string.restype = C.c_char_p
 
     def part(self, name: str) -> C.CDLL:

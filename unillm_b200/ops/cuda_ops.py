@@ -87,12 +87,14 @@ def gemm_tn(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = 
             residual: Optional[torch.Tensor] = None, act: Optional[str] = None, out: Optional[torch.Tensor] = None,
             out_dtype: torch.dtype = torch.bfloat16, out_scale: float = 1.0, tile_tokens: int = 0, splits: int = 0,
             dual_rows: int = 0, rs: Optional[dict] = None, ag: Optional[dict] = None,
-            grouped: Optional[dict] = None, cta_pair: int = 0, pair_splits: int = 0) -> torch.Tensor:
+            grouped: Optional[dict] = None, cta_pair: int = 0, pair_splits: int = 0,
+            act_params: Optional[tuple] = None) -> torch.Tensor:
     """``out[M, N] = act(x[M, K] @ w[N, K]^T * out_scale + bias) + residual`` on tcgen05 tensor cores.
 
     ``dual_rows = I`` switches to the gated form: ``w`` is ``[2*I, K]`` with gate rows first and the
     result is ``act(x @ w[:I]^T) * (x @ w[I:]^T)`` of shape ``[M, I]``.
     With fp32 operands everything runs in 32-bit arithmetic and the result is fp32.
+    ``act_params``: the two coefficients of ``act="xielu"``.
     ``rs`` / ``ag`` carry the peer pointers for the fused reduce-scatter / all-gather variants (see
     :mod:`unillm_b200.dist.fused`).
     """
@@ -125,6 +127,8 @@ def gemm_tn(x: torch.Tensor, w: torch.Tensor, *, bias: Optional[torch.Tensor] = 
     a.ldx, a.ldw, a.ldo = x.stride(0), w.stride(0), out.stride(0)
     a.ldr = residual.stride(0) if residual is not None else 0
     a.act = N.ACT[act]
+    if act_params is not None:
+        a.act_a, a.act_b = act_params
     a.dual = 1 if dual else 0
     a.up_row_off = dual_rows
     a.w_rows_total = w.shape[0]
@@ -228,7 +232,7 @@ def norm(x: torch.Tensor, weight: Optional[torch.Tensor], *, bias: Optional[torc
 # ---------------------------------------------------------------------------------------------
 # Norms around a 32-bit residual stream
 # ---------------------------------------------------------------------------------------------
-def _resid_args(what: str, x: torch.Tensor, weight, bias, out, H: int, eps: float, kind: str):
+def _resid_args(what: str, x: torch.Tensor, weight, bias, out, H: int, eps: float, kind: str, offset_one: bool = False):
     f32 = _elem(what, weight, bias, out)
     if x.dtype != torch.float32 or x.dim() != 2 or not x.is_contiguous() or out.shape[1:] != x.shape[1:]:
         raise ValueError(f"{what}: the residual stream is a contiguous fp32 [T, width] tensor, out has its rows' size")
@@ -239,19 +243,22 @@ def _resid_args(what: str, x: torch.Tensor, weight, bias, out, H: int, eps: floa
     a.err = err_word(x.device).data_ptr()
     a.T, a.H, a.Hp, a.x_rows = out.shape[0], H, x.shape[1], x.shape[0]
     a.kind, a.f32, a.eps = (0 if kind == "rms" else 1), int(f32), eps
+    a.w_off = 1.0 if offset_one else 0.0
     return a
 
 
 def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tensor, bias: Optional[torch.Tensor] = None, *,
                   eps: float, kind: str = "rms", width: Optional[int] = None, out: Optional[torch.Tensor] = None,
-                  experts: Optional[torch.Tensor] = None, routing: Optional["MoeRouting"] = None) -> torch.Tensor:
+                  experts: Optional[torch.Tensor] = None, routing: Optional["MoeRouting"] = None,
+                  offset_one: bool = False) -> torch.Tensor:
     """``x += norm(y)`` on the fp32 residual stream ``x`` (in place); returns the new rows in the type of ``weight``.
 
     ``experts`` / ``routing``: the rows to be normalised are ``y + sum_k w[t, k] * experts[row_slot[t, k]]`` (``y`` may then
-    be None).  ``width``: real row size when rows are zero-padded to a multiple of 8."""
+    be None).  ``width``: real row size when rows are zero-padded to a multiple of 8.  ``offset_one``: norm weights are
+    stored around zero."""
     if out is None:
         out = torch.empty(x.shape, dtype=weight.dtype, device=x.device)
-    a = _resid_args("residual_norm", x, weight, bias, out, width or x.shape[1], eps, kind)
+    a = _resid_args("residual_norm", x, weight, bias, out, width or x.shape[1], eps, kind, offset_one)
     for t in (y, experts):
         if t is not None and (t.dtype != weight.dtype or t.shape[1] != x.shape[1] or not t.is_contiguous()):
             raise ValueError("residual_norm: sublayer rows must be contiguous, of the weights' type and the stream's width")
@@ -268,13 +275,13 @@ def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], weight: torch.Tens
 
 
 def row_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None, *, eps: float, kind: str = "rms",
-             rows: Optional[torch.Tensor] = None, width: Optional[int] = None) -> torch.Tensor:
+             rows: Optional[torch.Tensor] = None, width: Optional[int] = None, offset_one: bool = False) -> torch.Tensor:
     """``norm(x[rows])`` of an fp32 residual stream (all rows when ``rows`` is None) in the type of ``weight``."""
     if rows is not None and rows.dtype != torch.int32:
         raise TypeError("rows must be int32")
     n = x.shape[0] if rows is None else rows.numel()
     out = torch.empty(n, x.shape[1], dtype=weight.dtype, device=x.device)
-    a = _resid_args("row_norm", x, weight, bias, out, width or x.shape[1], eps, kind)
+    a = _resid_args("row_norm", x, weight, bias, out, width or x.shape[1], eps, kind, offset_one)
     a.rows = _p(rows)
     N.check(N.cuda_lib().ub_row_norm(C.byref(a), _stream(x)), "ub_row_norm")
     return out
@@ -294,6 +301,244 @@ def embed_residual(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0):
     N.check(lib.ub_embed_residual(ids.data_ptr(), table.data_ptr(), x.data_ptr(), out.data_ptr(), T, Hp, V, scale, int(f32),
                                   err_word(table.device).data_ptr(), _stream(table)), "ub_embed_residual")
     return x, out
+
+
+# ---------------------------------------------------------------------------------------------
+# Layers with carried state: input of a sublayer, wkv recurrence
+# ---------------------------------------------------------------------------------------------
+class Portions:
+    """Rows [row0, row0 + rows) of a step as portions of sequences: ``q_start`` (int32 [n + 1], from 0) or one row per
+    sequence; ``state_in`` / ``state_out`` int32 [n] rows of the state tensors (negative: none)."""
+
+    __slots__ = ("row0", "rows", "n", "max_q", "q_start", "state_in", "state_out")
+
+    def __init__(self, row0: int, rows: int, n: int, max_q: int, q_start, state_in, state_out):
+        for t, k in ((q_start, n + 1), (state_in, n), (state_out, n)):
+            if t is not None and (t.dtype != torch.int32 or t.numel() != k or not t.is_cuda):
+                raise ValueError("portions: int32 CUDA tensors, one entry per sequence")
+        if q_start is None and (rows != n or max_q != 1):
+            raise ValueError("portions: without q_start every sequence has one row")
+        self.row0, self.rows, self.n, self.max_q = row0, rows, n, max_q
+        self.q_start, self.state_in, self.state_out = q_start, state_in, state_out
+
+
+def _state_rows(what: str, t: Optional[torch.Tensor], tail: tuple) -> None:
+    if t is not None and (t.dtype != torch.float32 or not t.is_contiguous() or tuple(t.shape[1:]) != tail):
+        raise ValueError(f"{what}: state must be contiguous fp32 [rows, {', '.join(map(str, tail))}]")
+
+
+def sublayer_in(x: torch.Tensor, portions: Sequence[Portions], weight: torch.Tensor, *, eps: float, y: Optional[torch.Tensor] = None,
+                y_weight: Optional[torch.Tensor] = None, conv: Optional[torch.Tensor] = None,
+                conv_state: Optional[torch.Tensor] = None, mu: Optional[torch.Tensor] = None,
+                shift_state: Optional[torch.Tensor] = None, width: Optional[int] = None, offset_one: bool = True, tile: int = 0):
+    """What the next sublayer reads: ``x' = x + norm(y)``, ``h = norm(x')`` plus its causal convolution over time with the taps
+    ``conv`` (fp32 [taps, width], the last one meets the token itself), and with ``mu`` (fp32 [n, width]) the n token-shift
+    mixes ``h + (previous h - h) * mu``.  Returns ``(x', out)``; out is [rows, width], or [n, rows, width] with ``mu``, in
+    the type of ``weight``.  The state tensors hold what the sequences of ``portions`` carry on."""
+    f32 = _elem("sublayer_in", weight, y, y_weight)
+    T, Hp = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or weight.numel() != Hp:
+        raise ValueError("sublayer_in: contiguous fp32 stream, weights of its width")
+    if y is not None and (y.shape != x.shape or not y.is_contiguous() or y_weight is None or y_weight.numel() != Hp):
+        raise ValueError("sublayer_in: y has the stream's shape and a norm weight")
+    taps = 0 if conv is None else conv.shape[0]
+    n_mix = 0 if mu is None else mu.shape[0]
+    for t in (conv, mu):
+        if t is not None and (t.dtype != torch.float32 or t.shape[1] != Hp or not t.is_contiguous()):
+            raise ValueError("sublayer_in: conv and mu are contiguous fp32 [n, width]")
+    _state_rows("sublayer_in conv", conv_state, (max(taps - 1, 0), Hp))
+    _state_rows("sublayer_in shift", shift_state, (Hp,))
+    states = [t for t in (conv_state, shift_state) if t is not None]
+    out = torch.empty((n_mix, T, Hp) if n_mix else (T, Hp), dtype=weight.dtype, device=x.device)
+    x_out = x if y is None else torch.empty_like(x)
+    for p in portions:
+        if p.row0 + p.rows > T:
+            raise ValueError("sublayer_in: portions outside the step")
+        a = N.UbSublayerInArgs()
+        a.x, a.y, a.wy, a.x_out, a.wn = x.data_ptr(), _p(y), _p(y_weight), x_out.data_ptr(), weight.data_ptr()
+        a.conv, a.conv_state, a.mu, a.shift_state, a.out = _p(conv), _p(conv_state), _p(mu), _p(shift_state), out.data_ptr()
+        if states:
+            a.state_in, a.state_out = _p(p.state_in), _p(p.state_out)
+            a.state_rows = states[0].shape[0]
+        a.q_start, a.err = _p(p.q_start), err_word(x.device).data_ptr()
+        a.row0, a.out_mix_stride = p.row0, T * Hp
+        a.H, a.Hp, a.taps, a.n_mix, a.num_seqs, a.max_q = width or Hp, Hp, taps, n_mix, p.n, p.max_q
+        # rows in front of a tile are computed again: larger tiles once there are enough of them for the SMs
+        a.tile = tile or (1 if p.max_q == 1 else 4 if p.rows <= 1024 else 8 if p.rows <= 4096 else 16)
+        a.f32, a.eps, a.w_off = int(f32), eps, 1.0 if offset_one else 0.0
+        N.check(N.cuda_lib().ub_sublayer_in(C.byref(a), _stream(x)), "ub_sublayer_in")
+    return x_out, out
+
+
+WKV_CHUNK = 64
+
+
+def wkv_mixer(rkvg: torch.Tensor, ww: torch.Tensor, u: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor,
+              portions: Sequence[Portions], *, eps: float, norm_dim: int = 0, chunk: Optional[int] = None) -> torch.Tensor:
+    """RWKV-6 style recurrence with head norm and SiLU gate: ``rkvg`` [4, T, H * D], ``ww`` fp32 [T, H * D] (decay =
+    exp(-exp(ww))), ``u`` fp32 [H, D], ``norm_w`` fp32 [H * D], ``state`` fp32 [rows, H, D, D] -> [T, H * D].  ``chunk``:
+    tokens per parallel chunk of long portions (0 = one CTA walks a portion, None = chosen here)."""
+    f32 = _elem("wkv_mixer", rkvg)
+    _, T, ld = rkvg.shape
+    H, D = u.shape
+    if not rkvg.is_contiguous() or ld != H * D or ww.dtype != torch.float32 or ww.shape != (T, ld) or not ww.is_contiguous():
+        raise ValueError("wkv_mixer: rkvg [4, T, H * D] and fp32 ww [T, H * D], contiguous")
+    if u.dtype != torch.float32 or norm_w.dtype != torch.float32 or norm_w.numel() != ld:
+        raise ValueError("wkv_mixer: fp32 u [H, D] and norm weight [H * D]")
+    _state_rows("wkv_mixer", state, (H, D, D))
+    out = torch.empty(T, ld, dtype=rkvg.dtype, device=rkvg.device)
+    lib = N.cuda_lib()
+    for p in portions:
+        if p.row0 + p.rows > T:
+            raise ValueError("wkv_mixer: portions outside the step")
+        a = N.UbWkvArgs()
+        e = rkvg.element_size() * T * ld
+        a.r, a.k, a.v, a.g = (rkvg.data_ptr() + i * e for i in range(4))
+        a.ww, a.u, a.norm_w, a.state, a.out = ww.data_ptr(), u.data_ptr(), norm_w.data_ptr(), state.data_ptr(), out.data_ptr()
+        a.state_in, a.state_out, a.q_start, a.err = _p(p.state_in), _p(p.state_out), _p(p.q_start), err_word(rkvg.device).data_ptr()
+        a.row0, a.ld, a.H, a.D, a.norm_dim, a.num_seqs = p.row0, ld, H, D, norm_dim or D, p.n
+        a.state_rows, a.f32, a.eps = state.shape[0], int(f32), eps
+        c = chunk
+        if c is None:       # chunks pay once a portion is long and the sequences alone do not fill the device
+            c = WKV_CHUNK if p.max_q > 2 * WKV_CHUNK and p.n * H < 4 * 148 else 0
+        if p.q_start is None:
+            c = 0
+        if c:
+            a.chunk, a.rows, a.max_chunks = c, p.rows, p.rows // c + p.n
+            ws = torch.empty(lib.ub_wkv_workspace_floats(p.rows, ld, H, D, a.max_chunks), dtype=torch.float32, device=rkvg.device)
+            a.ws = ws.data_ptr()
+        N.check(lib.ub_wkv_mixer(C.byref(a), _stream(rkvg)), "ub_wkv_mixer")
+    return out
+
+
+_GROUP_TILES: dict = {}
+
+
+def gemm_stacked(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """``out[e] = x[e] @ w[e]^T`` for a stack of equal products: x [E, T, K] (contiguous), w [E, N, K] -> [E, T, N].  Up to 16
+    rows on the weight-streaming kernel, beyond on the grouped GEMM with a tile table that is fixed by the sizes."""
+    f32 = _elem("gemm_stacked", x, w)
+    E, T, Kd = x.shape
+    n = w.shape[1]
+    if not x.is_contiguous() or not w.is_contiguous() or w.shape[0] != E or w.shape[2] != Kd:
+        raise ValueError("gemm_stacked: contiguous x [E, T, K] and w [E, N, K]")
+    out = torch.empty(E, T, n, dtype=x.dtype, device=x.device)
+    if T <= 16 and not f32:
+        a = N.UbGemmArgs()
+        a.x, a.w, a.out, a.err = x.data_ptr(), w.data_ptr(), out.data_ptr(), err_word(x.device).data_ptr()
+        a.M, a.N, a.K, a.ldx, a.ldw, a.ldo, a.w_rows_total = T, n, Kd, Kd, Kd, n, n
+        a.batch, a.x_batch, a.w_batch, a.out_batch = E, T * Kd, n * Kd, T * n
+        N.check(N.cuda_lib().ub_gemm_tn(C.byref(a), _stream(x)), "ub_gemm_tn(stacked)")
+        return out
+    tn = moe_tile_tokens(E * T, 1, E)
+    key = (E, T, tn, x.device)
+    tiles = _GROUP_TILES.get(key)
+    if tiles is None:
+        rows = [[e, e * T + t, (e + 1) * T, 0] for e in range(E) for t in range(0, T, tn)]
+        tiles = _GROUP_TILES[key] = torch.tensor(rows, dtype=torch.int32).to(x.device)
+    _gemm_grouped_plain(x.view(E * T, Kd), w.view(E * n, Kd), n, None, out.view(E * T, n),
+                        {"tiles": tiles.data_ptr(), "max_tiles": tiles.shape[0], "w_rows": n, "tile_tokens": tn}, f32)
+    return out
+
+
+# ---------------------------------------------------------------------------------------------
+# Multi-head latent attention
+# ---------------------------------------------------------------------------------------------
+def _latent_args(T: int, positions, inv_freq, rot: int, f32: bool, gain: float, device):
+    if positions.dtype != torch.int32 or inv_freq.dtype != torch.float32 or positions.numel() != T:
+        raise TypeError("latent attention: int32 positions, fp32 frequencies")
+    a = N.UbLatentArgs()
+    a.positions, a.inv_freq, a.err = positions.data_ptr(), inv_freq.data_ptr(), err_word(device).data_ptr()
+    a.T, a.rot, a.rot_dims, a.f32, a.gain = T, rot, 2 * inv_freq.numel(), int(f32), gain
+    return a
+
+
+def latent_rows(down: torch.Tensor, positions: torch.Tensor, slot_mapping: torch.Tensor, cache: torch.Tensor, q_norm_w: torch.Tensor,
+                kv_norm_w: torch.Tensor, inv_freq: torch.Tensor, *, eps: float, gain: float = 1.0, q_real: int = 0,
+                kv_real: int = 0) -> torch.Tensor:
+    """``down`` [T, q_rank + kv_rank + rot] -> normed query latents [T, q_rank]; the normed kv latent and the rotated key part
+    go to the rows ``slot_mapping`` of ``cache`` [num_blocks, 1, block_size, kv_rank + rot].  ``q_real`` / ``kv_real``:
+    elements that the norms average over when segments are padded."""
+    f32 = _elem("latent_rows", down, cache, q_norm_w, kv_norm_w)
+    T, qr, kvr = down.shape[0], q_norm_w.numel(), kv_norm_w.numel()
+    rot = down.shape[1] - qr - kvr
+    if cache.shape[-1] != kvr + rot or cache.shape[1] != 1 or not cache.is_contiguous() or not down.is_contiguous():
+        raise ValueError("latent_rows: cache rows are [kv latent | rotated part]")
+    if slot_mapping.dtype != torch.int32 or slot_mapping.numel() != T:
+        raise TypeError("latent_rows: int32 slots, one per token")
+    out = torch.empty(T, qr, dtype=down.dtype, device=down.device)
+    a = _latent_args(T, positions, inv_freq, rot, f32, gain, down.device)
+    a.down, a.q_latent, a.cache, a.q_norm_w, a.kv_norm_w = down.data_ptr(), out.data_ptr(), cache.data_ptr(), q_norm_w.data_ptr(), kv_norm_w.data_ptr()
+    a.slot_mapping, a.num_slots = slot_mapping.data_ptr(), cache.shape[0] * cache.shape[2]
+    a.q_rank, a.kv_rank, a.q_real, a.kv_real, a.eps = qr, kvr, q_real or qr, kv_real or kvr, eps
+    N.check(N.cuda_lib().ub_latent_rows(C.byref(a), _stream(down)), "ub_latent_rows")
+    return out
+
+
+def latent_rotate(q: torch.Tensor, positions: torch.Tensor, inv_freq: torch.Tensor, rot: int, out: Optional[torch.Tensor] = None,
+                  gain: float = 1.0) -> torch.Tensor:
+    """Turns the last ``rot`` elements of every head of ``q`` [T, heads, size] (rows may be strided) and puts them last in the
+    heads of ``out`` (default: in place)."""
+    out = q if out is None else out
+    f32 = _elem("latent_rotate", q, out)
+    T, H = q.shape[:2]
+    if q.stride(2) != 1 or out.stride(2) != 1 or out.shape[:2] != q.shape[:2]:
+        raise ValueError("latent_rotate: heads must be contiguous")
+    a = _latent_args(T, positions, inv_freq, rot, f32, gain, q.device)
+    a.H, a.q, a.q_out = H, q.data_ptr(), out.data_ptr()
+    a.q_stride, a.q_head, a.q_off = q.stride(0), q.stride(1), q.shape[2] - rot
+    a.qo_stride, a.qo_head, a.qo_off = out.stride(0), out.stride(1), out.shape[2] - rot
+    N.check(N.cuda_lib().ub_latent_rotate(C.byref(a), _stream(q)), "ub_latent_rotate")
+    return out
+
+
+def gemm_heads(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out[t, h] = x[t, h] @ w[h]^T``: x [T, H, K] and out [T, H, N] with any token and head strides, w [H, N, K]."""
+    f32 = _elem("gemm_heads", x, w, out)
+    T, H, Kd = x.shape
+    if w.shape != (H, out.shape[2], Kd) or out.shape[:2] != (T, H) or x.stride(2) != 1 or out.stride(2) != 1 or not w.is_contiguous():
+        raise ValueError("gemm_heads: x [T, H, K], w [H, N, K], out [T, H, N]")
+    a = N.UbHeadGemmArgs()
+    a.x, a.w, a.out = x.data_ptr(), w.data_ptr(), out.data_ptr()
+    a.x_stride, a.x_head, a.out_stride, a.out_head = x.stride(0), x.stride(1), out.stride(0), out.stride(1)
+    a.M, a.N, a.K, a.H, a.f32 = T, w.shape[1], Kd, H, int(f32)
+    N.check(N.cuda_lib().ub_gemm_heads(C.byref(a), _stream(x)), "ub_gemm_heads")
+    return out
+
+
+def attn_latent(q: torch.Tensor, cache: torch.Tensor, v_dim: int, block_tables: torch.Tensor, seq_lens: torch.Tensor, *, scale: float,
+                sinks: Optional[torch.Tensor] = None, q_start: Optional[torch.Tensor] = None, max_q_len: int = 1,
+                out: Optional[torch.Tensor] = None, splits: int = 0, scratch: Optional[torch.Tensor] = None,
+                max_seq_len: Optional[int] = None) -> torch.Tensor:
+    """Attention of all heads over one cached row per token: q [T, H, D], cache [num_blocks, 1, block_size, D]; keys are the
+    rows, values their first ``v_dim`` elements -> [T, H, v_dim].  With ``q_start`` prompt portions, else one query per
+    sequence; causal."""
+    f32 = _elem("attn_latent", q, cache, out)
+    T, H, D = q.shape
+    if cache.shape[1] != 1 or cache.shape[3] != D or not cache.is_contiguous() or q.stride(1) != D or q.stride(2) != 1:
+        raise ValueError("attn_latent: cache rows and query heads of one size")
+    if out is None:
+        out = torch.empty(T, H, v_dim, dtype=q.dtype, device=q.device)
+    a = _attn_args(q, cache, cache[..., :v_dim], out, None, block_tables, seq_lens, H, 1, D, scale, sinks)
+    a.kv_shared, a.causal = 1, 1
+    if q_start is not None or f32:
+        splits = 1
+    if splits <= 0:
+        ctx = max_seq_len if max_seq_len is not None else block_tables.shape[1] * cache.shape[2]
+        ctas, splits = T * -(-H // (16 if H <= 16 else 32)), 1
+        while ctas * splits < 148 and ctx // (splits * 2) >= 128 and splits < 16:
+            splits *= 2
+    if splits > 1:
+        need = T * H * splits * (v_dim + 2)
+        if scratch is None or scratch.numel() < need:
+            scratch = torch.empty(need, dtype=torch.float32, device=q.device)
+        a.scratch = scratch.data_ptr()
+    a.splits = splits
+    if q_start is not None:
+        a.q_start, a.total_q, a.max_q_len = q_start.data_ptr(), T, max_q_len
+    lib = N.cuda_lib()
+    N.check((lib.ub_attn_f32 if f32 else lib.ub_attn_latent)(C.byref(a), _stream(q)), "ub_attn_latent")
+    return out
 
 
 # ---------------------------------------------------------------------------------------------
