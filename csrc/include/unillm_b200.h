@@ -286,6 +286,26 @@ typedef struct UbAttnArgs {
   int Dv;                    /* value head size (0 = D): v_cache [.., Dv], out [T, Hq, Dv], scratch [.., Dv + 2] */
   int kv_shared;             /* ub_attn_f32: values are the first Dv elements of the key rows (ub_attn_latent: always so) */
 } UbAttnArgs;
+/* prompts over expanded latents (csrc/attn/attn_expanded_tc.cu): ub_latent_gather copies the cache rows of the sequences to
+   consecutive rows (each sequence from page_start[seq] * 16 on, zeros behind its end and up to `rows`), ub_attn_expanded
+   runs the attention on tcgen05 */
+typedef struct UbExpandArgs {
+  const void* cache;         /* bf16 [num_blocks, 16, row] */
+  void* lat;                 /* bf16 [rows, row], row = kv_rank + rot */
+  const void* q;             /* bf16 [T, H, dim + rot], rotated, tokens q_stride apart */
+  const void* kv;            /* bf16 [rows, H, dim + vdim]: unrotated key, value */
+  void* out;                 /* bf16 [T, H, vdim], tokens o_stride apart */
+  const float* sinks;        /* [H] or NULL */
+  const int *block_tables, *seq_lens, *q_start;
+  const int* page_start;     /* [num_seqs + 1] first 16-row page of every sequence */
+  int* err;
+  long long q_stride, o_stride;
+  int T, H, dim, rot, vdim, kv_rank, row, rows, num_seqs, max_q, block_size, num_blocks, max_blocks_per_seq;
+  float scale;
+} UbExpandArgs;
+int ub_latent_gather(const UbExpandArgs* args, void* stream);
+int ub_attn_expanded(const UbExpandArgs* args, void* stream);
+int ub_attn_expanded_supported(int dim, int rot, int vdim);
 /* one cache row per token for all heads: key = the row [D], value = its first Dv elements (csrc/attn/attn_latent.cu) */
 int ub_attn_latent(const UbAttnArgs* args, void* stream);
 /* merges the partials that a decode kernel left in args->scratch */

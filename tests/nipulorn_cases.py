@@ -46,7 +46,7 @@ CASES = {
     # one tap: no carried inputs; recurrences only
     "short": _cfg(96, 64, 1, [_wkv(4, 16, 32), _wkv(2, 40)]),
     # one tap and attention only: nothing is carried but the cache
-    "plain": _cfg(40, 72, 1, [_latent(4, 24, 24, 24, 32, 8, 0.25, 48), _latent(2, 8, 32, 40, 24, 16, 0.3)]),
+    "plain": _cfg(40, 72, 1, [_latent(4, 24, 24, 24, 32, 8, 0.25, 48), _latent(2, 32, 48, 40, 96, 16, 0.2)]),
 }
 
 
@@ -87,7 +87,8 @@ def make_weights(cfg, seed=0):
             w[p + "sink"], w[p + "o"] = vec(n, 1.0, 1.0), mat(H, n * m["vdim"])
         if lay["mlp"] is not None:
             ff = lay["mlp"]["ff"]
-            w[L + "mlp.up"], w[L + "mlp.down"], w[L + "mlp.act"] = mat(ff, H, 1.5), mat(H, ff), vec(2, 0.3, 0.8)
+            w[L + "mlp.up"], w[L + "mlp.down"], w[L + "mlp.act"] = mat(ff, H, 1.5), mat(H, ff), \
+                torch.tensor([-1.5, 1.5]) + 0.5 * torch.randn(2, generator=g)
     return {k: t.to(torch.bfloat16) for k, t in w.items()}
 
 

@@ -1,5 +1,5 @@
 """Prefill and decode throughput of one design beside the closest existing family at equal size, and the same
-comparison kernel by kernel (``python bench.py --design gekapel [--design-kernels]``).
+comparison kernel by kernel (``python bench.py --design gekapel|nipulorn [--design-kernels]``).
 
 Both models are random-weight stacks of a few layers with a real model's layer sizes, run by the same
 ``GpuModelRunner`` steps that serve requests: a prefill step is one batch of whole prompts, a decode step one token of
@@ -12,6 +12,11 @@ over the bf16 matrix throughput (MEASURED_PEAKS.json).
 
 The closest family to Gekapel is DeepSeek-MoE (routed experts plus always-on ones), here with Mistral's sliding window.
 Its experts have a gate, so at equal size they are two thirds as wide.
+
+Nipulorn's parts have two nearest relatives.  Whole steps are set beside Llama, the dense full-attention decoder of the same
+runner, with its feed-forward as wide as makes the parameters equal; the recurrence is set beside RWKV-6's kernel (a model
+of the whole-model path) at the same heads, tokens and state.  Arithmetic that is fp32 by design counts against the FMA
+rate of the device instead of the matrix rate.
 """
 from __future__ import annotations
 
@@ -23,7 +28,7 @@ import torch
 
 from ..engine.runner import GpuModelRunner, RunnerWeights, StepBatch
 from ..models import configs as C
-from ..models.families import GekapelModel
+from ..models.families import GekapelModel, NipulornModel
 from ..models.spec import DecoderSpec, MoESpec
 from ..ops import cuda_ops as K
 from .microbench import _peaks, time_ms
@@ -62,7 +67,47 @@ def closest_spec(z: dict) -> DecoderSpec:
                                    shared_intermediate_size=z["shared"] * 2 // 3))
 
 
-ARMS = {"gekapel": gekapel_spec, "deepseek_moe + window": closest_spec}
+# width, wkv heads and size, latent attention (heads, dim, vdim, q rank, kv rank, rotated), feed-forward, vocabulary, layers
+# (three wkv layers, then one of latent attention with a feed-forward)
+NIPULORN_SIZES = {
+    "1k": dict(width=1024, wkv=16, wdim=64, heads=16, dim=64, vdim=64, q_rank=384, kv_rank=256, rot=32, ff=4096, vocab=32000, layers=4),
+    "2k": dict(width=2048, wkv=32, wdim=64, heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, rot=64, ff=8192, vocab=32000, layers=4),
+    "4k": dict(width=4096, wkv=64, wdim=64, heads=32, dim=128, vdim=128, q_rank=1536, kv_rank=512, rot=64, ff=16384, vocab=32000, layers=4),
+}
+
+
+def nipulorn_spec(z: dict) -> DecoderSpec:
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 != 3:
+            layers.append({"type": "wkv", "mixer": {"heads": z["wkv"], "dim": z["wdim"]}, "mlp": None})
+            continue
+        layers.append({"type": "latent_attention", "mlp": {"kind": "dense", "ff": z["ff"]},
+                       "mixer": {"heads": z["heads"], "dim": z["dim"], "vdim": z["vdim"], "q_rank": z["q_rank"], "kv_rank": z["kv_rank"],
+                                 "rot_dim": z["rot"], "scale": (z["dim"] + z["rot"]) ** -0.5,
+                                 "rot": {"base": 10000.0, "dims": z["rot"],
+                                         "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}})
+    return NipulornModel.spec_from_config(C.NipulornConfig(vocab_size=z["vocab"], hidden_size=z["width"], num_hidden_layers=z["layers"],
+                                                           canon_taps=4, logit_scale=0.5, embedding_scale=z["width"] ** 0.5, layers=layers))
+
+
+def llama_spec(z: dict) -> DecoderSpec:
+    """As many parameters in the layers, in a dense decoder with the same attention heads over full-size keys."""
+    H, d, n = z["width"], z["dim"], z["layers"]
+    hq, hkv = H // d, max(1, H // d // 4)
+    wkv = 5 * H * z["wkv"] * z["wdim"] + 64 * (H + z["wkv"] * z["wdim"])
+    lat = H * (z["q_rank"] + z["kv_rank"] + z["rot"]) + z["q_rank"] * z["heads"] * (d + z["rot"]) + \
+        z["kv_rank"] * z["heads"] * (d + z["vdim"]) + H * z["heads"] * z["vdim"] + 2 * H * z["ff"]
+    total = n // 4 * (3 * wkv + lat)
+    attn = H * d * (hq + 2 * hkv) + H * hq * d
+    ff = (total - n * attn) // (n * 3 * H) // 128 * 128
+    return DecoderSpec(vocab_size=z["vocab"], hidden_size=H, num_layers=n, num_heads=hq, num_kv_heads=hkv, head_dim=d,
+                       intermediate_size=ff, max_position_embeddings=8192, tie_embeddings=True)
+
+
+DESIGNS = {"gekapel": (SIZES, {"gekapel": gekapel_spec, "deepseek_moe + window": closest_spec}),
+           "nipulorn": (NIPULORN_SIZES, {"nipulorn": nipulorn_spec, "llama": llama_spec})}
+FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12      # FMA pipe at the maximum clock
 
 
 def _runner(spec: DecoderSpec, tokens: int, max_len: int, seqs: int) -> GpuModelRunner:
@@ -71,8 +116,16 @@ def _runner(spec: DecoderSpec, tokens: int, max_len: int, seqs: int) -> GpuModel
                           max_model_len=max_len)
 
 
-def _batch(vocab: int, seqs: int, context: int, decode: bool, seed: int = 0) -> StepBatch:
+def _batch(spec: DecoderSpec, seqs: int, context: int, decode: bool, seed: int = 0) -> StepBatch:
     """Whole prompts of ``context`` tokens, or one token of every sequence at position ``context - 1``."""
+    b = _token_batch(spec.vocab_size, seqs, context, decode, seed)
+    if spec.has_state:
+        b.state_in = [2 * s if decode else -1 for s in range(seqs)]
+        b.state_out = [2 * s + 1 for s in range(seqs)]
+    return b
+
+
+def _token_batch(vocab: int, seqs: int, context: int, decode: bool, seed: int) -> StepBatch:
     g = torch.Generator().manual_seed(seed)
     nb = -(-context // 16)
     tables = [list(range(s * nb, (s + 1) * nb)) for s in range(seqs)]
@@ -106,7 +159,8 @@ def step_ms(runner: GpuModelRunner, b: StepBatch, iters: int = 20, warmup: int =
 # kernel by kernel
 # ------------------------------------------------------------------------------------------------
 RECORDED = ("gemm_tn", "grouped_gemm", "norm", "residual_norm", "row_norm", "embed_residual", "embed_gather", "rope_kv_append",
-            "attn_decode", "attn_prefill", "moe_route", "moe_gather", "moe_combine", "sample")
+            "attn_decode", "attn_prefill", "moe_route", "moe_gather", "moe_combine", "sample", "sublayer_in", "wkv_mixer",
+            "gemm_stacked", "latent_rows", "latent_rotate", "gemm_heads", "attn_latent", "latent_gather", "attn_expanded")
 
 
 @contextlib.contextmanager
@@ -141,7 +195,40 @@ def _nbytes(*ts) -> int:
 
 
 def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
-    """(label, bytes moved, multiply-add flops) of one call, counting every operand once."""
+    """(label, bytes moved, flops of the matrix pipe[, flops of the fp32 pipe]) of one call, counting every operand once."""
+    q_lens = [1] * b.num_decode + list(b.prefill_q_lens)
+    pairs_all = sum(q * n - q * (q - 1) // 2 for q, n in zip(q_lens, b.seq_lens))
+    if name == "sublayer_in":
+        x, parts = a[0], a[1]
+        live = sum(p.n for p in parts)
+        state = sum(2 * live * t[0].numel() * 4 for t in (kw.get("conv_state"), kw.get("shift_state")) if t is not None)
+        return (f"norms + conv" + (" + mixes" if kw.get("mu") is not None else ""),
+                _nbytes(x, kw.get("y"), r[1]) + (_nbytes(x) if kw.get("y") is not None else 0) + state, 0.0)
+    if name == "wkv_mixer":
+        rkvg, ww, u, st, parts = a[0], a[1], a[2], a[4], a[5]
+        per = st[0].numel()
+        live = sum(p.n for p in parts)
+        reads = live if b.num_decode else 0              # prompts start from nothing
+        return "wkv", _nbytes(rkvg, ww, r) + 4 * per * (live + reads), 0.0, 5.0 * rkvg.shape[1] * per
+    if name == "gemm_stacked":
+        x, w = a
+        return f"stacked gemm {x.shape[0]}x[{x.shape[1]}x{w.shape[1]}x{w.shape[2]}]", _nbytes(x, w, r), 2.0 * x.shape[1] * w.numel()
+    if name == "latent_rows":
+        return "latent norms + rotation + append", 2 * _nbytes(a[0]), 0.0
+    if name == "latent_rotate":
+        return "query rotation", 2 * a[0].shape[0] * a[0].shape[1] * a[3] * a[0].element_size(), 0.0
+    if name == "gemm_heads":
+        return (f"head gemm {a[0].shape[1]}x[{a[0].shape[0]}x{a[1].shape[1]}x{a[1].shape[2]}]", _nbytes(*a), 2.0 * a[0].shape[0] * a[1].numel())
+    if name == "attn_latent":
+        q, kc = a[0], a[1]
+        return (("attn_latent (prompt)" if kw.get("q_start") is not None else "attn_latent (decode)"),
+                _nbytes(q, r) + sum(b.seq_lens) * kc.shape[3] * kc.element_size(), 2.0 * pairs_all * q.shape[1] * (kc.shape[3] + a[2]))
+    if name == "latent_gather":
+        return "gather of cached latents", 2 * _nbytes(r), 0.0
+    if name == "attn_expanded":
+        q, kv, lat, vd = a[0], a[1], a[2], a[3]
+        return "attn_expanded", _nbytes(q, kv, r) + lat.shape[0] * 2 * (q.shape[2] - kv.shape[1] // q.shape[1] + vd), \
+            2.0 * pairs_all * q.shape[1] * (q.shape[2] + vd)
     if name == "gemm_tn":
         x, w = a[0], a[1]
         return (f"gemm {x.shape[0]}x{w.shape[0]}x{w.shape[1]}", _nbytes(x, w, r, kw.get("residual")),
@@ -197,28 +284,46 @@ def kernel_rows(runner: GpuModelRunner, b: StepBatch) -> List[dict]:
     torch.cuda.synchronize()
     rows: Dict[str, dict] = {}
     for name, fn, a, kw, r in calls:
-        label, nbytes, flops = _cost(name, a, kw, r, b)
+        label, nbytes, flops, *f32 = _cost(name, a, kw, r, b)
         if label in rows:
             rows[label]["calls"] += 1
             continue
         ms, _ = time_ms(lambda: fn(*a, **kw))
-        floor = max(nbytes / (hbm * 1e9), flops / (tf * 1e12)) * 1e6
+        floor = max(nbytes / (hbm * 1e9), flops / (tf * 1e12), (f32[0] if f32 else 0.0) / (FP32_TFLOPS * 1e12)) * 1e6
         rows[label] = {"kernel": label, "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2),
                        "fraction": round(floor / (ms * 1e3), 3)}
     return list(rows.values())
 
 
-def main(sizes: Optional[List[str]] = None, kernels: bool = False) -> List[dict]:
+def wkv6_row(z: dict, seqs: int, tokens: int) -> dict:
+    """RWKV-6's recurrence kernel at a Nipulorn layer's heads, in the same units as the table above (its output is neither
+    normalised nor gated, so it moves the gate's bytes less)."""
+    from ..ops import recurrent as R
+
+    hbm, _, _ = _peaks()
+    H, D = z["wkv"], z["wdim"]
+    g = torch.Generator(device="cuda").manual_seed(1)
+    r, k, v = (torch.randn(seqs, tokens, H * D, generator=g, device="cuda").to(torch.bfloat16) for _ in range(3))
+    w, u = torch.rand(seqs, tokens, H * D, generator=g, device="cuda") * 4 - 5, torch.randn(H * D, generator=g, device="cuda")
+    st = torch.zeros(seqs, H, D, D, device="cuda")
+    ms, _ = time_ms(lambda: R.wkv6(r, k, v, w, u, H, st))
+    nbytes = _nbytes(r, k, v, w, r) + 2 * _nbytes(st)
+    floor = max(nbytes / (hbm * 1e9), 5.0 * seqs * tokens * H * D * D / (FP32_TFLOPS * 1e12)) * 1e6
+    return {"kernel": "wkv6 (RWKV-6)", "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2), "fraction": round(floor / (ms * 1e3), 3)}
+
+
+def main(design: str = "gekapel", sizes: Optional[List[str]] = None, kernels: bool = False) -> List[dict]:
     out = []
-    for size in sizes or list(SIZES):
-        z = SIZES[size]
-        for arm, make in ARMS.items():
+    table, arms = DESIGNS[design]
+    for size in sizes or list(table):
+        z = table[size]
+        for arm, make in arms.items():
             spec = make(z)
             tokens = max([n * c for n, c in PREFILL] + [n * c for n, c in DECODE])
             runner = _runner(spec, tokens, max(c for _, c in PREFILL + DECODE) + 16, max(n for n, _ in DECODE))
             for kind, cases in (("prefill", PREFILL), ("decode", DECODE)):
                 for n, c in cases:
-                    b = _batch(spec.vocab_size, n, c, kind == "decode")
+                    b = _batch(spec, n, c, kind == "decode")
                     t = step_ms(runner, b)
                     row = {"size": size, "model": arm, "layers": spec.num_layers, "params_m": round(runner.w.nbytes() / 2e6),
                            "step": kind, "sequences": n, "context": c, **t,
@@ -226,7 +331,10 @@ def main(sizes: Optional[List[str]] = None, kernels: bool = False) -> List[dict]
                     out.append(row)
                     print(row, flush=True)
                     if kernels:
-                        for k in kernel_rows(runner, b):
+                        rows = kernel_rows(runner, b)
+                        if design == "nipulorn" and arm != "nipulorn":
+                            rows.append(wkv6_row(z, n, 1 if kind == "decode" else c))
+                        for k in rows:
                             out.append({"size": size, "model": arm, "step": kind, "sequences": n, "context": c, **k})
                             print("   ", k, flush=True)
             K.check_device_errors()

@@ -306,6 +306,8 @@ class RunnerWeights:
         uv = _pad(_pad(p[L + "w_uv"].reshape(n, ls.v_head_dim, ls.kv_rank), 1, kh.vdim), 2, kh.dv)
         t[L + "w_uk_t"] = dev(uk.transpose(1, 2))             # [heads, kv_rank, dim]: taken to the query side
         t[L + "w_uv"] = dev(uv)                               # [heads, vdim, kv_rank]
+        if self.dtype == torch.bfloat16 and self.expandable(i):
+            t[L + "w_ukv"] = dev(torch.cat([uk, uv], 1).flatten(0, 1))       # [heads * (dim + vdim), kv_rank]: long prompts
         if ls.sink:
             t[L + "sink"] = f32(p[L + "sink"])
         t[L + "wo"] = head_cols(p[L + "wo"], ls.v_head_dim, kh.vdim)
@@ -352,6 +354,11 @@ class RunnerWeights:
         """Cache bytes that one token takes on this rank over all layers that own keys and values."""
         e = torch.empty(0, dtype=self.dtype).element_size()
         return e * sum(k.cache_row for k in self.heads)
+
+    def expandable(self, i: int) -> bool:
+        """Layer ``i`` is latent attention of sizes that the tensor-core prompt kernel takes."""
+        kh = self.heads[i]
+        return self.spec.layer(i).mixer == "latent" and K.expanded_supported(kh.dim, kh.rot, kh.vdim)
 
     def state_bytes_per_seq(self) -> int:
         """Bytes of carried state of one live sequence (both halves of its slot)."""
@@ -512,6 +519,8 @@ class RunnerWeights:
                 self.t[L + "w_uq"] = rnd(kh.hq * (kh.dim + kh.rot), kh.q_rank)
                 self.t[L + "w_uk_t"] = rnd(kh.hq * kh.dv, kh.dim).view(kh.hq, kh.dv, kh.dim)
                 self.t[L + "w_uv"] = rnd(kh.hq * kh.vdim, kh.dv).view(kh.hq, kh.vdim, kh.dv)
+                if self.expandable(i):
+                    self.t[L + "w_ukv"] = torch.cat([self.t[L + "w_uk_t"].transpose(1, 2), self.t[L + "w_uv"]], 1).flatten(0, 1).contiguous()
                 self.t[L + "sink"], self.t[L + "wo"] = zeros(kh.hq).float(), rnd(H, kh.hq * kh.vdim)
                 continue
             self.t[L + "wqkv"] = rnd(kh.qkv_rows, H)
@@ -613,11 +622,12 @@ class TpContext:
 class StepPacker:
     """Packs a ``StepBatch`` into one int32 staging buffer (host-only logic, numpy views)."""
 
-    def __init__(self, buf: torch.Tensor, max_blocks_per_seq: int):
+    def __init__(self, buf: torch.Tensor, max_blocks_per_seq: int, kv_pages: bool = False):
         self.meta_host = buf
         self.np = buf.numpy()
         self.META_INTS = buf.numel()
         self.max_blocks_per_seq = max_blocks_per_seq
+        self.kv_pages = kv_pages
 
     @staticmethod
     def _bucket(n: int) -> int:
@@ -693,6 +703,15 @@ class StepPacker:
         for ql in q_lens:
             qs.append(qs[-1] + ql)
         put("q_start", qs)
+        if self.kv_pages and Pp:
+            # expanded prompts: where every sequence's rows start, in pages of 16, and a row count from a small set
+            pages, pairs = [0], 0
+            for n, q in zip(p_lens, q_lens):
+                pages.append(pages[-1] + (n + 15) // 16)
+                pairs += q * n - q * (q - 1) // 2
+            put("kv_pages", pages)
+            step = max(128, self._bucket(pages[-1] * 16) // 8)
+            lay["_kv_rows"], lay["_kv_pairs"] = -(-pages[-1] * 16 // step) * step, pairs
         if b.state_in is not None:
             for name, v in (("state_in", b.state_in), ("state_out", b.state_out)):
                 put(name, list(v[:D]) + [-1] * pad + list(v[D:]) + [-1] * (Pp - P))
@@ -794,7 +813,8 @@ class GpuModelRunner:
         # packed metadata: pinned host staging + device mirror with fixed addresses (graph friendly)
         # two staging buffers: the next step may be packed while the copy of the previous one is still queued
         self.meta_hosts = [torch.zeros(self.META_INTS, dtype=torch.int32, pin_memory=True) for _ in range(2)]
-        self.packers = [StepPacker(h, self.max_blocks_per_seq) for h in self.meta_hosts]
+        latent = any(ls.mixer == "latent" for ls in self.layers)
+        self.packers = [StepPacker(h, self.max_blocks_per_seq, kv_pages=latent) for h in self.meta_hosts]
         self._flip = 0
         self.meta_dev = torch.empty(self.META_INTS, dtype=torch.int32, device=dev)
         self.fmeta_hosts = [torch.empty(4 * max_num_seqs, dtype=torch.float32, pin_memory=True) for _ in range(2)]
@@ -843,6 +863,7 @@ class GpuModelRunner:
         pk = self.packers[self._flip]
         lay = pk.pack(b, bucketed, token_src=src)
         lay["_host"] = pk.meta_host
+        self._choose_expansion(lay)
         return lay
 
     def _feed_sampled_ids(self, lay) -> None:
@@ -1263,13 +1284,21 @@ class GpuModelRunner:
                                gain=gain, q_real=ls.q_rank, kv_real=ls.kv_rank)
         q = self._gemm(cq, t[L + "w_uq"]).view(T, kh.hq, kh.dim + kh.rot)
         bt = self._view(lay, "block_tables").view(Dp + P, self.max_blocks_per_seq)
+        out = torch.empty(T, kh.hq, kh.vdim, dtype=q.dtype, device=q.device)
+        kw = dict(scale=ls.scale, sinks=t.get(L + "sink"))
+        if P and lay["_xp"][i]:
+            self._latent_expanded(i, q[Dp:], pos[Dp:], bt[Dp:], lay, out[Dp:], freq, gain, kw)
+            if not Dp:
+                return out.view(T, kh.hq * kh.vdim)
+            q, pos, full, T, P = q[:Dp], pos[:Dp], out, Dp, 0
+            out = full[:Dp]
+        else:
+            full = out
         qa = torch.empty(T, kh.hq, kh.dk, dtype=q.dtype, device=q.device)
         lat = torch.empty(T, kh.hq, kh.dv, dtype=q.dtype, device=q.device)
-        out = torch.empty(T, kh.hq, kh.vdim, dtype=q.dtype, device=q.device)
         with self._prof("latent_query"):
             K.gemm_heads(q[..., :kh.dim], t[L + "w_uk_t"], qa[..., :kh.dv])
             K.latent_rotate(q, pos, freq, kh.rot, out=qa, gain=gain)
-        kw = dict(scale=ls.scale, sinks=t.get(L + "sink"))
         if Dp:
             with self._prof("attn_latent_decode"):
                 K.attn_latent(qa[:Dp], self.k_cache[i], kh.dv, bt[:Dp], self._view(lay, "seq_lens_d"), out=lat[:Dp],
@@ -1281,7 +1310,34 @@ class GpuModelRunner:
         with self._prof("latent_value"):
             K.gemm_heads(lat, t[L + "w_uv"], out)
         self.launches += 4 + (Dp > 0) + (P > 0)
-        return out.view(T, kh.hq * kh.vdim)
+        return full.view(-1, kh.hq * kh.vdim)
+
+    def _latent_expanded(self, i, q, pos, bt, lay, out, freq, gain, kw) -> None:
+        """Prompt portions long enough to pay for it: keys and values of all heads are computed from the cached latents of
+        their sequences, and the attention runs on those (a third of the multiply-adds of attention over the latents)."""
+        t, kh, L = self.w.t, self.w.heads[i], f"layers.{i}."
+        lens, pages = self._view(lay, "seq_lens_p"), self._view(lay, "kv_pages")
+        with self._prof("latent_expand"):
+            rows = K.latent_gather(self.k_cache[i], bt, lens, pages, lay["_kv_rows"])
+            K.latent_rotate(q, pos, freq, kh.rot, gain=gain)
+        kv = self._gemm(rows[:, :kh.dv], t[L + "w_ukv"])
+        with self._prof("attn_expanded"):
+            K.attn_expanded(q, kv, rows, kh.vdim, lens, self._view(lay, "q_start"), pages, lay["_max_q"], out=out, **kw)
+        self.launches += 3
+
+    def _choose_expansion(self, lay) -> None:
+        """Per latent layer, whether this step's prompt portions attend to expanded keys and values: their multiply-adds saved
+        (at about a third of the rate of the tensor-core kernel) against those of the expansion."""
+        pairs, rows = lay.get("_kv_pairs", 0), lay.get("_kv_rows", 0)
+        flags = []
+        for i, kh in enumerate(self.w.heads):
+            on = f"layers.{i}.w_ukv" in self.w.t and self.block_size == 16
+            if on:
+                on = pairs * 3 * max(2 * kh.dv - kh.dim - kh.vdim, 0) + pairs * 2 * (kh.dim + kh.rot + kh.vdim) > rows * kh.dv * (kh.dim + kh.vdim)
+            flags.append(bool(on))
+        lay["_xp"] = tuple(flags)
+        if not any(flags):
+            lay["_kv_rows"] = 0
 
     def _rotation(self, ls):
         """(device table of a layer's rotation frequencies, gain on cosine and sine)."""
@@ -1559,7 +1615,8 @@ class GpuModelRunner:
         if graphable:
             lay = self._pack(b, bucketed=True)
             lay["_pp"] = b.prefill_shares_prefix
-            key = (lay["_Dp"], lay["_P"], lay["_T"], lay["_max_q"], b.shared_prefix_len, b.prefill_shares_prefix)
+            key = (lay["_Dp"], lay["_P"], lay["_T"], lay["_max_q"], b.shared_prefix_len, b.prefill_shares_prefix, lay["_xp"],
+                   lay.get("_kv_rows", 0))
             g = self.graphs.get(key)
             self._graph_mode = True
             self._upload(lay)

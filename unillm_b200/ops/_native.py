@@ -109,6 +109,15 @@ class UbHeadGemmArgs(C.Structure):
     ]
 
 
+class UbExpandArgs(C.Structure):
+    _fields_ = [
+        ("cache", vp), ("lat", vp), ("q", vp), ("kv", vp), ("out", vp), ("sinks", vp), ("block_tables", vp), ("seq_lens", vp),
+        ("q_start", vp), ("page_start", vp), ("err", vp), ("q_stride", i64), ("o_stride", i64),
+        ("T", i32), ("H", i32), ("dim", i32), ("rot", i32), ("vdim", i32), ("kv_rank", i32), ("row", i32), ("rows", i32),
+        ("num_seqs", i32), ("max_q", i32), ("block_size", i32), ("num_blocks", i32), ("max_blocks_per_seq", i32), ("scale", f32),
+    ]
+
+
 class UbLatentArgs(C.Structure):
     _fields_ = [
         ("down", vp), ("q_latent", vp), ("cache", vp), ("q_norm_w", vp), ("kv_norm_w", vp), ("positions", vp),
@@ -223,7 +232,7 @@ class _CudaLibs:
     ARGS_AND_STREAM = {
         "serving": ("ub_gemm_tn", "ub_norm", "ub_rope_kv_append", "ub_attn_decode", "ub_attn_prefill", "ub_sample",
                     "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm", "ub_sublayer_in", "ub_wkv_mixer",
-                    "ub_gemm_heads", "ub_latent_rows", "ub_latent_rotate", "ub_attn_latent"),
+                    "ub_gemm_heads", "ub_latent_rows", "ub_latent_rotate", "ub_attn_latent", "ub_latent_gather", "ub_attn_expanded"),
         "more": ("ub_allreduce_oneshot", "ub_tp_argmax_merge"),
     }
 

@@ -541,6 +541,51 @@ def attn_latent(q: torch.Tensor, cache: torch.Tensor, v_dim: int, block_tables: 
     return out
 
 
+def expanded_supported(dim: int, rot: int, vdim: int) -> bool:
+    """Whether ``attn_expanded`` takes these (padded) head sizes."""
+    return dim % 16 == 0 and 16 <= dim <= 128 and vdim % 16 == 0 and 16 <= vdim <= 128 and rot % 8 == 0 and 8 <= rot <= 64
+
+
+def latent_gather(cache: torch.Tensor, block_tables: torch.Tensor, seq_lens: torch.Tensor, page_start: torch.Tensor,
+                  rows: int) -> torch.Tensor:
+    """Cache rows of sequences, one after the other: sequence i from row ``16 * page_start[i]`` on, zeros behind its end and
+    behind the last one -> [rows, row size] (``rows`` a multiple of 16)."""
+    _bf16c(cache, "cache")
+    if page_start.dtype != torch.int32 or page_start.numel() != seq_lens.numel() + 1 or cache.shape[1] != 1 or cache.shape[2] != 16:
+        raise ValueError("latent_gather: int32 page_start [n + 1], pages of 16 rows")
+    out = torch.empty(rows, cache.shape[3], dtype=cache.dtype, device=cache.device)
+    a = N.UbExpandArgs()
+    a.cache, a.lat, a.block_tables, a.seq_lens = cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(), seq_lens.data_ptr()
+    a.page_start, a.err, a.rows, a.row, a.num_seqs = page_start.data_ptr(), err_word(cache.device).data_ptr(), rows, cache.shape[3], seq_lens.numel()
+    a.block_size, a.num_blocks, a.max_blocks_per_seq = 16, cache.shape[0], block_tables.shape[1]
+    N.check(N.cuda_lib().ub_latent_gather(C.byref(a), _stream(cache)), "ub_latent_gather")
+    return out
+
+
+def attn_expanded(q: torch.Tensor, kv: torch.Tensor, lat: torch.Tensor, v_dim: int, seq_lens: torch.Tensor, q_start: torch.Tensor,
+                  page_start: torch.Tensor, max_q_len: int, *, scale: float, sinks: Optional[torch.Tensor] = None,
+                  out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Causal prompt attention over expanded latents on tcgen05: q [T, H, dim + rot] (rotated), kv [R, H * (dim + v_dim)], lat
+    [R, kv_rank + rot] as ``latent_gather`` gives them -> [T, H, v_dim]."""
+    for t, n in ((q, "q"), (kv, "kv"), (lat, "lat")):
+        _bf16c(t, n)
+    T, H, size = q.shape
+    dim = kv.shape[1] // H - v_dim
+    if kv.shape[0] != lat.shape[0] or not kv.is_contiguous() or not lat.is_contiguous() or q.stride(1) != size or q.stride(2) != 1:
+        raise ValueError("attn_expanded: contiguous kv and lat rows of the same number, contiguous heads")
+    if sinks is not None and (sinks.dtype != torch.float32 or sinks.numel() != H):
+        raise ValueError("sinks: fp32, one per query head")
+    if out is None:
+        out = torch.empty(T, H, v_dim, dtype=q.dtype, device=q.device)
+    a = N.UbExpandArgs()
+    a.q, a.kv, a.lat, a.out, a.sinks = q.data_ptr(), kv.data_ptr(), lat.data_ptr(), out.data_ptr(), _p(sinks)
+    a.seq_lens, a.q_start, a.page_start, a.err = seq_lens.data_ptr(), q_start.data_ptr(), page_start.data_ptr(), err_word(q.device).data_ptr()
+    a.q_stride, a.o_stride, a.T, a.H, a.dim, a.rot, a.vdim = q.stride(0), out.stride(0), T, H, dim, size - dim, v_dim
+    a.row, a.kv_rank, a.rows, a.num_seqs, a.max_q, a.scale = lat.shape[1], lat.shape[1] - a.rot, lat.shape[0], seq_lens.numel(), max_q_len, scale
+    N.check(N.cuda_lib().ub_attn_expanded(C.byref(a), _stream(q)), "ub_attn_expanded")
+    return out
+
+
 # ---------------------------------------------------------------------------------------------
 # RoPE + KV append
 # ---------------------------------------------------------------------------------------------
