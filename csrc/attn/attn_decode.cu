@@ -270,29 +270,46 @@ __global__ void __launch_bounds__(128) attn_decode_kernel(const UbAttnArgs a, co
 }
 
 // Merge the split partials: out = sum_i O_i * exp(lse_i - lse_max) / sum_i exp(lse_i - lse_max).
-// A softmax sink (one logit per head without a value) joins the denominator here, once.
-__global__ void attn_split_merge_kernel(const float* scratch, __nv_bfloat16* out, float* lse_out, int Hq, int D,
-                                        int splits, long long o_stride, const float* sinks) {
-  const int seq = blockIdx.x, h = blockIdx.y;
+// A softmax sink (one logit per head without a value) joins the denominator here, once.  The first warp turns the
+// log-sum-exps into weights, then every thread adds up one column.
+constexpr int MERGE_SPLITS = 64;
+__global__ void __launch_bounds__(128) attn_split_merge_kernel(const float* scratch, __nv_bfloat16* out, float* lse_out, int Hq, int D,
+                                                               int splits, long long o_stride, const float* sinks) {
+  __shared__ float w_s[MERGE_SPLITS];
+  const int seq = blockIdx.x, h = blockIdx.y, lane = threadIdx.x & 31;
   const float* sp = scratch + ((long long)seq * Hq + h) * splits * (D + 2);
-  float mx = sinks != nullptr ? sinks[h] : -CUDART_INF_F;
-  for (int i = 0; i < splits; ++i) mx = fmaxf(mx, sp[i * (D + 2) + D]);
-  float den = sinks != nullptr ? expf(sinks[h] - mx) : 0.f;
-  for (int i = 0; i < splits; ++i) {
-    const float ls = sp[i * (D + 2) + D];
-    den += (ls == -CUDART_INF_F) ? 0.f : expf(ls - mx);
-  }
-  for (int d = threadIdx.x; d < D; d += blockDim.x) {
-    float o = 0.f;
-    for (int i = 0; i < splits; ++i) {
-      const float ls = sp[i * (D + 2) + D];
-      const float w = (ls == -CUDART_INF_F) ? 0.f : expf(ls - mx);
-      o += sp[i * (D + 2) + d] * w;
+  if (threadIdx.x < 32) {
+    const float sink = sinks != nullptr ? sinks[h] : -CUDART_INF_F;
+    float l[MERGE_SPLITS / 32], mx = sink;
+#pragma unroll
+    for (int k = 0; k < MERGE_SPLITS / 32; ++k) {
+      const int i = lane + 32 * k;
+      l[k] = i < splits ? sp[(long long)i * (D + 2) + D] : -CUDART_INF_F;
+      mx = fmaxf(mx, l[k]);
     }
-    out[(long long)seq * o_stride + (long long)h * D + d] = __float2bfloat16(den > 0.f ? o / den : 0.f);
+    mx = warp_max(mx);
+    float den = 0.f;
+#pragma unroll
+    for (int k = 0; k < MERGE_SPLITS / 32; ++k) {
+      l[k] = l[k] == -CUDART_INF_F ? 0.f : expf(l[k] - mx);
+      den += l[k];
+    }
+    den = warp_sum(den) + (sink == -CUDART_INF_F ? 0.f : expf(sink - mx));
+    const float inv = den > 0.f ? 1.f / den : 0.f;
+#pragma unroll
+    for (int k = 0; k < MERGE_SPLITS / 32; ++k) w_s[lane + 32 * k] = l[k] * inv;
+    if (lane == 0 && blockIdx.z == 0 && lse_out != nullptr) lse_out[(long long)seq * Hq + h] = den > 0.f ? mx + logf(den) : -CUDART_INF_F;
   }
-  if (threadIdx.x == 0 && lse_out != nullptr)
-    lse_out[(long long)seq * Hq + h] = den > 0.f ? mx + logf(den) : -CUDART_INF_F;
+  __syncthreads();
+  const int d = blockIdx.z * blockDim.x + threadIdx.x;
+  if (d >= D) return;
+  float o = 0.f;
+#pragma unroll 8
+  for (int i = 0; i < splits; ++i) {
+    const float w = w_s[i];
+    o += w != 0.f ? sp[(long long)i * (D + 2) + d] * w : 0.f;        // a range without keys has left nothing
+  }
+  out[(long long)seq * o_stride + (long long)h * D + d] = __float2bfloat16(o);
 }
 
 // Merge two independently computed attention partials over disjoint key sets.
@@ -393,11 +410,7 @@ static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return -(int)e;
   if (a.splits > 1) {
-    dim3 g2(a.num_seqs, a.Hq);
-    attn_split_merge_kernel<<<g2, D <= 128 ? D : 128, 0, st>>>(a.scratch, reinterpret_cast<__nv_bfloat16*>(a.out),
-                                                               a.lse, a.Hq, D, a.splits, a.o_stride, nullptr);
-    e = cudaGetLastError();
-    if (e != cudaSuccess) return -(int)e;
+    return ub_attn_split_merge(&a, st);
   }
   return 0;
 }
@@ -406,7 +419,8 @@ static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
 
 extern "C" int ub_attn_split_merge(const UbAttnArgs* a, void* stream) {
   const int dv = a->Dv > 0 ? a->Dv : a->D;
-  ub::attn_split_merge_kernel<<<dim3(a->num_seqs, a->Hq), dv <= 128 ? dv : 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
+  if (a->splits > ub::MERGE_SPLITS) return -3;
+  ub::attn_split_merge_kernel<<<dim3(a->num_seqs, a->Hq, (dv + 127) / 128), 128, 0, reinterpret_cast<cudaStream_t>(stream)>>>(
       a->scratch, reinterpret_cast<__nv_bfloat16*>(a->out), a->lse, a->Hq, dv, a->splits, a->o_stride, a->sinks);
   const cudaError_t e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;

@@ -41,8 +41,10 @@ __device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], 
 constexpr int S_PITCH = KT + 4;            // floats
 constexpr int P_PITCH = KT * 2 + 16;       // bytes
 
+constexpr int BT_MAX = 512;                // block-table entries held in shared memory
+
 struct Layout {
-  int pitch, q, kv, s, p, row, total;      // byte offsets
+  int pitch, q, kv, s, p, row, bt, total;  // byte offsets
   __host__ __device__ Layout(int D, int mt) {
     pitch = (D + 15) / 16 * 32 + 16;
     q = 0;
@@ -50,7 +52,8 @@ struct Layout {
     s = kv + 2 * KT * pitch;
     p = s + 2 * 16 * mt * S_PITCH * 4;
     row = p + 16 * mt * P_PITCH;
-    total = row + 16 * mt * 3 * 4;         // alpha, max, sum per row
+    bt = row + 16 * mt * 3 * 4;            // behind alpha, max, sum per row
+    total = bt + BT_MAX * 4;
   }
 };
 
@@ -89,23 +92,30 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
     const int tok = ok ? row / a.Hq : 0, h = ok ? row % a.Hq : 0;
     cp_async16(q_u + r * L.pitch + c * 16, qg + (ok ? (long long)(qs + tok) * a.q_stride + (long long)h * D + c * 8 : 0), ok);
   }
+  int* bt_sm = reinterpret_cast<int*>(sm + L.bt);
+  const int page0 = kv_lo / a.block_size, pages = n_tiles > 0 ? (kv_hi - 1) / a.block_size - page0 + 1 : 0;
+  for (int i = threadIdx.x; i < min(pages, BT_MAX); i += THREADS) bt_sm[i] = page0 + i < a.max_blocks_per_seq ? bt[page0 + i] : -1;
+  __syncthreads();
+  const int bs_shift = 31 - __clz(a.block_size);           // a power of two (host check)
   auto issue = [&](int t) {
     if (t < n_tiles) {
       const uint32_t st = kv_u + (t & 1) * KT * L.pitch;
       const int base = kv_lo + t * KT;
-      // a warp fetches whole rows: one block-table lookup per row, 16-byte chunks at consecutive addresses
+      // a warp fetches whole rows: one block-table entry per row, 16-byte chunks at consecutive addresses
+#pragma unroll 4
       for (int r = warp; r < KT; r += THREADS / 32) {
         const int pos = base + r;
         long long src = -1;
         if (pos < kv_hi) {
-          const int bi = pos / a.block_size;
-          const int blk = bi < a.max_blocks_per_seq ? bt[bi] : -1;
+          const int bi = pos >> bs_shift;
+          const int blk = bi - page0 < BT_MAX ? bt_sm[bi - page0] : (bi < a.max_blocks_per_seq ? bt[bi] : -1);
           if (blk < 0 || blk >= a.num_blocks) set_err(a.err, ERR_BOUNDS, seq);
-          else src = ((long long)blk * a.block_size + pos % a.block_size) * D;
+          else src = (((long long)blk << bs_shift) + (pos & (a.block_size - 1))) * D;
         }
+        const __nv_bfloat16* g = cache + (src >= 0 ? src : 0);
         for (int c = lane; c < nck; c += 32) {
           const bool ok = src >= 0 && c < nch;
-          cp_async16(st + r * L.pitch + c * 16, cache + (ok ? src + c * 8 : 0), ok);
+          cp_async16(st + r * L.pitch + c * 16, ok ? g + c * 8 : cache, ok);
         }
       }
     }
@@ -131,33 +141,41 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
     issue(t + 1);
     const uint32_t kb = kv_u + (t & 1) * KT * L.pitch;
     {
-      float s[MT][2][4];
+      float s[MT][2][4], s2[MT][2][4];                     // even and odd steps: two chains of dependent MMAs
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
-        for (int j = 0; j < 2; ++j) s[mt][j][0] = s[mt][j][1] = s[mt][j][2] = s[mt][j][3] = 0.f;
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) s[mt][j][e] = s2[mt][j][e] = 0.f;
       const int mi = lane >> 3;
       const uint32_t baddr = kb + (tg * 16 + (mi >> 1) * 8 + (lane & 7)) * L.pitch + (mi & 1) * 16;
       const uint32_t aaddr = q_u + ((lane & 7) + ((lane >> 3) & 1) * 8) * L.pitch + (lane >> 4) * 16;
-#pragma unroll 4
-      for (int ks = ks0; ks < ks1; ++ks) {
+      auto step = [&](int ks, float (&acc)[MT][2][4]) {
         uint32_t b0, b1, b2, b3;
         ldsm_x4(baddr + ks * 32, b0, b1, b2, b3);
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt) {
           uint32_t af[4];
           ldsm_x4(aaddr + mt * 16 * L.pitch + ks * 32, af[0], af[1], af[2], af[3]);
-          mma_bf16(s[mt][0], af, b0, b1);
-          mma_bf16(s[mt][1], af, b2, b3);
+          mma_bf16(acc[mt][0], af, b0, b1);
+          mma_bf16(acc[mt][1], af, b2, b3);
         }
+      };
+      int ks = ks0;
+#pragma unroll 3
+      for (; ks + 1 < ks1; ks += 2) {
+        step(ks, s);
+        step(ks + 1, s2);
       }
+      if (ks < ks1) step(ks, s);
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           float* d = s_sm + (kh * ROWS + mt * 16 + (lane >> 2)) * S_PITCH + tg * 16 + j * 8 + (lane & 3) * 2;
-          *reinterpret_cast<float2*>(d) = make_float2(s[mt][j][0], s[mt][j][1]);
-          *reinterpret_cast<float2*>(d + 8 * S_PITCH) = make_float2(s[mt][j][2], s[mt][j][3]);
+          *reinterpret_cast<float2*>(d) = make_float2(s[mt][j][0] + s2[mt][j][0], s[mt][j][1] + s2[mt][j][1]);
+          *reinterpret_cast<float2*>(d + 8 * S_PITCH) = make_float2(s[mt][j][2] + s2[mt][j][2], s[mt][j][3] + s2[mt][j][3]);
         }
     }
     __syncthreads();
@@ -297,6 +315,7 @@ extern "C" int ub_attn_latent(const UbAttnArgs* a, void* stream) {
   if (a->D % 8 != 0 || a->Dv % 8 != 0 || a->Dv <= 0 || a->Dv >= a->D || a->Dv > 512 || a->D > 640 || a->Hq <= 0) return -2;
   if (a->q_stride % 8 != 0 || a->o_stride % 2 != 0 || a->splits < 1 || a->num_seqs > 65535) return -3;
   if (a->splits > 1 && (a->q_start != nullptr || a->scratch == nullptr)) return -3;
+  if (a->block_size <= 0 || (a->block_size & (a->block_size - 1))) return -5;
   if (a->window > 0 || a->alibi_slopes != nullptr || a->merge_o != nullptr || a->kv_start > 0) return -7;
   if ((reinterpret_cast<uintptr_t>(a->q) | reinterpret_cast<uintptr_t>(a->k_cache) | reinterpret_cast<uintptr_t>(a->out)) & 15) return -4;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);

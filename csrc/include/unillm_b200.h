@@ -158,9 +158,9 @@ typedef struct UbSublayerInArgs {
   const void* wy;           /* weight of the norm on y */
   float* x_out;             /* x + norm(y); another buffer than x; unused without y */
   const void* wn;           /* weight of the norm on the result */
-  const float* conv;        /* [taps, Hp] or NULL */
+  const void* conv;         /* [taps, Hp], of y's element type, or NULL */
   float* conv_state;        /* [state_rows, taps - 1, Hp] last values of the norm */
-  const float* mu;          /* [n_mix, Hp] or NULL */
+  const void* mu;           /* [n_mix, Hp], of y's element type, or NULL */
   float* shift_state;       /* [state_rows, Hp] last value after the convolution */
   void* out;                /* [rows, Hp], or n_mix of them out_mix_stride elements apart */
   const int* state_in;      /* per sequence: state row to read, negative = start of the sequence */
@@ -168,7 +168,7 @@ typedef struct UbSublayerInArgs {
   const int* q_start;       /* [num_seqs + 1] rows of the sequences from row0 on; NULL: one row each */
   int* err;
   long long row0, out_mix_stride;
-  int H, Hp, taps, n_mix, num_seqs, max_q, state_rows, tile /* tokens per CTA */, f32;
+  int H, Hp, taps, n_mix /* 0 or 5 */, num_seqs, max_q, state_rows, tile /* tokens per CTA */, f32;
   float eps, w_off;
 } UbSublayerInArgs;
 int ub_sublayer_in(const UbSublayerInArgs* args, void* stream);

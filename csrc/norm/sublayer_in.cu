@@ -10,7 +10,8 @@
 // from the sequence's state rows (the last taps - 1 values of n, the last h), and the portion leaves its own behind in
 // OTHER rows, so every CTA of the launch may read the old ones whenever it runs.
 //
-// A CTA takes `tile` consecutive tokens of one sequence and recomputes the few rows of n in front of them (x and y are read
+// One token per sequence (decoding) has a kernel of its own: what the state contributes does not depend on the norms, so all
+// loads are under way before the first sum.  Longer portions: a CTA takes `tile` consecutive tokens of one sequence and recomputes the few rows of n in front of them (x and y are read
 // again, x' goes to a buffer of its own), so tiles are independent.  The last taps - 1 rows of n stay in shared memory; a
 // thread touches only its own columns there.
 #include "../common/elem.cuh"
@@ -19,8 +20,34 @@
 namespace ub {
 namespace subin {
 
+constexpr int MIXES = 5;      // token-shift mixes of a recurrent mixer
+
+// eight weights as they lie in memory, widened when they are used
+template <typename T>
+struct Raw8;
+template <>
+struct Raw8<__nv_bfloat16> {
+  uint4 v;
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+    const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { f[2 * e] = bf16_lo(u[e]); f[2 * e + 1] = bf16_hi(u[e]); }
+  }
+};
+template <>
+struct Raw8<float> {
+  float v[8];
+  __device__ __forceinline__ void load(const float* p) { load8(p, v); }
+  __device__ __forceinline__ void get(float (&f)[8]) const {
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = v[e];
+  }
+};
+
 // one barrier per sum: the two halves of `red` alternate
-__device__ __forceinline__ float block_sum(float v, float (*red)[8], int& flip) {
+template <int NW>
+__device__ __forceinline__ float block_sum(float v, float (*red)[NW], int& flip) {
   v = warp_sum(v);
   const int nw = blockDim.x >> 5;
   if ((threadIdx.x & 31) == 0) red[flip][threadIdx.x >> 5] = v;
@@ -52,7 +79,8 @@ __global__ void __launch_bounds__(256) sublayer_in_kernel(const UbSublayerInArgs
   const T* y = reinterpret_cast<const T*>(a.y);
   const long long row0 = a.row0 + qs;
   int flip = 0;
-  auto slot = [&](int idx) { return ((idx % m) + m) % m; };
+  const int wrap = m > 0 ? m : 1;
+  auto slot = [&](int idx) { return (idx + wrap * ((m + wrap - 1) / wrap)) % wrap; };     // idx >= -m
   auto hrow = [&](int s, int half, int ch) { return reinterpret_cast<float4*>(hist + ((s * 2 + half) * nch + ch) * 4); };
 
   if (s0 == 0 && m > 0) {
@@ -139,12 +167,12 @@ __global__ void __launch_bounds__(256) sublayer_in_kernel(const UbSublayerInArgs
           const int s = slot(t - m + j);
           const float4 lo = *hrow(s, 0, ch), hi = *hrow(s, 1, ch);
           float k[8];
-          load8(a.conv + (long long)j * a.Hp + ch * 8, k);
+          load8(reinterpret_cast<const T*>(a.conv) + (long long)j * a.Hp + ch * 8, k);
           h[0] = fmaf(k[0], lo.x, h[0]); h[1] = fmaf(k[1], lo.y, h[1]); h[2] = fmaf(k[2], lo.z, h[2]); h[3] = fmaf(k[3], lo.w, h[3]);
           h[4] = fmaf(k[4], hi.x, h[4]); h[5] = fmaf(k[5], hi.y, h[5]); h[6] = fmaf(k[6], hi.z, h[6]); h[7] = fmaf(k[7], hi.w, h[7]);
         }
         float k[8];
-        load8(a.conv + (long long)m * a.Hp + ch * 8, k);
+        load8(reinterpret_cast<const T*>(a.conv) + (long long)m * a.Hp + ch * 8, k);
 #pragma unroll
         for (int e = 0; e < 8; ++e) h[e] = fmaf(k[e], n[c][e], h[e]);
       }
@@ -158,7 +186,7 @@ __global__ void __launch_bounds__(256) sublayer_in_kernel(const UbSublayerInArgs
         if (!mix) store8(out, h);
         for (int i = 0; i < a.n_mix; ++i) {
           float mu[8], o[8];
-          load8(a.mu + (long long)i * a.Hp + ch * 8, mu);
+          load8(reinterpret_cast<const T*>(a.mu) + (long long)i * a.Hp + ch * 8, mu);
 #pragma unroll
           for (int e = 0; e < 8; ++e) o[e] = h[e] + (prev[c][e] - h[e]) * mu[e];
           store8(out + (long long)i * a.out_mix_stride, o);
@@ -181,8 +209,263 @@ __global__ void __launch_bounds__(256) sublayer_in_kernel(const UbSublayerInArgs
   }
 }
 
+// Portions at up to 4096 columns and four taps: a thread owns one chunk, and the weights, the last rows of n and the
+// prefetched next token all stay in registers.
+template <typename T, int TAPS, bool MIX>
+__global__ void __launch_bounds__(512) sublayer_rows_kernel(const UbSublayerInArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  constexpr int M = TAPS - 1;
+  __shared__ float red[2][16];
+  const int seq = blockIdx.y, ch = threadIdx.x;
+  const int qs = a.q_start[seq], q_len = a.q_start[seq + 1] - qs;
+  const int t0 = blockIdx.x * a.tile, t1 = min(t0 + a.tile, q_len);
+  if (t0 >= t1) return;
+  int si = a.state_in != nullptr ? a.state_in[seq] : -1, so = a.state_out != nullptr ? a.state_out[seq] : -1;
+  if (si >= a.state_rows || so >= a.state_rows) {
+    if (threadIdx.x == 0) set_err(a.err, ERR_BOUNDS, seq);
+    si = so = -1;
+  }
+  const bool on = ch < a.Hp / 8;
+  const int s0 = max(0, t0 - M - (MIX ? 1 : 0));
+  const T* y = reinterpret_cast<const T*>(a.y);
+  const long long base = (a.row0 + qs) * a.Hp + ch * 8;
+  Raw8<T> wy8, wn8, k8[TAPS], mu8[MIX ? MIXES : 1];
+  float hist[M > 0 ? M : 1][8], prev[8], x[8], yv[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    prev[e] = x[e] = yv[e] = 0.f;
+#pragma unroll
+    for (int r = 0; r < M; ++r) hist[r][e] = 0.f;
+  }
+  auto fetch = [&](int t) {
+    load8(a.x + base + (long long)t * a.Hp, x);
+    if (y != nullptr) load8(y + base + (long long)t * a.Hp, yv);
+  };
+  if (on) {
+    fetch(s0);
+    if (y != nullptr) wy8.load(reinterpret_cast<const T*>(a.wy) + ch * 8);
+    wn8.load(reinterpret_cast<const T*>(a.wn) + ch * 8);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) k8[j].load(reinterpret_cast<const T*>(a.conv) + (long long)j * a.Hp + ch * 8);
+    if (MIX) {
+#pragma unroll
+      for (int i = 0; i < MIXES; ++i) mu8[i].load(reinterpret_cast<const T*>(a.mu) + (long long)i * a.Hp + ch * 8);
+    }
+    if (s0 == 0 && si >= 0) {
+#pragma unroll
+      for (int r = 0; r < M; ++r) load8(a.conv_state + ((long long)si * M + r) * a.Hp + ch * 8, hist[r]);
+      if (MIX) load8(a.shift_state + (long long)si * a.Hp + ch * 8, prev);
+    }
+  }
+  int flip = 0;
+  for (int t = s0; t < t1; ++t) {
+    if (y != nullptr) {
+      float sq = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sq += yv[e] * yv[e];
+      const float r = 1.f / sqrtf(block_sum(sq, red, flip) / a.H + a.eps);
+      if (on) {
+        float w[8];
+        wy8.get(w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[e] += yv[e] * r * (a.w_off + w[e]);
+        if (t >= t0) store8(a.x_out + base + (long long)t * a.Hp, x);
+      }
+    }
+    float n[8], sq = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      n[e] = x[e];
+      sq += n[e] * n[e];
+    }
+    if (on && t + 1 < t1) fetch(t + 1);
+    const float r = 1.f / sqrtf(block_sum(sq, red, flip) / a.H + a.eps);
+    if (!on) continue;
+    float w[8], h[8];
+    wn8.get(w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      n[e] *= r * (a.w_off + w[e]);
+      h[e] = n[e];
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) {
+      float k[8];
+      k8[j].get(k);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) h[e] = fmaf(k[e], j < M ? hist[j < M ? j : 0][e] : n[e], h[e]);
+    }
+#pragma unroll
+    for (int r2 = 0; r2 < M; ++r2)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) hist[r2][e] = r2 + 1 < M ? hist[r2 + 1 < M ? r2 + 1 : 0][e] : n[e];
+    if (t >= t0) {
+      T* out = reinterpret_cast<T*>(a.out) + base + (long long)t * a.Hp;
+      if (!MIX) {
+        store8(out, h);
+      } else {
+#pragma unroll
+        for (int i = 0; i < MIXES; ++i) {
+          float mu[8], o[8];
+          mu8[i].get(mu);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) o[e] = h[e] + (prev[e] - h[e]) * mu[e];
+          store8(out + (long long)i * a.out_mix_stride, o);
+        }
+      }
+    }
+    if (MIX) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) prev[e] = h[e];
+    }
+    if (t == q_len - 1 && so >= 0) {
+#pragma unroll
+      for (int r2 = 0; r2 < M; ++r2) store8(a.conv_state + ((long long)so * M + r2) * a.Hp + ch * 8, hist[r2]);
+      if (MIX) store8(a.shift_state + (long long)so * a.Hp + ch * 8, h);
+    }
+  }
+}
+
+template <typename T, int TAPS>
+static cudaError_t launch_rows(const UbSublayerInArgs& a, cudaStream_t st) {
+  const dim3 grid((a.max_q + a.tile - 1) / a.tile, a.num_seqs), block((a.Hp / 8 + 31) / 32 * 32);
+  return a.n_mix > 0 ? launch_pdl(sublayer_rows_kernel<T, TAPS, true>, grid, block, (size_t)0, st, a)
+                     : launch_pdl(sublayer_rows_kernel<T, TAPS, false>, grid, block, (size_t)0, st, a);
+}
+
+// One token of every sequence.
+template <typename T, int CH>
+__global__ void __launch_bounds__(512) sublayer_step_kernel(const UbSublayerInArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[2][16];
+  const int seq = blockIdx.x, nch = a.Hp / 8, m = a.taps > 0 ? a.taps - 1 : 0;
+  const long long row = a.row0 + seq;
+  const bool mix = a.n_mix > 0;
+  const T* y = reinterpret_cast<const T*>(a.y);
+  float x[CH][8], yv[CH][8], old[CH][8], prev[CH][8];
+  float sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int ch = threadIdx.x + c * blockDim.x;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[c][e] = yv[c][e] = old[c][e] = prev[c][e] = 0.f;
+    if (ch >= nch) continue;
+    load8(a.x + row * a.Hp + ch * 8, x[c]);
+    if (y != nullptr) load8(y + row * a.Hp + ch * 8, yv[c]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq += yv[c][e] * yv[c][e];
+  }
+  int si = a.state_in != nullptr ? a.state_in[seq] : -1, so = a.state_out != nullptr ? a.state_out[seq] : -1;
+  if (si >= a.state_rows || so >= a.state_rows) {
+    if (threadIdx.x == 0) set_err(a.err, ERR_BOUNDS, seq);
+    si = so = -1;
+  }
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int ch = threadIdx.x + c * blockDim.x;
+    if (ch >= nch) continue;
+    if (mix && si >= 0) load8(a.shift_state + (long long)si * a.Hp + ch * 8, prev[c]);
+#pragma unroll 3
+    for (int j = 0; j < m; ++j) {                     // the taps in front of the token; its predecessors move up one row
+      float v[8], k[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = 0.f;
+      if (si >= 0) load8(a.conv_state + ((long long)si * m + j) * a.Hp + ch * 8, v);
+      load8(reinterpret_cast<const T*>(a.conv) + (long long)j * a.Hp + ch * 8, k);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) old[c][e] = fmaf(k[e], v[e], old[c][e]);
+      if (so >= 0 && j > 0) store8(a.conv_state + ((long long)so * m + j - 1) * a.Hp + ch * 8, v);
+    }
+  }
+  Raw8<T> wy8[CH], wn8[CH], k8[CH], mu8[CH][MIXES];
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int ch = threadIdx.x + c * blockDim.x;
+    if (ch >= nch) continue;
+    if (y != nullptr) wy8[c].load(reinterpret_cast<const T*>(a.wy) + ch * 8);
+    wn8[c].load(reinterpret_cast<const T*>(a.wn) + ch * 8);
+    if (a.taps > 0) k8[c].load(reinterpret_cast<const T*>(a.conv) + (long long)m * a.Hp + ch * 8);
+    if (mix) {
+#pragma unroll
+      for (int i = 0; i < MIXES; ++i) mu8[c][i].load(reinterpret_cast<const T*>(a.mu) + (long long)i * a.Hp + ch * 8);
+    }
+  }
+  int flip = 0;
+  if (y != nullptr) {
+    const float r = 1.f / sqrtf(block_sum(sq, red, flip) / a.H + a.eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int ch = threadIdx.x + c * blockDim.x;
+      if (ch >= nch) continue;
+      float w[8];
+      wy8[c].get(w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[c][e] += yv[c][e] * r * (a.w_off + w[e]);
+      store8(a.x_out + row * a.Hp + ch * 8, x[c]);
+    }
+  }
+  sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq += x[c][e] * x[c][e];
+  const float r = 1.f / sqrtf(block_sum(sq, red, flip) / a.H + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int ch = threadIdx.x + c * blockDim.x;
+    if (ch >= nch) continue;
+    float w[8], k[8], n[8], h[8];
+    wn8[c].get(w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) k[e] = 0.f;
+    if (a.taps > 0) k8[c].get(k);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      n[e] = x[c][e] * r * (a.w_off + w[e]);
+      h[e] = fmaf(k[e], n[e], n[e] + old[c][e]);
+    }
+    T* out = reinterpret_cast<T*>(a.out) + row * a.Hp + ch * 8;
+    if (!mix) {
+      store8(out, h);
+    } else {
+#pragma unroll
+      for (int i = 0; i < MIXES; ++i) {
+        float mu[8], o[8];
+        mu8[c][i].get(mu);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = h[e] + (prev[c][e] - h[e]) * mu[e];
+        store8(out + (long long)i * a.out_mix_stride, o);
+      }
+    }
+    if (so >= 0) {
+      if (m > 0) store8(a.conv_state + ((long long)so * m + m - 1) * a.Hp + ch * 8, n);
+      if (mix) store8(a.shift_state + (long long)so * a.Hp + ch * 8, h);
+    }
+  }
+}
+
+template <typename T>
+static cudaError_t launch_step(const UbSublayerInArgs& a, cudaStream_t st) {
+  const int nch = a.Hp / 8;
+  const int threads = nch >= 512 ? 512 : (nch + 31) / 32 * 32;
+  const int ch = (nch + threads - 1) / threads;
+  const dim3 grid(a.num_seqs), block(threads);
+  if (ch <= 1) return launch_pdl(sublayer_step_kernel<T, 1>, grid, block, (size_t)0, st, a);
+  if (ch <= 2) return launch_pdl(sublayer_step_kernel<T, 2>, grid, block, (size_t)0, st, a);
+  return launch_pdl(sublayer_step_kernel<T, 4>, grid, block, (size_t)0, st, a);
+}
+
 template <typename T>
 static cudaError_t launch(const UbSublayerInArgs& a, cudaStream_t st) {
+  if (a.q_start == nullptr) return launch_step<T>(a, st);
+  if (a.Hp <= 4096 && a.taps >= 1 && a.taps <= 4) {
+    if (a.taps == 1) return launch_rows<T, 1>(a, st);
+    if (a.taps == 2) return launch_rows<T, 2>(a, st);
+    if (a.taps == 3) return launch_rows<T, 3>(a, st);
+    return launch_rows<T, 4>(a, st);
+  }
   const int nch = a.Hp / 8;
   const int threads = nch >= 256 ? 256 : (nch + 31) / 32 * 32;
   const int ch = (nch + threads - 1) / threads;
@@ -212,7 +495,7 @@ extern "C" int ub_sublayer_in(const UbSublayerInArgs* a, void* stream) {
   if (a->y != nullptr && (a->wy == nullptr || a->x_out == nullptr || a->x_out == a->x)) return -4;
   if (a->taps > 0 && a->conv == nullptr) return -5;
   if (a->taps > 1 && (a->conv_state == nullptr || (long long)(a->taps - 1) * a->Hp * 4 > 220 * 1024)) return -5;
-  if (a->n_mix > 0 && (a->mu == nullptr || a->shift_state == nullptr)) return -6;
+  if (a->n_mix != 0 && (a->n_mix != subin::MIXES || a->mu == nullptr || a->shift_state == nullptr)) return -6;
   cudaStream_t st = reinterpret_cast<cudaStream_t>(stream);
   cudaError_t e = a->f32 ? subin::launch<float>(*a, st) : subin::launch<__nv_bfloat16>(*a, st);
   if (e == cudaSuccess) e = cudaGetLastError();

@@ -7,8 +7,9 @@
 // State, decays and everything between the loads and `out` are fp32; r, k, v, g and out have the element type of the matrix
 // products.  A portion reads its sequence's state row (none: zero) and leaves the new state in another row.
 //
-// Four columns and D / RG rows of S live in the registers of a thread; RG = 8 neighbouring lanes hold the row groups of the
-// same columns, so a token's output needs four shuffles.  Tokens come in tiles of 16 through shared memory; the bonus term
+// Four columns and D / RG rows of S live in the registers of a thread, as pairs of neighbouring rows: the row factors r, k and
+// d come as pairs from shared memory and two multiply-adds are one instruction.  RG = 8 neighbouring lanes hold the row
+// groups of the same columns, so a token's output needs four shuffles.  Tokens come in tiles of 16 through shared memory; the bonus term
 // is one scalar per token, sum_i r u k, times v.
 //
 // Long prompts (wkv_chunk / wkv_carry / wkv_out): chunks of CL tokens run in parallel from a zero state and leave their
@@ -72,7 +73,7 @@ __device__ __forceinline__ void bonus_terms(const UbWkvArgs& a, Tile<DP>& s, int
 template <int DP>
 struct State {
   static constexpr int RPT = DP / RG;            // rows per thread
-  float S[RPT / 4][4][4];                        // [group of 4 rows][row][column]
+  uint64_t S[RPT / 2][4];                        // [pair of rows][column]
   int rg, cg;
 
   __device__ __forceinline__ State() {
@@ -80,45 +81,55 @@ struct State {
     rg = lane & 7;
     cg = (threadIdx.x >> 5) * 4 + (lane >> 3);
   }
-  __device__ __forceinline__ int row(int q, int e) const { return 4 * (rg + RG * q) + e; }
+  // first row of pair p: groups of four rows, RG groups apart
+  __device__ __forceinline__ int row(int p) const { return 4 * (rg + RG * (p >> 1)) + 2 * (p & 1); }
 
   __device__ __forceinline__ void load(const float* st, int D) {
 #pragma unroll
-    for (int q = 0; q < RPT / 4; ++q)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (st != nullptr && row(q, e) < D && cg * 4 < D) f = *reinterpret_cast<const float4*>(st + (long long)row(q, e) * D + cg * 4);
-        S[q][e][0] = f.x; S[q][e][1] = f.y; S[q][e][2] = f.z; S[q][e][3] = f.w;
+    for (int p = 0; p < RPT / 2; ++p) {
+      float4 f = make_float4(0.f, 0.f, 0.f, 0.f), g = f;
+      if (st != nullptr && row(p) < D && cg * 4 < D) {
+        f = *reinterpret_cast<const float4*>(st + (long long)row(p) * D + cg * 4);
+        g = *reinterpret_cast<const float4*>(st + (long long)(row(p) + 1) * D + cg * 4);
       }
+      S[p][0] = pack_f32x2(f.x, g.x); S[p][1] = pack_f32x2(f.y, g.y); S[p][2] = pack_f32x2(f.z, g.z); S[p][3] = pack_f32x2(f.w, g.w);
+    }
   }
   __device__ __forceinline__ void store(float* st, int D) const {
 #pragma unroll
-    for (int q = 0; q < RPT / 4; ++q)
-#pragma unroll
-      for (int e = 0; e < 4; ++e)
-        if (row(q, e) < D && cg * 4 < D)
-          *reinterpret_cast<float4*>(st + (long long)row(q, e) * D + cg * 4) = make_float4(S[q][e][0], S[q][e][1], S[q][e][2], S[q][e][3]);
+    for (int p = 0; p < RPT / 2; ++p) {
+      if (row(p) >= D || cg * 4 >= D) continue;
+      float4 f, g;
+      unpack_f32x2(S[p][0], f.x, g.x); unpack_f32x2(S[p][1], f.y, g.y); unpack_f32x2(S[p][2], f.z, g.z); unpack_f32x2(S[p][3], f.w, g.w);
+      *reinterpret_cast<float4*>(st + (long long)row(p) * D + cg * 4) = f;
+      *reinterpret_cast<float4*>(st + (long long)(row(p) + 1) * D + cg * 4) = g;
+    }
   }
   __device__ __forceinline__ void walk(Tile<DP>& s, int n) {
     for (int t = 0; t < n; ++t) {
-      const float4 v = *reinterpret_cast<const float4*>(&s.v[t][cg * 4]);
-      float y[4] = {0.f, 0.f, 0.f, 0.f};
+      const float4 v4 = *reinterpret_cast<const float4*>(&s.v[t][cg * 4]);
+      const uint64_t v[4] = {pack_f32x2(v4.x, v4.x), pack_f32x2(v4.y, v4.y), pack_f32x2(v4.z, v4.z), pack_f32x2(v4.w, v4.w)};
+      uint64_t y2[4] = {0ull, 0ull, 0ull, 0ull};
 #pragma unroll
       for (int q = 0; q < RPT / 4; ++q) {
         const int i = 4 * (rg + RG * q);
-        const float4 r4 = *reinterpret_cast<const float4*>(&s.r[t][i]);
-        const float4 k4 = *reinterpret_cast<const float4*>(&s.k[t][i]);
-        const float4 d4 = *reinterpret_cast<const float4*>(&s.d[t][i]);
-        const float r[4] = {r4.x, r4.y, r4.z, r4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w}, d[4] = {d4.x, d4.y, d4.z, d4.w};
+        const ulonglong2 r = *reinterpret_cast<const ulonglong2*>(&s.r[t][i]);
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&s.k[t][i]);
+        const ulonglong2 d = *reinterpret_cast<const ulonglong2*>(&s.d[t][i]);
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          float(&row)[4] = S[q][e];
-          y[0] = fmaf(r[e], row[0], y[0]); y[1] = fmaf(r[e], row[1], y[1]);
-          y[2] = fmaf(r[e], row[2], y[2]); y[3] = fmaf(r[e], row[3], y[3]);
-          row[0] = fmaf(d[e], row[0], k[e] * v.x); row[1] = fmaf(d[e], row[1], k[e] * v.y);
-          row[2] = fmaf(d[e], row[2], k[e] * v.z); row[3] = fmaf(d[e], row[3], k[e] * v.w);
+        for (int c = 0; c < 4; ++c) {
+          y2[c] = fma_f32x2(r.x, S[2 * q][c], y2[c]);
+          S[2 * q][c] = fma_f32x2(d.x, S[2 * q][c], mul_f32x2(k.x, v[c]));
+          y2[c] = fma_f32x2(r.y, S[2 * q + 1][c], y2[c]);
+          S[2 * q + 1][c] = fma_f32x2(d.y, S[2 * q + 1][c], mul_f32x2(k.y, v[c]));
         }
+      }
+      float y[4];
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        float lo, hi;
+        unpack_f32x2(y2[c], lo, hi);
+        y[c] = lo + hi;
       }
       // sum over the eight row groups, each step halving what a lane still carries: four shuffles for four columns
       const bool b2 = rg & 4, b1 = rg & 2;
@@ -181,11 +192,87 @@ __global__ void __launch_bounds__(DP * 2) wkv_seq_kernel(const UbWkvArgs a) {
     __syncthreads();
     bonus_terms<DP>(a, s, n, h);
     st.walk(s, n);
+    if (so >= 0 && t0 + n == q_len) st.store(a.state + ((long long)so * a.H + h) * per, a.D);
     __syncthreads();
     for (int t = warp; t < n; t += nw)
       finish_token<T>(a, row0 + t0 + t, h, lane, [&](int c) { return fmaf(s.bonus[t], s.v[t][c], s.y[t][c]); });
   }
-  if (so >= 0) st.store(a.state + ((long long)so * a.H + h) * per, a.D);
+}
+
+// One token of every sequence: a read and a write of the state.  Everything else that the CTA needs is requested in front of
+// the state, so that its latency runs under the state's.
+template <typename T, int DP>
+__global__ void __launch_bounds__(DP * 2) wkv_step_kernel(const UbWkvArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ __align__(16) float r_s[DP], k_s[DP], d_s[DP], v_s[DP], y_s[DP];
+  __shared__ float red[DP / 32 > 0 ? DP / 32 : 1], red2[DP / 32 > 0 ? DP / 32 : 1];
+  const int h = blockIdx.x, seq = blockIdx.y, i = threadIdx.x, D = a.D, warp = i >> 5, lane = i & 31;
+  const long long off = (a.row0 + seq) * a.ld + (long long)h * D + i;
+  const bool mine = i < D;
+  float r = 0.f, k = 0.f, v = 0.f, g = 0.f, ww = 0.f, u = 0.f, nw = 0.f;
+  if (mine) {
+    r = float(reinterpret_cast<const T*>(a.r)[off]);
+    k = float(reinterpret_cast<const T*>(a.k)[off]);
+    v = float(reinterpret_cast<const T*>(a.v)[off]);
+    g = float(reinterpret_cast<const T*>(a.g)[off]);
+    ww = a.ww[off];
+    u = a.u[h * D + i];
+    nw = a.norm_w[h * D + i];
+  }
+  const int si = state_row(a, a.state_in, seq), so = state_row(a, a.state_out, seq);
+  const long long per = (long long)D * D;
+  State<DP> st;
+  // four columns of a thread, its rows in pairs: the layout of State, loaded row by row
+  float4 f[State<DP>::RPT];
+  const float* src = a.state + ((long long)max(si, 0) * a.H + h) * per;
+#pragma unroll
+  for (int p = 0; p < State<DP>::RPT; ++p) {
+    const int row = st.row(p >> 1) + (p & 1);
+    f[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (si >= 0 && row < D && st.cg * 4 < D) f[p] = __ldcs(reinterpret_cast<const float4*>(src + (long long)row * D + st.cg * 4));
+  }
+  if (i < DP) {
+    r_s[i] = r;
+    k_s[i] = k;
+    v_s[i] = v;
+    d_s[i] = mine ? expf(-expf(ww)) : 1.f;
+    const float b = warp_sum(r * u * k);
+    if (lane == 0) red[warp] = b;
+  }
+  __syncthreads();
+  float bonus = 0.f;
+#pragma unroll
+  for (int w = 0; w < DP / 32; ++w) bonus += red[w];
+  float y[4] = {0.f, 0.f, 0.f, 0.f};
+  const float4 v4 = *reinterpret_cast<const float4*>(&v_s[st.cg * 4]);
+  float* dst = a.state + ((long long)max(so, 0) * a.H + h) * per;
+#pragma unroll
+  for (int p = 0; p < State<DP>::RPT; ++p) {
+    const int row = st.row(p >> 1) + (p & 1);
+    const float rr = r_s[row], kk = k_s[row], dd = d_s[row];
+    y[0] = fmaf(rr, f[p].x, y[0]); y[1] = fmaf(rr, f[p].y, y[1]); y[2] = fmaf(rr, f[p].z, y[2]); y[3] = fmaf(rr, f[p].w, y[3]);
+    f[p].x = fmaf(dd, f[p].x, kk * v4.x); f[p].y = fmaf(dd, f[p].y, kk * v4.y);
+    f[p].z = fmaf(dd, f[p].z, kk * v4.z); f[p].w = fmaf(dd, f[p].w, kk * v4.w);
+    if (so >= 0 && row < D && st.cg * 4 < D) __stcs(reinterpret_cast<float4*>(dst + (long long)row * D + st.cg * 4), f[p]);
+  }
+#pragma unroll
+  for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) y[c] += __shfl_xor_sync(0xffffffffu, y[c], o);
+  if (st.rg == 0) *reinterpret_cast<float4*>(&y_s[st.cg * 4]) = make_float4(y[0], y[1], y[2], y[3]);
+  __syncthreads();
+  const float o = mine ? fmaf(bonus, v, y_s[i]) : 0.f;
+  if (i < DP) {
+    const float sq = warp_sum(o * o);
+    if (lane == 0) red2[warp] = sq;
+  }
+  __syncthreads();
+  if (!mine) return;
+  float sq = 0.f;
+#pragma unroll
+  for (int w = 0; w < DP / 32; ++w) sq += red2[w];
+  reinterpret_cast<T*>(a.out)[off] = T(o * (1.f / sqrtf(sq / a.norm_dim + a.eps)) * nw * silu(g));
 }
 
 // (sequence, chunk inside it) of a chunk index of the launch; false past the last one
@@ -264,12 +351,24 @@ __global__ void __launch_bounds__(256) wkv_carry_kernel(const UbWkvArgs a) {
   if (e >= per) return;
   float4 S = make_float4(0.f, 0.f, 0.f, 0.f);
   if (si >= 0) S = *reinterpret_cast<const float4*>(a.state + ((long long)si * a.H + h) * per + e);
-  for (int c = 0; c < n; ++c) {
-    float4* q = reinterpret_cast<float4*>(ws_q(a, base + c, h) + e);
-    const float p = ws_p(a, base + c, h)[e / a.D];
-    const float4 v = *q;
-    *q = S;
-    S = make_float4(fmaf(p, S.x, v.x), fmaf(p, S.y, v.y), fmaf(p, S.z, v.z), fmaf(p, S.w, v.w));
+  // eight chunks are requested before the first of them is used
+  constexpr int U = 8;
+  const int row = e / a.D;
+  for (int c0 = 0; c0 < n; c0 += U) {
+    float4 v[U];
+    float p[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (c0 + u < n) {
+        v[u] = __ldcs(reinterpret_cast<const float4*>(ws_q(a, base + c0 + u, h) + e));
+        p[u] = __ldg(ws_p(a, base + c0 + u, h) + row);
+      }
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      if (c0 + u < n) {
+        *reinterpret_cast<float4*>(ws_q(a, base + c0 + u, h) + e) = S;
+        S = make_float4(fmaf(p[u], S.x, v[u].x), fmaf(p[u], S.y, v[u].y), fmaf(p[u], S.z, v[u].z), fmaf(p[u], S.w, v[u].w));
+      }
   }
   if (so >= 0) *reinterpret_cast<float4*>(a.state + ((long long)so * a.H + h) * per + e) = S;
 }
@@ -349,6 +448,7 @@ static cudaError_t launch(const UbWkvArgs& a, cudaStream_t st) {
   const dim3 block(DP * 2);
   const size_t tile = sizeof(Tile<DP>), out = sizeof(float) * (DP * DP + OT * (DP + 4));
   cudaError_t e;
+  if (a.q_start == nullptr) return launch_pdl(wkv_step_kernel<T, DP>, dim3(a.H, a.num_seqs), block, (size_t)0, st, a);
   if (a.chunk <= 0) {
     if ((e = allow_smem(wkv_seq_kernel<T, DP>, tile)) != cudaSuccess) return e;
     return launch_pdl(wkv_seq_kernel<T, DP>, dim3(a.H, a.num_seqs), block, tile, st, a);

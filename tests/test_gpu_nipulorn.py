@@ -80,7 +80,7 @@ CUTS = [[37], [2], [1], [33, 1, 2, 1, 27], [1, 17]]
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("H,taps,mix,tile", [(8, 2, 5, 0), (50, 4, 5, 0), (136, 7, 0, 1), (200, 1, 5, 3), (1000, 3, 0, 0), (2048, 4, 5, 16),
-                                             (4096, 5, 0, 2), (9000, 2, 3, 0), (264, 24, 5, 4)])
+                                             (4096, 5, 0, 2), (9000, 2, 5, 0), (4096, 4, 5, 0), (2048, 1, 0, 0), (264, 24, 5, 4)])
 def test_sublayer_input(dtype, H, taps, mix, tile):
     """Residual add of the normed sublayer rows, the next norm, its convolution and the token-shift mixes, in portions."""
     from unillm_b200.ops import cuda_ops as K
@@ -89,7 +89,7 @@ def test_sublayer_input(dtype, H, taps, mix, tile):
     x = [_rand(n, H, seed=10 + i, dtype=torch.float32, scale=2.0) for i, n in enumerate(LENS)]
     y = [_rand(n, H, seed=30 + i) for i, n in enumerate(LENS)]
     wy, wn = _rand(H, seed=1, scale=0.3), _rand(H, seed=2, scale=0.3)
-    conv, mu = _rand(H, taps, seed=3, scale=0.4), _rand(mix, H, seed=4, dtype=torch.float32) if mix else None
+    conv, mu = _rand(H, taps, seed=3, scale=0.4), _rand(mix, H, seed=4) if mix else None
     dev = lambda t: _pad(t, Hp).to("cuda", dtype).contiguous()
     f32 = lambda t: _pad(t.float(), Hp).cuda().contiguous()
     conv_state = torch.full((2 * len(LENS), taps - 1, Hp), 77.0, device="cuda")       # never to be read before it is written
@@ -101,8 +101,8 @@ def test_sublayer_input(dtype, H, taps, mix, tile):
             order, parts = _portions(step, half)
             cat = lambda ts: torch.cat([ts[s][a:b] for s, a, b in order])
             xs, out = K.sublayer_in(f32(cat(x)), parts, dev(wn), eps=1e-4, y=dev(cat(y)) if with_y else None,
-                                    y_weight=dev(wy) if with_y else None, conv=f32(conv.t()), conv_state=conv_state,
-                                    mu=None if mu is None else f32(mu), shift_state=shift, width=H, tile=tile)
+                                    y_weight=dev(wy) if with_y else None, conv=dev(conv.t()), conv_state=conv_state,
+                                    mu=None if mu is None else dev(mu), shift_state=shift, width=H, tile=tile)
             assert xs[:, H:].abs().sum() == 0 and out[..., H:].abs().sum() == 0
             r = 0
             for s, a, b in order:
@@ -412,7 +412,7 @@ def test_unequal_batch_with_blocks_and_slots_used_again(case, dtype):
     alone = _engine(m, dtype)
     for k in seqs:
         want = P.forward(cfg, w, seqs[k])
-        _check_rows(got[k], want, dtype if dtype == torch.float32 or len(seqs[k]) > 10 else None)
+        _check_rows(got[k], want, dtype if dtype == torch.float32 or len(seqs[k]) > 40 else None)
         err = C.row_error(got[k], C.score(alone, seqs[k], [(0, len(seqs[k]))]))
         assert err.max() < (5e-4 if dtype == torch.float32 else 0.3)
 

@@ -194,8 +194,8 @@ class RunnerWeights:
                 if L + n in p:
                     self.t[L + n] = dev(_pad(p[L + n], 0, H))
             for n in ("conv1", "conv2"):
-                if L + n in p:                                # [taps, H] in fp32: the kernel walks the taps of a channel
-                    self.t[L + n] = _pad(p[L + n].t(), 1, H).to(device=device, dtype=torch.float32).contiguous()
+                if L + n in p:                                # [taps, H]: neighbouring threads read neighbouring channels
+                    self.t[L + n] = dev(_pad(p[L + n].t(), 1, H))
             if L + "act" in p:
                 from ..models.mixers import xielu_coefficients
 
@@ -287,7 +287,7 @@ class RunnerWeights:
 
         if ls.mixer == "wkv":
             d, dp, rank = ls.head_dim, kh.dk, self._round(ls.decay_rank)
-            t[L + "mu"] = f32(_pad(p[L + "mu"], 1, H))
+            t[L + "mu"] = dev(_pad(p[L + "mu"], 1, H))
             t[L + "w_rkvg"] = dev(torch.stack([_pad(heads(w, n, d, dp, 0, n), 1, H) for w in p[L + "w_rkvg"]]))
             t[L + "w_d1"] = dev(_pad(_pad(p[L + "w_d1"], 0, rank), 1, H))
             t[L + "w_d2"] = dev(_pad(heads(p[L + "w_d2"], n, d, dp, 0, n), 1, rank))
@@ -497,7 +497,7 @@ class RunnerWeights:
                     self.t[L + n + ".b"] = zeros(H)
             if s.input_conv:
                 for n in ("conv1", "conv2"):
-                    self.t[L + n] = rnd(s.input_conv, H).float()
+                    self.t[L + n] = rnd(s.input_conv, H)
             if ls.mlp == "dense":
                 width = self._round(s.layer_intermediate(i))
                 self.t[L + "w_up"], self.t[L + "w_down"] = rnd(width, H), rnd(H, width)
@@ -507,7 +507,7 @@ class RunnerWeights:
                     self.act_params[i] = (0.8, 1.3)
             if ls.mixer == "wkv":
                 rank, C = self._round(ls.decay_rank or 64), kh.hq * kh.dk
-                self.t[L + "mu"] = torch.full((5, H), 0.5, device=self.t["embed"].device)
+                self.t[L + "mu"] = torch.full_like(rnd(5, H), 0.5)
                 self.t[L + "w_rkvg"] = torch.stack([rnd(C, H) for _ in range(4)])
                 self.t[L + "w_d1"], self.t[L + "w_d2"], self.t[L + "d0"] = rnd(rank, H), rnd(C, rank), zeros(C) - 2.0
                 self.t[L + "u"], self.t[L + "o_norm"] = rnd(kh.hq, kh.dk).float(), ones(C).float()

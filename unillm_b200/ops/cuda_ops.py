@@ -332,10 +332,10 @@ def sublayer_in(x: torch.Tensor, portions: Sequence[Portions], weight: torch.Ten
                 conv_state: Optional[torch.Tensor] = None, mu: Optional[torch.Tensor] = None,
                 shift_state: Optional[torch.Tensor] = None, width: Optional[int] = None, offset_one: bool = True, tile: int = 0):
     """What the next sublayer reads: ``x' = x + norm(y)``, ``h = norm(x')`` plus its causal convolution over time with the taps
-    ``conv`` (fp32 [taps, width], the last one meets the token itself), and with ``mu`` (fp32 [n, width]) the n token-shift
-    mixes ``h + (previous h - h) * mu``.  Returns ``(x', out)``; out is [rows, width], or [n, rows, width] with ``mu``, in
+    ``conv`` ([taps, width], the last one meets the token itself), and with ``mu`` ([5, width]) the five token-shift
+    mixes ``h + (previous h - h) * mu``.  Returns ``(x', out)``; out is [rows, width], or [5, rows, width] with ``mu``, in
     the type of ``weight``.  The state tensors hold what the sequences of ``portions`` carry on."""
-    f32 = _elem("sublayer_in", weight, y, y_weight)
+    f32 = _elem("sublayer_in", weight, y, y_weight, conv, mu)
     T, Hp = x.shape
     if x.dtype != torch.float32 or not x.is_contiguous() or weight.numel() != Hp:
         raise ValueError("sublayer_in: contiguous fp32 stream, weights of its width")
@@ -344,8 +344,10 @@ def sublayer_in(x: torch.Tensor, portions: Sequence[Portions], weight: torch.Ten
     taps = 0 if conv is None else conv.shape[0]
     n_mix = 0 if mu is None else mu.shape[0]
     for t in (conv, mu):
-        if t is not None and (t.dtype != torch.float32 or t.shape[1] != Hp or not t.is_contiguous()):
-            raise ValueError("sublayer_in: conv and mu are contiguous fp32 [n, width]")
+        if t is not None and (t.shape[1] != Hp or not t.is_contiguous()):
+            raise ValueError("sublayer_in: conv and mu are contiguous [n, width]")
+    if n_mix not in (0, 5):
+        raise ValueError("sublayer_in: five token-shift mixes or none")
     _state_rows("sublayer_in conv", conv_state, (max(taps - 1, 0), Hp))
     _state_rows("sublayer_in shift", shift_state, (Hp,))
     states = [t for t in (conv_state, shift_state) if t is not None]
@@ -363,8 +365,8 @@ def sublayer_in(x: torch.Tensor, portions: Sequence[Portions], weight: torch.Ten
         a.q_start, a.err = _p(p.q_start), err_word(x.device).data_ptr()
         a.row0, a.out_mix_stride = p.row0, T * Hp
         a.H, a.Hp, a.taps, a.n_mix, a.num_seqs, a.max_q = width or Hp, Hp, taps, n_mix, p.n, p.max_q
-        # rows in front of a tile are computed again: larger tiles once there are enough of them for the SMs
-        a.tile = tile or (1 if p.max_q == 1 else 4 if p.rows <= 1024 else 8 if p.rows <= 4096 else 16)
+        # rows in front of a tile are computed again: tiles as large as still leaves two CTAs per SM
+        a.tile = tile or min(max(-(-p.rows // 296), 2), 32)
         a.f32, a.eps, a.w_off = int(f32), eps, 1.0 if offset_one else 0.0
         N.check(N.cuda_lib().ub_sublayer_in(C.byref(a), _stream(x)), "ub_sublayer_in")
     return x_out, out
@@ -506,6 +508,22 @@ def gemm_heads(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Ten
     return out
 
 
+def latent_splits(seqs: int, heads: int, ctx: int, row: int, v_dim: int) -> int:
+    """Key ranges per sequence of a decode step: rounds of CTAs over the SMs at their share of the bandwidth, against what the
+    partial results cost to write and merge."""
+    ctas = seqs * -(-heads // (16 if heads <= 16 else 32))
+    resident = 148 * (2 if row <= 320 else 1)
+    best, cost = 1, None
+    for s in (1, 2, 4, 8, 16):
+        if s > 1 and ctx // s < 128:
+            break
+        us = -(-ctas * s // resident) * (ctx / s * row * 2 / 45e3 * (resident // 148) + 1.5)
+        us += 0.0 if s == 1 else 3.0 + seqs * heads * s * v_dim * 8 / 4e6
+        if cost is None or us < cost:
+            best, cost = s, us
+    return best
+
+
 def attn_latent(q: torch.Tensor, cache: torch.Tensor, v_dim: int, block_tables: torch.Tensor, seq_lens: torch.Tensor, *, scale: float,
                 sinks: Optional[torch.Tensor] = None, q_start: Optional[torch.Tensor] = None, max_q_len: int = 1,
                 out: Optional[torch.Tensor] = None, splits: int = 0, scratch: Optional[torch.Tensor] = None,
@@ -525,9 +543,7 @@ def attn_latent(q: torch.Tensor, cache: torch.Tensor, v_dim: int, block_tables: 
         splits = 1
     if splits <= 0:
         ctx = max_seq_len if max_seq_len is not None else block_tables.shape[1] * cache.shape[2]
-        ctas, splits = T * -(-H // (16 if H <= 16 else 32)), 1
-        while ctas * splits < 148 and ctx // (splits * 2) >= 128 and splits < 16:
-            splits *= 2
+        splits = latent_splits(T, H, ctx, D, v_dim)
     if splits > 1:
         need = T * H * splits * (v_dim + 2)
         if scratch is None or scratch.numel() < need:
