@@ -202,7 +202,7 @@ __global__ void __launch_bounds__(DP * 2) wkv_seq_kernel(const UbWkvArgs a) {
 // One token of every sequence: a read and a write of the state.  Everything else that the CTA needs is requested in front of
 // the state, so that its latency runs under the state's.
 template <typename T, int DP>
-__global__ void __launch_bounds__(DP * 2) wkv_step_kernel(const UbWkvArgs a) {
+__global__ void __launch_bounds__(DP * 2, DP <= 64 ? 1024 / (DP * 2) : 2) wkv_step_kernel(const UbWkvArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ __align__(16) float r_s[DP], k_s[DP], d_s[DP], v_s[DP], y_s[DP];
