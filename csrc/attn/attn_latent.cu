@@ -23,7 +23,7 @@ constexpr float LOG2E = 1.4426950408889634f, LN2 = 0.6931471805599453f;
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool pred) {
   const int sz = pred ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz) : "memory");
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(sz));
 }
 __device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
@@ -101,21 +101,29 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
     if (t < n_tiles) {
       const uint32_t st = kv_u + (t & 1) * KT * L.pitch;
       const int base = kv_lo + t * KT;
-      // a warp fetches whole rows: one block-table entry per row, 16-byte chunks at consecutive addresses
-#pragma unroll 4
-      for (int r = warp; r < KT; r += THREADS / 32) {
-        const int pos = base + r;
-        long long src = -1;
+      // A warp fetches eight whole rows; lane r looks row r's page up, then every row is at most three 16-byte chunks per
+      // lane.  Nothing but the shuffled offset stands between the copies: with a look-up and a bounds check in front of
+      // every row the issue of a tile took longer than its arithmetic.
+      constexpr int RPW = KT / (THREADS / 32), CPR = 3;     // rows per warp, chunks per lane and row (D <= 640, with padding)
+      long long src = -1;
+      if (lane < RPW) {
+        const int pos = base + warp * RPW + lane;
         if (pos < kv_hi) {
           const int bi = pos >> bs_shift;
           const int blk = bi - page0 < BT_MAX ? bt_sm[bi - page0] : (bi < a.max_blocks_per_seq ? bt[bi] : -1);
           if (blk < 0 || blk >= a.num_blocks) set_err(a.err, ERR_BOUNDS, seq);
           else src = (((long long)blk << bs_shift) + (pos & (a.block_size - 1))) * D;
         }
-        const __nv_bfloat16* g = cache + (src >= 0 ? src : 0);
-        for (int c = lane; c < nck; c += 32) {
-          const bool ok = src >= 0 && c < nch;
-          cp_async16(st + r * L.pitch + c * 16, ok ? g + c * 8 : cache, ok);
+      }
+      const uint32_t dst = st + warp * RPW * L.pitch + lane * 16;
+#pragma unroll
+      for (int r = 0; r < RPW; ++r) {
+        const long long o = __shfl_sync(0xffffffffu, src, r);
+        const __nv_bfloat16* g = cache + (o >= 0 ? o : 0) + lane * 8;
+#pragma unroll
+        for (int k = 0; k < CPR; ++k) {
+          const int c = lane + 32 * k;
+          if (c < nck) cp_async16(dst + r * L.pitch + k * 512, o >= 0 && c < nch ? g + k * 256 : cache, o >= 0 && c < nch);
         }
       }
     }

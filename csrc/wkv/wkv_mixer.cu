@@ -144,16 +144,47 @@ struct State {
   }
 };
 
-// head norm, weight and gate of one token by one warp; o(c) is the recurrence's output in column c
-template <typename T, typename F>
-__device__ __forceinline__ void finish_token(const UbWkvArgs& a, long long row, int h, int lane, F o) {
-  float sq = 0.f;
-  for (int c = lane; c < a.D; c += 32) { const float v = o(c); sq += v * v; }
-  const float r = 1.f / sqrtf(warp_sum(sq) / a.norm_dim + a.eps);
-  const long long off = row * a.ld + (long long)h * a.D;
-  for (int c = lane; c < a.D; c += 32) {
-    const float g = float(reinterpret_cast<const T*>(a.g)[off + c]);
-    reinterpret_cast<T*>(a.out)[off + c] = T(o(c) * r * a.norm_w[h * a.D + c] * silu(g));
+// head norm, weight and gate of the tokens warp, warp + nw, ... < n; o(t, c) is the recurrence's output of token t in column
+// c.  Four tokens of a warp go together, so that their gates are under way at the same time.
+template <typename T, int DP, typename F>
+__device__ __forceinline__ void finish_tokens(const UbWkvArgs& a, long long row, int n, int h, F o) {
+  constexpr int CPL = DP / 32, U = 4;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const T* gp = reinterpret_cast<const T*>(a.g);
+  T* out = reinterpret_cast<T*>(a.out);
+  float w[CPL];
+#pragma unroll
+  for (int j = 0; j < CPL; ++j) w[j] = lane + 32 * j < a.D ? a.norm_w[h * a.D + lane + 32 * j] : 0.f;
+  for (int t0 = warp; t0 < n; t0 += U * nw) {
+    float v[U][CPL], g[U][CPL], sq[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int t = t0 + u * nw;
+      sq[u] = 0.f;
+#pragma unroll
+      for (int j = 0; j < CPL; ++j) {
+        const int c = lane + 32 * j;
+        const bool ok = t < n && c < a.D;
+        g[u][j] = ok ? float(gp[(row + t) * a.ld + (long long)h * a.D + c]) : 0.f;
+        v[u][j] = ok ? o(t, c) : 0.f;
+        sq[u] = fmaf(v[u][j], v[u][j], sq[u]);
+      }
+    }
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1)
+#pragma unroll
+      for (int u = 0; u < U; ++u) sq[u] += __shfl_xor_sync(0xffffffffu, sq[u], x);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int t = t0 + u * nw;
+      if (t >= n) continue;
+      const float r = 1.f / sqrtf(sq[u] / a.norm_dim + a.eps);
+#pragma unroll
+      for (int j = 0; j < CPL; ++j) {
+        const int c = lane + 32 * j;
+        if (c < a.D) out[(row + t) * a.ld + (long long)h * a.D + c] = T(v[u][j] * r * w[j] * silu(g[u][j]));
+      }
+    }
   }
 }
 
@@ -177,7 +208,7 @@ __global__ void __launch_bounds__(DP * 2) wkv_seq_kernel(const UbWkvArgs a) {
   pdl_wait();
   extern __shared__ __align__(16) uint8_t raw[];
   Tile<DP>& s = *reinterpret_cast<Tile<DP>*>(raw);
-  const int h = blockIdx.x, seq = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int h = blockIdx.x, seq = blockIdx.y;
   int qs, q_len;
   seq_rows(a, seq, qs, q_len);
   if (q_len <= 0) return;
@@ -194,8 +225,7 @@ __global__ void __launch_bounds__(DP * 2) wkv_seq_kernel(const UbWkvArgs a) {
     st.walk(s, n);
     if (so >= 0 && t0 + n == q_len) st.store(a.state + ((long long)so * a.H + h) * per, a.D);
     __syncthreads();
-    for (int t = warp; t < n; t += nw)
-      finish_token<T>(a, row0 + t0 + t, h, lane, [&](int c) { return fmaf(s.bonus[t], s.v[t][c], s.y[t][c]); });
+    finish_tokens<T, DP>(a, row0 + t0, n, h, [&](int t, int c) { return fmaf(s.bonus[t], s.v[t][c], s.y[t][c]); });
   }
 }
 
@@ -323,9 +353,12 @@ __global__ void __launch_bounds__(DP * 2) wkv_chunk_kernel(const UbWkvArgs a) {
     st.walk(s, n);
     __syncthreads();
     const long long off = (long long)(qs + t0) * a.ld + (long long)h * a.D;
-    for (int i = threadIdx.x; i < n * a.D; i += blockDim.x) {
-      const int t = i / a.D, c = i % a.D;
-      ws_y(a)[off + (long long)t * a.ld + c] = fmaf(s.bonus[t], s.v[t][c], s.y[t][c]);
+    for (int i = threadIdx.x; i < n * (DP / 4); i += blockDim.x) {
+      const int t = i / (DP / 4), c = i % (DP / 4) * 4;
+      if (c >= a.D) continue;
+      const float b = s.bonus[t];
+      const float4 v = *reinterpret_cast<const float4*>(&s.v[t][c]), y = *reinterpret_cast<const float4*>(&s.y[t][c]);
+      *reinterpret_cast<float4*>(ws_y(a) + off + (long long)t * a.ld + c) = make_float4(fmaf(b, v.x, y.x), fmaf(b, v.y, y.y), fmaf(b, v.z, y.z), fmaf(b, v.w, y.w));
     }
     if (threadIdx.x < a.D) {
       for (int t = 0; t < n; ++t) {
@@ -373,8 +406,8 @@ __global__ void __launch_bounds__(256) wkv_carry_kernel(const UbWkvArgs a) {
   if (so >= 0) *reinterpret_cast<float4*>(a.state + ((long long)so * a.H + h) * per + e) = S;
 }
 
-// 32 tokens of a chunk per CTA: y += (r * product) S_entering, then norm, weight and gate
-constexpr int OT = 32;
+// 64 tokens of a chunk per CTA: y += (r * product) S_entering, then norm, weight and gate
+constexpr int OT = 64, OG = OT / 8;      // tokens per CTA, per thread
 
 template <typename T, int DP>
 __global__ void __launch_bounds__(DP * 2) wkv_out_kernel(const UbWkvArgs a) {
@@ -383,7 +416,7 @@ __global__ void __launch_bounds__(DP * 2) wkv_out_kernel(const UbWkvArgs a) {
   extern __shared__ __align__(16) uint8_t raw[];
   float(*S)[DP] = reinterpret_cast<float(*)[DP]>(raw);
   float(*rp)[DP + 4] = reinterpret_cast<float(*)[DP + 4]>(raw + sizeof(float) * DP * DP);
-  const int h = blockIdx.x, chunk = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int h = blockIdx.x, chunk = blockIdx.y;
   int seq, c0, c1, qs;
   if (!find_chunk(a, chunk, seq, c0, c1, qs)) return;
   const int t0 = c0 + blockIdx.z * OT, n = min(OT, c1 - t0), D = a.D;
@@ -403,11 +436,11 @@ __global__ void __launch_bounds__(DP * 2) wkv_out_kernel(const UbWkvArgs a) {
     *reinterpret_cast<float4*>(&rp[t][c]) = f;
   }
   __syncthreads();
-  // DP / 4 column groups x 8 token groups of 4 tokens
+  // DP / 4 column groups x 8 token groups
   const int cg = threadIdx.x % (DP / 4), tg = threadIdx.x / (DP / 4);
-  float acc[4][4];
+  float acc[OG][4];
 #pragma unroll
-  for (int t = 0; t < 4; ++t)
+  for (int t = 0; t < OG; ++t)
 #pragma unroll
     for (int c = 0; c < 4; ++c) acc[t][c] = 0.f;
   for (int i = 0; i < D; i += 4) {
@@ -415,8 +448,8 @@ __global__ void __launch_bounds__(DP * 2) wkv_out_kernel(const UbWkvArgs a) {
 #pragma unroll
     for (int e = 0; e < 4; ++e) s4[e] = *reinterpret_cast<const float4*>(&S[i + e][cg * 4]);
 #pragma unroll
-    for (int t = 0; t < 4; ++t) {
-      const float4 p4 = *reinterpret_cast<const float4*>(&rp[tg * 4 + t][i]);
+    for (int t = 0; t < OG; ++t) {
+      const float4 p4 = *reinterpret_cast<const float4*>(&rp[tg * OG + t][i]);
       const float p[4] = {p4.x, p4.y, p4.z, p4.w};
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
@@ -427,15 +460,14 @@ __global__ void __launch_bounds__(DP * 2) wkv_out_kernel(const UbWkvArgs a) {
   }
   __syncthreads();
 #pragma unroll
-  for (int t = 0; t < 4; ++t) {
-    const int tt = tg * 4 + t;
+  for (int t = 0; t < OG; ++t) {
+    const int tt = tg * OG + t;
     float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
     if (tt < n && cg * 4 < D) f = *reinterpret_cast<const float4*>(ws_y(a) + off + (long long)tt * a.ld + cg * 4);
     *reinterpret_cast<float4*>(&rp[tt][cg * 4]) = make_float4(acc[t][0] + f.x, acc[t][1] + f.y, acc[t][2] + f.z, acc[t][3] + f.w);
   }
   __syncthreads();
-  for (int t = warp; t < n; t += nw)
-    finish_token<T>(a, a.row0 + qs + t0 + t, h, lane, [&](int c) { return rp[t][c]; });
+  finish_tokens<T, DP>(a, a.row0 + qs + t0, n, h, [&](int t, int c) { return rp[t][c]; });
 }
 
 template <typename K>

@@ -216,7 +216,7 @@ def test_matrices_per_head(dtype, M, H, N, Kd):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("E,T,N,Kd", [(4, 1, 40, 56), (4, 16, 256, 192), (4, 17, 64, 96), (3, 300, 136, 72), (4, 1000, 512, 256)])
+@pytest.mark.parametrize("E,T,N,Kd", [(4, 1, 40, 56), (4, 16, 256, 192), (4, 17, 64, 96), (3, 300, 136, 72), (4, 1000, 512, 256), (2, 4100, 136, 64)])
 def test_stacked_products(dtype, E, T, N, Kd):
     from unillm_b200.ops import cuda_ops as K
 

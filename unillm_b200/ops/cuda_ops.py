@@ -418,7 +418,8 @@ _GROUP_TILES: dict = {}
 
 def gemm_stacked(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     """``out[e] = x[e] @ w[e]^T`` for a stack of equal products: x [E, T, K] (contiguous), w [E, N, K] -> [E, T, N].  Up to 16
-    rows on the weight-streaming kernel, beyond on the grouped GEMM with a tile table that is fixed by the sizes."""
+    rows on the weight-streaming kernel, beyond on the grouped GEMM with a tile table that is fixed by the sizes; thousands of
+    rows fill the device one product at a time, in the CTA-pair kernel that the grouped form does not have."""
     f32 = _elem("gemm_stacked", x, w)
     E, T, Kd = x.shape
     n = w.shape[1]
@@ -431,6 +432,10 @@ def gemm_stacked(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
         a.M, a.N, a.K, a.ldx, a.ldw, a.ldo, a.w_rows_total = T, n, Kd, Kd, Kd, n, n
         a.batch, a.x_batch, a.w_batch, a.out_batch = E, T * Kd, n * Kd, T * n
         N.check(N.cuda_lib().ub_gemm_tn(C.byref(a), _stream(x)), "ub_gemm_tn(stacked)")
+        return out
+    if T >= 4096 and not f32:
+        for e in range(E):
+            gemm_tn(x[e], w[e], out=out[e])
         return out
     tn = moe_tile_tokens(E * T, 1, E)
     key = (E, T, tn, x.device)
