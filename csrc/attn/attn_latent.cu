@@ -3,11 +3,14 @@
 // row is the key of every head, its first Dv elements are the value.  Paged like the other caches, one row per position.
 //
 // A CTA takes 16 * MT rows -- a row is (query token, head) -- of one sequence and one range of its keys; with one query per
-// sequence these are the heads, so a tile of cache rows fetched once serves all of them, as key and as value.  Tiles of 64
-// positions come through a two-stage cp.async ring into rows padded by 16 bytes (ldmatrix without bank conflicts).  Per
-// tile: eight warps form the scores, four groups of 16 positions times two halves of the row; all threads do the online
-// softmax in fp32 on the summed halves; the warps then share the value columns.  Causal by position; softmax sinks join in
-// the epilogue, or for split ranges in the merge, once.
+// sequence these are the heads, so a tile of cache rows fetched once serves all of them, as key and as value.
+//
+// Four warps fetch: tiles of 64 positions by cp.async into a ring of two or three stages whose rows are padded by 16 bytes
+// (ldmatrix without bank conflicts), the block table read once, ahead.  The fill of a tile is bound by the path from L2 into
+// shared memory and takes about as long as the tile's arithmetic, so it has warps of its own.  Eight warps compute: the
+// scores in four groups of 16 positions times two halves of the row, the online softmax in fp32 on the summed halves, then
+// the value columns among them.  Causal by position; softmax sinks join in the epilogue, or for split ranges in the merge,
+// once.
 #include <math_constants.h>
 
 #include "../common/ptx.cuh"
@@ -18,7 +21,7 @@ extern "C" int ub_attn_split_merge(const UbAttnArgs* a, void* stream);
 namespace ub {
 namespace latent {
 
-constexpr int KT = 64, THREADS = 256;
+constexpr int KT = 64, THREADS = 256, LOADERS = 128;   // computing and fetching threads
 constexpr float LOG2E = 1.4426950408889634f, LN2 = 0.6931471805599453f;
 
 __device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool pred) {
@@ -45,11 +48,11 @@ constexpr int BT_MAX = 512;                // block-table entries held in shared
 
 struct Layout {
   int pitch, q, kv, s, p, row, bt, total;  // byte offsets
-  __host__ __device__ Layout(int D, int mt) {
+  __host__ __device__ Layout(int D, int mt, int stages) {
     pitch = (D + 15) / 16 * 32 + 16;
     q = 0;
     kv = 16 * mt * pitch;
-    s = kv + 2 * KT * pitch;
+    s = kv + stages * KT * pitch;
     p = s + 2 * 16 * mt * S_PITCH * 4;
     row = p + 16 * mt * P_PITCH;
     bt = row + 16 * mt * 3 * 4;            // behind alpha, max, sum per row
@@ -57,13 +60,20 @@ struct Layout {
   }
 };
 
+// Narrow rows: two CTAs on an SM, so that one computes while the other one's warps meet at a barrier.
 template <int MT, int VP>
-__global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a) {
+struct Residency { static constexpr int CTAS = MT == 1 && VP <= 2 ? 2 : 1; };
+
+template <int MT, int VP>
+__global__ void __launch_bounds__(THREADS + LOADERS, (Residency<MT, VP>::CTAS)) attn_latent_kernel(const UbAttnArgs a, const int stages) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int ROWS = 16 * MT, TPR = THREADS / ROWS, CPT = KT / TPR;
   extern __shared__ __align__(128) uint8_t sm[];
-  const Layout L(a.D, MT);
+  __shared__ uint64_t full[3], empty[3];
+  __shared__ int abort_word;
+  volatile int* abort_flag = &abort_word;
+  const Layout L(a.D, MT, stages);
   const int D = a.D, Dv = a.Dv, nch = D / 8, nck = (D + 15) / 16 * 2;
   float* s_sm = reinterpret_cast<float*>(sm + L.s);
   float* alpha_sm = reinterpret_cast<float*>(sm + L.row);
@@ -86,28 +96,41 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
   const __nv_bfloat16* qg = reinterpret_cast<const __nv_bfloat16*>(a.q);
   const uint32_t q_u = smem_u32(sm + L.q), kv_u = smem_u32(sm + L.kv), p_u = smem_u32(sm + L.p);
 
-  for (int i = threadIdx.x; i < ROWS * nck; i += THREADS) {
+  for (int i = threadIdx.x; i < ROWS * nck; i += THREADS + LOADERS) {
     const int r = i / nck, c = i % nck, row = row0 + r;
     const bool ok = row < rows_total && c < nch;
     const int tok = ok ? row / a.Hq : 0, h = ok ? row % a.Hq : 0;
     cp_async16(q_u + r * L.pitch + c * 16, qg + (ok ? (long long)(qs + tok) * a.q_stride + (long long)h * D + c * 8 : 0), ok);
   }
+  asm volatile("cp.async.commit_group;" ::: "memory");
   int* bt_sm = reinterpret_cast<int*>(sm + L.bt);
   const int page0 = kv_lo / a.block_size, pages = n_tiles > 0 ? (kv_hi - 1) / a.block_size - page0 + 1 : 0;
-  for (int i = threadIdx.x; i < min(pages, BT_MAX); i += THREADS) bt_sm[i] = page0 + i < a.max_blocks_per_seq ? bt[page0 + i] : -1;
+  for (int i = threadIdx.x; i < min(pages, BT_MAX); i += THREADS + LOADERS) bt_sm[i] = page0 + i < a.max_blocks_per_seq ? bt[page0 + i] : -1;
+  if (threadIdx.x == 0) {
+    abort_word = 0;
+    for (int i = 0; i < stages; ++i) {
+      mbar_init(&full[i], LOADERS);
+      mbar_init(&empty[i], THREADS);
+    }
+    fence_mbar_init();
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
   __syncthreads();
-  const int bs_shift = 31 - __clz(a.block_size);           // a power of two (host check)
-  auto issue = [&](int t) {
-    if (t < n_tiles) {
-      const uint32_t st = kv_u + (t & 1) * KT * L.pitch;
+
+  // A wait that gives up has set the error word and the abort flag; the later ones then return at once, and every thread
+  // goes on to its end in step with the others.
+  if (warp >= THREADS / 32) {
+    // ------------------------------ fetching warps ------------------------------
+    const int bs_shift = 31 - __clz(a.block_size);         // a power of two (host check)
+    const int w = warp - THREADS / 32;
+    constexpr int RPW = KT / (LOADERS / 32), CPR = 3;      // rows per warp, chunks per lane and row (D <= 640, with padding)
+    int st = 0, ph = 1;
+    for (int t = 0; t < n_tiles; ++t) {
       const int base = kv_lo + t * KT;
-      // A warp fetches eight whole rows; lane r looks row r's page up, then every row is at most three 16-byte chunks per
-      // lane.  Nothing but the shuffled offset stands between the copies: with a look-up and a bounds check in front of
-      // every row the issue of a tile took longer than its arithmetic.
-      constexpr int RPW = KT / (THREADS / 32), CPR = 3;     // rows per warp, chunks per lane and row (D <= 640, with padding)
+      // lane r looks row r's page up; nothing but the shuffled offset then stands between the copies
       long long src = -1;
       if (lane < RPW) {
-        const int pos = base + warp * RPW + lane;
+        const int pos = base + w * RPW + lane;
         if (pos < kv_hi) {
           const int bi = pos >> bs_shift;
           const int blk = bi - page0 < BT_MAX ? bt_sm[bi - page0] : (bi < a.max_blocks_per_seq ? bt[bi] : -1);
@@ -115,21 +138,29 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
           else src = (((long long)blk << bs_shift) + (pos & (a.block_size - 1))) * D;
         }
       }
-      const uint32_t dst = st + warp * RPW * L.pitch + lane * 16;
+      const bool ok = __all_sync(0xffffffffu, mbar_wait(&empty[st], ph, abort_flag, a.err, 710 + st));
+      if (ok) {
+        const uint32_t dst = kv_u + (st * KT + w * RPW) * L.pitch + lane * 16;
 #pragma unroll
-      for (int r = 0; r < RPW; ++r) {
-        const long long o = __shfl_sync(0xffffffffu, src, r);
-        const __nv_bfloat16* g = cache + (o >= 0 ? o : 0) + lane * 8;
+        for (int r = 0; r < RPW; ++r) {
+          const long long off = __shfl_sync(0xffffffffu, src, r);
+          const __nv_bfloat16* g = cache + (off >= 0 ? off : 0) + lane * 8;
 #pragma unroll
-        for (int k = 0; k < CPR; ++k) {
-          const int c = lane + 32 * k;
-          if (c < nck) cp_async16(dst + r * L.pitch + k * 512, o >= 0 && c < nch ? g + k * 256 : cache, o >= 0 && c < nch);
+          for (int k = 0; k < CPR; ++k) {
+            const int c = lane + 32 * k;
+            const bool in = off >= 0 && c < nch;
+            if (c < nck) cp_async16(dst + r * L.pitch + k * 512, in ? g + k * 256 : cache, in);
+          }
         }
       }
+      asm volatile("cp.async.mbarrier.arrive.noinc.shared::cta.b64 [%0];" ::"r"(smem_u32(&full[st])) : "memory");
+      if (++st == stages) { st = 0; ph ^= 1; }
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  issue(0);
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    return;
+  }
+  // ------------------------------ computing warps ------------------------------
+  auto sync = [] { asm volatile("bar.sync 1, 256;" ::: "memory"); };
 
   float o[MT][VP * 2][4];
 #pragma unroll
@@ -143,11 +174,10 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
   const int tg = warp & 3, kh = warp >> 2, nks = nck / 2, half = (nks + 1) / 2;
   const int ks0 = kh * half, ks1 = min(nks, ks0 + half);
 
+  int st = 0, ph = 0;
   for (int t = 0; t < n_tiles; ++t) {
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();                                       // tile t is there; everyone is done with tile t - 1
-    issue(t + 1);
-    const uint32_t kb = kv_u + (t & 1) * KT * L.pitch;
+    mbar_wait(&full[st], ph, abort_flag, a.err, 700 + st);
+    const uint32_t kb = kv_u + st * KT * L.pitch;
     {
       float s[MT][2][4], s2[MT][2][4];                     // even and odd steps: two chains of dependent MMAs
 #pragma unroll
@@ -186,7 +216,7 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
           *reinterpret_cast<float2*>(d + 8 * S_PITCH) = make_float2(s[mt][j][2] + s2[mt][j][2], s[mt][j][3] + s2[mt][j][3]);
         }
     }
-    __syncthreads();
+    sync();
     {
       const float* s0 = s_sm + my_row * S_PITCH;
       const float* s1 = s0 + ROWS * S_PITCH;
@@ -215,7 +245,7 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
       l_run = l_run * al + sum;
       if (part == 0) alpha_sm[my_row] = al;
     }
-    __syncthreads();
+    sync();
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt) {
       const float al_a = alpha_sm[mt * 16 + (lane >> 2)], al_b = alpha_sm[mt * 16 + (lane >> 2) + 8];
@@ -243,13 +273,14 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
         }
       }
     }
+    mbar_arrive(&empty[st]);
+    if (++st == stages) { st = 0; ph ^= 1; }
   }
-  asm volatile("cp.async.wait_group 0;" ::: "memory");
   if (part == 0) {
     m_sm[my_row] = m_run;
     l_sm[my_row] = l_run;
   }
-  __syncthreads();
+  sync();
 #pragma unroll
   for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -289,7 +320,10 @@ __global__ void __launch_bounds__(THREADS) attn_latent_kernel(const UbAttnArgs a
 
 template <int MT, int VP>
 static int launch(const UbAttnArgs& a, int mq, cudaStream_t st) {
-  const Layout L(a.D, MT);
+  // two stages where that lets a second CTA onto the SM, else as many as fit
+  const bool pair = Residency<MT, VP>::CTAS == 2 && Layout(a.D, MT, 2).total <= 112 * 1024;
+  const int stages = !pair && Layout(a.D, MT, 3).total <= 225 * 1024 ? 3 : 2;
+  const Layout L(a.D, MT, stages);
   static int allowed[UB_MAX_DEVICES] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -299,7 +333,7 @@ static int launch(const UbAttnArgs& a, int mq, cudaStream_t st) {
     allowed[dev] = L.total;
   }
   const dim3 grid((mq * a.Hq + 16 * MT - 1) / (16 * MT), a.splits, a.num_seqs);
-  cudaError_t e = launch_pdl(attn_latent_kernel<MT, VP>, grid, dim3(THREADS), (size_t)L.total, st, a);
+  cudaError_t e = launch_pdl(attn_latent_kernel<MT, VP>, grid, dim3(THREADS + LOADERS), (size_t)L.total, st, a, stages);
   if (e == cudaSuccess) e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
 }

@@ -351,6 +351,12 @@ __device__ __forceinline__ uint32_t pack_bf16x2(float lo, float hi) {
   __nv_bfloat162 t = __floats2bfloat162_rn(lo, hi);
   return *reinterpret_cast<uint32_t*>(&t);
 }
+// e^v - 1 - v for v <= 0, for epilogues that round to bf16: the Taylor polynomial near zero (its remainder there is below
+// 2e-8), where the difference of the fast exponential would cancel.
+__device__ __forceinline__ float exp_tail(float v) {
+  const float near = v * v * fmaf(v, fmaf(v, fmaf(v, 1.f / 120.f, 1.f / 24.f), 1.f / 6.f), 0.5f);
+  return v > -0.125f ? near : __expf(v) - 1.f - v;
+}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -115,7 +115,7 @@ __device__ __forceinline__ float apply_act(float v, int act, float pa, float pb)
     case UB_ACT_QUICK_GELU: return v / (1.f + __expf(-1.702f * v));
     case UB_ACT_SIGMOID: return 1.f / (1.f + __expf(-v));
     case UB_ACT_TANH: return tanhf(v);
-    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? pa * v * v : pb * (expm1f(v) - v));
+    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? pa * v * v : pb * exp_tail(v));
     default: return v;
   }
 }

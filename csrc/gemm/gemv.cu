@@ -39,7 +39,7 @@ __device__ __forceinline__ float act_apply(float v, const UbGemmArgs& a) {
     case UB_ACT_SIGMOID: return 1.f / (1.f + __expf(-v));
     case UB_ACT_TANH: return tanhf(v);
     case UB_ACT_SOFTPLUS: return v > 20.f ? v : log1pf(__expf(v));
-    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? a.act_a * v * v : a.act_b * (expm1f(v) - v));
+    case UB_ACT_XIELU: return fmaf(0.5f, v, v > 0.f ? a.act_a * v * v : a.act_b * exp_tail(v));
     default: return v;
   }
 }
