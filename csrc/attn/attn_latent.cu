@@ -62,7 +62,7 @@ struct Layout {
 
 // Narrow rows: two CTAs on an SM, so that one computes while the other one's warps meet at a barrier.
 template <int MT, int VP>
-struct Residency { static constexpr int CTAS = MT == 1 && VP <= 2 ? 2 : 1; };
+struct Residency { static constexpr int CTAS = MT == 1 && VP <= 2 ? 2 : 0; };     // 0: left to the compiler
 
 template <int MT, int VP>
 __global__ void __launch_bounds__(THREADS + LOADERS, (Residency<MT, VP>::CTAS)) attn_latent_kernel(const UbAttnArgs a, const int stages) {

@@ -519,8 +519,8 @@ def latent_splits(seqs: int, heads: int, ctx: int, row: int, v_dim: int) -> int:
     ctas = seqs * -(-heads // (16 if heads <= 16 else 32))
     resident = 148 * (2 if row <= 328 and heads <= 16 else 1)
     best, cost = 1, None
-    for s in (1, 2, 4, 8, 16):
-        if s > 1 and ctx // s < 128:
+    for s in (1, 2, 4, 8, 16, 32):
+        if s > 1 and ctx // s < 64:
             break
         us = -(-ctas * s // resident) * (ctx / s * row * 2 / 45e3 * (resident // 148) + 3.0)
         us += 0.0 if s == 1 else 3.0 + seqs * heads * s * v_dim * 8 / 4e6
