@@ -186,7 +186,8 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
     if (ra < gn) slope_a = a.alibi_slopes[h0 + ra] * LOG2E;
     if (rb < gn) slope_b = a.alibi_slopes[h0 + rb] * LOG2E;
   }
-  const float sc = a.scale * LOG2E;
+  const float sc = (a.softcap > 0.f ? a.softcap : a.scale) * LOG2E;
+  const float cap_in = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
   float o[DV / 8][4];
 #pragma unroll
   for (int i = 0; i < DV / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
@@ -230,6 +231,12 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
       ldsm_x4(smem_u32(kb + tile_off<DK>(r, c)), b0, b1, b2, b3);
       mma_bf16(s[0], qf[ks], b0, b1);
       mma_bf16(s[1], qf[ks], b2, b3);
+    }
+    if (cap_in != 0.f) {
+#pragma unroll
+      for (int j = 0; j < 2; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[j][e] = tanh_by_exp(s[j][e] * cap_in);
     }
     float mx_a = m_a, mx_b = m_b;
 #pragma unroll
@@ -385,7 +392,7 @@ static int launch_sized(const UbAttnArgs& a, cudaStream_t st) {
 extern "C" int ub_attn_decode_mma_supported(const UbAttnArgs* a) {
   const int dv = a->Dv > 0 ? a->Dv : a->D;
   if (a->D > 256 || dv > 256 || a->D % 8 != 0 || dv % 8 != 0) return 0;
-  if (a->merge_o != nullptr && (a->D != dv || (dv != 64 && dv != 128) || a->sinks != nullptr)) return 0;
+  if (a->merge_o != nullptr && (a->D != dv || (dv != 64 && dv != 128) || a->sinks != nullptr || a->softcap > 0.f)) return 0;
   if (a->block_size < 8 || a->block_size > 64 || (a->block_size & (a->block_size - 1))) return 0;   // whole pages per 64-token tile
   if (a->Hkv <= 0 || a->Hq % a->Hkv != 0 || a->q_stride % 8 != 0) return 0;
   if ((reinterpret_cast<uintptr_t>(a->q) & 15) || (reinterpret_cast<uintptr_t>(a->k_cache) & 15) ||

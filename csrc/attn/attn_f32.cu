@@ -63,7 +63,9 @@ __global__ void __launch_bounds__(WARPS * 32) attn_f32_kernel(const UbAttnArgs a
         d0 = fmaf(q_s[warp][d + 2], kv.z, d0);
         d0 = fmaf(q_s[warp][d + 3], kv.w, d0);
       }
-      s = d0 * a.scale + slope * (float)(pos - qpos);
+      d0 *= a.scale;
+      if (a.softcap > 0.f) d0 = a.softcap * tanhf(d0 / a.softcap);
+      s = d0 + slope * (float)(pos - qpos);
     }
     const float mx = fmaxf(m, warp_max(s));
     if (mx == -CUDART_INF_F) continue;

@@ -152,7 +152,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
     slope_a = a.alibi_slopes[kvh * G + min(rowa, rows_total - 1) % G] * P_LOG2E;
     slope_b = a.alibi_slopes[kvh * G + min(rowb, rows_total - 1) % G] * P_LOG2E;
   }
-  const float sc = a.scale * P_LOG2E;
+  const float sc = (a.softcap > 0.f ? a.softcap : a.scale) * P_LOG2E;
+  const float cap_in = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
 
   float o[DV / 8][4];
 #pragma unroll
@@ -202,6 +203,12 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
       }
     }
     // scale, mask, online softmax
+    if (cap_in != 0.f) {
+#pragma unroll
+      for (int j = 0; j < KT / 8; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[j][e] = tanh_by_exp(s[j][e] * cap_in);
+    }
     float mx_a = m_a, mx_b = m_b;
 #pragma unroll
     for (int j = 0; j < KT / 8; ++j) {
@@ -344,7 +351,7 @@ extern "C" int ub_attn_prefill_last_path() { return g_last_path; }
 extern "C" int ub_attn_prefill(const UbAttnArgs* a, void* stream_v) {
   using namespace ub;
   if (a->num_seqs <= 0 || a->max_q_len <= 0) return 0;
-  const bool plain = a->sinks == nullptr && (a->Dv == 0 || a->Dv == a->D);   // what the tensor-core kernel takes
+  const bool plain = a->sinks == nullptr && a->softcap <= 0.f && (a->Dv == 0 || a->Dv == a->D);   // what the tensor-core kernel takes
   if (plain && tc_enabled() && ub_attn_prefill_tc_supported(a)) {
     g_last_path = 1;
     return ub_attn_prefill_tc(a, stream_v);

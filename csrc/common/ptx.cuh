@@ -313,6 +313,9 @@ __device__ __forceinline__ void publish_to_peers(uint32_t* local_count, uint32_t
 // ----------------------------------------------------------------------------
 // Small numeric helpers
 // ----------------------------------------------------------------------------
+// tanh(x) = 1 - 2 / (1 + e^(2x)) to a few 1e-7 absolute, for scores that are capped (|x| of any size).
+__device__ __forceinline__ float tanh_by_exp(float x) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * x)); }
+
 // Two fp32 values per instruction (fma.rn.f32x2 / add.f32x2 / mul.f32x2 on a 64-bit register pair) and a three-input
 // maximum: epilogues and softmax loops are bound by the instruction issue of a few warps, and these halve their
 // arithmetic instructions.

@@ -170,6 +170,14 @@ typedef struct UbSublayerInArgs {
   long long row0, out_mix_stride;
   int H, Hp, taps, n_mix /* 0 or 5 */, num_seqs, max_q, state_rows, tile /* tokens per CTA */, f32;
   float eps, w_off;
+  /* Without convolution and mixes rows do not depend on one another: n_rows of them in one launch, whatever the portions are
+     (x_out may then be x, or NULL).  Their y may be a mixture: y_gate[t] * y + sum_k topk_w[t, k] * yx[row_slot[t, k]]. */
+  const void* yx;           /* [slots, Hp] expert rows, or NULL */
+  const int* row_slot;      /* [T, K], negative = none */
+  const float* topk_w;      /* [T, K] */
+  const float* y_gate;      /* [T] or NULL */
+  const int* rows;          /* row of x and y per output row, or NULL */
+  int n_rows, x_rows, K, slots;
 } UbSublayerInArgs;
 int ub_sublayer_in(const UbSublayerInArgs* args, void* stream);
 
@@ -192,6 +200,27 @@ typedef struct UbWkvArgs {
 } UbWkvArgs;
 int ub_wkv_mixer(const UbWkvArgs* args, void* stream);
 long long ub_wkv_workspace_floats(int rows, int ld, int H, int D, int max_chunks);
+
+/* ---------------- K16d : gated delta rule over ragged portions (csrc/delta/delta_mixer.cu) ---------------- */
+typedef struct UbDeltaArgs {
+  const void *qkv;           /* rows [Q: G * dk | K: G * dk | V: H * dv] in front of the convolutions */
+  const void *gate;          /* rows of H * dv */
+  const void *b, *a;         /* rows of H: write strength and decay, before their non-linearities */
+  const void* conv;          /* [taps, 2 * G * dk + H * dv], of qkv's element type */
+  const float *a_log, *dt_bias, *norm_w;       /* [H], [H], [dv] */
+  float* conv_state;         /* [state_rows, taps - 1, 2 * G * dk + H * dv] last inputs of the convolutions */
+  float* state;              /* [state_rows, H, dk, dv] */
+  const int *state_in, *state_out, *q_start;   /* as in UbSublayerInArgs */
+  void* out;                 /* rows of H * dv */
+  float* ws;                 /* portions: ub_delta_workspace_floats(..) floats */
+  int* err;
+  long long row0, ld, ld_out;                  /* ld: elements between rows of qkv, gate, b and a */
+  int H, G, dk, dv /* padded to 8, <= 256 */, dk_real, dv_real, taps, num_seqs, max_q, rows, state_rows, f32;
+  int lanes;                 /* portions: lanes that share a column of the state (8, 16, 32), 0 = chosen here */
+  float eps;
+} UbDeltaArgs;
+int ub_delta_mixer(const UbDeltaArgs* args, void* stream);
+long long ub_delta_workspace_floats(int rows, int H, int G, int dk, int dv);
 
 /* ---------------- K1h : one matrix per head, out[t, h] = x[t, h] @ w[h]^T (csrc/gemm/gemm_heads.cu) ---------------- */
 typedef struct UbHeadGemmArgs {
@@ -248,6 +277,8 @@ typedef struct UbRopeArgs {
   int norm_dim;              /* elements of a head that the RMS norm averages over (0 = D; less when heads are padded) */
   int f32;                   /* qkv, caches and norm weights are fp32 */
   int k_cache_only;          /* 1: the rotated k need not be written back into qkv (it is in the cache) */
+  int row_norm;              /* 1: one norm over all q of a token and one over all k; the weights have Hq * D and Hkv * D elements */
+  long long ld;              /* elements between rows of qkv (0: rows are dense) */
 } UbRopeArgs;
 int ub_rope_kv_append(const UbRopeArgs* args, void* stream);
 
@@ -285,6 +316,7 @@ typedef struct UbAttnArgs {
   const float* sinks;
   int Dv;                    /* value head size (0 = D): v_cache [.., Dv], out [T, Hq, Dv], scratch [.., Dv + 2] */
   int kv_shared;             /* ub_attn_f32: values are the first Dv elements of the key rows (ub_attn_latent: always so) */
+  float softcap;             /* > 0: scores become softcap * tanh(score / softcap), before masks, ALiBi and sinks */
 } UbAttnArgs;
 /* prompts over expanded latents (csrc/attn/attn_expanded_tc.cu): ub_latent_gather copies the cache rows of the sequences to
    consecutive rows (each sequence from page_start[seq] * 16 on, zeros behind its end and up to `rows`), ub_attn_expanded
@@ -414,6 +446,12 @@ typedef struct UbMoeRouteArgs {
   const void* router_b;     /* [E] added to the logits (router_w mode), or NULL */
   int x_f32;                /* x is fp32 (the residual stream itself) */
   int router_f32;           /* router_w and router_b are fp32 */
+  /* router_w mode: experts are chosen by softmax(logits) + correction, within the keep_groups of `groups` equal groups of
+     neighbours that have the largest such score; the weights are the chosen softmax values over their sum + 1e-20 */
+  const void* correction;   /* [E] of the router's type, or NULL */
+  int groups, keep_groups;  /* 0 or 1: no groups */
+  const void* shared_w;     /* [H] of the router's type: shared_gate[t] = sigmoid(x . shared_w), or NULL */
+  float* shared_gate;       /* [T] */
 } UbMoeRouteArgs;
 int ub_moe_route(const UbMoeRouteArgs* args, void* stream);
 int ub_moe_gather(const void* x, const int* sorted_rows, void* out, int rows, int K, int H, void* stream);

@@ -24,13 +24,16 @@ constexpr int MOE_MAX_K = 16;
 template <typename XT, typename WT, int TB>
 __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) {
   constexpr int EB = 4;
-  __shared__ float logits_s[TB][MOE_MAX_E];
+  __shared__ float logits_s[TB][MOE_MAX_E + 1];   // the last one in use may be the gate of the always-on expert
+  __shared__ float choice_s[TB][MOE_MAX_E];
   const int t0 = blockIdx.x * TB, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int E = a.E, K = a.K;
   if (a.router_w != nullptr) {
     const XT* x = reinterpret_cast<const XT*>(a.x);
     const WT* w = reinterpret_cast<const WT*>(a.router_w);
-    for (int e0 = warp * EB; e0 < E; e0 += 4 * EB) {
+    const int rows = E + (a.shared_w != nullptr);
+    const WT* sw = reinterpret_cast<const WT*>(a.shared_w);
+    for (int e0 = warp * EB; e0 < rows; e0 += 4 * EB) {
       float acc[TB][EB];
 #pragma unroll
       for (int i = 0; i < TB; ++i)
@@ -39,7 +42,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
       for (int h = lane * 8; h < a.H; h += 256) {
         float ws[EB][8];
 #pragma unroll
-        for (int j = 0; j < EB; ++j) load8(w + (long long)min(e0 + j, E - 1) * a.H + h, ws[j]);
+        for (int j = 0; j < EB; ++j) load8((e0 + j == E && sw != nullptr ? sw : w + (long long)min(e0 + j, E - 1) * a.H) + h, ws[j]);
 #pragma unroll
         for (int i = 0; i < TB; ++i) {
           float xs[8];
@@ -56,7 +59,10 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
         for (int j = 0; j < EB; ++j) {
           float v = warp_sum(acc[i][j]);
           const int e = e0 + j;
-          if (e >= E) continue;
+          if (e >= E) {
+            if (e == E && sw != nullptr && lane == 0) logits_s[i][E] = v;
+            continue;
+          }
           if (a.router_b != nullptr) v += (float)reinterpret_cast<const WT*>(a.router_b)[e];
           // the reference model keeps router logits in the activation dtype: round like a bf16 linear layer would
           if (lane == 0) logits_s[i][e] = a.round_logits_bf16 ? __bfloat162float(__float2bfloat16(v)) : v;
@@ -82,6 +88,44 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
     float den = 0.f;
     for (int e = lane; e < E; e += 32) den += expf(logit[e] - mx);
     den = warp_sum(den);
+    if (a.shared_gate != nullptr && lane == 0) a.shared_gate[t] = 1.f / (1.f + expf(-logit[E]));
+    const bool scored = a.correction != nullptr || a.groups > 1;
+    const float* pick = logit;                    // what the choice goes by
+    if (scored) {
+      float* sc = choice_s[i];
+      for (int e = lane; e < E; e += 32)
+        sc[e] = expf(logit[e] - mx) / den + (a.correction != nullptr ? (float)reinterpret_cast<const WT*>(a.correction)[e] : 0.f);
+      __syncwarp();
+      if (a.groups > 1 && a.keep_groups < a.groups) {
+        // a lane holds the best score of groups lane, lane + 32, ..; the best groups are taken out one by one, then the
+        // experts of those that are left over are closed
+        const int size = E / a.groups;
+        uint32_t kept = 0;
+        for (int k = 0; k < a.keep_groups; ++k) {
+          float best = -INFINITY;
+          int bi = 0x7fffffff;
+          for (int g = lane, j = 0; g < a.groups; g += 32, ++j) {
+            if (kept >> j & 1u) continue;
+            float m = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, sc[e]);
+            if (m > best || (m == best && g < bi)) { best = m; bi = g; }
+          }
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) {
+            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+          }
+          if (bi < a.groups && (bi & 31) == lane) kept |= 1u << (bi >> 5);
+        }
+        __syncwarp();
+        for (int g = lane, j = 0; g < a.groups; g += 32, ++j)
+          if (!(kept >> j & 1u))
+            for (int e = g * size; e < (g + 1) * size; ++e) sc[e] = -INFINITY;
+        __syncwarp();
+      }
+      pick = sc;
+    }
     uint32_t taken = 0;  // bit j: expert lane + 32*j already selected
     float mine = 0.f;    // lane k keeps the k-th choice
     int mine_e = 0;
@@ -90,7 +134,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
       int bi = 0x7fffffff;
       for (int e = lane, j = 0; e < E; e += 32, ++j) {
         if (taken >> j & 1u) continue;
-        const float v = logit[e];
+        const float v = pick[e];
         if (v > best || (v == best && e < bi)) { best = v; bi = e; }
       }
 #pragma unroll
@@ -100,10 +144,10 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
         if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
       }
       if (bi < E && (bi & 31) == lane) taken |= 1u << (bi >> 5);
-      if (lane == k) { mine = expf(best - mx); mine_e = bi < E ? bi : 0; }
+      if (lane == k) { mine_e = bi < E ? bi : 0; mine = expf(logit[mine_e] - mx); }
     }
     const float s = warp_sum(lane < K ? mine : 0.f);
-    const float inv = a.norm_topk ? 1.f / s : 1.f / den;
+    const float inv = !a.norm_topk ? 1.f / den : scored ? 1.f / (den * (s / den + 1e-20f)) : 1.f / s;
     if (lane < K) {
       a.topk_ids[(long long)t * K + lane] = mine_e;
       a.topk_w[(long long)t * K + lane] = mine * inv * a.weight_scale;
@@ -448,6 +492,10 @@ extern "C" int ub_moe_route(const UbMoeRouteArgs* a, void* stream_v) {
   if (a->E <= 0 || a->E > ub::MOE_MAX_E || a->K <= 0 || a->K > ub::MOE_MAX_K || a->K > a->E) return -2;
   if (a->router_w != nullptr && (a->H % 8 != 0 || a->x == nullptr)) return -3;
   if (a->tiles != nullptr && (a->tile_tokens <= 0 || a->max_tiles <= 0)) return -4;
+  if (a->router_w == nullptr && (a->correction != nullptr || a->shared_w != nullptr)) return -5;
+  if ((a->shared_w != nullptr) != (a->shared_gate != nullptr)) return -5;
+  if (a->groups > 1 && (a->E % a->groups != 0 || a->keep_groups < 1 || a->keep_groups > a->groups || a->K > a->keep_groups * (a->E / a->groups)))
+    return -6;
   UbMoeRouteArgs b = *a;
   if (b.weight_scale == 0.f) b.weight_scale = 1.f;
   if (b.router_w != nullptr && b.x_f32 && b.router_f32) ub::launch_route<float, float>(b, st);

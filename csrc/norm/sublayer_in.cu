@@ -10,6 +10,9 @@
 // from the sequence's state rows (the last taps - 1 values of n, the last h), and the portion leaves its own behind in
 // OTHER rows, so every CTA of the launch may read the old ones whenever it runs.
 //
+// Without convolution and mixes a row depends on nothing but itself: sublayer_alone_kernel, one CTA per row, in which y may
+// also be a mixture-of-experts result that is summed here, with a gate on its always-on part.
+//
 // One token per sequence (decoding) has a kernel of its own: what the state contributes does not depend on the norms, so all
 // loads are under way before the first sum.  Longer portions: a CTA takes `tile` consecutive tokens of one sequence and recomputes the few rows of n in front of them (x and y are read
 // again, x' goes to a buffer of its own), so tiles are independent.  The last taps - 1 rows of n stay in shared memory; a
@@ -446,6 +449,109 @@ __global__ void __launch_bounds__(512) sublayer_step_kernel(const UbSublayerInAr
   }
 }
 
+// Rows that depend on nothing but themselves.
+template <typename T, int CH>
+__global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float red[2][16];
+  const int nch = a.Hp / 8;
+  long long src = blockIdx.x;
+  if (a.rows != nullptr) {
+    src = a.rows[blockIdx.x];
+    if (src < 0 || src >= a.x_rows) {
+      if (threadIdx.x == 0) set_err(a.err, ERR_BOUNDS, blockIdx.x);
+      src = 0;
+    }
+  }
+  const T* y = reinterpret_cast<const T*>(a.y);
+  const T* yx = reinterpret_cast<const T*>(a.yx);
+  const float gate = a.y_gate != nullptr ? a.y_gate[src] : 1.f;
+  float x[CH][8], f[CH][8];
+  Raw8<T> wy8[CH], wn8[CH];
+  float sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int ch = threadIdx.x + c * blockDim.x;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[c][e] = f[c][e] = 0.f;
+    if (ch >= nch) continue;
+    load8(a.x + src * a.Hp + ch * 8, x[c]);
+    wn8[c].load(reinterpret_cast<const T*>(a.wn) + ch * 8);
+    if (y == nullptr && yx == nullptr) continue;
+    wy8[c].load(reinterpret_cast<const T*>(a.wy) + ch * 8);
+    if (y != nullptr) {
+      load8(y + src * a.Hp + ch * 8, f[c]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[c][e] *= gate;
+    }
+    for (int k0 = 0; yx != nullptr && k0 < a.K; k0 += 4) {         // four experts' rows are under way at a time
+      float g[4][8], w[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        w[j] = 0.f;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) g[j][e] = 0.f;
+        if (k0 + j >= a.K) continue;
+        const int slot = __ldg(a.row_slot + src * a.K + k0 + j);
+        if (slot >= a.slots) {
+          set_err(a.err, ERR_BOUNDS, blockIdx.x);
+        } else if (slot >= 0) {
+          w[j] = __ldg(a.topk_w + src * a.K + k0 + j);
+          load8(yx + (long long)slot * a.Hp + ch * 8, g[j]);
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[c][e] = fmaf(w[j], g[j][e], f[c][e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq += f[c][e] * f[c][e];           // pad columns are zero
+  }
+  int flip = 0;
+  if (y != nullptr || yx != nullptr) {
+    const float r = 1.f / sqrtf(block_sum(sq, red, flip) / a.H + a.eps);
+#pragma unroll
+    for (int c = 0; c < CH; ++c) {
+      const int ch = threadIdx.x + c * blockDim.x;
+      if (ch >= nch) continue;
+      float w[8];
+      wy8[c].get(w);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) x[c][e] += f[c][e] * r * (a.w_off + w[e]);
+      if (a.x_out != nullptr) store8(a.x_out + (long long)blockIdx.x * a.Hp + ch * 8, x[c]);
+    }
+  }
+  sq = 0.f;
+#pragma unroll
+  for (int c = 0; c < CH; ++c)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) sq += x[c][e] * x[c][e];
+  const float r = 1.f / sqrtf(block_sum(sq, red, flip) / a.H + a.eps);
+#pragma unroll
+  for (int c = 0; c < CH; ++c) {
+    const int ch = threadIdx.x + c * blockDim.x;
+    if (ch >= nch) continue;
+    float w[8];
+    wn8[c].get(w);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[c][e] *= r * (a.w_off + w[e]);
+    store8(reinterpret_cast<T*>(a.out) + (long long)blockIdx.x * a.Hp + ch * 8, x[c]);
+  }
+}
+
+template <typename T>
+static cudaError_t launch_alone(const UbSublayerInArgs& a, cudaStream_t st) {
+  const int nch = a.Hp / 8;
+  const int threads = nch >= 512 ? 512 : (nch + 31) / 32 * 32;
+  const int ch = (nch + threads - 1) / threads;
+  const dim3 grid(a.n_rows), block(threads);
+  if (ch <= 1) return launch_pdl(sublayer_alone_kernel<T, 1>, grid, block, (size_t)0, st, a);
+  if (ch <= 2) return launch_pdl(sublayer_alone_kernel<T, 2>, grid, block, (size_t)0, st, a);
+  return launch_pdl(sublayer_alone_kernel<T, 4>, grid, block, (size_t)0, st, a);
+}
+
 template <typename T>
 static cudaError_t launch_step(const UbSublayerInArgs& a, cudaStream_t st) {
   const int nch = a.Hp / 8;
@@ -489,7 +595,19 @@ static cudaError_t launch(const UbSublayerInArgs& a, cudaStream_t st) {
 
 extern "C" int ub_sublayer_in(const UbSublayerInArgs* a, void* stream) {
   using namespace ub;
+  if (a->n_rows > 0) {
+    if (a->H <= 0 || a->Hp % 8 != 0 || a->Hp < a->H || a->Hp > 16384) return -2;
+    if (a->x == nullptr || a->wn == nullptr || a->out == nullptr || a->taps != 0 || a->n_mix != 0) return -3;
+    if ((a->y != nullptr || a->yx != nullptr) && a->wy == nullptr) return -4;
+    if (a->yx != nullptr && (a->row_slot == nullptr || a->topk_w == nullptr || a->K <= 0)) return -4;
+    if (a->rows != nullptr && a->x_out != nullptr) return -4;
+    cudaStream_t s = reinterpret_cast<cudaStream_t>(stream);
+    cudaError_t e = a->f32 ? subin::launch_alone<float>(*a, s) : subin::launch_alone<__nv_bfloat16>(*a, s);
+    if (e == cudaSuccess) e = cudaGetLastError();
+    return e == cudaSuccess ? 0 : -(int)e;
+  }
   if (a->num_seqs <= 0 || a->max_q <= 0) return 0;
+  if (a->yx != nullptr || a->y_gate != nullptr || a->rows != nullptr) return -4;
   if (a->H <= 0 || a->Hp % 8 != 0 || a->Hp < a->H || a->Hp > 16384) return -2;
   if (a->x == nullptr || a->wn == nullptr || a->out == nullptr || a->tile <= 0 || a->num_seqs > 65535) return -3;
   if (a->y != nullptr && (a->wy == nullptr || a->x_out == nullptr || a->x_out == a->x)) return -4;

@@ -5,7 +5,8 @@
 // One CTA per token, one warp per head (round-robin).  cos/sin are computed on the fly from the
 // position (no table in HBM); partial rotary, linear position scaling and Llama-3 frequency
 // scaling are parameters (or a table of frequencies).  Heads with a norm, interleaved pairs or a value size of its own go
-// through a second kernel in which a few lanes own a head, eight elements each; it also has a 32-bit form.
+// through a second kernel in which a few lanes own a head, eight elements each; it also has a 32-bit form, and one norm over
+// all query (key) elements of a token instead of one per head.
 // Slots are bounds-checked: a bad slot sets the error word and is skipped.
 //
 // Replaces in the reference: apply_rope / apply_rope_with_offset (crates/runtime/src/models_v2/
@@ -208,7 +209,26 @@ __global__ void __launch_bounds__(128) head_norm_rope_kernel(const UbRopeArgs a)
     if (threadIdx.x == 0) set_err(a.err, ERR_BOUNDS, t);
   }
   const long long blk = slot_ok ? slot / a.block_size : 0, off = slot_ok ? slot % a.block_size : 0;
-  T* row = reinterpret_cast<T*>(a.qkv) + (long long)t * ((long long)(a.Hq + a.Hkv) * D + (long long)a.Hkv * Dv);
+  T* row = reinterpret_cast<T*>(a.qkv) + (long long)t * a.ld;
+  float rq = 1.f, rk = 1.f;                       // row norms: one factor for all queries, one for all keys
+  if (a.row_norm) {
+    __shared__ float red[2][4];
+    float sq = 0.f, sk = 0.f;
+    const int nq = a.Hq * D / 8, nk = a.Hkv * D / 8;
+    for (int i = threadIdx.x; i < nq + nk; i += 128) {
+      float v[8], ss = 0.f;
+      load8(row + (long long)i * 8, v);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
+      if (i < nq) sq += ss; else sk += ss;
+    }
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
+    __syncthreads();
+    rq = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)(a.Hq * a.norm_dim) + a.norm_eps);
+    if (a.Hkv > 0) rk = 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)(a.Hkv * a.norm_dim) + a.norm_eps);
+  }
   const int grp = threadIdx.x / LPH, c = threadIdx.x % LPH, ngrp = 128 / LPH;
   const int nrot = a.Hq + a.Hkv;
   const bool have = c * 8 < D;                    // the last lanes of a group may own nothing
@@ -222,14 +242,24 @@ __global__ void __launch_bounds__(128) head_norm_rope_kernel(const UbRopeArgs a)
     for (int e = 0; e < 8; ++e) v[e] = 0.f;
     if (ok) load8(row + (long long)h * D + c * 8, v);
     const T* nw = reinterpret_cast<const T*>(h < a.Hq ? a.q_norm_w : a.k_norm_w);
-    if (a.q_norm_w != nullptr || a.k_norm_w != nullptr) {
+    float r = 1.f;
+    if (a.row_norm) {
+      r = h < a.Hq ? rq : rk;
+      nw += (long long)(h < a.Hq ? h : h - a.Hq) * D;
+      if (ok) {
+        float w[8];
+        load8(nw + c * 8, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = v[e] * r * w[e];
+      }
+    } else if (a.q_norm_w != nullptr || a.k_norm_w != nullptr) {
       float ss = 0.f;
 #pragma unroll
       for (int e = 0; e < 8; ++e) ss += v[e] * v[e];
 #pragma unroll
       for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
       if (ok && nw != nullptr) {
-        const float r = 1.f / sqrtf(ss * inv_n + a.norm_eps);
+        r = 1.f / sqrtf(ss * inv_n + a.norm_eps);
         float w[8];
         load8(nw + c * 8, w);
 #pragma unroll
@@ -246,7 +276,22 @@ __global__ void __launch_bounds__(128) head_norm_rope_kernel(const UbRopeArgs a)
           v[e + 1] = x1 * co + x0 * si;
         }
       }
-    } else if (half > 0) {                        // half % 8 == 0 (host check)
+    } else if (half > 0 && half % 8 != 0) {       // the other half of a pair lies across chunks: fetched element by element
+      float o[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int i = c * 8 + e, j = i < half ? i + half : i - half;
+        o[e] = 0.f;
+        if (ok && i < 2 * half) o[e] = (float)row[(long long)h * D + j] * r * (nw != nullptr ? (float)nw[j] : 1.f);
+      }
+      __syncwarp();                               // a head's lanes have read it before one of them writes
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int i = c * 8 + e;
+        if (i < half) v[e] = v[e] * cs[i] - o[e] * cs[half + i];
+        else if (i < 2 * half) v[e] = v[e] * cs[i - half] + o[e] * cs[i];
+      }
+    } else if (half > 0) {
       const int partner = c < hc ? c + hc : (c < 2 * hc ? c - hc : c);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
@@ -288,12 +333,17 @@ extern "C" int ub_rope_kv_append(const UbRopeArgs* a, void* stream_v) {
   if (a->T <= 0) return 0;
   if (a->D > 512 || (a->rotary_dim & 1) || a->rotary_dim > a->D) return -2;
   const int Dv = a->Dv > 0 ? a->Dv : a->D;
-  const bool general = a->f32 || Dv != a->D || a->inv_freq != nullptr || (a->norm_dim > 0 && a->norm_dim != a->D);
-  const bool wide_ok = a->D % 8 == 0 && Dv % 8 == 0 && a->D <= 256 && (a->interleaved || a->rotary_dim % 16 == 0);
+  const long long dense = (long long)(a->Hq + a->Hkv) * a->D + (long long)a->Hkv * Dv;
+  const long long ld = a->ld > 0 ? a->ld : dense;
+  const bool general = a->f32 || Dv != a->D || a->inv_freq != nullptr || (a->norm_dim > 0 && a->norm_dim != a->D) || a->row_norm || ld != dense;
+  const bool wide_ok = a->D % 8 == 0 && Dv % 8 == 0 && a->D <= 256 && ld % 8 == 0 && ld >= dense;
+  if (a->row_norm && (a->q_norm_w == nullptr || (a->Hkv > 0 && a->k_norm_w == nullptr))) return -5;
   if (general && !wide_ok) return -4;
   if (wide_ok && (general || a->interleaved || a->q_norm_w != nullptr || a->k_norm_w != nullptr)) {
     UbRopeArgs b = *a;
     b.Dv = Dv;
+    b.ld = ld;
+    if (b.norm_dim <= 0) b.norm_dim = b.D;
     cudaError_t e = b.f32 ? ub::launch_head_norm_rope<float>(b, (cudaStream_t)stream_v)
                           : ub::launch_head_norm_rope<__nv_bfloat16>(b, (cudaStream_t)stream_v);
     if (e == cudaSuccess) e = cudaGetLastError();

@@ -4,7 +4,7 @@ The shared objects are produced next to this file's package, so that they travel
 tree and are visible to whatever inspects the process's loaded libraries:
 
 * ``unillm_b200/_native/libunillm_b200_cuda.so``  -- the CUDA kernels that serving a decoder on one GPU
-  launches (``csrc/{gemm,attn,norm,norm_rope,moe,wkv,eltwise,sample,kv}``), compiled with
+  launches (``csrc/{gemm,attn,norm,norm_rope,moe,wkv,delta,eltwise,sample,kv}``), compiled with
   ``nvcc -gencode arch=compute_100a,code=sm_100a`` (Blackwell only; no other arch is built).
 * ``unillm_b200/_native/libunillm_b200_cuda_more.so``  -- the rest of ``csrc/**/*.cu``: peer-memory
   collectives, recurrences, block-quantised matrices, probes.  A process that needs none of them neither
@@ -66,7 +66,7 @@ def nvcc_path() -> str:
     return p
 
 
-SERVING_DIRS = ("attn", "eltwise", "gemm", "kv", "moe", "norm", "norm_rope", "sample", "wkv")
+SERVING_DIRS = ("attn", "delta", "eltwise", "gemm", "kv", "moe", "norm", "norm_rope", "sample", "wkv")
 CUDA_LIBS = {"serving": "libunillm_b200_cuda.so", "more": "libunillm_b200_cuda_more.so"}
 
 

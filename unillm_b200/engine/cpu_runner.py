@@ -97,7 +97,10 @@ class CpuModelRunner:
         if ls.mixer == "wkv":
             y = self._per_sequence(h, b, st, lambda x, d: MX.wkv(m.p, L, ls, x, d, self.spec.norm_eps))
             return ops_fn.linear(y, m.p[L + "wo"])
-        return self._attention(i, h, b, pos, slots)
+        if ls.mixer == "delta":
+            return self._per_sequence(h, b, st, lambda x, d: m._delta(i, x, d))
+        a = self._attention(i, h, b, pos, slots)
+        return a if ls.beside is None else m._side_by_side(i, a, self._per_sequence(h, b, st, lambda x, d: m._delta(i, x, d)))
 
     @torch.no_grad()
     def forward_logits(self, b: StepBatch) -> torch.Tensor:

@@ -42,6 +42,9 @@ def why_not_gpu(model) -> Optional[str]:
             return f"layer {i}: wkv heads above 128"
         if ls.mixer == "latent" and (ls.kv_rank > 512 or ls.kv_rank + ls.rot_dim > 624):
             return f"layer {i}: a latent above 512, or above 624 with its rotated part"
+        for mx in ls.mixers:
+            if mx.mixer == "delta" and (max(mx.head_dim, mx.v_head_dim) > 256 or not 1 <= mx.conv_taps <= 16):
+                return f"layer {i}: delta heads above 256 or more than 16 taps"
         if ls.mixer == "attention" and s.layers is not None and max(ls.head_dim, ls.v_head_dim) > 256:
             return f"layer {i}: head sizes above 256"
         if ls.moe is not None and (ls.moe.num_experts > 256 or ls.moe.top_k > 16):

@@ -33,7 +33,8 @@ def _experts(runner, i: int, h: torch.Tensor, router_x: torch.Tensor):
     with runner._prof("moe_route"):
         r = K.moe_route(router_x, t[L + "router"], m.top_k, norm_topk=m.normalize_topk, round_logits_bf16=False,
                         expert_lo=runner.w.expert_lo if runner.w.ep else 0,
-                        num_local_experts=runner.w.experts_local if runner.w.ep else 0, router_b=t.get(L + "router_b"))
+                        num_local_experts=runner.w.experts_local if runner.w.ep else 0, router_b=t.get(L + "router_b"),
+                        correction=t.get(L + "correction"), groups=m.groups, keep_groups=m.keep_groups, shared_w=t.get(L + "shared_sg"))
         xs = K.moe_gather(h, r)
     runner.launches += 3
     gu, dn = t[L + "experts_gate_up"], t[L + "experts_down"]
@@ -59,7 +60,8 @@ def _shared_expert(runner, i: int, h: torch.Tensor, residual=None) -> torch.Tens
 
 def moe_branch(runner, i: int, h: torch.Tensor, router_x: torch.Tensor):
     """The mixture's output for a layer that normalises it before the residual add: ``(base rows or None, expert rows or
-    None, routing)``, to be summed by the norm kernel.  ``router_x``: what the router reads (the 32-bit stream)."""
+    None, routing)``, to be summed by the norm kernel (which also applies ``routing.shared_gate`` to the base rows).
+    ``router_x``: what the router reads (the 32-bit stream, or the normed rows)."""
     m = runner.layers[i].moe
     y, r = _experts(runner, i, h, router_x)
     base = _shared_expert(runner, i, h) if m.num_shared_experts else None

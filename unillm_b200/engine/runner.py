@@ -24,6 +24,7 @@ Reference counterpart: the per-token loop of ``UniLLMBackend::generate`` / ``Lla
 """
 from __future__ import annotations
 
+import dataclasses
 import math
 import os
 import time
@@ -142,6 +143,7 @@ class KernelHeads:
     rot: int = 0
     vdim: int = 0
     q_rank: int = 0
+    delta: Optional["DeltaHeads"] = None         # of the layer's gated delta rule (beside the attention, or its only mixer)
 
     @property
     def qkv_rows(self) -> int:
@@ -152,6 +154,33 @@ class KernelHeads:
         if not self.own_kv:
             return 0
         return self.dk if self.q_rank else self.hkv * (self.dk + self.dv)
+
+
+@dataclass(frozen=True)
+class DeltaHeads:
+    """A gated delta rule as the kernels see it: ``hq`` heads of ``dk`` x ``dv`` states, ``hk`` query / key heads, head sizes
+    rounded up to multiples of 8.  Its rows of the layer's input projection are [Q | K | V | gate | b | a], behind those of an
+    attention it stands beside; its columns of the output projection follow that one's."""
+
+    hq: int
+    hk: int
+    dk: int
+    dv: int
+    taps: int
+    row0: int
+    col0: int
+
+    @property
+    def conv_rows(self) -> int:
+        return 2 * self.hk * self.dk + self.hq * self.dv
+
+    @property
+    def rows(self) -> int:
+        return self.conv_rows + self.hq * self.dv + _round8(2 * self.hq)
+
+    @property
+    def cols(self) -> int:
+        return self.hq * self.dv
 
 
 class RunnerWeights:
@@ -202,11 +231,15 @@ class RunnerWeights:
                 self.act_params[i] = xielu_coefficients(p[L + "act"])
             if ls.mixer != "attention":
                 self._mixer_weights(i, p, device, dev, heads)
-                self._dense_weights(i, p, dev)
+                self._ff_weights(i, p, dev)
                 continue
-            for n in ("q_norm", "k_norm"):
-                if L + n in p:
+            for n, cnt in (("q_norm", ls.num_heads), ("k_norm", ls.num_kv_heads)):
+                if L + n in p and s.qk_norm_kind(i) == "row":
+                    self.t[L + n] = dev(heads(p[L + n], cnt, ls.head_dim, kh.dk, 0, cnt))
+                elif L + n in p:
                     self.t[L + n] = dev(_pad(p[L + n], 0, kh.dk))
+            if ls.fixed_sink is not None:
+                self.t[L + "sink"] = torch.full((kh.hq,), ls.fixed_sink, dtype=torch.float32, device=device)
             if L + "sink" in p:
                 self.t[L + "sink"] = p[L + "sink"][rank * kh.hq:(rank + 1) * kh.hq].to(device=device, dtype=torch.float32).contiguous()
 
@@ -225,44 +258,56 @@ class RunnerWeights:
             self.t[L + "wo"] = dev(_pad(heads(wo, ls.num_heads, ls.v_head_dim, kh.dv, rank * kh.hq, kh.hq).t(), 0, H))
             if L + "bo" in p:
                 self.t[L + "bo"] = dev(p[L + "bo"] if rank == 0 else torch.zeros_like(p[L + "bo"]))
-            self._dense_weights(i, p, dev)
-            if L + "router" in p:
-                # experts: tensor-parallel inside each expert here; expert-parallel layouts are built by MoeRunner
-                m = ls.moe
-                self.t[L + "router"] = dev(_pad(p[L + "router"], 1, H))
-                if m.router_bias:
-                    self.t[L + "router_b"] = dev(p[L + "router_b"])
+            if kh.delta is not None:
+                self._beside_weights(i, p, device, dev, heads)
+            self._ff_weights(i, p, dev)
 
-                def up_rows(t, r, w):
-                    """This rank's rows of an up (or [gate; up]) matrix [.., rows, H], each half padded to 8."""
-                    halves = t.chunk(2, -2) if m.gated else (t,)
-                    n = halves[0].shape[-2] // w
-                    cut = [_pad(h[..., r * n:(r + 1) * n, :], h.dim() - 2, self._round(n)) for h in halves]
-                    return _pad(torch.cat(cut, -2), t.dim() - 1, H)
+    def _ff_weights(self, i: int, p, dev) -> None:
+        """Feed-forward of one layer, dense or a mixture."""
+        self._dense_weights(i, p, dev)
+        L, ls, H, rank, world = f"layers.{i}.", self.spec.layer(i), self.width, self.rank, self.world
+        if L + "router" not in p:
+            return
+        # experts: tensor-parallel inside each expert here; expert-parallel layouts are built by MoeRunner
+        m = ls.moe
+        self.t[L + "router"] = dev(_pad(p[L + "router"], 1, H))
+        if m.router_bias:
+            self.t[L + "router_b"] = dev(p[L + "router_b"])
+        if m.correction:
+            self.t[L + "correction"] = dev(p[L + "correction"])
+        if m.shared_gate:
+            self.t[L + "shared_sg"] = dev(_pad(p[L + "shared_sg"], 1, H)).view(-1)
 
-                def down_cols(t, r, w):
-                    n = t.shape[-1] // w
-                    return _pad(_pad(t[..., r * n:(r + 1) * n], t.dim() - 1, self._round(n)), t.dim() - 2, H)
+        def up_rows(t, r, w):
+            """This rank's rows of an up (or [gate; up]) matrix [.., rows, H], each half padded to 8."""
+            halves = t.chunk(2, -2) if m.gated else (t,)
+            n = halves[0].shape[-2] // w
+            cut = [_pad(h[..., r * n:(r + 1) * n, :], h.dim() - 2, self._round(n)) for h in halves]
+            return _pad(torch.cat(cut, -2), t.dim() - 1, H)
 
-                gu, dn = p[L + "experts_gate_up"], p[L + "experts_down"]
-                if self.ep:
-                    # expert parallel: whole experts [expert_lo, expert_lo + experts_local) live here
-                    lo, hi = self.expert_lo, self.expert_lo + self.experts_local
-                    self.t[L + "experts_gate_up"] = dev(up_rows(gu[lo:hi], 0, 1))
-                    self.t[L + "experts_down"] = dev(down_cols(dn[lo:hi], 0, 1))
-                else:
-                    self.t[L + "experts_gate_up"] = dev(up_rows(gu, rank, world))
-                    self.t[L + "experts_down"] = dev(down_cols(dn, rank, world))
-                if L + "shared_gate_up" in p:
-                    self.t[L + "shared_gate_up"] = dev(up_rows(p[L + "shared_gate_up"], rank, world))
-                    self.t[L + "shared_down"] = dev(down_cols(p[L + "shared_down"], rank, world))
+        def down_cols(t, r, w):
+            n = t.shape[-1] // w
+            return _pad(_pad(t[..., r * n:(r + 1) * n], t.dim() - 1, self._round(n)), t.dim() - 2, H)
+
+        gu, dn = p[L + "experts_gate_up"], p[L + "experts_down"]
+        if self.ep:
+            # expert parallel: whole experts [expert_lo, expert_lo + experts_local) live here
+            lo, hi = self.expert_lo, self.expert_lo + self.experts_local
+            self.t[L + "experts_gate_up"] = dev(up_rows(gu[lo:hi], 0, 1))
+            self.t[L + "experts_down"] = dev(down_cols(dn[lo:hi], 0, 1))
+        else:
+            self.t[L + "experts_gate_up"] = dev(up_rows(gu, rank, world))
+            self.t[L + "experts_down"] = dev(down_cols(dn, rank, world))
+        if L + "shared_gate_up" in p:
+            self.t[L + "shared_gate_up"] = dev(up_rows(p[L + "shared_gate_up"], rank, world))
+            self.t[L + "shared_down"] = dev(down_cols(p[L + "shared_down"], rank, world))
 
     def _dense_weights(self, i: int, p, dev) -> None:
         """Dense feed-forward of one layer."""
         L, rank, world = f"layers.{i}.", self.rank, self.world
         if L + "w_gate_up" in p:
-            g, u = p[L + "w_gate_up"].chunk(2, 0)
-            self.t[L + "w_gate_up"] = dev(torch.cat([shard_rows(g, rank, world), shard_rows(u, rank, world)], 0))
+            halves = [shard_rows(t, rank, world) for t in p[L + "w_gate_up"].chunk(2, 0)]
+            self.t[L + "w_gate_up"] = dev(_pad(torch.cat([_pad(t, 0, self._round(t.shape[0])) for t in halves], 0), 1, self.width))
         if L + "w_up" in p:
             up = shard_rows(p[L + "w_up"], rank, world)
             self.t[L + "w_up"] = dev(_pad(_pad(up, 0, self._round(up.shape[0])), 1, self.width))
@@ -274,8 +319,41 @@ class RunnerWeights:
             if L + "b_down" in p:
                 self.t[L + "b_down"] = dev(p[L + "b_down"] if rank == 0 else torch.zeros_like(p[L + "b_down"]))
 
+    def _beside_weights(self, i: int, p, device, dev, heads) -> None:
+        """The gated delta rule beside a layer's attention: one input and one output projection for both mixers.  The output
+        projection's result is multiplied by the first mixer's factor, so the second one's norm weight carries the ratio."""
+        L, ls, d = f"layers.{i}.", self.spec.layer(i), self.heads[i].delta
+        sa, sb = ls.scales
+        first = self.t.pop(L + "wqkv")
+        w, wo = self._delta_weights(L + "beside.", ls.beside, d, p, L, device, heads, sb / sa if sa else sb)
+        self.t[L + "w_in"] = torch.cat([first, dev(w)], 0)
+        if L + "bqkv" in self.t:
+            b = self.t.pop(L + "bqkv")
+            self.t[L + "b_in"] = _pad(b, 0, b.shape[0] + d.rows)
+        self.t[L + "wo"] = torch.cat([self.t[L + "wo"] * (1.0 if sa else 0.0), dev(wo)], 1).contiguous()
+
+    def _delta_weights(self, src: str, ls, d: "DeltaHeads", p, L: str, device, heads, factor: float):
+        """Parameters ``src`` of a gated delta rule into kernel layout; returns the rows of its input projection and its output
+        projection."""
+        t, H, n, g = self.t, self.width, ls.num_heads, ls.num_kv_heads
+
+        def f32(x):
+            return x.to(device=device, dtype=torch.float32).contiguous()
+
+        def qkv_rows(x):
+            q, k, v = x.split([ls.k_size, ls.k_size, ls.o_size])
+            return torch.cat([heads(q, g, ls.head_dim, d.dk, 0, g), heads(k, g, ls.head_dim, d.dk, 0, g),
+                              heads(v, n, ls.v_head_dim, d.dv, 0, n)])
+
+        t[L + "delta_conv"] = qkv_rows(p[src + "conv"]).t().to(device=device, dtype=self.dtype).contiguous()
+        t[L + "a_log"], t[L + "dt_bias"] = f32(p[src + "A_log"]), f32(p[src + "dt_bias"])
+        t[L + "o_norm"] = f32(_pad(p[src + "o_norm"].float() * factor, 0, d.dv))
+        ba = torch.cat([p[src + "w_b"], p[src + "w_a"]])
+        w = torch.cat([qkv_rows(p[src + "w_qkv"]), heads(p[src + "w_g"], n, ls.v_head_dim, d.dv, 0, n), _pad(ba, 0, _round8(2 * n))])
+        return _pad(w, 1, H), _pad(heads(p[src + "wo"].t(), n, ls.v_head_dim, d.dv, 0, n).t(), 0, H)
+
     def _mixer_weights(self, i: int, p, device, dev, heads) -> None:
-        """Latent attention or wkv parameters of one layer in kernel layout."""
+        """Latent attention, wkv or delta parameters of one layer in kernel layout."""
         L, ls, kh, H = f"layers.{i}.", self.spec.layer(i), self.heads[i], self.width
         n, t = ls.num_heads, self.t
 
@@ -285,6 +363,10 @@ class RunnerWeights:
         def head_cols(w, d, dp):                              # [H, heads * d] -> [width, heads * dp]
             return dev(_pad(heads(w.t(), n, d, dp, 0, n).t(), 0, H))
 
+        if ls.mixer == "delta":
+            w, wo = self._delta_weights(L, ls, kh.delta, p, L, device, heads, 1.0)
+            t[L + "w_in"], t[L + "wo"] = dev(w), dev(wo)
+            return
         if ls.mixer == "wkv":
             d, dp, rank = ls.head_dim, kh.dk, self._round(ls.decay_rank)
             t[L + "mu"] = dev(_pad(p[L + "mu"], 1, H))
@@ -328,7 +410,10 @@ class RunnerWeights:
             ls = spec.layer(i)
             if ls.mixer != "attention" or spec.norm_placement == "both":
                 if world > 1:
-                    raise UnsupportedOperation("latent attention, wkv layers and norms on both sides of a sublayer: one rank")
+                    raise UnsupportedOperation("latent attention, wkv and delta layers and norms on both sides of a sublayer: one rank")
+            if ls.mixer == "delta":
+                self.heads.append(KernelHeads(ls.num_heads, 0, 0, 8, 8, False, delta=self._delta_heads(ls, 0, 0)))
+                continue
             if ls.mixer == "wkv":
                 d = r8(ls.head_dim)
                 self.heads.append(KernelHeads(ls.num_heads, 0, 0, d, d, False))
@@ -343,12 +428,18 @@ class RunnerWeights:
             if ls.moe is not None and not self.ep and (ls.moe.intermediate_size % world or ls.moe.shared_width % world):
                 raise InvalidInput(f"layer {i}: expert widths not divisible by tensor parallel size {world}")
             hkv, kv_lo = self.kv_layout(ls.num_kv_heads, rank, world)
-            self.heads.append(KernelHeads(ls.num_heads // world, hkv, kv_lo, self._round(ls.head_dim), self._round(ls.v_head_dim),
-                                          ls.kv_from is None))
+            kh = KernelHeads(ls.num_heads // world, hkv, kv_lo, self._round(ls.head_dim), self._round(ls.v_head_dim), ls.kv_from is None)
+            if ls.beside is not None:
+                kh = dataclasses.replace(kh, delta=self._delta_heads(ls.beside, kh.qkv_rows, kh.hq * kh.dv))
+            self.heads.append(kh)
         # uniform specs: one layout for all layers
         self.hq = self.heads[0].hq if self.heads else spec.num_heads // world
         self.hkv, self.kv_lo = (self.heads[0].hkv, self.heads[0].kv_lo) if self.heads else \
             self.kv_layout(spec.num_kv_heads, rank, world)
+
+    @staticmethod
+    def _delta_heads(ls, row0: int, col0: int) -> "DeltaHeads":
+        return DeltaHeads(ls.num_heads, ls.num_kv_heads, _round8(ls.head_dim), _round8(ls.v_head_dim), ls.conv_taps, row0, col0)
 
     def kv_bytes_per_token(self) -> int:
         """Cache bytes that one token takes on this rank over all layers that own keys and values."""
@@ -373,6 +464,9 @@ class RunnerWeights:
                 out += [((i, n), (s.input_conv - 1, self.width)) for n in (("conv1", "conv2") if ls.mlp is not None else ("conv1",))]
             if ls.mixer == "wkv":
                 out += [((i, "shift"), (self.width,)), ((i, "wkv"), (kh.hq, kh.dk, kh.dv))]
+            d = kh.delta
+            if d is not None:
+                out += [((i, "delta_conv"), (d.taps - 1, d.conv_rows)), ((i, "delta"), (d.hq, d.dk, d.dv))]
         return out
 
     @staticmethod
@@ -505,6 +599,11 @@ class RunnerWeights:
                     self.t[L + "w_gate_up"] = torch.cat([self.t.pop(L + "w_up"), rnd(width, H)])
                 if s.act == "xielu":
                     self.act_params[i] = (0.8, 1.3)
+            d = kh.delta
+            if d is not None:
+                self.t[L + "delta_conv"] = rnd(d.taps, d.conv_rows) + 0.3
+                self.t[L + "a_log"], self.t[L + "dt_bias"] = zeros(d.hq).float(), zeros(d.hq).float() - 3.0
+                self.t[L + "o_norm"] = ones(d.dv).float()
             if ls.mixer == "wkv":
                 rank, C = self._round(ls.decay_rank or 64), kh.hq * kh.dk
                 self.t[L + "mu"] = torch.full_like(rnd(5, H), 0.5)
@@ -523,14 +622,24 @@ class RunnerWeights:
                     self.t[L + "w_ukv"] = torch.cat([self.t[L + "w_uk_t"].transpose(1, 2), self.t[L + "w_uv"]], 1).flatten(0, 1).contiguous()
                 self.t[L + "sink"], self.t[L + "wo"] = zeros(kh.hq).float(), rnd(H, kh.hq * kh.vdim)
                 continue
-            self.t[L + "wqkv"] = rnd(kh.qkv_rows, H)
-            self.t[L + "wo"] = rnd(H, kh.hq * kh.dv)
-            if s.qk_norm:
-                self.t[L + "q_norm"] = ones(kh.dk)
+            kind = s.qk_norm_kind(i)
+            if ls.mixer == "delta":
+                self.t[L + "w_in"], self.t[L + "wo"] = rnd(d.rows, H), rnd(H, d.cols)
+            elif d is not None:
+                self.t[L + "w_in"], self.t[L + "wo"] = rnd(kh.qkv_rows + d.rows, H), rnd(H, kh.hq * kh.dv + d.cols)
+                if s.has_qkv_bias(i):
+                    self.t[L + "b_in"] = zeros(kh.qkv_rows + d.rows)
+            else:
+                self.t[L + "wqkv"] = rnd(kh.qkv_rows, H)
+                self.t[L + "wo"] = rnd(H, kh.hq * kh.dv)
+                if s.has_qkv_bias(i):
+                    self.t[L + "bqkv"] = zeros(kh.qkv_rows)
+            if kind and ls.mixer == "attention":
+                self.t[L + "q_norm"] = ones(kh.dk * (kh.hq if kind == "row" else 1))
                 if kh.own_kv:
-                    self.t[L + "k_norm"] = ones(kh.dk)
-            if ls.sink:
-                self.t[L + "sink"] = zeros(kh.hq).float()
+                    self.t[L + "k_norm"] = ones(kh.dk * (kh.hkv if kind == "row" else 1))
+            if ls.sink or ls.fixed_sink is not None:
+                self.t[L + "sink"] = zeros(kh.hq).float() + (ls.fixed_sink or 0.0)
             m = ls.moe
             if m is None:
                 continue
@@ -538,6 +647,10 @@ class RunnerWeights:
             self.t[L + "router"] = rnd(m.num_experts, H)
             if m.router_bias:
                 self.t[L + "router_b"] = zeros(m.num_experts)
+            if m.correction:
+                self.t[L + "correction"] = zeros(m.num_experts)
+            if m.shared_gate:
+                self.t[L + "shared_sg"] = rnd(1, H).view(-1)
             self.t[L + "experts_gate_up"] = torch.stack([rnd(up, H) for _ in range(m.num_experts)])
             self.t[L + "experts_down"] = torch.stack([rnd(H, self._round(m.intermediate_size)) for _ in range(m.num_experts)])
             if m.num_shared_experts:
@@ -770,12 +883,12 @@ class GpuModelRunner:
             raise UnsupportedOperation("norms on sublayer outputs: 32-bit residual stream, no learned positions")
         if spec.norm_placement == "both" and (not spec.residual_fp32 or spec.norm != "rms" or spec.norm_bias or spec.pos == "learned"
                                               or spec.embed_norm or spec.residual_scale != 1.0 or spec.parallel_residual
-                                              or any(spec.layer_is_moe(i) for i in range(spec.num_layers))):
-            raise UnsupportedOperation("norms on both sides of a sublayer: RMS, 32-bit residual stream, dense feed-forwards")
-        if spec.norm_placement != "both" and (spec.input_conv or any(spec.layer(i).mixer != "attention" for i in range(spec.num_layers))):
-            raise UnsupportedOperation("input convolutions, latent attention and wkv layers: with norms on both sides of a sublayer")
-        if spec.norm_placement == "both" and any(spec.layer(i).mixer == "attention" for i in range(spec.num_layers)):
-            raise UnsupportedOperation("norms on both sides of a sublayer: latent attention and wkv layers")
+                                              or spec.mlp_bias or spec.o_bias
+                                              or (spec.input_conv and any(spec.layer_is_moe(i) for i in range(spec.num_layers)))):
+            raise UnsupportedOperation("norms on both sides of a sublayer: RMS, 32-bit residual stream, no mixtures behind convolutions")
+        if spec.norm_placement != "both" and (spec.input_conv or any(spec.layer(i).mixer != "attention" or spec.layer(i).beside is not None
+                                                                     for i in range(spec.num_layers))):
+            raise UnsupportedOperation("input convolutions, latent attention, wkv and delta layers: with norms on both sides of a sublayer")
         if spec.norm_placement == "input" and (spec.residual_fp32 or weights.dtype != torch.bfloat16):
             raise UnsupportedOperation("a 32-bit residual stream or 32-bit weights: only with norms on sublayer outputs")
         self.spec, self.w = spec, weights
@@ -974,22 +1087,23 @@ class GpuModelRunner:
                              self.v_cache[i] if own else None, num_q_heads=kh.hq, num_kv_heads=kh.hkv if own else 0,
                              head_dim=kh.dk, rotary_dim=ls.rotary_dim, pos_scale=s.rope_pos_scale,
                              interleaved=s.rope_interleaved, q_norm_w=t.get(L + "q_norm"), k_norm_w=t.get(L + "k_norm"),
-                             norm_eps=s.norm_eps, k_cache_only=own, **kw)
+                             norm_eps=s.norm_eps, k_cache_only=own, row_norm=s.qk_norm_kind(i) == "row", **kw)
         self.launches += 1
 
-    def _attention(self, i, qkv, lay, shared_prefix_len):
-        """qkv [T, q | k | v] already rotated and appended -> attention output [T, hq * Dv]."""
+    def _attention(self, i, qkv, lay, shared_prefix_len, out=None):
+        """qkv [T, q | k | v] already rotated and appended -> attention output [T, hq * Dv] (``out``: columns of a wider tensor)."""
         kh, ls = self.w.heads[i], self.layers[i]
         D, hq, hkv, window = kh.dk, kh.hq, kh.hkv, self.windows[i]
         sinks = self.w.t.get(f"layers.{i}.sink")
         T, Dp, P = lay["_T"], lay["_Dp"], lay["_P"]
         q = qkv[:, :hq * D].unflatten(1, (hq, D))          # strided view: row stride of the fused projection
-        out = torch.empty(T, hq, kh.dv, dtype=qkv.dtype, device=qkv.device)
+        flat = torch.empty(T, hq * kh.dv, dtype=qkv.dtype, device=qkv.device) if out is None else out
+        out = flat.unflatten(1, (hq, kh.dv))
         kc, vc = self.k_cache[i], self.v_cache[i]
         bt = self._view(lay, "block_tables").view(Dp + P, self.max_blocks_per_seq)
         scale = ls.scale if ls.scale is not None else 1.0 / math.sqrt(ls.head_dim)
         # the shared-prefix pass has no window, position bias or sink
-        plain = window == 0 and self.alibi is None and sinks is None and kh.dk == kh.dv and qkv.dtype == torch.bfloat16
+        plain = window == 0 and self.alibi is None and sinks is None and not ls.softcap and kh.dk == kh.dv and qkv.dtype == torch.bfloat16
         cascade = plain and shared_prefix_len >= 4 * self.block_size and Dp >= 8
         # prefill rows join the cascade when their chunks start after the shared prefix and share its blocks
         pp = cascade and P > 0 and lay.get("_pp", False)
@@ -1052,16 +1166,16 @@ class GpuModelRunner:
         elif Dp > 0:
             with self._prof("attn_decode"):
                 K.attn_decode(q[:Dp], kc, vc, bt[:Dp], self._view(lay, "seq_lens_d"), scale=scale, window=window,
-                              alibi_slopes=self.alibi, sinks=sinks, out=out[:Dp], scratch=self.attn_scratch,
+                              alibi_slopes=self.alibi, sinks=sinks, softcap=ls.softcap, out=out[:Dp], scratch=self.attn_scratch,
                               max_seq_len=self.max_model_len if self._graph_mode else int(self._max_len_d))
             self.launches += 1
         if P > 0 and not pp:
             with self._prof("attn_prefill"):
                 K.attn_prefill(q[Dp:], kc, vc, bt[Dp:], self._view(lay, "seq_lens_p"), self._view(lay, "q_start"),
                                lay["_max_q"], scale=scale, causal=True, window=window, alibi_slopes=self.alibi,
-                               sinks=sinks, out=out[Dp:])
+                               sinks=sinks, softcap=ls.softcap, out=out[Dp:])
             self.launches += 1
-        return out.view(T, hq * kh.dv)
+        return flat
 
     def _side_stream(self):
         if self._side is None:
@@ -1137,7 +1251,7 @@ class GpuModelRunner:
         if s.norm_placement == "output":
             return self._forward_tokens_output_norm(lay, shared_prefix_len)
         if s.norm_placement == "both":
-            return self._forward_tokens_both_norms(lay)
+            return self._forward_tokens_both_norms(lay, shared_prefix_len)
         ids = self._view(lay, "token_ids")
         pos = self._view(lay, "positions")
         slots = self._view(lay, "slot_mapping")
@@ -1209,31 +1323,70 @@ class GpuModelRunner:
                 h = self._residual_norm(x, y, L + "ln2")
         return x
 
-    def _forward_tokens_both_norms(self, lay) -> torch.Tensor:
+    def _forward_tokens_both_norms(self, lay, shared_prefix_len: int) -> torch.Tensor:
         """Layers of the form ``x += norm_b(f(conv(norm(x))))`` around a 32-bit residual stream.  Adding a sublayer's normed
-        output, the next norm, its convolution over time and (in front of a recurrent mixer) the token-shift mixes are one
-        kernel; what it needs from earlier steps is in the sequences' state rows."""
+        output (for a mixture-of-experts also its weighted sum), the next norm, its convolution over time and (in front of a wkv
+        mixer) the token-shift mixes are one kernel; what it needs from earlier steps is in the sequences' state rows.  The last
+        sublayer's output is added by the final norm, for the rows that are asked for."""
         s, t = self.spec, self.w.t
         pos, slots = self._view(lay, "positions"), self._view(lay, "slot_mapping")
         parts = self._portions(lay)
         x, _ = K.embed_residual(self._view(lay, "token_ids"), t["embed"], scale=s.embed_scale)
         self.launches += 1
-        y = y_name = None
+        y: dict = {}                                         # the sublayer output that has not been added yet
         for i, ls in enumerate(self.layers):
             L = f"layers.{i}."
-            x, h = self._sublayer_in(i, 1, x, parts, y, y_name)
+            x, h = self._sublayer_in(i, 1, x, parts, y)
+            scale = 1.0
             if ls.mixer == "wkv":
                 a = self._wkv(i, h, parts)
-            else:
+            elif ls.mixer == "latent":
                 a = self._latent_attention(i, h, pos, slots, lay)
-            y, y_name = self._gemm(a, t[L + "wo"]), L + "ln1b"
-            if ls.mlp is not None:
-                x, h = self._sublayer_in(i, 2, x, parts, y, y_name)
+            else:
+                a, scale = self._attention_and_delta(i, h, pos, slots, lay, parts, shared_prefix_len)
+            y = dict(y=self._gemm(a, t[L + "wo"], out_scale=scale), y_weight=t[L + "ln1b.w"])
+            if ls.mlp is None:
+                continue
+            x, h = self._sublayer_in(i, 2, x, parts, y)
+            y = dict(y_weight=t[L + "ln2b.w"])
+            if ls.mlp == "moe":
+                from .moe_runner import moe_branch
+
+                y["y"], y["experts"], y["routing"] = moe_branch(self, i, h, router_x=h)
+            elif s.mlp == "gated":
+                w = t[L + "w_gate_up"]
+                y["y"] = self._gemm(self._gemm(h, w, dual_rows=w.shape[0] // 2, act=s.act), t[L + "w_down"])
+            else:
                 up = self._gemm(h, t[L + "w_up"], act=s.act, act_params=self.w.act_params.get(i))
-                y, y_name = self._gemm(up, t[L + "w_down"]), L + "ln2b"
-        if y is not None:
-            self._residual_norm(x, y, y_name)
+                y["y"] = self._gemm(up, t[L + "w_down"])
+        self._last_y = y
         return x
+
+    def _attention_and_delta(self, i, h, pos, slots, lay, parts, shared_prefix_len):
+        """Attention, a gated delta rule, or both side by side on one input projection: (rows for the output projection, the
+        factor on its result)."""
+        t, L, ls, kh = self.w.t, f"layers.{i}.", self.layers[i], self.w.heads[i]
+        d = kh.delta
+        if d is None:
+            qkv = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
+            self._rope_append(i, qkv, pos, slots)
+            return self._attention(i, qkv, lay, shared_prefix_len), 1.0
+        proj = self._gemm(h, t[L + "w_in"], bias=t.get(L + "b_in"))
+        out = torch.empty(h.shape[0], d.col0 + d.cols, dtype=proj.dtype, device=proj.device)
+        mx = ls
+        if ls.beside is not None:
+            mx = ls.beside
+            qkv = proj[:, :d.row0]
+            self._rope_append(i, qkv, pos, slots)
+            self._attention(i, qkv, lay, shared_prefix_len, out=out[:, :d.col0])
+        with self._prof("delta"):
+            K.delta_mixer(proj, d.row0, t[L + "delta_conv"], t[L + "a_log"], t[L + "dt_bias"], t[L + "o_norm"],
+                          self.state[(i, "delta_conv")], self.state[(i, "delta")], parts, kv_heads=d.hk, eps=self.spec.norm_eps,
+                          dk_real=mx.head_dim, dv_real=mx.v_head_dim, out=out[:, d.col0:])
+        self.launches += sum(1 if p.q_start is None else 3 for p in parts)
+        if ls.beside is None:
+            return out, 1.0
+        return out, ls.scales[0] or 1.0
 
     def _portions(self, lay) -> List["K.Portions"]:
         """The step's rows as portions of sequences: one-token rows of decoding sequences, then pieces of prompts."""
@@ -1249,16 +1402,16 @@ class GpuModelRunner:
             out.append(K.Portions(Dp, T - Dp, P, lay["_max_q"], self._view(lay, "q_start"), cut(si, Dp, Dp + P), cut(so, Dp, Dp + P)))
         return out
 
-    def _sublayer_in(self, i, which, x, parts, y, y_name):
+    def _sublayer_in(self, i, which, x, parts, y: dict):
+        """``y``: the previous sublayer's output and norm weight, as keyword arguments of ``cuda_ops.sublayer_in``."""
         s, t, L = self.spec, self.w.t, f"layers.{i}."
         conv = f"conv{which}"
         mix = which == 1 and self.layers[i].mixer == "wkv"
-        self.launches += len(parts)
+        self.launches += len(parts) if s.input_conv or mix else 1
         with self._prof("sublayer_in"):
-            return K.sublayer_in(x, parts, t[f"{L}ln{which}.w"], eps=s.norm_eps, y=y, y_weight=None if y is None else t[y_name + ".w"],
-                                 conv=t.get(L + conv), conv_state=self.state.get((i, conv)), mu=t[L + "mu"] if mix else None,
-                                 shift_state=self.state[(i, "shift")] if mix else None, width=s.hidden_size,
-                                 offset_one=s.norm_weight_offset_one)
+            return K.sublayer_in(x, parts, t[f"{L}ln{which}.w"], eps=s.norm_eps, conv=t.get(L + conv), conv_state=self.state.get((i, conv)),
+                                 mu=t[L + "mu"] if mix else None, shift_state=self.state[(i, "shift")] if mix else None,
+                                 width=s.hidden_size, offset_one=s.norm_weight_offset_one, **y)
 
     def _wkv(self, i, h, parts):
         """``h`` [5, T, width]: the mixes for receptance, key, value, gate and decay."""
@@ -1341,7 +1494,7 @@ class GpuModelRunner:
 
     def _rotation(self, ls):
         """(device table of a layer's rotation frequencies, gain on cosine and sine)."""
-        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3, ls.rope_yarn)
+        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3, ls.rope_yarn, ls.rope_linear)
         if key not in self._inv_freq:
             self._inv_freq[key] = rope_inv_freq(*key).to(self.device)
         return self._inv_freq[key], rope_gain(ls.rope_yarn)
@@ -1482,6 +1635,11 @@ class GpuModelRunner:
         """Final-normed rows of the step whose logits are asked for."""
         s, t = self.spec, self.w.t
         rows = self._view(lay, "sample_rows")
+        if s.norm_placement == "both":
+            self.launches += 1
+            with self._prof("norm"):
+                return K.sublayer_in(x, (), t["final_norm.w"], eps=s.norm_eps, rows=rows, width=s.hidden_size,
+                                     offset_one=s.norm_weight_offset_one, **self._last_y)
         if s.residual_fp32:
             self.launches += 1
             with self._prof("norm"):

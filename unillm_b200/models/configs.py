@@ -1,4 +1,4 @@
-"""Configuration classes of all architectures: the reference's 47, Gekapel and Nipulorn.
+"""Configuration classes of all architectures: the reference's 47, Bakasun, Gekapel and Nipulorn.
 
 Field names and defaults follow the reference's ``model_config!`` blocks one for one
 (``crates/runtime/src/models_v2/<family>.rs``, e.g. ``llama.rs:20-38``, ``mixtral.rs:16-38``), so a
@@ -54,6 +54,29 @@ class BaichuanConfig:
     use_alibi: bool = True
     model_max_length: int = 4096
     z_loss_weight: float = 0.0
+
+
+@model_config
+class BakasunConfig:
+    """Bakasun: every layer is described on its own.  ``layers[i]`` holds ``type`` ("attention", or "parallel": attention and a
+    gated delta rule side by side), ``mixer`` (for "parallel": ``left``, ``right``, ``left_scale``, ``right_scale``) and
+    ``mlp`` (kind "dense" with ``ff``, kind "moe" with ``router``, ``expert`` and ``shared``, or null)."""
+
+    vocab_size: int = 32000
+    hidden_size: int = 2048
+    num_hidden_layers: int = 0
+    norm_eps: float = 1e-6
+    layers: List[Any] = []
+    max_position_embeddings: int = 131072
+    initializer_range: float = 0.02
+
+    @classmethod
+    def from_hf_config(cls, d):
+        if "layers" not in d or "width" not in d:
+            return super(BakasunConfig, cls).from_hf_config(d)
+        kw = {k: d[k] for k in ("max_position_embeddings", "initializer_range") if k in d}
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], num_hidden_layers=len(d["layers"]), norm_eps=d["norm"]["eps"],
+                   layers=list(d["layers"]), **kw)
 
 
 @model_config

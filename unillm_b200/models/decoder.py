@@ -91,17 +91,20 @@ class DecoderModel(Model):
                 shp.update({L + n: t for n, t in MX.mixer_shapes(ls, H).items()})
             else:
                 shp[L + "wqkv"] = (ls.qkv_size, H)
-                if s.qkv_bias:
+                if s.has_qkv_bias(i):
                     shp[L + "bqkv"] = (ls.qkv_size,)
-                if s.qk_norm:
-                    shp[L + "q_norm"] = (ls.head_dim,)
+                kind = s.qk_norm_kind(i)
+                if kind:
+                    shp[L + "q_norm"] = (ls.q_size if kind == "row" else ls.head_dim,)
                     if ls.kv_from is None:
-                        shp[L + "k_norm"] = (ls.head_dim,)
+                        shp[L + "k_norm"] = (ls.k_size if kind == "row" else ls.head_dim,)
                 if ls.sink:
                     shp[L + "sink"] = (ls.num_heads,)
                 shp[L + "wo"] = (H, ls.o_size)
                 if s.o_bias:
                     shp[L + "bo"] = (H,)
+            if ls.beside is not None:
+                shp.update({L + "beside." + n: t for n, t in MX.mixer_shapes(ls.beside, H).items()})
             moe = ls.mlp == "moe"
             if ls.mlp == "dense" or (moe and ls.moe.dense_parallel):
                 I = s.layer_intermediate(i)
@@ -121,12 +124,16 @@ class DecoderModel(Model):
                 shp[L + "router"] = (m.num_experts, H)
                 if m.router_bias:
                     shp[L + "router_b"] = (m.num_experts,)
+                if m.correction:
+                    shp[L + "correction"] = (m.num_experts,)
                 shp[L + "experts_gate_up"] = (m.num_experts, (2 if m.gated else 1) * m.intermediate_size, H)
                 shp[L + "experts_down"] = (m.num_experts, H, m.intermediate_size)
                 if m.num_shared_experts:
                     Is = m.shared_width
                     shp[L + "shared_gate_up"] = ((2 if m.gated else 1) * Is, H)
                     shp[L + "shared_down"] = (H, Is)
+                    if m.shared_gate:
+                        shp[L + "shared_sg"] = (1, H)
         if s.final_norm:
             shp["final_norm.w"] = (H,)
             if s.norm_bias:
@@ -145,11 +152,13 @@ class DecoderModel(Model):
             is_norm_w = name.endswith((".w", "q_norm", "k_norm")) and len(shape) == 1
             if init == "zeros":
                 t = torch.zeros(shape, dtype=dtype)
+            elif name.endswith(("q_norm", "k_norm")) and self.spec.layers is not None:
+                t = torch.ones(shape, dtype=dtype)
             elif is_norm_w:
                 t = torch.zeros(shape, dtype=dtype) if self.spec.norm_weight_offset_one else torch.ones(shape, dtype=dtype)
             elif name.endswith(("q_a_norm", "kv_a_norm", "o_norm")):         # weights that are not stored around zero
                 t = torch.ones(shape, dtype=dtype)
-            elif name.endswith((".b", "bqkv", "bo", "b_up", "b_down", "lm_head_bias", "router_b", "sink")):
+            elif name.endswith((".b", "bqkv", "bo", "b_up", "b_down", "lm_head_bias", "router_b", "sink", "correction", "A_log", "dt_bias")):
                 t = torch.zeros(shape, dtype=dtype)
             else:
                 t = (torch.randn(shape, generator=g, dtype=torch.float32) * std).to(dtype)
@@ -187,14 +196,21 @@ class DecoderModel(Model):
                 layers[i] = dataclasses.replace(ls, decay_rank=t.shape[0])
         return dataclasses.replace(s, layers=tuple(layers))
 
-    def _load_mixer(self, weights: ModelWeights, i: int, pre, out: Dict[str, torch.Tensor]) -> None:
-        """Parameters of a layer's latent or wkv mixer, each put together from the tensors the scheme names."""
-        ls = self.spec.layer(i)
+    def _side(self, names, i: int, second: bool = False):
+        """A mixer's tensor names in layer ``i``: another prefix where two mixers stand side by side."""
+        if self.spec.layer(i).beside is None or self.scheme.sides is None:
+            return tuple(names)
+        old, new = self.scheme.sides[0], self.scheme.sides[2 if second else 1]
+        return tuple(new + n[len(old):] if n.startswith(old) else n for n in names)
+
+    def _load_mixer(self, weights: ModelWeights, i: int, ls: LayerSpec, pre, out: Dict[str, torch.Tensor], second: bool = False) -> None:
+        """Parameters of a layer's mixer that is not plain attention, each put together from the tensors the scheme names."""
         for name, shape in MX.mixer_shapes(ls, self.spec.hidden_size).items():
-            parts = [self._find(weights, pre, (n,)) for n in self.scheme.mixers[ls.mixer][name]]
+            names = self._side(self.scheme.mixers[ls.mixer][name], i, second)
+            parts = [self._find(weights, pre, (n,)) for n in names]
             if any(t is None for t in parts):
-                raise LoadingError(f"{type(self).__name__}: missing weight layer {i} {name} {self.scheme.mixers[ls.mixer][name]}")
-            out[f"layers.{i}.{name}"] = MX.join_parts(parts, shape)
+                raise LoadingError(f"{type(self).__name__}: missing weight layer {i} {name} {names}")
+            out[f"layers.{i}.{'beside.' if second else ''}{name}"] = MX.join_parts(parts, shape)
 
     def _load(self, weights: ModelWeights, dtype=None, device=None):
         self.spec = self._complete_spec(weights)
@@ -250,9 +266,11 @@ class DecoderModel(Model):
                     out[L + n] = need(self._find(weights, pre, names), f"layer {i} {n}")
             # ---- mixer ----
             if ls.mixer != "attention":
-                self._load_mixer(weights, i, pre, out)
+                self._load_mixer(weights, i, ls, pre, out)
             else:
                 self._load_attention(weights, i, pre, out, T, need, deq)
+            if ls.beside is not None:
+                self._load_mixer(weights, i, ls.beside, pre, out, second=True)
             # ---- MLP ----
             moe = ls.mlp == "moe"
             if ls.mlp == "dense" or (moe and ls.moe.dense_parallel):
@@ -283,6 +301,8 @@ class DecoderModel(Model):
                 out[L + "router"] = need(self._find(weights, pre, k.router), f"layer {i} router")
                 if m.router_bias:
                     out[L + "router_b"] = need(self._find(weights, pre, k.router, ".bias"), f"layer {i} router bias")
+                if m.correction:
+                    out[L + "correction"] = need(self._find(weights, pre, k.correction), f"layer {i} router correction")
                 gus, dns = [], []
                 for e in range(m.num_experts):
                     epre = tuple(p + x.format(e=e) for p in pre for x in k.expert)
@@ -300,6 +320,8 @@ class DecoderModel(Model):
                         g = torch.cat([g, need(self._find(weights, pre, k.shared_up), "shared up")], 0)
                     out[L + "shared_gate_up"] = g
                     out[L + "shared_down"] = need(self._find(weights, pre, k.shared_down), "shared down")
+                    if m.shared_gate:
+                        out[L + "shared_sg"] = need(self._find(weights, pre, k.shared_sg), f"layer {i} gate of the shared expert")
         if s.final_norm:
             out["final_norm.w"] = need(self._find(weights, root, k.final_norm), "final norm")
             if s.norm_bias:
@@ -326,18 +348,19 @@ class DecoderModel(Model):
         """Projections, head norms and sinks of one layer's attention."""
         s, k, ls = self.spec, self.scheme, self.spec.layer(i)
         L = f"layers.{i}."
+        nq, nk, nv, no, nqn, nkn, nsink = (self._side(n, i) for n in (k.q, k.k, k.v, k.o, k.q_norm, k.k_norm, k.sink))
         packed = T(self._find(weights, pre, k.qkv)) if k.qkv else None
         pb = self._find(weights, pre, k.qkv, ".bias") if k.qkv else None
         if packed is not None:
             out[L + "wqkv"], bq = self._unpack_qkv(packed, pb)
         else:
-            q = T(self._find(weights, pre, k.q))
-            kk = T(self._find(weights, pre, k.k))
-            v = T(self._find(weights, pre, k.v))
+            q = T(self._find(weights, pre, nq))
+            kk = T(self._find(weights, pre, nk))
+            v = T(self._find(weights, pre, nv))
             if q is None:
-                names = [p + n + ".weight" for p in pre for n in k.q]
-                q, kk, v = deq(names), deq([n.replace(k.q[0], k.k[0]) for n in names]), \
-                    deq([n.replace(k.q[0], k.v[0]) for n in names])
+                names = [p + n + ".weight" for p in pre for n in nq]
+                q, kk, v = deq(names), deq([n.replace(nq[0], nk[0]) for n in names]), \
+                    deq([n.replace(nq[0], nv[0]) for n in names])
             need(q, f"layer {i} q_proj")
             if ls.kv_from is None:
                 need(kk, f"layer {i} k_proj"), need(v, f"layer {i} v_proj")
@@ -345,26 +368,26 @@ class DecoderModel(Model):
             else:
                 out[L + "wqkv"] = q
             bq = None
-            qb = self._find(weights, pre, k.q, ".bias")
+            qb = self._find(weights, pre, nq, ".bias")
             if qb is not None:
-                kb = self._find(weights, pre, k.k, ".bias")
-                vb = self._find(weights, pre, k.v, ".bias")
-                bq = torch.cat([qb, kb if kb is not None else torch.zeros(s.kv_size),
-                                vb if vb is not None else torch.zeros(s.kv_size)])
-        if s.qkv_bias:
-            out[L + "bqkv"] = bq if bq is not None else torch.zeros(s.q_size + 2 * s.kv_size)
-        if s.qk_norm:
-            out[L + "q_norm"] = need(self._find(weights, pre, k.q_norm), "q_norm")
+                kb = self._find(weights, pre, nk, ".bias")
+                vb = self._find(weights, pre, nv, ".bias")
+                bq = torch.cat([qb, kb if kb is not None else torch.zeros(ls.k_size),
+                                vb if vb is not None else torch.zeros(ls.v_size)])
+        if s.has_qkv_bias(i):
+            out[L + "bqkv"] = bq if bq is not None else torch.zeros(ls.qkv_size)
+        if s.qk_norm_kind(i):
+            out[L + "q_norm"] = need(self._find(weights, pre, nqn), "q_norm")
             if ls.kv_from is None:
-                out[L + "k_norm"] = need(self._find(weights, pre, k.k_norm), "k_norm")
+                out[L + "k_norm"] = need(self._find(weights, pre, nkn), "k_norm")
         if ls.sink:
-            out[L + "sink"] = need(self._find(weights, pre, k.sink, ""), f"layer {i} sinks")
-        wo = T(self._find(weights, pre, k.o))
+            out[L + "sink"] = need(self._find(weights, pre, nsink, ""), f"layer {i} sinks")
+        wo = T(self._find(weights, pre, no))
         if wo is None:
-            wo = deq([p + n + ".weight" for p in pre for n in k.o])
+            wo = deq([p + n + ".weight" for p in pre for n in no])
         out[L + "wo"] = need(wo, f"layer {i} o_proj")
         if s.o_bias:
-            b = self._find(weights, pre, k.o, ".bias")
+            b = self._find(weights, pre, no, ".bias")
             out[L + "bo"] = b if b is not None else torch.zeros(s.hidden_size)
 
     def _unpack_qkv(self, w: torch.Tensor, b: Optional[torch.Tensor]):
@@ -436,34 +459,37 @@ class DecoderModel(Model):
                                      ("act", k.act, WS)):
                 if L + n in self.p:
                     out[pre + names[0] + suffix] = self.p[L + n]
-            if ls.mixer != "attention":
-                for n in MX.mixer_shapes(ls, s.hidden_size):
-                    names = k.mixers[ls.mixer][n]
-                    for name, t in zip(names, MX.split_parts(self.p[L + n], ls, n, len(names))):
+            side = lambda names: self._side(names, i)[0]
+            for mx, at in zip(ls.mixers, ("", "beside.")):
+                if mx.mixer == "attention":
+                    continue
+                for n in MX.mixer_shapes(mx, s.hidden_size):
+                    names = self._side(k.mixers[mx.mixer][n], i, bool(at))
+                    for name, t in zip(names, MX.split_parts(self.p[L + at + n], mx, n, len(names))):
                         out[pre + name + WS] = t
-            else:
+            if ls.mixer == "attention":
                 wqkv = self.p[L + "wqkv"]
                 if k.qkv:
                     out[pre + k.qkv[0] + WS] = T(self._pack_qkv(wqkv))
                     if s.qkv_bias:
                         out[pre + k.qkv[0] + BS] = self._pack_qkv(self.p[L + "bqkv"][:, None])[:, 0]
                 elif ls.kv_from is not None:
-                    out[pre + k.q[0] + WS] = T(wqkv)
+                    out[pre + side(k.q) + WS] = T(wqkv)
                 else:
                     q, kk, v = wqkv.split([ls.q_size, ls.k_size, ls.v_size])
-                    out[pre + k.q[0] + WS], out[pre + k.k[0] + WS], out[pre + k.v[0] + WS] = T(q), T(kk), T(v)
-                    if s.qkv_bias:
-                        qb, kb, vb = self.p[L + "bqkv"].split([s.q_size, s.kv_size, s.kv_size])
-                        out[pre + k.q[0] + BS], out[pre + k.k[0] + BS], out[pre + k.v[0] + BS] = qb, kb, vb
-                if s.qk_norm:
-                    out[pre + k.q_norm[0] + WS] = self.p[L + "q_norm"]
+                    out[pre + side(k.q) + WS], out[pre + side(k.k) + WS], out[pre + side(k.v) + WS] = T(q), T(kk), T(v)
+                    if s.has_qkv_bias(i):
+                        qb, kb, vb = self.p[L + "bqkv"].split([ls.q_size, ls.k_size, ls.v_size])
+                        out[pre + side(k.q) + BS], out[pre + side(k.k) + BS], out[pre + side(k.v) + BS] = qb, kb, vb
+                if s.qk_norm_kind(i):
+                    out[pre + side(k.q_norm) + WS] = self.p[L + "q_norm"]
                     if ls.kv_from is None:
-                        out[pre + k.k_norm[0] + WS] = self.p[L + "k_norm"]
+                        out[pre + side(k.k_norm) + WS] = self.p[L + "k_norm"]
                 if ls.sink:
-                    out[pre + k.sink[0]] = self.p[L + "sink"]
-                out[pre + k.o[0] + WS] = T(self.p[L + "wo"])
+                    out[pre + side(k.sink)] = self.p[L + "sink"]
+                out[pre + side(k.o) + WS] = T(self.p[L + "wo"])
                 if s.o_bias:
-                    out[pre + k.o[0] + BS] = self.p[L + "bo"]
+                    out[pre + side(k.o) + BS] = self.p[L + "bo"]
             if L + "w_gate_up" in self.p:
                 if k.gate_up:
                     out[pre + k.gate_up[0] + WS] = T(self.p[L + "w_gate_up"])
@@ -483,6 +509,8 @@ class DecoderModel(Model):
                 out[pre + k.router[0] + WS] = self.p[L + "router"]
                 if m.router_bias:
                     out[pre + k.router[0] + BS] = self.p[L + "router_b"]
+                if m.correction:
+                    out[pre + k.correction[0] + WS] = self.p[L + "correction"]
                 for e in range(m.num_experts):
                     ep = pre + k.expert[0].format(e=e)
                     gu = self.p[L + "experts_gate_up"][e]
@@ -499,6 +527,8 @@ class DecoderModel(Model):
                     else:
                         out[pre + k.shared_gate[0] + WS] = self.p[L + "shared_gate_up"]
                     out[pre + k.shared_down[0] + WS] = self.p[L + "shared_down"]
+                    if m.shared_gate:
+                        out[pre + k.shared_sg[0] + WS] = self.p[L + "shared_sg"]
         if s.final_norm:
             out[k.final_norm[0] + WS] = self.p["final_norm.w"]
             if s.norm_bias:
@@ -540,7 +570,7 @@ class DecoderModel(Model):
         """Tables of one rotation; layers with the same rotation share them."""
         s = self.spec
         ls = ls or s.layer(0)
-        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3, ls.rope_yarn)
+        key = (ls.rotary_dim, ls.rope_theta, ls.rope_llama3, ls.rope_yarn, ls.rope_linear)
         if self._rope is None:
             self._rope = {}
         c = self._rope.get(key)
@@ -548,7 +578,7 @@ class DecoderModel(Model):
             n = max(need_len, min(s.max_position_embeddings, 8192))
             c = self._rope[key] = RoPECache(ls.head_dim, n, ls.rope_theta, rotary_dim=ls.rotary_dim,
                                             position_scale=s.rope_pos_scale, llama3=ls.rope_llama3, yarn=ls.rope_yarn,
-                                            device=self.device)
+                                            linear=ls.rope_linear, device=self.device)
         return c
 
     def _project_qkv(self, i: int, h: torch.Tensor):
@@ -559,14 +589,19 @@ class DecoderModel(Model):
         qkv = ops_fn.linear(h, self.p[L + "wqkv"], self.p.get(L + "bqkv"))
         lead = h.shape[:-1]
         k = v = None
+        kind = s.qk_norm_kind(i)
         if ls.kv_from is None:
             q, k, v = qkv.split([ls.q_size, ls.k_size, ls.v_size], dim=-1)
+            if kind == "row":
+                k = ops_fn.rms_norm(k.contiguous(), self.p[L + "k_norm"], s.norm_eps)
             k = k.reshape(*lead, ls.num_kv_heads, ls.head_dim)
             v = v.reshape(*lead, ls.num_kv_heads, ls.v_head_dim)
         else:
             q = qkv
+        if kind == "row":
+            q = ops_fn.rms_norm(q.contiguous(), self.p[L + "q_norm"], s.norm_eps)
         q = q.reshape(*lead, ls.num_heads, ls.head_dim)
-        if s.qk_norm:
+        if kind == "head":
             q = ops_fn.rms_norm(q, self.p[L + "q_norm"], s.norm_eps)
             if k is not None:
                 k = ops_fn.rms_norm(k, self.p[L + "k_norm"], s.norm_eps)
@@ -587,7 +622,21 @@ class DecoderModel(Model):
         ls, L = self.spec.layer(i), f"layers.{i}."
         if ls.mixer == "wkv":
             return ops_fn.linear(MX.wkv(self.p, L, ls, h, st, self.spec.norm_eps), self.p[L + "wo"])
-        return self._attention(i, h, past, cache, shared)
+        if ls.mixer == "delta":
+            return self._delta(i, h, st)
+        a = self._attention(i, h, past, cache, shared)
+        return a if ls.beside is None else self._side_by_side(i, a, self._delta(i, h, st))
+
+    def _delta(self, i: int, h: torch.Tensor, st: dict) -> torch.Tensor:
+        """Gated delta rule of layer ``i`` (its only mixer, or the one beside another) with its output projection."""
+        ls, L = self.spec.layer(i), f"layers.{i}."
+        if ls.beside is not None:
+            ls, L = ls.beside, L + "beside."
+        return ops_fn.linear(MX.delta(self.p, L, ls, h, st, self.spec.norm_eps), self.p[L + "wo"])
+
+    def _side_by_side(self, i: int, a: torch.Tensor, b: torch.Tensor) -> torch.Tensor:
+        sa, sb = self.spec.layer(i).scales
+        return (sa * _f(a) + sb * _f(b)).to(a.dtype)
 
     def _attend(self, i: int, q, k, v, bias):
         """q [B, Hq, T, Dk], k / v [B, Hkv, S, ...] in fp32, additive ``bias`` [T, S] or [Hq, T, S] -> [B, Hq, T, Dv]."""
@@ -596,10 +645,18 @@ class DecoderModel(Model):
         if g > 1:
             k, v = k.repeat_interleave(g, dim=1), v.repeat_interleave(g, dim=1)
         scale = ls.scale if ls.scale is not None else 1.0 / math.sqrt(ls.head_dim)
-        if not ls.sink:
+        if not ls.sink and ls.fixed_sink is None and not ls.softcap:
             return F.scaled_dot_product_attention(q, k, v, attn_mask=bias, scale=scale)
-        sc = torch.matmul(q, k.transpose(-1, -2)) * scale + bias
-        sink = self.p[f"layers.{i}.sink"].to(sc).reshape(-1, 1, 1).expand(*sc.shape[:-1], 1)
+        sc = torch.matmul(q, k.transpose(-1, -2)) * scale
+        if ls.softcap:
+            sc = ls.softcap * torch.tanh(sc / ls.softcap)
+        sc = sc + bias
+        if ls.sink:
+            sink = self.p[f"layers.{i}.sink"].to(sc).reshape(-1, 1, 1).expand(*sc.shape[:-1], 1)
+        elif ls.fixed_sink is not None:
+            sink = torch.full((*sc.shape[:-1], 1), ls.fixed_sink, dtype=sc.dtype, device=sc.device)
+        else:
+            return torch.matmul(torch.softmax(sc, dim=-1), v)
         # the sink is one more column of the softmax that has no value
         p = torch.softmax(torch.cat([sc, sink], dim=-1), dim=-1)[..., :-1]
         return torch.matmul(p, v)
@@ -666,7 +723,18 @@ class DecoderModel(Model):
         x2 = x.reshape(-1, shape[-1])
         rb = self.p.get(L + "router_b")
         logits = F.linear(_f(x2), _f(self.p[L + "router"]), None if rb is None else _f(rb))
-        if m.normalize_topk:
+        if m.correction or m.groups > 1:
+            sc = torch.softmax(logits, dim=-1)
+            choice = sc + _f(self.p[L + "correction"]) if m.correction else sc
+            if m.keep_groups < m.groups:
+                best = choice.reshape(-1, m.groups, m.num_experts // m.groups).amax(-1).topk(m.keep_groups, dim=-1).indices
+                shut = torch.ones(choice.shape[0], m.groups, dtype=torch.bool, device=x.device).scatter_(1, best, False)
+                choice = choice.masked_fill(shut.repeat_interleave(m.num_experts // m.groups, dim=1), float("-inf"))
+            idx = choice.topk(m.top_k, dim=-1).indices
+            w = sc.gather(1, idx)
+            if m.normalize_topk:
+                w = w / (w.sum(-1, keepdim=True) + 1e-20)
+        elif m.normalize_topk:
             v, idx = torch.topk(logits, m.top_k, dim=-1)
             w = torch.softmax(v, dim=-1)
         else:
@@ -684,8 +752,11 @@ class DecoderModel(Model):
             out.index_add_(0, tok, _f(y) * w[tok, slot].unsqueeze(-1))
         if m.num_shared_experts:
             w = self.p[L + "shared_gate_up"]
-            out = out + _f(self._dense_mlp(x2, w_gate_up=w if m.gated else None, w_up=None if m.gated else w,
-                                           w_down=self.p[L + "shared_down"], act=m.act))
+            y = _f(self._dense_mlp(x2, w_gate_up=w if m.gated else None, w_up=None if m.gated else w,
+                                   w_down=self.p[L + "shared_down"], act=m.act))
+            if m.shared_gate:
+                y = y * torch.sigmoid(F.linear(_f(x2), _f(self.p[L + "shared_sg"])))
+            out = out + y
         return out.to(x.dtype).reshape(shape)
 
     def _mlp(self, i: int, x: torch.Tensor) -> torch.Tensor:

@@ -552,6 +552,83 @@ class NipulornModel(DecoderModel):
                            logit_scale=c.logit_scale, tie_embeddings=True, initializer_range=c.initializer_range)
 
 
+class BakasunModel(DecoderModel):
+    """Bakasun: norms before and after each sublayer around a 32-bit residual stream; layers of windowed attention with query
+    and key norms over the whole projection, and layers of windowed attention (biased projections, capped scores) and a gated
+    delta rule side by side; a constant term in every softmax denominator; dense GELU feed-forwards, or mixtures whose experts
+    are chosen within the best groups with a correction, beside a gated shared expert.  Not one of the reference's families."""
+
+    config_class = C.BakasunConfig
+    scheme = KeyScheme(embed=("embed",), layer=("l{i}.",), ln1=("norm1",), ln2=("norm2",), ln1b=("norm1b",), ln2b=("norm2b",),
+                       q=("mix.q",), k=("mix.k",), v=("mix.v",), q_norm=("mix.q.norm",), k_norm=("mix.k.norm",), o=("mix.o",),
+                       gate=("mlp.gate",), up=("mlp.up",), down=("mlp.down",), router=("mlp.router",), correction=("mlp.correction",),
+                       expert=("mlp.e{e}.",), e_gate=("gate",), e_up=("up",), e_down=("down",), shared_gate=("mlp.shared.gate",),
+                       shared_up=("mlp.shared.up",), shared_down=("mlp.shared.down",), shared_sg=("mlp.shared.sg",),
+                       final_norm=("final.norm",), lm_head=("head",), weight_suffix="", bias_suffix=".b",
+                       sides=("mix.", "mix.left.", "mix.right."),
+                       mixers={"delta": {"w_qkv": ("mix.q", "mix.k", "mix.v"), "conv": ("mix.q.conv", "mix.k.conv", "mix.v.conv"),
+                                         "w_b": ("mix.b",), "w_a": ("mix.a",), "A_log": ("mix.A_log",), "dt_bias": ("mix.dt_bias",),
+                                         "w_g": ("mix.g",), "o_norm": ("mix.norm",), "wo": ("mix.o",)}})
+
+    @staticmethod
+    def _moe_spec(i: int, mlp: dict) -> MoESpec:
+        r, sh = mlp["router"], mlp.get("shared")
+        g = r.get("groups") or {"count": 1, "keep": 1}
+        E, top = r["experts"], r["top"]
+        if E % g["count"] or not 1 <= g["keep"] <= g["count"] or top > g["keep"] * (E // g["count"]):
+            raise ConfigurationError(f"layer {i}: {top} of {E} experts from {g['keep']} of {g['count']} groups")
+        return MoESpec(num_experts=E, top_k=top, intermediate_size=mlp["expert"]["ff"], act="silu", correction=True,
+                       groups=g["count"], keep_groups=g["keep"], num_shared_experts=0 if sh is None else 1,
+                       shared_intermediate_size=None if sh is None else sh["ff"], shared_gate=sh is not None)
+
+    @staticmethod
+    def _heads(i: int, mx: dict) -> dict:
+        if mx["heads"] % mx["kv_heads"]:
+            raise ConfigurationError(f"layer {i}: {mx['heads']} heads over {mx['kv_heads']} key heads")
+        return dict(num_heads=mx["heads"], num_kv_heads=mx["kv_heads"], head_dim=mx["dim"], v_head_dim=mx["vdim"])
+
+    @classmethod
+    def _attention_spec(cls, i: int, mx: dict, **kw) -> LayerSpec:
+        rot = mx.get("rot")
+        if rot and (rot["dims"] > mx["dim"] or rot["dims"] % 2):
+            raise ConfigurationError(f"layer {i}: {rot['dims']} rotated dimensions of {mx['dim']}")
+        sc = rot.get("scaling") if rot else None
+        return LayerSpec(**cls._heads(i, mx), window=mx["mask"]["size"] if mx.get("mask") else 0, scale=float(mx["scale"]),
+                         rotary_dim=rot["dims"] if rot else 0, rope_theta=float(rot["base"]) if rot else 10000.0,
+                         rope_linear=float(sc["factor"]) if sc else 1.0, fixed_sink=0.0, softcap=float(mx.get("softcap") or 0.0), **kw)
+
+    @classmethod
+    def _layer_spec(cls, i: int, d: dict) -> LayerSpec:
+        mx, mlp = d["mixer"], d.get("mlp")
+        ff = {"mlp": None}
+        if mlp is not None:
+            kind = mlp.get("kind")
+            if kind == "dense":
+                ff = dict(mlp="dense", intermediate_size=mlp["ff"])
+            elif kind == "moe":
+                ff = dict(mlp="moe", moe=cls._moe_spec(i, mlp))
+            else:
+                raise ConfigurationError(f"layer {i}: unknown feed-forward {kind!r}")
+        if d["type"] == "attention":
+            return cls._attention_spec(i, mx, qkv_bias=False, qk_norm="row", **ff)
+        if d["type"] != "parallel":
+            raise ConfigurationError(f"layer {i}: unknown mixer {d['type']!r}")
+        right = LayerSpec(**cls._heads(i, mx["right"]), mixer="delta", conv_taps=mx["right"]["conv"], mlp=None)
+        return cls._attention_spec(i, mx["left"], qkv_bias=True, qk_norm="", beside=right,
+                                   scales=(float(mx["left_scale"]), float(mx["right_scale"])), **ff)
+
+    @classmethod
+    def spec_from_config(cls, c):
+        layers = tuple(cls._layer_spec(i, d) for i, d in enumerate(c.layers))
+        first = layers[0] if layers else None
+        return DecoderSpec(vocab_size=c.vocab_size, hidden_size=c.hidden_size, num_layers=len(layers), layers=layers,
+                           num_heads=first.num_heads if first else 0, num_kv_heads=first.num_kv_heads if first else 0,
+                           head_dim=first.head_dim if first else 0, intermediate_size=0,
+                           max_position_embeddings=c.max_position_embeddings, norm="rms", norm_eps=c.norm_eps,
+                           norm_weight_offset_one=True, norm_placement="both", residual_fp32=True, act="gelu_tanh",
+                           initializer_range=c.initializer_range)
+
+
 DECODER_FAMILIES = {
     "llama": LlamaModel, "qwen": QwenModel, "gemma": GemmaModel, "phi": PhiModel, "deepseek": DeepSeekModel,
     "mistral": MistralModel, "mixtral": MixtralModel, "gpt2": GPT2Model, "gptj": GPTJModel, "gptneox": GPTNeoXModel,
@@ -559,5 +636,5 @@ DECODER_FAMILIES = {
     "olmo": OlmoModel, "granite": GraniteModel, "yi": YiModel, "falcon": FalconModel, "baichuan": BaichuanModel,
     "internlm": InternLMModel, "chatglm": ChatGLMModel, "minicpm": MiniCPMModel, "deepseek_moe": DeepSeekMoEModel,
     "dbrx": DbrxModel, "grok": GrokModel, "arctic": ArcticModel, "gekapel": GekapelModel,
-    "nipulorn": NipulornModel,
+    "nipulorn": NipulornModel, "bakasun": BakasunModel,
 }

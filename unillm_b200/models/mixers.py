@@ -1,11 +1,13 @@
-"""Sublayer parts of per-layer specs beyond plain attention: latent attention, the wkv recurrence, the input convolution and
-the xIELU activation, as PyTorch on any device -- the whole-model path and the CPU runner; the serving kernels are
-``csrc/attn/attn_latent.cu``, ``csrc/scan/wkv_mixer.cu`` and ``csrc/norm/sublayer_in.cu``.
+"""Sublayer parts of per-layer specs beyond plain attention: latent attention, the wkv recurrence, the gated delta rule, the
+input convolution and the xIELU activation, as PyTorch on any device -- the whole-model path and the CPU runner; the serving
+kernels are ``csrc/attn/attn_latent.cu``, ``csrc/wkv/wkv_mixer.cu``, ``csrc/delta/delta_mixer.cu`` and
+``csrc/norm/sublayer_in.cu``.
 
 State that a sequence carries lives in a dictionary per layer (``st``); a missing entry stands for the start of a sequence.
 
 Latent attention follows DeepSeek-V2 ("DeepSeek-V2: A Strong, Economical, and Efficient Mixture-of-Experts Language
-Model"), the recurrence RWKV-6 (the reference's ``models_v2/rwkv6.rs:483-553`` in another parametrisation).
+Model"), the recurrence RWKV-6 (the reference's ``models_v2/rwkv6.rs:483-553`` in another parametrisation), the delta rule
+with decay "Gated Delta Networks: Improving Mamba2 with Delta Rule" (Yang, Kautz, Hatamizadeh).
 """
 from __future__ import annotations
 
@@ -22,7 +24,7 @@ MU = ("r", "k", "v", "g", "w")           # order of the token-shift mixes in the
 
 
 def mixer_shapes(ls: LayerSpec, H: int) -> Dict[str, Tuple[int, ...]]:
-    """Canonical parameters of a latent or wkv mixer."""
+    """Canonical parameters of a latent, wkv or delta mixer."""
     n, d = ls.num_heads, ls.head_dim
     if ls.mixer == "latent":
         return {"w_dqkv": (ls.q_rank + ls.kv_rank + ls.rot_dim, H), "q_a_norm": (ls.q_rank,), "kv_a_norm": (ls.kv_rank,),
@@ -32,6 +34,9 @@ def mixer_shapes(ls: LayerSpec, H: int) -> Dict[str, Tuple[int, ...]]:
         C = n * d
         return {"mu": (5, H), "w_rkvg": (4, C, H), "w_d1": (ls.decay_rank, H), "w_d2": (C, ls.decay_rank), "d0": (C,),
                 "u": (n, d), "o_norm": (C,), "wo": (H, C)}
+    if ls.mixer == "delta":
+        return {"w_qkv": (ls.conv_rows, H), "conv": (ls.conv_rows, ls.conv_taps), "w_b": (n, H), "w_a": (n, H), "A_log": (n,),
+                "dt_bias": (n,), "w_g": (ls.o_size, H), "o_norm": (ls.v_head_dim,), "wo": (H, ls.o_size)}
     raise ValueError(f"no such mixer: {ls.mixer!r}")
 
 
@@ -48,6 +53,8 @@ def split_parts(t: torch.Tensor, ls: LayerSpec, name: str, n: int):
         return [t]
     if name == "w_dqkv":
         return list(t.split([ls.q_rank, ls.kv_rank + ls.rot_dim]))
+    if name in ("w_qkv", "conv"):
+        return list(t.split([ls.k_size, ls.k_size, ls.o_size]))
     return list(t.unbind(0))
 
 
@@ -75,6 +82,25 @@ def wkv(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, st: 
     y = R.wkv6(r, k, v, ww.contiguous(), p[L + "u"].float(), n, st["wkv"]).float().reshape(B, T, n, d)
     y = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)
     return (y.reshape(B, T, n * d) * p[L + "o_norm"].float() * F.silu(g.float())).to(h.dtype)
+
+
+def delta(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, st: dict, eps: float) -> torch.Tensor:
+    """Gated delta rule: h [B, T, H] -> [B, T, heads * value size], before the output projection."""
+    B, T, _ = h.shape
+    n, g, dk, dv = ls.num_heads, ls.num_kv_heads, ls.head_dim, ls.v_head_dim
+    y = ops_fn.linear(h, p[L + "w_qkv"]).float()
+    if "conv" not in st:
+        st["conv"] = torch.zeros(B, ls.conv_taps - 1, y.shape[2], dtype=torch.float32, device=h.device)
+        st["delta"] = torch.zeros(B, n, dk, dv, dtype=torch.float32, device=h.device)
+    y = F.silu(R.causal_dwconv1d(y, p[L + "conv"], None, st["conv"]))
+    q, k, v = y.split([ls.k_size, ls.k_size, ls.o_size], dim=-1)
+    unit = lambda x: x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
+    q, k = (unit(x.reshape(B, T, g, dk)).repeat_interleave(n // g, dim=2) for x in (q, k))
+    beta = torch.sigmoid(ops_fn.linear(h, p[L + "w_b"]).float())
+    keep = torch.exp(-torch.exp(p[L + "A_log"].float()) * F.softplus(ops_fn.linear(h, p[L + "w_a"]).float() + p[L + "dt_bias"].float()))
+    o, st["delta"] = R.delta_rule(q * dk ** -0.5, k, v.reshape(B, T, n, dv), keep, beta, st["delta"])
+    o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * p[L + "o_norm"].float()
+    return (o.reshape(B, T, n * dv) * F.silu(ops_fn.linear(h, p[L + "w_g"]).float())).to(h.dtype)
 
 
 def latent_project(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, eps: float):

@@ -34,6 +34,10 @@ class MoESpec:
     gated: bool = True                   # False: down(act(up x)) experts (and shared experts)
     router_bias: bool = False            # logits = W x + b
     shared_intermediate_size: Optional[int] = None   # width of the always-on expert; None: num_shared * intermediate_size
+    correction: bool = False             # experts are chosen by softmax(logits) + correction, weighted without it
+    groups: int = 1                      # equal groups of neighbouring experts; only those of the ``keep_groups`` groups with
+    keep_groups: int = 1                 # the largest score in them can be chosen
+    shared_gate: bool = False            # the always-on expert's output is multiplied by sigmoid(w . x), one number per token
 
     @property
     def shared_width(self) -> int:
@@ -50,8 +54,13 @@ class LayerSpec:
 
     ``mixer``: "attention"; "latent" (multi-head latent attention: queries through a normalised latent of ``q_rank``, keys
     and values of all heads from one cached, normalised latent of ``kv_rank`` and one cached rotated key part of
-    ``rot_dim`` shared by the heads; ``head_dim`` is the unrotated key size); or "wkv" (RWKV-6 style recurrence with a
-    ``head_dim`` x ``head_dim`` state per head, five token-shift mixes and a low-rank decay of ``decay_rank``)."""
+    ``rot_dim`` shared by the heads; ``head_dim`` is the unrotated key size); "wkv" (RWKV-6 style recurrence with a
+    ``head_dim`` x ``head_dim`` state per head, five token-shift mixes and a low-rank decay of ``decay_rank``); or "delta"
+    (gated delta rule with a ``head_dim`` x ``v_head_dim`` state per head, queries and keys of ``num_kv_heads`` heads, and
+    causal convolutions of ``conv_taps`` taps on queries, keys and values).
+
+    ``beside``: a second mixer that reads the same input; the first one's output times ``scales[0]`` and the second one's
+    times ``scales[1]`` are added."""
 
     num_heads: int
     num_kv_heads: int
@@ -64,7 +73,12 @@ class LayerSpec:
     rope_llama3: Optional[Tuple[float, float, float, float]] = None
     rope_yarn: Optional[Tuple[float, float, float, float]] = None   # (factor, original_ctx, fast turns, slow turns)
     kv_from: Optional[int] = None
+    rope_linear: float = 1.0             # frequencies are divided by this
     sink: bool = False                   # one learned logit per head in the softmax denominator
+    fixed_sink: Optional[float] = None   # a constant logit there instead
+    softcap: float = 0.0                 # scores become softcap * tanh(score / softcap); 0 = as they are
+    qkv_bias: Optional[bool] = None      # None = as the model says
+    qk_norm: Optional[str] = None        # "head", "row" (over the whole projection), "" = none; None = as the model says
     mlp: Optional[str] = "dense"
     moe: Optional[MoESpec] = None
     mixer: str = "attention"
@@ -73,11 +87,23 @@ class LayerSpec:
     rot_dim: int = 0
     decay_rank: int = 0
     intermediate_size: Optional[int] = None   # dense feed-forward width (None: the model's)
+    conv_taps: int = 0
+    beside: Optional["LayerSpec"] = None
+    scales: Tuple[float, float] = (1.0, 1.0)
 
     @property
     def has_kv(self) -> bool:
         """The layer owns cache rows."""
-        return self.mixer != "wkv" and self.kv_from is None
+        return self.mixer not in ("wkv", "delta") and self.kv_from is None
+
+    @property
+    def mixers(self) -> Tuple["LayerSpec", ...]:
+        return (self,) if self.beside is None else (self, self.beside)
+
+    @property
+    def conv_rows(self) -> int:
+        """Channels of a delta mixer's convolutions: [Q; K; V]."""
+        return 2 * self.k_size + self.o_size
 
     @property
     def cache_row(self) -> int:
@@ -199,6 +225,14 @@ class DecoderSpec:
         """Layers that own cache rows (the others read one of these, or have no keys)."""
         return tuple(i for i in range(self.num_layers) if self.layer(i).has_kv)
 
+    def qk_norm_kind(self, i: int) -> str:
+        kind = self.layer(i).qk_norm
+        return ("head" if self.qk_norm else "") if kind is None else kind
+
+    def has_qkv_bias(self, i: int) -> bool:
+        b = self.layer(i).qkv_bias
+        return self.qkv_bias if b is None else b
+
     def layer_intermediate(self, i: int) -> int:
         n = self.layer(i).intermediate_size
         return self.intermediate_size if n is None else n
@@ -206,7 +240,7 @@ class DecoderSpec:
     @property
     def state_elements(self) -> int:
         """fp32 elements of state that one sequence carries from token to token besides cache rows: the last inputs of the
-        convolutions, the previous token's input and the recurrent state of the wkv layers."""
+        convolutions, the previous token's input of the wkv layers and the recurrent state of the wkv and delta mixers."""
         n = 0
         for i in range(self.num_layers):
             ls = self.layer(i)
@@ -214,6 +248,9 @@ class DecoderSpec:
                 n += (self.input_conv - 1) * self.hidden_size * (2 if ls.mlp is not None else 1)
             if ls.mixer == "wkv":
                 n += self.hidden_size + ls.num_heads * ls.head_dim * ls.head_dim
+            for mx in ls.mixers:
+                if mx.mixer == "delta":
+                    n += (mx.conv_taps - 1) * mx.conv_rows + mx.num_heads * mx.head_dim * mx.v_head_dim
         return n
 
     @property
@@ -255,11 +292,15 @@ class KeyScheme:
     conv1: Tuple[str, ...] = ()          # input convolutions
     conv2: Tuple[str, ...] = ()
     act: Tuple[str, ...] = ()            # learned numbers of the activation
-    mixers: Optional[dict] = None        # {mixer: {parameter: names, several = stacked or concatenated}}, see decoder.MIXER_PARAMS
+    mixers: Optional[dict] = None        # {mixer: {parameter: names, several = stacked or concatenated}}, see mixers.mixer_shapes
+    sides: Optional[Tuple[str, str, str]] = None   # prefix of a mixer's names; what replaces it for the first and the second
+    #                                                of two mixers side by side
     weight_suffix: str = ".weight"
     bias_suffix: str = ".bias"
     transposed: bool = False             # GPT-2 Conv1D stores [in, out]
     router: Tuple[str, ...] = ("block_sparse_moe.gate",)
+    correction: Tuple[str, ...] = ()
+    shared_sg: Tuple[str, ...] = ()      # gate of the always-on expert
     expert: Tuple[str, ...] = ("block_sparse_moe.experts.{e}.",)
     e_gate: Tuple[str, ...] = ("w1",)
     e_up: Tuple[str, ...] = ("w3",)

@@ -70,7 +70,7 @@ class UbRopeArgs(C.Structure):
         ("T", i32), ("Hq", i32), ("Hkv", i32), ("D", i32), ("rotary_dim", i32), ("block_size", i32),
         ("num_slots", i64), ("theta", f32), ("pos_scale", f32), ("norm_eps", f32), ("interleaved", i32),
         ("l3_factor", f32), ("l3_low_freq_factor", f32), ("l3_high_freq_factor", f32), ("l3_orig_ctx", f32),
-        ("inv_freq", vp), ("Dv", i32), ("norm_dim", i32), ("f32", i32), ("k_cache_only", i32),
+        ("inv_freq", vp), ("Dv", i32), ("norm_dim", i32), ("f32", i32), ("k_cache_only", i32), ("row_norm", i32), ("ld", i64),
     ]
 
 
@@ -89,6 +89,8 @@ class UbSublayerInArgs(C.Structure):
         ("row0", i64), ("out_mix_stride", i64),
         ("H", i32), ("Hp", i32), ("taps", i32), ("n_mix", i32), ("num_seqs", i32), ("max_q", i32), ("state_rows", i32),
         ("tile", i32), ("f32", i32), ("eps", f32), ("w_off", f32),
+        ("yx", vp), ("row_slot", vp), ("topk_w", vp), ("y_gate", vp), ("rows", vp), ("n_rows", i32), ("x_rows", i32), ("K", i32),
+        ("slots", i32),
     ]
 
 
@@ -99,6 +101,16 @@ class UbWkvArgs(C.Structure):
         ("row0", i64), ("ld", i64),
         ("H", i32), ("D", i32), ("norm_dim", i32), ("num_seqs", i32), ("state_rows", i32), ("f32", i32),
         ("chunk", i32), ("rows", i32), ("max_chunks", i32), ("eps", f32),
+    ]
+
+
+class UbDeltaArgs(C.Structure):
+    _fields_ = [
+        ("qkv", vp), ("gate", vp), ("b", vp), ("a", vp), ("conv", vp), ("a_log", vp), ("dt_bias", vp), ("norm_w", vp),
+        ("conv_state", vp), ("state", vp), ("state_in", vp), ("state_out", vp), ("q_start", vp), ("out", vp), ("ws", vp), ("err", vp),
+        ("row0", i64), ("ld", i64), ("ld_out", i64),
+        ("H", i32), ("G", i32), ("dk", i32), ("dv", i32), ("dk_real", i32), ("dv_real", i32), ("taps", i32), ("num_seqs", i32),
+        ("max_q", i32), ("rows", i32), ("state_rows", i32), ("f32", i32), ("lanes", i32), ("eps", f32),
     ]
 
 
@@ -137,7 +149,7 @@ class UbAttnArgs(C.Structure):
         ("block_size", i32), ("max_blocks_per_seq", i32), ("num_blocks", i32),
         ("q_stride", i64), ("o_stride", i64), ("scale", f32),
         ("causal", i32), ("window", i32), ("splits", i32), ("kv_start", i32), ("total_q", i32), ("max_q_len", i32),
-        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32), ("kv_shared", i32),
+        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32), ("kv_shared", i32), ("softcap", f32),
     ]
 
 
@@ -166,6 +178,7 @@ class UbMoeRouteArgs(C.Structure):
         ("logits_f32", i32), ("T", i32), ("E", i32), ("K", i32), ("H", i32), ("norm_topk", i32),
         ("round_logits_bf16", i32), ("weight_scale", f32), ("tile_tokens", i32), ("max_tiles", i32),
         ("expert_lo", i32), ("num_local_experts", i32), ("router_b", vp), ("x_f32", i32), ("router_f32", i32),
+        ("correction", vp), ("groups", i32), ("keep_groups", i32), ("shared_w", vp), ("shared_gate", vp),
     ]
 
 
@@ -231,7 +244,7 @@ class _CudaLibs:
 
     ARGS_AND_STREAM = {
         "serving": ("ub_gemm_tn", "ub_norm", "ub_rope_kv_append", "ub_attn_decode", "ub_attn_prefill", "ub_sample",
-                    "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm", "ub_sublayer_in", "ub_wkv_mixer",
+                    "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm", "ub_sublayer_in", "ub_wkv_mixer", "ub_delta_mixer",
                     "ub_gemm_heads", "ub_latent_rows", "ub_latent_rotate", "ub_attn_latent", "ub_latent_gather", "ub_attn_expanded"),
         "more": ("ub_allreduce_oneshot", "ub_tp_argmax_merge"),
     }
@@ -244,6 +257,7 @@ class _CudaLibs:
         lib.ub_gemm_streamk_reset.restype = i32
         lib.ub_gemm_streamk_reset.argtypes = [vp]
         lib.ub_wkv_workspace_floats.restype = i64
+        lib.ub_delta_workspace_floats.restype = i64
         lib.ub_cuda_error_string.restype = C.c_char_p
 
     def part(self, name: str) -> C.CDLL:

@@ -330,12 +330,21 @@ def _state_rows(what: str, t: Optional[torch.Tensor], tail: tuple) -> None:
 def sublayer_in(x: torch.Tensor, portions: Sequence[Portions], weight: torch.Tensor, *, eps: float, y: Optional[torch.Tensor] = None,
                 y_weight: Optional[torch.Tensor] = None, conv: Optional[torch.Tensor] = None,
                 conv_state: Optional[torch.Tensor] = None, mu: Optional[torch.Tensor] = None,
-                shift_state: Optional[torch.Tensor] = None, width: Optional[int] = None, offset_one: bool = True, tile: int = 0):
+                shift_state: Optional[torch.Tensor] = None, width: Optional[int] = None, offset_one: bool = True, tile: int = 0,
+                experts: Optional[torch.Tensor] = None, routing: Optional["MoeRouting"] = None, rows: Optional[torch.Tensor] = None):
     """What the next sublayer reads: ``x' = x + norm(y)``, ``h = norm(x')`` plus its causal convolution over time with the taps
     ``conv`` ([taps, width], the last one meets the token itself), and with ``mu`` ([5, width]) the five token-shift
     mixes ``h + (previous h - h) * mu``.  Returns ``(x', out)``; out is [rows, width], or [5, rows, width] with ``mu``, in
-    the type of ``weight``.  The state tensors hold what the sequences of ``portions`` carry on."""
-    f32 = _elem("sublayer_in", weight, y, y_weight, conv, mu)
+    the type of ``weight``.  The state tensors hold what the sequences of ``portions`` carry on.
+
+    Without ``conv`` and ``mu`` rows stand alone: ``y`` may be a mixture (``experts`` in the order of ``routing``, ``y`` the rows
+    of its always-on expert or None), and ``rows`` (int32) picks the rows to compute -- only ``out`` of those is returned then,
+    and ``x`` stays as it is; otherwise ``x`` is changed in place."""
+    f32 = _elem("sublayer_in", weight, y, y_weight, conv, mu, experts)
+    if conv is None and mu is None:
+        return _sublayer_alone(x, weight, eps, y, y_weight, width, offset_one, experts, routing, rows, f32)
+    if experts is not None or rows is not None:
+        raise ValueError("sublayer_in: mixtures and picked rows go without convolution and mixes")
     T, Hp = x.shape
     if x.dtype != torch.float32 or not x.is_contiguous() or weight.numel() != Hp:
         raise ValueError("sublayer_in: contiguous fp32 stream, weights of its width")
@@ -370,6 +379,81 @@ def sublayer_in(x: torch.Tensor, portions: Sequence[Portions], weight: torch.Ten
         a.f32, a.eps, a.w_off = int(f32), eps, 1.0 if offset_one else 0.0
         N.check(N.cuda_lib().ub_sublayer_in(C.byref(a), _stream(x)), "ub_sublayer_in")
     return x_out, out
+
+
+def _sublayer_alone(x, weight, eps, y, y_weight, width, offset_one, experts, routing, rows, f32):
+    T, Hp = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous() or weight.numel() != Hp:
+        raise ValueError("sublayer_in: contiguous fp32 stream, weights of its width")
+    if y is not None and (y.shape != x.shape or not y.is_contiguous()):
+        raise ValueError("sublayer_in: y has the stream's shape")
+    if (y is not None or experts is not None) and (y_weight is None or y_weight.numel() != Hp):
+        raise ValueError("sublayer_in: a norm weight for y")
+    if rows is not None and rows.dtype != torch.int32:
+        raise TypeError("sublayer_in: rows must be int32")
+    a = N.UbSublayerInArgs()
+    n = T if rows is None else rows.numel()
+    out = torch.empty(n, Hp, dtype=weight.dtype, device=x.device)
+    if n == 0:
+        return out if rows is not None else (x, out)
+    a.x, a.y, a.wy, a.wn, a.out, a.rows = x.data_ptr(), _p(y), _p(y_weight), weight.data_ptr(), out.data_ptr(), _p(rows)
+    a.x_out = x.data_ptr() if rows is None else None
+    if experts is not None:
+        if routing.T != T or experts.shape[1] != Hp or not experts.is_contiguous():
+            raise ValueError("sublayer_in: the routing is of another step, or expert rows of another width")
+        a.yx, a.row_slot, a.topk_w = experts.data_ptr(), routing.row_slot.data_ptr(), routing.topk_w.data_ptr()
+        a.K, a.slots, a.y_gate = routing.K, experts.shape[0], _p(routing.shared_gate if y is not None else None)
+    a.err = err_word(x.device).data_ptr()
+    a.H, a.Hp, a.n_rows, a.x_rows, a.f32, a.eps, a.w_off = width or Hp, Hp, n, T, int(f32), eps, 1.0 if offset_one else 0.0
+    N.check(N.cuda_lib().ub_sublayer_in(C.byref(a), _stream(x)), "ub_sublayer_in")
+    return out if rows is not None else (x, out)
+
+
+def delta_mixer(proj: torch.Tensor, col: int, conv: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor,
+                conv_state: Optional[torch.Tensor], state: torch.Tensor, portions: Sequence[Portions], *, kv_heads: int, eps: float,
+                dk_real: int = 0, dv_real: int = 0, out: Optional[torch.Tensor] = None, lanes: int = 0) -> torch.Tensor:
+    """Gated delta rule with its convolutions, head norm and SiLU gate.  ``proj`` [T, ld]: from column ``col`` on, rows of
+    [Q | K | V | gate | b | a] with ``kv_heads`` * Dk, the same, H * Dv, H * Dv, H and H columns.  ``conv`` [taps, Q + K + V],
+    ``state`` fp32 [rows, H, Dk, Dv], ``conv_state`` fp32 [rows, taps - 1, Q + K + V] -> [T, H * Dv] (``out`` may be columns of a
+    wider tensor).  ``dk_real`` / ``dv_real``: head sizes before padding.  ``lanes``: see ``UbDeltaArgs``."""
+    f32 = _elem("delta_mixer", proj, conv, out)
+    T, ld = proj.shape
+    _, H, dk, dv = state.shape
+    taps, Cn = conv.shape
+    qk = kv_heads * dk
+    if proj.stride(1) != 1 or not conv.is_contiguous() or Cn != 2 * qk + H * dv or col + Cn + H * dv + 2 * H > ld:
+        raise ValueError("delta_mixer: rows of [Q | K | V | gate | b | a], taps over [Q | K | V]")
+    for t, n in ((a_log, H), (dt_bias, H), (norm_w, dv)):
+        if t.dtype != torch.float32 or t.numel() != n:
+            raise ValueError("delta_mixer: fp32 a_log [H], dt_bias [H] and norm weight [Dv]")
+    _state_rows("delta_mixer", state, (H, dk, dv))
+    if taps > 1:
+        _state_rows("delta_mixer convolutions", conv_state, (taps - 1, Cn))
+        if conv_state.shape[0] != state.shape[0]:
+            raise ValueError("delta_mixer: as many rows of either state")
+    if out is None:
+        out = torch.empty(T, H * dv, dtype=proj.dtype, device=proj.device)
+    if out.shape != (T, H * dv) or out.stride(1) != 1:
+        raise ValueError("delta_mixer: out is [T, H * Dv]")
+    lib, e = N.cuda_lib(), proj.element_size()
+    at = lambda c: proj.data_ptr() + (col + c) * e
+    for p in portions:
+        if p.row0 + p.rows > T:
+            raise ValueError("delta_mixer: portions outside the step")
+        a = N.UbDeltaArgs()
+        a.qkv, a.gate, a.b, a.a = at(0), at(Cn), at(Cn + H * dv), at(Cn + H * dv + H)
+        a.conv, a.a_log, a.dt_bias, a.norm_w = conv.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr()
+        a.conv_state, a.state = _p(conv_state if taps > 1 else None), state.data_ptr()
+        a.state_in, a.state_out, a.q_start = _p(p.state_in), _p(p.state_out), _p(p.q_start)
+        a.out, a.err = out.data_ptr(), err_word(proj.device).data_ptr()
+        a.row0, a.ld, a.ld_out = p.row0, proj.stride(0), out.stride(0)
+        a.H, a.G, a.dk, a.dv, a.dk_real, a.dv_real, a.taps = H, kv_heads, dk, dv, dk_real or dk, dv_real or dv, taps
+        a.num_seqs, a.max_q, a.rows, a.state_rows, a.f32, a.lanes, a.eps = p.n, p.max_q, p.rows, state.shape[0], int(f32), lanes, eps
+        if p.q_start is not None:
+            ws = torch.empty(lib.ub_delta_workspace_floats(p.rows, H, kv_heads, dk, dv), dtype=torch.float32, device=proj.device)
+            a.ws = ws.data_ptr()
+        N.check(lib.ub_delta_mixer(C.byref(a), _stream(proj)), "ub_delta_mixer")
+    return out
 
 
 WKV_CHUNK = 64
@@ -616,15 +700,18 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
                    pos_scale: float = 1.0, interleaved: bool = False, q_norm_w: Optional[torch.Tensor] = None,
                    k_norm_w: Optional[torch.Tensor] = None, norm_eps: float = 1e-6,
                    llama3_scaling: Optional[Sequence[float]] = None, v_head_dim: Optional[int] = None,
-                   norm_dim: int = 0, inv_freq: Optional[torch.Tensor] = None, k_cache_only: bool = False) -> torch.Tensor:
+                   norm_dim: int = 0, inv_freq: Optional[torch.Tensor] = None, k_cache_only: bool = False,
+                   row_norm: bool = False) -> torch.Tensor:
     """Rotates q and k inside ``qkv`` [T, (Hq+Hkv)*D + Hkv*Dv] in place and appends k, v to the paged cache.
 
     ``num_kv_heads = 0``: rows hold queries only (a layer that reads another layer's keys).  ``inv_freq`` (fp32
     [rotary_dim / 2]) replaces the frequencies that ``theta`` and the scaling give; ``norm_dim`` is the number of elements
-    the head norm averages over when heads are zero-padded.  ``k_cache_only``: the rotated k is needed in the cache only."""
+    the head norm averages over when heads are zero-padded.  ``k_cache_only``: the rotated k is needed in the cache only.
+    ``row_norm``: one norm over all queries of a token and one over all its keys (weights of that size).  ``qkv`` may be the
+    first columns of wider rows."""
     f32 = _elem("rope_kv_append", qkv, k_cache, v_cache, q_norm_w, k_norm_w)
-    if not qkv.is_contiguous():
-        raise ValueError("qkv must be contiguous")
+    if qkv.stride(1) != 1:
+        raise ValueError("qkv: rows must be contiguous")
     T = qkv.shape[0]
     if positions.dtype != torch.int32 or (slot_mapping is not None and slot_mapping.dtype != torch.int32):
         raise TypeError("positions / slot_mapping must be int32")
@@ -644,7 +731,10 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
     a.theta, a.pos_scale, a.norm_eps = theta, pos_scale, norm_eps
     a.interleaved = 1 if interleaved else 0
     a.Dv, a.norm_dim, a.f32 = v_head_dim or head_dim, norm_dim, int(f32)
-    a.k_cache_only = int(k_cache_only)
+    a.k_cache_only, a.row_norm, a.ld = int(k_cache_only), int(row_norm), qkv.stride(0)
+    if row_norm and (q_norm_w is None or q_norm_w.numel() != num_q_heads * head_dim or
+                     (num_kv_heads and (k_norm_w is None or k_norm_w.numel() != num_kv_heads * head_dim))):
+        raise ValueError("rope_kv_append: row norms take weights over all heads")
     if qkv.shape[1] != (num_q_heads + num_kv_heads) * head_dim + num_kv_heads * a.Dv:
         raise ValueError(f"rope_kv_append: rows of {qkv.shape[1]} elements do not hold these heads")
     if k_cache is not None and (k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]) != (num_kv_heads, head_dim, a.Dv):
@@ -662,7 +752,7 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
 # ---------------------------------------------------------------------------------------------
 # Attention
 # ---------------------------------------------------------------------------------------------
-def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks=None):
+def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks=None, softcap=0.0):
     a = N.UbAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out, a.lse = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(lse)
     a.block_tables, a.seq_lens = block_tables.data_ptr(), seq_lens.data_ptr()
@@ -671,7 +761,7 @@ def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D
     a.block_size, a.max_blocks_per_seq, a.num_blocks = k_cache.shape[2], block_tables.shape[1], k_cache.shape[0]
     a.q_stride, a.o_stride = q.stride(0), out.stride(0)
     a.scale = scale if scale is not None else 1.0 / math.sqrt(D)
-    a.Dv = v_cache.shape[3]
+    a.Dv, a.softcap = v_cache.shape[3], softcap
     if k_cache.shape[3] != D or out.shape[-1] != a.Dv:
         raise ValueError("attention: head sizes of q, caches and out do not match")
     if sinks is not None:
@@ -686,10 +776,10 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, b
                 alibi_slopes: Optional[torch.Tensor] = None, splits: int = 0, scratch: Optional[torch.Tensor] = None,
                 out: Optional[torch.Tensor] = None, return_lse: bool = False, lse: Optional[torch.Tensor] = None,
                 max_seq_len: Optional[int] = None, merge: Optional[tuple] = None, kernel: Optional[str] = None,
-                sinks: Optional[torch.Tensor] = None):
+                sinks: Optional[torch.Tensor] = None, softcap: float = 0.0):
     """One query token per sequence.  q: [B, Hq, D] (last two dims contiguous); caches [nb, Hkv, bs, D] (the value cache may
-    have a head size of its own).  ``sinks``: fp32 [Hq], one logit per head that joins the softmax denominator.  fp32
-    operands run in 32-bit arithmetic.
+    have a head size of its own).  ``sinks``: fp32 [Hq], one logit per head that joins the softmax denominator.
+    ``softcap`` > 0: scores become softcap * tanh(score / softcap).  fp32 operands run in 32-bit arithmetic.
 
     ``kernel="warp"`` calls the warp-per-item kernel directly (page size 16, head size 64 / 128, ``splits == 1``, no
     window, no ALiBi) instead of going through the dispatcher's choice."""
@@ -710,7 +800,7 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, b
         splits = 1
         while ctas * splits < 2 * 148 and ctx // (splits * 2) >= 256 and splits < 16:
             splits *= 2
-    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks)
+    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks, softcap)
     if splits > 1:
         need = B * Hq * splits * (Dv + 2)
         if scratch is None or scratch.numel() < need:
@@ -737,7 +827,8 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
                  causal: bool = True, window: int = 0, kv_start: int = 0,
                  alibi_slopes: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
                  return_lse: bool = False, lse: Optional[torch.Tensor] = None, merge: Optional[tuple] = None,
-                 kv_splits: int = 1, scratch: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None):
+                 kv_splits: int = 1, scratch: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
+                 softcap: float = 0.0):
     """Ragged prefill: q [T, Hq, D]; sequence i owns query rows q_start[i]:q_start[i+1] and sees
     seq_lens[i] keys, its last query at kv position seq_lens[i]-1.
 
@@ -752,7 +843,7 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
         out = torch.empty((T, Hq, v_cache.shape[3]), dtype=q.dtype, device=q.device)
     if return_lse and lse is None:
         lse = torch.empty((T, Hq), dtype=torch.float32, device=q.device)
-    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks)
+    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks, softcap)
     a.q_start = q_start.data_ptr()
     a.causal, a.window, a.kv_start = (1 if causal else 0), window, kv_start
     a.total_q, a.max_q_len = T, max_q_len
@@ -1013,9 +1104,9 @@ class MoeRouting:
     """Device-side routing state of one MoE layer call (all int32 / fp32 tensors, sized from T, K, E)."""
 
     __slots__ = ("T", "K", "E", "tile_tokens", "max_tiles", "topk_ids", "topk_w", "counts", "offsets", "sorted_rows",
-                 "row_slot", "tiles")
+                 "row_slot", "tiles", "shared_gate")
 
-    def __init__(self, T: int, K: int, E: int, tile_tokens: int, device):
+    def __init__(self, T: int, K: int, E: int, tile_tokens: int, device, shared_gate: bool = False):
         self.T, self.K, self.E, self.tile_tokens = T, K, E, tile_tokens
         self.max_tiles = (T * K + tile_tokens - 1) // tile_tokens + E
         i32 = dict(dtype=torch.int32, device=device)
@@ -1026,6 +1117,7 @@ class MoeRouting:
         self.sorted_rows = torch.empty(T * K, **i32)
         self.row_slot = torch.empty(T * K, **i32)
         self.tiles = torch.empty(self.max_tiles, 4, **i32)
+        self.shared_gate = torch.empty(T, dtype=torch.float32, device=device) if shared_gate else None
 
 
 def moe_tile_tokens(T: int, K: int, E: int) -> int:
@@ -1040,14 +1132,18 @@ def moe_tile_tokens(T: int, K: int, E: int) -> int:
 def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k: int, *, norm_topk: bool = True,
               logits: Optional[torch.Tensor] = None, weight_scale: float = 1.0, tile_tokens: int = 0,
               round_logits_bf16: bool = True, routing: Optional[MoeRouting] = None, expert_lo: int = 0,
-              num_local_experts: int = 0, router_b: Optional[torch.Tensor] = None) -> MoeRouting:
+              num_local_experts: int = 0, router_b: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None,
+              groups: int = 1, keep_groups: int = 1, shared_w: Optional[torch.Tensor] = None) -> MoeRouting:
     """Router GEMV (+ bias) + top-k + softmax weights + expert sort + grouped-GEMM tile table, two launches.  ``x`` may be
     bf16 or an fp32 residual stream, whatever the type of the router.
 
     ``expert_lo`` / ``num_local_experts`` restrict the sort to the experts of this rank (expert parallelism): pairs
-    routed to other ranks get ``row_slot = -1`` and take no part in the grouped GEMMs."""
+    routed to other ranks get ``row_slot = -1`` and take no part in the grouped GEMMs.
+
+    ``correction`` ([E]) and / or ``groups``: experts are chosen by softmax + correction within the ``keep_groups`` best groups of
+    neighbours, and weighted by their softmax values.  ``shared_w`` ([H]): ``routing.shared_gate[t] = sigmoid(x[t] . shared_w)``."""
     if router_w is not None:
-        _elem("moe_route x", x), _elem("moe_route router", router_w, router_b)
+        _elem("moe_route x", x), _elem("moe_route router", router_w, router_b, correction, shared_w)
         T, H = x.shape
         if router_w.shape[1] != H or not x.is_contiguous() or not router_w.is_contiguous():
             raise ValueError("moe_route: x [T, H] and router [E, H] must be contiguous")
@@ -1060,7 +1156,10 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
         if not logits.is_contiguous():
             raise ValueError("logits must be contiguous")
     tn = tile_tokens or moe_tile_tokens(T, top_k, E)
-    r = routing if routing is not None else MoeRouting(T, top_k, E, tn, dev)
+    r = routing if routing is not None else MoeRouting(T, top_k, E, tn, dev, shared_w is not None)
+    for t, n in ((correction, E), (shared_w, H)):
+        if t is not None and (router_w is None or t.numel() != n or not t.is_contiguous()):
+            raise ValueError("moe_route: correction [E] and shared_w [H] go with a router matrix")
     a = N.UbMoeRouteArgs()
     a.logits, a.x, a.router_w = _p(logits), _p(x) if router_w is not None else None, _p(router_w)
     a.topk_ids, a.topk_w = r.topk_ids.data_ptr(), r.topk_w.data_ptr()
@@ -1076,6 +1175,8 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
         a.router_b, a.x_f32, a.router_f32 = _p(router_b), int(x.dtype == torch.float32), int(router_w.dtype == torch.float32)
     a.tile_tokens, a.max_tiles = r.tile_tokens, r.max_tiles
     a.expert_lo, a.num_local_experts = expert_lo, num_local_experts
+    a.correction, a.groups, a.keep_groups = _p(correction), groups, keep_groups
+    a.shared_w, a.shared_gate = _p(shared_w), _p(r.shared_gate if shared_w is not None else None)
     N.check(N.cuda_lib().ub_moe_route(C.byref(a), torch.cuda.current_stream(dev).cuda_stream), "ub_moe_route")
     return r
 

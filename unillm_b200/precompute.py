@@ -17,8 +17,8 @@ import torch
 
 
 def rope_inv_freq(rotary_dim: int, base: float, llama3: Optional[Tuple[float, float, float, float]] = None,
-                  yarn: Optional[Tuple[float, float, float, float]] = None) -> torch.Tensor:
-    """Frequencies of the rotated pairs.  ``yarn`` = (factor, original context, fast, slow): pairs that turn more than ``fast``
+                  yarn: Optional[Tuple[float, float, float, float]] = None, linear: float = 1.0) -> torch.Tensor:
+    """Frequencies of the rotated pairs.  ``linear``: all of them divided by that.  ``yarn`` = (factor, original context, fast, slow): pairs that turn more than ``fast``
     times within the original context keep their frequency, those that turn less than ``slow`` times are slowed down by
     ``factor``, with a linear ramp over the pair index between the two (see ``rope_gain`` for the other half of it)."""
     inv = base ** (-torch.arange(0, rotary_dim // 2, dtype=torch.float64) * 2.0 / rotary_dim)
@@ -35,7 +35,7 @@ def rope_inv_freq(rotary_dim: int, base: float, llama3: Optional[Tuple[float, fl
         lo, hi = max(math.floor(pair(fast)), 0), min(math.ceil(pair(slow)), rotary_dim - 1)
         ramp = ((torch.arange(rotary_dim // 2, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
         inv = inv / factor * ramp + inv * (1 - ramp)
-    return inv.float()
+    return (inv / linear).float()
 
 
 def rope_gain(yarn: Optional[Tuple[float, float, float, float]]) -> float:
@@ -46,10 +46,10 @@ def rope_gain(yarn: Optional[Tuple[float, float, float, float]]) -> float:
 class RoPECache:
     def __init__(self, head_dim: int, max_seq_len: int = 2048, base: float = 10000.0, *, rotary_dim: Optional[int] = None,
                  position_scale: float = 1.0, llama3: Optional[Tuple[float, float, float, float]] = None,
-                 yarn: Optional[Tuple[float, float, float, float]] = None, device="cpu"):
+                 yarn: Optional[Tuple[float, float, float, float]] = None, linear: float = 1.0, device="cpu"):
         self.head_dim, self.max_seq_len, self.base = head_dim, max_seq_len, base
         self.rotary_dim = rotary_dim if rotary_dim is not None else head_dim
-        inv = rope_inv_freq(self.rotary_dim, base, llama3, yarn).to(device)
+        inv = rope_inv_freq(self.rotary_dim, base, llama3, yarn, linear).to(device)
         pos = torch.arange(max_seq_len, dtype=torch.float32, device=device) * position_scale
         ang = pos[:, None] * inv[None, :]
         g = rope_gain(yarn)
