@@ -13,16 +13,18 @@
 //
 // One token per sequence (delta_step): a CTA per head and sequence; the state passes through registers once.
 //
-// Portions: delta_prep makes q, k and v of 16 tokens, their products k.k and q.k among themselves, and running sums of the
-// log decays; delta_scan carries the state through blocks of 16 tokens; delta_finish normalises and gates.  Within a block
-// with the log decays' running sum c,
+// Portions: delta_prep makes q, k and v of blocks of 16 tokens and two triangular matrices per block and head; delta_scan
+// carries the state through the blocks; delta_finish normalises and gates.  Within a block, with the running sum c of the log
+// decays, the definition above is
 //
-//   u_i = beta_i (v_i - e^(c_i) S^T k_i - sum_(j < i) e^(c_i - c_j) (k_i . k_j) u_j)
+//   u_i + beta_i sum_(j < i) e^(c_i - c_j) (k_i . k_j) u_j = beta_i (v_i - e^(c_i) S^T k_i)
 //   o_i = e^(c_i) S^T q_i + sum_(j <= i) e^(c_i - c_j) (q_i . k_j) u_j
 //   S  <- e^(c_end) S + sum_j e^(c_end - c_j) k_j u_j^T
 //
-// so the products with S of all 16 tokens are independent, and what is left of the recurrence is a triangular solve of 16
-// scalars per column.  Exponents are never positive.  Columns of S do not meet: a warp owns a few of them.
+// with the S that enters the block.  So with x_j = v_j - e^(c_j) S^T k_j and the inverse T of the unit triangular system (times
+// beta), u = T x and o = e^c S^T q + W x, W = (decayed q k^T) T: T and W hold no column of S, are made once per block and head,
+// and the scan is left with products.  Entries of T are at most one (products of contractions), exponents never positive.
+// Columns of S do not meet: a warp owns a few of them.
 #include "../common/elem.cuh"
 #include "../include/unillm_b200.h"
 
@@ -31,7 +33,7 @@ namespace delta {
 
 constexpr int BT = 16;        // tokens per block
 
-__device__ __forceinline__ float silu(float v) { return v / (1.f + expf(-v)); }
+__device__ __forceinline__ float silu(float v) { return __fdividef(v, 1.f + __expf(-v)); }
 __device__ __forceinline__ float softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float log_decay(const UbDeltaArgs& a, float x, int h) { return -expf(a.a_log[h]) * softplus(x + a.dt_bias[h]); }
 
@@ -47,17 +49,15 @@ __device__ __forceinline__ int state_row(const UbDeltaArgs& a, const int* rows, 
 // ------------------------------------------------------------------------------------------------------------------------
 // one token per sequence
 // ------------------------------------------------------------------------------------------------------------------------
-constexpr int STEP_T = 256;
-
-// ROWS: rows of S that a thread holds (four columns each); 0: S is read twice instead (heads too large for registers).
-template <typename T, int ROWS>
-__global__ void __launch_bounds__(STEP_T) delta_step_kernel(const UbDeltaArgs a, const int cl /* threads across the columns */) {
+// NT threads; ROWS: rows of S that a thread holds (four columns each); 0: S is read twice instead (heads too large for registers).
+template <typename T, int NT, int ROWS>
+__global__ void __launch_bounds__(NT) delta_step_kernel(const UbDeltaArgs a, const int cl /* threads across the columns */) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int HELD = ROWS > 0 ? ROWS : 1;
   extern __shared__ __align__(16) float sm[];
   const int h = blockIdx.x, seq = blockIdx.y, dk = a.dk, dv = a.dv, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int nrg = STEP_T / cl, rg = tid / cl, col = (tid % cl) * 4;
+  const int nrg = NT / cl, rg = tid / cl, col = (tid % cl) * 4;
   float* qkv = sm;                               // [2 dk + dv] after the convolutions
   float* part = qkv + 2 * dk + dv;               // [8][2][dv] partial products with the old state
   float* u_s = part + 8 * 2 * dv;            // [dv]
@@ -81,7 +81,7 @@ __global__ void __launch_bounds__(STEP_T) delta_step_kernel(const UbDeltaArgs a,
     }
   }
   // convolutions of this head's channels; the oldest input leaves, the current one joins
-  for (int c = tid; c < 2 * dk + dv; c += STEP_T) {
+  for (int c = tid; c < 2 * dk + dv; c += NT) {
     const int ch = c < dk ? g * dk + c : c < 2 * dk ? a.G * dk + g * dk + (c - dk) : 2 * a.G * dk + h * dv + (c - 2 * dk);
     const bool keep = so >= 0 && (c >= 2 * dk || h % group == 0);
     const T* w = reinterpret_cast<const T*>(a.conv) + ch;
@@ -95,7 +95,7 @@ __global__ void __launch_bounds__(STEP_T) delta_step_kernel(const UbDeltaArgs a,
     if (keep && m > 0) a.conv_state[((long long)so * m + m - 1) * C + ch] = cur;
     qkv[c] = silu(fmaf((float)w[(long long)m * C], cur, acc));
   }
-  float gate = 0.f, nw = 0.f;                    // dv <= STEP_T (host check)
+  float gate = 0.f, nw = 0.f;                    // dv <= NT (launch_step)
   if (tid < dv) {
     gate = (float)reinterpret_cast<const T*>(a.gate)[row * a.ld + (long long)h * dv + tid];
     nw = a.norm_w[tid];
@@ -134,7 +134,7 @@ __global__ void __launch_bounds__(STEP_T) delta_step_kernel(const UbDeltaArgs a,
     R.x += __shfl_xor_sync(0xffffffffu, R.x, o); R.y += __shfl_xor_sync(0xffffffffu, R.y, o);
     R.z += __shfl_xor_sync(0xffffffffu, R.z, o); R.w += __shfl_xor_sync(0xffffffffu, R.w, o);
   }
-  const int slot = cl >= 32 ? rg : warp, nslots = cl >= 32 ? nrg : STEP_T / 32;
+  const int slot = cl >= 32 ? rg : warp, nslots = cl >= 32 ? nrg : NT / 32;
   if (on && (cl >= 32 || lane < cl)) {
     *reinterpret_cast<float4*>(part + (slot * 2) * dv + col) = P;
     *reinterpret_cast<float4*>(part + (slot * 2 + 1) * dv + col) = R;
@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(STEP_T) delta_step_kernel(const UbDeltaArgs a,
   if (tid < dv) {
     float s = 0.f;
 #pragma unroll
-    for (int w = 0; w < STEP_T / 32; ++w) s += sc[8 + w];
+    for (int w = 0; w < NT / 32; ++w) s += sc[8 + w];
     reinterpret_cast<T*>(a.out)[row * a.ld_out + (long long)h * dv + tid] = T(o * (1.f / sqrtf(s / a.dv_real + a.eps)) * nw * silu(gate));
   }
   if (so >= 0 && on) {
@@ -181,31 +181,95 @@ template <typename T>
 static cudaError_t launch_step(const UbDeltaArgs& a, cudaStream_t st) {
   int cl = 2;
   while (cl * 4 < a.dv) cl <<= 1;                // <= 64
-  const int nrg = STEP_T / cl, need = (a.dk + nrg - 1) / nrg;
+  const int nt = a.dv <= 128 && a.dk * a.dv <= 64 * 64 ? 128 : 256;          // small states: more CTAs per SM
+  const int nrg = nt / cl, need = (a.dk + nrg - 1) / nrg;
   const size_t smem = sizeof(float) * (2 * a.dk + a.dv + 16 * a.dv + 2 * a.dv + 16);
-  const dim3 grid(a.H, a.num_seqs), block(STEP_T);
+  const dim3 grid(a.H, a.num_seqs), block(nt);
   auto go = [&](auto kern) { return launch_pdl(kern, grid, block, smem, st, a, cl); };
-  if (need <= 1) return go(delta_step_kernel<T, 1>);
-  if (need <= 4) return go(delta_step_kernel<T, 4>);
-  if (need <= 8) return go(delta_step_kernel<T, 8>);
-  if (need <= 16) return go(delta_step_kernel<T, 16>);
-  if (need <= 32) return go(delta_step_kernel<T, 32>);
-  return go(delta_step_kernel<T, 0>);
+  if (nt == 128) {
+    if (need <= 2) return go(delta_step_kernel<T, 128, 2>);
+    if (need <= 8) return go(delta_step_kernel<T, 128, 8>);
+    if (need <= 32) return go(delta_step_kernel<T, 128, 32>);
+    return go(delta_step_kernel<T, 128, 0>);
+  }
+  if (need <= 8) return go(delta_step_kernel<T, 256, 8>);
+  if (need <= 16) return go(delta_step_kernel<T, 256, 16>);
+  if (need <= 32) return go(delta_step_kernel<T, 256, 32>);
+  return go(delta_step_kernel<T, 256, 0>);
 }
 
 // ------------------------------------------------------------------------------------------------------------------------
 // portions: what the scan reads
 // ------------------------------------------------------------------------------------------------------------------------
-// workspace, per row of the launch: q and k [2 G dk], v (later o) [H dv], k.k and q.k with the tokens of the row's block
-// [G][2][16], running log decay and beta [H][2]
+// workspace, per row of the launch: q and k [2 G dk], v (later o) [H dv], the row's entries of T and W [H][2][16], e^c and
+// e^(c_end - c) [H][2]
 __device__ __forceinline__ float* ws_qk(const UbDeltaArgs& a) { return a.ws; }
 __device__ __forceinline__ float* ws_v(const UbDeltaArgs& a) { return a.ws + (long long)a.rows * 2 * a.G * a.dk; }
-__device__ __forceinline__ float* ws_gram(const UbDeltaArgs& a) { return ws_v(a) + (long long)a.rows * a.H * a.dv; }
-__device__ __forceinline__ float* ws_cb(const UbDeltaArgs& a) { return ws_gram(a) + (long long)a.rows * a.G * 2 * BT; }
+__device__ __forceinline__ float* ws_tw(const UbDeltaArgs& a) { return ws_v(a) + (long long)a.rows * a.H * a.dv; }
+__device__ __forceinline__ float* ws_gl(const UbDeltaArgs& a) { return ws_tw(a) + (long long)a.rows * a.H * 2 * BT; }
 
 constexpr int PREP_T = 256;
+constexpr int LDM = BT + 1;                      // row of a 16 x 16 matrix in shared memory
+constexpr int LDH = 2 * BT * LDM + BT;           // two of them per value head, half the banks apart from the next head's
 
-// One block of 16 tokens of one query / key head, or of one value head (units G ..).
+// Two tokens of eight neighbouring channels behind convolution and silu: channel `ch` of the rows, c8 on their own axis.
+template <typename T>
+__device__ __forceinline__ void conv_pair(const UbDeltaArgs& a, long long row, int t, int q_len, int si, int ch, int C, float (&y)[2][8]) {
+  const int m = a.taps - 1;
+#pragma unroll
+  for (int e = 0; e < 8; ++e) y[0][e] = y[1][e] = 0.f;
+  const T* w = reinterpret_cast<const T*>(a.conv) + ch;
+  auto input = [&](int tt, float (&v)[8]) {
+    if (tt >= 0 && tt < q_len) {
+      load8(reinterpret_cast<const T*>(a.qkv) + (row + tt) * a.ld + ch, v);
+    } else if (tt < 0 && si >= 0) {
+      load8(a.conv_state + ((long long)si * m + m + tt) * C + ch, v);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) v[e] = 0.f;
+    }
+  };
+  // input t - m + j meets tap j of token t and tap j - 1 of token t + 1
+  float before[8];
+#pragma unroll
+  for (int e = 0; e < 8; ++e) before[e] = 0.f;
+#pragma unroll 4
+  for (int j = 0; j <= m; ++j) {
+    float v[8], k[8];
+    input(t - m + j, v);
+    load8(w + (long long)j * C, k);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      y[0][e] = fmaf(k[e], v[e], y[0][e]);
+      y[1][e] = fmaf(before[e], v[e], y[1][e]);
+      before[e] = k[e];
+    }
+  }
+  float v[8];
+  input(t + 1, v);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) {
+    y[0][e] = silu(y[0][e]);
+    y[1][e] = silu(fmaf(before[e], v[e], y[1][e]));
+  }
+}
+
+// The last taps - 1 inputs of a portion are the sequence's state: eight channels of them.
+template <typename T>
+__device__ __forceinline__ void keep_inputs(const UbDeltaArgs& a, long long row, int q_len, int si, int so, int ch, int C) {
+  const int m = a.taps - 1;
+  for (int r = 0; r < m; ++r) {
+    const int t = q_len - m + r;
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = 0.f;
+    if (t >= 0) load8(reinterpret_cast<const T*>(a.qkv) + (row + t) * a.ld + ch, v);
+    else if (si >= 0) load8(a.conv_state + ((long long)si * m + m + t) * C + ch, v);
+    store8(a.conv_state + ((long long)so * m + r) * C + ch, v);
+  }
+}
+
+// One block of 16 tokens of one query / key head with its value heads' matrices, or (units G ..) 256 value channels.
 template <typename T>
 __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a) {
   pdl_launch_dependents();
@@ -214,90 +278,62 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
   const int unit = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int qs = a.q_start[seq], q_len = a.q_start[seq + 1] - qs, t0 = blockIdx.x * BT;
   if (t0 >= q_len) return;
-  const int n = min(BT, q_len - t0), m = a.taps - 1, dk = a.dk, dv = a.dv;
-  const bool is_qk = unit < a.G;
-  const int h = unit - a.G, C = 2 * a.G * dk + a.H * dv;
-  const int width = is_qk ? 2 * dk : dv;         // channels of this unit
+  const int n = min(BT, q_len - t0), dk = a.dk, C = 2 * a.G * dk + a.H * a.dv;
   const int si = state_row(a, a.state_in, seq), so = state_row(a, a.state_out, seq);
-  auto channel = [&](int c) { return is_qk ? (c < dk ? unit * dk + c : a.G * dk + unit * dk + (c - dk)) : 2 * a.G * dk + h * dv + c; };
-  float* in = sm;                                // [16 + m][width] inputs
-  float* y = in + (BT + m) * width;              // [16][width + 4]
-  const int ldy = width + 4;
+  const bool last = so >= 0 && t0 + n == q_len;
   const long long row = a.row0 + qs, wrow = qs;  // rows of the step / of the workspace
-  for (int i = tid; i < (n + m) * (width / 8); i += PREP_T) {
-    const int r = i / (width / 8), c = i % (width / 8) * 8, t = t0 - m + r, ch = channel(c);
-    float v[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) v[e] = 0.f;
-    if (t >= 0) load8(reinterpret_cast<const T*>(a.qkv) + (row + t) * a.ld + ch, v);
-    else if (si >= 0) load8(a.conv_state + ((long long)si * m + m + t) * C + ch, v);
-    store8(in + r * width + c, v);
-  }
-  __syncthreads();
-  if (so >= 0 && t0 + n == q_len) {              // the last inputs are the sequence's state
-    for (int i = tid; i < m * width; i += PREP_T) {
-      const int r = i / width, c = i % width;
-      a.conv_state[((long long)so * m + r) * C + channel(c)] = in[(n + r) * width + c];
+  float y[2][8];
+  if (unit >= a.G) {
+    const int c = (unit - a.G) * PREP_T + (tid % 32) * 8, t = t0 + (tid / 32) * 2;
+    if (c >= a.H * a.dv) return;
+    const int ch = 2 * a.G * dk + c;
+    if (t < q_len) {
+      conv_pair<T>(a, row, t, q_len, si, ch, C, y);
+      store8(ws_v(a) + (wrow + t) * a.H * a.dv + c, y[0]);
+      if (t + 1 < q_len) store8(ws_v(a) + (wrow + t + 1) * a.H * a.dv + c, y[1]);
     }
-  }
-  for (int c = tid; c < width; c += PREP_T) {
-    const T* w = reinterpret_cast<const T*>(a.conv) + channel(c);
-    float acc[BT];
-#pragma unroll
-    for (int r = 0; r < BT; ++r) acc[r] = 0.f;
-    for (int j = 0; j <= m; ++j) {
-      const float wj = (float)w[(long long)j * C];
-#pragma unroll
-      for (int r = 0; r < BT; ++r)
-        if (r < n) acc[r] = fmaf(wj, in[(r + j) * width + c], acc[r]);
-    }
-#pragma unroll
-    for (int r = 0; r < BT; ++r) {
-      if (r >= n) break;
-      const float s = silu(acc[r]);
-      if (is_qk) y[r * ldy + c] = s;
-      else ws_v(a)[(wrow + t0 + r) * a.H * dv + (long long)h * dv + c] = s;
-    }
-  }
-  if (!is_qk) {
-    if (warp == 0) {
-      const bool ok = lane < n;
-      const long long at = (row + t0 + lane) * a.ld + h;
-      float c = ok ? log_decay(a, (float)reinterpret_cast<const T*>(a.a)[at], h) : 0.f;
-#pragma unroll
-      for (int o = 1; o < BT; o <<= 1) {
-        const float v = __shfl_up_sync(0xffffffffu, c, o);
-        if (lane >= o) c += v;
-      }
-      if (ok) {
-        const float beta = 1.f / (1.f + expf(-(float)reinterpret_cast<const T*>(a.b)[at]));
-        *reinterpret_cast<float2*>(ws_cb(a) + ((wrow + t0 + lane) * a.H + h) * 2) = make_float2(c, beta);
-      }
-    }
+    if (last && tid < 32) keep_inputs<T>(a, row, q_len, si, so, ch, C);
     return;
   }
-  __syncthreads();
-  const float qs_ = 1.f / sqrtf((float)a.dk_real);
-  for (int i = warp; i < 2 * n; i += PREP_T / 32) {             // unit vectors: q rows, then k rows
-    const int r = i >> 1, part = i & 1;
-    float* p = y + r * ldy + part * dk;
-    float s = 0.f;
-    for (int c = lane; c < dk; c += 32) s = fmaf(p[c], p[c], s);
-    s = 1.f / sqrtf(warp_sum(s) + 1e-6f);
-    if (part == 0) s *= qs_;
-    float* dst = ws_qk(a) + (wrow + t0 + r) * 2 * a.G * dk + (long long)part * a.G * dk + (long long)unit * dk;
-    for (int c = lane; c < dk; c += 32) {
-      const float v = p[c] * s;
-      p[c] = v;
-      dst[c] = v;
+  const int ldy = dk + 4, group = a.H / a.G;
+  float* qk_s = sm;                              // [2][16][dk + 4] q, then k
+  float* mat = qk_s + 2 * BT * ldy;              // [2][16][17] k.k and q.k
+  float* work = mat + 2 * BT * LDM;              // per value head in flight: the system and the decayed q.k, [2][16][17] each
+  // lanes of one (q or k, two tokens) row pair lie side by side
+  const int nch = dk / 8;
+  int L = 1;
+  while (L < nch) L <<= 1;                       // <= 32
+  for (int task = tid / L; task < BT; task += PREP_T / L) {      // q of tokens 0, 1 | k of tokens 0, 1 | q of tokens 2, 3 | ..
+    const int part = task & 1, r = (task >> 1) * 2, c = (tid % L) * 8, t = t0 + r;
+    const bool on = c < dk && t < q_len;
+    const int ch = part * a.G * dk + unit * dk + c;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) y[0][e] = y[1][e] = 0.f;
+    if (on) conv_pair<T>(a, row, t, q_len, si, ch, C, y);
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { s0 = fmaf(y[0][e], y[0][e], s0); s1 = fmaf(y[1][e], y[1][e], s1); }
+    for (int o = L / 2; o > 0; o >>= 1) { s0 += __shfl_xor_sync(0xffffffffu, s0, o); s1 += __shfl_xor_sync(0xffffffffu, s1, o); }
+    const float f = part == 0 ? 1.f / sqrtf((float)a.dk_real) : 1.f;
+    const float f0 = f / sqrtf(s0 + 1e-6f), f1 = f / sqrtf(s1 + 1e-6f);
+    if (c < dk) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) { y[0][e] *= f0; y[1][e] = t + 1 < q_len ? y[1][e] * f1 : 0.f; }
+      store8(qk_s + (part * BT + r) * ldy + c, y[0]);
+      store8(qk_s + (part * BT + r + 1) * ldy + c, y[1]);
+      float* dst = ws_qk(a) + (wrow + t) * 2 * a.G * dk + (long long)part * a.G * dk + (long long)unit * dk + c;
+      if (t < q_len) store8(dst, y[0]);
+      if (t + 1 < q_len) store8(dst + 2LL * a.G * dk, y[1]);
     }
+    if (last && on && r == 0) keep_inputs<T>(a, row, q_len, si, so, ch, C);
   }
   __syncthreads();
-  const int i = tid / BT, j = tid % BT;          // PREP_T = 16 * 16 pairs
-  if (i < n) {
+  {
+    const int i = tid / BT, j = tid % BT;        // PREP_T = 16 * 16 pairs
     float kk = 0.f, qk = 0.f;
     if (j <= i) {
-      const float *ki = y + i * ldy + dk, *qi = y + i * ldy, *kj = y + j * ldy + dk;
+      const float *qi = qk_s + i * ldy, *ki = qk_s + (BT + i) * ldy, *kj = qk_s + (BT + j) * ldy;
+#pragma unroll 4
       for (int c = 0; c < dk; c += 4) {
         const float4 x = *reinterpret_cast<const float4*>(ki + c), q = *reinterpret_cast<const float4*>(qi + c);
         const float4 z = *reinterpret_cast<const float4*>(kj + c);
@@ -305,9 +341,57 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
         qk = fmaf(q.x, z.x, fmaf(q.y, z.y, fmaf(q.z, z.z, fmaf(q.w, z.w, qk))));
       }
     }
-    float* dst = ws_gram(a) + ((wrow + t0 + i) * a.G + unit) * 2 * BT;
-    dst[j] = j < i ? kk : 0.f;
-    dst[BT + j] = qk;
+    mat[i * LDM + j] = j < i ? kk : 0.f;
+    mat[(BT + i) * LDM + j] = qk;
+  }
+  __syncthreads();
+  // sixteen lanes per value head: lane j makes column j of T and W
+  const int half = lane / BT, j = lane % BT;
+  float* sys = work + (warp * 2 + half) * LDH;
+  for (int h0 = warp * 2; h0 < group; h0 += PREP_T / 32 * 2) {
+    const bool on = h0 + half < group;
+    const int h = unit * group + min(h0 + half, group - 1);
+    const bool tok = j < n;
+    const long long at = (row + t0 + min(j, n - 1)) * a.ld + h;
+    float c = tok ? log_decay(a, (float)reinterpret_cast<const T*>(a.a)[at], h) : 0.f;      // tokens past the end: no decay
+    const float beta = tok ? 1.f / (1.f + expf(-(float)reinterpret_cast<const T*>(a.b)[at])) : 0.f;
+#pragma unroll
+    for (int o = 1; o < BT; o <<= 1) {
+      const float v = __shfl_up_sync(0xffffffffu, c, o, BT);
+      if (j >= o) c += v;
+    }
+    const float c_end = __shfl_sync(0xffffffffu, c, BT - 1, BT);
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < BT; ++i) {
+      const float ci = __shfl_sync(0xffffffffu, c, i, BT), bi = __shfl_sync(0xffffffffu, beta, i, BT);
+      const float e = j <= i ? expf(ci - c) : 0.f;
+      sys[i * LDM + j] = bi * e * mat[i * LDM + j];
+      sys[(BT + i) * LDM + j] = e * mat[(BT + i) * LDM + j];
+    }
+    __syncwarp();
+    float x[BT];                                 // column j of the inverse, then of T
+#pragma unroll
+    for (int i = 0; i < BT; ++i) {
+      float v = i == j ? 1.f : 0.f;
+#pragma unroll
+      for (int k = 0; k < i; ++k) v = fmaf(-sys[i * LDM + k], x[k], v);
+      x[i] = v;
+    }
+#pragma unroll
+    for (int i = 0; i < BT; ++i) x[i] *= beta;
+    float* dst = ws_tw(a) + ((wrow + t0) * a.H + h) * 2 * BT + j;
+#pragma unroll
+    for (int i = 0; i < BT; ++i) {
+      float w = 0.f;
+#pragma unroll
+      for (int k = 0; k <= i; ++k) w = fmaf(sys[(BT + i) * LDM + k], x[k], w);
+      if (on && i < n) {
+        dst[(long long)i * a.H * 2 * BT] = x[i];
+        dst[(long long)i * a.H * 2 * BT + BT] = w;
+      }
+    }
+    if (on && tok) *reinterpret_cast<float2*>(ws_gl(a) + ((wrow + t0 + j) * a.H + h) * 2) = make_float2(expf(c), expf(c_end - c));
   }
 }
 
@@ -327,14 +411,13 @@ struct Scan {
   static constexpr int DK = RPL * LPG;           // rows that fit
   static constexpr int CPW = 4 * (32 / LPG);     // columns per warp
   static constexpr int COLS = CPW * SCAN_W;      // ... per CTA
+  static constexpr int GT = RPL >= 16 ? 2 : 4;   // tokens whose products with S are under way together
   struct Stage {
-    float k[BT][DK], q[BT][DK], v[BT][COLS], gram[BT][2 * BT + 4], cb[BT][2];
+    float k[BT][DK], q[BT][DK], v[BT][COLS], tw[BT][2 * BT], gl[BT][2];
   };
   struct Smem {
     Stage st[2];
-    float mat[2][BT][BT];                        // by column j: -e^(c_i - c_j) k_i.k_j (i > j), e^(c_i - c_j) q_i.k_j (i >= j)
-    float grow[BT], left[BT];                    // e^(c_i), e^(c_end - c_j)
-    float u[SCAN_W][BT][CPW];
+    float2 u[SCAN_W][BT][CPW];                   // u e^(c_end - c), twice each
   };
 };
 
@@ -370,7 +453,7 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
       S[p][0] = pack_f32x2(x.x, y.x); S[p][1] = pack_f32x2(x.y, y.y); S[p][2] = pack_f32x2(x.z, y.z); S[p][3] = pack_f32x2(x.w, y.w);
     }
   }
-  const float *qk = ws_qk(a), *gram = ws_gram(a), *cbp = ws_cb(a);
+  const float *qk = ws_qk(a), *tw = ws_tw(a), *gl = ws_gl(a);
   float* vo = ws_v(a);
   const int blocks = (q_len + BT - 1) / BT;
   auto fetch = [&](int b) {
@@ -390,14 +473,14 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
         const bool ok = t < n && cta_col + c < dv;
         cp16(&st.v[t][c], vo + (ok ? (row + t) * a.H * dv + (long long)h * dv + cta_col + c : 0), ok);
       }
-      for (int i = tid; i < BT * (2 * BT / 4); i += SCAN_W * 32) {
-        const int t = i / (2 * BT / 4), c = i % (2 * BT / 4) * 4;
-        cp16(&st.gram[t][c], gram + (t < n ? ((row + t) * a.G + g) * 2 * BT + c : 0), t < n);
+      {
+        const int t = tid / 8, c = tid % 8 * 4;  // 128 threads: 16 rows of 32
+        cp16(&st.tw[t][c], tw + (t < n ? ((row + t) * a.H + h) * 2 * BT + c : 0), t < n);
       }
-      // tokens past the end repeat the last one's decay; their k and v are zero, so they write nothing
+      // tokens past the end repeat the last one's decay; their k, v and matrix rows are zero, so they write nothing
       if (tid < BT) {
-        const float* p = cbp + ((row + min(tid, n - 1)) * a.H + h) * 2;
-        asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(&st.cb[tid][0])), "l"(p) : "memory");
+        const float* p = gl + ((row + min(tid, n - 1)) * a.H + h) * 2;
+        asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(&st.gl[tid][0])), "l"(p) : "memory");
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -409,100 +492,108 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
     fetch(b + 1);
     const typename C::Stage& st = s.st[b & 1];
     const int t0 = b * BT, n = min(BT, q_len - t0);
-    const float c_end = st.cb[BT - 1][0];
-    for (int i = tid; i < BT * BT; i += SCAN_W * 32) {
-      const int r = i % BT, j = i / BT;
-      const float e = j <= r ? expf(st.cb[r][0] - st.cb[j][0]) : 0.f;
-      s.mat[0][j][r] = j < r ? -e * st.gram[r][j] : 0.f;
-      s.mat[1][j][r] = j <= r ? e * st.gram[r][BT + j] : 0.f;
-    }
-    if (tid < BT) s.grow[tid] = expf(st.cb[tid][0]);
-    else if (tid < 2 * BT) s.left[tid - BT] = expf(c_end - st.cb[tid - BT][0]);
-    __syncthreads();
 
-    // products of all tokens with the entering state
+    // products of all tokens with the entering state: x (of the tokens' k) or e^c S^T q
     float val[BT];
 #pragma unroll
-    for (int t = 0; t < BT; ++t) {
-      uint64_t P[4] = {0ull, 0ull, 0ull, 0ull}, R[4] = {0ull, 0ull, 0ull, 0ull};
+    for (int tg = 0; tg < BT; tg += C::GT) {
+      uint64_t P[C::GT][4], R[C::GT][4];
 #pragma unroll
-      for (int x = 0; x < RPL / 4; ++x) {
-        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&st.k[t][4 * (l + LPG * x)]);
-        const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(&st.q[t][4 * (l + LPG * x)]);
+      for (int t = 0; t < C::GT; ++t)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) P[t][c] = R[t][c] = 0ull;
+#pragma unroll
+      for (int x = 0; x < RPL / 4; ++x)
+#pragma unroll
+        for (int t = 0; t < C::GT; ++t) {
+          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&st.k[tg + t][4 * (l + LPG * x)]);
+          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(&st.q[tg + t][4 * (l + LPG * x)]);
+#pragma unroll
+          for (int c = 0; c < 4; ++c) {
+            P[t][c] = fma_f32x2(k.x, S[2 * x][c], P[t][c]);
+            R[t][c] = fma_f32x2(q.x, S[2 * x][c], R[t][c]);
+            P[t][c] = fma_f32x2(k.y, S[2 * x + 1][c], P[t][c]);
+            R[t][c] = fma_f32x2(q.y, S[2 * x + 1][c], R[t][c]);
+          }
+        }
+      // each step halves what a lane still carries: 4 + 2 + 1 shuffles per token, then whole sums over lanes that hold the same
+      float f[C::GT][4], z[C::GT];
+#pragma unroll
+      for (int t = 0; t < C::GT; ++t)
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          P[c] = fma_f32x2(k.x, S[2 * x][c], P[c]);
-          R[c] = fma_f32x2(q.x, S[2 * x][c], R[c]);
-          P[c] = fma_f32x2(k.y, S[2 * x + 1][c], P[c]);
-          R[c] = fma_f32x2(q.y, S[2 * x + 1][c], R[c]);
+          float p0, p1, r0, r1;
+          unpack_f32x2(P[t][c], p0, p1);
+          unpack_f32x2(R[t][c], r0, r1);
+          const float p = p0 + p1, r = r0 + r1;
+          f[t][c] = (type ? r : p) + __shfl_xor_sync(0xffffffffu, type ? p : r, LPG / 2);
         }
-      }
-      float p[4], r[4];
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        float lo, hi;
-        unpack_f32x2(P[c], lo, hi);
-        p[c] = lo + hi;
-        unpack_f32x2(R[c], lo, hi);
-        r[c] = lo + hi;
-      }
-      // each step halves what a lane still carries: 4 + 2 + 1 shuffles, then whole sums over lanes that hold the same
-      float f[4];
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const float mine = type ? r[c] : p[c], other = type ? p[c] : r[c];
-        f[c] = mine + __shfl_xor_sync(0xffffffffu, other, LPG / 2);
-      }
       const bool b1 = mycol & 2, b0 = mycol & 1;
-      float f0 = b1 ? f[2] : f[0], f1 = b1 ? f[3] : f[1];
-      f0 += __shfl_xor_sync(0xffffffffu, b1 ? f[0] : f[2], LPG / 4);
-      f1 += __shfl_xor_sync(0xffffffffu, b1 ? f[1] : f[3], LPG / 4);
-      float z = b0 ? f1 : f0;
-      z += __shfl_xor_sync(0xffffffffu, b0 ? f0 : f1, LPG / 8);
 #pragma unroll
-      for (int o = LPG / 16; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-      z *= s.grow[t];
-      val[t] = type ? z : st.v[t][wcol + mycol] - z;
+      for (int t = 0; t < C::GT; ++t) {
+        f[t][0] = (b1 ? f[t][2] : f[t][0]) + __shfl_xor_sync(0xffffffffu, b1 ? f[t][0] : f[t][2], LPG / 4);
+        f[t][1] = (b1 ? f[t][3] : f[t][1]) + __shfl_xor_sync(0xffffffffu, b1 ? f[t][1] : f[t][3], LPG / 4);
+      }
+#pragma unroll
+      for (int t = 0; t < C::GT; ++t) z[t] = (b0 ? f[t][1] : f[t][0]) + __shfl_xor_sync(0xffffffffu, b0 ? f[t][0] : f[t][1], LPG / 8);
+#pragma unroll
+      for (int o = LPG / 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int t = 0; t < C::GT; ++t) z[t] += __shfl_xor_sync(0xffffffffu, z[t], o);
+#pragma unroll
+      for (int t = 0; t < C::GT; ++t) {
+        z[t] *= st.gl[tg + t][0];
+        val[tg + t] = type ? z[t] : st.v[tg + t][wcol + mycol] - z[t];
+      }
     }
-    // the triangular solve: u_j is final when its turn comes
-    const int from = lane & ~(LPG / 2);          // the lane of this column that solves
+    // u = T x in the lanes that hold x, o = e^c S^T q + W x in the others
+    float x[BT];
 #pragma unroll
     for (int j = 0; j < BT; ++j) {
-      const float u = __shfl_sync(0xffffffffu, val[j] * st.cb[j][1], from);
-      if (type == 0 && rep == 0) s.u[warp][j][grp * 4 + mycol] = u * s.left[j];
-#pragma unroll
-      for (int x = j / 4; x < BT / 4; ++x) {
-        const float4 m = *reinterpret_cast<const float4*>(&s.mat[type][j][4 * x]);
-        if (4 * x >= j) val[4 * x] = fmaf(m.x, u, val[4 * x]);
-        if (4 * x + 1 >= j) val[4 * x + 1] = fmaf(m.y, u, val[4 * x + 1]);
-        if (4 * x + 2 >= j) val[4 * x + 2] = fmaf(m.z, u, val[4 * x + 2]);
-        if (4 * x + 3 >= j) val[4 * x + 3] = fmaf(m.w, u, val[4 * x + 3]);
-      }
+      x[j] = __shfl_sync(0xffffffffu, val[j], lane & ~(LPG / 2));
+      if (type == 0) val[j] = 0.f;
     }
-    if (type == 1 && rep == 0 && on) {
-      float* dst = vo + ((long long)qs + t0) * a.H * dv + (long long)h * dv + col + mycol;
 #pragma unroll
-      for (int t = 0; t < BT; ++t)
-        if (t < n) dst[(long long)t * a.H * dv] = val[t];
+    for (int i = 0; i < BT; ++i)
+#pragma unroll
+      for (int j4 = 0; j4 <= i / 4; ++j4) {      // beyond the diagonal the rows hold zeros
+        const float4 m = *reinterpret_cast<const float4*>(&st.tw[i][type * BT + 4 * j4]);
+        val[i] = fmaf(m.x, x[4 * j4], fmaf(m.y, x[4 * j4 + 1], fmaf(m.z, x[4 * j4 + 2], fmaf(m.w, x[4 * j4 + 3], val[i]))));
+      }
+    if (rep == 0) {
+      if (type == 0) {
+#pragma unroll
+        for (int t = 0; t < BT; ++t) {
+          const float u = val[t] * st.gl[t][1];
+          s.u[warp][t][grp * 4 + mycol] = make_float2(u, u);
+        }
+      } else if (on) {
+        float* dst = vo + ((long long)qs + t0) * a.H * dv + (long long)h * dv + col + mycol;
+#pragma unroll
+        for (int t = 0; t < BT; ++t)
+          if (t < n) dst[(long long)t * a.H * dv] = val[t];
+      }
     }
     __syncwarp();
     // the state behind the block
-    const uint64_t fade = pack_f32x2(s.grow[BT - 1], s.grow[BT - 1]);
+    const float end = st.gl[BT - 1][0];
+    const uint64_t fade = pack_f32x2(end, end);
 #pragma unroll
     for (int p = 0; p < RPL / 2; ++p)
 #pragma unroll
       for (int c = 0; c < 4; ++c) S[p][c] = mul_f32x2(S[p][c], fade);
 #pragma unroll
     for (int j = 0; j < BT; ++j) {
-      const float4 u4 = *reinterpret_cast<const float4*>(&s.u[warp][j][grp * 4]);
-      const uint64_t u[4] = {pack_f32x2(u4.x, u4.x), pack_f32x2(u4.y, u4.y), pack_f32x2(u4.z, u4.z), pack_f32x2(u4.w, u4.w)};
+      const ulonglong2 u01 = *reinterpret_cast<const ulonglong2*>(&s.u[warp][j][grp * 4]);
+      const ulonglong2 u23 = *reinterpret_cast<const ulonglong2*>(&s.u[warp][j][grp * 4 + 2]);
+      const uint64_t u[4] = {u01.x, u01.y, u23.x, u23.y};
 #pragma unroll
-      for (int x = 0; x < RPL / 4; ++x) {
-        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&st.k[j][4 * (l + LPG * x)]);
+      for (int x2 = 0; x2 < RPL / 4; ++x2) {
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&st.k[j][4 * (l + LPG * x2)]);
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
-          S[2 * x][c] = fma_f32x2(k.x, u[c], S[2 * x][c]);
-          S[2 * x + 1][c] = fma_f32x2(k.y, u[c], S[2 * x + 1][c]);
+          S[2 * x2][c] = fma_f32x2(k.x, u[c], S[2 * x2][c]);
+          S[2 * x2 + 1][c] = fma_f32x2(k.y, u[c], S[2 * x2 + 1][c]);
         }
       }
     }
@@ -523,29 +614,29 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
 }
 
 // ------------------------------------------------------------------------------------------------------------------------
-// portions: norm and gate of the outputs, a warp per row and head
+// portions: norm and gate of the outputs, eight columns per lane
 // ------------------------------------------------------------------------------------------------------------------------
 template <typename T>
-__global__ void __launch_bounds__(256) delta_finish_kernel(const UbDeltaArgs a) {
+__global__ void __launch_bounds__(256) delta_finish_kernel(const UbDeltaArgs a, const int L /* lanes per row and head */) {
   pdl_launch_dependents();
   pdl_wait();
-  const long long i = blockIdx.x * 8LL + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31, dv = a.dv;
-  if (i >= (long long)a.rows * a.H) return;
+  const int dv = a.dv, c = (threadIdx.x % L) * 8;
+  const long long i = (long long)blockIdx.x * (256 / L) + threadIdx.x / L;
+  const bool on = i < (long long)a.rows * a.H && c < dv;
   const long long t = i / a.H;
-  const int h = int(i % a.H), c = lane * 8;
+  const int h = int(i % a.H);
   float o[8], g[8], w[8], sq = 0.f;
 #pragma unroll
   for (int e = 0; e < 8; ++e) o[e] = 0.f;
-  if (c < dv) {
+  if (on) {
     load8(ws_v(a) + t * a.H * dv + (long long)h * dv + c, o);
     load8(reinterpret_cast<const T*>(a.gate) + (a.row0 + t) * a.ld + (long long)h * dv + c, g);
     load8(a.norm_w + c, w);
   }
 #pragma unroll
   for (int e = 0; e < 8; ++e) sq = fmaf(o[e], o[e], sq);
-  sq = warp_sum(sq);
-  if (c >= dv) return;
+  for (int x = L / 2; x > 0; x >>= 1) sq += __shfl_xor_sync(0xffffffffu, sq, x);
+  if (!on) return;
   const float r = 1.f / sqrtf(sq / a.dv_real + a.eps);
 #pragma unroll
   for (int e = 0; e < 8; ++e) o[e] *= r * w[e] * silu(g[e]);
@@ -565,13 +656,14 @@ static cudaError_t launch_scan(const UbDeltaArgs& a, cudaStream_t st) {
 
 template <typename T>
 static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
-  const int width = 2 * a.dk > a.dv ? 2 * a.dk : a.dv;
-  const size_t smem = sizeof(float) * ((size_t)(BT + a.taps - 1) * width + (size_t)BT * (2 * a.dk + 4));
+  const int group = a.H / a.G;
+  const size_t smem = sizeof(float) * (2 * BT * (a.dk + 4) + 2 * BT * LDM + (size_t)(group < PREP_T / BT ? (group + 1) / 2 * 2 : PREP_T / BT) * LDH);
+  const dim3 grid((a.max_q + BT - 1) / BT, a.G + (a.H * a.dv + PREP_T - 1) / PREP_T, a.num_seqs);
   if (smem > 48 * 1024) {
     const cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
   }
-  cudaError_t e = launch_pdl(delta_prep_kernel<T>, dim3((a.max_q + BT - 1) / BT, a.G + a.H, a.num_seqs), dim3(PREP_T), smem, st, a);
+  cudaError_t e = launch_pdl(delta_prep_kernel<T>, grid, dim3(PREP_T), smem, st, a);
   if (e != cudaSuccess) return e;
   // few lanes per column keep the reductions short, many of them spread a small launch over the device
   const long long cols = (long long)a.num_seqs * a.H * a.dv;
@@ -583,14 +675,17 @@ static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
   else if (a.dk <= 128) e = lanes <= 8 ? launch_scan<16, 8>(a, st) : lanes <= 16 ? launch_scan<8, 16>(a, st) : launch_scan<4, 32>(a, st);
   else e = lanes <= 16 ? launch_scan<16, 16>(a, st) : launch_scan<8, 32>(a, st);
   if (e != cudaSuccess) return e;
-  return launch_pdl(delta_finish_kernel<T>, dim3((unsigned)(((long long)a.rows * a.H + 7) / 8)), dim3(256), (size_t)0, st, a);
+  int L = 1;
+  while (L * 8 < a.dv) L <<= 1;
+  const long long per = 256 / L;
+  return launch_pdl(delta_finish_kernel<T>, dim3((unsigned)(((long long)a.rows * a.H + per - 1) / per)), dim3(256), (size_t)0, st, a, L);
 }
 
 }  // namespace delta
 }  // namespace ub
 
 extern "C" long long ub_delta_workspace_floats(int rows, int H, int G, int dk, int dv) {
-  return (long long)rows * (2LL * G * dk + (long long)H * dv + 2LL * ub::delta::BT * G + 2LL * H);
+  return (long long)rows * (2LL * G * dk + (long long)H * dv + 2LL * ub::delta::BT * H + 2LL * H);
 }
 
 extern "C" int ub_delta_mixer(const UbDeltaArgs* a, void* stream) {
@@ -610,7 +705,7 @@ extern "C" int ub_delta_mixer(const UbDeltaArgs* a, void* stream) {
     if (a->rows != a->num_seqs) return -6;
     e = a->f32 ? delta::launch_step<float>(*a, st) : delta::launch_step<__nv_bfloat16>(*a, st);
   } else {
-    if (a->ws == nullptr || a->G + a->H > 65535) return -6;
+    if (a->ws == nullptr || a->G + a->H * a->dv / 256 + 1 > 65535) return -6;
     e = a->f32 ? delta::launch_portions<float>(*a, st) : delta::launch_portions<__nv_bfloat16>(*a, st);
   }
   if (e == cudaSuccess) e = cudaGetLastError();

@@ -17,28 +17,29 @@ namespace ub {
 constexpr int MOE_MAX_E = 256;
 constexpr int MOE_MAX_K = 16;
 
-// Logits of TB tokens per CTA of 128 threads (from x and the router matrix, or given), then top-k and weights, one warp
-// per token.  XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.  A warp
+// Logits of TB tokens per CTA (from x and the router matrix, or given), then top-k and weights, one warp per token.  A CTA has
+// a warp for every four router rows, up to sixteen.  XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.  A warp
 // takes four experts at a time for all TB tokens, so a router row is read once per TB tokens and an activation once per
 // four experts.  A logit's sum runs over h in the same order whatever TB is.
 template <typename XT, typename WT, int TB>
-__global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) {
+__global__ void __launch_bounds__(512) moe_route_kernel(const UbMoeRouteArgs a) {
   constexpr int EB = 4;
   __shared__ float logits_s[TB][MOE_MAX_E + 1];   // the last one in use may be the gate of the always-on expert
   __shared__ float choice_s[TB][MOE_MAX_E];
-  const int t0 = blockIdx.x * TB, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = blockIdx.x * TB, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
   const int E = a.E, K = a.K;
   if (a.router_w != nullptr) {
     const XT* x = reinterpret_cast<const XT*>(a.x);
     const WT* w = reinterpret_cast<const WT*>(a.router_w);
     const int rows = E + (a.shared_w != nullptr);
     const WT* sw = reinterpret_cast<const WT*>(a.shared_w);
-    for (int e0 = warp * EB; e0 < rows; e0 += 4 * EB) {
+    for (int e0 = warp * EB; e0 < rows; e0 += nw * EB) {
       float acc[TB][EB];
 #pragma unroll
       for (int i = 0; i < TB; ++i)
 #pragma unroll
         for (int j = 0; j < EB; ++j) acc[i][j] = 0.f;
+#pragma unroll 2
       for (int h = lane * 8; h < a.H; h += 256) {
         float ws[EB][8];
 #pragma unroll
@@ -69,7 +70,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
         }
     }
   } else {
-    for (int i = threadIdx.x; i < TB * E; i += 128) {
+    for (int i = threadIdx.x; i < TB * E; i += blockDim.x) {
       const int t = t0 + i / E, e = i % E;
       if (t >= a.T) continue;
       logits_s[i / E][e] = a.logits_f32 ? reinterpret_cast<const float*>(a.logits)[(long long)t * E + e]
@@ -77,7 +78,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const UbMoeRouteArgs a) 
     }
   }
   __syncthreads();
-  for (int i = warp; i < TB; i += 4) {
+  for (int i = warp; i < TB; i += nw) {
     const int t = t0 + i;
     if (t >= a.T) continue;                       // warp-uniform
     const float* logit = logits_s[i];
@@ -241,8 +242,10 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const UbMoeRouteArgs a) 
 
 template <typename XT, typename WT>
 static void launch_route(const UbMoeRouteArgs& a, cudaStream_t st) {
-  if (a.T >= 148 * 8) moe_route_kernel<XT, WT, 4><<<(a.T + 3) / 4, 128, 0, st>>>(a);
-  else moe_route_kernel<XT, WT, 1><<<a.T, 128, 0, st>>>(a);
+  const int rows = a.router_w != nullptr ? a.E + (a.shared_w != nullptr) : 16;
+  const int nt = 32 * (rows <= 16 ? 4 : rows > 60 ? 16 : (rows + 3) / 4);
+  if (a.T >= 148 * 8) moe_route_kernel<XT, WT, 4><<<(a.T + 3) / 4, nt, 0, st>>>(a);
+  else moe_route_kernel<XT, WT, 1><<<a.T, nt, 0, st>>>(a);
 }
 
 // out[slot, :] = x[sorted_rows[slot] / K, :]; V 16-byte vectors per 8 bf16 / 4 fp32 elements

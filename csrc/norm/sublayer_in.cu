@@ -451,7 +451,7 @@ __global__ void __launch_bounds__(512) sublayer_step_kernel(const UbSublayerInAr
 
 // Rows that depend on nothing but themselves.
 template <typename T, int CH>
-__global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInArgs a) {
+__global__ void __launch_bounds__(CH == 1 ? 512 : 256, CH == 1 ? 2 : 1) sublayer_alone_kernel(const UbSublayerInArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   __shared__ float red[2][16];
@@ -468,7 +468,6 @@ __global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInA
   const T* yx = reinterpret_cast<const T*>(a.yx);
   const float gate = a.y_gate != nullptr ? a.y_gate[src] : 1.f;
   float x[CH][8], f[CH][8];
-  Raw8<T> wy8[CH], wn8[CH];
   float sq = 0.f;
 #pragma unroll
   for (int c = 0; c < CH; ++c) {
@@ -477,34 +476,34 @@ __global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInA
     for (int e = 0; e < 8; ++e) x[c][e] = f[c][e] = 0.f;
     if (ch >= nch) continue;
     load8(a.x + src * a.Hp + ch * 8, x[c]);
-    wn8[c].load(reinterpret_cast<const T*>(a.wn) + ch * 8);
     if (y == nullptr && yx == nullptr) continue;
-    wy8[c].load(reinterpret_cast<const T*>(a.wy) + ch * 8);
     if (y != nullptr) {
       load8(y + src * a.Hp + ch * 8, f[c]);
 #pragma unroll
       for (int e = 0; e < 8; ++e) f[c][e] *= gate;
     }
     for (int k0 = 0; yx != nullptr && k0 < a.K; k0 += 4) {         // four experts' rows are under way at a time
-      float g[4][8], w[4];
+      Raw8<T> g[4];
+      float w[4];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         w[j] = 0.f;
-#pragma unroll
-        for (int e = 0; e < 8; ++e) g[j][e] = 0.f;
-        if (k0 + j >= a.K) continue;
-        const int slot = __ldg(a.row_slot + src * a.K + k0 + j);
+        const int slot = k0 + j < a.K ? __ldg(a.row_slot + src * a.K + k0 + j) : -1;
         if (slot >= a.slots) {
           set_err(a.err, ERR_BOUNDS, blockIdx.x);
         } else if (slot >= 0) {
           w[j] = __ldg(a.topk_w + src * a.K + k0 + j);
-          load8(yx + (long long)slot * a.Hp + ch * 8, g[j]);
+          g[j].load(yx + (long long)slot * a.Hp + ch * 8);
         }
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j)
+      for (int j = 0; j < 4; ++j) {
+        if (w[j] == 0.f) continue;               // uniform
+        float v[8];
+        g[j].get(v);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) f[c][e] = fmaf(w[j], g[j][e], f[c][e]);
+        for (int e = 0; e < 8; ++e) f[c][e] = fmaf(w[j], v[e], f[c][e]);
+      }
     }
 #pragma unroll
     for (int e = 0; e < 8; ++e) sq += f[c][e] * f[c][e];           // pad columns are zero
@@ -517,7 +516,7 @@ __global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInA
       const int ch = threadIdx.x + c * blockDim.x;
       if (ch >= nch) continue;
       float w[8];
-      wy8[c].get(w);
+      load8(reinterpret_cast<const T*>(a.wy) + ch * 8, w);
 #pragma unroll
       for (int e = 0; e < 8; ++e) x[c][e] += f[c][e] * r * (a.w_off + w[e]);
       if (a.x_out != nullptr) store8(a.x_out + (long long)blockIdx.x * a.Hp + ch * 8, x[c]);
@@ -534,7 +533,7 @@ __global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInA
     const int ch = threadIdx.x + c * blockDim.x;
     if (ch >= nch) continue;
     float w[8];
-    wn8[c].get(w);
+    load8(reinterpret_cast<const T*>(a.wn) + ch * 8, w);
 #pragma unroll
     for (int e = 0; e < 8; ++e) x[c][e] *= r * (a.w_off + w[e]);
     store8(reinterpret_cast<T*>(a.out) + (long long)blockIdx.x * a.Hp + ch * 8, x[c]);
@@ -544,12 +543,10 @@ __global__ void __launch_bounds__(512) sublayer_alone_kernel(const UbSublayerInA
 template <typename T>
 static cudaError_t launch_alone(const UbSublayerInArgs& a, cudaStream_t st) {
   const int nch = a.Hp / 8;
-  const int threads = nch >= 512 ? 512 : (nch + 31) / 32 * 32;
-  const int ch = (nch + threads - 1) / threads;
-  const dim3 grid(a.n_rows), block(threads);
-  if (ch <= 1) return launch_pdl(sublayer_alone_kernel<T, 1>, grid, block, (size_t)0, st, a);
-  if (ch <= 2) return launch_pdl(sublayer_alone_kernel<T, 2>, grid, block, (size_t)0, st, a);
-  return launch_pdl(sublayer_alone_kernel<T, 4>, grid, block, (size_t)0, st, a);
+  const dim3 grid(a.n_rows);
+  if (nch <= 512) return launch_pdl(sublayer_alone_kernel<T, 1>, grid, dim3((nch + 31) / 32 * 32), (size_t)0, st, a);
+  if (nch <= 1024) return launch_pdl(sublayer_alone_kernel<T, 4>, grid, dim3(256), (size_t)0, st, a);
+  return launch_pdl(sublayer_alone_kernel<T, 8>, grid, dim3(256), (size_t)0, st, a);
 }
 
 template <typename T>

@@ -1,5 +1,5 @@
 """Prefill and decode throughput of one design beside the closest existing family at equal size, and the same
-comparison kernel by kernel (``python bench.py --design gekapel|nipulorn [--design-kernels]``).
+comparison kernel by kernel (``python bench.py --design gekapel|nipulorn|bakasun [--design-kernels]``).
 
 Both models are random-weight stacks of a few layers with a real model's layer sizes, run by the same
 ``GpuModelRunner`` steps that serve requests: a prefill step is one batch of whole prompts, a decode step one token of
@@ -17,6 +17,10 @@ Nipulorn's parts have two nearest relatives.  Whole steps are set beside Llama, 
 runner, with its feed-forward as wide as makes the parameters equal; the recurrence is set beside RWKV-6's kernel (a model
 of the whole-model path) at the same heads, tokens and state.  Arithmetic that is fp32 by design counts against the FMA
 rate of the device instead of the matrix rate.
+
+Bakasun's steps are set beside DeepSeek-MoE with Mistral's sliding window (the same gated experts and always-on expert, windowed
+attention in every layer), its experts as wide as makes the parameters equal; its gated delta rule is set beside Nipulorn's
+recurrence at the same heads, tokens and state.
 """
 from __future__ import annotations
 
@@ -28,7 +32,7 @@ import torch
 
 from ..engine.runner import GpuModelRunner, RunnerWeights, StepBatch
 from ..models import configs as C
-from ..models.families import GekapelModel, NipulornModel
+from ..models.families import BakasunModel, GekapelModel, NipulornModel
 from ..models.spec import DecoderSpec, MoESpec
 from ..ops import cuda_ops as K
 from .microbench import _peaks, time_ms
@@ -105,8 +109,42 @@ def llama_spec(z: dict) -> DecoderSpec:
                        intermediate_size=ff, max_position_embeddings=8192, tie_embeddings=True)
 
 
+# width, attention (heads, kv heads, size of a head, window), delta rule (heads, query / key heads, size), experts, expert width,
+# shared width, vocabulary, layers (attention, two with both mixers, attention; a mixture of experts in each)
+BAKASUN_SIZES = {
+    "1k": dict(width=1024, heads=16, kv=4, dim=64, window=256, dh=16, dg=8, dd=64, experts=64, top=8, ff=256, shared=512, vocab=32000, layers=4),
+    "2k": dict(width=2048, heads=16, kv=4, dim=128, window=512, dh=16, dg=8, dd=128, experts=32, top=4, ff=1024, shared=2048, vocab=32000, layers=4),
+    "4k": dict(width=4096, heads=32, kv=8, dim=128, window=1024, dh=32, dg=16, dd=128, experts=16, top=2, ff=4096, shared=4096, vocab=32000, layers=4),
+}
+
+
+def bakasun_spec(z: dict) -> DecoderSpec:
+    attn = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "mask": {"size": z["window"]},
+            "rot": {"base": 10000.0, "dims": z["dim"]}, "scale": z["dim"] ** -0.5}
+    left = dict(attn, softcap=30.0, rot={"base": 10000.0, "dims": z["dim"] // 2, "scaling": {"factor": 4.0}})
+    right = {"heads": z["dh"], "kv_heads": z["dg"], "dim": z["dd"], "vdim": z["dd"], "conv": 4}
+    mlp = {"kind": "moe", "router": {"experts": z["experts"], "top": z["top"], "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": z["ff"]}, "shared": {"ff": z["shared"]}}
+    both = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.8}
+    layers = [{"type": "parallel", "mixer": both, "mlp": mlp} if i % 4 in (1, 2) else {"type": "attention", "mixer": attn, "mlp": mlp}
+              for i in range(z["layers"])]
+    return BakasunModel.spec_from_config(C.BakasunConfig(vocab_size=z["vocab"], hidden_size=z["width"], num_hidden_layers=z["layers"],
+                                                         layers=layers))
+
+
+def windowed_moe_spec(z: dict) -> DecoderSpec:
+    """As many parameters in the layers, in layers of windowed attention and a mixture of experts."""
+    H, n = z["width"], z["layers"]
+    delta = n // 2 * H * z["dd"] * (2 * z["dg"] + 3 * z["dh"])
+    ff = z["ff"] + delta // (n * 3 * H * (z["experts"] + z["shared"] // z["ff"])) // 8 * 8
+    return DecoderSpec(vocab_size=z["vocab"], hidden_size=H, num_layers=n, num_heads=z["heads"], num_kv_heads=z["kv"], head_dim=z["dim"],
+                       intermediate_size=ff, max_position_embeddings=8192, window=z["window"],
+                       moe=MoESpec(num_experts=z["experts"], top_k=z["top"], intermediate_size=ff, num_shared_experts=z["shared"] // z["ff"]))
+
+
 DESIGNS = {"gekapel": (SIZES, {"gekapel": gekapel_spec, "deepseek_moe + window": closest_spec}),
-           "nipulorn": (NIPULORN_SIZES, {"nipulorn": nipulorn_spec, "llama": llama_spec})}
+           "nipulorn": (NIPULORN_SIZES, {"nipulorn": nipulorn_spec, "llama": llama_spec}),
+           "bakasun": (BAKASUN_SIZES, {"bakasun": bakasun_spec, "deepseek_moe + window": windowed_moe_spec})}
 FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12      # FMA pipe at the maximum clock
 
 
@@ -159,7 +197,7 @@ def step_ms(runner: GpuModelRunner, b: StepBatch, iters: int = 20, warmup: int =
 # kernel by kernel
 # ------------------------------------------------------------------------------------------------
 RECORDED = ("gemm_tn", "grouped_gemm", "norm", "residual_norm", "row_norm", "embed_residual", "embed_gather", "rope_kv_append",
-            "attn_decode", "attn_prefill", "moe_route", "moe_gather", "moe_combine", "sample", "sublayer_in", "wkv_mixer",
+            "attn_decode", "attn_prefill", "moe_route", "moe_gather", "moe_combine", "sample", "sublayer_in", "wkv_mixer", "delta_mixer",
             "gemm_stacked", "latent_rows", "latent_rotate", "gemm_heads", "attn_latent", "latent_gather", "attn_expanded")
 
 
@@ -200,6 +238,14 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
     pairs_all = sum(q * n - q * (q - 1) // 2 for q, n in zip(q_lens, b.seq_lens))
     if name == "sublayer_in":
         x, parts = a[0], a[1]
+        if kw.get("conv") is None and kw.get("mu") is None:
+            y, ex = kw.get("y"), kw.get("experts")
+            if kw.get("rows") is not None:
+                n = r.shape[0] / x.shape[0]
+                k = kw["routing"].K if ex is not None else 0
+                return "final norm", int(n * (_nbytes(x, y) + k * _nbytes(y if y is not None else x)) + _nbytes(r)), 0.0
+            return ("norms" + (" + expert sum" if ex is not None else ""),
+                    _nbytes(x, y, ex, r[1]) + (_nbytes(x) if y is not None or ex is not None else 0), 0.0)
         live = sum(p.n for p in parts)
         state = sum(2 * live * t[0].numel() * 4 for t in (kw.get("conv_state"), kw.get("shift_state")) if t is not None)
         return (f"norms + conv" + (" + mixes" if kw.get("mu") is not None else ""),
@@ -210,6 +256,15 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
         live = sum(p.n for p in parts)
         reads = live if b.num_decode else 0              # prompts start from nothing
         return "wkv", _nbytes(rkvg, ww, r) + 4 * per * (live + reads), 0.0, 5.0 * rkvg.shape[1] * per
+    if name == "delta_mixer":
+        proj, state, parts = a[0], a[7], a[8]
+        per, conv = state[0].numel(), a[6][0].numel() if a[6] is not None else 0
+        H = state.shape[1]
+        used = a[2].shape[1] + H * state.shape[3] + 2 * H
+        live = sum(p.n for p in parts)
+        reads = live if b.num_decode else 0              # prompts start from nothing
+        return ("delta rule", proj.shape[0] * used * proj.element_size() + _nbytes(r) + 4 * (per + conv) * (live + reads), 0.0,
+                6.0 * proj.shape[0] * per)
     if name == "gemm_stacked":
         x, w = a
         return f"stacked gemm {x.shape[0]}x[{x.shape[1]}x{w.shape[1]}x{w.shape[2]}]", _nbytes(x, w, r), 2.0 * x.shape[1] * w.numel()
@@ -312,6 +367,23 @@ def wkv6_row(z: dict, seqs: int, tokens: int) -> dict:
     return {"kernel": "wkv6 (RWKV-6)", "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2), "fraction": round(floor / (ms * 1e3), 3)}
 
 
+def wkv_row(z: dict, seqs: int, tokens: int, decode: bool) -> dict:
+    """Nipulorn's recurrence kernel at the heads and state of a Bakasun layer's delta rule, in the units of the table above."""
+    hbm, _, _ = _peaks()
+    H, D, T = z["dh"], z["dd"], seqs * tokens
+    g = torch.Generator(device="cuda").manual_seed(1)
+    rkvg = torch.randn(4, T, H * D, generator=g, device="cuda").to(torch.bfloat16)
+    ww, u = torch.rand(T, H * D, generator=g, device="cuda") * 4 - 5, torch.randn(H, D, generator=g, device="cuda")
+    st, nw = torch.zeros(2 * seqs, H, D, D, device="cuda"), torch.ones(H * D, device="cuda")
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    si, so = i32([2 * s if decode else -1 for s in range(seqs)]), i32([2 * s + 1 for s in range(seqs)])
+    p = K.Portions(0, T, seqs, tokens, None if decode else i32([s * tokens for s in range(seqs + 1)]), si, so)
+    ms, _ = time_ms(lambda: K.wkv_mixer(rkvg, ww, u, nw, st, [p], eps=1e-5))
+    nbytes = _nbytes(rkvg, ww, rkvg[0]) + 4 * st[0].numel() * seqs * (2 if decode else 1)
+    floor = max(nbytes / (hbm * 1e9), 5.0 * T * H * D * D / (FP32_TFLOPS * 1e12)) * 1e6
+    return {"kernel": "wkv (Nipulorn)", "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2), "fraction": round(floor / (ms * 1e3), 3)}
+
+
 def main(design: str = "gekapel", sizes: Optional[List[str]] = None, kernels: bool = False) -> List[dict]:
     out = []
     table, arms = DESIGNS[design]
@@ -334,6 +406,8 @@ def main(design: str = "gekapel", sizes: Optional[List[str]] = None, kernels: bo
                         rows = kernel_rows(runner, b)
                         if design == "nipulorn" and arm != "nipulorn":
                             rows.append(wkv6_row(z, n, 1 if kind == "decode" else c))
+                        if design == "bakasun" and arm != "bakasun":
+                            rows.append(wkv_row(z, n, 1 if kind == "decode" else c, kind == "decode"))
                         for k in rows:
                             out.append({"size": size, "model": arm, "step": kind, "sequences": n, "context": c, **k})
                             print("   ", k, flush=True)
