@@ -13,7 +13,7 @@
 //
 // One token per sequence (delta_step): a CTA per head and sequence; the state passes through registers once.
 //
-// Portions: delta_prep makes q, k and v of blocks of 16 tokens and two triangular matrices per block and head; delta_scan
+// Portions: delta_prep makes q, k and v of blocks of 16 tokens, delta_solve two triangular matrices per block and head; delta_scan
 // carries the state through the blocks; delta_finish normalises and gates.  Within a block, with the running sum c of the log
 // decays, the definition above is
 //
@@ -201,12 +201,13 @@ static cudaError_t launch_step(const UbDeltaArgs& a, cudaStream_t st) {
 // ------------------------------------------------------------------------------------------------------------------------
 // portions: what the scan reads
 // ------------------------------------------------------------------------------------------------------------------------
-// workspace, per row of the launch: q and k [2 G dk], v (later o) [H dv], the row's entries of T and W [H][2][16], e^c and
-// e^(c_end - c) [H][2]
+// workspace, per row of the launch: q and k [2 G dk], v (later o) [H dv], the row's entries of T and W [H][2][16], (-e^c, e^c,
+// e^(c_end - c), 0) [H][4], k.k and q.k with the tokens of the row's block [G][2][16]
 __device__ __forceinline__ float* ws_qk(const UbDeltaArgs& a) { return a.ws; }
 __device__ __forceinline__ float* ws_v(const UbDeltaArgs& a) { return a.ws + (long long)a.rows * 2 * a.G * a.dk; }
 __device__ __forceinline__ float* ws_tw(const UbDeltaArgs& a) { return ws_v(a) + (long long)a.rows * a.H * a.dv; }
 __device__ __forceinline__ float* ws_gl(const UbDeltaArgs& a) { return ws_tw(a) + (long long)a.rows * a.H * 2 * BT; }
+__device__ __forceinline__ float* ws_gram(const UbDeltaArgs& a) { return ws_gl(a) + (long long)a.rows * a.H * 4; }
 
 constexpr int PREP_T = 256;
 constexpr int LDM = BT + 1;                      // row of a 16 x 16 matrix in shared memory
@@ -269,13 +270,13 @@ __device__ __forceinline__ void keep_inputs(const UbDeltaArgs& a, long long row,
   }
 }
 
-// One block of 16 tokens of one query / key head with its value heads' matrices, or (units G ..) 256 value channels.
+// One block of 16 tokens of one query / key head, or (units G ..) of 256 value channels.
 template <typename T>
 __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
-  const int unit = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int unit = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
   const int qs = a.q_start[seq], q_len = a.q_start[seq + 1] - qs, t0 = blockIdx.x * BT;
   if (t0 >= q_len) return;
   const int n = min(BT, q_len - t0), dk = a.dk, C = 2 * a.G * dk + a.H * a.dv;
@@ -295,10 +296,8 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
     if (last && tid < 32) keep_inputs<T>(a, row, q_len, si, so, ch, C);
     return;
   }
-  const int ldy = dk + 4, group = a.H / a.G;
+  const int ldy = dk + 4;
   float* qk_s = sm;                              // [2][16][dk + 4] q, then k
-  float* mat = qk_s + 2 * BT * ldy;              // [2][16][17] k.k and q.k
-  float* work = mat + 2 * BT * LDM;              // per value head in flight: the system and the decayed q.k, [2][16][17] each
   // lanes of one (q or k, two tokens) row pair lie side by side
   const int nch = dk / 8;
   int L = 1;
@@ -341,57 +340,72 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
         qk = fmaf(q.x, z.x, fmaf(q.y, z.y, fmaf(q.z, z.z, fmaf(q.w, z.w, qk))));
       }
     }
-    mat[i * LDM + j] = j < i ? kk : 0.f;
-    mat[(BT + i) * LDM + j] = qk;
+    if (i < n) {
+      float* dst = ws_gram(a) + ((wrow + t0 + i) * a.G + unit) * 2 * BT;
+      dst[j] = j < i ? kk : 0.f;
+      dst[BT + j] = qk;
+    }
   }
-  __syncthreads();
-  // sixteen lanes per value head: lane j makes column j of T and W
-  const int half = lane / BT, j = lane % BT;
-  float* sys = work + (warp * 2 + half) * LDH;
-  for (int h0 = warp * 2; h0 < group; h0 += PREP_T / 32 * 2) {
-    const bool on = h0 + half < group;
-    const int h = unit * group + min(h0 + half, group - 1);
-    const bool tok = j < n;
-    const long long at = (row + t0 + min(j, n - 1)) * a.ld + h;
-    float c = tok ? log_decay(a, (float)reinterpret_cast<const T*>(a.a)[at], h) : 0.f;      // tokens past the end: no decay
-    const float beta = tok ? 1.f / (1.f + expf(-(float)reinterpret_cast<const T*>(a.b)[at])) : 0.f;
+}
+
+constexpr int SOLVE_T = 128;                     // eight (block, head) pairs per CTA
+
+// T and W of a block and head: sixteen lanes, lane j makes column j of both.
+template <typename T>
+__global__ void __launch_bounds__(SOLVE_T) delta_solve_kernel(const UbDeltaArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  __shared__ float sm[SOLVE_T / BT][LDH];
+  const int seq = blockIdx.z, unit = threadIdx.x / BT, j = threadIdx.x % BT;
+  const int qs = a.q_start[seq], q_len = a.q_start[seq + 1] - qs, t0 = blockIdx.x * BT;
+  if (t0 >= q_len) return;
+  const int n = min(BT, q_len - t0), h_ = blockIdx.y * (SOLVE_T / BT) + unit, h = min(h_, a.H - 1), g = h / (a.H / a.G);
+  const bool on = h_ < a.H, tok = j < n;
+  const long long row = a.row0 + qs, wrow = qs;
+  float* sys = sm[unit];
+  const long long at = (row + t0 + min(j, n - 1)) * a.ld + h;
+  float c = tok ? log_decay(a, (float)reinterpret_cast<const T*>(a.a)[at], h) : 0.f;        // tokens past the end: no decay
+  const float beta = tok ? 1.f / (1.f + expf(-(float)reinterpret_cast<const T*>(a.b)[at])) : 0.f;
 #pragma unroll
-    for (int o = 1; o < BT; o <<= 1) {
-      const float v = __shfl_up_sync(0xffffffffu, c, o, BT);
-      if (j >= o) c += v;
+  for (int o = 1; o < BT; o <<= 1) {
+    const float v = __shfl_up_sync(0xffffffffu, c, o, BT);
+    if (j >= o) c += v;
+  }
+  const float c_end = __shfl_sync(0xffffffffu, c, BT - 1, BT);
+  const float* gram = ws_gram(a) + ((wrow + t0) * a.G + g) * 2 * BT + j;
+#pragma unroll
+  for (int i = 0; i < BT; ++i) {
+    const float ci = __shfl_sync(0xffffffffu, c, i, BT), bi = __shfl_sync(0xffffffffu, beta, i, BT);
+    const float e = j <= i && i < n ? expf(ci - c) : 0.f;
+    const float* p = gram + (long long)min(i, n - 1) * a.G * 2 * BT;
+    sys[i * LDM + j] = bi * e * p[0];
+    sys[(BT + i) * LDM + j] = e * p[BT];
+  }
+  __syncwarp();
+  float x[BT];                                   // column j of the inverse, then of T
+#pragma unroll
+  for (int i = 0; i < BT; ++i) {
+    float v = i == j ? 1.f : 0.f;
+#pragma unroll
+    for (int k = 0; k < i; ++k) v = fmaf(-sys[i * LDM + k], x[k], v);
+    x[i] = v;
+  }
+#pragma unroll
+  for (int i = 0; i < BT; ++i) x[i] *= beta;
+  float* dst = ws_tw(a) + ((wrow + t0) * a.H + h) * 2 * BT + j;
+#pragma unroll
+  for (int i = 0; i < BT; ++i) {
+    float w = 0.f;
+#pragma unroll
+    for (int k = 0; k <= i; ++k) w = fmaf(sys[(BT + i) * LDM + k], x[k], w);
+    if (on && i < n) {
+      dst[(long long)i * a.H * 2 * BT] = x[i];
+      dst[(long long)i * a.H * 2 * BT + BT] = w;
     }
-    const float c_end = __shfl_sync(0xffffffffu, c, BT - 1, BT);
-    __syncwarp();
-#pragma unroll
-    for (int i = 0; i < BT; ++i) {
-      const float ci = __shfl_sync(0xffffffffu, c, i, BT), bi = __shfl_sync(0xffffffffu, beta, i, BT);
-      const float e = j <= i ? expf(ci - c) : 0.f;
-      sys[i * LDM + j] = bi * e * mat[i * LDM + j];
-      sys[(BT + i) * LDM + j] = e * mat[(BT + i) * LDM + j];
-    }
-    __syncwarp();
-    float x[BT];                                 // column j of the inverse, then of T
-#pragma unroll
-    for (int i = 0; i < BT; ++i) {
-      float v = i == j ? 1.f : 0.f;
-#pragma unroll
-      for (int k = 0; k < i; ++k) v = fmaf(-sys[i * LDM + k], x[k], v);
-      x[i] = v;
-    }
-#pragma unroll
-    for (int i = 0; i < BT; ++i) x[i] *= beta;
-    float* dst = ws_tw(a) + ((wrow + t0) * a.H + h) * 2 * BT + j;
-#pragma unroll
-    for (int i = 0; i < BT; ++i) {
-      float w = 0.f;
-#pragma unroll
-      for (int k = 0; k <= i; ++k) w = fmaf(sys[(BT + i) * LDM + k], x[k], w);
-      if (on && i < n) {
-        dst[(long long)i * a.H * 2 * BT] = x[i];
-        dst[(long long)i * a.H * 2 * BT + BT] = w;
-      }
-    }
-    if (on && tok) *reinterpret_cast<float2*>(ws_gl(a) + ((wrow + t0 + j) * a.H + h) * 2) = make_float2(expf(c), expf(c_end - c));
+  }
+  if (on && tok) {
+    const float e = expf(c);
+    *reinterpret_cast<float4*>(ws_gl(a) + ((wrow + t0 + j) * a.H + h) * 4) = make_float4(-e, e, expf(c_end - c), 0.f);
   }
 }
 
@@ -406,6 +420,10 @@ __device__ __forceinline__ void cp16(float* dst, const float* src, bool ok) {
 }
 
 // RPL rows and four columns of S per lane, LPG lanes per column group.
+//
+// Sums over the lanes of a group are taken by halving: a lane hands over what its partner keeps.  So that this needs no
+// selection, lanes hold things in the order in which they give them away: the first operand of an odd half-group's lane is q
+// where the others' is k, and its four columns are numbered from its own one (slot s holds column s ^ own).
 template <int RPL, int LPG>
 struct Scan {
   static constexpr int DK = RPL * LPG;           // rows that fit
@@ -413,11 +431,11 @@ struct Scan {
   static constexpr int COLS = CPW * SCAN_W;      // ... per CTA
   static constexpr int GT = RPL >= 16 ? 2 : 4;   // tokens whose products with S are under way together
   struct Stage {
-    float k[BT][DK], q[BT][DK], v[BT][COLS], tw[BT][2 * BT], gl[BT][2];
+    float kq[2][BT][DK], v[2][BT][COLS], tw[BT][2 * BT], gl[BT][4];          // v[1] stays zero
   };
   struct Smem {
     Stage st[2];
-    float2 u[SCAN_W][BT][CPW];                   // u e^(c_end - c), twice each
+    float2 u[SCAN_W][2][BT][CPW];                // u e^(c_end - c), twice each; in the second copy neighbouring columns change places
   };
 };
 
@@ -434,10 +452,14 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
   const int grp = lane / LPG, l = lane % LPG, g = h / (a.H / a.G), dk = a.dk, dv = a.dv;
   const int cta_col = blockIdx.x * C::COLS, wcol = warp * C::CPW + grp * 4, col = cta_col + wcol;
   const bool on = col < dv;
-  // after the reduction a lane holds one number per token: of S^T k (even half of the group) or S^T q, for one column
+  // after the reduction a lane holds one number per token: of S^T k (even half of the group) or S^T q, for its own column
   const int type = l / (LPG / 2), mycol = (l / (LPG / 8)) & 3, rep = l % (LPG / 8);
   const int si = state_row(a, a.state_in, seq), so = state_row(a, a.state_out, seq);
   auto first_row = [&](int p) { return 4 * (l + LPG * (p >> 1)) + 2 * (p & 1); };     // of pair p
+  auto turn = [&](const float4 f) {              // columns 0 .. 3 <-> slots 0 .. 3
+    const float4 h2 = mycol & 2 ? make_float4(f.z, f.w, f.x, f.y) : f;
+    return mycol & 1 ? make_float4(h2.y, h2.x, h2.w, h2.z) : h2;
+  };
 
   uint64_t S[RPL / 2][4];
   {
@@ -447,41 +469,44 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
       float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
       const int r = first_row(p);
       if (si >= 0 && on && r < dk) {
-        x = *reinterpret_cast<const float4*>(src + (long long)r * dv);
-        y = *reinterpret_cast<const float4*>(src + (long long)(r + 1) * dv);
+        x = turn(*reinterpret_cast<const float4*>(src + (long long)r * dv));
+        y = turn(*reinterpret_cast<const float4*>(src + (long long)(r + 1) * dv));
       }
       S[p][0] = pack_f32x2(x.x, y.x); S[p][1] = pack_f32x2(x.y, y.y); S[p][2] = pack_f32x2(x.z, y.z); S[p][3] = pack_f32x2(x.w, y.w);
     }
   }
+  for (int i = tid; i < 2 * BT * C::COLS; i += SCAN_W * 32) s.st[i / (BT * C::COLS)].v[1][0][i % (BT * C::COLS)] = 0.f;
   const float *qk = ws_qk(a), *tw = ws_tw(a), *gl = ws_gl(a);
   float* vo = ws_v(a);
   const int blocks = (q_len + BT - 1) / BT;
+  // this thread's share of the copies: chunk (row, column) of k and q, of v, of the matrices, and of the decays
+  constexpr int KC = C::DK / 4, KR = SCAN_W * 32 / KC, VC = C::COLS / 4, VR = SCAN_W * 32 / VC;
+  static_assert(SCAN_W * 32 % KC == 0 && BT % KR == 0, "whole rows of k per pass");
+  const int kr = tid / KC, kc = tid % KC * 4, vr = tid / VC, vc = tid % VC * 4;
   auto fetch = [&](int b) {
     if (b < blocks) {
       typename C::Stage& st = s.st[b & 1];
       const int t0 = b * BT, n = min(BT, q_len - t0);
       const long long row = (long long)qs + t0;
-      for (int i = tid; i < BT * (C::DK / 4); i += SCAN_W * 32) {
-        const int t = i / (C::DK / 4), c = i % (C::DK / 4) * 4;
-        const bool ok = t < n && c < dk;
-        const float* p = qk + (ok ? (row + t) * 2 * a.G * dk + (long long)g * dk + c : 0);
-        cp16(&st.q[t][c], p, ok);
-        cp16(&st.k[t][c], ok ? p + (long long)a.G * dk : p, ok);
+      {
+        const float* p = qk + (row + kr) * 2 * a.G * dk + (long long)g * dk + kc;
+#pragma unroll
+        for (int i = 0; i < BT / KR; ++i, p += 2LL * KR * a.G * dk) {
+          const bool ok = kr + i * KR < n && kc < dk;
+          cp16(&st.kq[1][kr + i * KR][kc], ok ? p : qk, ok);
+          cp16(&st.kq[0][kr + i * KR][kc], ok ? p + (long long)a.G * dk : qk, ok);
+        }
       }
-      for (int i = tid; i < BT * (C::COLS / 4); i += SCAN_W * 32) {
-        const int t = i / (C::COLS / 4), c = i % (C::COLS / 4) * 4;
-        const bool ok = t < n && cta_col + c < dv;
-        cp16(&st.v[t][c], vo + (ok ? (row + t) * a.H * dv + (long long)h * dv + cta_col + c : 0), ok);
+      for (int t = vr; t < BT; t += VR) {
+        const bool ok = t < n && cta_col + vc < dv;
+        cp16(&st.v[0][t][vc], vo + (ok ? (row + t) * a.H * dv + (long long)h * dv + cta_col + vc : 0), ok);
       }
       {
         const int t = tid / 8, c = tid % 8 * 4;  // 128 threads: 16 rows of 32
         cp16(&st.tw[t][c], tw + (t < n ? ((row + t) * a.H + h) * 2 * BT + c : 0), t < n);
       }
       // tokens past the end repeat the last one's decay; their k, v and matrix rows are zero, so they write nothing
-      if (tid < BT) {
-        const float* p = gl + ((row + min(tid, n - 1)) * a.H + h) * 2;
-        asm volatile("cp.async.ca.shared.global [%0], [%1], 8;" ::"r"(smem_u32(&st.gl[tid][0])), "l"(p) : "memory");
-      }
+      if (tid < BT) cp16(&st.gl[tid][0], gl + ((row + min(tid, n - 1)) * a.H + h) * 4, true);
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
@@ -492,6 +517,7 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
     fetch(b + 1);
     const typename C::Stage& st = s.st[b & 1];
     const int t0 = b * BT, n = min(BT, q_len - t0);
+    const float *mine = &st.kq[type][0][4 * l], *theirs = &st.kq[type ^ 1][0][4 * l];
 
     // products of all tokens with the entering state: x (of the tokens' k) or e^c S^T q
     float val[BT];
@@ -503,20 +529,22 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
 #pragma unroll
         for (int c = 0; c < 4; ++c) P[t][c] = R[t][c] = 0ull;
 #pragma unroll
-      for (int x = 0; x < RPL / 4; ++x)
+      for (int x = 0; x < RPL / 4; ++x) {
+        ulonglong2 k[C::GT], q[C::GT];
 #pragma unroll
         for (int t = 0; t < C::GT; ++t) {
-          const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&st.k[tg + t][4 * (l + LPG * x)]);
-          const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(&st.q[tg + t][4 * (l + LPG * x)]);
-#pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            P[t][c] = fma_f32x2(k.x, S[2 * x][c], P[t][c]);
-            R[t][c] = fma_f32x2(q.x, S[2 * x][c], R[t][c]);
-            P[t][c] = fma_f32x2(k.y, S[2 * x + 1][c], P[t][c]);
-            R[t][c] = fma_f32x2(q.y, S[2 * x + 1][c], R[t][c]);
-          }
+          k[t] = *reinterpret_cast<const ulonglong2*>(mine + (tg + t) * C::DK + 4 * LPG * x);
+          q[t] = *reinterpret_cast<const ulonglong2*>(theirs + (tg + t) * C::DK + 4 * LPG * x);
         }
-      // each step halves what a lane still carries: 4 + 2 + 1 shuffles per token, then whole sums over lanes that hold the same
+#pragma unroll
+        for (int t = 0; t < C::GT; ++t)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) { P[t][c] = fma_f32x2(k[t].x, S[2 * x][c], P[t][c]); R[t][c] = fma_f32x2(q[t].x, S[2 * x][c], R[t][c]); }
+#pragma unroll
+        for (int t = 0; t < C::GT; ++t)
+#pragma unroll
+          for (int c = 0; c < 4; ++c) { P[t][c] = fma_f32x2(k[t].y, S[2 * x + 1][c], P[t][c]); R[t][c] = fma_f32x2(q[t].y, S[2 * x + 1][c], R[t][c]); }
+      }
       float f[C::GT][4], z[C::GT];
 #pragma unroll
       for (int t = 0; t < C::GT; ++t)
@@ -525,26 +553,21 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
           float p0, p1, r0, r1;
           unpack_f32x2(P[t][c], p0, p1);
           unpack_f32x2(R[t][c], r0, r1);
-          const float p = p0 + p1, r = r0 + r1;
-          f[t][c] = (type ? r : p) + __shfl_xor_sync(0xffffffffu, type ? p : r, LPG / 2);
+          f[t][c] = p0 + p1 + __shfl_xor_sync(0xffffffffu, r0 + r1, LPG / 2);
         }
-      const bool b1 = mycol & 2, b0 = mycol & 1;
 #pragma unroll
       for (int t = 0; t < C::GT; ++t) {
-        f[t][0] = (b1 ? f[t][2] : f[t][0]) + __shfl_xor_sync(0xffffffffu, b1 ? f[t][0] : f[t][2], LPG / 4);
-        f[t][1] = (b1 ? f[t][3] : f[t][1]) + __shfl_xor_sync(0xffffffffu, b1 ? f[t][1] : f[t][3], LPG / 4);
+        f[t][0] += __shfl_xor_sync(0xffffffffu, f[t][2], LPG / 4);
+        f[t][1] += __shfl_xor_sync(0xffffffffu, f[t][3], LPG / 4);
       }
 #pragma unroll
-      for (int t = 0; t < C::GT; ++t) z[t] = (b0 ? f[t][1] : f[t][0]) + __shfl_xor_sync(0xffffffffu, b0 ? f[t][0] : f[t][1], LPG / 8);
+      for (int t = 0; t < C::GT; ++t) z[t] = f[t][0] + __shfl_xor_sync(0xffffffffu, f[t][1], LPG / 8);
 #pragma unroll
       for (int o = LPG / 16; o > 0; o >>= 1)
 #pragma unroll
         for (int t = 0; t < C::GT; ++t) z[t] += __shfl_xor_sync(0xffffffffu, z[t], o);
 #pragma unroll
-      for (int t = 0; t < C::GT; ++t) {
-        z[t] *= st.gl[tg + t][0];
-        val[tg + t] = type ? z[t] : st.v[tg + t][wcol + mycol] - z[t];
-      }
+      for (int t = 0; t < C::GT; ++t) val[tg + t] = fmaf(z[t], st.gl[tg + t][type], st.v[type][tg + t][wcol + mycol]);
     }
     // u = T x in the lanes that hold x, o = e^c S^T q + W x in the others
     float x[BT];
@@ -554,9 +577,9 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
       if (type == 0) val[j] = 0.f;
     }
 #pragma unroll
-    for (int i = 0; i < BT; ++i)
+    for (int j4 = 0; j4 < BT / 4; ++j4)
 #pragma unroll
-      for (int j4 = 0; j4 <= i / 4; ++j4) {      // beyond the diagonal the rows hold zeros
+      for (int i = 4 * j4; i < BT; ++i) {        // beyond the diagonal the rows hold zeros
         const float4 m = *reinterpret_cast<const float4*>(&st.tw[i][type * BT + 4 * j4]);
         val[i] = fmaf(m.x, x[4 * j4], fmaf(m.y, x[4 * j4 + 1], fmaf(m.z, x[4 * j4 + 2], fmaf(m.w, x[4 * j4 + 3], val[i]))));
       }
@@ -564,32 +587,34 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
       if (type == 0) {
 #pragma unroll
         for (int t = 0; t < BT; ++t) {
-          const float u = val[t] * st.gl[t][1];
-          s.u[warp][t][grp * 4 + mycol] = make_float2(u, u);
+          const float u = val[t] * st.gl[t][2];
+          s.u[warp][0][t][grp * 4 + mycol] = make_float2(u, u);
+          s.u[warp][1][t][grp * 4 + (mycol ^ 1)] = make_float2(u, u);
         }
       } else if (on) {
         float* dst = vo + ((long long)qs + t0) * a.H * dv + (long long)h * dv + col + mycol;
 #pragma unroll
-        for (int t = 0; t < BT; ++t)
-          if (t < n) dst[(long long)t * a.H * dv] = val[t];
+        for (int t = 0; t < BT; ++t, dst += (long long)a.H * dv)
+          if (t < n) *dst = val[t];
       }
     }
     __syncwarp();
     // the state behind the block
-    const float end = st.gl[BT - 1][0];
+    const float end = st.gl[BT - 1][1];
     const uint64_t fade = pack_f32x2(end, end);
+    const float* kk = &st.kq[0][0][4 * l];
+    const float2 *ua = &s.u[warp][mycol & 1][0][grp * 4 + (mycol & 2)], *ub = &s.u[warp][mycol & 1][0][grp * 4 + ((mycol & 2) ^ 2)];
 #pragma unroll
     for (int p = 0; p < RPL / 2; ++p)
 #pragma unroll
       for (int c = 0; c < 4; ++c) S[p][c] = mul_f32x2(S[p][c], fade);
 #pragma unroll
     for (int j = 0; j < BT; ++j) {
-      const ulonglong2 u01 = *reinterpret_cast<const ulonglong2*>(&s.u[warp][j][grp * 4]);
-      const ulonglong2 u23 = *reinterpret_cast<const ulonglong2*>(&s.u[warp][j][grp * 4 + 2]);
+      const ulonglong2 u01 = *reinterpret_cast<const ulonglong2*>(ua + j * C::CPW), u23 = *reinterpret_cast<const ulonglong2*>(ub + j * C::CPW);
       const uint64_t u[4] = {u01.x, u01.y, u23.x, u23.y};
 #pragma unroll
       for (int x2 = 0; x2 < RPL / 4; ++x2) {
-        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(&st.k[j][4 * (l + LPG * x2)]);
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(kk + j * C::DK + 4 * LPG * x2);
 #pragma unroll
         for (int c = 0; c < 4; ++c) {
           S[2 * x2][c] = fma_f32x2(k.x, u[c], S[2 * x2][c]);
@@ -607,8 +632,8 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
       if (r >= dk) continue;
       float4 x, y;
       unpack_f32x2(S[p][0], x.x, y.x); unpack_f32x2(S[p][1], x.y, y.y); unpack_f32x2(S[p][2], x.z, y.z); unpack_f32x2(S[p][3], x.w, y.w);
-      *reinterpret_cast<float4*>(dst + (long long)r * dv) = x;
-      *reinterpret_cast<float4*>(dst + (long long)(r + 1) * dv) = y;
+      *reinterpret_cast<float4*>(dst + (long long)r * dv) = turn(x);
+      *reinterpret_cast<float4*>(dst + (long long)(r + 1) * dv) = turn(y);
     }
   }
 }
@@ -656,14 +681,12 @@ static cudaError_t launch_scan(const UbDeltaArgs& a, cudaStream_t st) {
 
 template <typename T>
 static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
-  const int group = a.H / a.G;
-  const size_t smem = sizeof(float) * (2 * BT * (a.dk + 4) + 2 * BT * LDM + (size_t)(group < PREP_T / BT ? (group + 1) / 2 * 2 : PREP_T / BT) * LDH);
-  const dim3 grid((a.max_q + BT - 1) / BT, a.G + (a.H * a.dv + PREP_T - 1) / PREP_T, a.num_seqs);
-  if (smem > 48 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return e;
-  }
+  const size_t smem = sizeof(float) * 2 * BT * (a.dk + 4);
+  const int blocks = (a.max_q + BT - 1) / BT;
+  const dim3 grid(blocks, a.G + (a.H * a.dv + PREP_T - 1) / PREP_T, a.num_seqs);
   cudaError_t e = launch_pdl(delta_prep_kernel<T>, grid, dim3(PREP_T), smem, st, a);
+  if (e != cudaSuccess) return e;
+  e = launch_pdl(delta_solve_kernel<T>, dim3(blocks, (a.H + SOLVE_T / BT - 1) / (SOLVE_T / BT), a.num_seqs), dim3(SOLVE_T), (size_t)0, st, a);
   if (e != cudaSuccess) return e;
   // few lanes per column keep the reductions short, many of them spread a small launch over the device
   const long long cols = (long long)a.num_seqs * a.H * a.dv;
@@ -685,7 +708,7 @@ static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
 }  // namespace ub
 
 extern "C" long long ub_delta_workspace_floats(int rows, int H, int G, int dk, int dv) {
-  return (long long)rows * (2LL * G * dk + (long long)H * dv + 2LL * ub::delta::BT * H + 2LL * H);
+  return (long long)rows * (2LL * G * dk + (long long)H * dv + 2LL * ub::delta::BT * (H + G) + 4LL * H);
 }
 
 extern "C" int ub_delta_mixer(const UbDeltaArgs* a, void* stream) {

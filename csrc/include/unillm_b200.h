@@ -446,12 +446,13 @@ typedef struct UbMoeRouteArgs {
   const void* router_b;     /* [E] added to the logits (router_w mode), or NULL */
   int x_f32;                /* x is fp32 (the residual stream itself) */
   int router_f32;           /* router_w and router_b are fp32 */
-  /* router_w mode: experts are chosen by softmax(logits) + correction, within the keep_groups of `groups` equal groups of
-     neighbours that have the largest such score; the weights are the chosen softmax values over their sum + 1e-20 */
+  /* With a correction or groups, experts are chosen by softmax(logits) + correction, within the keep_groups of `groups` equal
+     groups of neighbours that have the largest such score; the weights are the chosen softmax values over their sum + 1e-20 */
   const void* correction;   /* [E] of the router's type, or NULL */
   int groups, keep_groups;  /* 0 or 1: no groups */
   const void* shared_w;     /* [H] of the router's type: shared_gate[t] = sigmoid(x . shared_w), or NULL */
-  float* shared_gate;       /* [T] */
+  float* shared_gate;       /* [T]; with given logits, of their column E */
+  int ld_logits;            /* elements between rows of given logits, 0 = E */
 } UbMoeRouteArgs;
 int ub_moe_route(const UbMoeRouteArgs* args, void* stream);
 int ub_moe_gather(const void* x, const int* sorted_rows, void* out, int rows, int K, int H, void* stream);

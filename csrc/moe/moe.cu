@@ -17,8 +17,8 @@ namespace ub {
 constexpr int MOE_MAX_E = 256;
 constexpr int MOE_MAX_K = 16;
 
-// Logits of TB tokens per CTA (from x and the router matrix, or given), then top-k and weights, one warp per token.  A CTA has
-// a warp for every four router rows, up to sixteen.  XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.  A warp
+// Logits of TB tokens per CTA (from x and the router matrix, or given), then top-k and weights, one warp per token.  A CTA of
+// one token has a warp for every four router rows, up to sixteen.  XT / WT: element types of the activations (bf16, or the fp32 residual stream) and of the router.  A warp
 // takes four experts at a time for all TB tokens, so a router row is read once per TB tokens and an activation once per
 // four experts.  A logit's sum runs over h in the same order whatever TB is.
 template <typename XT, typename WT, int TB>
@@ -70,11 +70,13 @@ __global__ void __launch_bounds__(512) moe_route_kernel(const UbMoeRouteArgs a) 
         }
     }
   } else {
-    for (int i = threadIdx.x; i < TB * E; i += blockDim.x) {
-      const int t = t0 + i / E, e = i % E;
+    const long long ldl = a.ld_logits > 0 ? a.ld_logits : E;
+    const int cols = E + (a.shared_gate != nullptr);
+    for (int i = threadIdx.x; i < TB * cols; i += blockDim.x) {
+      const int t = t0 + i / cols, e = i % cols;
       if (t >= a.T) continue;
-      logits_s[i / E][e] = a.logits_f32 ? reinterpret_cast<const float*>(a.logits)[(long long)t * E + e]
-                                        : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.logits)[(long long)t * E + e]);
+      logits_s[i / cols][e] = a.logits_f32 ? reinterpret_cast<const float*>(a.logits)[t * ldl + e]
+                                        : __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(a.logits)[t * ldl + e]);
     }
   }
   __syncthreads();
@@ -244,7 +246,7 @@ template <typename XT, typename WT>
 static void launch_route(const UbMoeRouteArgs& a, cudaStream_t st) {
   const int rows = a.router_w != nullptr ? a.E + (a.shared_w != nullptr) : 16;
   const int nt = 32 * (rows <= 16 ? 4 : rows > 60 ? 16 : (rows + 3) / 4);
-  if (a.T >= 148 * 8) moe_route_kernel<XT, WT, 4><<<(a.T + 3) / 4, nt, 0, st>>>(a);
+  if (a.T >= 148 * 8) moe_route_kernel<XT, WT, 4><<<(a.T + 3) / 4, 128, 0, st>>>(a);
   else moe_route_kernel<XT, WT, 1><<<a.T, nt, 0, st>>>(a);
 }
 
@@ -495,15 +497,15 @@ extern "C" int ub_moe_route(const UbMoeRouteArgs* a, void* stream_v) {
   if (a->E <= 0 || a->E > ub::MOE_MAX_E || a->K <= 0 || a->K > ub::MOE_MAX_K || a->K > a->E) return -2;
   if (a->router_w != nullptr && (a->H % 8 != 0 || a->x == nullptr)) return -3;
   if (a->tiles != nullptr && (a->tile_tokens <= 0 || a->max_tiles <= 0)) return -4;
-  if (a->router_w == nullptr && (a->correction != nullptr || a->shared_w != nullptr)) return -5;
-  if ((a->shared_w != nullptr) != (a->shared_gate != nullptr)) return -5;
+  if (a->router_w == nullptr ? a->shared_w != nullptr : (a->shared_w != nullptr) != (a->shared_gate != nullptr)) return -5;
+  if (a->ld_logits != 0 && a->ld_logits < a->E + (a->shared_gate != nullptr)) return -5;
   if (a->groups > 1 && (a->E % a->groups != 0 || a->keep_groups < 1 || a->keep_groups > a->groups || a->K > a->keep_groups * (a->E / a->groups)))
     return -6;
   UbMoeRouteArgs b = *a;
   if (b.weight_scale == 0.f) b.weight_scale = 1.f;
   if (b.router_w != nullptr && b.x_f32 && b.router_f32) ub::launch_route<float, float>(b, st);
   else if (b.router_w != nullptr && b.x_f32) ub::launch_route<float, __nv_bfloat16>(b, st);
-  else if (b.router_w != nullptr && b.router_f32) ub::launch_route<__nv_bfloat16, float>(b, st);
+  else if (b.router_f32) ub::launch_route<__nv_bfloat16, float>(b, st);
   else ub::launch_route<__nv_bfloat16, __nv_bfloat16>(b, st);
   ub::moe_sort_kernel<<<1, 1024, 0, st>>>(b);
   cudaError_t e = cudaGetLastError();

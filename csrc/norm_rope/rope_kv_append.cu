@@ -188,17 +188,21 @@ __global__ void __launch_bounds__(128) rope_kv_append_kernel(const UbRopeArgs a)
 // LPH lanes per head (a power of two, LPH * 8 >= D), eight consecutive elements of the head per lane: the norm is a shuffle
 // reduction among the lanes of the head, interleaved pairs are lane-local, half-split pairs come from the lane that holds
 // the other half.  K goes to the cache and, unless k_cache_only, back into the row; V is copied to the cache.  A thread
-// requests its chunks of up to U heads (and its share of V) before it works out the angles.
-template <typename T, int LPH>
-__global__ void __launch_bounds__(256) head_norm_rope_kernel(const UbRopeArgs a) {
+// requests its chunks of U heads (and its share of V) before it works out the angles; a lane meets the same angles in every
+// head, so they stay in registers.
+enum { PAIR_HALVES = 0, PAIR_NEIGHBOURS = 1, PAIR_ODD = 2 /* halves that are no whole chunks */ };
+
+template <typename T, int LPH, int PAIR>
+__global__ void __launch_bounds__(128, 8) head_norm_rope_kernel(const UbRopeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  constexpr int U = 3;
+  constexpr int U = 2;
   extern __shared__ float cs[];                   // cos [half] then sin [half]
-  __shared__ float red[2][8];
-  const int t = blockIdx.x, D = a.D, Dv = a.Dv, half = a.rotary_dim / 2, nt = blockDim.x;
-  const int grp = threadIdx.x / LPH, c = threadIdx.x % LPH, ngrp = nt / LPH;
-  const int nrot = a.Hq + a.Hkv, batch = U * ngrp;
+  __shared__ float red[2][4];
+  const int t = blockIdx.x, D = a.D, Dv = a.Dv, half = a.rotary_dim / 2;
+  constexpr int ngrp = 128 / LPH, batch = U * ngrp;
+  const int grp = threadIdx.x / LPH, c = threadIdx.x % LPH;
+  const int nrot = a.Hq + a.Hkv;
   const bool have = c * 8 < D;                    // the last lanes of a group may own nothing
   T* row = reinterpret_cast<T*>(a.qkv) + (long long)t * a.ld;
   float v[U][8];
@@ -208,7 +212,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const UbRopeArgs a)
       const int h = h0 + u * ngrp + grp;
 #pragma unroll
       for (int e = 0; e < 8; ++e) v[u][e] = 0.f;
-      if (h < nrot && have) load8(row + (long long)h * D + c * 8, v[u]);
+      if (h < nrot && have) load8(row + h * D + c * 8, v[u]);
     }
   };
   load(0);
@@ -220,7 +224,7 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const UbRopeArgs a)
   }
   const long long blk = slot_ok ? slot / a.block_size : 0, off = slot_ok ? slot % a.block_size : 0;
   const float pos = (float)a.positions[t] * a.pos_scale;
-  for (int i = threadIdx.x; i < half; i += nt) {
+  for (int i = threadIdx.x; i < half; i += 128) {
     float s, co;
     sincosf(pos * (a.inv_freq != nullptr ? a.inv_freq[i] : rope_inv_freq(i, a)), &s, &co);
     cs[i] = co;
@@ -228,15 +232,15 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const UbRopeArgs a)
   }
   if (slot_ok && a.v_cache != nullptr) {
     const int cpr = Dv / 8;
-    const T* vr = row + (long long)nrot * D;
-    for (int it = threadIdx.x; it < a.Hkv * cpr; it += nt) {
+    const T* vr = row + nrot * D;
+    T* vd = reinterpret_cast<T*>(a.v_cache) + (blk * a.Hkv * a.block_size + off) * Dv;
+    for (int it = threadIdx.x; it < a.Hkv * cpr; it += 128) {
       const int hk = it / cpr, ch = it - hk * cpr;
       float w[8];
-      load8(vr + (long long)hk * Dv + ch * 8, w);
-      store8(reinterpret_cast<T*>(a.v_cache) + ((blk * a.Hkv + hk) * a.block_size + off) * Dv + ch * 8, w);
+      load8(vr + it * 8, w);
+      store8(vd + (long long)hk * a.block_size * Dv + ch * 8, w);
     }
   }
-  float rq = 1.f, rk = 1.f;                       // row norms: one factor for all queries, one for all keys
   if (a.row_norm) {
     float sq = 0.f, sk = 0.f;
     for (int h0 = 0; h0 < nrot; h0 += batch) {
@@ -255,14 +259,34 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const UbRopeArgs a)
     if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
   }
   __syncthreads();                                // angles and sums complete; nobody has written to the row yet
+  float rq = 1.f, rk = 1.f;                       // row norms: one factor for all queries, one for all keys
   if (a.row_norm) {
-    float sq = 0.f, sk = 0.f;
-    for (int w = 0; w < nt >> 5; ++w) { sq += red[0][w]; sk += red[1][w]; }
-    rq = 1.f / sqrtf(sq / (float)(a.Hq * a.norm_dim) + a.norm_eps);
-    if (a.Hkv > 0) rk = 1.f / sqrtf(sk / (float)(a.Hkv * a.norm_dim) + a.norm_eps);
+    rq = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)(a.Hq * a.norm_dim) + a.norm_eps);
+    if (a.Hkv > 0) rk = 1.f / sqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)(a.Hkv * a.norm_dim) + a.norm_eps);
   }
-  const float inv_n = 1.f / (float)a.norm_dim;
-  const int hc = half / 8;                        // half-split form: chunks per half
+  const bool normed = a.q_norm_w != nullptr || a.k_norm_w != nullptr;
+  // element e of this lane's chunk becomes x * co[e] + other * si[e]
+  constexpr int NA = PAIR == PAIR_NEIGHBOURS ? 4 : 8;
+  float co[NA], si[NA];
+  int partner = c;
+#pragma unroll
+  for (int e = 0; e < NA; ++e) {
+    co[e] = 1.f;
+    si[e] = 0.f;
+    if (PAIR == PAIR_NEIGHBOURS) {
+      const int i = c * 4 + e;
+      if (i < half) { co[e] = cs[i]; si[e] = cs[half + i]; }
+    } else {
+      const int i = c * 8 + e;
+      if (i < half) { co[e] = cs[i]; si[e] = -cs[half + i]; }
+      else if (i < 2 * half) { co[e] = cs[i - half]; si[e] = cs[i]; }
+    }
+  }
+  if (PAIR == PAIR_HALVES) {
+    const int hc = half / 8;                      // chunks per half
+    partner = c < hc ? c + hc : (c < 2 * hc ? c - hc : c);
+  }
+  T* kd = reinterpret_cast<T*>(a.k_cache) + (blk * a.Hkv * a.block_size + off) * D + c * 8;
   for (int h0 = 0; h0 < nrot; h0 += batch) {
     if (h0 > 0) load(h0);
 #pragma unroll
@@ -273,77 +297,70 @@ __global__ void __launch_bounds__(256) head_norm_rope_kernel(const UbRopeArgs a)
       float (&x)[8] = v[u];
       const T* nw = reinterpret_cast<const T*>(h < a.Hq ? a.q_norm_w : a.k_norm_w);
       float r = 1.f;
-      if (a.row_norm) {
-        r = h < a.Hq ? rq : rk;
-        nw += (long long)(h < a.Hq ? h : h - a.Hq) * D;
-      } else if (a.q_norm_w != nullptr || a.k_norm_w != nullptr) {
-        float ss = 0.f;
+      if (normed) {
+        if (a.row_norm) {
+          r = h < a.Hq ? rq : rk;
+          nw += (h < a.Hq ? h : h - a.Hq) * D;
+        } else {
+          float ss = 0.f;
 #pragma unroll
-        for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
+          for (int e = 0; e < 8; ++e) ss += x[e] * x[e];
 #pragma unroll
-        for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-        if (nw != nullptr) r = 1.f / sqrtf(ss * inv_n + a.norm_eps);
+          for (int o = LPH / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+          if (nw != nullptr) r = 1.f / sqrtf(ss / (float)a.norm_dim + a.norm_eps);
+        }
+        if (ok && nw != nullptr) {
+          float w[8];
+          load8(nw + c * 8, w);
+#pragma unroll
+          for (int e = 0; e < 8; ++e) x[e] = x[e] * r * w[e];
+        }
       }
-      if (ok && nw != nullptr) {
-        float w[8];
-        load8(nw + c * 8, w);
+      if (half > 0) {
+        if (PAIR == PAIR_NEIGHBOURS) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[e] = x[e] * r * w[e];
-      }
-      if (a.interleaved) {
-#pragma unroll
-        for (int e = 0; e < 8; e += 2) {
-          const int i = c * 4 + e / 2;
-          if (i < half) {
-            const float co = cs[i], si = cs[half + i], x0 = x[e], x1 = x[e + 1];
-            x[e] = x0 * co - x1 * si;
-            x[e + 1] = x1 * co + x0 * si;
+          for (int e = 0; e < 4; ++e) {
+            const float x0 = x[2 * e], x1 = x[2 * e + 1];
+            x[2 * e] = x0 * co[e] - x1 * si[e];
+            x[2 * e + 1] = x1 * co[e] + x0 * si[e];
           }
-        }
-      } else if (half > 0 && half % 8 != 0) {     // the other half of a pair lies across chunks: fetched element by element
-        float o[8];
+        } else if (PAIR == PAIR_ODD) {            // the other half of a pair lies across chunks: fetched element by element
+          float o[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const int i = c * 8 + e, j = i < half ? i + half : i - half;
-          o[e] = 0.f;
-          if (ok && i < 2 * half) o[e] = (float)row[(long long)h * D + j] * r * (nw != nullptr ? (float)nw[j] : 1.f);
-        }
-        __syncwarp();                             // a head's lanes have read it before one of them writes
+          for (int e = 0; e < 8; ++e) {
+            const int i = c * 8 + e, j = i < half ? i + half : i - half;
+            o[e] = 0.f;
+            if (ok && i < 2 * half) o[e] = (float)row[h * D + j] * r * (nw != nullptr ? (float)nw[j] : 1.f);
+          }
+          __syncwarp();                           // a head's lanes have read it before one of them writes
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const int i = c * 8 + e;
-          if (i < half) x[e] = x[e] * cs[i] - o[e] * cs[half + i];
-          else if (i < 2 * half) x[e] = x[e] * cs[i - half] + o[e] * cs[i];
-        }
-      } else if (half > 0) {
-        const int partner = c < hc ? c + hc : (c < 2 * hc ? c - hc : c);
-        const float sign = c < hc ? -1.f : 1.f;
-        const int at = (c < hc ? c : c - hc) * 8;
-        const bool turn = c < 2 * hc;
+          for (int e = 0; e < 8; ++e) x[e] = x[e] * co[e % NA] + o[e] * si[e % NA];
+        } else {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float other = __shfl_sync(0xffffffffu, x[e], partner, LPH);
-          if (turn) x[e] = x[e] * cs[at + e] + sign * other * cs[half + at + e];
+          for (int e = 0; e < 8; ++e) x[e] = x[e] * co[e % NA] + __shfl_sync(0xffffffffu, x[e], partner, LPH) * si[e % NA];
         }
       }
       if (!ok) continue;
-      if (h < a.Hq || !a.k_cache_only || !slot_ok) store8(row + (long long)h * D + c * 8, x);
-      if (h >= a.Hq && slot_ok && a.k_cache != nullptr)
-        store8(reinterpret_cast<T*>(a.k_cache) + ((blk * a.Hkv + (h - a.Hq)) * a.block_size + off) * D + c * 8, x);
+      if (h < a.Hq || !a.k_cache_only || !slot_ok) store8(row + h * D + c * 8, x);
+      if (h >= a.Hq && slot_ok && a.k_cache != nullptr) store8(kd + (long long)(h - a.Hq) * a.block_size * D, x);
     }
   }
 }
 
-template <typename T>
+template <typename T, int PAIR>
 static cudaError_t launch_head_norm_rope(const UbRopeArgs& a, cudaStream_t st) {
   const size_t smem = (size_t)(a.rotary_dim > 0 ? a.rotary_dim : 1) * sizeof(float);
-  const int lph = a.D <= 32 ? 4 : a.D <= 64 ? 8 : a.D <= 128 ? 16 : 32;
-  const int nt = (a.Hq + a.Hkv) * lph > 3 * 128 ? 256 : 128;          // a few heads per thread
-  const dim3 grid(a.T), block(nt);
-  if (lph == 4) return launch_pdl(head_norm_rope_kernel<T, 4>, grid, block, smem, st, a);
-  if (lph == 8) return launch_pdl(head_norm_rope_kernel<T, 8>, grid, block, smem, st, a);
-  if (lph == 16) return launch_pdl(head_norm_rope_kernel<T, 16>, grid, block, smem, st, a);
-  return launch_pdl(head_norm_rope_kernel<T, 32>, grid, block, smem, st, a);
+  const dim3 grid(a.T), block(128);
+  if (a.D <= 32) return launch_pdl(head_norm_rope_kernel<T, 4, PAIR>, grid, block, smem, st, a);
+  if (a.D <= 64) return launch_pdl(head_norm_rope_kernel<T, 8, PAIR>, grid, block, smem, st, a);
+  if (a.D <= 128) return launch_pdl(head_norm_rope_kernel<T, 16, PAIR>, grid, block, smem, st, a);
+  return launch_pdl(head_norm_rope_kernel<T, 32, PAIR>, grid, block, smem, st, a);
+}
+
+template <typename T>
+static cudaError_t launch_head_norm_rope(const UbRopeArgs& a, cudaStream_t st) {
+  if (a.interleaved) return launch_head_norm_rope<T, PAIR_NEIGHBOURS>(a, st);
+  return a.rotary_dim % 16 != 0 ? launch_head_norm_rope<T, PAIR_ODD>(a, st) : launch_head_norm_rope<T, PAIR_HALVES>(a, st);
 }
 
 }  // namespace ub

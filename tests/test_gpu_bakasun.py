@@ -283,14 +283,21 @@ ROUTERS = [(8, 3, 2, 1, 40), (9, 4, 3, 2, 96), (5, 1, 1, 1, 16), (40, 6, 8, 3, 2
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("T", [1, 7, 1300])
 @pytest.mark.parametrize("E,top,count,keep,H", ROUTERS)
-def test_router(dtype, T, E, top, count, keep, H):
-    """Choice by corrected scores inside the best groups, weights without the correction, gate of the shared expert."""
+@pytest.mark.parametrize("given", [False, True])
+def test_router(dtype, T, E, top, count, keep, H, given):
+    """Choice by corrected scores inside the best groups, weights without the correction, gate of the shared expert; from the rows
+    or from logits in wider rows."""
     from unillm_b200.ops import cuda_ops as K
 
     x, w, sg = _rand(T, H, seed=1), _rand(E, H, seed=2, scale=1.5 * H ** -0.5), _rand(H, seed=3, scale=2 * H ** -0.5)
     corr = (_rand(E, seed=4, dtype=torch.float32, scale=1.5 / E) - 0.6 / E).to(torch.bfloat16)      # choice scores of both signs
     dev = lambda t: t.to("cuda", dtype).contiguous()
-    r = K.moe_route(dev(x), dev(w), top, round_logits_bf16=False, correction=dev(corr), groups=count, keep_groups=keep, shared_w=dev(sg))
+    kw = dict(correction=dev(corr), groups=count, keep_groups=keep)
+    if given:
+        full = torch.cat([x.double() @ w.double().T, x.double() @ sg.double()[:, None], torch.full((T, 5), 1e3)], 1).float().cuda()
+        r = K.moe_route(None, None, top, logits=full, num_experts=E, shared_gate=True, **kw)
+    else:
+        r = K.moe_route(dev(x), dev(w), top, round_logits_bf16=False, shared_w=dev(sg), **kw)
     s = torch.softmax(x.double() @ w.double().T, -1)
     choice = s + corr.double()
     _close(r.shared_gate, P.sigmoid(x.double() @ sg.double()), torch.float32)
@@ -317,7 +324,9 @@ def test_router_refuses_groups_that_do_not_fit():
         with pytest.raises(RuntimeError):
             K.moe_route(x, w, top, groups=groups, keep_groups=keep)
     with pytest.raises(ValueError):
-        K.moe_route(None, None, 2, logits=_rand(2, 8).cuda(), correction=_rand(8).cuda())
+        K.moe_route(None, None, 2, logits=_rand(2, 8).cuda(), shared_w=_rand(8).cuda())
+    with pytest.raises(ValueError):
+        K.moe_route(x, w, 2, correction=_rand(7).cuda())
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -352,6 +361,26 @@ def test_norms_around_a_mixture(dtype, H, T, top):
         _close(out[:, :H], P.norm(want_x, wn.double(), 1e-4), dtype, f32_tol=5e-5)
         assert xs[:, H:].abs().sum() == 0 and out[:, H:].abs().sum() == 0
     K.check_device_errors()
+
+
+def test_router_of_many_rows_is_a_matrix_product():
+    """From a thousand rows on, logits and gates come from the tensor cores; the choice is that of the router kernel."""
+    from unillm_b200.engine import moe_runner
+    from unillm_b200.engine.runner import GpuModelRunner, RunnerWeights
+
+    cfg = C.CASES["mixed"]
+    m = C.load_model(cfg, C.make_weights(cfg))
+    runner = GpuModelRunner(m.spec, RunnerWeights(m.spec, m.p, "cuda"), num_blocks=8, max_num_seqs=4, max_num_batched_tokens=2048,
+                            max_model_len=256, use_cuda_graphs=False)
+    h = _rand(1100, cfg["width"], seed=3).cuda()
+    base, y, r = moe_runner.moe_branch(runner, 1, h, h)
+    few = [moe_runner.moe_branch(runner, 1, h[i:i + 550].contiguous(), h[i:i + 550].contiguous()) for i in (0, 550)]
+    ids = torch.cat([x[2].topk_ids for x in few])
+    same = (r.topk_ids == ids).all(1)
+    assert same.float().mean() > 0.99
+    for got, want in ((r.topk_w, torch.cat([x[2].topk_w for x in few])), (r.shared_gate, torch.cat([x[2].shared_gate for x in few]))):
+        assert (got - want)[same].abs().max() < 1e-4
+    assert _close(base, torch.cat([x[0] for x in few]).cpu(), torch.bfloat16, bf16_tol=3e-2) is None
 
 
 # ------------------------------------------------------------------------------------------------

@@ -244,7 +244,9 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
                 n = r.shape[0] / x.shape[0]
                 k = kw["routing"].K if ex is not None else 0
                 return "final norm", int(n * (_nbytes(x, y) + k * _nbytes(y if y is not None else x)) + _nbytes(r)), 0.0
-            return ("norms" + (" + expert sum" if ex is not None else ""),
+            if y is None and ex is None:
+                return "norm", _nbytes(x, r[1]), 0.0
+            return ("norm + residual" + (" + expert sum" if ex is not None else "") + " + norm",
                     _nbytes(x, y, ex, r[1]) + (_nbytes(x) if y is not None or ex is not None else 0), 0.0)
         live = sum(p.n for p in parts)
         state = sum(2 * live * t[0].numel() * 4 for t in (kw.get("conv_state"), kw.get("shift_state")) if t is not None)
@@ -317,6 +319,8 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
         q = kw["num_q_heads"] * kw["head_dim"] / a[0].shape[1]
         kv = 1.0 - q
         return "rope + append", int(_nbytes(a[0]) * (2 * q + 2 * kv)), 0.0
+    if name == "moe_route" and a[0] is None:
+        return "route + sort (logits given)", _nbytes(kw["logits"], r.topk_ids, r.topk_w, r.sorted_rows, r.row_slot), 0.0
     if name == "moe_route":
         return "route + sort", _nbytes(a[0], a[1]), 2.0 * a[0].shape[0] * a[1].numel()
     if name == "moe_gather":

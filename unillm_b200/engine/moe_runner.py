@@ -24,17 +24,29 @@ import torch
 from ..ops import cuda_ops as K
 
 
+ROUTER_GEMM_ROWS = 1024
+
+
 def _experts(runner, i: int, h: torch.Tensor, router_x: torch.Tensor):
     """Routing of ``router_x`` and the experts' outputs for ``h``: (rows in expert order, routing)."""
     t = runner.w.t
     m = runner.layers[i].moe
     L = f"layers.{i}."
     T = h.shape[0]
-    with runner._prof("moe_route"):
-        r = K.moe_route(router_x, t[L + "router"], m.top_k, norm_topk=m.normalize_topk, round_logits_bf16=False,
-                        expert_lo=runner.w.expert_lo if runner.w.ep else 0,
-                        num_local_experts=runner.w.experts_local if runner.w.ep else 0, router_b=t.get(L + "router_b"),
-                        correction=t.get(L + "correction"), groups=m.groups, keep_groups=m.keep_groups, shared_w=t.get(L + "shared_sg"))
+    kw = dict(norm_topk=m.normalize_topk, expert_lo=runner.w.expert_lo if runner.w.ep else 0,
+              num_local_experts=runner.w.experts_local if runner.w.ep else 0, correction=t.get(L + "correction"), groups=m.groups,
+              keep_groups=m.keep_groups)
+    full = t.get(L + "router_full")
+    if full is not None and T >= ROUTER_GEMM_ROWS and router_x.dtype == full.dtype:
+        # many rows: the logits (and the shared expert's gate) are a tensor-core product with fp32 results
+        logits = runner._gemm(router_x, full, out_dtype=torch.float32)
+        with runner._prof("moe_route"):
+            r = K.moe_route(None, None, m.top_k, logits=logits, num_experts=m.num_experts, shared_gate=m.shared_gate, **kw)
+    else:
+        with runner._prof("moe_route"):
+            r = K.moe_route(router_x, t[L + "router"], m.top_k, round_logits_bf16=False, router_b=t.get(L + "router_b"),
+                            shared_w=t.get(L + "shared_sg"), **kw)
+    with runner._prof("moe_gather"):
         xs = K.moe_gather(h, r)
     runner.launches += 3
     gu, dn = t[L + "experts_gate_up"], t[L + "experts_down"]

@@ -277,6 +277,7 @@ class RunnerWeights:
             self.t[L + "correction"] = dev(p[L + "correction"])
         if m.shared_gate:
             self.t[L + "shared_sg"] = dev(_pad(p[L + "shared_sg"], 1, H)).view(-1)
+        self._router_full(L, m)
 
         def up_rows(t, r, w):
             """This rank's rows of an up (or [gate; up]) matrix [.., rows, H], each half padded to 8."""
@@ -301,6 +302,14 @@ class RunnerWeights:
         if L + "shared_gate_up" in p:
             self.t[L + "shared_gate_up"] = dev(up_rows(p[L + "shared_gate_up"], rank, world))
             self.t[L + "shared_down"] = dev(down_cols(p[L + "shared_down"], rank, world))
+
+    def _router_full(self, L: str, m) -> None:
+        """Router rows and the shared expert's gate as one matrix of whole 8-row groups, for steps with many tokens."""
+        if self.dtype != torch.bfloat16 or m.router_bias or self.ep:
+            return
+        rows = [self.t[L + "router"]] + ([self.t[L + "shared_sg"][None]] if m.shared_gate else [])
+        w = torch.cat(rows)
+        self.t[L + "router_full"] = _pad(w, 0, _round8(w.shape[0]))
 
     def _dense_weights(self, i: int, p, dev) -> None:
         """Dense feed-forward of one layer."""
@@ -546,6 +555,7 @@ class RunnerWeights:
             if s.layer_is_moe(i):
                 m = s.moe
                 self.t[L + "router"] = rnd(m.num_experts, H)
+                self._router_full(L, m)
                 # tensor parallel inside every expert, or (expert parallel) whole experts of this rank
                 Ie = m.intermediate_size if self.ep else m.intermediate_size // world
                 c0 = 0 if self.ep else rank * Ie
@@ -651,6 +661,7 @@ class RunnerWeights:
                 self.t[L + "correction"] = zeros(m.num_experts)
             if m.shared_gate:
                 self.t[L + "shared_sg"] = rnd(1, H).view(-1)
+            self._router_full(L, m)
             self.t[L + "experts_gate_up"] = torch.stack([rnd(up, H) for _ in range(m.num_experts)])
             self.t[L + "experts_down"] = torch.stack([rnd(H, self._round(m.intermediate_size)) for _ in range(m.num_experts)])
             if m.num_shared_experts:

@@ -178,7 +178,7 @@ class UbMoeRouteArgs(C.Structure):
         ("logits_f32", i32), ("T", i32), ("E", i32), ("K", i32), ("H", i32), ("norm_topk", i32),
         ("round_logits_bf16", i32), ("weight_scale", f32), ("tile_tokens", i32), ("max_tiles", i32),
         ("expert_lo", i32), ("num_local_experts", i32), ("router_b", vp), ("x_f32", i32), ("router_f32", i32),
-        ("correction", vp), ("groups", i32), ("keep_groups", i32), ("shared_w", vp), ("shared_gate", vp),
+        ("correction", vp), ("groups", i32), ("keep_groups", i32), ("shared_w", vp), ("shared_gate", vp), ("ld_logits", i32),
     ]
 
 

@@ -1133,7 +1133,8 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
               logits: Optional[torch.Tensor] = None, weight_scale: float = 1.0, tile_tokens: int = 0,
               round_logits_bf16: bool = True, routing: Optional[MoeRouting] = None, expert_lo: int = 0,
               num_local_experts: int = 0, router_b: Optional[torch.Tensor] = None, correction: Optional[torch.Tensor] = None,
-              groups: int = 1, keep_groups: int = 1, shared_w: Optional[torch.Tensor] = None) -> MoeRouting:
+              groups: int = 1, keep_groups: int = 1, shared_w: Optional[torch.Tensor] = None, shared_gate: bool = False,
+              num_experts: Optional[int] = None) -> MoeRouting:
     """Router GEMV (+ bias) + top-k + softmax weights + expert sort + grouped-GEMM tile table, two launches.  ``x`` may be
     bf16 or an fp32 residual stream, whatever the type of the router.
 
@@ -1141,7 +1142,9 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
     routed to other ranks get ``row_slot = -1`` and take no part in the grouped GEMMs.
 
     ``correction`` ([E]) and / or ``groups``: experts are chosen by softmax + correction within the ``keep_groups`` best groups of
-    neighbours, and weighted by their softmax values.  ``shared_w`` ([H]): ``routing.shared_gate[t] = sigmoid(x[t] . shared_w)``."""
+    neighbours, and weighted by their softmax values.  ``shared_w`` ([H]): ``routing.shared_gate[t] = sigmoid(x[t] . shared_w)``;
+    with given ``logits`` and ``shared_gate`` the gates are those of the column after the experts'.  ``num_experts``: columns
+    of ``logits`` that are experts (the first ones; default all)."""
     if router_w is not None:
         _elem("moe_route x", x), _elem("moe_route router", router_w, router_b, correction, shared_w)
         T, H = x.shape
@@ -1150,16 +1153,18 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
         E = router_w.shape[0]
         dev = x.device
     else:
-        T, E = logits.shape
+        T, cols = logits.shape
+        E = cols - int(shared_gate) if num_experts is None else num_experts
         H = 0
         dev = logits.device
-        if not logits.is_contiguous():
-            raise ValueError("logits must be contiguous")
+        if not logits.is_contiguous() or cols < E + int(shared_gate) or shared_w is not None:
+            raise ValueError("moe_route: contiguous logits [T, experts (+ gate)]")
     tn = tile_tokens or moe_tile_tokens(T, top_k, E)
-    r = routing if routing is not None else MoeRouting(T, top_k, E, tn, dev, shared_w is not None)
+    gated = shared_w is not None or shared_gate
+    r = routing if routing is not None else MoeRouting(T, top_k, E, tn, dev, gated)
     for t, n in ((correction, E), (shared_w, H)):
-        if t is not None and (router_w is None or t.numel() != n or not t.is_contiguous()):
-            raise ValueError("moe_route: correction [E] and shared_w [H] go with a router matrix")
+        if t is not None and (t.numel() != n or not t.is_contiguous()):
+            raise ValueError("moe_route: correction [E] and shared_w [H]")
     a = N.UbMoeRouteArgs()
     a.logits, a.x, a.router_w = _p(logits), _p(x) if router_w is not None else None, _p(router_w)
     a.topk_ids, a.topk_w = r.topk_ids.data_ptr(), r.topk_w.data_ptr()
@@ -1176,7 +1181,10 @@ def moe_route(x: Optional[torch.Tensor], router_w: Optional[torch.Tensor], top_k
     a.tile_tokens, a.max_tiles = r.tile_tokens, r.max_tiles
     a.expert_lo, a.num_local_experts = expert_lo, num_local_experts
     a.correction, a.groups, a.keep_groups = _p(correction), groups, keep_groups
-    a.shared_w, a.shared_gate = _p(shared_w), _p(r.shared_gate if shared_w is not None else None)
+    if correction is not None:
+        a.router_f32 = int(correction.dtype == torch.float32)
+    a.shared_w, a.shared_gate = _p(shared_w), _p(r.shared_gate if gated else None)
+    a.ld_logits = 0 if router_w is not None else logits.shape[1]
     N.check(N.cuda_lib().ub_moe_route(C.byref(a), torch.cuda.current_stream(dev).cuda_stream), "ub_moe_route")
     return r
 
