@@ -51,7 +51,7 @@ __device__ __forceinline__ int state_row(const UbDeltaArgs& a, const int* rows, 
 // ------------------------------------------------------------------------------------------------------------------------
 // NT threads; ROWS: rows of S that a thread holds (four columns each); 0: S is read twice instead (heads too large for registers).
 template <typename T, int NT, int ROWS>
-__global__ void __launch_bounds__(NT) delta_step_kernel(const UbDeltaArgs a, const int cl /* threads across the columns */) {
+__global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / NT : 1) delta_step_kernel(const UbDeltaArgs a, const int cl /* threads across the columns */) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int HELD = ROWS > 0 ? ROWS : 1;
@@ -80,20 +80,46 @@ __global__ void __launch_bounds__(NT) delta_step_kernel(const UbDeltaArgs a, con
       if (r < dk) S[i] = __ldcs(reinterpret_cast<const float4*>(src + (long long)r * dv));
     }
   }
-  // convolutions of this head's channels; the oldest input leaves, the current one joins
-  for (int c = tid; c < 2 * dk + dv; c += NT) {
-    const int ch = c < dk ? g * dk + c : c < 2 * dk ? a.G * dk + g * dk + (c - dk) : 2 * a.G * dk + h * dv + (c - 2 * dk);
-    const bool keep = so >= 0 && (c >= 2 * dk || h % group == 0);
-    const T* w = reinterpret_cast<const T*>(a.conv) + ch;
-    const float cur = (float)reinterpret_cast<const T*>(a.qkv)[row * a.ld + ch];
-    float acc = 0.f;
-    for (int j = 0; j < m; ++j) {
-      const float v = si >= 0 ? a.conv_state[((long long)si * m + j) * C + ch] : 0.f;
-      acc = fmaf((float)w[(long long)j * C], v, acc);
-      if (keep && j > 0) a.conv_state[((long long)so * m + j - 1) * C + ch] = v;
+  // convolutions of this head's channels; the oldest input leaves, the current one joins.  Four taps (of two
+  // channels, where a thread holds little of S) are requested together.
+  constexpr int CU = NT == 128 ? 2 : 1;
+  for (int c0 = tid; c0 < 2 * dk + dv; c0 += CU * NT) {
+    float acc[CU], cur[CU];
+    int ch[CU];
+    bool in[CU], keep[CU];
+#pragma unroll
+    for (int u = 0; u < CU; ++u) {
+      const int c = c0 + u * NT;
+      acc[u] = 0.f;
+      in[u] = c < 2 * dk + dv;
+      ch[u] = !in[u] ? 0 : c < dk ? g * dk + c : c < 2 * dk ? a.G * dk + g * dk + (c - dk) : 2 * a.G * dk + h * dv + (c - 2 * dk);
+      keep[u] = in[u] && so >= 0 && (c >= 2 * dk || h % group == 0);
+      cur[u] = (float)reinterpret_cast<const T*>(a.qkv)[row * a.ld + ch[u]];
     }
-    if (keep && m > 0) a.conv_state[((long long)so * m + m - 1) * C + ch] = cur;
-    qkv[c] = silu(fmaf((float)w[(long long)m * C], cur, acc));
+    const T* w = reinterpret_cast<const T*>(a.conv);
+    for (int j0 = 0; j0 < a.taps; j0 += 4) {
+      float v[CU][4], k[CU][4];
+#pragma unroll
+      for (int u = 0; u < CU; ++u)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int r = j0 + j;
+          k[u][j] = r < a.taps ? (float)w[(long long)r * C + ch[u]] : 0.f;
+          v[u][j] = r < m ? (si >= 0 ? a.conv_state[((long long)si * m + r) * C + ch[u]] : 0.f) : cur[u];
+        }
+#pragma unroll
+      for (int u = 0; u < CU; ++u)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          const int r = j0 + j;
+          if (r >= a.taps) break;
+          acc[u] = fmaf(k[u][j], v[u][j], acc[u]);
+          if (keep[u] && r > 0) a.conv_state[((long long)so * m + r - 1) * C + ch[u]] = v[u][j];
+        }
+    }
+#pragma unroll
+    for (int u = 0; u < CU; ++u)
+      if (in[u]) qkv[c0 + u * NT] = silu(acc[u]);
   }
   float gate = 0.f, nw = 0.f;                    // dv <= NT (launch_step)
   if (tid < dv) {
@@ -423,13 +449,16 @@ __device__ __forceinline__ void cp16(float* dst, const float* src, bool ok) {
 //
 // Sums over the lanes of a group are taken by halving: a lane hands over what its partner keeps.  So that this needs no
 // selection, lanes hold things in the order in which they give them away: the first operand of an odd half-group's lane is q
-// where the others' is k, and its four columns are numbered from its own one (slot s holds column s ^ own).
+// where the others' is k, the LPG / 8 lanes that share a column take LPG / 8 tokens at a time and number them from their own one
+// (slot s holds token s ^ own), and likewise the four columns.  In the end a lane has one number for every LPG / 8th token.
 template <int RPL, int LPG>
 struct Scan {
   static constexpr int DK = RPL * LPG;           // rows that fit
   static constexpr int CPW = 4 * (32 / LPG);     // columns per warp
   static constexpr int COLS = CPW * SCAN_W;      // ... per CTA
-  static constexpr int GT = RPL >= 16 ? 2 : 4;   // tokens whose products with S are under way together
+  static constexpr int REPS = LPG / 8;           // lanes per column and kind of product
+  static constexpr int OWN = BT / REPS;          // tokens a lane ends up with: q * REPS + rep
+  static constexpr int GT = RPL >= 16 ? (REPS > 2 ? REPS : 2) : 4;             // tokens whose products with S are under way together
   struct Stage {
     float kq[2][BT][DK], v[2][BT][COLS], tw[BT][2 * BT], gl[BT][4];          // v[1] stays zero
   };
@@ -520,7 +549,7 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
     const float *mine = &st.kq[type][0][4 * l], *theirs = &st.kq[type ^ 1][0][4 * l];
 
     // products of all tokens with the entering state: x (of the tokens' k) or e^c S^T q
-    float val[BT];
+    float f[C::OWN][4];
 #pragma unroll
     for (int tg = 0; tg < BT; tg += C::GT) {
       uint64_t P[C::GT][4], R[C::GT][4];
@@ -533,8 +562,9 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
         ulonglong2 k[C::GT], q[C::GT];
 #pragma unroll
         for (int t = 0; t < C::GT; ++t) {
-          k[t] = *reinterpret_cast<const ulonglong2*>(mine + (tg + t) * C::DK + 4 * LPG * x);
-          q[t] = *reinterpret_cast<const ulonglong2*>(theirs + (tg + t) * C::DK + 4 * LPG * x);
+          const int at = (C::REPS == 1 ? tg + t : (tg + t) ^ rep) * C::DK + 4 * LPG * x;
+          k[t] = *reinterpret_cast<const ulonglong2*>(mine + at);
+          q[t] = *reinterpret_cast<const ulonglong2*>(theirs + at);
         }
 #pragma unroll
         for (int t = 0; t < C::GT; ++t)
@@ -545,7 +575,7 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
 #pragma unroll
           for (int c = 0; c < 4; ++c) { P[t][c] = fma_f32x2(k[t].y, S[2 * x + 1][c], P[t][c]); R[t][c] = fma_f32x2(q[t].y, S[2 * x + 1][c], R[t][c]); }
       }
-      float f[C::GT][4], z[C::GT];
+      float w[C::GT][4];
 #pragma unroll
       for (int t = 0; t < C::GT; ++t)
 #pragma unroll
@@ -553,50 +583,63 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
           float p0, p1, r0, r1;
           unpack_f32x2(P[t][c], p0, p1);
           unpack_f32x2(R[t][c], r0, r1);
-          f[t][c] = p0 + p1 + __shfl_xor_sync(0xffffffffu, r0 + r1, LPG / 2);
+          w[t][c] = p0 + p1 + __shfl_xor_sync(0xffffffffu, r0 + r1, LPG / 2);
         }
+      // the tokens that share lanes
 #pragma unroll
-      for (int t = 0; t < C::GT; ++t) {
-        f[t][0] += __shfl_xor_sync(0xffffffffu, f[t][2], LPG / 4);
-        f[t][1] += __shfl_xor_sync(0xffffffffu, f[t][3], LPG / 4);
-      }
+      for (int o = C::REPS / 2; o > 0; o >>= 1)
 #pragma unroll
-      for (int t = 0; t < C::GT; ++t) z[t] = f[t][0] + __shfl_xor_sync(0xffffffffu, f[t][1], LPG / 8);
+        for (int t = 0; t < C::GT; ++t)
+          if (t % (2 * o) < o && t % C::REPS < 2 * o) {
 #pragma unroll
-      for (int o = LPG / 16; o > 0; o >>= 1)
+            for (int c = 0; c < 4; ++c) w[t][c] += __shfl_xor_sync(0xffffffffu, w[t + o][c], o);
+          }
 #pragma unroll
-        for (int t = 0; t < C::GT; ++t) z[t] += __shfl_xor_sync(0xffffffffu, z[t], o);
+      for (int t = 0; t < C::GT; t += C::REPS)
 #pragma unroll
-      for (int t = 0; t < C::GT; ++t) val[tg + t] = fmaf(z[t], st.gl[tg + t][type], st.v[type][tg + t][wcol + mycol]);
+        for (int c = 0; c < 4; ++c) f[(tg + t) / C::REPS][c] = w[t][c];
+    }
+    float val[C::OWN];
+#pragma unroll
+    for (int q = 0; q < C::OWN; ++q) {
+      f[q][0] += __shfl_xor_sync(0xffffffffu, f[q][2], LPG / 4);
+      f[q][1] += __shfl_xor_sync(0xffffffffu, f[q][3], LPG / 4);
+    }
+#pragma unroll
+    for (int q = 0; q < C::OWN; ++q) val[q] = f[q][0] + __shfl_xor_sync(0xffffffffu, f[q][1], LPG / 8);
+#pragma unroll
+    for (int q = 0; q < C::OWN; ++q) {
+      const int t = q * C::REPS + rep;
+      val[q] = fmaf(val[q], st.gl[t][type], st.v[type][t][wcol + mycol]);
     }
     // u = T x in the lanes that hold x, o = e^c S^T q + W x in the others
     float x[BT];
 #pragma unroll
-    for (int j = 0; j < BT; ++j) {
-      x[j] = __shfl_sync(0xffffffffu, val[j], lane & ~(LPG / 2));
-      if (type == 0) val[j] = 0.f;
+    for (int j = 0; j < BT; ++j) x[j] = __shfl_sync(0xffffffffu, val[j / C::REPS], (lane & ~(LPG / 2 | (C::REPS - 1))) + j % C::REPS);
+    if (type == 0) {
+#pragma unroll
+      for (int q = 0; q < C::OWN; ++q) val[q] = 0.f;
     }
 #pragma unroll
     for (int j4 = 0; j4 < BT / 4; ++j4)
 #pragma unroll
-      for (int i = 4 * j4; i < BT; ++i) {        // beyond the diagonal the rows hold zeros
-        const float4 m = *reinterpret_cast<const float4*>(&st.tw[i][type * BT + 4 * j4]);
-        val[i] = fmaf(m.x, x[4 * j4], fmaf(m.y, x[4 * j4 + 1], fmaf(m.z, x[4 * j4 + 2], fmaf(m.w, x[4 * j4 + 3], val[i]))));
+      for (int q = 4 * j4 / C::REPS; q < C::OWN; ++q) {          // beyond the diagonal the rows hold zeros
+        const float4 m = *reinterpret_cast<const float4*>(&st.tw[q * C::REPS + rep][type * BT + 4 * j4]);
+        val[q] = fmaf(m.x, x[4 * j4], fmaf(m.y, x[4 * j4 + 1], fmaf(m.z, x[4 * j4 + 2], fmaf(m.w, x[4 * j4 + 3], val[q]))));
       }
-    if (rep == 0) {
-      if (type == 0) {
+    if (type == 0) {
 #pragma unroll
-        for (int t = 0; t < BT; ++t) {
-          const float u = val[t] * st.gl[t][2];
-          s.u[warp][0][t][grp * 4 + mycol] = make_float2(u, u);
-          s.u[warp][1][t][grp * 4 + (mycol ^ 1)] = make_float2(u, u);
-        }
-      } else if (on) {
-        float* dst = vo + ((long long)qs + t0) * a.H * dv + (long long)h * dv + col + mycol;
-#pragma unroll
-        for (int t = 0; t < BT; ++t, dst += (long long)a.H * dv)
-          if (t < n) *dst = val[t];
+      for (int q = 0; q < C::OWN; ++q) {
+        const int t = q * C::REPS + rep;
+        const float u = val[q] * st.gl[t][2];
+        s.u[warp][0][t][grp * 4 + mycol] = make_float2(u, u);
+        s.u[warp][1][t][grp * 4 + (mycol ^ 1)] = make_float2(u, u);
       }
+    } else if (on) {
+      float* dst = vo + ((long long)qs + t0 + rep) * a.H * dv + (long long)h * dv + col + mycol;
+#pragma unroll
+      for (int q = 0; q < C::OWN; ++q, dst += (long long)C::REPS * a.H * dv)
+        if (q * C::REPS + rep < n) *dst = val[q];
     }
     __syncwarp();
     // the state behind the block
@@ -691,7 +734,7 @@ static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
   // few lanes per column keep the reductions short, many of them spread a small launch over the device
   const long long cols = (long long)a.num_seqs * a.H * a.dv;
   int lanes = a.lanes;
-  if (lanes == 0) lanes = cols / 16 >= 2 * 592 ? 8 : cols / 8 >= 592 ? 16 : 32;
+  if (lanes == 0) lanes = cols / 16 >= 888 ? 8 : cols / 8 >= 400 ? 16 : 32;
   if (a.dk > 128 && lanes < 16) lanes = 16;
   if (a.dk <= 32) e = launch_scan<4, 8>(a, st);
   else if (a.dk <= 64) e = lanes <= 8 ? launch_scan<8, 8>(a, st) : launch_scan<4, 16>(a, st);
