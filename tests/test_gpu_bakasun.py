@@ -490,3 +490,24 @@ def test_trace_runner(tmp_path, dtype):
     for step, rows in ((0, [3, 69, 8]), (1, [1]), (2, [32, 71])):
         got = torch.frombuffer(bytearray((tmp_path / f"{step}.f32").read_bytes()), dtype=torch.float32).reshape(len(rows), -1)
         assert C.row_error(got.double(), ref[rows]).median() < (5e-4 if dtype == "float32" else 0.3)
+
+
+def test_layers_with_the_delta_rule_alone():
+    """The mechanism as a layer's only mixer (another design's use of it): the GPU engine against the host engine."""
+    import dataclasses
+
+    from unillm_b200.engine.factory import build_cpu_engine
+
+    cfg = C.CASES["mixed"]
+    m = C.load_model(cfg, C.make_weights(cfg))
+    rule = dataclasses.replace(m.spec.layer(1).beside, mlp="dense", intermediate_size=40)
+    m.spec = dataclasses.replace(m.spec, layers=(rule, dataclasses.replace(rule, mlp=None), m.spec.layer(3)), num_layers=3, initializer_range=0.15)
+    m._init_params("random", seed=3)
+    m.p["layers.0.dt_bias"] = m.p["layers.0.dt_bias"] - 3.0
+    toks = C.tokens(cfg, 90, 2)
+    want = C.score(build_cpu_engine(m, num_blocks=16), toks, [(0, 90)])
+    for dtype in DTYPES:
+        for sizes in ([90], [33, 1, 2, 17], [1]):
+            eng = _engine(m, dtype)
+            _check_rows(C.score(eng, toks, C.portions(90, sizes)), want, dtype)
+            eng.runner.raise_on_device_error()
