@@ -33,8 +33,8 @@ class CpuModelRunner:
                 self.v_cache.append(self.v_cache[ls.kv_from])
                 continue
             heads, dk, dv = (1, ls.cache_row, 0) if ls.mixer == "latent" else (ls.num_kv_heads, ls.head_dim, ls.v_head_dim)
-            for cache, d in ((self.k_cache, dk), (self.v_cache, dv)):
-                cache.append(torch.zeros(num_blocks, heads, block_size, d, dtype=dt, device=dev) if ls.has_kv else None)
+            for cache, n, d in ((self.k_cache, heads * ls.maps, dk), (self.v_cache, heads, dv)):
+                cache.append(torch.zeros(num_blocks, n, block_size, d, dtype=dt, device=dev) if ls.has_kv else None)
         self.states: Dict[int, List[dict]] = {}         # state row -> what each layer carries on
         self._alibi = alibi_slopes(s.num_heads).to(dev) if s.pos == "alibi" else None
         self.launches = 0
@@ -46,6 +46,7 @@ class CpuModelRunner:
         L = f"layers.{i}."
         T = h.shape[0]
         rope = m._rope_cache(int(pos.max()) + 1, ls).at(pos) if ls.rotary_dim > 0 else None
+        vrope = m._value_rope(int(pos.max()) + 1, ls).at(pos) if ls.value_rope else None
         latent = ls.mixer == "latent"
         if latent:
             q, rows = m._latent_rows(i, h, rope)
@@ -56,12 +57,14 @@ class CpuModelRunner:
                 q = apply_rope(q, *rope, ls.rotary_dim, s.rope_interleaved)
                 if k is not None:
                     k = apply_rope(k, *rope, ls.rotary_dim, s.rope_interleaved)
+            if vrope is not None and v is not None:
+                v = apply_rope(v, *vrope, ls.v_head_dim, s.rope_interleaved)
         if k is not None:
             ok = slots >= 0
             blk, off = slots[ok] // self.block_size, slots[ok] % self.block_size
             self.k_cache[i][blk, :, off] = k[ok]
             self.v_cache[i][blk, :, off] = v[ok]
-        out = torch.empty(T, ls.num_heads, ls.v_head_dim, dtype=h.dtype, device=h.device)
+        out = torch.empty(T, ls.num_heads * ls.maps, ls.v_head_dim, dtype=h.dtype, device=h.device)
         row = 0
         q_lens = [1] * b.num_decode + list(b.prefill_q_lens)
         for si, ql in enumerate(q_lens):
@@ -71,7 +74,7 @@ class CpuModelRunner:
             if latent:
                 kk, vv = MX.latent_expand(m.p, L, ls, self.k_cache[i][bt][:, 0].flatten(0, 1)[:kv_len])
             else:
-                kk = self.k_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.head_dim)[:, :kv_len]
+                kk = self.k_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads * ls.maps, -1, ls.head_dim)[:, :kv_len]
                 vv = self.v_cache[i][bt].permute(1, 0, 2, 3).reshape(ls.num_kv_heads, -1, ls.v_head_dim)[:, :kv_len]
             qq = q[row:row + ql].transpose(0, 1).float()              # [H, ql, D]
             qpos = torch.arange(kv_len - ql, kv_len, device=h.device)[:, None]
@@ -79,13 +82,15 @@ class CpuModelRunner:
             vis = kpos <= qpos
             if ls.window > 0:
                 vis = vis & (kpos > qpos - ls.window)
+            if ls.chunk > 0:
+                vis = vis & (kpos // ls.chunk == qpos // ls.chunk)
             bias = torch.zeros(ql, kv_len, device=h.device).masked_fill(~vis, float("-inf"))
             if self._alibi is not None:
                 bias = bias[None] + self._alibi[:, None, None] * (kpos - qpos)[None].float()
             y = m._attend(i, qq[None], kk.float()[None], vv.float()[None], bias if bias.dim() == 2 else bias[None])[0]
             out[row:row + ql] = y.transpose(0, 1).to(h.dtype)
             row += ql
-        return ops_fn.linear(out.reshape(T, ls.o_size), m.p[L + "wo"], m.p.get(L + "bo"))
+        return ops_fn.linear(m._finish_attention(i, out, h, vrope), m.p[L + "wo"], m.p.get(L + "bo"))
 
     def _per_sequence(self, h: torch.Tensor, b: StepBatch, st: List[dict], fn) -> torch.Tensor:
         """``fn(rows [1, n, H], state)`` on the rows of each sequence of the step."""
@@ -121,11 +126,13 @@ class CpuModelRunner:
         nseq = len(b.seq_lens)
         read = b.state_in if b.state_in is not None else [-1] * nseq
         states = [copy.deepcopy(self.states[r]) if r >= 0 else [{} for _ in range(s.num_layers)] for r in read]
+        streams = [x]
         for i in range(s.num_layers):
             st = [d[i] for d in states]
             conv = lambda h, n, i=i, st=st: self._per_sequence(
-                h[0], b, st, lambda y, d: MX.input_conv(y, m.p[f"layers.{i}.{n}"], d, n))[None]
+                h[0], b, st, lambda y, d: MX.before_sublayer(y, m.p[f"layers.{i}.{n}"], d, n))[None]
             x = m.block(i, x[None], lambda h, i=i, st=st: self._mixer(i, h[0], b, pos, slots, st)[None], conv)[0]
+            x = m.after_layer(i, x, streams)
         for w, d in zip(b.state_out or (), states):
             if w >= 0:
                 self.states[w] = d

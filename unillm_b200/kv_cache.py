@@ -31,11 +31,11 @@ class LayerKVCache:
         return self.k is not None
 
     def append(self, k: torch.Tensor, v: torch.Tensor) -> None:
-        """k, v: ``[B, H, T_new, D]``."""
+        """k, v: ``[B, H, T_new, D]`` (either may have a head count and size of its own)."""
         B, H, T, D = k.shape
         if self.k is None:
             self.k = torch.zeros(B, H, self.max_seq_len, D, dtype=k.dtype, device=k.device)
-            self.v = torch.zeros(B, H, self.max_seq_len, v.shape[-1], dtype=v.dtype, device=v.device)
+            self.v = torch.zeros(B, v.shape[1], self.max_seq_len, v.shape[-1], dtype=v.dtype, device=v.device)
         if self.len + T > self.max_seq_len:
             raise MemoryError_(f"KV cache overflow: {self.len} + {T} > max_seq_len {self.max_seq_len}")
         self.k[:, :, self.len:self.len + T] = k

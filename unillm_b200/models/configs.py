@@ -1,4 +1,4 @@
-"""Configuration classes of all architectures: the reference's 47, Bakasun, Gekapel and Nipulorn.
+"""Configuration classes of all architectures: the reference's 47, Bakasun, Gekapel, Nipulorn and Tasadra.
 
 Field names and defaults follow the reference's ``model_config!`` blocks one for one
 (``crates/runtime/src/models_v2/<family>.rs``, e.g. ``llama.rs:20-38``, ``mixtral.rs:16-38``), so a
@@ -1057,6 +1057,30 @@ class T5Config:
     is_gated_act: bool = False
     hidden_size: int = 512
     num_hidden_layers: int = 6
+
+
+@model_config
+class TasadraConfig:
+    """Tasadra: every layer is described on its own.  ``layers[i]`` holds ``type`` ("attention"; "channel_delta": a gated delta
+    rule with one decay per key channel; "attention_2": differential attention in chunks), ``mixer`` and ``mlp`` (kind "dense"
+    with ``ff``, or null)."""
+
+    vocab_size: int = 32000
+    hidden_size: int = 2048
+    num_hidden_layers: int = 0
+    norm_eps: float = 1e-6
+    residual_mult: float = 1.0
+    layers: List[Any] = []
+    max_position_embeddings: int = 131072
+    initializer_range: float = 0.02
+
+    @classmethod
+    def from_hf_config(cls, d):
+        if "layers" not in d or "width" not in d:
+            return super(TasadraConfig, cls).from_hf_config(d)
+        kw = {k: d[k] for k in ("max_position_embeddings", "initializer_range", "residual_mult") if k in d}
+        return cls(vocab_size=d["vocab"], hidden_size=d["width"], num_hidden_layers=len(d["layers"]), norm_eps=d["norm"]["eps"],
+                   layers=list(d["layers"]), **kw)
 
 
 @model_config

@@ -79,6 +79,12 @@ class DecoderModel(Model):
                 shp[L + "ln2.w"] = (H,)
                 if s.norm_bias:
                     shp[L + "ln2.b"] = (H,)
+            if s.norm == "tanh":
+                shp.update({L + n + ".alpha": () for n in ("ln1", "ln2") if L + n + ".w" in shp})
+            if s.token_shift:
+                shp[L + "shift"] = (H,)
+            if s.depth_average:
+                shp[L + "dwa"] = (i + 2,)
             if s.norm_placement == "both":
                 shp[L + "ln1b.w"] = (H,)
                 if ls.mlp is not None:
@@ -100,6 +106,10 @@ class DecoderModel(Model):
                         shp[L + "k_norm"] = (ls.k_size if kind == "row" else ls.head_dim,)
                 if ls.sink:
                     shp[L + "sink"] = (ls.num_heads,)
+                if ls.out_gate:
+                    shp[L + "w_og"] = (ls.gate_size, H)
+                if ls.maps == 2:
+                    shp[L + "lambdas"] = (4, ls.head_dim)
                 shp[L + "wo"] = (H, ls.o_size)
                 if s.o_bias:
                     shp[L + "bo"] = (H,)
@@ -138,6 +148,8 @@ class DecoderModel(Model):
             shp["final_norm.w"] = (H,)
             if s.norm_bias:
                 shp["final_norm.b"] = (H,)
+            if s.norm == "tanh":
+                shp["final_norm.alpha"] = ()
         if not s.tie_embeddings:
             shp["lm_head"] = (s.vocab_size, E)
         if s.lm_head_bias:
@@ -154,6 +166,11 @@ class DecoderModel(Model):
                 t = torch.zeros(shape, dtype=dtype)
             elif name.endswith(("q_norm", "k_norm")) and self.spec.layers is not None:
                 t = torch.ones(shape, dtype=dtype)
+            elif name.endswith(".alpha"):
+                t = torch.full(shape, 0.5, dtype=dtype)
+            elif name.endswith(".dwa"):                                      # the layer's own result
+                t = torch.zeros(shape, dtype=dtype)
+                t[-1] = 1.0
             elif is_norm_w:
                 t = torch.zeros(shape, dtype=dtype) if self.spec.norm_weight_offset_one else torch.ones(shape, dtype=dtype)
             elif name.endswith(("q_a_norm", "kv_a_norm", "o_norm")):         # weights that are not stored around zero
@@ -183,17 +200,26 @@ class DecoderModel(Model):
         return None
 
     def _complete_spec(self, weights: ModelWeights) -> DecoderSpec:
-        """The spec with the sizes that only the tensors' shapes give (the rank of a wkv layer's decay)."""
+        """The spec with the sizes that only the tensors' shapes give (the ranks of low-rank decays and gates)."""
         s = self.spec
-        if s.layers is None or all(ls.mixer != "wkv" or ls.decay_rank for ls in s.layers):
+        if s.layers is None:
             return s
         layers = list(s.layers)
         for i, ls in enumerate(layers):
-            if ls.mixer == "wkv" and not ls.decay_rank:
-                t = self._find(weights, tuple(p.format(i=i) for p in self.scheme.layer), self.scheme.mixers["wkv"]["w_d1"])
+            need = {}
+            if ls.mixer == "wkv":
+                need["decay_rank"] = "w_d1"
+            if ls.mixer == "delta" and ls.decay == "channel":
+                need["decay_rank"] = "w_a1"
+            if ls.mixer == "delta" and ls.low_rank_gate:
+                need["gate_rank"] = "w_g1"
+            for rank, name in need.items():
+                if getattr(ls, rank):
+                    continue
+                t = self._find(weights, tuple(p.format(i=i) for p in self.scheme.layer), self.scheme.mixers[ls.mixer][name])
                 if t is None:
-                    raise LoadingError(f"{type(self).__name__}: missing weight layer {i} decay")
-                layers[i] = dataclasses.replace(ls, decay_rank=t.shape[0])
+                    raise LoadingError(f"{type(self).__name__}: missing weight layer {i} {name}")
+                layers[i] = dataclasses.replace(layers[i], **{rank: t.shape[0]})
         return dataclasses.replace(s, layers=tuple(layers))
 
     def _side(self, names, i: int, second: bool = False):
@@ -261,7 +287,10 @@ class DecoderModel(Model):
                 if s.norm_bias:
                     b = self._find(weights, pre, k.ln2, ".bias")
                     out[L + "ln2.b"] = b if b is not None else torch.zeros(s.hidden_size)
-            for n, names in (("ln1b.w", k.ln1b), ("ln2b.w", k.ln2b), ("conv1", k.conv1), ("conv2", k.conv2), ("act", k.act)):
+            for n, names in (("ln1", k.ln1), ("ln2", k.ln2)):
+                if L + n + ".alpha" in shapes:
+                    out[L + n + ".alpha"] = need(self._find_slope(weights, pre, names), f"layer {i} {n} slope")
+            for n, names in (("shift", k.shift), ("dwa", k.depth_average), ("ln1b.w", k.ln1b), ("ln2b.w", k.ln2b), ("conv1", k.conv1), ("conv2", k.conv2), ("act", k.act)):
                 if L + n in shapes:
                     out[L + n] = need(self._find(weights, pre, names), f"layer {i} {n}")
             # ---- mixer ----
@@ -288,7 +317,7 @@ class DecoderModel(Model):
                     out[L + "w_up"] = need(T(self._find(weights, pre, k.up)), f"layer {i} fc1")
                     if s.mlp_bias:
                         b = self._find(weights, pre, k.up, ".bias")
-                        out[L + "b_up"] = b if b is not None else torch.zeros(s.intermediate_size)
+                        out[L + "b_up"] = b if b is not None else torch.zeros(s.layer_intermediate(i))
                 dn = T(self._find(weights, pre, k.down))
                 if dn is None:
                     dn = deq([p + n + ".weight" for p in pre for n in k.down])
@@ -327,6 +356,8 @@ class DecoderModel(Model):
             if s.norm_bias:
                 b = self._find(weights, root, k.final_norm, ".bias")
                 out["final_norm.b"] = b if b is not None else torch.zeros(s.hidden_size)
+            if s.norm == "tanh":
+                out["final_norm.alpha"] = need(self._find_slope(weights, root, k.final_norm), "final norm slope")
         if not s.tie_embeddings:
             lm = self._find(weights, root, k.lm_head)
             if lm is None:
@@ -343,6 +374,11 @@ class DecoderModel(Model):
         self.p = {n: t.to(device=dev, dtype=dtype).contiguous() for n, t in out.items() if n in shapes}
         self.device, self.dtype = dev, dtype
         self._rope = self._alibi = None
+
+    def _find_slope(self, weights: ModelWeights, pre, names):
+        """The scalar slope of a Dynamic Tanh (stored with or without an axis)."""
+        t = self._find(weights, pre, tuple(n + self.scheme.alpha_suffix for n in names))
+        return None if t is None else t.reshape(())
 
     def _load_attention(self, weights: ModelWeights, i: int, pre, out: Dict[str, torch.Tensor], T, need, deq) -> None:
         """Projections, head norms and sinks of one layer's attention."""
@@ -382,6 +418,10 @@ class DecoderModel(Model):
                 out[L + "k_norm"] = need(self._find(weights, pre, nkn), "k_norm")
         if ls.sink:
             out[L + "sink"] = need(self._find(weights, pre, nsink, ""), f"layer {i} sinks")
+        if ls.out_gate:
+            out[L + "w_og"] = need(self._find(weights, pre, k.out_gate), f"layer {i} output gate")
+        if ls.maps == 2:
+            out[L + "lambdas"] = torch.stack([need(self._find(weights, pre, (n,)), f"layer {i} {n}") for n in k.lambdas])
         wo = T(self._find(weights, pre, no))
         if wo is None:
             wo = deq([p + n + ".weight" for p in pre for n in no])
@@ -455,7 +495,10 @@ class DecoderModel(Model):
                 out[pre + k.ln2[0] + WS] = self.p[L + "ln2.w"]
                 if s.norm_bias:
                     out[pre + k.ln2[0] + BS] = self.p[L + "ln2.b"]
-            for n, names, suffix in (("ln1b.w", k.ln1b, WS), ("ln2b.w", k.ln2b, WS), ("conv1", k.conv1, WS), ("conv2", k.conv2, WS),
+            for n, names in (("ln1", k.ln1), ("ln2", k.ln2)):
+                if L + n + ".alpha" in self.p:
+                    out[pre + names[0] + k.alpha_suffix + WS] = self.p[L + n + ".alpha"]
+            for n, names, suffix in (("shift", k.shift, WS), ("dwa", k.depth_average, WS), ("ln1b.w", k.ln1b, WS), ("ln2b.w", k.ln2b, WS), ("conv1", k.conv1, WS), ("conv2", k.conv2, WS),
                                      ("act", k.act, WS)):
                 if L + n in self.p:
                     out[pre + names[0] + suffix] = self.p[L + n]
@@ -487,6 +530,10 @@ class DecoderModel(Model):
                         out[pre + side(k.k_norm) + WS] = self.p[L + "k_norm"]
                 if ls.sink:
                     out[pre + side(k.sink)] = self.p[L + "sink"]
+                if ls.out_gate:
+                    out[pre + k.out_gate[0] + WS] = self.p[L + "w_og"]
+                if ls.maps == 2:
+                    out.update({pre + n + WS: t for n, t in zip(k.lambdas, self.p[L + "lambdas"].unbind(0))})
                 out[pre + side(k.o) + WS] = T(self.p[L + "wo"])
                 if s.o_bias:
                     out[pre + side(k.o) + BS] = self.p[L + "bo"]
@@ -533,6 +580,8 @@ class DecoderModel(Model):
             out[k.final_norm[0] + WS] = self.p["final_norm.w"]
             if s.norm_bias:
                 out[k.final_norm[0] + BS] = self.p["final_norm.b"]
+            if s.norm == "tanh":
+                out[k.final_norm[0] + k.alpha_suffix + WS] = self.p["final_norm.alpha"]
         if not s.tie_embeddings:
             out[k.lm_head[0] + WS] = self.p["lm_head"]
         if s.lm_head_bias:
@@ -560,6 +609,8 @@ class DecoderModel(Model):
                 eps = s.ref_layer_eps
             if s.ref_ln_star:
                 return ops_fn.layer_norm(x, w, None, eps)
+        if s.norm == "tanh":
+            return (torch.tanh(_f(self.p[name + ".alpha"]) * _f(x)) * _f(w) + _f(b)).to(x.dtype)
         if s.norm == "layer":
             return ops_fn.layer_norm(x, w, b, eps)
         if s.norm_weight_offset_one:
@@ -581,9 +632,14 @@ class DecoderModel(Model):
                                             linear=ls.rope_linear, device=self.device)
         return c
 
+    def _value_rope(self, need_len: int, ls: LayerSpec) -> RoPECache:
+        """Tables of the rotation of a layer's values: all their dimensions, no scaling."""
+        return self._rope_cache(need_len, dataclasses.replace(ls, head_dim=ls.v_head_dim, rotary_dim=ls.v_head_dim, rope_llama3=None,
+                                                              rope_yarn=None, rope_linear=1.0))
+
     def _project_qkv(self, i: int, h: torch.Tensor):
         """(q, k, v) of layer ``i`` as [..., heads, size] before rotation, normalised where the design has it; k and v
-        are None when the layer reads another layer's."""
+        are None when the layer reads another layer's.  With two maps a head's two queries (keys) lie side by side."""
         s, ls = self.spec, self.spec.layer(i)
         L = f"layers.{i}."
         qkv = ops_fn.linear(h, self.p[L + "wqkv"], self.p.get(L + "bqkv"))
@@ -594,13 +650,13 @@ class DecoderModel(Model):
             q, k, v = qkv.split([ls.q_size, ls.k_size, ls.v_size], dim=-1)
             if kind == "row":
                 k = ops_fn.rms_norm(k.contiguous(), self.p[L + "k_norm"], s.norm_eps)
-            k = k.reshape(*lead, ls.num_kv_heads, ls.head_dim)
+            k = k.reshape(*lead, ls.num_kv_heads * ls.maps, ls.head_dim)
             v = v.reshape(*lead, ls.num_kv_heads, ls.v_head_dim)
         else:
             q = qkv
         if kind == "row":
             q = ops_fn.rms_norm(q.contiguous(), self.p[L + "q_norm"], s.norm_eps)
-        q = q.reshape(*lead, ls.num_heads, ls.head_dim)
+        q = q.reshape(*lead, ls.num_heads * ls.maps, ls.head_dim)
         if kind == "head":
             q = ops_fn.rms_norm(q, self.p[L + "q_norm"], s.norm_eps)
             if k is not None:
@@ -639,10 +695,14 @@ class DecoderModel(Model):
         return (sa * _f(a) + sb * _f(b)).to(a.dtype)
 
     def _attend(self, i: int, q, k, v, bias):
-        """q [B, Hq, T, Dk], k / v [B, Hkv, S, ...] in fp32, additive ``bias`` [T, S] or [Hq, T, S] -> [B, Hq, T, Dv]."""
+        """q [B, Hq, T, Dk], k / v [B, Hkv, S, ...] in fp32, additive ``bias`` [T, S] or [Hq, T, S] -> [B, Hq, T, Dv]; with two
+        maps per head q, k and the result have twice the heads."""
         ls = self.spec.layer(i)
         g = ls.num_heads // ls.num_kv_heads
-        if g > 1:
+        if ls.maps > 1:
+            k = k.unflatten(1, (ls.num_kv_heads, ls.maps)).repeat_interleave(g, dim=1).flatten(1, 2)
+            v = v.repeat_interleave(g * ls.maps, dim=1)
+        elif g > 1:
             k, v = k.repeat_interleave(g, dim=1), v.repeat_interleave(g, dim=1)
         scale = ls.scale if ls.scale is not None else 1.0 / math.sqrt(ls.head_dim)
         if not ls.sink and ls.fixed_sink is None and not ls.softcap:
@@ -661,11 +721,25 @@ class DecoderModel(Model):
         p = torch.softmax(torch.cat([sc, sink], dim=-1), dim=-1)[..., :-1]
         return torch.matmul(p, v)
 
+    def _finish_attention(self, i: int, y: torch.Tensor, h: torch.Tensor, vrope) -> torch.Tensor:
+        """y [.., T, heads, Dv] of the attention over what the layer read, h [.., T, H] -> rows for the output projection: values
+        turned back, maps subtracted, output gate."""
+        s, ls, L = self.spec, self.spec.layer(i), f"layers.{i}."
+        if ls.maps == 2:
+            y = MX.difference(ls, self.p[L + "lambdas"], _f(y), s.norm_eps)
+        if vrope is not None:
+            y = apply_rope(y, vrope[0], -vrope[1], ls.v_head_dim, s.rope_interleaved)
+        if ls.out_gate:
+            g = torch.sigmoid(_f(ops_fn.linear(h, self.p[L + "w_og"])))
+            y = _f(y) * (g.unsqueeze(-1) if ls.out_gate == "head" else g.unflatten(-1, (ls.num_heads, ls.v_head_dim)))
+        return y.flatten(-2).to(h.dtype)
+
     def _attention(self, i: int, h: torch.Tensor, past: int, cache: Optional[KVCache], shared: dict) -> torch.Tensor:
         s, ls = self.spec, self.spec.layer(i)
         L = f"layers.{i}."
         B, T, _ = h.shape
         rope = self._rope_cache(past + T, ls).get_range(past, past + T) if ls.rotary_dim > 0 else None
+        vrope = self._value_rope(past + T, ls).get_range(past, past + T) if ls.value_rope else None
         if ls.mixer == "latent":
             q, rows = self._latent_rows(i, h, rope)
             rows = rows[:, None]                              # one row of width kv_rank + rot_dim for all heads
@@ -679,6 +753,8 @@ class DecoderModel(Model):
                 q = apply_rope(q, *rope, ls.rotary_dim, s.rope_interleaved)
                 if k is not None:
                     k = apply_rope(k, *rope, ls.rotary_dim, s.rope_interleaved)
+            if vrope is not None and v is not None:
+                v = apply_rope(v, *vrope, ls.v_head_dim, s.rope_interleaved)
         if ls.mixer == "latent":
             pass
         elif ls.kv_from is not None:
@@ -697,13 +773,15 @@ class DecoderModel(Model):
         vis = kpos <= qpos
         if ls.window > 0:
             vis = vis & (kpos > qpos - ls.window)
+        if ls.chunk > 0:
+            vis = vis & (kpos // ls.chunk == qpos // ls.chunk)
         bias = torch.zeros(T, S, device=h.device, dtype=torch.float32).masked_fill(~vis, float("-inf"))
         if s.pos == "alibi":
             if self._alibi is None or self._alibi.device != h.device:
                 self._alibi = alibi_slopes(s.num_heads).to(h.device)
             bias = bias[None] + self._alibi[:, None, None] * (kpos - qpos)[None].float()
         y = self._attend(i, _f(q), _f(k), _f(v), bias)
-        y = y.transpose(1, 2).reshape(B, T, ls.o_size).to(h.dtype)
+        y = self._finish_attention(i, y.transpose(1, 2), h, vrope)
         return ops_fn.linear(y, self.p[L + "wo"], self.p.get(L + "bo"))
 
     def _dense_mlp(self, x, w_gate_up=None, w_up=None, b_up=None, w_down=None, b_down=None, act="silu", act_p=None):
@@ -773,7 +851,7 @@ class DecoderModel(Model):
 
     def block(self, i: int, x: torch.Tensor, attention, conv=None) -> torch.Tensor:
         """One layer around ``attention(h)``: where the norms sit and how the sublayers join the residual stream.
-        ``conv(h, name)`` puts the input convolution of that name in front of a sublayer."""
+        ``conv(h, name)`` puts the input convolution of that name (or the token shift) in front of a sublayer."""
         s = self.spec
         L = f"layers.{i}."
         rs = s.residual_scale
@@ -791,12 +869,19 @@ class DecoderModel(Model):
             h = self._norm(x, L + "ln2")
             return x + self._norm(self._mlp(i, conv(h, "conv2") if s.input_conv else h), L + "ln2b") * rs
         h = self._norm(x, L + "ln1")
-        a = attention(h)
+        a = attention(conv(h, "shift") if s.token_shift else h)
         if s.parallel_residual:
             m_in = h if s.parallel_shared_norm else self._norm(x, L + "ln2")
             return x + (a + self._mlp(i, m_in)) * rs
         x = x + a * rs
         return x if s.layer(i).mlp is None else x + self._mlp(i, self._norm(x, L + "ln2")) * rs
+
+    def after_layer(self, i: int, x: torch.Tensor, streams: List[torch.Tensor]) -> torch.Tensor:
+        """What goes on behind layer ``i``, whose result is ``x``; ``streams`` collects the results."""
+        if not self.spec.depth_average:
+            return x
+        streams.append(x)
+        return sum(w * t.to(w.dtype) for w, t in zip(_f(self.p[f"layers.{i}.dwa"]), streams)).to(x.dtype)
 
     def hidden_states(self, input_ids: torch.Tensor, cache: Optional[KVCache] = None,
                       inputs_embeds: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -820,11 +905,13 @@ class DecoderModel(Model):
             x = x + self.p["pos_embed"][pos][None]
         if s.embed_norm:
             x = ops_fn.layer_norm(x, self.p["embed_norm.w"], self.p["embed_norm.b"], s.norm_eps)
+        streams = [x]                         # for the depth average
         shared: dict = {}                     # keys and values of this call's layers, for those that read an earlier one's
         for i in range(s.num_layers):
             st: dict = cache.layer(i).state if cache is not None else {}
             x = self.block(i, x, lambda h, i=i, st=st: self.mixer(i, h, past, cache, shared, st),
-                           lambda h, n, i=i, st=st: MX.input_conv(h, self.p[f"layers.{i}.{n}"], st, n))
+                           lambda h, n, i=i, st=st: MX.before_sublayer(h, self.p[f"layers.{i}.{n}"], st, n))
+            x = self.after_layer(i, x, streams)
         if cache is not None:
             cache.set_seq_len(past + T)
         if s.final_norm:

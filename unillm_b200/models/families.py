@@ -629,6 +629,78 @@ class BakasunModel(DecoderModel):
                            initializer_range=c.initializer_range)
 
 
+class TasadraModel(DecoderModel):
+    """Tasadra: Dynamic Tanh in front of every sublayer of a 32-bit residual stream whose additions are scaled, a token shift in
+    front of every mixer, and behind every layer a learned average over the embedding and all layers so far.  Mixers: attention
+    with query and key norms, YaRN rotation, rotated values, capped scores and a gate per head; a gated delta rule whose state
+    decays per key channel; differential attention in chunks with a gate per element, whose keys and values a later layer may
+    share.  Squared-relu feed-forwards with biases.  Not one of the reference's families."""
+
+    config_class = C.TasadraConfig
+    scheme = KeyScheme(embed=("embed",), layer=("l{i}.",), ln1=("norm1",), ln2=("norm2",), q=("mix.q",), k=("mix.k",), v=("mix.v",),
+                       q_norm=("mix.q.norm",), k_norm=("mix.k.norm",), out_gate=("mix.g",), o=("mix.o",), up=("mlp.up",),
+                       down=("mlp.down",), shift=("shift",), depth_average=("dwa",), final_norm=("final.norm",), lm_head=("head",),
+                       weight_suffix="", bias_suffix=".b", lambdas=("mix.lq1", "mix.lk1", "mix.lq2", "mix.lk2"),
+                       mixers={"delta": {"w_qkv": ("mix.q", "mix.k", "mix.v"), "conv": ("mix.q.conv", "mix.k.conv", "mix.v.conv"),
+                                         "w_b": ("mix.b",), "w_a1": ("mix.a1",), "w_a2": ("mix.a2",), "A_log": ("mix.A_log",),
+                                         "dt_bias": ("mix.dt_bias",), "w_g1": ("mix.g1",), "w_g2": ("mix.g2",),
+                                         "o_norm": ("mix.norm",), "wo": ("mix.o",)}})
+
+    @staticmethod
+    def _heads(i: int, mx: dict) -> dict:
+        if mx["heads"] % mx["kv_heads"]:
+            raise ConfigurationError(f"layer {i}: {mx['heads']} heads over {mx['kv_heads']} key heads")
+        return dict(num_heads=mx["heads"], num_kv_heads=mx["kv_heads"], head_dim=mx["dim"], v_head_dim=mx["vdim"])
+
+    @classmethod
+    def _attention_spec(cls, i: int, mx: dict, ff: dict) -> LayerSpec:
+        rot = mx["rot"]
+        sc = rot.get("scaling")
+        if rot["dims"] > mx["dim"] or rot["dims"] % 2 or mx["vdim"] % 2:
+            raise ConfigurationError(f"layer {i}: {rot['dims']} rotated dimensions of {mx['dim']}, values of {mx['vdim']}")
+        return LayerSpec(**cls._heads(i, mx), chunk=mx["mask"]["size"] if mx.get("mask") else 0, scale=float(mx["scale"]),
+                         rotary_dim=rot["dims"], rope_theta=float(rot["base"]), value_rope=True,
+                         rope_yarn=None if sc is None else tuple(float(sc[n]) for n in ("factor", "original", "fast", "slow")),
+                         softcap=float(mx.get("softcap") or 0.0), qk_norm="head", out_gate="head", **ff)
+
+    @classmethod
+    def _differential_spec(cls, i: int, mx: dict, layers, ff: dict) -> LayerSpec:
+        src = mx.get("kv_from")
+        if src is not None:
+            if not 0 <= src < i or layers[src]["type"] != "attention_2" or layers[src]["mixer"].get("kv_from") is not None:
+                raise ConfigurationError(f"layer {i}: kv_from {src} is not an earlier layer of this kind with keys of its own")
+            if any(layers[src]["mixer"][n] != mx[n] for n in ("kv_heads", "dim", "vdim")):
+                raise ConfigurationError(f"layer {i}: keys of layer {src} have other sizes")
+        return LayerSpec(**cls._heads(i, mx), chunk=mx["mask"]["size"] if mx.get("mask") else 0, scale=float(mx["scale"]), kv_from=src,
+                         softcap=float(mx.get("softcap") or 0.0), qk_norm="", maps=2, diff=float(mx["diff"]), out_gate="element", **ff)
+
+    @classmethod
+    def _layer_spec(cls, i: int, d: dict, layers) -> LayerSpec:
+        mx, mlp = d["mixer"], d.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ConfigurationError(f"layer {i}: unknown feed-forward {mlp.get('kind')!r}")
+        ff = dict(mlp=None if mlp is None else "dense", intermediate_size=None if mlp is None else mlp["ff"])
+        if d["type"] == "attention":
+            return cls._attention_spec(i, mx, ff)
+        if d["type"] == "channel_delta":
+            return LayerSpec(**cls._heads(i, mx), mixer="delta", conv_taps=mx["conv"], decay="channel", low_rank_gate=True,
+                             gate_act="sigmoid", **ff)
+        if d["type"] == "attention_2":
+            return cls._differential_spec(i, mx, layers, ff)
+        raise ConfigurationError(f"layer {i}: unknown mixer {d['type']!r}")
+
+    @classmethod
+    def spec_from_config(cls, c):
+        layers = tuple(cls._layer_spec(i, d, c.layers) for i, d in enumerate(c.layers))
+        first = layers[0] if layers else None
+        return DecoderSpec(vocab_size=c.vocab_size, hidden_size=c.hidden_size, num_layers=len(layers), layers=layers,
+                           num_heads=first.num_heads if first else 0, num_kv_heads=first.num_kv_heads if first else 0,
+                           head_dim=first.head_dim if first else 0, intermediate_size=0,
+                           max_position_embeddings=c.max_position_embeddings, norm="tanh", norm_eps=c.norm_eps, norm_bias=True,
+                           residual_fp32=True, residual_scale=c.residual_mult, token_shift=True, depth_average=True, mlp="plain",
+                           act="relu2", mlp_bias=True, initializer_range=c.initializer_range)
+
+
 DECODER_FAMILIES = {
     "llama": LlamaModel, "qwen": QwenModel, "gemma": GemmaModel, "phi": PhiModel, "deepseek": DeepSeekModel,
     "mistral": MistralModel, "mixtral": MixtralModel, "gpt2": GPT2Model, "gptj": GPTJModel, "gptneox": GPTNeoXModel,
@@ -636,5 +708,5 @@ DECODER_FAMILIES = {
     "olmo": OlmoModel, "granite": GraniteModel, "yi": YiModel, "falcon": FalconModel, "baichuan": BaichuanModel,
     "internlm": InternLMModel, "chatglm": ChatGLMModel, "minicpm": MiniCPMModel, "deepseek_moe": DeepSeekMoEModel,
     "dbrx": DbrxModel, "grok": GrokModel, "arctic": ArcticModel, "gekapel": GekapelModel,
-    "nipulorn": NipulornModel, "bakasun": BakasunModel,
+    "nipulorn": NipulornModel, "bakasun": BakasunModel, "tasadra": TasadraModel,
 }

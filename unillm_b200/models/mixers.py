@@ -1,13 +1,14 @@
 """Sublayer parts of per-layer specs beyond plain attention: latent attention, the wkv recurrence, the gated delta rule, the
-input convolution and the xIELU activation, as PyTorch on any device -- the whole-model path and the CPU runner; the serving
-kernels are ``csrc/attn/attn_latent.cu``, ``csrc/wkv/wkv_mixer.cu``, ``csrc/delta/delta_mixer.cu`` and
-``csrc/norm/sublayer_in.cu``.
+difference of two attention maps, the input convolution, the token shift and the xIELU activation, as PyTorch on any device --
+the whole-model path and the CPU runner; the serving kernels are ``csrc/attn/attn_latent.cu``, ``csrc/attn/attn_finish.cu``,
+``csrc/wkv/wkv_mixer.cu``, ``csrc/delta/delta_mixer.cu``, ``csrc/norm/sublayer_in.cu`` and ``csrc/norm/stream_in.cu``.
 
 State that a sequence carries lives in a dictionary per layer (``st``); a missing entry stands for the start of a sequence.
 
 Latent attention follows DeepSeek-V2 ("DeepSeek-V2: A Strong, Economical, and Efficient Mixture-of-Experts Language
 Model"), the recurrence RWKV-6 (the reference's ``models_v2/rwkv6.rs:483-553`` in another parametrisation), the delta rule
-with decay "Gated Delta Networks: Improving Mamba2 with Delta Rule" (Yang, Kautz, Hatamizadeh).
+with decay "Gated Delta Networks: Improving Mamba2 with Delta Rule" (Yang, Kautz, Hatamizadeh), the difference of maps
+"Differential Transformer" (Ye et al.).
 """
 from __future__ import annotations
 
@@ -35,8 +36,11 @@ def mixer_shapes(ls: LayerSpec, H: int) -> Dict[str, Tuple[int, ...]]:
         return {"mu": (5, H), "w_rkvg": (4, C, H), "w_d1": (ls.decay_rank, H), "w_d2": (C, ls.decay_rank), "d0": (C,),
                 "u": (n, d), "o_norm": (C,), "wo": (H, C)}
     if ls.mixer == "delta":
-        return {"w_qkv": (ls.conv_rows, H), "conv": (ls.conv_rows, ls.conv_taps), "w_b": (n, H), "w_a": (n, H), "A_log": (n,),
-                "dt_bias": (n,), "w_g": (ls.o_size, H), "o_norm": (ls.v_head_dim,), "wo": (H, ls.o_size)}
+        channels = n * d
+        decay = {"w_a1": (ls.decay_rank, H), "w_a2": (channels, ls.decay_rank)} if ls.decay == "channel" else {"w_a": (n, H)}
+        gate = {"w_g1": (ls.gate_rank, H), "w_g2": (ls.o_size, ls.gate_rank)} if ls.low_rank_gate else {"w_g": (ls.o_size, H)}
+        return {"w_qkv": (ls.conv_rows, H), "conv": (ls.conv_rows, ls.conv_taps), "w_b": (n, H), **decay, "A_log": (n,),
+                "dt_bias": (channels if ls.decay == "channel" else n,), **gate, "o_norm": (ls.v_head_dim,), "wo": (H, ls.o_size)}
     raise ValueError(f"no such mixer: {ls.mixer!r}")
 
 
@@ -64,6 +68,19 @@ def input_conv(h: torch.Tensor, w: torch.Tensor, st: dict, key: str) -> torch.Te
     if key not in st:
         st[key] = torch.zeros(h.shape[0], n, h.shape[2], dtype=h.dtype, device=h.device)
     return h + R.causal_dwconv1d(h, w, None, st[key])
+
+
+def token_shift(h: torch.Tensor, mix: torch.Tensor, st: dict) -> torch.Tensor:
+    """h [B, T, H]: every token's values mixed with those of the token before it."""
+    first = st["shift"] if "shift" in st else torch.zeros(h.shape[0], h.shape[2], dtype=h.dtype, device=h.device)
+    back = torch.cat([first[:, None], h[:, :-1]], 1)
+    st["shift"] = h[:, -1].clone()
+    return h + (back - h) * mix.to(h.dtype)
+
+
+def before_sublayer(h: torch.Tensor, w: torch.Tensor, st: dict, key: str) -> torch.Tensor:
+    """What stands between a norm and its sublayer: a token shift or an input convolution, by the parameter's name."""
+    return token_shift(h, w, st) if key == "shift" else input_conv(h, w, st, key)
 
 
 def wkv(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, st: dict, eps: float) -> torch.Tensor:
@@ -97,10 +114,28 @@ def delta(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, st
     unit = lambda x: x / torch.sqrt(x.pow(2).sum(-1, keepdim=True) + 1e-6)
     q, k = (unit(x.reshape(B, T, g, dk)).repeat_interleave(n // g, dim=2) for x in (q, k))
     beta = torch.sigmoid(ops_fn.linear(h, p[L + "w_b"]).float())
-    keep = torch.exp(-torch.exp(p[L + "A_log"].float()) * F.softplus(ops_fn.linear(h, p[L + "w_a"]).float() + p[L + "dt_bias"].float()))
+    if ls.decay == "channel":
+        raw = F.linear(ops_fn.linear(h, p[L + "w_a1"]).float(), p[L + "w_a2"].float()) + p[L + "dt_bias"].float()
+        keep = torch.exp(-torch.exp(p[L + "A_log"].float())[:, None] * F.softplus(raw).reshape(B, T, n, dk))
+    else:
+        keep = torch.exp(-torch.exp(p[L + "A_log"].float()) * F.softplus(ops_fn.linear(h, p[L + "w_a"]).float() + p[L + "dt_bias"].float()))
     o, st["delta"] = R.delta_rule(q * dk ** -0.5, k, v.reshape(B, T, n, dv), keep, beta, st["delta"])
     o = o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * p[L + "o_norm"].float()
-    return (o.reshape(B, T, n * dv) * F.silu(ops_fn.linear(h, p[L + "w_g"]).float())).to(h.dtype)
+    g = ops_fn.linear(ops_fn.linear(h, p[L + "w_g1"]), p[L + "w_g2"]) if ls.low_rank_gate else ops_fn.linear(h, p[L + "w_g"])
+    return (o.reshape(B, T, n * dv) * ops_fn.activation(ls.gate_act)(g.float())).to(h.dtype)
+
+
+def diff_lambda(ls: LayerSpec, lambdas: torch.Tensor) -> float:
+    """The factor on the second map of a differential attention; ``lambdas`` [4, head_dim]: q and k of map 1, of map 2."""
+    a = lambdas.detach().double().cpu()
+    return float(torch.exp((a[0] * a[1]).sum()) - torch.exp((a[2] * a[3]).sum())) + ls.diff
+
+
+def difference(ls: LayerSpec, lambdas: torch.Tensor, y: torch.Tensor, eps: float) -> torch.Tensor:
+    """y [.., heads * 2, v size], the two maps of a head side by side -> [.., heads, v size]."""
+    a1, a2 = y.unflatten(-2, (ls.num_heads, 2)).unbind(-2)
+    o = a1 - diff_lambda(ls, lambdas) * a2
+    return o / torch.sqrt(o.pow(2).mean(-1, keepdim=True) + eps) * (1.0 - ls.diff)
 
 
 def latent_project(p: Dict[str, torch.Tensor], L: str, ls: LayerSpec, h: torch.Tensor, eps: float):

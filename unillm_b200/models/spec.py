@@ -57,7 +57,11 @@ class LayerSpec:
     ``rot_dim`` shared by the heads; ``head_dim`` is the unrotated key size); "wkv" (RWKV-6 style recurrence with a
     ``head_dim`` x ``head_dim`` state per head, five token-shift mixes and a low-rank decay of ``decay_rank``); or "delta"
     (gated delta rule with a ``head_dim`` x ``v_head_dim`` state per head, queries and keys of ``num_kv_heads`` heads, and
-    causal convolutions of ``conv_taps`` taps on queries, keys and values).
+    causal convolutions of ``conv_taps`` taps on queries, keys and values; ``decay="channel"``: every row of the state decays at
+    its own rate, through a low-rank map of ``decay_rank``; ``low_rank_gate``: the output gate is a product of rank ``gate_rank``).
+
+    ``maps`` = 2: differential attention, two softmax maps per head over the same values (query and key rows lie head by head as
+    [map 1, map 2]); o = (a1 - lambda a2) / rms * (1 - ``diff``) with one learned lambda per layer.
 
     ``beside``: a second mixer that reads the same input; the first one's output times ``scales[0]`` and the second one's
     times ``scales[1]`` are added."""
@@ -67,6 +71,7 @@ class LayerSpec:
     head_dim: int                        # query / key size
     v_head_dim: int
     window: int = 0                      # keys p - window + 1 .. p; 0 = all
+    chunk: int = 0                       # keys of the query's own chunk of this many positions, counted from 0; 0 = all
     scale: Optional[float] = None        # None = 1/sqrt(head_dim)
     rotary_dim: int = 0
     rope_theta: float = 10000.0
@@ -88,6 +93,14 @@ class LayerSpec:
     decay_rank: int = 0
     intermediate_size: Optional[int] = None   # dense feed-forward width (None: the model's)
     conv_taps: int = 0
+    decay: str = "head"                  # delta: one decay per "head", or one per "channel" of its keys
+    low_rank_gate: bool = False
+    gate_rank: int = 0
+    gate_act: str = "silu"               # delta: activation of the output gate
+    value_rope: bool = False             # values turn by their position over all their dimensions, outputs turn back by the query's
+    out_gate: str = ""                   # the attention's output times sigmoid(W h): "head" = one number per head, "element", "" = none
+    maps: int = 1
+    diff: float = 0.0
     beside: Optional["LayerSpec"] = None
     scales: Tuple[float, float] = (1.0, 1.0)
 
@@ -112,11 +125,11 @@ class LayerSpec:
 
     @property
     def q_size(self) -> int:
-        return self.num_heads * (self.head_dim + self.rot_dim)
+        return self.num_heads * self.maps * (self.head_dim + self.rot_dim)
 
     @property
     def k_size(self) -> int:
-        return self.num_kv_heads * self.head_dim
+        return self.num_kv_heads * self.maps * self.head_dim
 
     @property
     def v_size(self) -> int:
@@ -125,6 +138,11 @@ class LayerSpec:
     @property
     def o_size(self) -> int:
         return self.num_heads * self.v_head_dim
+
+    @property
+    def gate_size(self) -> int:
+        """Rows of the attention's output gate."""
+        return {"": 0, "head": self.num_heads, "element": self.o_size}[self.out_gate]
 
     @property
     def qkv_size(self) -> int:
@@ -143,7 +161,7 @@ class DecoderSpec:
     intermediate_size: int = 11008
     max_position_embeddings: int = 2048
     # norms
-    norm: str = "rms"                    # "rms" | "layer"
+    norm: str = "rms"                    # "rms" | "layer" | "tanh" (Dynamic Tanh: tanh(alpha x) w + b, no statistics)
     norm_eps: float = 1e-6
     norm_bias: bool = False
     norm_weight_offset_one: bool = False  # Gemma: y * (1 + w)
@@ -173,6 +191,8 @@ class DecoderSpec:
     norm_placement: str = "input"        # "input": x + f(norm(x)) | "output": x + norm(f(x)), sublayers read x itself |
     #                                      "both": x + norm_b(f(norm(x)))
     input_conv: int = 0                  # taps of the causal depthwise convolution added to what every sublayer reads (0: none)
+    token_shift: bool = False            # a mixer reads h + (h of the previous token - h) * shift, per channel
+    depth_average: bool = False          # what leaves layer i is a learned weighted sum of the embedding and all layers' results
     residual_fp32: bool = False          # the residual stream is kept in 32 bits between the layers
     layers: Optional[Tuple[LayerSpec, ...]] = None   # per-layer description; None: all layers as the fields above say
     # scalings
@@ -240,12 +260,14 @@ class DecoderSpec:
     @property
     def state_elements(self) -> int:
         """fp32 elements of state that one sequence carries from token to token besides cache rows: the last inputs of the
-        convolutions, the previous token's input of the wkv layers and the recurrent state of the wkv and delta mixers."""
+        convolutions, the previous token's input of the wkv layers and of token shifts, and the recurrent state of the wkv and delta mixers."""
         n = 0
         for i in range(self.num_layers):
             ls = self.layer(i)
             if self.input_conv:
                 n += (self.input_conv - 1) * self.hidden_size * (2 if ls.mlp is not None else 1)
+            if self.token_shift:
+                n += self.hidden_size
             if ls.mixer == "wkv":
                 n += self.hidden_size + ls.num_heads * ls.head_dim * ls.head_dim
             for mx in ls.mixers:
@@ -292,6 +314,11 @@ class KeyScheme:
     conv1: Tuple[str, ...] = ()          # input convolutions
     conv2: Tuple[str, ...] = ()
     act: Tuple[str, ...] = ()            # learned numbers of the activation
+    shift: Tuple[str, ...] = ()          # token shift
+    depth_average: Tuple[str, ...] = ()  # weights of the depth average
+    out_gate: Tuple[str, ...] = ()       # output gate of an attention
+    lambdas: Tuple[str, ...] = ()        # the four vectors of a differential attention's lambda: q and k of map 1, of map 2
+    alpha_suffix: str = ".alpha"         # slope of a Dynamic Tanh, behind the norm's name
     mixers: Optional[dict] = None        # {mixer: {parameter: names, several = stacked or concatenated}}, see mixers.mixer_shapes
     sides: Optional[Tuple[str, str, str]] = None   # prefix of a mixer's names; what replaces it for the first and the second
     #                                                of two mixers side by side

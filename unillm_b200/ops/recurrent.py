@@ -224,12 +224,12 @@ def wkv6(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, w: torch.Tensor, u: 
 
 def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, keep: torch.Tensor, beta: torch.Tensor, state: torch.Tensor):
     """Delta rule with decay, token by token in fp32 (host form; on the device ``cuda_ops.delta_mixer``): ``q``, ``k``
-    [B, T, H, Dk], ``v`` [B, T, H, Dv], ``keep`` and ``beta`` [B, T, H], ``state`` [B, H, Dk, Dv] -> (outputs, new state)."""
+    [B, T, H, Dk], ``v`` [B, T, H, Dv], ``beta`` [B, T, H], ``keep`` [B, T, H] or one per row of the state [B, T, H, Dk], ``state`` [B, H, Dk, Dv] -> (outputs, new state)."""
     out = torch.empty_like(v)
     S = state
     for t in range(v.shape[1]):
         kt = k[:, t, :, :, None]
-        S = S * keep[:, t, :, None, None]
+        S = S * (keep[:, t, :, None, None] if keep.dim() == 3 else keep[:, t, :, :, None])
         u = beta[:, t, :, None] * (v[:, t] - (S * kt).sum(2))
         S = S + kt * u[:, :, None, :]
         out[:, t] = (S * q[:, t, :, :, None]).sum(2)
