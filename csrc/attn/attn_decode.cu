@@ -382,7 +382,7 @@ static int launch_mma(const UbAttnArgs& a, cudaStream_t st) {
 
 template <int D>
 static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
-  const bool plain = a.sinks == nullptr && a.softcap <= 0.f && (a.Dv == 0 || a.Dv == D);     // what the older kernels take
+  const bool plain = a.sinks == nullptr && a.softcap <= 0.f && a.chunk <= 0 && (a.Dv == 0 || a.Dv == D);     // what the older kernels take
   const bool mma_ok = (D <= 128 || !plain) && (decode_mma_enabled() || !plain) && ub_attn_decode_mma_supported(&a);
   if (a.merge_o != nullptr && (!mma_ok || a.splits != 1)) return -7;   // fused merge lives in the warp-MMA kernels only
   // one warp per item needs enough items to keep every SM's copy engines busy; with fewer, an item is better served by

@@ -89,7 +89,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
   // block-table entries together with the length instead of behind it (one dependent global latency less).
   int* bt_sm = reinterpret_cast<int*>(dsm + S::BT_OFF);
   const int* bt = a.block_tables + (long long)seq * a.max_blocks_per_seq;
-  const bool bt_early = a.window == 0 && a.splits == 1;
+  const bool bt_early = a.window == 0 && a.chunk == 0 && a.splits == 1;
   const int bs_shift = 31 - __clz(a.block_size);
   if (bt_early) {
     const int first = max(a.kv_start, 0) >> bs_shift;
@@ -98,6 +98,7 @@ __global__ void __launch_bounds__(128) attn_decode_mma_kernel(const UbAttnArgs a
   const int kv_len = a.seq_lens[seq];
   int lo = a.kv_start;
   if (a.window > 0) lo = max(lo, kv_len - a.window);
+  if (a.chunk > 0) lo = max(lo, max(kv_len - 1, 0) / a.chunk * a.chunk);
   lo = max(lo, 0);
   const int span = max(kv_len - lo, 0);
   int per = (span + a.splits - 1) / a.splits;
@@ -392,7 +393,7 @@ static int launch_sized(const UbAttnArgs& a, cudaStream_t st) {
 extern "C" int ub_attn_decode_mma_supported(const UbAttnArgs* a) {
   const int dv = a->Dv > 0 ? a->Dv : a->D;
   if (a->D > 256 || dv > 256 || a->D % 8 != 0 || dv % 8 != 0) return 0;
-  if (a->merge_o != nullptr && (a->D != dv || (dv != 64 && dv != 128) || a->sinks != nullptr || a->softcap > 0.f)) return 0;
+  if (a->merge_o != nullptr && (a->D != dv || (dv != 64 && dv != 128) || a->sinks != nullptr || a->softcap > 0.f || a->chunk > 0)) return 0;
   if (a->block_size < 8 || a->block_size > 64 || (a->block_size & (a->block_size - 1))) return 0;   // whole pages per 64-token tile
   if (a->Hkv <= 0 || a->Hq % a->Hkv != 0 || a->q_stride % 8 != 0) return 0;
   if ((reinterpret_cast<uintptr_t>(a->q) & 15) || (reinterpret_cast<uintptr_t>(a->k_cache) & 15) ||

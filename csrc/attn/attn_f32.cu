@@ -39,6 +39,7 @@ __global__ void __launch_bounds__(WARPS * 32) attn_f32_kernel(const UbAttnArgs a
   const int hi = a.causal || a.q_start == nullptr ? min(kv_len, qpos + 1) : kv_len;
   int lo = max(a.kv_start, 0);
   if (a.window > 0) lo = max(lo, qpos - a.window + 1);
+  if (a.chunk > 0) lo = max(lo, qpos / a.chunk * a.chunk);
   const float slope = a.alibi_slopes != nullptr ? a.alibi_slopes[h] : 0.f;
   float m = -CUDART_INF_F, l = 0.f, acc[MAX_D / 32];
 #pragma unroll

@@ -102,6 +102,7 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
   int kv_end = a.causal ? min(kv_len, last_qpos + 1) : kv_len;
   int kv_begin = max(a.kv_start, 0);
   if (a.window > 0) kv_begin = max(kv_begin, first_qpos - a.window + 1);
+  if (a.chunk > 0) kv_begin = max(kv_begin, max(first_qpos, 0) / a.chunk * a.chunk);
   kv_begin = kv_begin / KT * KT;
   const int ntiles = kv_end > kv_begin ? (kv_end - kv_begin + KT - 1) / KT : 0;
 
@@ -147,6 +148,14 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
   const int rowa = row0 + ra, rowb = row0 + rb;
   const int qpos_a = kv_len - q_len + min(rowa, rows_total - 1) / G;
   const int qpos_b = kv_len - q_len + min(rowb, rows_total - 1) / G;
+  // first key that a row sees
+  auto first_key = [&](int qpos) {
+    int lo = a.kv_start;
+    if (a.window > 0) lo = max(lo, qpos - a.window + 1);
+    if (a.chunk > 0) lo = max(lo, max(qpos, 0) / a.chunk * a.chunk);
+    return lo;
+  };
+  const int lo_a = first_key(qpos_a), lo_b = first_key(qpos_b);
   float slope_a = 0.f, slope_b = 0.f;
   if (a.alibi_slopes != nullptr) {
     slope_a = a.alibi_slopes[kvh * G + min(rowa, rows_total - 1) % G] * P_LOG2E;
@@ -217,9 +226,8 @@ __global__ void __launch_bounds__(128) attn_prefill_kernel(const UbAttnArgs a) {
         const int kpos = t0 + j * 8 + (lane & 3) * 2 + (e & 1);
         const bool rowsel_b = e >= 2;
         const int qpos = rowsel_b ? qpos_b : qpos_a;
-        bool vis = kpos < kv_end && kpos >= a.kv_start;
+        bool vis = kpos < kv_end && kpos >= (rowsel_b ? lo_b : lo_a);
         if (a.causal) vis = vis && kpos <= qpos;
-        if (a.window > 0) vis = vis && kpos > qpos - a.window;
         float v = s[j][e] * sc + (rowsel_b ? slope_b : slope_a) * (float)(kpos - qpos);
         v = vis ? v : -CUDART_INF_F;
         s[j][e] = v;
@@ -351,7 +359,7 @@ extern "C" int ub_attn_prefill_last_path() { return g_last_path; }
 extern "C" int ub_attn_prefill(const UbAttnArgs* a, void* stream_v) {
   using namespace ub;
   if (a->num_seqs <= 0 || a->max_q_len <= 0) return 0;
-  const bool plain = a->sinks == nullptr && a->softcap <= 0.f && (a->Dv == 0 || a->Dv == a->D);   // what the tensor-core kernel takes
+  const bool plain = a->sinks == nullptr && (a->Dv == 0 || a->Dv == a->D);   // what the tensor-core kernel takes
   if (plain && tc_enabled() && ub_attn_prefill_tc_supported(a)) {
     g_last_path = 1;
     return ub_attn_prefill_tc(a, stream_v);

@@ -18,8 +18,8 @@
 // 3-D tensor map (d, head, token) so that the packed-row order is produced by the copy itself.
 //
 // Handles head_dim 128, page size 16, causal (with offset, for chunked prefill and prefix-cache hits) or
-// bidirectional masks, optional log-sum-exp output for merging partial results.  Sliding windows, ALiBi and other
-// head sizes stay on the warp-MMA kernel (attn_prefill.cu).
+// bidirectional masks, chunks (a query sees its own chunk only), capped scores, optional log-sum-exp output for merging partial
+// results.  Sliding windows, ALiBi and other head sizes stay on the warp-MMA kernel (attn_prefill.cu).
 //
 // Replaces in the reference: ops_fn::flash_attention (crates/runtime/src/tensor_core.rs:1318-1383).
 #include <cuda.h>
@@ -89,6 +89,8 @@ struct Params {
   float scale_log2;
   int causal;
   int kv_start;     // first key position to attend (suffix pass after a shared prefix); 0 = all
+  int chunk;        // > 0: keys of the query's own chunk of this many positions only
+  float cap_in;     // scores s become cap * tanh(s * cap_in), scale_log2 then holds cap * log2(e); 0 = as they are
   const __nv_bfloat16* merge_o;   // optional partial over a disjoint key set, [T, Hq, HD] contiguous
   const float* merge_lse;         // its log-sum-exp, [T, Hq]
   // Key split: grid.z = num_seqs * kv_splits; CTA (seq, split) walks 1 / kv_splits of the visible KV tiles and writes
@@ -99,7 +101,44 @@ struct Params {
   int total_q;
 };
 
-template <bool P_TMEM>
+// tanh of a thread's 64 scores.  Where they are small for the whole warp (scores far below the cap), the first six terms of the
+// Taylor series, whose remainder is below 3e-8 up to the bound; else by the exponential.
+constexpr float TANH_SERIES = 0.4f;
+__device__ __forceinline__ void cap_scores(uint32_t (&sv)[2][32], float cap_in) {
+  const uint64_t in2 = pack_f32x2(cap_in, cap_in);
+  float mx = 0.f;
+#pragma unroll
+  for (int c = 0; c < 2; ++c)
+#pragma unroll
+    for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fabsf(__uint_as_float(sv[c][i])));
+  if (__all_sync(0xffffffffu, mx * cap_in < TANH_SERIES)) {
+    const uint64_t one = pack_f32x2(1.f, 1.f), c1 = pack_f32x2(-1.f / 3.f, -1.f / 3.f), c2 = pack_f32x2(2.f / 15.f, 2.f / 15.f);
+    const uint64_t c3 = pack_f32x2(-17.f / 315.f, -17.f / 315.f), c4 = pack_f32x2(62.f / 2835.f, 62.f / 2835.f);
+    const uint64_t c5 = pack_f32x2(-1382.f / 155925.f, -1382.f / 155925.f);
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int i = 0; i < 32; i += 2) {
+        const uint64_t x = mul_f32x2(pack_f32x2(__uint_as_float(sv[c][i]), __uint_as_float(sv[c][i + 1])), in2), q = mul_f32x2(x, x);
+        uint64_t p = fma_f32x2(q, c5, c4);
+        p = fma_f32x2(q, p, c3);
+        p = fma_f32x2(q, p, c2);
+        p = fma_f32x2(q, p, c1);
+        p = fma_f32x2(q, p, one);
+        float a, b;
+        unpack_f32x2(mul_f32x2(x, p), a, b);
+        sv[c][i] = __float_as_uint(a);
+        sv[c][i + 1] = __float_as_uint(b);
+      }
+  } else {
+#pragma unroll
+    for (int c = 0; c < 2; ++c)
+#pragma unroll
+      for (int i = 0; i < 32; ++i) sv[c][i] = __float_as_uint(tanh_by_exp(__uint_as_float(sv[c][i]) * cap_in));
+  }
+}
+
+template <bool P_TMEM, bool CAP>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                        const __grid_constant__ CUtensorMap tmap_v, const Params p) {
@@ -136,7 +175,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
   const int t_last = min(t0 + TOK, q_end) - 1;
   int kv_hi = p.causal ? min(kv_len, kv_len - q_len + (t_last - q_begin) + 1) : kv_len;
   if (kv_hi < 0) kv_hi = 0;
-  const int kv_lo = max(p.kv_start, 0);
+  int kv_lo = max(p.kv_start, 0);
+  if (p.chunk > 0) kv_lo = max(kv_lo, max(kv_len - q_len + (t0 - q_begin), 0) / p.chunk * p.chunk);     // of the first row
   int tile0 = kv_lo / BN;                                   // first KV tile that holds a visible key
   int n_tiles = kv_hi > kv_lo ? (kv_hi + BN - 1) / BN - tile0 : 0;
   if (p.kv_splits > 1) {
@@ -332,6 +372,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
     int limit = kv_len;
     if (p.causal) limit = min(kv_len, kv_len - q_len + (tok - q_begin) + 1);
     if (!row_valid || limit < 0) limit = 0;
+    int row_lo = kv_lo;                         // first key of this row
+    if (p.chunk > 0) row_lo = max(p.kv_start, max(limit - 1, 0) / p.chunk * p.chunk);
     // m is the exponent reference of this half row (log2 domain).  It follows the running maximum lazily: it moves
     // only when a tile's maximum exceeds it by more than 8, so probabilities stay below 2^8 and the O rows in TMEM
     // are rescaled rarely.  The final O / l does not depend on the reference.
@@ -352,11 +394,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
       const uint32_t s_addr = tmem_s + b * BN + half * 64 + lane_off;      // this half's 64 S columns
       const int key0 = (tile0 + j) * BN + half * 64;
       // Tiles that lie completely inside [kv_lo, limit) need no per-key predicate (all but the first and last ones).
-      const bool full = key0 >= kv_lo && key0 + 64 <= limit;
+      const bool full = key0 >= row_lo && key0 + 64 <= limit;
       uint32_t sv[2][32];
       tmem_ld_32x32(s_addr, sv[0]);
       tmem_ld_32x32(s_addr + 32, sv[1]);
       tmem_ld_wait();
+      if (CAP) cap_scores(sv, p.cap_in);
       if (stamp) g_attn_ts[j][1] = clock64();
       if (!P_TMEM) {
         tc_fence_before();
@@ -376,7 +419,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
             const int k = key0 + c * 32 + i;
-            if (k < limit && k >= kv_lo) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[c][i]));
+            if (k < limit && k >= row_lo) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sv[c][i]));
           }
       }
       const float m_tile = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * p.scale_log2;
@@ -402,8 +445,8 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_
           float p0 = ex2_approx(x0), p1 = ex2_approx(x1);
           if (!full) {
             const int k0 = key0 + c * 32 + 2 * i;
-            if (!(k0 < limit && k0 >= kv_lo)) p0 = 0.f;
-            if (!(k0 + 1 < limit && k0 + 1 >= kv_lo)) p1 = 0.f;
+            if (!(k0 < limit && k0 >= row_lo)) p0 = 0.f;
+            if (!(k0 + 1 < limit && k0 + 1 >= row_lo)) p1 = 0.f;
           }
           ps2[i & 1] = add_f32x2(ps2[i & 1], pack_f32x2(p0, p1));
           packed[c * 16 + i] = pack_bf16x2(p0, p1);
@@ -654,7 +697,9 @@ extern "C" int ub_attn_prefill_tc(const UbAttnArgs* a, void* stream_v) {
   p.max_blocks_per_seq = a->max_blocks_per_seq;
   p.num_blocks = a->num_blocks;
   p.o_stride = a->o_stride;
-  p.scale_log2 = a->scale * LOG2E;
+  p.scale_log2 = (a->softcap > 0.f ? a->softcap : a->scale) * LOG2E;
+  p.cap_in = a->softcap > 0.f ? a->scale / a->softcap : 0.f;
+  p.chunk = a->chunk;
   p.causal = a->causal;
   p.kv_start = a->kv_start;
   p.merge_o = reinterpret_cast<const __nv_bfloat16*>(a->merge_o);
@@ -681,17 +726,21 @@ extern "C" int ub_attn_prefill_tc(const UbAttnArgs* a, void* stream_v) {
   int dev = 0;
   cudaGetDevice(&dev);
   if (dev < UB_MAX_DEVICES && !attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+    cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_prefill_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+      e = cudaFuncSetAttribute(attn_prefill_tc_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_prefill_tc_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL);
     if (e != cudaSuccess) return -(int)e;
     attr_set[dev] = true;
   }
   dim3 grid((a->max_q_len + TOK - 1) / TOK, a->Hkv, a->num_seqs * S);
-  if (p_tmem)
-    launch_pdl(attn_prefill_tc_kernel<true>, grid, dim3(THREADS), (size_t)SMEM_TOTAL, reinterpret_cast<cudaStream_t>(stream_v), tq, tk, tv, p);
+  if (p.cap_in > 0.f)
+    launch_pdl(attn_prefill_tc_kernel<true, true>, grid, dim3(THREADS), (size_t)SMEM_TOTAL, reinterpret_cast<cudaStream_t>(stream_v), tq, tk, tv, p);
+  else if (p_tmem)
+    launch_pdl(attn_prefill_tc_kernel<true, false>, grid, dim3(THREADS), (size_t)SMEM_TOTAL, reinterpret_cast<cudaStream_t>(stream_v), tq, tk, tv, p);
   else
-    launch_pdl(attn_prefill_tc_kernel<false>, grid, dim3(THREADS), (size_t)SMEM_TOTAL, reinterpret_cast<cudaStream_t>(stream_v), tq, tk, tv, p);
+    launch_pdl(attn_prefill_tc_kernel<false, false>, grid, dim3(THREADS), (size_t)SMEM_TOTAL, reinterpret_cast<cudaStream_t>(stream_v), tq, tk, tv, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return -(int)e;
   if (S > 1) {

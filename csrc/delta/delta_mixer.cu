@@ -7,6 +7,9 @@
 //   S <- decay * S,  u = beta * (v - S^T k),  S <- S + k u^T,  o = S^T q                  S [dk, dv]
 //   out = o / sqrt(mean(o^2) + eps) * w * silu(gate)
 //
+// (or sigmoid(gate)).  With one decay per key channel, decay = exp(-exp(a_log) * softplus(raw + dt_bias)) is a vector over the rows
+// of S, raw and dt_bias have a value per head and channel.
+//
 // Everything between the loads and `out` is fp32; the projected rows and `out` have the element type of the matrix products.
 // A portion reads its sequence's state rows (none: zero) and leaves the new state in other rows, so every CTA of a launch may
 // read the old ones whenever it runs.  Rows of heads are padded to multiples of 8 with zeros, which stay zero.
@@ -25,6 +28,11 @@
 // beta), u = T x and o = e^c S^T q + W x, W = (decayed q k^T) T: T and W hold no column of S, are made once per block and head,
 // and the scan is left with products.  Entries of T are at most one (products of contractions), exponents never positive.
 // Columns of S do not meet: a warp owns a few of them.
+//
+// Decays per channel put vectors in the place of e^c: with D(i, j) the diagonal of the products of the decays of tokens j + 1 .. i,
+// the pair products are k_i^T D(i, j) k_j and q_i^T D(i, j) k_j, made per value head by walking i upwards with the running product
+// (delta_prep_channel): no exponential, nothing is divided by a decay, all factors are at most one.  What the scan reads are then
+// D(i, -1) k_i and D(i, -1) q_i in front of S and D(end, j) k_j behind it.
 #include "../common/elem.cuh"
 #include "../include/unillm_b200.h"
 
@@ -36,6 +44,14 @@ constexpr int BT = 16;        // tokens per block
 __device__ __forceinline__ float silu(float v) { return __fdividef(v, 1.f + __expf(-v)); }
 __device__ __forceinline__ float softplus(float v) { return v > 20.f ? v : log1pf(expf(v)); }
 __device__ __forceinline__ float log_decay(const UbDeltaArgs& a, float x, int h) { return -expf(a.a_log[h]) * softplus(x + a.dt_bias[h]); }
+
+__device__ __forceinline__ float channel_decay(const UbDeltaArgs& a, long long row, int h, int d, float rate /* exp(a_log) */) {
+  return expf(-rate * softplus(a.decay[row * a.ld_decay + (long long)h * a.dk + d] + a.dt_bias[(long long)h * a.dk + d]));
+}
+__device__ __forceinline__ float out_gate(const UbDeltaArgs& a, float v) {
+  const float s = __fdividef(1.f, 1.f + __expf(-v));
+  return a.gate_act == 1 ? s : v * s;
+}
 
 __device__ __forceinline__ int state_row(const UbDeltaArgs& a, const int* rows, int seq) {
   const int r = rows != nullptr ? rows[seq] : -1;
@@ -50,7 +66,7 @@ __device__ __forceinline__ int state_row(const UbDeltaArgs& a, const int* rows, 
 // one token per sequence
 // ------------------------------------------------------------------------------------------------------------------------
 // NT threads; ROWS: rows of S that a thread holds (four columns each); 0: S is read twice instead (heads too large for registers).
-template <typename T, int NT, int ROWS>
+template <typename T, int NT, int ROWS, bool CH>
 __global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / NT : 1) delta_step_kernel(const UbDeltaArgs a, const int cl /* threads across the columns */) {
   pdl_launch_dependents();
   pdl_wait();
@@ -63,6 +79,7 @@ __global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / 
   float* u_s = part + 8 * 2 * dv;            // [dv]
   float* o_s = u_s + dv;                         // [dv]
   float* sc = o_s + dv;                          // scalars: 1 / |q|, 1 / |k|, q . k, beta, decay; then eight sums
+  float* dec = sc + 16;                          // [dk] decays of the rows (CH)
   const int group = a.H / a.G, g = h / group, m = a.taps - 1, C = 2 * a.G * dk + a.H * dv;
   const long long row = a.row0 + seq;
   const int si = state_row(a, a.state_in, seq), so = state_row(a, a.state_out, seq);
@@ -123,12 +140,16 @@ __global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / 
   }
   float gate = 0.f, nw = 0.f;                    // dv <= NT (launch_step)
   if (tid < dv) {
-    gate = (float)reinterpret_cast<const T*>(a.gate)[row * a.ld + (long long)h * dv + tid];
+    gate = (float)reinterpret_cast<const T*>(a.gate)[row * a.ld_gate + (long long)h * dv + tid];
     nw = a.norm_w[tid];
+  }
+  if (CH) {
+    const float rate = expf(a.a_log[h]);
+    for (int d = tid; d < dk; d += NT) dec[d] = channel_decay(a, row, h, d, rate);
   }
   if (tid == 0) {
     sc[3] = 1.f / (1.f + expf(-(float)reinterpret_cast<const T*>(a.b)[row * a.ld + h]));
-    sc[4] = expf(log_decay(a, (float)reinterpret_cast<const T*>(a.a)[row * a.ld + h], h));
+    sc[4] = CH ? 1.f : expf(log_decay(a, (float)reinterpret_cast<const T*>(a.a)[row * a.ld + h], h));
   }
   __syncthreads();
   if (warp < 3) {                                // |q|^2, |k|^2, q . k
@@ -140,7 +161,8 @@ __global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / 
   }
   float4 P = make_float4(0.f, 0.f, 0.f, 0.f), R = P;          // S^T k and S^T q, up to the factors of k and q
   auto meet = [&](const float4 s, int r) {
-    const float kk = qkv[dk + r], qq = qkv[r];
+    float kk = qkv[dk + r], qq = qkv[r];
+    if (CH) { kk *= dec[r]; qq *= dec[r]; }
     P.x = fmaf(s.x, kk, P.x); P.y = fmaf(s.y, kk, P.y); P.z = fmaf(s.z, kk, P.z); P.w = fmaf(s.w, kk, P.w);
     R.x = fmaf(s.x, qq, R.x); R.y = fmaf(s.y, qq, R.y); R.z = fmaf(s.z, qq, R.z); R.w = fmaf(s.w, qq, R.w);
   };
@@ -182,14 +204,14 @@ __global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / 
     float s = 0.f;
 #pragma unroll
     for (int w = 0; w < NT / 32; ++w) s += sc[8 + w];
-    reinterpret_cast<T*>(a.out)[row * a.ld_out + (long long)h * dv + tid] = T(o * (1.f / sqrtf(s / a.dv_real + a.eps)) * nw * silu(gate));
+    reinterpret_cast<T*>(a.out)[row * a.ld_out + (long long)h * dv + tid] = T(o * (1.f / sqrtf(s / a.dv_real + a.eps)) * nw * out_gate(a, gate));
   }
   if (so >= 0 && on) {
     const float4 u = *reinterpret_cast<const float4*>(u_s + col);
     auto write = [&](float4 s, int r) {
-      const float kk = qkv[dk + r] * rk;
-      s.x = fmaf(kk, u.x, decay * s.x); s.y = fmaf(kk, u.y, decay * s.y);
-      s.z = fmaf(kk, u.z, decay * s.z); s.w = fmaf(kk, u.w, decay * s.w);
+      const float kk = qkv[dk + r] * rk, g = CH ? dec[r] : decay;
+      s.x = fmaf(kk, u.x, g * s.x); s.y = fmaf(kk, u.y, g * s.y);
+      s.z = fmaf(kk, u.z, g * s.z); s.w = fmaf(kk, u.w, g * s.w);
       __stcs(reinterpret_cast<float4*>(dst + (long long)r * dv), s);
     };
     if (ROWS > 0) {
@@ -203,37 +225,44 @@ __global__ void __launch_bounds__(NT, ROWS <= 8 ? 768 / NT : ROWS <= 16 ? 512 / 
   }
 }
 
-template <typename T>
+template <typename T, bool CH>
 static cudaError_t launch_step(const UbDeltaArgs& a, cudaStream_t st) {
   int cl = 2;
   while (cl * 4 < a.dv) cl <<= 1;                // <= 64
   const int nt = a.dv <= 128 && a.dk * a.dv <= 64 * 64 ? 128 : 256;          // small states: more CTAs per SM
   const int nrg = nt / cl, need = (a.dk + nrg - 1) / nrg;
-  const size_t smem = sizeof(float) * (2 * a.dk + a.dv + 16 * a.dv + 2 * a.dv + 16);
+  const size_t smem = sizeof(float) * (2 * a.dk + a.dv + 16 * a.dv + 2 * a.dv + 16 + (CH ? a.dk : 0));
   const dim3 grid(a.H, a.num_seqs), block(nt);
   auto go = [&](auto kern) { return launch_pdl(kern, grid, block, smem, st, a, cl); };
   if (nt == 128) {
-    if (need <= 2) return go(delta_step_kernel<T, 128, 2>);
-    if (need <= 8) return go(delta_step_kernel<T, 128, 8>);
-    if (need <= 32) return go(delta_step_kernel<T, 128, 32>);
-    return go(delta_step_kernel<T, 128, 0>);
+    if (need <= 2) return go(delta_step_kernel<T, 128, 2, CH>);
+    if (need <= 8) return go(delta_step_kernel<T, 128, 8, CH>);
+    if (need <= 32) return go(delta_step_kernel<T, 128, 32, CH>);
+    return go(delta_step_kernel<T, 128, 0, CH>);
   }
-  if (need <= 8) return go(delta_step_kernel<T, 256, 8>);
-  if (need <= 16) return go(delta_step_kernel<T, 256, 16>);
-  if (need <= 32) return go(delta_step_kernel<T, 256, 32>);
-  return go(delta_step_kernel<T, 256, 0>);
+  if (need <= 8) return go(delta_step_kernel<T, 256, 8, CH>);
+  if (need <= 16) return go(delta_step_kernel<T, 256, 16, CH>);
+  if (need <= 32) return go(delta_step_kernel<T, 256, 32, CH>);
+  return go(delta_step_kernel<T, 256, 0, CH>);
 }
 
 // ------------------------------------------------------------------------------------------------------------------------
 // portions: what the scan reads
 // ------------------------------------------------------------------------------------------------------------------------
 // workspace, per row of the launch: q and k [2 G dk], v (later o) [H dv], the row's entries of T and W [H][2][16], (-e^c, e^c,
-// e^(c_end - c), 0) [H][4], k.k and q.k with the tokens of the row's block [G][2][16]
+// e^(c_end - c), 0) [H][4], k.k and q.k with the tokens of the row's block [G][2][16].  With decays per channel: decayed q, decayed k
+// and k decayed to the block's end [3 H dk], the products per value head [H][2][16], and behind them, per block and head, the
+// products of the block's decays [dk].
+__device__ __forceinline__ int qk_row(const UbDeltaArgs& a) { return a.decay != nullptr ? 3 * a.H * a.dk : 2 * a.G * a.dk; }
 __device__ __forceinline__ float* ws_qk(const UbDeltaArgs& a) { return a.ws; }
-__device__ __forceinline__ float* ws_v(const UbDeltaArgs& a) { return a.ws + (long long)a.rows * 2 * a.G * a.dk; }
+__device__ __forceinline__ float* ws_v(const UbDeltaArgs& a) { return a.ws + (long long)a.rows * qk_row(a); }
 __device__ __forceinline__ float* ws_tw(const UbDeltaArgs& a) { return ws_v(a) + (long long)a.rows * a.H * a.dv; }
 __device__ __forceinline__ float* ws_gl(const UbDeltaArgs& a) { return ws_tw(a) + (long long)a.rows * a.H * 2 * BT; }
 __device__ __forceinline__ float* ws_gram(const UbDeltaArgs& a) { return ws_gl(a) + (long long)a.rows * a.H * 4; }
+
+__device__ __forceinline__ float* ws_end(const UbDeltaArgs& a) { return ws_gram(a) + (long long)a.rows * a.H * 2 * BT; }
+// number of a sequence's first block among those of the launch: the gaps between sequences are harmless
+__device__ __forceinline__ long long first_block(int qs, int seq) { return qs / BT + seq; }
 
 constexpr int PREP_T = 256;
 constexpr int LDM = BT + 1;                      // row of a 16 x 16 matrix in shared memory
@@ -296,6 +325,22 @@ __device__ __forceinline__ void keep_inputs(const UbDeltaArgs& a, long long row,
   }
 }
 
+// Sixteen tokens of 256 value channels.
+template <typename T>
+__device__ __forceinline__ void prep_values(const UbDeltaArgs& a, int unit, long long row, long long wrow, int t0, int q_len, int si, int so, bool last) {
+  const int tid = threadIdx.x, C = 2 * a.G * a.dk + a.H * a.dv;
+  const int c = unit * PREP_T + (tid % 32) * 8, t = t0 + (tid / 32) * 2;
+  if (c >= a.H * a.dv) return;
+  const int ch = 2 * a.G * a.dk + c;
+  float y[2][8];
+  if (t < q_len) {
+    conv_pair<T>(a, row, t, q_len, si, ch, C, y);
+    store8(ws_v(a) + (wrow + t) * a.H * a.dv + c, y[0]);
+    if (t + 1 < q_len) store8(ws_v(a) + (wrow + t + 1) * a.H * a.dv + c, y[1]);
+  }
+  if (last && tid < 32) keep_inputs<T>(a, row, q_len, si, so, ch, C);
+}
+
 // One block of 16 tokens of one query / key head, or (units G ..) of 256 value channels.
 template <typename T>
 __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a) {
@@ -311,15 +356,7 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
   const long long row = a.row0 + qs, wrow = qs;  // rows of the step / of the workspace
   float y[2][8];
   if (unit >= a.G) {
-    const int c = (unit - a.G) * PREP_T + (tid % 32) * 8, t = t0 + (tid / 32) * 2;
-    if (c >= a.H * a.dv) return;
-    const int ch = 2 * a.G * dk + c;
-    if (t < q_len) {
-      conv_pair<T>(a, row, t, q_len, si, ch, C, y);
-      store8(ws_v(a) + (wrow + t) * a.H * a.dv + c, y[0]);
-      if (t + 1 < q_len) store8(ws_v(a) + (wrow + t + 1) * a.H * a.dv + c, y[1]);
-    }
-    if (last && tid < 32) keep_inputs<T>(a, row, q_len, si, so, ch, C);
+    prep_values<T>(a, unit - a.G, row, wrow, t0, q_len, si, so, last);
     return;
   }
   const int ldy = dk + 4;
@@ -374,10 +411,121 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
   }
 }
 
+// The same with decays per channel: one block of 16 tokens of one VALUE head, or (units H ..) of 256 value channels.
+template <typename T>
+__global__ void __launch_bounds__(PREP_T) delta_prep_channel_kernel(const UbDeltaArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];
+  const int unit = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x;
+  const int qs = a.q_start[seq], q_len = a.q_start[seq + 1] - qs, t0 = blockIdx.x * BT;
+  if (t0 >= q_len) return;
+  const int n = min(BT, q_len - t0), dk = a.dk, C = 2 * a.G * dk + a.H * a.dv;
+  const int si = state_row(a, a.state_in, seq), so = state_row(a, a.state_out, seq);
+  const bool last = so >= 0 && t0 + n == q_len;
+  const long long row = a.row0 + qs, wrow = qs;
+  if (unit >= a.H) {
+    prep_values<T>(a, unit - a.H, row, wrow, t0, q_len, si, so, last);
+    return;
+  }
+  const int h = unit, group = a.H / a.G, g = h / group, ldy = dk + 4;
+  float *q_s = sm, *k_s = sm + BT * ldy, *d_s = sm + 2 * BT * ldy;           // [16][dk + 4] each
+  const float rate = expf(a.a_log[h]);
+  for (int i = tid; i < BT * dk; i += PREP_T) {
+    const int t = i / dk, d = i % dk;
+    d_s[t * ldy + d] = t < n ? channel_decay(a, row + t0 + t, h, d, rate) : 1.f;
+  }
+  const int nch = dk / 8;
+  int L = 1;
+  while (L < nch) L <<= 1;                       // <= 32
+  for (int task = tid / L; task < BT; task += PREP_T / L) {
+    const int part = task & 1, r = (task >> 1) * 2, c = (tid % L) * 8, t = t0 + r;
+    const bool on = c < dk && t < q_len;
+    const int ch = part * a.G * dk + g * dk + c;
+    float y[2][8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) y[0][e] = y[1][e] = 0.f;
+    if (on) conv_pair<T>(a, row, t, q_len, si, ch, C, y);
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) { s0 = fmaf(y[0][e], y[0][e], s0); s1 = fmaf(y[1][e], y[1][e], s1); }
+    for (int o = L / 2; o > 0; o >>= 1) { s0 += __shfl_xor_sync(0xffffffffu, s0, o); s1 += __shfl_xor_sync(0xffffffffu, s1, o); }
+    const float f = part == 0 ? 1.f / sqrtf((float)a.dk_real) : 1.f;
+    const float f0 = f / sqrtf(s0 + 1e-6f), f1 = f / sqrtf(s1 + 1e-6f);
+    if (c < dk) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) { y[0][e] *= f0; y[1][e] = t + 1 < q_len ? y[1][e] * f1 : 0.f; }
+      store8((part == 0 ? q_s : k_s) + r * ldy + c, y[0]);
+      store8((part == 0 ? q_s : k_s) + (r + 1) * ldy + c, y[1]);
+    }
+    if (last && on && r == 0 && h % group == 0) keep_inputs<T>(a, row, q_len, si, so, ch, C);
+  }
+  __syncthreads();
+  // products of the decays from the block's start and to its end; a thread owns a channel
+  const long long HK = (long long)a.H * dk;
+  float* dst = ws_qk(a) + (wrow + t0) * 3 * HK + (long long)h * dk;
+  for (int i = tid; i < 2 * dk; i += PREP_T) {
+    const int d = i < dk ? i : i - dk;
+    float p = 1.f;
+    if (i < dk) {
+#pragma unroll
+      for (int t = 0; t < BT; ++t) {
+        p *= d_s[t * ldy + d];
+        if (t < n) {
+          dst[t * 3 * HK + d] = q_s[t * ldy + d] * p;
+          dst[t * 3 * HK + HK + d] = k_s[t * ldy + d] * p;
+        }
+      }
+      ws_end(a)[((first_block(qs, seq) + blockIdx.x) * a.H + h) * dk + d] = p;
+    } else {
+#pragma unroll
+      for (int t = BT - 1; t >= 0; --t) {
+        if (t < n) dst[t * 3 * HK + 2 * HK + d] = k_s[t * ldy + d] * p;
+        p *= d_s[t * ldy + d];
+      }
+    }
+  }
+  // k_j with the decayed keys and queries of the tokens behind it: sixteen lanes share a j and split the channels
+  const int j = tid / BT, l = tid % BT;
+  float kk[BT], qk[BT];
+#pragma unroll
+  for (int i = 0; i < BT; ++i) kk[i] = qk[i] = 0.f;
+  for (int c = l * 4; c < dk; c += 4 * BT) {
+    float4 w = *reinterpret_cast<const float4*>(k_s + j * ldy + c);
+#pragma unroll
+    for (int i = 0; i < BT; ++i) {
+      if (i < j) continue;
+      const float4 q = *reinterpret_cast<const float4*>(q_s + i * ldy + c);
+      if (i > j) {
+        const float4 f = *reinterpret_cast<const float4*>(d_s + i * ldy + c), k = *reinterpret_cast<const float4*>(k_s + i * ldy + c);
+        w.x *= f.x; w.y *= f.y; w.z *= f.z; w.w *= f.w;
+        kk[i] = fmaf(k.x, w.x, fmaf(k.y, w.y, fmaf(k.z, w.z, fmaf(k.w, w.w, kk[i]))));
+      }
+      qk[i] = fmaf(q.x, w.x, fmaf(q.y, w.y, fmaf(q.z, w.z, fmaf(q.w, w.w, qk[i]))));
+    }
+  }
+  // sums over the sixteen lanes; lane i is left with those of token i
+#pragma unroll
+  for (int o = BT / 2; o > 0; o >>= 1) {
+    const bool up = l & o;
+#pragma unroll
+    for (int m = 0; m < o; ++m) {
+      const float k0 = __shfl_xor_sync(0xffffffffu, up ? kk[m] : kk[m + o], o), q0 = __shfl_xor_sync(0xffffffffu, up ? qk[m] : qk[m + o], o);
+      kk[m] = (up ? kk[m + o] : kk[m]) + k0;
+      qk[m] = (up ? qk[m + o] : qk[m]) + q0;
+    }
+  }
+  if (l < n) {
+    float* gr = ws_gram(a) + ((wrow + t0 + l) * a.H + h) * 2 * BT + j;
+    gr[0] = kk[0];
+    gr[BT] = qk[0];
+  }
+}
+
 constexpr int SOLVE_T = 128;                     // eight (block, head) pairs per CTA
 
 // T and W of a block and head: sixteen lanes, lane j makes column j of both.
-template <typename T>
+template <typename T, bool CH>
 __global__ void __launch_bounds__(SOLVE_T) delta_solve_kernel(const UbDeltaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
@@ -390,7 +538,8 @@ __global__ void __launch_bounds__(SOLVE_T) delta_solve_kernel(const UbDeltaArgs 
   const long long row = a.row0 + qs, wrow = qs;
   float* sys = sm[unit];
   const long long at = (row + t0 + min(j, n - 1)) * a.ld + h;
-  float c = tok ? log_decay(a, (float)reinterpret_cast<const T*>(a.a)[at], h) : 0.f;        // tokens past the end: no decay
+  // tokens past the end: no decay; decays per channel are in the products already
+  float c = tok && !CH ? log_decay(a, (float)reinterpret_cast<const T*>(a.a)[at], h) : 0.f;
   const float beta = tok ? 1.f / (1.f + expf(-(float)reinterpret_cast<const T*>(a.b)[at])) : 0.f;
 #pragma unroll
   for (int o = 1; o < BT; o <<= 1) {
@@ -398,12 +547,13 @@ __global__ void __launch_bounds__(SOLVE_T) delta_solve_kernel(const UbDeltaArgs 
     if (j >= o) c += v;
   }
   const float c_end = __shfl_sync(0xffffffffu, c, BT - 1, BT);
-  const float* gram = ws_gram(a) + ((wrow + t0) * a.G + g) * 2 * BT + j;
+  const int units = CH ? a.H : a.G;              // heads that have products of their own
+  const float* gram = ws_gram(a) + ((wrow + t0) * units + (CH ? h : g)) * 2 * BT + j;
 #pragma unroll
   for (int i = 0; i < BT; ++i) {
     const float ci = __shfl_sync(0xffffffffu, c, i, BT), bi = __shfl_sync(0xffffffffu, beta, i, BT);
     const float e = j <= i && i < n ? expf(ci - c) : 0.f;
-    const float* p = gram + (long long)min(i, n - 1) * a.G * 2 * BT;
+    const float* p = gram + (long long)min(i, n - 1) * units * 2 * BT;
     sys[i * LDM + j] = bi * e * p[0];
     sys[(BT + i) * LDM + j] = e * p[BT];
   }
@@ -451,7 +601,7 @@ __device__ __forceinline__ void cp16(float* dst, const float* src, bool ok) {
 // selection, lanes hold things in the order in which they give them away: the first operand of an odd half-group's lane is q
 // where the others' is k, the LPG / 8 lanes that share a column take LPG / 8 tokens at a time and number them from their own one
 // (slot s holds token s ^ own), and likewise the four columns.  In the end a lane has one number for every LPG / 8th token.
-template <int RPL, int LPG>
+template <int RPL, int LPG, bool CH>
 struct Scan {
   static constexpr int DK = RPL * LPG;           // rows that fit
   static constexpr int CPW = 4 * (32 / LPG);     // columns per warp
@@ -460,7 +610,8 @@ struct Scan {
   static constexpr int OWN = BT / REPS;          // tokens a lane ends up with: q * REPS + rep
   static constexpr int GT = RPL >= 16 ? (REPS > 2 ? REPS : 2) : 4;             // tokens whose products with S are under way together
   struct Stage {
-    float kq[2][BT][DK], v[2][BT][COLS], tw[BT][2 * BT], gl[BT][4];          // v[1] stays zero
+    float kq[CH ? 3 : 2][BT][DK], v[2][BT][COLS], tw[BT][2 * BT], gl[BT][4];          // v[1] stays zero
+    float end[CH ? DK : 4];                      // decays of the rows over the block
   };
   struct Smem {
     Stage st[2];
@@ -468,11 +619,11 @@ struct Scan {
   };
 };
 
-template <int RPL, int LPG>
+template <int RPL, int LPG, bool CH>
 __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
-  using C = Scan<RPL, LPG>;
+  using C = Scan<RPL, LPG, CH>;
   extern __shared__ __align__(16) uint8_t raw[];
   typename C::Smem& s = *reinterpret_cast<typename C::Smem*>(raw);
   const int h = blockIdx.y, seq = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -518,13 +669,17 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
       const int t0 = b * BT, n = min(BT, q_len - t0);
       const long long row = (long long)qs + t0;
       {
-        const float* p = qk + (row + kr) * 2 * a.G * dk + (long long)g * dk + kc;
+        const long long ld = qk_row(a), next = (long long)(CH ? a.H : a.G) * dk;         // next: q to k, k to the k behind S
+        const float* p = qk + (row + kr) * ld + (long long)(CH ? h : g) * dk + kc;
 #pragma unroll
-        for (int i = 0; i < BT / KR; ++i, p += 2LL * KR * a.G * dk) {
+        for (int i = 0; i < BT / KR; ++i, p += KR * ld) {
           const bool ok = kr + i * KR < n && kc < dk;
           cp16(&st.kq[1][kr + i * KR][kc], ok ? p : qk, ok);
-          cp16(&st.kq[0][kr + i * KR][kc], ok ? p + (long long)a.G * dk : qk, ok);
+          cp16(&st.kq[0][kr + i * KR][kc], ok ? p + next : qk, ok);
+          if (CH) cp16(&st.kq[CH ? 2 : 0][kr + i * KR][kc], ok ? p + 2 * next : qk, ok);
         }
+        if (CH && tid < C::DK / 4)
+          cp16(&st.end[CH ? 4 * tid : 0], ws_end(a) + ((first_block(qs, seq) + b) * a.H + h) * dk + (4 * tid < dk ? 4 * tid : 0), 4 * tid < dk);
       }
       for (int t = vr; t < BT; t += VR) {
         const bool ok = t < n && cta_col + vc < dv;
@@ -645,12 +800,21 @@ __global__ void __launch_bounds__(SCAN_W * 32) delta_scan_kernel(const UbDeltaAr
     // the state behind the block
     const float end = st.gl[BT - 1][1];
     const uint64_t fade = pack_f32x2(end, end);
-    const float* kk = &st.kq[0][0][4 * l];
+    const float* kk = &st.kq[CH ? 2 : 0][0][4 * l];
     const float2 *ua = &s.u[warp][mycol & 1][0][grp * 4 + (mycol & 2)], *ub = &s.u[warp][mycol & 1][0][grp * 4 + ((mycol & 2) ^ 2)];
+    if (CH) {
 #pragma unroll
-    for (int p = 0; p < RPL / 2; ++p)
+      for (int x2 = 0; x2 < RPL / 4; ++x2) {
+        const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(&st.end[CH ? 4 * l + 4 * LPG * x2 : 0]);
 #pragma unroll
-      for (int c = 0; c < 4; ++c) S[p][c] = mul_f32x2(S[p][c], fade);
+        for (int c = 0; c < 4; ++c) { S[2 * x2][c] = mul_f32x2(S[2 * x2][c], f.x); S[2 * x2 + 1][c] = mul_f32x2(S[2 * x2 + 1][c], f.y); }
+      }
+    } else {
+#pragma unroll
+      for (int p = 0; p < RPL / 2; ++p)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) S[p][c] = mul_f32x2(S[p][c], fade);
+    }
 #pragma unroll
     for (int j = 0; j < BT; ++j) {
       const ulonglong2 u01 = *reinterpret_cast<const ulonglong2*>(ua + j * C::CPW), u23 = *reinterpret_cast<const ulonglong2*>(ub + j * C::CPW);
@@ -698,7 +862,7 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const UbDeltaArgs a, 
   for (int e = 0; e < 8; ++e) o[e] = 0.f;
   if (on) {
     load8(ws_v(a) + t * a.H * dv + (long long)h * dv + c, o);
-    load8(reinterpret_cast<const T*>(a.gate) + (a.row0 + t) * a.ld + (long long)h * dv + c, g);
+    load8(reinterpret_cast<const T*>(a.gate) + (a.row0 + t) * a.ld_gate + (long long)h * dv + c, g);
     load8(a.norm_w + c, w);
   }
 #pragma unroll
@@ -707,39 +871,45 @@ __global__ void __launch_bounds__(256) delta_finish_kernel(const UbDeltaArgs a, 
   if (!on) return;
   const float r = 1.f / sqrtf(sq / a.dv_real + a.eps);
 #pragma unroll
-  for (int e = 0; e < 8; ++e) o[e] *= r * w[e] * silu(g[e]);
+  for (int e = 0; e < 8; ++e) o[e] *= r * w[e] * out_gate(a, g[e]);
   store8(reinterpret_cast<T*>(a.out) + (a.row0 + t) * a.ld_out + (long long)h * dv + c, o);
 }
 
-template <int RPL, int LPG>
+template <int RPL, int LPG, bool CH>
 static cudaError_t launch_scan(const UbDeltaArgs& a, cudaStream_t st) {
-  using C = Scan<RPL, LPG>;
+  using C = Scan<RPL, LPG, CH>;
   constexpr size_t smem = sizeof(typename C::Smem);
   if (smem > 48 * 1024) {
-    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPL, LPG>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    const cudaError_t e = cudaFuncSetAttribute(delta_scan_kernel<RPL, LPG, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return e;
   }
-  return launch_pdl(delta_scan_kernel<RPL, LPG>, dim3((a.dv + C::COLS - 1) / C::COLS, a.H, a.num_seqs), dim3(SCAN_W * 32), smem, st, a);
+  return launch_pdl(delta_scan_kernel<RPL, LPG, CH>, dim3((a.dv + C::COLS - 1) / C::COLS, a.H, a.num_seqs), dim3(SCAN_W * 32), smem, st, a);
 }
 
-template <typename T>
+template <typename T, bool CH>
 static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
-  const size_t smem = sizeof(float) * 2 * BT * (a.dk + 4);
+  const size_t smem = sizeof(float) * (CH ? 3 : 2) * BT * (a.dk + 4);
   const int blocks = (a.max_q + BT - 1) / BT;
-  const dim3 grid(blocks, a.G + (a.H * a.dv + PREP_T - 1) / PREP_T, a.num_seqs);
-  cudaError_t e = launch_pdl(delta_prep_kernel<T>, grid, dim3(PREP_T), smem, st, a);
+  const dim3 grid(blocks, (CH ? a.H : a.G) + (a.H * a.dv + PREP_T - 1) / PREP_T, a.num_seqs);
+  cudaError_t e = cudaSuccess;
+  if constexpr (CH) {
+    if (smem > 48 * 1024) e = cudaFuncSetAttribute(delta_prep_channel_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e == cudaSuccess) e = launch_pdl(delta_prep_channel_kernel<T>, grid, dim3(PREP_T), smem, st, a);
+  } else {
+    e = launch_pdl(delta_prep_kernel<T>, grid, dim3(PREP_T), smem, st, a);
+  }
   if (e != cudaSuccess) return e;
-  e = launch_pdl(delta_solve_kernel<T>, dim3(blocks, (a.H + SOLVE_T / BT - 1) / (SOLVE_T / BT), a.num_seqs), dim3(SOLVE_T), (size_t)0, st, a);
+  e = launch_pdl(delta_solve_kernel<T, CH>, dim3(blocks, (a.H + SOLVE_T / BT - 1) / (SOLVE_T / BT), a.num_seqs), dim3(SOLVE_T), (size_t)0, st, a);
   if (e != cudaSuccess) return e;
   // few lanes per column keep the reductions short, many of them spread a small launch over the device
   const long long cols = (long long)a.num_seqs * a.H * a.dv;
   int lanes = a.lanes;
   if (lanes == 0) lanes = cols / 16 >= 888 ? 8 : cols / 8 >= 400 ? 16 : 32;
   if (a.dk > 128 && lanes < 16) lanes = 16;
-  if (a.dk <= 32) e = launch_scan<4, 8>(a, st);
-  else if (a.dk <= 64) e = lanes <= 8 ? launch_scan<8, 8>(a, st) : launch_scan<4, 16>(a, st);
-  else if (a.dk <= 128) e = lanes <= 8 ? launch_scan<16, 8>(a, st) : lanes <= 16 ? launch_scan<8, 16>(a, st) : launch_scan<4, 32>(a, st);
-  else e = lanes <= 16 ? launch_scan<16, 16>(a, st) : launch_scan<8, 32>(a, st);
+  if (a.dk <= 32) e = launch_scan<4, 8, CH>(a, st);
+  else if (a.dk <= 64) e = lanes <= 8 ? launch_scan<8, 8, CH>(a, st) : launch_scan<4, 16, CH>(a, st);
+  else if (a.dk <= 128) e = lanes <= 8 ? launch_scan<16, 8, CH>(a, st) : lanes <= 16 ? launch_scan<8, 16, CH>(a, st) : launch_scan<4, 32, CH>(a, st);
+  else e = lanes <= 16 ? launch_scan<16, 16, CH>(a, st) : launch_scan<8, 32, CH>(a, st);
   if (e != cudaSuccess) return e;
   int L = 1;
   while (L * 8 < a.dv) L <<= 1;
@@ -750,18 +920,25 @@ static cudaError_t launch_portions(const UbDeltaArgs& a, cudaStream_t st) {
 }  // namespace delta
 }  // namespace ub
 
-extern "C" long long ub_delta_workspace_floats(int rows, int H, int G, int dk, int dv) {
-  return (long long)rows * (2LL * G * dk + (long long)H * dv + 2LL * ub::delta::BT * (H + G) + 4LL * H);
+extern "C" long long ub_delta_workspace_floats(int rows, int num_seqs, int H, int G, int dk, int dv, int channel_decay) {
+  constexpr int BT = ub::delta::BT;
+  const long long qk = channel_decay ? 3LL * H * dk : 2LL * G * dk, units = channel_decay ? H : G;
+  const long long end = channel_decay ? (rows / BT + num_seqs + 1LL) * H * dk : 0;
+  return (long long)rows * (qk + (long long)H * dv + 2LL * BT * (H + units) + 4LL * H) + end;
 }
 
-extern "C" int ub_delta_mixer(const UbDeltaArgs* a, void* stream) {
+extern "C" int ub_delta_mixer(const UbDeltaArgs* args, void* stream) {
   using namespace ub;
+  UbDeltaArgs full = *args;
+  if (full.ld_gate <= 0) full.ld_gate = full.ld;
+  const UbDeltaArgs* a = &full;
+  const bool ch = a->decay != nullptr;
   if (a->num_seqs <= 0 || a->max_q <= 0 || a->rows <= 0) return 0;
   if (a->H <= 0 || a->G <= 0 || a->H % a->G != 0 || a->H > 65535 || a->num_seqs > 65535) return -2;
   if (a->dk % 8 != 0 || a->dv % 8 != 0 || a->dk <= 0 || a->dv <= 0 || a->dk > 256 || a->dv > 256) return -3;
   if (a->dk_real <= 0 || a->dk_real > a->dk || a->dv_real <= 0 || a->dv_real > a->dv) return -3;
-  if (a->taps < 1 || a->taps > 16 || a->ld % 8 != 0 || a->ld_out % 8 != 0) return -4;
-  if (a->qkv == nullptr || a->gate == nullptr || a->b == nullptr || a->a == nullptr || a->conv == nullptr || a->state == nullptr ||
+  if (a->taps < 1 || a->taps > 16 || a->ld % 8 != 0 || a->ld_out % 8 != 0 || a->ld_gate % 8 != 0) return -4;
+  if (a->qkv == nullptr || a->gate == nullptr || a->b == nullptr || (a->a == nullptr && !ch) || a->conv == nullptr || a->state == nullptr ||
       a->out == nullptr || a->norm_w == nullptr || a->a_log == nullptr || a->dt_bias == nullptr)
     return -5;
   if (a->taps > 1 && a->conv_state == nullptr) return -5;
@@ -769,10 +946,12 @@ extern "C" int ub_delta_mixer(const UbDeltaArgs* a, void* stream) {
   cudaError_t e;
   if (a->q_start == nullptr) {
     if (a->rows != a->num_seqs) return -6;
-    e = a->f32 ? delta::launch_step<float>(*a, st) : delta::launch_step<__nv_bfloat16>(*a, st);
+    if (ch) e = a->f32 ? delta::launch_step<float, true>(*a, st) : delta::launch_step<__nv_bfloat16, true>(*a, st);
+    else e = a->f32 ? delta::launch_step<float, false>(*a, st) : delta::launch_step<__nv_bfloat16, false>(*a, st);
   } else {
-    if (a->ws == nullptr || a->G + a->H * a->dv / 256 + 1 > 65535) return -6;
-    e = a->f32 ? delta::launch_portions<float>(*a, st) : delta::launch_portions<__nv_bfloat16>(*a, st);
+    if (a->ws == nullptr || (ch ? a->H : a->G) + a->H * a->dv / 256 + 1 > 65535) return -6;
+    if (ch) e = a->f32 ? delta::launch_portions<float, true>(*a, st) : delta::launch_portions<__nv_bfloat16, true>(*a, st);
+    else e = a->f32 ? delta::launch_portions<float, false>(*a, st) : delta::launch_portions<__nv_bfloat16, false>(*a, st);
   }
   if (e == cudaSuccess) e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;

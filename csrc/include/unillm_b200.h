@@ -181,6 +181,29 @@ typedef struct UbSublayerInArgs {
 } UbSublayerInArgs;
 int ub_sublayer_in(const UbSublayerInArgs* args, void* stream);
 
+/* ---------------- K5t : input of a sublayer behind a norm without statistics (csrc/norm/stream_in.cu) ---------------- */
+typedef struct UbStreamInArgs {
+  const float* x;           /* residual stream [rows, Hp], or NULL: the rows of `table` for `ids` */
+  const int* ids;
+  const void* table;        /* [vocab, Hp] */
+  const void* y;            /* the previous sublayer's rows, x' = x + scale * y; or NULL */
+  const float* hist;        /* n_hist streams [rows, Hp], hist_stride elements apart */
+  const float* mix;         /* [n_hist + 1] weights of the streams and of x', or NULL: no average */
+  float* x_res;             /* receives x', or NULL */
+  float* x_out;             /* receives the stream that goes on, or NULL; with a shift not the buffer x */
+  const void *w, *b;        /* [Hp] of the norm tanh(alpha * s) * w + b */
+  const void* shift;        /* [Hp], or NULL: rows stand alone (n_rows of them, picked by `rows` where given) */
+  float* shift_state;       /* [state_rows, Hp] last h of a sequence */
+  const int *state_in, *state_out, *q_start;   /* as in UbSublayerInArgs */
+  const int* rows;          /* row of x, y and hist per output row, or NULL */
+  void* out;
+  int* err;
+  long long row0, hist_stride;
+  int Hp, n_hist, vocab, num_seqs, max_q, state_rows, tile /* tokens per CTA */, n_rows, x_rows, f32;
+  float scale, alpha;
+} UbStreamInArgs;
+int ub_stream_in(const UbStreamInArgs* args, void* stream);
+
 /* ---------------- K16c : matrix-state recurrence with head norm and gate (csrc/wkv/wkv_mixer.cu) ---------------- */
 typedef struct UbWkvArgs {
   const void *r, *k, *v, *g; /* [.., ld] rows of heads * D elements */
@@ -204,10 +227,10 @@ long long ub_wkv_workspace_floats(int rows, int ld, int H, int D, int max_chunks
 /* ---------------- K16d : gated delta rule over ragged portions (csrc/delta/delta_mixer.cu) ---------------- */
 typedef struct UbDeltaArgs {
   const void *qkv;           /* rows [Q: G * dk | K: G * dk | V: H * dv] in front of the convolutions */
-  const void *gate;          /* rows of H * dv */
+  const void *gate;          /* rows of H * dv, ld_gate apart */
   const void *b, *a;         /* rows of H: write strength and decay, before their non-linearities */
   const void* conv;          /* [taps, 2 * G * dk + H * dv], of qkv's element type */
-  const float *a_log, *dt_bias, *norm_w;       /* [H], [H], [dv] */
+  const float *a_log, *dt_bias, *norm_w;       /* [H], [H] (with `decay`: [H * dk]), [dv] */
   float* conv_state;         /* [state_rows, taps - 1, 2 * G * dk + H * dv] last inputs of the convolutions */
   float* state;              /* [state_rows, H, dk, dv] */
   const int *state_in, *state_out, *q_start;   /* as in UbSublayerInArgs */
@@ -218,9 +241,13 @@ typedef struct UbDeltaArgs {
   int H, G, dk, dv /* padded to 8, <= 256 */, dk_real, dv_real, taps, num_seqs, max_q, rows, state_rows, f32;
   int lanes;                 /* portions: lanes that share a column of the state (8, 16, 32), 0 = chosen here */
   float eps;
+  /* one decay per key channel instead of one per head (`a` is then unused): fp32 rows of H * dk, before the non-linearities */
+  const float* decay;
+  long long ld_gate, ld_decay;
+  int gate_act;              /* 0 SiLU, 1 sigmoid */
 } UbDeltaArgs;
 int ub_delta_mixer(const UbDeltaArgs* args, void* stream);
-long long ub_delta_workspace_floats(int rows, int H, int G, int dk, int dv);
+long long ub_delta_workspace_floats(int rows, int num_seqs, int H, int G, int dk, int dv, int channel_decay);
 
 /* ---------------- K1h : one matrix per head, out[t, h] = x[t, h] @ w[h]^T (csrc/gemm/gemm_heads.cu) ---------------- */
 typedef struct UbHeadGemmArgs {
@@ -279,8 +306,24 @@ typedef struct UbRopeArgs {
   int k_cache_only;          /* 1: the rotated k need not be written back into qkv (it is in the cache) */
   int row_norm;              /* 1: one norm over all q of a token and one over all k; the weights have Hq * D and Hkv * D elements */
   long long ld;              /* elements between rows of qkv (0: rows are dense) */
+  float gain;                /* factor on cosine and sine (0: 1); with inv_freq only */
+  const float* v_inv_freq;   /* [v_rot / 2]: values are cached turned by position * frequency, pairs (i, i + v_rot / 2); or NULL */
+  int v_rot;
 } UbRopeArgs;
 int ub_rope_kv_append(const UbRopeArgs* args, void* stream);
+
+/* ---------------- K6d : queries, keys and values of a differential attention (csrc/norm_rope/map_rows.cu) ---------------- */
+typedef struct UbMapRowsArgs {
+  const void* src;           /* rows [Q: H * maps * dim | K: G * maps * dim | V: G * dv] */
+  void* q_out;               /* [T, H * maps, maps * dim] */
+  void* k_cache;             /* [num_blocks, G, block_size, maps * dim] */
+  void* v_cache;             /* [num_blocks, G, block_size, dv] */
+  const int* slot_mapping;   /* NULL: rows hold queries only */
+  int* err;
+  long long num_slots, ld;
+  int T, H, G, maps, dim, dv, block_size, f32;
+} UbMapRowsArgs;
+int ub_map_rows(const UbMapRowsArgs* args, void* stream);
 
 /* ---------------- K3 / K4 : paged attention ---------------- */
 typedef struct UbAttnArgs {
@@ -317,7 +360,20 @@ typedef struct UbAttnArgs {
   int Dv;                    /* value head size (0 = D): v_cache [.., Dv], out [T, Hq, Dv], scratch [.., Dv + 2] */
   int kv_shared;             /* ub_attn_f32: values are the first Dv elements of the key rows (ub_attn_latent: always so) */
   float softcap;             /* > 0: scores become softcap * tanh(score / softcap), before masks, ALiBi and sinks */
+  int chunk;                 /* > 0: a query sees keys of its own chunk of this many positions only (counted from position 0) */
 } UbAttnArgs;
+/* between an attention's outputs and its output projection (csrc/attn/attn_finish.cu) */
+typedef struct UbAttnFinishArgs {
+  const void* att;           /* [T, H * maps, dv] */
+  const void* gate;          /* gate_kind 1: rows of H, 2: rows of H * dv, before the sigmoid */
+  const int* positions;      /* [T] */
+  const float* inv_freq;     /* [dv_real / 2], or NULL: no rotation */
+  void* out;                 /* [T, H * dv] */
+  long long ld_att, ld_gate, ld_out;
+  int T, H, dv /* padded to 8 */, dv_real, maps, gate_kind, f32;
+  float lambda, factor, eps; /* maps = 2 */
+} UbAttnFinishArgs;
+int ub_attn_finish(const UbAttnFinishArgs* args, void* stream);
 /* prompts over expanded latents (csrc/attn/attn_expanded_tc.cu): ub_latent_gather copies the cache rows of the sequences to
    consecutive rows (each sequence from page_start[seq] * 16 on, zeros behind its end and up to `rows`), ub_attn_expanded
    runs the attention on tcgen05 */

@@ -192,12 +192,13 @@ __global__ void __launch_bounds__(128) rope_kv_append_kernel(const UbRopeArgs a)
 // head, so they stay in registers.
 enum { PAIR_HALVES = 0, PAIR_NEIGHBOURS = 1, PAIR_ODD = 2 /* halves that are no whole chunks */ };
 
-template <typename T, int LPH, int PAIR>
-__global__ void __launch_bounds__(128, 8) head_norm_rope_kernel(const UbRopeArgs a) {
+// VTURN: values are cached turned by their position.
+template <typename T, int LPH, int PAIR, bool VTURN>
+__global__ void __launch_bounds__(128, VTURN ? 6 : 8) head_norm_rope_kernel(const UbRopeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int U = 2;
-  extern __shared__ float cs[];                   // cos [half] then sin [half]
+  extern __shared__ float cs[];                   // cos [half] then sin [half], the same for the values
   __shared__ float red[2][4];
   const int t = blockIdx.x, D = a.D, Dv = a.Dv, half = a.rotary_dim / 2;
   constexpr int ngrp = 128 / LPH, batch = U * ngrp;
@@ -227,10 +228,18 @@ __global__ void __launch_bounds__(128, 8) head_norm_rope_kernel(const UbRopeArgs
   for (int i = threadIdx.x; i < half; i += 128) {
     float s, co;
     sincosf(pos * (a.inv_freq != nullptr ? a.inv_freq[i] : rope_inv_freq(i, a)), &s, &co);
-    cs[i] = co;
-    cs[half + i] = s;
+    cs[i] = co * a.gain;
+    cs[half + i] = s * a.gain;
   }
-  if (slot_ok && a.v_cache != nullptr) {
+  const int vh = VTURN ? a.v_rot / 2 : 0;
+  float* vcs = cs + 2 * half;
+  for (int i = threadIdx.x; i < vh; i += 128) {
+    float s, co;
+    sincosf(pos * a.v_inv_freq[i], &s, &co);
+    vcs[i] = co;
+    vcs[vh + i] = s;
+  }
+  if (slot_ok && a.v_cache != nullptr && !VTURN) {
     const int cpr = Dv / 8;
     const T* vr = row + nrot * D;
     T* vd = reinterpret_cast<T*>(a.v_cache) + (blk * a.Hkv * a.block_size + off) * Dv;
@@ -259,6 +268,30 @@ __global__ void __launch_bounds__(128, 8) head_norm_rope_kernel(const UbRopeArgs
     if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
   }
   __syncthreads();                                // angles and sums complete; nobody has written to the row yet
+  if (VTURN && slot_ok && a.v_cache != nullptr) {                    // turned values go to the cache only, the row stays
+    const int cpr = Dv / 8;
+    const T* vr = row + nrot * D;
+    T* vd = reinterpret_cast<T*>(a.v_cache) + (blk * a.Hkv * a.block_size + off) * Dv;
+    for (int it = threadIdx.x; it < a.Hkv * cpr; it += 128) {
+      const int hk = it / cpr, i0 = (it - hk * cpr) * 8;
+      const T* head = vr + hk * Dv;
+      float x[8], o[8];
+      load8(head + i0, x);
+      if (vh % 8 == 0) {
+        if (i0 < 2 * vh) load8(head + (i0 < vh ? i0 + vh : i0 - vh), o);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) o[e] = i0 + e < 2 * vh ? (float)head[i0 + e < vh ? i0 + e + vh : i0 + e - vh] : 0.f;
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const int i = i0 + e;
+        if (i < vh) x[e] = x[e] * vcs[i] - o[e] * vcs[vh + i];
+        else if (i < 2 * vh) x[e] = x[e] * vcs[i - vh] + o[e] * vcs[i];
+      }
+      store8(vd + (long long)hk * a.block_size * Dv + i0, x);
+    }
+  }
   float rq = 1.f, rk = 1.f;                       // row norms: one factor for all queries, one for all keys
   if (a.row_norm) {
     rq = 1.f / sqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)(a.Hq * a.norm_dim) + a.norm_eps);
@@ -347,14 +380,19 @@ __global__ void __launch_bounds__(128, 8) head_norm_rope_kernel(const UbRopeArgs
   }
 }
 
+template <typename T, int PAIR, bool VTURN>
+static cudaError_t launch_head_norm_rope(const UbRopeArgs& a, cudaStream_t st) {
+  const size_t smem = (size_t)(a.rotary_dim + (a.v_inv_freq != nullptr ? a.v_rot : 0) + 1) * sizeof(float);
+  const dim3 grid(a.T), block(128);
+  if (a.D <= 32) return launch_pdl(head_norm_rope_kernel<T, 4, PAIR, VTURN>, grid, block, smem, st, a);
+  if (a.D <= 64) return launch_pdl(head_norm_rope_kernel<T, 8, PAIR, VTURN>, grid, block, smem, st, a);
+  if (a.D <= 128) return launch_pdl(head_norm_rope_kernel<T, 16, PAIR, VTURN>, grid, block, smem, st, a);
+  return launch_pdl(head_norm_rope_kernel<T, 32, PAIR, VTURN>, grid, block, smem, st, a);
+}
+
 template <typename T, int PAIR>
 static cudaError_t launch_head_norm_rope(const UbRopeArgs& a, cudaStream_t st) {
-  const size_t smem = (size_t)(a.rotary_dim > 0 ? a.rotary_dim : 1) * sizeof(float);
-  const dim3 grid(a.T), block(128);
-  if (a.D <= 32) return launch_pdl(head_norm_rope_kernel<T, 4, PAIR>, grid, block, smem, st, a);
-  if (a.D <= 64) return launch_pdl(head_norm_rope_kernel<T, 8, PAIR>, grid, block, smem, st, a);
-  if (a.D <= 128) return launch_pdl(head_norm_rope_kernel<T, 16, PAIR>, grid, block, smem, st, a);
-  return launch_pdl(head_norm_rope_kernel<T, 32, PAIR>, grid, block, smem, st, a);
+  return a.v_inv_freq != nullptr ? launch_head_norm_rope<T, PAIR, true>(a, st) : launch_head_norm_rope<T, PAIR, false>(a, st);
 }
 
 template <typename T>
@@ -371,7 +409,8 @@ extern "C" int ub_rope_kv_append(const UbRopeArgs* a, void* stream_v) {
   const int Dv = a->Dv > 0 ? a->Dv : a->D;
   const long long dense = (long long)(a->Hq + a->Hkv) * a->D + (long long)a->Hkv * Dv;
   const long long ld = a->ld > 0 ? a->ld : dense;
-  const bool general = a->f32 || Dv != a->D || a->inv_freq != nullptr || (a->norm_dim > 0 && a->norm_dim != a->D) || a->row_norm || ld != dense;
+  if (a->v_inv_freq != nullptr && ((a->v_rot & 1) || a->v_rot <= 0 || a->v_rot > Dv)) return -2;
+  const bool general = a->f32 || a->v_inv_freq != nullptr || Dv != a->D || a->inv_freq != nullptr || (a->norm_dim > 0 && a->norm_dim != a->D) || a->row_norm || ld != dense;
   const bool wide_ok = a->D % 8 == 0 && Dv % 8 == 0 && a->D <= 256 && ld % 8 == 0 && ld >= dense;
   if (a->row_norm && (a->q_norm_w == nullptr || (a->Hkv > 0 && a->k_norm_w == nullptr))) return -5;
   if (general && !wide_ok) return -4;
@@ -380,6 +419,7 @@ extern "C" int ub_rope_kv_append(const UbRopeArgs* a, void* stream_v) {
     b.Dv = Dv;
     b.ld = ld;
     if (b.norm_dim <= 0) b.norm_dim = b.D;
+    if (b.gain <= 0.f) b.gain = 1.f;
     cudaError_t e = b.f32 ? ub::launch_head_norm_rope<float>(b, (cudaStream_t)stream_v)
                           : ub::launch_head_norm_rope<__nv_bfloat16>(b, (cudaStream_t)stream_v);
     if (e == cudaSuccess) e = cudaGetLastError();

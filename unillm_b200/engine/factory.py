@@ -28,7 +28,7 @@ def why_not_gpu(model) -> Optional[str]:
     if not isinstance(model, DecoderModel):
         return f"{type(model).__name__} is not a decoder-only model of the parametric block"
     s = model.spec
-    if s.norm not in ("rms", "layer") or s.post_ln or s.embed_proj_dim:
+    if s.norm not in ("rms", "layer", "tanh") or s.post_ln or s.embed_proj_dim:
         return "post-LN / projected-embedding topologies run on the whole-model path"
     if getattr(model, "reference_quirks", False):
         return "reference_quirks changes the normalisation; the kernels implement the published architecture"
@@ -45,8 +45,8 @@ def why_not_gpu(model) -> Optional[str]:
         for mx in ls.mixers:
             if mx.mixer == "delta" and (max(mx.head_dim, mx.v_head_dim) > 256 or not 1 <= mx.conv_taps <= 16):
                 return f"layer {i}: delta heads above 256 or more than 16 taps"
-        if ls.mixer == "attention" and s.layers is not None and max(ls.head_dim, ls.v_head_dim) > 256:
-            return f"layer {i}: head sizes above 256"
+        if ls.mixer == "attention" and s.layers is not None and max((ls.head_dim + 7) // 8 * 8 * ls.maps, ls.v_head_dim) > 256:
+            return f"layer {i}: head sizes above 256 (of all maps together)"
         if ls.moe is not None and (ls.moe.num_experts > 256 or ls.moe.top_k > 16):
             return f"layer {i}: more than 256 experts or more than 16 per token"
     if (s.input_conv - 1) * s.hidden_size * 4 > 220 * 1024:

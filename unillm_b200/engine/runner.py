@@ -131,7 +131,10 @@ class KernelHeads:
     rows); the pad entries of the projections are zero, so they add nothing to scores or outputs.
 
     Latent attention: one cache row of ``dk`` = kv_rank + rot elements whose first ``dv`` = kv_rank are the value; ``dim``,
-    ``rot``, ``vdim`` and ``q_rank`` are the padded sizes around it.  wkv: ``dk`` x ``dv`` states, no cache row."""
+    ``rot``, ``vdim`` and ``q_rank`` are the padded sizes around it.  wkv: ``dk`` x ``dv`` states, no cache row.
+
+    With ``maps`` > 1 a key row holds the keys of all maps and every (head, map) is a query head of the kernels: ``hq`` counts
+    those, ``dk`` is the whole row.  ``gate_rows``: rows of an output gate behind Q, K and V of the input projection."""
 
     hq: int
     hkv: int
@@ -144,10 +147,12 @@ class KernelHeads:
     vdim: int = 0
     q_rank: int = 0
     delta: Optional["DeltaHeads"] = None         # of the layer's gated delta rule (beside the attention, or its only mixer)
+    maps: int = 1
+    gate_rows: int = 0
 
     @property
     def qkv_rows(self) -> int:
-        return self.hq * self.dk + (self.hkv * (self.dk + self.dv) if self.own_kv else 0)
+        return self.hq * (self.dk // self.maps) + (self.hkv * (self.dk + self.dv) if self.own_kv else 0)
 
     @property
     def cache_row(self) -> int:
@@ -160,7 +165,8 @@ class KernelHeads:
 class DeltaHeads:
     """A gated delta rule as the kernels see it: ``hq`` heads of ``dk`` x ``dv`` states, ``hk`` query / key heads, head sizes
     rounded up to multiples of 8.  Its rows of the layer's input projection are [Q | K | V | gate | b | a], behind those of an
-    attention it stands beside; its columns of the output projection follow that one's."""
+    attention it stands beside; its columns of the output projection follow that one's.  With low-rank decays per channel and a
+    low-rank gate (``ra``, ``rg`` > 0, rounded up) they are [Q | K | V | b | first product of the decays | of the gate]."""
 
     hq: int
     hk: int
@@ -169,13 +175,22 @@ class DeltaHeads:
     taps: int
     row0: int
     col0: int
+    ra: int = 0
+    rg: int = 0
 
     @property
     def conv_rows(self) -> int:
         return 2 * self.hk * self.dk + self.hq * self.dv
 
     @property
+    def low_col(self) -> int:
+        """First column of the low-rank products."""
+        return self.conv_rows + _round8(self.hq)
+
+    @property
     def rows(self) -> int:
+        if self.ra:
+            return self.low_col + self.ra + self.rg
         return self.conv_rows + self.hq * self.dv + _round8(2 * self.hq)
 
     @property
@@ -208,6 +223,8 @@ class RunnerWeights:
         for n in ("embed_norm.w", "embed_norm.b", "final_norm.w", "final_norm.b"):
             if n in p:
                 self.t[n] = dev(_pad(p[n], 0, H))
+        if "final_norm.alpha" in p:
+            self.slopes["final_norm"] = float(p["final_norm.alpha"])
         for n in ("pos_embed", "project_in", "project_out"):
             if n in p:
                 self.t[n] = dev(p[n])
@@ -225,6 +242,15 @@ class RunnerWeights:
             for n in ("conv1", "conv2"):
                 if L + n in p:                                # [taps, H]: neighbouring threads read neighbouring channels
                     self.t[L + n] = dev(_pad(p[L + n].t(), 1, H))
+            self.slopes.update({L + n: float(p[L + n + ".alpha"]) for n in ("ln1", "ln2") if L + n + ".alpha" in p})
+            if L + "shift" in p:
+                self.t[L + "shift"] = dev(_pad(p[L + "shift"], 0, H))
+            if L + "dwa" in p:
+                self.t[L + "dwa"] = p[L + "dwa"].to(device=device, dtype=torch.float32).contiguous()
+            if L + "lambdas" in p:
+                from ..models.mixers import diff_lambda
+
+                self.lams[i] = diff_lambda(ls, p[L + "lambdas"])
             if L + "act" in p:
                 from ..models.mixers import xielu_coefficients
 
@@ -245,17 +271,24 @@ class RunnerWeights:
 
             def fused_rows(t):
                 parts = t.split([ls.q_size, ls.k_size, ls.v_size]) if kh.own_kv else (t,)
-                out = [heads(parts[0], ls.num_heads, ls.head_dim, kh.dk, rank * kh.hq, kh.hq)]
+                n, d = ls.maps, kh.dk // ls.maps
+                out = [heads(parts[0], ls.num_heads * n, ls.head_dim, d, rank * kh.hq, kh.hq)]
                 if kh.own_kv:
-                    out.append(heads(parts[1], ls.num_kv_heads, ls.head_dim, kh.dk, kh.kv_lo, kh.hkv))
+                    out.append(heads(parts[1], ls.num_kv_heads * n, ls.head_dim, d, kh.kv_lo * n, kh.hkv * n))
                     out.append(heads(parts[2], ls.num_kv_heads, ls.v_head_dim, kh.dv, kh.kv_lo, kh.hkv))
                 return torch.cat(out, 0)
 
-            self.t[L + "wqkv"] = dev(_pad(fused_rows(p[L + "wqkv"]), 1, H))
+            w_in = fused_rows(p[L + "wqkv"])
+            if ls.out_gate:
+                g = p[L + "w_og"]
+                g = _pad(g, 0, kh.gate_rows) if ls.out_gate == "head" else heads(g, ls.num_heads, ls.v_head_dim, kh.dv, 0, ls.num_heads)
+                w_in = torch.cat([w_in, g])
+            self.t[L + "wqkv"] = dev(_pad(w_in, 1, H))
             if L + "bqkv" in p:
-                self.t[L + "bqkv"] = dev(fused_rows(p[L + "bqkv"]))
+                self.t[L + "bqkv"] = dev(_pad(fused_rows(p[L + "bqkv"]), 0, kh.qkv_rows + kh.gate_rows))
             wo = p[L + "wo"].t()                              # [heads * v size, H]: sharded and padded like the head rows
-            self.t[L + "wo"] = dev(_pad(heads(wo, ls.num_heads, ls.v_head_dim, kh.dv, rank * kh.hq, kh.hq).t(), 0, H))
+            n = kh.hq // ls.maps
+            self.t[L + "wo"] = dev(_pad(heads(wo, ls.num_heads, ls.v_head_dim, kh.dv, rank * n, n).t(), 0, H))
             if L + "bo" in p:
                 self.t[L + "bo"] = dev(p[L + "bo"] if rank == 0 else torch.zeros_like(p[L + "bo"]))
             if kh.delta is not None:
@@ -321,12 +354,12 @@ class RunnerWeights:
             up = shard_rows(p[L + "w_up"], rank, world)
             self.t[L + "w_up"] = dev(_pad(_pad(up, 0, self._round(up.shape[0])), 1, self.width))
             if L + "b_up" in p:
-                self.t[L + "b_up"] = dev(shard_rows(p[L + "b_up"], rank, world))
+                self.t[L + "b_up"] = dev(_pad(shard_rows(p[L + "b_up"], rank, world), 0, self._round(up.shape[0])))
         if L + "w_down" in p:
             dn = shard_cols(p[L + "w_down"], rank, world)
             self.t[L + "w_down"] = dev(_pad(_pad(dn, 1, self._round(dn.shape[1])), 0, self.width))
             if L + "b_down" in p:
-                self.t[L + "b_down"] = dev(p[L + "b_down"] if rank == 0 else torch.zeros_like(p[L + "b_down"]))
+                self.t[L + "b_down"] = dev(_pad(p[L + "b_down"] if rank == 0 else torch.zeros_like(p[L + "b_down"]), 0, self.width))
 
     def _beside_weights(self, i: int, p, device, dev, heads) -> None:
         """The gated delta rule beside a layer's attention: one input and one output projection for both mixers.  The output
@@ -357,9 +390,18 @@ class RunnerWeights:
         t[L + "delta_conv"] = qkv_rows(p[src + "conv"]).t().to(device=device, dtype=self.dtype).contiguous()
         t[L + "a_log"], t[L + "dt_bias"] = f32(p[src + "A_log"]), f32(p[src + "dt_bias"])
         t[L + "o_norm"] = f32(_pad(p[src + "o_norm"].float() * factor, 0, d.dv))
+        wo = _pad(heads(p[src + "wo"].t(), n, ls.v_head_dim, d.dv, 0, n).t(), 0, H)
+        if d.ra:
+            low = lambda x, r: x.to(device=device, dtype=self.dtype).contiguous() if x.shape[1] == r else _pad(x, 1, r).to(device=device, dtype=self.dtype)
+            t[L + "dt_bias"] = f32(heads(p[src + "dt_bias"], n, ls.head_dim, d.dk, 0, n))
+            t[L + "w_a2"] = low(heads(p[src + "w_a2"], n, ls.head_dim, d.dk, 0, n), d.ra)
+            t[L + "w_g2"] = low(heads(p[src + "w_g2"], n, ls.v_head_dim, d.dv, 0, n), d.rg)
+            w = torch.cat([qkv_rows(p[src + "w_qkv"]), _pad(p[src + "w_b"], 0, _round8(n)), _pad(p[src + "w_a1"], 0, d.ra),
+                           _pad(p[src + "w_g1"], 0, d.rg)])
+            return _pad(w, 1, H), wo
         ba = torch.cat([p[src + "w_b"], p[src + "w_a"]])
         w = torch.cat([qkv_rows(p[src + "w_qkv"]), heads(p[src + "w_g"], n, ls.v_head_dim, d.dv, 0, n), _pad(ba, 0, _round8(2 * n))])
-        return _pad(w, 1, H), _pad(heads(p[src + "wo"].t(), n, ls.v_head_dim, d.dv, 0, n).t(), 0, H)
+        return _pad(w, 1, H), wo
 
     def _mixer_weights(self, i: int, p, device, dev, heads) -> None:
         """Latent attention, wkv or delta parameters of one layer in kernel layout."""
@@ -414,12 +456,15 @@ class RunnerWeights:
         self.width = self._round(spec.hidden_size)
         self.heads: List[KernelHeads] = []
         self.act_params: Dict[int, Tuple[float, float]] = {}   # coefficients of activations with learned numbers, per layer
+        self.slopes: Dict[str, float] = {}                     # of Dynamic Tanh norms, by the norm's name
+        self.lams: Dict[int, float] = {}                       # factor on the second map of differential attentions, per layer
         r8 = self._round
         for i in range(spec.num_layers):
             ls = spec.layer(i)
-            if ls.mixer != "attention" or spec.norm_placement == "both":
+            if ls.mixer != "attention" or spec.norm_placement == "both" or spec.norm == "tanh" or ls.maps > 1 or ls.out_gate or ls.value_rope:
                 if world > 1:
-                    raise UnsupportedOperation("latent attention, wkv and delta layers and norms on both sides of a sublayer: one rank")
+                    raise UnsupportedOperation("latent attention, wkv and delta layers, output gates, rotated values, differential attention, "
+                                               "Dynamic Tanh and norms on both sides of a sublayer: one rank")
             if ls.mixer == "delta":
                 self.heads.append(KernelHeads(ls.num_heads, 0, 0, 8, 8, False, delta=self._delta_heads(ls, 0, 0)))
                 continue
@@ -437,7 +482,10 @@ class RunnerWeights:
             if ls.moe is not None and not self.ep and (ls.moe.intermediate_size % world or ls.moe.shared_width % world):
                 raise InvalidInput(f"layer {i}: expert widths not divisible by tensor parallel size {world}")
             hkv, kv_lo = self.kv_layout(ls.num_kv_heads, rank, world)
-            kh = KernelHeads(ls.num_heads // world, hkv, kv_lo, self._round(ls.head_dim), self._round(ls.v_head_dim), ls.kv_from is None)
+            dv = self._round(ls.v_head_dim)
+            gate = {"": 0, "head": _round8(ls.num_heads), "element": ls.num_heads * dv}[ls.out_gate]
+            kh = KernelHeads(ls.num_heads * ls.maps // world, hkv, kv_lo, self._round(ls.head_dim) * ls.maps, dv, ls.kv_from is None,
+                             maps=ls.maps, gate_rows=gate)
             if ls.beside is not None:
                 kh = dataclasses.replace(kh, delta=self._delta_heads(ls.beside, kh.qkv_rows, kh.hq * kh.dv))
             self.heads.append(kh)
@@ -448,7 +496,10 @@ class RunnerWeights:
 
     @staticmethod
     def _delta_heads(ls, row0: int, col0: int) -> "DeltaHeads":
-        return DeltaHeads(ls.num_heads, ls.num_kv_heads, _round8(ls.head_dim), _round8(ls.v_head_dim), ls.conv_taps, row0, col0)
+        if (ls.decay == "channel") != ls.low_rank_gate:
+            raise UnsupportedOperation("delta rule: decays per channel go with a low-rank gate")
+        ranks = (_round8(ls.decay_rank or 64), _round8(ls.gate_rank or 64)) if ls.low_rank_gate else (0, 0)
+        return DeltaHeads(ls.num_heads, ls.num_kv_heads, _round8(ls.head_dim), _round8(ls.v_head_dim), ls.conv_taps, row0, col0, *ranks)
 
     def kv_bytes_per_token(self) -> int:
         """Cache bytes that one token takes on this rank over all layers that own keys and values."""
@@ -471,8 +522,10 @@ class RunnerWeights:
             ls, kh = s.layer(i), self.heads[i]
             if s.input_conv:
                 out += [((i, n), (s.input_conv - 1, self.width)) for n in (("conv1", "conv2") if ls.mlp is not None else ("conv1",))]
+            if ls.mixer == "wkv" or s.token_shift:
+                out.append(((i, "shift"), (self.width,)))
             if ls.mixer == "wkv":
-                out += [((i, "shift"), (self.width,)), ((i, "wkv"), (kh.hq, kh.dk, kh.dv))]
+                out.append(((i, "wkv"), (kh.hq, kh.dk, kh.dv)))
             d = kh.delta
             if d is not None:
                 out += [((i, "delta_conv"), (d.taps - 1, d.conv_rows)), ((i, "delta"), (d.hq, d.dk, d.dv))]
@@ -592,9 +645,17 @@ class RunnerWeights:
         zeros = lambda n: torch.zeros_like(ones(n))
         if s.norm_bias:
             self.t["final_norm.b"] = zeros(H)
+        if s.norm == "tanh":
+            self.slopes = {n: 0.5 for n in ("final_norm", *(f"layers.{i}.{k}" for i in range(s.num_layers) for k in ("ln1", "ln2")))}
         for i, (kh, ls) in enumerate(zip(self.heads, s.layers)):
             L = f"layers.{i}."
             norm_w = zeros if s.norm_weight_offset_one else ones
+            if s.token_shift:
+                self.t[L + "shift"] = zeros(H) + 0.3
+            if s.depth_average:
+                self.t[L + "dwa"] = torch.cat([rnd(1, i + 1).view(-1), ones(1)]).float()
+            if ls.maps > 1:
+                self.lams[i] = ls.diff
             for n in ("ln1", "ln2") if s.norm_placement != "both" else ("ln1", "ln2", "ln1b", "ln2b"):
                 self.t[L + n + ".w"] = norm_w(H)
                 if s.norm_bias:
@@ -605,6 +666,8 @@ class RunnerWeights:
             if ls.mlp == "dense":
                 width = self._round(s.layer_intermediate(i))
                 self.t[L + "w_up"], self.t[L + "w_down"] = rnd(width, H), rnd(H, width)
+                if s.mlp_bias:
+                    self.t[L + "b_up"], self.t[L + "b_down"] = zeros(width), zeros(H)
                 if s.mlp == "gated":
                     self.t[L + "w_gate_up"] = torch.cat([self.t.pop(L + "w_up"), rnd(width, H)])
                 if s.act == "xielu":
@@ -612,8 +675,10 @@ class RunnerWeights:
             d = kh.delta
             if d is not None:
                 self.t[L + "delta_conv"] = rnd(d.taps, d.conv_rows) + 0.3
-                self.t[L + "a_log"], self.t[L + "dt_bias"] = zeros(d.hq).float(), zeros(d.hq).float() - 3.0
+                self.t[L + "a_log"], self.t[L + "dt_bias"] = zeros(d.hq).float(), zeros(d.hq * (d.dk if d.ra else 1)).float() - 3.0
                 self.t[L + "o_norm"] = ones(d.dv).float()
+                if d.ra:
+                    self.t[L + "w_a2"], self.t[L + "w_g2"] = rnd(d.hq * d.dk, d.ra), rnd(d.hq * d.dv, d.rg)
             if ls.mixer == "wkv":
                 rank, C = self._round(ls.decay_rank or 64), kh.hq * kh.dk
                 self.t[L + "mu"] = torch.full_like(rnd(5, H), 0.5)
@@ -640,10 +705,10 @@ class RunnerWeights:
                 if s.has_qkv_bias(i):
                     self.t[L + "b_in"] = zeros(kh.qkv_rows + d.rows)
             else:
-                self.t[L + "wqkv"] = rnd(kh.qkv_rows, H)
-                self.t[L + "wo"] = rnd(H, kh.hq * kh.dv)
+                self.t[L + "wqkv"] = rnd(kh.qkv_rows + kh.gate_rows, H)
+                self.t[L + "wo"] = rnd(H, kh.hq // kh.maps * kh.dv)
                 if s.has_qkv_bias(i):
-                    self.t[L + "bqkv"] = zeros(kh.qkv_rows)
+                    self.t[L + "bqkv"] = zeros(kh.qkv_rows + kh.gate_rows)
             if kind and ls.mixer == "attention":
                 self.t[L + "q_norm"] = ones(kh.dk * (kh.hq if kind == "row" else 1))
                 if kh.own_kv:
@@ -887,8 +952,20 @@ class GpuModelRunner:
     def __init__(self, spec: DecoderSpec, weights: RunnerWeights, *, num_blocks: int, block_size: int = 16,
                  max_num_seqs: int = 256, max_num_batched_tokens: int = 8192, max_model_len: int = 8192,
                  tp: Optional[TpContext] = None, device=None, use_cuda_graphs: bool = True):
-        if spec.norm not in ("rms", "layer") or spec.post_ln or spec.embed_proj_dim:
+        if spec.norm not in ("rms", "layer", "tanh") or spec.post_ln or spec.embed_proj_dim:
             raise UnsupportedOperation("this spec is served by the generic model path, not the fused runner")
+        tanh = spec.norm == "tanh"
+        if tanh and (spec.norm_placement != "input" or not spec.residual_fp32 or not spec.norm_bias or not spec.final_norm or spec.pos == "learned"
+                     or spec.embed_norm or spec.embed_scale != 1.0 or spec.parallel_residual or spec.input_conv
+                     or any(spec.layer(i).mixer == "wkv" or spec.layer(i).mlp == "moe" for i in range(spec.num_layers))):
+            raise UnsupportedOperation("Dynamic Tanh: in front of the sublayers of a 32-bit residual stream, no mixtures, wkv layers or convolutions")
+        if not tanh and (spec.token_shift or spec.depth_average):
+            raise UnsupportedOperation("token shifts and depth averages: behind Dynamic Tanh norms")
+        if any(spec.layer(i).maps > 1 and (spec.layer(i).rotary_dim or spec.qk_norm_kind(i) or spec.layer(i).maps != 2) for i in range(spec.num_layers)):
+            raise UnsupportedOperation("differential attention: two maps, no rotation, no query and key norms")
+        if any(spec.layer(i).beside is not None and (spec.layer(i).out_gate or spec.layer(i).maps > 1 or spec.layer(i).value_rope or
+                                                     spec.layer(i).beside.low_rank_gate) for i in range(spec.num_layers)):
+            raise UnsupportedOperation("two mixers side by side: plain attention and a delta rule with one decay per head")
         if spec.norm_placement == "output" and (not spec.residual_fp32 or spec.pos == "learned" or spec.embed_norm
                                                 or spec.residual_scale != 1.0 or spec.parallel_residual):
             raise UnsupportedOperation("norms on sublayer outputs: 32-bit residual stream, no learned positions")
@@ -897,10 +974,10 @@ class GpuModelRunner:
                                               or spec.mlp_bias or spec.o_bias
                                               or (spec.input_conv and any(spec.layer_is_moe(i) for i in range(spec.num_layers)))):
             raise UnsupportedOperation("norms on both sides of a sublayer: RMS, 32-bit residual stream, no mixtures behind convolutions")
-        if spec.norm_placement != "both" and (spec.input_conv or any(spec.layer(i).mixer != "attention" or spec.layer(i).beside is not None
+        if spec.norm_placement != "both" and not tanh and (spec.input_conv or any(spec.layer(i).mixer != "attention" or spec.layer(i).beside is not None
                                                                      for i in range(spec.num_layers))):
             raise UnsupportedOperation("input convolutions, latent attention, wkv and delta layers: with norms on both sides of a sublayer")
-        if spec.norm_placement == "input" and (spec.residual_fp32 or weights.dtype != torch.bfloat16):
+        if spec.norm_placement == "input" and not tanh and (spec.residual_fp32 or weights.dtype != torch.bfloat16):
             raise UnsupportedOperation("a 32-bit residual stream or 32-bit weights: only with norms on sublayer outputs")
         self.spec, self.w = spec, weights
         self.tp = tp or TpContext()
@@ -914,6 +991,7 @@ class GpuModelRunner:
         self.layers = [s.layer(i) for i in range(s.num_layers)]
         # a window that no sequence can outgrow is full attention (and keeps the kernels for that)
         self.windows = [ls.window if 0 < ls.window < max_model_len else 0 for ls in self.layers]
+        self.chunks = [ls.chunk if 0 < ls.chunk < max_model_len else 0 for ls in self.layers]
         self.k_cache: List[torch.Tensor] = []
         self.v_cache: List[torch.Tensor] = []
         for ls, kh in zip(self.layers, weights.heads):
@@ -1091,7 +1169,9 @@ class GpuModelRunner:
         kw = dict(theta=ls.rope_theta, llama3_scaling=ls.rope_llama3)
         if s.layers is not None:
             # frequencies from the host in 64 bits, and only for the layers' own rotation
-            kw = dict(inv_freq=self._rotation(ls)[0] if ls.rotary_dim > 0 else None, v_head_dim=kh.dv, norm_dim=ls.head_dim)
+            kw = dict(v_head_dim=kh.dv, norm_dim=ls.head_dim, v_inv_freq=self._value_rotation(ls) if ls.value_rope and kh.own_kv else None)
+            if ls.rotary_dim > 0:
+                kw["inv_freq"], kw["gain"] = self._rotation(ls)
         own = kh.own_kv
         with self._prof("rope_kv_append"):
             K.rope_kv_append(qkv, pos, slots if own else None, self.k_cache[i] if own else None,
@@ -1101,10 +1181,32 @@ class GpuModelRunner:
                              norm_eps=s.norm_eps, k_cache_only=own, row_norm=s.qk_norm_kind(i) == "row", **kw)
         self.launches += 1
 
+    def _attention_layer(self, i, h, pos, slots, lay, shared_prefix_len):
+        """Attention of layer ``i`` on what it reads, up to the rows for its output projection."""
+        t, ls, kh, L = self.w.t, self.layers[i], self.w.heads[i], f"layers.{i}."
+        proj = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
+        qkv = proj[:, :kh.qkv_rows] if kh.gate_rows else proj
+        if kh.maps > 1:
+            own = kh.own_kv
+            with self._prof("map_rows"):
+                qkv = K.map_rows(qkv, slots if own else None, self.k_cache[i] if own else None, self.v_cache[i] if own else None,
+                                 num_heads=kh.hq // kh.maps, maps=kh.maps, dim=kh.dk // kh.maps).flatten(1)
+            self.launches += 1
+        else:
+            self._rope_append(i, qkv, pos, slots)
+        a = self._attention(i, qkv, lay, shared_prefix_len)
+        if kh.maps == 1 and not ls.out_gate and not ls.value_rope:
+            return a
+        self.launches += 1
+        with self._prof("attn_finish"):
+            return K.attn_finish(a, kh.dv, gate=proj[:, kh.qkv_rows:] if kh.gate_rows else None, gate_kind=ls.out_gate, maps=kh.maps,
+                                 lam=self.w.lams.get(i, 0.0), factor=1.0 - ls.diff, eps=self.spec.norm_eps, dv_real=ls.v_head_dim,
+                                 positions=pos if ls.value_rope else None, inv_freq=self._value_rotation(ls) if ls.value_rope else None)
+
     def _attention(self, i, qkv, lay, shared_prefix_len, out=None):
         """qkv [T, q | k | v] already rotated and appended -> attention output [T, hq * Dv] (``out``: columns of a wider tensor)."""
         kh, ls = self.w.heads[i], self.layers[i]
-        D, hq, hkv, window = kh.dk, kh.hq, kh.hkv, self.windows[i]
+        D, hq, hkv, window, chunk = kh.dk, kh.hq, kh.hkv, self.windows[i], self.chunks[i]
         sinks = self.w.t.get(f"layers.{i}.sink")
         T, Dp, P = lay["_T"], lay["_Dp"], lay["_P"]
         q = qkv[:, :hq * D].unflatten(1, (hq, D))          # strided view: row stride of the fused projection
@@ -1113,8 +1215,8 @@ class GpuModelRunner:
         kc, vc = self.k_cache[i], self.v_cache[i]
         bt = self._view(lay, "block_tables").view(Dp + P, self.max_blocks_per_seq)
         scale = ls.scale if ls.scale is not None else 1.0 / math.sqrt(ls.head_dim)
-        # the shared-prefix pass has no window, position bias or sink
-        plain = window == 0 and self.alibi is None and sinks is None and not ls.softcap and kh.dk == kh.dv and qkv.dtype == torch.bfloat16
+        # the shared-prefix pass has no window, chunk, position bias or sink
+        plain = window == 0 and chunk == 0 and self.alibi is None and sinks is None and not ls.softcap and kh.dk == kh.dv and qkv.dtype == torch.bfloat16
         cascade = plain and shared_prefix_len >= 4 * self.block_size and Dp >= 8
         # prefill rows join the cascade when their chunks start after the shared prefix and share its blocks
         pp = cascade and P > 0 and lay.get("_pp", False)
@@ -1177,14 +1279,14 @@ class GpuModelRunner:
         elif Dp > 0:
             with self._prof("attn_decode"):
                 K.attn_decode(q[:Dp], kc, vc, bt[:Dp], self._view(lay, "seq_lens_d"), scale=scale, window=window,
-                              alibi_slopes=self.alibi, sinks=sinks, softcap=ls.softcap, out=out[:Dp], scratch=self.attn_scratch,
+                              alibi_slopes=self.alibi, sinks=sinks, softcap=ls.softcap, chunk=chunk, out=out[:Dp], scratch=self.attn_scratch,
                               max_seq_len=self.max_model_len if self._graph_mode else int(self._max_len_d))
             self.launches += 1
         if P > 0 and not pp:
             with self._prof("attn_prefill"):
                 K.attn_prefill(q[Dp:], kc, vc, bt[Dp:], self._view(lay, "seq_lens_p"), self._view(lay, "q_start"),
                                lay["_max_q"], scale=scale, causal=True, window=window, alibi_slopes=self.alibi,
-                               sinks=sinks, softcap=ls.softcap, out=out[Dp:])
+                               sinks=sinks, softcap=ls.softcap, chunk=chunk, out=out[Dp:])
             self.launches += 1
         return flat
 
@@ -1263,6 +1365,8 @@ class GpuModelRunner:
             return self._forward_tokens_output_norm(lay, shared_prefix_len)
         if s.norm_placement == "both":
             return self._forward_tokens_both_norms(lay, shared_prefix_len)
+        if s.norm == "tanh":
+            return self._forward_tokens_stream(lay, shared_prefix_len)
         ids = self._view(lay, "token_ids")
         pos = self._view(lay, "positions")
         slots = self._view(lay, "slot_mapping")
@@ -1276,9 +1380,7 @@ class GpuModelRunner:
         for i in range(s.num_layers):
             L = f"layers.{i}."
             h = self._norm(x, L + "ln1")
-            qkv = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
-            self._rope_append(i, qkv, pos, slots)
-            a = self._attention(i, qkv, lay, shared_prefix_len)
+            a = self._attention_layer(i, h, pos, slots, lay, shared_prefix_len)
             if s.parallel_residual:
                 m_in = h if s.parallel_shared_norm else self._norm(x, L + "ln2")
                 o = self._gemm(a, t[L + "wo"], bias=t.get(L + "bo"))
@@ -1317,9 +1419,7 @@ class GpuModelRunner:
         self.launches += 1
         for i, ls in enumerate(self.layers):
             L = f"layers.{i}."
-            qkv = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
-            self._rope_append(i, qkv, pos, slots)
-            a = self._attention(i, qkv, lay, shared_prefix_len)
+            a = self._attention_layer(i, h, pos, slots, lay, shared_prefix_len)
             y = self._gemm(a, t[L + "wo"], bias=t.get(L + "bo"))
             tp.all_reduce(y)
             h = self._residual_norm(x, y, L + "ln1")
@@ -1373,15 +1473,55 @@ class GpuModelRunner:
         self._last_y = y
         return x
 
+    def _forward_tokens_stream(self, lay, shared_prefix_len: int) -> torch.Tensor:
+        """Layers of the form ``x += m f(norm(x))`` with a norm that needs no statistics, around a 32-bit residual stream.  Adding a
+        sublayer's output, the average over depth behind a layer, the next norm and the token shift are one kernel; the embedding
+        rows are gathered by the first of them, the last layer's output is added and averaged by the final norm, for the rows that
+        are asked for."""
+        s, t, m = self.spec, self.w.t, self.spec.residual_scale
+        pos, slots = self._view(lay, "positions"), self._view(lay, "slot_mapping")
+        parts = self._portions(lay)
+        buf = lambda: torch.empty(lay["_T"], self.w.width, dtype=torch.float32, device=self.device)
+        # results of the layers so far, the embedding first
+        streams = torch.empty(s.num_layers, lay["_T"], self.w.width, dtype=torch.float32, device=self.device) if s.depth_average else None
+        y: dict = dict(ids=self._view(lay, "token_ids"), table=t["embed"])
+        for i, ls in enumerate(self.layers):
+            L = f"layers.{i}."
+            if streams is not None:
+                y["x_res"] = streams[i]
+            x = streams[0] if i == 0 and streams is not None else buf()
+            if i > 0 or streams is None:
+                y["x_out"] = x
+            h = self._stream_in(L + "ln1", parts, shift=t.get(L + "shift"), shift_state=self.state.get((i, "shift")), **y)
+            if ls.mixer == "latent":
+                a = self._latent_attention(i, h, pos, slots, lay)
+            elif ls.mixer == "delta":
+                a, _ = self._attention_and_delta(i, h, pos, slots, lay, parts, shared_prefix_len)
+            else:
+                a = self._attention_layer(i, h, pos, slots, lay, shared_prefix_len)
+            y = dict(x=x, y=self._gemm(a, t[L + "wo"], bias=t.get(L + "bo")), scale=m)
+            if ls.mlp is not None:
+                x = buf() if i == 0 and streams is not None else x
+                h = self._stream_in(L + "ln2", (), x_out=x, **y)
+                y = dict(x=x, y=self._mlp_noresid(i, h), scale=m)
+            if streams is not None:
+                y.update(streams=streams, mix=t[L + "dwa"])
+        self._last_y = y
+        return y["x"]
+
+    def _stream_in(self, name, parts, **kw):
+        t = self.w.t
+        self.launches += len(parts) if kw.get("shift") is not None else 1
+        with self._prof("stream_in"):
+            return K.stream_in(parts, t[name + ".w"], t[name + ".b"], self.w.slopes[name], **kw)
+
     def _attention_and_delta(self, i, h, pos, slots, lay, parts, shared_prefix_len):
         """Attention, a gated delta rule, or both side by side on one input projection: (rows for the output projection, the
         factor on its result)."""
         t, L, ls, kh = self.w.t, f"layers.{i}.", self.layers[i], self.w.heads[i]
         d = kh.delta
         if d is None:
-            qkv = self._gemm(h, t[L + "wqkv"], bias=t.get(L + "bqkv"))
-            self._rope_append(i, qkv, pos, slots)
-            return self._attention(i, qkv, lay, shared_prefix_len), 1.0
+            return self._attention_layer(i, h, pos, slots, lay, shared_prefix_len), 1.0
         proj = self._gemm(h, t[L + "w_in"], bias=t.get(L + "b_in"))
         out = torch.empty(h.shape[0], d.col0 + d.cols, dtype=proj.dtype, device=proj.device)
         mx = ls
@@ -1390,11 +1530,15 @@ class GpuModelRunner:
             qkv = proj[:, :d.row0]
             self._rope_append(i, qkv, pos, slots)
             self._attention(i, qkv, lay, shared_prefix_len, out=out[:, :d.col0])
+        low = {}
+        if d.ra:
+            mid = proj[:, d.row0 + d.low_col:]
+            low = dict(decay=self._gemm(mid[:, :d.ra], t[L + "w_a2"], out_dtype=torch.float32), gate=self._gemm(mid[:, d.ra:d.ra + d.rg], t[L + "w_g2"]))
         with self._prof("delta"):
             K.delta_mixer(proj, d.row0, t[L + "delta_conv"], t[L + "a_log"], t[L + "dt_bias"], t[L + "o_norm"],
                           self.state[(i, "delta_conv")], self.state[(i, "delta")], parts, kv_heads=d.hk, eps=self.spec.norm_eps,
-                          dk_real=mx.head_dim, dv_real=mx.v_head_dim, out=out[:, d.col0:])
-        self.launches += sum(1 if p.q_start is None else 3 for p in parts)
+                          dk_real=mx.head_dim, dv_real=mx.v_head_dim, out=out[:, d.col0:], gate_act=mx.gate_act, **low)
+        self.launches += sum(1 if p.q_start is None else 4 for p in parts)
         if ls.beside is None:
             return out, 1.0
         return out, ls.scales[0] or 1.0
@@ -1509,6 +1653,13 @@ class GpuModelRunner:
         if key not in self._inv_freq:
             self._inv_freq[key] = rope_inv_freq(*key).to(self.device)
         return self._inv_freq[key], rope_gain(ls.rope_yarn)
+
+    def _value_rotation(self, ls):
+        """Frequencies of a layer's rotated values: all their dimensions, no scaling."""
+        key = (ls.v_head_dim, ls.rope_theta)
+        if key not in self._inv_freq:
+            self._inv_freq[key] = rope_inv_freq(*key).to(self.device)
+        return self._inv_freq[key]
 
     def _residual_norm(self, x, y, name, **kw):
         s, t = self.spec, self.w.t
@@ -1651,6 +1802,8 @@ class GpuModelRunner:
             with self._prof("norm"):
                 return K.sublayer_in(x, (), t["final_norm.w"], eps=s.norm_eps, rows=rows, width=s.hidden_size,
                                      offset_one=s.norm_weight_offset_one, **self._last_y)
+        if s.norm == "tanh":
+            return self._stream_in("final_norm", (), rows=rows, **self._last_y)
         if s.residual_fp32:
             self.launches += 1
             with self._prof("norm"):

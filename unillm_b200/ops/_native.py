@@ -71,6 +71,33 @@ class UbRopeArgs(C.Structure):
         ("num_slots", i64), ("theta", f32), ("pos_scale", f32), ("norm_eps", f32), ("interleaved", i32),
         ("l3_factor", f32), ("l3_low_freq_factor", f32), ("l3_high_freq_factor", f32), ("l3_orig_ctx", f32),
         ("inv_freq", vp), ("Dv", i32), ("norm_dim", i32), ("f32", i32), ("k_cache_only", i32), ("row_norm", i32), ("ld", i64),
+        ("gain", f32), ("v_inv_freq", vp), ("v_rot", i32),
+    ]
+
+
+class UbMapRowsArgs(C.Structure):
+    _fields_ = [
+        ("src", vp), ("q_out", vp), ("k_cache", vp), ("v_cache", vp), ("slot_mapping", vp), ("err", vp),
+        ("num_slots", i64), ("ld", i64),
+        ("T", i32), ("H", i32), ("G", i32), ("maps", i32), ("dim", i32), ("dv", i32), ("block_size", i32), ("f32", i32),
+    ]
+
+
+class UbStreamInArgs(C.Structure):
+    _fields_ = [
+        ("x", vp), ("ids", vp), ("table", vp), ("y", vp), ("hist", vp), ("mix", vp), ("x_res", vp), ("x_out", vp), ("w", vp), ("b", vp),
+        ("shift", vp), ("shift_state", vp), ("state_in", vp), ("state_out", vp), ("q_start", vp), ("rows", vp), ("out", vp), ("err", vp),
+        ("row0", i64), ("hist_stride", i64),
+        ("Hp", i32), ("n_hist", i32), ("vocab", i32), ("num_seqs", i32), ("max_q", i32), ("state_rows", i32), ("tile", i32),
+        ("n_rows", i32), ("x_rows", i32), ("f32", i32), ("scale", f32), ("alpha", f32),
+    ]
+
+
+class UbAttnFinishArgs(C.Structure):
+    _fields_ = [
+        ("att", vp), ("gate", vp), ("positions", vp), ("inv_freq", vp), ("out", vp), ("ld_att", i64), ("ld_gate", i64), ("ld_out", i64),
+        ("T", i32), ("H", i32), ("dv", i32), ("dv_real", i32), ("maps", i32), ("gate_kind", i32), ("f32", i32),
+        ("lambda_", f32), ("factor", f32), ("eps", f32),
     ]
 
 
@@ -111,6 +138,7 @@ class UbDeltaArgs(C.Structure):
         ("row0", i64), ("ld", i64), ("ld_out", i64),
         ("H", i32), ("G", i32), ("dk", i32), ("dv", i32), ("dk_real", i32), ("dv_real", i32), ("taps", i32), ("num_seqs", i32),
         ("max_q", i32), ("rows", i32), ("state_rows", i32), ("f32", i32), ("lanes", i32), ("eps", f32),
+        ("decay", vp), ("ld_gate", i64), ("ld_decay", i64), ("gate_act", i32),
     ]
 
 
@@ -149,7 +177,7 @@ class UbAttnArgs(C.Structure):
         ("block_size", i32), ("max_blocks_per_seq", i32), ("num_blocks", i32),
         ("q_stride", i64), ("o_stride", i64), ("scale", f32),
         ("causal", i32), ("window", i32), ("splits", i32), ("kv_start", i32), ("total_q", i32), ("max_q_len", i32),
-        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32), ("kv_shared", i32), ("softcap", f32),
+        ("merge_o", vp), ("merge_lse", vp), ("sinks", vp), ("Dv", i32), ("kv_shared", i32), ("softcap", f32), ("chunk", i32),
     ]
 
 
@@ -245,7 +273,8 @@ class _CudaLibs:
     ARGS_AND_STREAM = {
         "serving": ("ub_gemm_tn", "ub_norm", "ub_rope_kv_append", "ub_attn_decode", "ub_attn_prefill", "ub_sample",
                     "ub_moe_route", "ub_gemm_f32", "ub_attn_f32", "ub_residual_norm", "ub_row_norm", "ub_sublayer_in", "ub_wkv_mixer", "ub_delta_mixer",
-                    "ub_gemm_heads", "ub_latent_rows", "ub_latent_rotate", "ub_attn_latent", "ub_latent_gather", "ub_attn_expanded"),
+                    "ub_gemm_heads", "ub_latent_rows", "ub_latent_rotate", "ub_attn_latent", "ub_latent_gather", "ub_attn_expanded",
+                    "ub_stream_in", "ub_map_rows", "ub_attn_finish"),
         "more": ("ub_allreduce_oneshot", "ub_tp_argmax_merge"),
     }
 

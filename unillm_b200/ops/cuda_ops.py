@@ -411,21 +411,32 @@ def _sublayer_alone(x, weight, eps, y, y_weight, width, offset_one, experts, rou
 
 def delta_mixer(proj: torch.Tensor, col: int, conv: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, norm_w: torch.Tensor,
                 conv_state: Optional[torch.Tensor], state: torch.Tensor, portions: Sequence[Portions], *, kv_heads: int, eps: float,
-                dk_real: int = 0, dv_real: int = 0, out: Optional[torch.Tensor] = None, lanes: int = 0) -> torch.Tensor:
-    """Gated delta rule with its convolutions, head norm and SiLU gate.  ``proj`` [T, ld]: from column ``col`` on, rows of
-    [Q | K | V | gate | b | a] with ``kv_heads`` * Dk, the same, H * Dv, H * Dv, H and H columns.  ``conv`` [taps, Q + K + V],
-    ``state`` fp32 [rows, H, Dk, Dv], ``conv_state`` fp32 [rows, taps - 1, Q + K + V] -> [T, H * Dv] (``out`` may be columns of a
-    wider tensor).  ``dk_real`` / ``dv_real``: head sizes before padding.  ``lanes``: see ``UbDeltaArgs``."""
-    f32 = _elem("delta_mixer", proj, conv, out)
+                dk_real: int = 0, dv_real: int = 0, out: Optional[torch.Tensor] = None, lanes: int = 0,
+                decay: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, gate_act: str = "silu") -> torch.Tensor:
+    """Gated delta rule with its convolutions, head norm and gate (``gate_act``: "silu" or "sigmoid").  ``proj`` [T, ld]: from
+    column ``col`` on, rows of [Q | K | V | gate | b | a] with ``kv_heads`` * Dk, the same, H * Dv, H * Dv, H and H columns.
+    ``conv`` [taps, Q + K + V], ``state`` fp32 [rows, H, Dk, Dv], ``conv_state`` fp32 [rows, taps - 1, Q + K + V] -> [T, H * Dv]
+    (``out`` may be columns of a wider tensor).  ``dk_real`` / ``dv_real``: head sizes before padding.  ``lanes``: see
+    ``UbDeltaArgs``.
+
+    ``decay`` (fp32 [T, H * Dk], before its non-linearities, ``dt_bias`` then [H * Dk]): one decay per key channel; with it and
+    ``gate`` [T, H * Dv] the rows of ``proj`` are [Q | K | V | b]."""
+    f32 = _elem("delta_mixer", proj, conv, out, gate)
     T, ld = proj.shape
     _, H, dk, dv = state.shape
     taps, Cn = conv.shape
     qk = kv_heads * dk
-    if proj.stride(1) != 1 or not conv.is_contiguous() or Cn != 2 * qk + H * dv or col + Cn + H * dv + 2 * H > ld:
+    chan = decay is not None
+    if chan != (gate is not None):
+        raise ValueError("delta_mixer: decays per channel go with gate rows of their own")
+    need = Cn + (H if chan else H * dv + 2 * H)
+    if proj.stride(1) != 1 or not conv.is_contiguous() or Cn != 2 * qk + H * dv or col + need > ld:
         raise ValueError("delta_mixer: rows of [Q | K | V | gate | b | a], taps over [Q | K | V]")
-    for t, n in ((a_log, H), (dt_bias, H), (norm_w, dv)):
+    if chan and (decay.dtype != torch.float32 or decay.shape != (T, H * dk) or gate.shape != (T, H * dv) or decay.stride(1) != 1 or gate.stride(1) != 1):
+        raise ValueError("delta_mixer: fp32 decays [T, H * Dk] and gates [T, H * Dv]")
+    for t, n in ((a_log, H), (dt_bias, H * dk if chan else H), (norm_w, dv)):
         if t.dtype != torch.float32 or t.numel() != n:
-            raise ValueError("delta_mixer: fp32 a_log [H], dt_bias [H] and norm weight [Dv]")
+            raise ValueError("delta_mixer: fp32 a_log [H], dt_bias [H] (or [H * Dk]) and norm weight [Dv]")
     _state_rows("delta_mixer", state, (H, dk, dv))
     if taps > 1:
         _state_rows("delta_mixer convolutions", conv_state, (taps - 1, Cn))
@@ -441,7 +452,12 @@ def delta_mixer(proj: torch.Tensor, col: int, conv: torch.Tensor, a_log: torch.T
         if p.row0 + p.rows > T:
             raise ValueError("delta_mixer: portions outside the step")
         a = N.UbDeltaArgs()
-        a.qkv, a.gate, a.b, a.a = at(0), at(Cn), at(Cn + H * dv), at(Cn + H * dv + H)
+        if chan:
+            a.qkv, a.gate, a.b, a.decay = at(0), gate.data_ptr(), at(Cn), decay.data_ptr()
+            a.ld_gate, a.ld_decay = gate.stride(0), decay.stride(0)
+        else:
+            a.qkv, a.gate, a.b, a.a = at(0), at(Cn), at(Cn + H * dv), at(Cn + H * dv + H)
+        a.gate_act = {"silu": 0, "sigmoid": 1}[gate_act]
         a.conv, a.a_log, a.dt_bias, a.norm_w = conv.data_ptr(), a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr()
         a.conv_state, a.state = _p(conv_state if taps > 1 else None), state.data_ptr()
         a.state_in, a.state_out, a.q_start = _p(p.state_in), _p(p.state_out), _p(p.q_start)
@@ -450,9 +466,71 @@ def delta_mixer(proj: torch.Tensor, col: int, conv: torch.Tensor, a_log: torch.T
         a.H, a.G, a.dk, a.dv, a.dk_real, a.dv_real, a.taps = H, kv_heads, dk, dv, dk_real or dk, dv_real or dv, taps
         a.num_seqs, a.max_q, a.rows, a.state_rows, a.f32, a.lanes, a.eps = p.n, p.max_q, p.rows, state.shape[0], int(f32), lanes, eps
         if p.q_start is not None:
-            ws = torch.empty(lib.ub_delta_workspace_floats(p.rows, H, kv_heads, dk, dv), dtype=torch.float32, device=proj.device)
+            ws = torch.empty(lib.ub_delta_workspace_floats(p.rows, p.n, H, kv_heads, dk, dv, int(chan)), dtype=torch.float32, device=proj.device)
             a.ws = ws.data_ptr()
         N.check(lib.ub_delta_mixer(C.byref(a), _stream(proj)), "ub_delta_mixer")
+    return out
+
+
+def stream_in(portions: Sequence[Portions], weight: torch.Tensor, bias: torch.Tensor, alpha: float, *, x: Optional[torch.Tensor] = None,
+              ids: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None, scale: float = 1.0,
+              streams: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, x_res: Optional[torch.Tensor] = None,
+              x_out: Optional[torch.Tensor] = None, shift: Optional[torch.Tensor] = None, shift_state: Optional[torch.Tensor] = None,
+              rows: Optional[torch.Tensor] = None, tile: int = 0) -> torch.Tensor:
+    """What a sublayer behind a Dynamic Tanh reads: ``x' = x + scale * y``, ``s = sum_j mix[j] * streams[j] + mix[-1] * x'`` (without
+    ``mix``: x'), ``h = tanh(alpha * s) * weight + bias``, and with ``shift`` every row mixed with the row of the token before it.
+
+    ``x``: fp32 [T, width], or ``ids`` (int32 [T]) and ``table`` for the embedding itself.  ``streams``: fp32 [n, T, width].
+    ``x_res`` / ``x_out`` receive x' / s.  ``rows`` (int32, without ``shift``) picks the rows to compute.  Returns h in the type of
+    ``weight``."""
+    f32 = _elem("stream_in", weight, bias, y, shift, table)
+    Hp = weight.numel()
+    T = x.shape[0] if ids is None else ids.numel()
+    if (x is None) == (ids is None) or (ids is not None and (ids.dtype != torch.int32 or table is None or table.shape[1] != Hp or not table.is_contiguous())):
+        raise ValueError("stream_in: a stream, or ids and their table")
+    for t in (x, x_res, x_out):
+        if t is not None and (t.dtype != torch.float32 or t.shape != (T, Hp) or not t.is_contiguous()):
+            raise ValueError("stream_in: streams are contiguous fp32 [T, width]")
+    if bias.numel() != Hp or (y is not None and (y.shape != (T, Hp) or not y.is_contiguous())) or (shift is not None and shift.numel() != Hp):
+        raise ValueError("stream_in: weights and sublayer rows of the stream's width")
+    a = N.UbStreamInArgs()
+    if mix is not None:
+        n = mix.numel() - 1
+        if mix.dtype != torch.float32 or (n and (streams is None or streams.dtype != torch.float32 or streams.shape[0] < n
+                                                 or streams.shape[1:] != (T, Hp) or streams[0].stride() != (Hp, 1))):
+            raise ValueError("stream_in: fp32 weights of n streams [n, T, width] and of x'")
+        a.mix, a.n_hist = mix.data_ptr(), n
+        if n:
+            a.hist, a.hist_stride = streams.data_ptr(), streams.stride(0)
+    a.x, a.ids, a.table, a.y, a.scale = _p(x), _p(ids), _p(table), _p(y), scale
+    a.vocab = table.shape[0] if table is not None else 0
+    a.x_res, a.x_out, a.w, a.b, a.alpha = _p(x_res), _p(x_out), weight.data_ptr(), bias.data_ptr(), alpha
+    a.err, a.Hp, a.f32 = err_word(weight.device).data_ptr(), Hp, int(f32)
+    lib = N.cuda_lib()
+    cols = -(-Hp // 1024)
+    if shift is None:
+        n = T if rows is None else rows.numel()
+        if rows is not None and rows.dtype != torch.int32:
+            raise TypeError("stream_in: rows must be int32")
+        out = torch.empty(n, Hp, dtype=weight.dtype, device=weight.device)
+        a.out, a.rows, a.n_rows, a.x_rows = out.data_ptr(), _p(rows), n, T
+        a.tile = tile or max(min(n * cols // 1184, 4), -(-n // 65535), 1)
+        N.check(lib.ub_stream_in(C.byref(a), _stream(weight)), "ub_stream_in")
+        return out
+    if rows is not None:
+        raise ValueError("stream_in: picked rows go without a shift")
+    _state_rows("stream_in shift", shift_state, (Hp,))
+    out = torch.empty(T, Hp, dtype=weight.dtype, device=weight.device)
+    a.out, a.shift, a.shift_state = out.data_ptr(), shift.data_ptr(), _p(shift_state)
+    for p in portions:
+        if p.row0 + p.rows > T:
+            raise ValueError("stream_in: portions outside the step")
+        if shift_state is not None:
+            a.state_in, a.state_out, a.state_rows = _p(p.state_in), _p(p.state_out), shift_state.shape[0]
+        a.q_start, a.row0, a.num_seqs, a.max_q = _p(p.q_start), p.row0, p.n, p.max_q
+        # the row in front of a tile is computed again: tiles as large as still leaves some CTAs per SM
+        a.tile = tile or max(min(p.rows * cols // 592, 16), -(-p.max_q // 65535), 1)
+        N.check(lib.ub_stream_in(C.byref(a), _stream(weight)), "ub_stream_in")
     return out
 
 
@@ -701,15 +779,18 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
                    k_norm_w: Optional[torch.Tensor] = None, norm_eps: float = 1e-6,
                    llama3_scaling: Optional[Sequence[float]] = None, v_head_dim: Optional[int] = None,
                    norm_dim: int = 0, inv_freq: Optional[torch.Tensor] = None, k_cache_only: bool = False,
-                   row_norm: bool = False) -> torch.Tensor:
+                   row_norm: bool = False, gain: float = 1.0, v_inv_freq: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Rotates q and k inside ``qkv`` [T, (Hq+Hkv)*D + Hkv*Dv] in place and appends k, v to the paged cache.
 
     ``num_kv_heads = 0``: rows hold queries only (a layer that reads another layer's keys).  ``inv_freq`` (fp32
     [rotary_dim / 2]) replaces the frequencies that ``theta`` and the scaling give; ``norm_dim`` is the number of elements
     the head norm averages over when heads are zero-padded.  ``k_cache_only``: the rotated k is needed in the cache only.
     ``row_norm``: one norm over all queries of a token and one over all its keys (weights of that size).  ``qkv`` may be the
-    first columns of wider rows."""
+    first columns of wider rows.  ``gain``: factor on cosine and sine (with ``inv_freq``).  ``v_inv_freq`` (fp32 [n]): values are
+    cached turned by their position, element i with element i + n."""
     f32 = _elem("rope_kv_append", qkv, k_cache, v_cache, q_norm_w, k_norm_w)
+    if gain != 1.0 and inv_freq is None:
+        raise ValueError("rope_kv_append: a gain goes with a frequency table")
     if qkv.stride(1) != 1:
         raise ValueError("qkv: rows must be contiguous")
     T = qkv.shape[0]
@@ -742,17 +823,75 @@ def rope_kv_append(qkv: torch.Tensor, positions: torch.Tensor, slot_mapping: Opt
     if inv_freq is not None:
         if inv_freq.dtype != torch.float32 or inv_freq.numel() != a.rotary_dim // 2:
             raise ValueError("inv_freq: fp32, one entry per rotated pair")
-        a.inv_freq = inv_freq.data_ptr()
+        a.inv_freq, a.gain = inv_freq.data_ptr(), gain
+    if v_inv_freq is not None:
+        if v_inv_freq.dtype != torch.float32 or 2 * v_inv_freq.numel() > a.Dv:
+            raise ValueError("v_inv_freq: fp32, one entry per turned pair")
+        a.v_inv_freq, a.v_rot = v_inv_freq.data_ptr(), 2 * v_inv_freq.numel()
     if llama3_scaling is not None:
         a.l3_factor, a.l3_low_freq_factor, a.l3_high_freq_factor, a.l3_orig_ctx = llama3_scaling
     N.check(N.cuda_lib().ub_rope_kv_append(C.byref(a), _stream(qkv)), "ub_rope_kv_append")
     return qkv
 
 
+def map_rows(qkv: torch.Tensor, slot_mapping: Optional[torch.Tensor], k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], *,
+             num_heads: int, maps: int, dim: int) -> torch.Tensor:
+    """Queries of a differential attention for the attention kernels, keys and values into the cache.  ``qkv`` [T, ..]: rows of
+    [Q: heads * maps * dim | K: kv heads * maps * dim | V: kv heads * Dv] (``slot_mapping`` None: Q alone is read); ``k_cache``
+    [.., kv heads, block, maps * dim] -> [T, heads * maps, maps * dim], each query zero where the other maps' keys lie."""
+    f32 = _elem("map_rows", qkv, k_cache, v_cache)
+    if qkv.stride(1) != 1 or dim % 8:
+        raise ValueError("map_rows: contiguous rows, sizes in multiples of 8")
+    out = torch.empty(qkv.shape[0], num_heads * maps, maps * dim, dtype=qkv.dtype, device=qkv.device)
+    a = N.UbMapRowsArgs()
+    a.src, a.q_out, a.err = qkv.data_ptr(), out.data_ptr(), err_word(qkv.device).data_ptr()
+    a.T, a.H, a.maps, a.dim, a.ld, a.f32 = qkv.shape[0], num_heads, maps, dim, qkv.stride(0), int(f32)
+    need = num_heads * maps * dim
+    if slot_mapping is not None:
+        if slot_mapping.dtype != torch.int32 or k_cache.shape[:3] != v_cache.shape[:3] or k_cache.shape[3] != maps * dim:
+            raise ValueError("map_rows: caches do not match the heads")
+        a.G, a.block_size, a.dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+        a.slot_mapping, a.k_cache, a.v_cache = slot_mapping.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr()
+        a.num_slots = k_cache.shape[0] * k_cache.shape[2]
+        need += a.G * (maps * dim + a.dv)
+    if qkv.shape[1] < need:
+        raise ValueError(f"map_rows: rows of {qkv.shape[1]} elements do not hold these heads")
+    N.check(N.cuda_lib().ub_map_rows(C.byref(a), _stream(qkv)), "ub_map_rows")
+    return out
+
+
+def attn_finish(att: torch.Tensor, v_dim: int, *, gate: Optional[torch.Tensor] = None, gate_kind: str = "", maps: int = 1, lam: float = 0.0,
+                factor: float = 1.0, eps: float = 0.0, positions: Optional[torch.Tensor] = None, inv_freq: Optional[torch.Tensor] = None,
+                dv_real: int = 0) -> torch.Tensor:
+    """Between an attention's outputs ``att`` [T, heads * maps * v_dim] and its output projection: maps subtracted
+    (``(a1 - lam * a2) / rms * factor``), outputs turned back by their position (``inv_freq`` fp32 [dv_real / 2]), times the sigmoid
+    of ``gate`` (``gate_kind`` "head": [T, >= heads], "element": [T, heads * v_dim]) -> [T, heads * v_dim]."""
+    f32 = _elem("attn_finish", att, gate)
+    T, H = att.shape[0], att.shape[1] // (v_dim * maps)
+    if att.stride(1) != 1 or H * v_dim * maps != att.shape[1]:
+        raise ValueError("attn_finish: rows of whole heads")
+    out = torch.empty(T, H * v_dim, dtype=att.dtype, device=att.device)
+    a = N.UbAttnFinishArgs()
+    a.att, a.out, a.ld_att, a.ld_out = att.data_ptr(), out.data_ptr(), att.stride(0), out.stride(0)
+    a.gate_kind = {"": 0, "head": 1, "element": 2}[gate_kind]
+    if a.gate_kind:
+        if gate.shape[0] != T or gate.stride(1) != 1 or gate.shape[1] < (H if gate_kind == "head" else H * v_dim):
+            raise ValueError("attn_finish: one gate row per token")
+        a.gate, a.ld_gate = gate.data_ptr(), gate.stride(0)
+    a.T, a.H, a.dv, a.dv_real, a.maps, a.f32 = T, H, v_dim, dv_real or v_dim, maps, int(f32)
+    a.lambda_, a.factor, a.eps = lam, factor, eps
+    if inv_freq is not None:
+        if inv_freq.dtype != torch.float32 or positions.dtype != torch.int32 or inv_freq.numel() != a.dv_real // 2 or positions.numel() != T:
+            raise ValueError("attn_finish: fp32 frequencies per pair, int32 positions")
+        a.inv_freq, a.positions = inv_freq.data_ptr(), positions.data_ptr()
+    N.check(N.cuda_lib().ub_attn_finish(C.byref(a), _stream(att)), "ub_attn_finish")
+    return out
+
+
 # ---------------------------------------------------------------------------------------------
 # Attention
 # ---------------------------------------------------------------------------------------------
-def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks=None, softcap=0.0):
+def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks=None, softcap=0.0, chunk=0):
     a = N.UbAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out, a.lse = q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), out.data_ptr(), _p(lse)
     a.block_tables, a.seq_lens = block_tables.data_ptr(), seq_lens.data_ptr()
@@ -761,7 +900,7 @@ def _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D
     a.block_size, a.max_blocks_per_seq, a.num_blocks = k_cache.shape[2], block_tables.shape[1], k_cache.shape[0]
     a.q_stride, a.o_stride = q.stride(0), out.stride(0)
     a.scale = scale if scale is not None else 1.0 / math.sqrt(D)
-    a.Dv, a.softcap = v_cache.shape[3], softcap
+    a.Dv, a.softcap, a.chunk = v_cache.shape[3], softcap, chunk
     if k_cache.shape[3] != D or out.shape[-1] != a.Dv:
         raise ValueError("attention: head sizes of q, caches and out do not match")
     if sinks is not None:
@@ -776,10 +915,11 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, b
                 alibi_slopes: Optional[torch.Tensor] = None, splits: int = 0, scratch: Optional[torch.Tensor] = None,
                 out: Optional[torch.Tensor] = None, return_lse: bool = False, lse: Optional[torch.Tensor] = None,
                 max_seq_len: Optional[int] = None, merge: Optional[tuple] = None, kernel: Optional[str] = None,
-                sinks: Optional[torch.Tensor] = None, softcap: float = 0.0):
+                sinks: Optional[torch.Tensor] = None, softcap: float = 0.0, chunk: int = 0):
     """One query token per sequence.  q: [B, Hq, D] (last two dims contiguous); caches [nb, Hkv, bs, D] (the value cache may
     have a head size of its own).  ``sinks``: fp32 [Hq], one logit per head that joins the softmax denominator.
-    ``softcap`` > 0: scores become softcap * tanh(score / softcap).  fp32 operands run in 32-bit arithmetic.
+    ``softcap`` > 0: scores become softcap * tanh(score / softcap).  ``chunk`` > 0: a query sees keys of its own chunk of that many
+    positions only.  fp32 operands run in 32-bit arithmetic.
 
     ``kernel="warp"`` calls the warp-per-item kernel directly (page size 16, head size 64 / 128, ``splits == 1``, no
     window, no ALiBi) instead of going through the dispatcher's choice."""
@@ -796,11 +936,13 @@ def attn_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, b
         ctx = max_seq_len if max_seq_len is not None else block_tables.shape[1] * k_cache.shape[2]
         if window > 0:
             ctx = min(ctx, window)
+        if chunk > 0:
+            ctx = min(ctx, chunk)
         ctas = B * Hkv
         splits = 1
         while ctas * splits < 2 * 148 and ctx // (splits * 2) >= 256 and splits < 16:
             splits *= 2
-    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks, softcap)
+    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks, softcap, chunk)
     if splits > 1:
         need = B * Hq * splits * (Dv + 2)
         if scratch is None or scratch.numel() < need:
@@ -828,9 +970,9 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
                  alibi_slopes: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
                  return_lse: bool = False, lse: Optional[torch.Tensor] = None, merge: Optional[tuple] = None,
                  kv_splits: int = 1, scratch: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None,
-                 softcap: float = 0.0):
+                 softcap: float = 0.0, chunk: int = 0):
     """Ragged prefill: q [T, Hq, D]; sequence i owns query rows q_start[i]:q_start[i+1] and sees
-    seq_lens[i] keys, its last query at kv position seq_lens[i]-1.
+    seq_lens[i] keys, its last query at kv position seq_lens[i]-1.  ``softcap``, ``chunk``: see :func:`attn_decode`.
 
     ``kv_splits > 1`` (tensor-core kernel only, no ``merge``) divides every CTA's key tiles over that many CTAs and
     folds the partial results with a second small kernel: for launches with few query tiles and many keys, such as
@@ -843,7 +985,7 @@ def attn_prefill(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
         out = torch.empty((T, Hq, v_cache.shape[3]), dtype=q.dtype, device=q.device)
     if return_lse and lse is None:
         lse = torch.empty((T, Hq), dtype=torch.float32, device=q.device)
-    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks, softcap)
+    a = _attn_args(q, k_cache, v_cache, out, lse, block_tables, seq_lens, Hq, Hkv, D, scale, sinks, softcap, chunk)
     a.q_start = q_start.data_ptr()
     a.causal, a.window, a.kv_start = (1 if causal else 0), window, kv_start
     a.total_q, a.max_q_len = T, max_q_len
