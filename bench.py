@@ -228,7 +228,7 @@ def main(argv=None) -> int:
                     help="1 GPU: run the per-rank shapes of W-way tensor parallelism (heads, KV heads, MLP width and "
                          "vocabulary divided by W) without any communication -- the compute floor of one rank; "
                          "the token counts it prints are not a throughput of the full model")
-    ap.add_argument("--design", default=None, choices=["gekapel", "nipulorn", "bakasun"],
+    ap.add_argument("--design", default=None, choices=["gekapel", "nipulorn", "bakasun", "tasadra"],
                     help="1 GPU: instead of the serving workload, prefill and decode steps of this design beside the closest "
                          "existing family at equal size (random weights, a few layers)")
     ap.add_argument("--design-sizes", default=None, help="--design: comma-separated subset of the sizes (1k,2k,4k)")

@@ -48,7 +48,7 @@ def _cfg(vocab, width, layers, mult, eps=1e-5):
 CASES = {
     # every kind of layer, sharing across a layer of another kind
     "mixed": _cfg(151, 96, [_layer(_diff(4, 2, 16, 40, 13, 0.3, 0.35), 72),
-                            _layer(_attn(6, 3, 24, 32, 16, 0.25, yarn=(3.0, 40, 4.0, 0.5), cap=9.0), 56),
+                            _layer(_attn(6, 3, 24, 32, 16, 0.25, yarn=(12.0, 40, 4.0, 0.5), cap=9.0), 56),
                             _layer(_delta(4, 2, 32, 24, 4), None),
                             _layer(_diff(4, 2, 16, 40, 24, 0.25, 0.6, src=0), 40),
                             _layer(_attn(4, 1, 16, 16, 16, 0.3, base=500.0), None)], 0.7),

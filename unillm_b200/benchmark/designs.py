@@ -1,5 +1,5 @@
 """Prefill and decode throughput of one design beside the closest existing family at equal size, and the same
-comparison kernel by kernel (``python bench.py --design gekapel|nipulorn|bakasun [--design-kernels]``).
+comparison kernel by kernel (``python bench.py --design gekapel|nipulorn|bakasun|tasadra [--design-kernels]``).
 
 Both models are random-weight stacks of a few layers with a real model's layer sizes, run by the same
 ``GpuModelRunner`` steps that serve requests: a prefill step is one batch of whole prompts, a decode step one token of
@@ -21,6 +21,9 @@ rate of the device instead of the matrix rate.
 Bakasun's steps are set beside DeepSeek-MoE with Mistral's sliding window (the same gated experts and always-on expert, windowed
 attention in every layer), its experts as wide as makes the parameters equal; its gated delta rule is set beside Nipulorn's
 recurrence at the same heads, tokens and state.
+
+Tasadra's steps are set beside Llama with its feed-forward as wide as makes the parameters equal, its delta rule with decays per
+channel beside Bakasun's with decays per head at the same heads, tokens and state.
 """
 from __future__ import annotations
 
@@ -32,7 +35,7 @@ import torch
 
 from ..engine.runner import GpuModelRunner, RunnerWeights, StepBatch
 from ..models import configs as C
-from ..models.families import BakasunModel, GekapelModel, NipulornModel
+from ..models.families import BakasunModel, GekapelModel, NipulornModel, TasadraModel
 from ..models.spec import DecoderSpec, MoESpec
 from ..ops import cuda_ops as K
 from .microbench import _peaks, time_ms
@@ -142,9 +145,52 @@ def windowed_moe_spec(z: dict) -> DecoderSpec:
                        moe=MoESpec(num_experts=z["experts"], top_k=z["top"], intermediate_size=ff, num_shared_experts=z["shared"] // z["ff"]))
 
 
+# width, attention (heads, kv heads, size of a head), delta rule (heads, size), differential attention (heads, kv heads, size of a
+# map's head; values are twice that), chunk, feed-forward, vocabulary, layers (attention, delta rule, differential, differential on
+# the third layer's keys, and again)
+TASADRA_SIZES = {
+    "1k": dict(width=1024, heads=16, kv=4, dim=64, dh=16, dd=64, xh=8, xkv=2, xdim=64, chunk=1024, ff=4096, vocab=32000, layers=4),
+    "2k": dict(width=2048, heads=16, kv=4, dim=128, dh=16, dd=128, xh=16, xkv=4, xdim=64, chunk=1024, ff=8192, vocab=32000, layers=4),
+    "4k": dict(width=4096, heads=32, kv=8, dim=128, dh=32, dd=128, xh=32, xkv=8, xdim=64, chunk=1024, ff=16384, vocab=32000, layers=4),
+}
+
+
+def tasadra_spec(z: dict) -> DecoderSpec:
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 == 0:
+            kind = "attention"
+            mx = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["dim"], "vdim": z["dim"], "scale": z["dim"] ** -0.5, "softcap": 50.0,
+                  "rot": {"base": 10000.0, "dims": z["dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+        elif i % 4 == 1:
+            kind, mx = "channel_delta", {"heads": z["dh"], "kv_heads": z["dh"], "dim": z["dd"], "vdim": z["dd"], "conv": 4}
+        else:
+            kind = "attention_2"
+            mx = {"heads": z["xh"], "kv_heads": z["xkv"], "dim": z["xdim"], "vdim": 2 * z["xdim"], "scale": z["xdim"] ** -0.5, "diff": 0.5,
+                  "mask": {"size": z["chunk"]}}
+            if i % 4 == 3:
+                mx["kv_from"] = i - 1
+        layers.append({"type": kind, "mixer": mx, "mlp": {"kind": "dense", "ff": z["ff"]}})
+    return TasadraModel.spec_from_config(C.TasadraConfig(vocab_size=z["vocab"], hidden_size=z["width"], num_hidden_layers=z["layers"],
+                                                         residual_mult=0.5, layers=layers))
+
+
+def plain_llama_spec(z: dict) -> DecoderSpec:
+    """As many parameters in the layers, in a dense decoder with the attention heads of the first layer in every layer."""
+    H, d, n, xv = z["width"], z["dim"], z["layers"], 2 * z["xdim"]
+    attn = H * d * (2 * z["heads"] + 2 * z["kv"])
+    delta = H * z["dd"] * 4 * z["dh"] + 2 * 64 * (H + z["dh"] * z["dd"])
+    own = H * (3 * z["xh"] + 2 * z["xkv"]) * xv
+    total = n // 4 * (attn + delta + 2 * own - H * 2 * z["xkv"] * xv) + n * 2 * H * z["ff"]
+    ff = (total - n * attn) // (n * 3 * H) // 128 * 128
+    return DecoderSpec(vocab_size=z["vocab"], hidden_size=H, num_layers=n, num_heads=z["heads"], num_kv_heads=z["kv"], head_dim=d,
+                       intermediate_size=ff, max_position_embeddings=8192)
+
+
 DESIGNS = {"gekapel": (SIZES, {"gekapel": gekapel_spec, "deepseek_moe + window": closest_spec}),
            "nipulorn": (NIPULORN_SIZES, {"nipulorn": nipulorn_spec, "llama": llama_spec}),
-           "bakasun": (BAKASUN_SIZES, {"bakasun": bakasun_spec, "deepseek_moe + window": windowed_moe_spec})}
+           "bakasun": (BAKASUN_SIZES, {"bakasun": bakasun_spec, "deepseek_moe + window": windowed_moe_spec}),
+           "tasadra": (TASADRA_SIZES, {"tasadra": tasadra_spec, "llama": plain_llama_spec})}
 FP32_TFLOPS = 148 * 128 * 2 * 1.965e9 / 1e12      # FMA pipe at the maximum clock
 
 
@@ -198,7 +244,8 @@ def step_ms(runner: GpuModelRunner, b: StepBatch, iters: int = 20, warmup: int =
 # ------------------------------------------------------------------------------------------------
 RECORDED = ("gemm_tn", "grouped_gemm", "norm", "residual_norm", "row_norm", "embed_residual", "embed_gather", "rope_kv_append",
             "attn_decode", "attn_prefill", "moe_route", "moe_gather", "moe_combine", "sample", "sublayer_in", "wkv_mixer", "delta_mixer",
-            "gemm_stacked", "latent_rows", "latent_rotate", "gemm_heads", "attn_latent", "latent_gather", "attn_expanded")
+            "gemm_stacked", "latent_rows", "latent_rotate", "gemm_heads", "attn_latent", "latent_gather", "attn_expanded",
+            "stream_in", "map_rows", "attn_finish")
 
 
 @contextlib.contextmanager
@@ -258,14 +305,28 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
         live = sum(p.n for p in parts)
         reads = live if b.num_decode else 0              # prompts start from nothing
         return "wkv", _nbytes(rkvg, ww, r) + 4 * per * (live + reads), 0.0, 5.0 * rkvg.shape[1] * per
+    if name == "stream_in":
+        x, y, n = kw.get("x"), kw.get("y"), 0 if kw.get("mix") is None else kw["mix"].numel() - 1
+        share = r.shape[0] / (x if x is not None else kw["ids"]).shape[0]
+        reads = (_nbytes(x, y) if x is not None else _nbytes(r)) + n * (_nbytes(kw["streams"][0]) if n else 0)
+        label = ("embedding" if x is None else "residual") + (f" + average of {n + 1}" if n else "") + " + norm"
+        return (label + (" + shift" if kw.get("shift") is not None else "") + (" (last rows)" if kw.get("rows") is not None else ""),
+                int(share * reads) + _nbytes(r, kw.get("x_res"), kw.get("x_out")), 0.0)
+    if name == "map_rows":
+        own = kw["num_heads"] * kw["maps"] * kw["dim"] if a[1] is None else a[0].shape[1]
+        kv = 0 if a[1] is None else a[0].shape[1] - kw["num_heads"] * kw["maps"] * kw["dim"]
+        return "rows of two maps" + (" + append" if kv else ""), _nbytes(r) + (own + kv) * a[0].shape[0] * a[0].element_size(), 0.0
+    if name == "attn_finish":
+        gate = kw["gate"].element_size() * r.shape[0] * (r.shape[1] if kw["gate_kind"] == "element" else kw["gate"].shape[1])
+        return ("difference of maps + gate" if kw["maps"] == 2 else "rotation back + gate"), _nbytes(a[0], r) + gate, 0.0
     if name == "delta_mixer":
         proj, state, parts = a[0], a[7], a[8]
         per, conv = state[0].numel(), a[6][0].numel() if a[6] is not None else 0
         H = state.shape[1]
-        used = a[2].shape[1] + H * state.shape[3] + 2 * H
+        used = a[2].shape[1] + H + (0 if kw.get("decay") is not None else H * state.shape[3] + H)
         live = sum(p.n for p in parts)
         reads = live if b.num_decode else 0              # prompts start from nothing
-        return ("delta rule", proj.shape[0] * used * proj.element_size() + _nbytes(r) + 4 * (per + conv) * (live + reads), 0.0,
+        return ("delta rule", proj.shape[0] * used * proj.element_size() + _nbytes(r, kw.get("decay"), kw.get("gate")) + 4 * (per + conv) * (live + reads), 0.0,
                 6.0 * proj.shape[0] * per)
     if name == "gemm_stacked":
         x, w = a
@@ -298,6 +359,7 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
     if name in ("attn_decode", "attn_prefill"):
         q, kc, vc = a[0], a[1], a[2]
         win = kw.get("window") or 10 ** 9
+        chunk = kw.get("chunk") or 0
         lens = b.seq_lens
         q_lens = [1] * b.num_decode + list(b.prefill_q_lens)
         row = (kc.shape[3] + vc.shape[3]) * kc.shape[1] * kc.element_size()
@@ -307,6 +369,10 @@ def _cost(name: str, a, kw, r, b: StepBatch) -> tuple:
             first = n - ql + 1
             full = max(0, min(n, win) - first + 1) if first <= win else 0       # queries that see fewer keys than the window
             pairs += full * (first + first + full - 1) // 2 + (ql - full) * min(n, win)
+        if chunk:                                        # the chunked attentions of these designs have two maps: half a row per query
+            seen = [sum(p % chunk + 1 for p in range(n - ql, n)) for n, ql in zip(lens, q_lens)]
+            keys = sum(n - (n - ql) // chunk * chunk for n, ql in zip(lens, q_lens))
+            return name + " (chunks, two maps)", _nbytes(q) // 2 + _nbytes(r) + keys * row, 2.0 * sum(seen) * q.shape[1] * (kc.shape[3] // 2 + vc.shape[3])
         return name, _nbytes(q, r) + keys * row, 2.0 * pairs * q.shape[1] * (kc.shape[3] + vc.shape[3])
     if name == "residual_norm":
         x, y, ex = a[0], a[1], kw.get("experts")
@@ -388,6 +454,27 @@ def wkv_row(z: dict, seqs: int, tokens: int, decode: bool) -> dict:
     return {"kernel": "wkv (Nipulorn)", "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2), "fraction": round(floor / (ms * 1e3), 3)}
 
 
+def delta_row(z: dict, seqs: int, tokens: int, decode: bool) -> dict:
+    """Bakasun's delta rule (one decay per head, full gate) at the heads and state of a Tasadra layer, in the units of the table
+    above."""
+    hbm, _, _ = _peaks()
+    H, D, T = z["dh"], z["dd"], seqs * tokens
+    g = torch.Generator(device="cuda").manual_seed(1)
+    used = 4 * H * D + 2 * H
+    proj = torch.randn(T, (used + 7) // 8 * 8, generator=g, device="cuda").to(torch.bfloat16)
+    conv = torch.full((4, 3 * H * D), 0.3, device="cuda", dtype=torch.bfloat16)
+    zero, st = torch.zeros(H, device="cuda"), torch.zeros(2 * seqs, H, D, D, device="cuda")
+    cs = torch.zeros(2 * seqs, 3, 3 * H * D, device="cuda")
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")
+    si, so = i32([2 * s if decode else -1 for s in range(seqs)]), i32([2 * s + 1 for s in range(seqs)])
+    p = K.Portions(0, T, seqs, tokens, None if decode else i32([s * tokens for s in range(seqs + 1)]), si, so)
+    nw = torch.ones(D, device="cuda")
+    ms, _ = time_ms(lambda: K.delta_mixer(proj, 0, conv, zero, zero, nw, cs, st, [p], kv_heads=H, eps=1e-5))
+    nbytes = T * (used + H * D) * 2 + 4 * (st[0].numel() + cs[0].numel()) * seqs * (2 if decode else 1)
+    floor = max(nbytes / (hbm * 1e9), 6.0 * T * H * D * D / (FP32_TFLOPS * 1e12)) * 1e6
+    return {"kernel": "delta rule (Bakasun)", "calls": 1, "us": round(ms * 1e3, 2), "roofline_us": round(floor, 2), "fraction": round(floor / (ms * 1e3), 3)}
+
+
 def main(design: str = "gekapel", sizes: Optional[List[str]] = None, kernels: bool = False) -> List[dict]:
     out = []
     table, arms = DESIGNS[design]
@@ -412,6 +499,8 @@ def main(design: str = "gekapel", sizes: Optional[List[str]] = None, kernels: bo
                             rows.append(wkv6_row(z, n, 1 if kind == "decode" else c))
                         if design == "bakasun" and arm != "bakasun":
                             rows.append(wkv_row(z, n, 1 if kind == "decode" else c, kind == "decode"))
+                        if design == "tasadra" and arm != "tasadra":
+                            rows.append(delta_row(z, n, 1 if kind == "decode" else c, kind == "decode"))
                         for k in rows:
                             out.append({"size": size, "model": arm, "step": kind, "sequences": n, "context": c, **k})
                             print("   ", k, flush=True)
