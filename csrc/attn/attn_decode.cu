@@ -388,7 +388,7 @@ static int launch_decode(const UbAttnArgs& a, cudaStream_t st) {
   // one warp per item needs enough items to keep every SM's copy engines busy; with fewer, an item is better served by
   // the four warps of a CTA
   if (!plain && !mma_ok) return -4;
-  if (plain && mma_ok && a.splits == 1 && a.num_seqs * a.Hkv >= 256 && decode_warp_enabled() && ub_attn_decode_warp_supported(&a))
+  if (mma_ok && a.splits == 1 && a.num_seqs * a.Hkv >= 256 && decode_warp_enabled() && ub_attn_decode_warp_supported(&a))
     return ub_attn_decode_warp(&a, st);
   if (plain && mma_ok && a.kv_start > 0 && decode_persist_enabled() && ub_attn_decode_persist_supported(&a))
     return ub_attn_decode_persist(&a, st);

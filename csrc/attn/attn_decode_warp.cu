@@ -16,6 +16,7 @@
 //   * the next item's sequence length and block-table entries are requested while the current item streams.
 //
 // Same math as attn_decode_mma.cu (m16n8k16 warp MMAs, the GQA group as MMA rows, base-2 online softmax).
+// Chunks (a query sees its own chunk only) move the first key of an item, capped scores are a compiled variant.
 // Restrictions: page size 16, head size 64 / 128, no sliding window, no ALiBi, no KV splits; the caller falls back
 // to the other kernels otherwise.
 //
@@ -59,8 +60,9 @@ __device__ __forceinline__ float ex2a(float x) {        // 2^x, approximate; 2^-
   return y;
 }
 
-// D = head size, S = ring stages per warp, SMALLG = the GQA group has at most 8 heads (MMA rows 8..15 stay zero)
-template <int D, int S, bool SMALLG>
+// D = head size, S = ring stages per warp, SMALLG = the GQA group has at most 8 heads (MMA rows 8..15 stay zero), CAP = capped
+// scores
+template <int D, int S, bool SMALLG, bool CAP>
 __global__ void __launch_bounds__(WARPS * 32, (D == 128 ? (S <= 3 ? 2 : 1) : 3))
 attn_decode_warp_kernel(const UbAttnArgs a, const int gchunks, const int n_items) {
   constexpr int CPR = D / 8;                       // 16-byte chunks per key row
@@ -77,12 +79,15 @@ attn_decode_warp_kernel(const UbAttnArgs a, const int gchunks, const int n_items
   const uint32_t ring = smem_u32(dsm) + warp * (S * STAGE);
   const int Gtot = a.Hq / a.Hkv;
   const int per_seq = a.Hkv * gchunks;
-  const int kv_lo = max(a.kv_start, 0);
-  const int p0 = kv_lo / PAGE;
+  auto first_key = [&](int len) {
+    const int lo = max(a.kv_start, 0);
+    return a.chunk > 0 ? max(lo, max(len - 1, 0) / a.chunk * a.chunk) : lo;
+  };
   const __nv_bfloat16* kc = reinterpret_cast<const __nv_bfloat16*>(a.k_cache);
   const __nv_bfloat16* vc = reinterpret_cast<const __nv_bfloat16*>(a.v_cache);
   const __nv_bfloat16* mo = reinterpret_cast<const __nv_bfloat16*>(a.merge_o);
-  const float sc = a.scale * LOG2E;
+  const float sc = (CAP ? a.softcap : a.scale) * LOG2E;
+  const float cap_in = CAP ? a.scale / a.softcap : 0.f;
 
   // destination of this lane's i-th 16-byte copy inside a page (swizzled by the row), and its row
   uint32_t dsto[NI];
@@ -106,7 +111,7 @@ attn_decode_warp_kernel(const UbAttnArgs a, const int gchunks, const int n_items
   auto request = [&](int it) {
     const int seq = it / per_seq;
     nx_len = a.seq_lens[seq];
-    const int bi = p0 + lane;
+    const int bi = (a.chunk > 0 ? first_key(nx_len) : max(a.kv_start, 0)) / PAGE + lane;
     nx_bt = bi < a.max_blocks_per_seq ? a.block_tables[(long long)seq * a.max_blocks_per_seq + bi] : -1;
   };
   request(item);
@@ -118,7 +123,7 @@ attn_decode_warp_kernel(const UbAttnArgs a, const int gchunks, const int n_items
     const int kvh = rem / gchunks, gc = rem - kvh * gchunks;
     const int h0 = kvh * Gtot + gc * 16;
     const int gn = min(16, Gtot - gc * 16);
-    const int kv_hi = nx_len;
+    const int kv_hi = nx_len, kv_lo = first_key(nx_len), p0 = kv_lo / PAGE;
     int bt = nx_bt;                                  // block-table entries p0 + lane (reloaded every 32 pages)
     const int P = kv_hi > kv_lo ? (kv_hi + PAGE - 1) / PAGE - p0 : 0;
     const int next_item = item + gstride;
@@ -198,6 +203,12 @@ attn_decode_warp_kernel(const UbAttnArgs a, const int gchunks, const int n_items
         ldsm_x4(kb + krow + (((ks * 2 + kcb) ^ kx) << 4), b0, b1, b2, b3);
         mma_bf16(s[0], qf[ks], b0, b1);
         mma_bf16(s[1], qf[ks], b2, b3);
+      }
+      if (CAP) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j)
+#pragma unroll
+          for (int e = 0; e < (SMALLG ? 2 : 4); ++e) s[j][e] = tanh_by_exp(s[j][e] * cap_in);
       }
       float mx_a = m_a, mx_b = m_b;
       if (t0 >= kv_lo && t0 + PAGE <= kv_hi) {
@@ -313,7 +324,7 @@ attn_decode_warp_kernel(const UbAttnArgs a, const int gchunks, const int n_items
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
-template <int D, int S, bool SMALLG>
+template <int D, int S, bool SMALLG, bool CAP>
 static int launch(const UbAttnArgs& a, cudaStream_t st, int gchunks, int n_items, int ctas) {
   constexpr int SMEM = WARPS * S * 2 * PAGE * D * 2;
   static bool attr_set[UB_MAX_DEVICES] = {};
@@ -321,14 +332,20 @@ static int launch(const UbAttnArgs& a, cudaStream_t st, int gchunks, int n_items
   cudaGetDevice(&dev);
   if (dev >= UB_MAX_DEVICES) return -1;
   if (!attr_set[dev]) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_warp_kernel<D, S, SMALLG>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_warp_kernel<D, S, SMALLG, CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM);
     if (e != cudaSuccess) return -(int)e;
     attr_set[dev] = true;
   }
-  cudaError_t e = ub::launch_pdl(attn_decode_warp_kernel<D, S, SMALLG>, dim3(ctas), dim3(WARPS * 32), (size_t)SMEM, st, a,
+  cudaError_t e = ub::launch_pdl(attn_decode_warp_kernel<D, S, SMALLG, CAP>, dim3(ctas), dim3(WARPS * 32), (size_t)SMEM, st, a,
                                  gchunks, n_items);
   if (e == cudaSuccess) e = cudaGetLastError();
   return e == cudaSuccess ? 0 : -(int)e;
+}
+
+template <int D, int S>
+static int launch(const UbAttnArgs& a, cudaStream_t st, int gchunks, int n_items, int ctas, bool smallg) {
+  if (a.softcap > 0.f) return smallg ? launch<D, S, true, true>(a, st, gchunks, n_items, ctas) : launch<D, S, false, true>(a, st, gchunks, n_items, ctas);
+  return smallg ? launch<D, S, true, false>(a, st, gchunks, n_items, ctas) : launch<D, S, false, false>(a, st, gchunks, n_items, ctas);
 }
 
 static int num_sms() {
@@ -351,7 +368,8 @@ extern "C" int ub_attn_decode_warp_supported(const UbAttnArgs* a) {
   if (a->D != 64 && a->D != 128) return 0;
   if (a->block_size != ub::dwarp::PAGE) return 0;
   if (a->Hkv <= 0 || a->Hq % a->Hkv != 0 || a->q_stride % 2 != 0 || a->o_stride % 2 != 0) return 0;
-  if (a->window > 0 || a->alibi_slopes != nullptr || a->splits != 1) return 0;
+  if (a->window > 0 || a->alibi_slopes != nullptr || a->splits != 1 || a->sinks != nullptr) return 0;
+  if (a->Dv > 0 && a->Dv != a->D) return 0;
   if ((reinterpret_cast<uintptr_t>(a->q) & 3) || (reinterpret_cast<uintptr_t>(a->out) & 3) ||
       (reinterpret_cast<uintptr_t>(a->k_cache) & 15) || (reinterpret_cast<uintptr_t>(a->v_cache) & 15))
     return 0;
@@ -371,16 +389,16 @@ extern "C" int ub_attn_decode_warp(const UbAttnArgs* a, void* stream) {
   if (a->D == 64) {
     int ctas = 3 * sms;
     if (ctas * WARPS > n_items) ctas = (n_items + WARPS - 1) / WARPS;
-    return smallg ? launch<64, 4, true>(*a, st, gchunks, n_items, ctas) : launch<64, 4, false>(*a, st, gchunks, n_items, ctas);
+    return launch<64, 4>(*a, st, gchunks, n_items, ctas, smallg);
   }
   // Many items: two CTAs per SM with three stages per warp.  Fewer items than half of those warps: one CTA per SM
   // with six stages per warp, i.e. five pages in flight for each of the few streams.
   if (n_items * 2 > 2 * sms * WARPS) {
     int ctas = 2 * sms;
     if (ctas * WARPS > n_items) ctas = (n_items + WARPS - 1) / WARPS;
-    return smallg ? launch<128, 3, true>(*a, st, gchunks, n_items, ctas) : launch<128, 3, false>(*a, st, gchunks, n_items, ctas);
+    return launch<128, 3>(*a, st, gchunks, n_items, ctas, smallg);
   }
   int ctas = sms;
   if (ctas * WARPS > n_items) ctas = (n_items + WARPS - 1) / WARPS;
-  return smallg ? launch<128, 6, true>(*a, st, gchunks, n_items, ctas) : launch<128, 6, false>(*a, st, gchunks, n_items, ctas);
+  return launch<128, 6>(*a, st, gchunks, n_items, ctas, smallg);
 }

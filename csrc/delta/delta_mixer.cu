@@ -413,7 +413,7 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
 
 // The same with decays per channel: one block of 16 tokens of one VALUE head, or (units H ..) of 256 value channels.
 template <typename T>
-__global__ void __launch_bounds__(PREP_T) delta_prep_channel_kernel(const UbDeltaArgs a) {
+__global__ void __launch_bounds__(PREP_T, 3) delta_prep_channel_kernel(const UbDeltaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];
@@ -430,10 +430,15 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_channel_kernel(const UbDelt
   }
   const int h = unit, group = a.H / a.G, g = h / group, ldy = dk + 4;
   float *q_s = sm, *k_s = sm + BT * ldy, *d_s = sm + 2 * BT * ldy;           // [16][dk + 4] each
-  const float rate = expf(a.a_log[h]);
-  for (int i = tid; i < BT * dk; i += PREP_T) {
-    const int t = i / dk, d = i % dk;
-    d_s[t * ldy + d] = t < n ? channel_decay(a, row + t0 + t, h, d, rate) : 1.f;
+  // the decays of four channels of a token per item; the loads are under way while the convolutions run
+  constexpr int DI = BT * 256 / 4 / PREP_T;
+  const int quads = dk / 4;
+  float4 raw[DI];
+#pragma unroll
+  for (int u = 0; u < DI; ++u) {
+    const int i = tid + u * PREP_T, t = i / quads;
+    raw[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t < n) raw[u] = *reinterpret_cast<const float4*>(a.decay + (row + t0 + t) * a.ld_decay + (long long)h * dk + (i - t * quads) * 4);
   }
   const int nch = dk / 8;
   int L = 1;
@@ -459,6 +464,19 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_channel_kernel(const UbDelt
       store8((part == 0 ? q_s : k_s) + (r + 1) * ldy + c, y[1]);
     }
     if (last && on && r == 0 && h % group == 0) keep_inputs<T>(a, row, q_len, si, so, ch, C);
+  }
+  const float rate = -expf(a.a_log[h]);
+#pragma unroll
+  for (int u = 0; u < DI; ++u) {
+    const int i = tid + u * PREP_T, t = i / quads, d = (i - t * quads) * 4;
+    if (t >= BT) continue;
+    float4 g = make_float4(1.f, 1.f, 1.f, 1.f);               // tokens past the end: no decay
+    if (t < n) {
+      const float4 b = *reinterpret_cast<const float4*>(a.dt_bias + (long long)h * dk + d);
+      g = make_float4(expf(rate * softplus(raw[u].x + b.x)), expf(rate * softplus(raw[u].y + b.y)), expf(rate * softplus(raw[u].z + b.z)),
+                      expf(rate * softplus(raw[u].w + b.w)));
+    }
+    *reinterpret_cast<float4*>(d_s + t * ldy + d) = g;
   }
   __syncthreads();
   // products of the decays from the block's start and to its end; a thread owns a channel
@@ -937,7 +955,7 @@ extern "C" int ub_delta_mixer(const UbDeltaArgs* args, void* stream) {
   if (a->H <= 0 || a->G <= 0 || a->H % a->G != 0 || a->H > 65535 || a->num_seqs > 65535) return -2;
   if (a->dk % 8 != 0 || a->dv % 8 != 0 || a->dk <= 0 || a->dv <= 0 || a->dk > 256 || a->dv > 256) return -3;
   if (a->dk_real <= 0 || a->dk_real > a->dk || a->dv_real <= 0 || a->dv_real > a->dv) return -3;
-  if (a->taps < 1 || a->taps > 16 || a->ld % 8 != 0 || a->ld_out % 8 != 0 || a->ld_gate % 8 != 0) return -4;
+  if (a->taps < 1 || a->taps > 16 || a->ld % 8 != 0 || a->ld_out % 8 != 0 || a->ld_gate % 8 != 0 || (ch && a->ld_decay % 4 != 0)) return -4;
   if (a->qkv == nullptr || a->gate == nullptr || a->b == nullptr || (a->a == nullptr && !ch) || a->conv == nullptr || a->state == nullptr ||
       a->out == nullptr || a->norm_w == nullptr || a->a_log == nullptr || a->dt_bias == nullptr)
     return -5;

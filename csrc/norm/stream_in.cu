@@ -60,23 +60,23 @@ __global__ void __launch_bounds__(THREADS) stream_in_kernel(const UbStreamInArgs
 #pragma unroll
       for (int e = 0; e < 8; ++e) x[e] = fmaf(a.scale, y[e], x[e]);
     }
-    if (dst >= 0 && a.x_res != nullptr) store8(a.x_res + dst * Hp + c, x);
-    if (a.mix != nullptr) {
-      float acc[8];
+    float acc[8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
+    if (a.mix != nullptr) {                        // all loads of a row are under way before the first store
       const float* p = a.hist + src * Hp + c;
 #pragma unroll 4
       for (int j = 0; j < a.n_hist; ++j, p += a.hist_stride) {
         float v[8];
         load8(p, v);
-        const float m = a.mix[j];
+        const float m = __ldg(a.mix + j);
 #pragma unroll
         for (int e = 0; e < 8; ++e) acc[e] = fmaf(m, v[e], acc[e]);
       }
-#pragma unroll
-      for (int e = 0; e < 8; ++e) x[e] = fmaf(m_own, x[e], acc[e]);
     }
+    if (dst >= 0 && a.x_res != nullptr) store8(a.x_res + dst * Hp + c, x);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) x[e] = fmaf(m_own, x[e], acc[e]);              // without an average 1 * x + 0
     if (dst >= 0 && a.x_out != nullptr) store8(a.x_out + dst * Hp + c, x);
 #pragma unroll
     for (int e = 0; e < 8; ++e) h[e] = fmaf(tanhf(a.alpha * x[e]), w[e], b[e]);

@@ -232,6 +232,21 @@ __global__ void __launch_bounds__(128, VTURN ? 6 : 8) head_norm_rope_kernel(cons
     cs[half + i] = s * a.gain;
   }
   const int vh = VTURN ? a.v_rot / 2 : 0;
+  // the first chunk of V that this thread turns, and its partners
+  float vx[8], vo[8];
+  auto load_v = [&](int it) {
+    const int cpr = Dv / 8, hk = it / cpr, i0 = (it - hk * cpr) * 8;
+    const T* head = row + nrot * D + hk * Dv;
+    load8(head + i0, vx);
+    if (vh % 8 == 0) {
+      if (i0 < 2 * vh) load8(head + (i0 < vh ? i0 + vh : i0 - vh), vo);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) vo[e] = i0 + e < 2 * vh ? (float)head[i0 + e < vh ? i0 + e + vh : i0 + e - vh] : 0.f;
+    }
+  };
+  const bool turn_v = VTURN && slot_ok && a.v_cache != nullptr;
+  if (turn_v && threadIdx.x < a.Hkv * (Dv / 8)) load_v(threadIdx.x);
   float* vcs = cs + 2 * half;
   for (int i = threadIdx.x; i < vh; i += 128) {
     float s, co;
@@ -268,28 +283,19 @@ __global__ void __launch_bounds__(128, VTURN ? 6 : 8) head_norm_rope_kernel(cons
     if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
   }
   __syncthreads();                                // angles and sums complete; nobody has written to the row yet
-  if (VTURN && slot_ok && a.v_cache != nullptr) {                    // turned values go to the cache only, the row stays
+  if (turn_v) {                    // turned values go to the cache only, the row stays
     const int cpr = Dv / 8;
-    const T* vr = row + nrot * D;
     T* vd = reinterpret_cast<T*>(a.v_cache) + (blk * a.Hkv * a.block_size + off) * Dv;
     for (int it = threadIdx.x; it < a.Hkv * cpr; it += 128) {
       const int hk = it / cpr, i0 = (it - hk * cpr) * 8;
-      const T* head = vr + hk * Dv;
-      float x[8], o[8];
-      load8(head + i0, x);
-      if (vh % 8 == 0) {
-        if (i0 < 2 * vh) load8(head + (i0 < vh ? i0 + vh : i0 - vh), o);
-      } else {
-#pragma unroll
-        for (int e = 0; e < 8; ++e) o[e] = i0 + e < 2 * vh ? (float)head[i0 + e < vh ? i0 + e + vh : i0 + e - vh] : 0.f;
-      }
+      if (it >= 128) load_v(it);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
         const int i = i0 + e;
-        if (i < vh) x[e] = x[e] * vcs[i] - o[e] * vcs[vh + i];
-        else if (i < 2 * vh) x[e] = x[e] * vcs[i - vh] + o[e] * vcs[i];
+        if (i < vh) vx[e] = vx[e] * vcs[i] - vo[e] * vcs[vh + i];
+        else if (i < 2 * vh) vx[e] = vx[e] * vcs[i - vh] + vo[e] * vcs[i];
       }
-      store8(vd + (long long)hk * a.block_size * Dv + i0, x);
+      store8(vd + (long long)hk * a.block_size * Dv + i0, vx);
     }
   }
   float rq = 1.f, rk = 1.f;                       // row norms: one factor for all queries, one for all keys
