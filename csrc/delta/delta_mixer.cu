@@ -413,7 +413,7 @@ __global__ void __launch_bounds__(PREP_T) delta_prep_kernel(const UbDeltaArgs a)
 
 // The same with decays per channel: one block of 16 tokens of one VALUE head, or (units H ..) of 256 value channels.
 template <typename T>
-__global__ void __launch_bounds__(PREP_T, 3) delta_prep_channel_kernel(const UbDeltaArgs a) {
+__global__ void __launch_bounds__(PREP_T, 4) delta_prep_channel_kernel(const UbDeltaArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   extern __shared__ __align__(16) float sm[];

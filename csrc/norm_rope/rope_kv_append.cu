@@ -194,7 +194,7 @@ enum { PAIR_HALVES = 0, PAIR_NEIGHBOURS = 1, PAIR_ODD = 2 /* halves that are no 
 
 // VTURN: values are cached turned by their position.
 template <typename T, int LPH, int PAIR, bool VTURN>
-__global__ void __launch_bounds__(128, VTURN ? 6 : 8) head_norm_rope_kernel(const UbRopeArgs a) {
+__global__ void __launch_bounds__(128, 8) head_norm_rope_kernel(const UbRopeArgs a) {
   pdl_launch_dependents();
   pdl_wait();
   constexpr int U = 2;
@@ -225,12 +225,6 @@ __global__ void __launch_bounds__(128, VTURN ? 6 : 8) head_norm_rope_kernel(cons
   }
   const long long blk = slot_ok ? slot / a.block_size : 0, off = slot_ok ? slot % a.block_size : 0;
   const float pos = (float)a.positions[t] * a.pos_scale;
-  for (int i = threadIdx.x; i < half; i += 128) {
-    float s, co;
-    sincosf(pos * (a.inv_freq != nullptr ? a.inv_freq[i] : rope_inv_freq(i, a)), &s, &co);
-    cs[i] = co * a.gain;
-    cs[half + i] = s * a.gain;
-  }
   const int vh = VTURN ? a.v_rot / 2 : 0;
   // the first chunk of V that this thread turns, and its partners
   float vx[8], vo[8];
@@ -248,11 +242,18 @@ __global__ void __launch_bounds__(128, VTURN ? 6 : 8) head_norm_rope_kernel(cons
   const bool turn_v = VTURN && slot_ok && a.v_cache != nullptr;
   if (turn_v && threadIdx.x < a.Hkv * (Dv / 8)) load_v(threadIdx.x);
   float* vcs = cs + 2 * half;
-  for (int i = threadIdx.x; i < vh; i += 128) {
+  for (int i = threadIdx.x; i < half + vh; i += 128) {
+    const bool v_angle = VTURN && i >= half;
+    const float f = v_angle ? a.v_inv_freq[i - half] : a.inv_freq != nullptr ? a.inv_freq[i] : rope_inv_freq(i, a);
     float s, co;
-    sincosf(pos * a.v_inv_freq[i], &s, &co);
-    vcs[i] = co;
-    vcs[vh + i] = s;
+    sincosf(pos * f, &s, &co);
+    if (v_angle) {
+      vcs[i - half] = co;
+      vcs[vh + i - half] = s;
+    } else {
+      cs[i] = co * a.gain;
+      cs[half + i] = s * a.gain;
+    }
   }
   if (slot_ok && a.v_cache != nullptr && !VTURN) {
     const int cpr = Dv / 8;
