@@ -1,4 +1,4 @@
-// K7: what stands between an attention's outputs and its output projection, per token and head, in 32 bits:
+// K3o: what stands between an attention's outputs and its output projection, per token and head, in 32 bits:
 //
 //   maps = 2:   o = a1 - lambda * a2,   o = o / sqrt(mean(o^2) + eps) * factor      (a1, a2: the outputs of heads 2 h and 2 h + 1)
 //   rotation:   pair (u, v) = (o_i, o_(i + half)) becomes (u cos + v sin, v cos - u sin), angle = position * freq_i
